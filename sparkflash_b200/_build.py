@@ -1,10 +1,13 @@
 """In-tree native build.
 
-Two shared libraries with a plain C ABI (loaded through ctypes, see ``_lib.py``):
+Four shared libraries with a plain C ABI (loaded through ctypes, see ``_lib.py``), each built on its own when it is first
+needed, so that a model compiles what it uses:
 
-* ``lib/libsfb_host.so``  - g++: codecs, CPU oracle ops, scheduler core, lane planner, radix cache,
-  constrained-decoding automaton, tool-call parser, Engram hash, rank-file converter/loader.
-* ``lib/libsfb_cuda.so``  - nvcc for sm_100a only: every device kernel and its launcher, the
+* ``lib/libsfb_core.so``  - g++: what every model needs - scheduler core, radix cache and page allocator, safetensors and
+  rank-file reader.
+* ``lib/libsfb_host.so``  - g++: codecs, CPU oracle ops, speculation policy, constrained-decoding automaton, Engram hash.
+* ``lib/libsfb_rows.so``  - nvcc for sm_100a only: kernels of the layered decoders (models/layered.py) and the sampler.
+* ``lib/libsfb_cuda.so``  - nvcc for sm_100a only: every other device kernel and its launcher, the
   symmetric-memory helpers and the lane (virtual memory) allocator.
 
 Objects are rebuilt only when the hash of the source (plus headers and flags) changes, so importing
@@ -32,6 +35,18 @@ NVCC_FLAGS = [
 ]
 if os.environ.get("SFB_KERNEL_MARKS") == "1":      # in-kernel phase marks (utils/kernel_marks.py): a measurement build
     NVCC_FLAGS.append("-DSFB_KERNEL_MARKS")
+_CORE = ("host_sched.cpp", "host_radix.cpp", "host_weights.cpp")
+
+
+def _sources(lib: str) -> list[Path]:
+    cu, cpp = sorted(CSRC.rglob("*.cu")), sorted(CSRC.rglob("*.cpp"))
+    return {"core": [s for s in cpp if s.name in _CORE],
+            "host": [s for s in cpp if s.name not in _CORE],
+            "rows": [s for s in cu if s.name.startswith("k_rows") or s.name == "k_sample.cu"],
+            "cuda": [s for s in cu if not s.name.startswith("k_rows")]}[lib]
+
+
+LIBRARIES = ("core", "host", "rows", "cuda")
 GXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-Wall", "-Wno-unused-function", "-pthread"]
 
 
@@ -72,43 +87,44 @@ def _compile_one(cmd: list[str], src: Path, obj: Path, stamp: Path, digest: str,
     return f"[built] {src.name}"
 
 
-def build(verbose: bool = False, force: bool = False) -> dict[str, Path]:
-    """Compile every native source for sm_100a / the host and link both libraries."""
+def build(verbose: bool = False, force: bool = False, only: tuple[str, ...] | None = None) -> dict[str, Path]:
+    """Compile the native sources for sm_100a / the host and link the libraries (``only``: names out of LIBRARIES)."""
+    names = tuple(only or LIBRARIES)
     LIBDIR.mkdir(exist_ok=True)
     OBJDIR.mkdir(exist_ok=True)
     hdr = _headers_digest()
-    nvcc = _nvcc()
-    cuda_srcs = sorted(CSRC.rglob("*.cu"))
-    host_srcs = sorted(CSRC.rglob("*.cpp"))
-    jobs = []
-    cuda_objs, host_objs = [], []
-    for s in cuda_srcs:
-        o = OBJDIR / (s.stem + ".cu.o")
-        cuda_objs.append(o)
-        cmd = [nvcc, *NVCC_FLAGS, "-I", str(CSRC), "-c", str(s), "-o", str(o)]
-        jobs.append((cmd, s, o, OBJDIR / (s.stem + ".cu.stamp"), _digest(s, NVCC_FLAGS, hdr)))
-    for s in host_srcs:
-        o = OBJDIR / (s.stem + ".cpp.o")
-        host_objs.append(o)
-        cmd = ["g++", *GXX_FLAGS, "-I", str(CSRC), "-c", str(s), "-o", str(o)]
-        jobs.append((cmd, s, o, OBJDIR / (s.stem + ".cpp.stamp"), _digest(s, GXX_FLAGS, hdr)))
+    jobs, objs = {}, {n: [] for n in names}
+    for n in names:
+        for s in _sources(n):
+            cuda = s.suffix == ".cu"
+            cc, flags = (_nvcc(), NVCC_FLAGS) if cuda else ("g++", GXX_FLAGS)
+            o = OBJDIR / (s.name + ".o")
+            objs[n].append(o)
+            jobs[s.name] = ([cc, *flags, "-I", str(CSRC), "-c", str(s), "-o", str(o)], s, o, OBJDIR / (s.name + ".stamp"), _digest(s, flags, hdr))
     if force:
-        for j in jobs:
+        for j in jobs.values():
             if j[3].exists():
                 j[3].unlink()
     with ThreadPoolExecutor(max_workers=max(2, (os.cpu_count() or 4))) as ex:
-        results = list(ex.map(lambda j: _compile_one(*j, verbose), jobs))
-    rebuilt = any(r.startswith("[built]") for r in results)
+        results = dict(zip(jobs, ex.map(lambda j: _compile_one(*j, verbose), jobs.values())))
     if verbose:
-        print("\n".join(results))
-    out = {"host": LIBDIR / "libsfb_host.so", "cuda": LIBDIR / "libsfb_cuda.so"}
-    if rebuilt or not out["host"].exists():
-        subprocess.run(["g++", "-shared", "-o", str(out["host"]), *map(str, host_objs), "-pthread"],
-                       check=True)
-    if rebuilt or not out["cuda"].exists():
-        subprocess.run([nvcc, "-shared", "-o", str(out["cuda"]), *map(str, cuda_objs),
-                        "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC"],
-                       check=True)
+        print("\n".join(results.values()))
+    out = {}
+    for n in names:
+        so = LIBDIR / f"libsfb_{n}.so"
+        out[n] = so
+        stamp = OBJDIR / f"lib{n}.stamp"
+        want = hashlib.sha256(" ".join(j[4] for j in (jobs[s.name] for s in _sources(n))).encode()).hexdigest()
+        if so.exists() and stamp.exists() and stamp.read_text() == want:
+            continue
+        part = LIBDIR / f".libsfb_{n}.{os.getpid()}.so"      # linked beside, then renamed: a reader never sees half a file
+        if n in ("core", "host"):
+            cmd = ["g++", "-shared", "-o", str(part), *map(str, objs[n]), "-pthread"]
+        else:
+            cmd = [_nvcc(), "-shared", "-o", str(part), *map(str, objs[n]), "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC"]
+        subprocess.run(cmd, check=True, capture_output=True)
+        os.replace(part, so)
+        stamp.write_text(want)
     return out
 
 

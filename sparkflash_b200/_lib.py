@@ -1,8 +1,7 @@
-"""ctypes access to the two native libraries.
+"""ctypes access to the native libraries (``_build.py`` lists what each holds).
 
-``host()`` returns ``libsfb_host.so`` (built on demand with g++ when missing); ``cuda()`` returns
-``libsfb_cuda.so`` and refuses to fall back: when a CUDA device is present and the library is
-missing or fails to load, the error is raised to the caller.
+Each accessor loads its library, compiling it first when it is missing.  ``cuda()`` and ``rows()`` refuse to fall back: when a
+CUDA device is present and the library is missing or fails to load, the error is raised to the caller.
 """
 from __future__ import annotations
 
@@ -11,8 +10,7 @@ import os
 from pathlib import Path
 
 _ROOT = Path(__file__).resolve().parent
-_host = None
-_cuda = None
+_loaded: dict[str, ctypes.CDLL] = {}
 
 c_void_p = ctypes.c_void_p
 c_int = ctypes.c_int
@@ -22,30 +20,32 @@ c_u8 = ctypes.c_uint8
 c_u64 = ctypes.c_uint64
 
 
-def _ensure_built() -> None:
-    h = _ROOT / "lib" / "libsfb_host.so"
-    c = _ROOT / "lib" / "libsfb_cuda.so"
-    if h.exists() and c.exists() and not os.environ.get("SFB_REBUILD"):
-        return
-    from . import _build
-    _build.build()
+def _load(name: str) -> ctypes.CDLL:
+    if name not in _loaded:
+        path = _ROOT / "lib" / f"libsfb_{name}.so"
+        if not path.exists() or os.environ.get("SFB_REBUILD"):
+            from . import _build
+            _build.build(only=(name,))
+        _loaded[name] = ctypes.CDLL(str(path))
+        if name == "host":
+            _declare_host(_loaded[name])
+    return _loaded[name]
+
+
+def core() -> ctypes.CDLL:
+    return _load("core")
 
 
 def host() -> ctypes.CDLL:
-    global _host
-    if _host is None:
-        _ensure_built()
-        _host = ctypes.CDLL(str(_ROOT / "lib" / "libsfb_host.so"))
-        _declare_host(_host)
-    return _host
+    return _load("host")
+
+
+def rows() -> ctypes.CDLL:
+    return _load("rows")
 
 
 def cuda() -> ctypes.CDLL:
-    global _cuda
-    if _cuda is None:
-        _ensure_built()
-        _cuda = ctypes.CDLL(str(_ROOT / "lib" / "libsfb_cuda.so"))
-    return _cuda
+    return _load("cuda")
 
 
 def _declare_host(L: ctypes.CDLL) -> None:

@@ -1,5 +1,5 @@
 """Command line: ``python -m sparkflash_b200 <models|doctor|trace|convert|pack-engram|serve|bench-serving|web|device-chain|
-inkling-tp4|plan|roofline|gates|served-gate>``.
+inkling-tp4|plan|roofline|gates|served-gate|generate|trace-run>``.
 Reference: crates/sparkflash-cli/src/main.rs:50-76 (subcommand table), convert.rs:76 (convert usage),
 serve.rs:6418-6590 (serve orchestration)."""
 from __future__ import annotations
@@ -207,6 +207,22 @@ def _served_gate(args) -> int:
                        (["--api-key", args.api_key] if args.api_key else []))
 
 
+def _trace_run(args) -> int:
+    from .serve import replay
+    return replay.run(args)
+
+
+def _generate(args) -> int:
+    """Continue prompts of token ids with a model folder, through the scheduler and the serving driver (no HTTP)."""
+    from .models import registry
+    from .serve.driver import generate_all
+    prompts = [[int(t) for t in p.split(",")] for p in args.tokens]
+    eng = registry.layered_engine(args.model, args.dtype, max_context=args.max_context, max_lanes=args.lanes, max_rows=args.max_rows)
+    for prompt, out in zip(prompts, generate_all(eng, prompts, args.max_new, args.temperature, args.seed)):
+        print(json.dumps({"prompt_tokens": len(prompt), "tokens": out}))
+    return 0
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(prog="sparkflash_b200")
     sub = ap.add_subparsers(dest="cmd")
@@ -226,6 +242,9 @@ def main(argv=None) -> int:
     e.add_argument("--dry-run", action="store_true"); e.set_defaults(fn=_pack_engram)
     s = sub.add_parser("serve")
     s.add_argument("--weights", help="directory of converted rank files"); s.add_argument("--synthetic", choices=["tiny", "reduced", "full"])
+    s.add_argument("--model", help="model folder (config.json + safetensors) served by the layered engine")
+    s.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"]); s.add_argument("--max-context", type=int, default=32768)
+    s.add_argument("--pool-tokens", type=int, default=0, help="cache pool of --model in tokens (0: every lane can be full)")
     s.add_argument("--tokenizer"); s.add_argument("--host", default="127.0.0.1"); s.add_argument("--port", type=int, default=8000)
     s.add_argument("--api-key", default=os.environ.get("SFB_API_KEY")); s.add_argument("--config", help="TOML settings file")
     s.add_argument("--model-id", default="deepseek-v4.1-flash"); s.add_argument("--control-port", type=int, default=29600)
@@ -252,6 +271,16 @@ def main(argv=None) -> int:
     gt = sub.add_parser("gates"); gt.add_argument("--skip-tests", action="store_true"); gt.set_defaults(fn=_gates)
     sg = sub.add_parser("served-gate"); sg.add_argument("--url", default="http://127.0.0.1:8000"); sg.add_argument("--tokens", type=int, default=48)
     sg.add_argument("--concurrency", type=int, default=4); sg.add_argument("--api-key"); sg.set_defaults(fn=_served_gate)
+    ge = sub.add_parser("generate", help="continue token ids with a model folder, through the scheduler")
+    ge.add_argument("--model", required=True); ge.add_argument("--tokens", action="append", required=True, help="comma-separated ids; repeat for several prompts")
+    ge.add_argument("--max-new", type=int, default=32); ge.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
+    ge.add_argument("--temperature", type=float, default=0.0); ge.add_argument("--seed", type=int, default=0)
+    ge.add_argument("--lanes", type=int, default=4); ge.add_argument("--max-context", type=int, default=4096); ge.add_argument("--max-rows", type=int, default=1024)
+    ge.set_defaults(fn=_generate)
+    tr = sub.add_parser("trace-run", help="replay a token trace from standard input and write logits")
+    tr.add_argument("--model", required=True); tr.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
+    tr.add_argument("--out", required=True); tr.add_argument("--max-tokens", type=int, required=True, help="most tokens live requests hold at any time")
+    tr.set_defaults(fn=_trace_run)
     args = ap.parse_args(argv)
     if not getattr(args, "fn", None):
         ap.print_help()

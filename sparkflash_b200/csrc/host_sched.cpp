@@ -11,7 +11,9 @@
 //      speculative step of at most `max_rows` verify rows (anchors first, then drafts in order of the
 //      drafter's confidence); more sequences take one plain row each.
 // Admission: `max_lanes` running + `queue_depth` waiting, beyond that the request is refused (HTTP 503).
-// When lane memory runs out the newest running sequence is preempted and later recomputed.
+// When lane memory runs out the newest running sequence is preempted and later recomputed.  With a paged cache
+// (sfb_sched_set_pages) a sequence is placed only when the pages of its whole length are free, so that nothing that runs is
+// ever short of a page; prefixes that free lanes still hold are dropped, least recently used first, to make room.
 //
 // Every rank executes the same plan from the same tick, so the planner is deterministic: no clocks, no
 // hashing of pointers, ties broken by sequence id.
@@ -57,6 +59,8 @@ struct Config {
   int64_t ring_slack = (int64_t)1 << 40;
   int decoder_tail = 0;     // > 0: prompt rows more than this far before the prompt's end run the cache-owning layers only
   int64_t lane_row_budget = -1;  // total rows all lanes may hold (-1: unlimited)
+  int page = 0;                  // rows per cache page (0: lanes are not paged)
+  int64_t pages = 0;             // pages in the pool
 };
 
 struct Scheduler {
@@ -88,6 +92,20 @@ int64_t rows_held(const Scheduler& s) {
   return n;
 }
 
+int64_t pages_of(const Scheduler& s, int64_t rows) { return (rows + s.cfg.page - 1) / s.cfg.page; }
+int64_t pages_for(const Scheduler& s, const Seq& q) { return pages_of(s, (int64_t)q.prompt_len + q.max_new); }
+
+// pages promised to running sequences plus pages that free lanes (other than `skip`) still hold
+int64_t pages_taken(const Scheduler& s, int skip, bool with_free) {
+  int64_t n = 0;
+  for (int i = 0; i < (int)s.lanes.size(); ++i) {
+    const Lane& L = s.lanes[i];
+    if (L.owner >= 0) n += pages_for(s, s.seqs.at(L.owner));
+    else if (with_free && i != skip) n += pages_of(s, (int64_t)L.held.size());
+  }
+  return n;
+}
+
 void place_waiting(Scheduler& s) {
   while (!s.waiting.empty()) {
     // any free lane?
@@ -96,6 +114,7 @@ void place_waiting(Scheduler& s) {
       if (s.lanes[i].owner < 0) free_lanes.push_back(i);
     if (free_lanes.empty()) return;
     Seq& q = s.seqs[s.waiting.front()];
+    if (s.cfg.page > 0 && pages_taken(s, -1, false) + pages_for(s, q) > s.cfg.pages) return;
     // longest reusable prefix among the free lanes (never the whole prompt: the last row must be computed)
     int best = -1, best_len = 0;
     for (int li : free_lanes) {
@@ -119,6 +138,17 @@ void place_waiting(Scheduler& s) {
     } else {
       s.prefix_hits++;
       s.prefix_rows += best_len;
+    }
+    if (s.cfg.page > 0) {
+      while (pages_taken(s, best, true) + pages_for(s, q) > s.cfg.pages) {
+        int victim = -1;
+        for (int i = 0; i < (int)s.lanes.size(); ++i)
+          if (i != best && s.lanes[i].owner < 0 && !s.lanes[i].held.empty() &&
+              (victim < 0 || s.lanes[i].last_used < s.lanes[victim].last_used))
+            victim = i;
+        if (victim < 0) break;       // cannot happen: the running sequences and q fit
+        s.lanes[victim].held.clear();
+      }
     }
     Lane& L = s.lanes[best];
     if (best_len < L.full_from) L.full_from = best_len;      // rows kept are all before the old boundary: nothing upper-layer is kept
@@ -178,12 +208,19 @@ void* sfb_sched_create(int max_lanes, int queue_depth, int max_rows, int prefill
 }
 void sfb_sched_set_ring_slack(void* h, int64_t rows) { ((Scheduler*)h)->cfg.ring_slack = rows; }
 void sfb_sched_set_decoder_tail(void* h, int rows) { ((Scheduler*)h)->cfg.decoder_tail = rows; }
+void sfb_sched_set_pages(void* h, int page, int64_t pages) { ((Scheduler*)h)->cfg.page = page; ((Scheduler*)h)->cfg.pages = pages; }
+// rows every lane holds by the scheduler's book (out: one entry per lane); an engine gives back what lies beyond
+void sfb_sched_lane_rows(void* h, int64_t* out) {
+  Scheduler& s = *(Scheduler*)h;
+  for (size_t i = 0; i < s.lanes.size(); ++i) out[i] = (int64_t)s.lanes[i].held.size();
+}
 void sfb_sched_destroy(void* h) { delete (Scheduler*)h; }
 
 // 0 = accepted, 1 = refused (lanes and queue full), 2 = prompt too long / invalid
 int sfb_sched_submit(void* h, int64_t id, const int32_t* prompt, int n, int max_new) {
   Scheduler& s = *(Scheduler*)h;
   if (n <= 0 || n + max_new > s.cfg.max_context || s.seqs.count(id)) return 2;
+  if (s.cfg.page > 0 && pages_of(s, (int64_t)n + max_new) > s.cfg.pages) return 2;
   int running = 0;
   for (auto& kv : s.seqs)
     if (kv.second.state == PREFILL || kv.second.state == DECODE) ++running;

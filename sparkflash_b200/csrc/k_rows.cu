@@ -1,0 +1,626 @@
+// Row kernels of the layered decoders (models/layered.py): everything of a layer between its matrix products except
+// attention.  A step holds n rows of any mix of lanes; the rows of one lane are a *segment* (consecutive, in position order).
+//
+//   seam       residual += norm(sublayer output), then the next sublayer's norm, in one pass over a row; options: the output is
+//              half the sum of two branches with an RMS norm each; the row starts from the embedding table; a loop pass adds
+//              the embedding output and a vector; a step of single-row segments also applies the input convolution.
+//   conv       causal depthwise convolution with carried inputs, optionally added to its input, optionally with a bias.
+//   qk_append  RMS norm over a whole query / key projection, keys and values into the paged cache.
+//   gated scan real-gated linear recurrence S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t with a = exp(-c r softplus(lam)):
+//              a chunk summary kernel and an output kernel for prompts, one fused kernel (convolution, gates, recurrence,
+//              output gate) for single rows.
+//   silu_mul   silu(gate) * up.
+//
+// Recurrent state (scan state, convolution inputs) has two versions per lane.  A segment reads version `src` (-1: zeros) and
+// writes version `dst`, so every block of a launch sees the state before the step, a replayed graph repeats the same result,
+// and a step can be undone by going back to `src`.
+#include "k_rows.cuh"
+
+namespace sfb {
+namespace rows {
+
+// ---- seam ------------------------------------------------------------------------------------------------------------
+struct SeamArgs {
+  float* x;                 // [rows, d] residual, 32-bit
+  const void* y;            // [rows, d] sublayer output (T) or null: no residual update
+  const void* y2;           // second branch (T) or null
+  const float *mw, *mw2;    // RMS weights of the two branches
+  const float *pw, *pb;     // post-norm
+  const void* embed;        // [vocab, d] (T)
+  const int* tokens;        // [rows]
+  const float* step_vec;    // [d] or null: added after the update
+  float* tap;               // [rows, d] or null: the residual right after the update
+  const float *nw, *nb;     // next norm, or null: none
+  void* h;                  // [rows, d] (T) its output
+  const int* row_map;       // null: row = block; otherwise the residual row of output row `block`
+  const float* cw;          // [taps, d] input convolution, or null
+  void* hist;               // [slots, taps - 1, d] (T)
+  const int *src, *dst;     // [rows] state versions of single-row segments
+  int from_embed, add_embed, taps, d, vocab;
+  float eps;
+  Status* status;
+};
+
+template <typename T, int V, int NV>
+__global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
+  __shared__ float sh[2 * 2 * 32];
+  int phase = 0;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int out_row = blockIdx.x, row = a.row_map ? a.row_map[out_row] : out_row;
+  const int d = a.d, step = blockDim.x * V, c0 = threadIdx.x * V;
+  const float inv_d = 1.f / (float)d;
+  float x[NV][V], e[NV][V];
+  const bool want_embed = a.from_embed || a.add_embed;
+  if (want_embed) {
+    int tok = a.tokens[row];
+    if (tok < 0 || tok >= a.vocab) { if (threadIdx.x == 0) status_set(a.status, ST_BOUNDS, 60, tok, a.vocab); tok = 0; }
+    const T* er = (const T*)a.embed + (size_t)tok * d;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (c0 + i * step < d) load_v<T, V>(er + c0 + i * step, e[i]);
+  }
+  float* xr = a.x + (size_t)row * d;
+  if (!a.from_embed) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (c0 + i * step < d) load_v<float, V>(xr + c0 + i * step, x[i]);
+  }
+  if (a.y) {
+    float y[NV][V];
+    const T* yr = (const T*)a.y + (size_t)row * d;
+    float s[2] = {0.f, 0.f};
+    if (a.y2) {
+      const T* zr = (const T*)a.y2 + (size_t)row * d;
+      float z[NV][V];
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (c0 + i * step < d) {
+          load_v<T, V>(yr + c0 + i * step, y[i]);
+          load_v<T, V>(zr + c0 + i * step, z[i]);
+#pragma unroll
+          for (int k = 0; k < V; ++k) { s[0] += y[i][k] * y[i][k]; s[1] += z[i][k] * z[i][k]; }
+        }
+      block_sums<2>(s, sh, phase);
+      const float r0 = 0.5f / sqrtf(s[0] * inv_d + a.eps), r1 = 0.5f / sqrtf(s[1] * inv_d + a.eps);
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (c0 + i * step < d) {
+          float w0[V], w1[V];
+          load_v<float, V>(a.mw + c0 + i * step, w0);
+          load_v<float, V>(a.mw2 + c0 + i * step, w1);
+#pragma unroll
+          for (int k = 0; k < V; ++k) y[i][k] = y[i][k] * r0 * w0[k] + z[i][k] * r1 * w1[k];
+        }
+    } else {
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+        if (c0 + i * step < d) load_v<T, V>(yr + c0 + i * step, y[i]);
+    }
+    float m[1] = {0.f}, q[1] = {0.f};
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (c0 + i * step < d) {
+#pragma unroll
+        for (int k = 0; k < V; ++k) m[0] += y[i][k];
+      }
+    block_sums<1>(m, sh, phase);
+    const float mu = m[0] * inv_d;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (c0 + i * step < d) {
+#pragma unroll
+        for (int k = 0; k < V; ++k) { const float t = y[i][k] - mu; q[0] += t * t; }
+      }
+    block_sums<1>(q, sh, phase);
+    const float rs = 1.f / sqrtf(q[0] * inv_d + a.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+      if (c0 + i * step < d) {
+        float w[V], b[V];
+        load_v<float, V>(a.pw + c0 + i * step, w);
+        load_v<float, V>(a.pb + c0 + i * step, b);
+#pragma unroll
+        for (int k = 0; k < V; ++k) x[i][k] += (y[i][k] - mu) * rs * w[k] + b[k];
+        if (a.tap) store_v<float, V>(a.tap + (size_t)row * d + c0 + i * step, x[i]);
+      }
+  }
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+    if (c0 + i * step < d) {
+      if (a.from_embed) {
+#pragma unroll
+        for (int k = 0; k < V; ++k) x[i][k] = e[i][k];
+      } else if (a.add_embed) {
+#pragma unroll
+        for (int k = 0; k < V; ++k) x[i][k] += e[i][k];
+      }
+      if (a.step_vec) {
+        float sv[V];
+        load_v<float, V>(a.step_vec + c0 + i * step, sv);
+#pragma unroll
+        for (int k = 0; k < V; ++k) x[i][k] += sv[k];
+      }
+      store_v<float, V>(xr + c0 + i * step, x[i]);
+    }
+  if (!a.nw) return;
+  float m[1] = {0.f}, q[1] = {0.f};
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+    if (c0 + i * step < d) {
+#pragma unroll
+      for (int k = 0; k < V; ++k) m[0] += x[i][k];
+    }
+  block_sums<1>(m, sh, phase);
+  const float mu = m[0] * inv_d;
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+    if (c0 + i * step < d) {
+#pragma unroll
+      for (int k = 0; k < V; ++k) { const float t = x[i][k] - mu; q[0] += t * t; }
+    }
+  block_sums<1>(q, sh, phase);
+  const float rs = 1.f / sqrtf(q[0] * inv_d + a.eps);
+  T* hr = (T*)a.h + (size_t)out_row * d;
+  const int W = a.taps - 1;
+  const int src = a.cw ? a.src[row] : -1;
+  T* hd = a.cw ? (T*)a.hist + (size_t)a.dst[row] * W * d : nullptr;
+  const T* hs = src >= 0 ? (const T*)a.hist + (size_t)src * W * d : nullptr;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = c0 + i * step;
+    if (c >= d) continue;
+    float w[V], b[V], o[V];
+    load_v<float, V>(a.nw + c, w);
+    load_v<float, V>(a.nb + c, b);
+#pragma unroll
+    for (int k = 0; k < V; ++k) o[k] = (x[i][k] - mu) * rs * w[k] + b[k];
+    if (a.cw) {
+      // the convolution sees the norm's output at activation precision, as the many-row kernel does
+      float acc[V], t[V];
+#pragma unroll
+      for (int k = 0; k < V; ++k) o[k] = to_f<T>(from_f<T>(o[k]));
+      load_v<float, V>(a.cw + (size_t)W * d + c, t);
+#pragma unroll
+      for (int k = 0; k < V; ++k) acc[k] = t[k] * o[k];
+      for (int j = 0; j < W; ++j) {
+        float g[V];
+        if (hs) load_v<T, V>(hs + (size_t)j * d + c, g);
+        else {
+#pragma unroll
+          for (int k = 0; k < V; ++k) g[k] = 0.f;
+        }
+        load_v<float, V>(a.cw + (size_t)j * d + c, t);
+#pragma unroll
+        for (int k = 0; k < V; ++k) acc[k] += t[k] * g[k];
+        if (j > 0) store_v<T, V>(hd + (size_t)(j - 1) * d + c, g);
+      }
+      if (W > 0) store_v<T, V>(hd + (size_t)(W - 1) * d + c, o);
+#pragma unroll
+      for (int k = 0; k < V; ++k) o[k] += acc[k];
+    }
+    store_v<T, V>(hr + c, o);
+  }
+}
+
+// ---- causal depthwise convolution over segments -------------------------------------------------------------------------
+struct ConvRowsArgs {
+  const void* x;            // [n, x_stride] (T)
+  int64_t x_stride;
+  const float* w;           // [taps, C], last = current row
+  const float* bias;        // [C] or null
+  void* y;                  // [n, C] (T)
+  void* hist;               // [slots, taps - 1, C] (T), oldest first
+  const int *row_seg, *seg_row0, *seg_len, *seg_src, *seg_dst;
+  int n, C, residual;       // residual: y = x + conv(x)
+};
+constexpr int CONV_RT = 8;  // rows per block: their loads are all in flight before the first product
+
+template <typename T, int V, int TAPS>
+__global__ void __launch_bounds__(128) conv_rows_kernel(ConvRowsArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (c >= a.C) return;
+  constexpr int W = TAPS - 1;
+  const int r0 = blockIdx.y * CONV_RT, r1 = min(r0 + CONV_RT, a.n);
+  const T* X = (const T*)a.x;
+  float in[CONV_RT][V], w[TAPS][V], win[W > 0 ? W : 1][V], bias[V];
+#pragma unroll
+  for (int i = 0; i < CONV_RT; ++i)
+    if (r0 + i < r1) load_v<T, V>(X + (size_t)(r0 + i) * a.x_stride + c, in[i]);
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) load_v<float, V>(a.w + (size_t)j * a.C + c, w[j]);
+#pragma unroll
+  for (int k = 0; k < V; ++k) bias[k] = 0.f;
+  if (a.bias) load_v<float, V>(a.bias + c, bias);
+  int seg = a.row_seg[r0], s0 = a.seg_row0[seg], s1 = s0 + a.seg_len[seg];
+  {
+    const int src = a.seg_src[seg];
+#pragma unroll
+    for (int j = 0; j < W; ++j) {         // win[j] = the input of row r0 - W + j
+      const int r = r0 - W + j;
+      if (r >= s0) load_v<T, V>(X + (size_t)r * a.x_stride + c, win[j]);
+      else if (src >= 0) load_v<T, V>((const T*)a.hist + ((size_t)src * W + (W - (s0 - r))) * a.C + c, win[j]);
+      else {
+#pragma unroll
+        for (int k = 0; k < V; ++k) win[j][k] = 0.f;
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < CONV_RT; ++i) {
+    const int r = r0 + i;
+    if (r >= r1) break;
+    if (r == s1) {                        // next segment: its window comes from its own state
+      seg = a.row_seg[r]; s0 = r; s1 = s0 + a.seg_len[seg];
+      const int src = a.seg_src[seg];
+#pragma unroll
+      for (int j = 0; j < W; ++j) {
+        if (src >= 0) load_v<T, V>((const T*)a.hist + ((size_t)src * W + j) * a.C + c, win[j]);
+        else {
+#pragma unroll
+          for (int k = 0; k < V; ++k) win[j][k] = 0.f;
+        }
+      }
+    }
+    float o[V];
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      float acc = bias[k] + w[W][k] * in[i][k];
+#pragma unroll
+      for (int j = 0; j < W; ++j) acc += w[j][k] * win[j][k];
+      o[k] = a.residual ? in[i][k] + acc : acc;
+    }
+    store_v<T, V>((T*)a.y + (size_t)r * a.C + c, o);
+#pragma unroll
+    for (int j = 0; j < W; ++j) {
+#pragma unroll
+      for (int k = 0; k < V; ++k) win[j][k] = j + 1 < W ? win[j + 1 < W ? j + 1 : j][k] : in[i][k];
+    }
+    if (r == s1 - 1) {
+      const int dst = a.seg_dst[seg];
+#pragma unroll
+      for (int j = 0; j < W; ++j) store_v<T, V>((T*)a.hist + ((size_t)dst * W + j) * a.C + c, win[j]);
+    }
+  }
+}
+
+// ---- query / key norm over the whole projection, cache append -------------------------------------------------------------
+struct QkAppendArgs {
+  const void* proj;         // [n, stride] (T): q at 0, k at HD, v at HD + GD
+  int64_t stride;
+  const float *qw, *kw;     // [HD], [GD]
+  void* q;                  // [n, HD] (T)
+  void *kpool, *vpool;      // [pages, G, 64, dim] / [pages, G, 64, vdim] (T)
+  const int* table;         // [lanes, max_pages]
+  const int *row_lane, *row_pos;
+  int max_pages, n_pages, H, G, dim, vdim;
+  float eps;
+  Status* status;
+};
+constexpr int PAGE = 64;
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256) qk_append_kernel(QkAppendArgs a) {
+  __shared__ float sh[2 * 2 * 32];
+  int phase = 0;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x;
+  const int HD = a.H * a.dim, GD = a.G * a.dim, GV = a.G * a.vdim;
+  const T* p = (const T*)a.proj + (size_t)row * a.stride;
+  float s[2] = {0.f, 0.f};
+  for (int c = threadIdx.x * V; c < HD + GD; c += blockDim.x * V) {
+    float f[V];
+    load_v<T, V>(p + c, f);
+    float t = 0.f;
+#pragma unroll
+    for (int k = 0; k < V; ++k) t += f[k] * f[k];
+    if (c < HD) s[0] += t; else s[1] += t;
+  }
+  block_sums<2>(s, sh, phase);
+  const float rq = 1.f / sqrtf(s[0] / (float)HD + a.eps), rk = 1.f / sqrtf(s[1] / (float)GD + a.eps);
+  const int pos = a.row_pos[row];
+  const int page = a.table[(size_t)a.row_lane[row] * a.max_pages + pos / PAGE], slot = pos % PAGE;
+  const bool ok = page >= 0 && page < a.n_pages;
+  if (!ok && threadIdx.x == 0) status_set(a.status, ST_BOUNDS, 61, page, a.n_pages);
+  for (int c = threadIdx.x * V; c < HD + GD + GV; c += blockDim.x * V) {
+    float f[V], w[V];
+    load_v<T, V>(p + c, f);
+    if (c < HD) {
+      load_v<float, V>(a.qw + c, w);
+#pragma unroll
+      for (int k = 0; k < V; ++k) f[k] = f[k] * rq * w[k];
+      store_v<T, V>((T*)a.q + (size_t)row * HD + c, f);
+    } else if (c < HD + GD) {
+      const int cc = c - HD, g = cc / a.dim, x = cc - g * a.dim;
+      load_v<float, V>(a.kw + cc, w);
+#pragma unroll
+      for (int k = 0; k < V; ++k) f[k] = f[k] * rk * w[k];
+      if (ok) store_v<T, V>((T*)a.kpool + (((size_t)page * a.G + g) * PAGE + slot) * a.dim + x, f);
+    } else {
+      const int cc = c - HD - GD, g = cc / a.vdim, x = cc - g * a.vdim;
+      if (ok) store_v<T, V>((T*)a.vpool + (((size_t)page * a.G + g) * PAGE + slot) * a.vdim + x, f);
+    }
+  }
+}
+
+// ---- real-gated linear recurrence -------------------------------------------------------------------------------------------
+struct ScanArgs {
+  const float* gates;       // [blocks, n, 2 bs]: pre-activations of r, then of i
+  const float *rb, *ib;     // [width] gate biases
+  const float* decay;       // [width] c * softplus(lam)
+  const void* u;            // [n, width] (T)
+  const void* y;            // [n, y_stride] (T) output branch before its gelu
+  int64_t y_stride;
+  void* out;                // [n, width] (T)
+  float* S;                 // [slots, width]
+  float2* sums;             // [chunks, width] (product of a, end value from a zero start)
+  const int *chunk_seg, *chunk_row0, *chunk_rows, *chunk_first;   // chunk_first: first chunk of the same segment
+  const int *seg_src, *seg_dst, *seg_row0, *seg_len;
+  int n, width, bs;
+};
+
+// decay a and input b of one step from the gate pre-activations; sqrt(1 - a^2) through expm1, which keeps its digits near a = 1
+__device__ __forceinline__ void gate_step(float zr, float zi, float decay, float u, float& a, float& b) {
+  const float la = -decay * sigmoid_f(zr);
+  a = expf(la);
+  b = sqrtf(-expm1f(2.f * la)) * (sigmoid_f(zi) * u);
+}
+
+template <typename T, bool OUT>
+__global__ void __launch_bounds__(128) scan_kernel(ScanArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= a.width) return;
+  const int ch = blockIdx.y, seg = a.chunk_seg[ch], row0 = a.chunk_row0[ch], rows = a.chunk_rows[ch], first = a.chunk_first[ch];
+  const bool last = row0 + rows == a.seg_row0[seg] + a.seg_len[seg];
+  if (!OUT && last) return;                 // nobody reads the last chunk's summary
+  float S = 0.f, P = 1.f;
+  if (OUT) {
+    const int src = a.seg_src[seg];
+    if (src >= 0) S = a.S[(size_t)src * a.width + c];
+    for (int k = first; k < ch; ++k) {
+      const float2 t = a.sums[(size_t)k * a.width + c];
+      S = fmaf(t.x, S, t.y);
+    }
+  }
+  const int b = c / a.bs, j = c - b * a.bs;
+  const float* g = a.gates + ((size_t)b * a.n + row0) * 2 * a.bs + j;
+  const T* U = (const T*)a.u + (size_t)row0 * a.width + c;
+  const T* Y = (const T*)a.y + (size_t)row0 * a.y_stride + c;
+  T* O = (T*)a.out + (size_t)row0 * a.width + c;
+  const float rb = a.rb[c], ib = a.ib[c], dec = a.decay[c];
+#pragma unroll 4
+  for (int t = 0; t < rows; ++t) {
+    float at, bt;
+    gate_step(g[(size_t)t * 2 * a.bs] + rb, g[(size_t)t * 2 * a.bs + a.bs] + ib, dec, to_f<T>(U[(size_t)t * a.width]), at, bt);
+    S = fmaf(at, S, bt);
+    if (OUT) O[(size_t)t * a.width] = from_f<T>(S * gelu_tanh_f(to_f<T>(Y[(size_t)t * a.y_stride])));
+    else P *= at;
+  }
+  if (!OUT) a.sums[(size_t)ch * a.width + c] = make_float2(P, S);
+  else if (last) a.S[(size_t)a.seg_dst[seg] * a.width + c] = S;
+}
+
+// Single-row segments: convolution, gates, recurrence and output gate of one part of the width in one kernel.
+// grid (parts * tiles, row groups of RB); 8 warps, a warp owns one output channel at a time.
+struct GatedRowArgs {
+  const void* x;            // [n, x_stride] (T) convolution input
+  const void* y;            // [n, y_stride] (T)
+  int64_t x_stride, y_stride;
+  const float *cw, *cb;     // [taps, width], [width]
+  void* hist;               // [slots, taps - 1, width] (T)
+  const void* wg;           // [parts, 2 bs, bs] (T): rows of r, then rows of i
+  const float *rb, *ib, *decay;
+  float* S;
+  void* out;                // [n, width] (T)
+  const int *src, *dst;     // [n]
+  int n, width, bs, taps, tiles, per_tile;
+};
+constexpr int GATED_RB = 4;
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256) gated_row_kernel(GatedRowArgs a) {
+  extern __shared__ float us[];             // [RB][bs rounded up to 8]
+  pdl_launch_dependents();
+  pdl_wait();
+  const int part = blockIdx.x / a.tiles, tile = blockIdx.x % a.tiles;
+  const int r0 = blockIdx.y * GATED_RB, nr = min(GATED_RB, a.n - r0);
+  const int W = a.taps - 1, ld = (a.bs + 7) & ~7;
+  for (int idx = threadIdx.x; idx < GATED_RB * a.bs; idx += blockDim.x) {
+    const int i = idx / a.bs, j = idx - i * a.bs, c = part * a.bs + j;
+    float acc = 0.f;
+    if (i < nr) {
+      const int row = r0 + i, src = a.src[row];
+      const T xt = ((const T*)a.x)[(size_t)row * a.x_stride + c];
+      acc = a.cb[c] + a.cw[(size_t)W * a.width + c] * to_f<T>(xt);
+      T* hd = (T*)a.hist + (size_t)a.dst[row] * W * a.width + c;
+      const T* hs = (const T*)a.hist + (size_t)(src >= 0 ? src : 0) * W * a.width + c;
+      for (int k = 0; k < W; ++k) {
+        const T g = src >= 0 ? hs[(size_t)k * a.width] : from_f<T>(0.f);
+        acc += a.cw[(size_t)k * a.width + c] * to_f<T>(g);
+        if (tile == 0 && k > 0) hd[(size_t)(k - 1) * a.width] = g;
+      }
+      if (tile == 0 && W > 0) hd[(size_t)(W - 1) * a.width] = xt;
+      acc = to_f<T>(from_f<T>(acc));        // activation precision, as the many-row convolution stores it
+    }
+    us[i * ld + j] = acc;
+  }
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int j1 = min((tile + 1) * a.per_tile, a.bs);
+  for (int j = tile * a.per_tile + warp; j < j1; j += 8) {
+    const T* wr = (const T*)a.wg + ((size_t)part * 2 * a.bs + j) * a.bs;
+    const T* wi = wr + (size_t)a.bs * a.bs;
+    float dr[GATED_RB], di[GATED_RB];
+#pragma unroll
+    for (int i = 0; i < GATED_RB; ++i) dr[i] = di[i] = 0.f;
+    for (int k = lane * V; k < a.bs; k += 32 * V) {
+      float fr[V], fi[V];
+      if constexpr (V == 8) { load8<T>(wr + k, fr); load8<T>(wi + k, fi); }
+      else { load_v<T, 1>(wr + k, fr); load_v<T, 1>(wi + k, fi); }
+#pragma unroll
+      for (int i = 0; i < GATED_RB; ++i) {
+#pragma unroll
+        for (int v = 0; v < V; ++v) { dr[i] += fr[v] * us[i * ld + k + v]; di[i] += fi[v] * us[i * ld + k + v]; }
+      }
+    }
+    float zr = 0.f, zi = 0.f;
+#pragma unroll
+    for (int i = 0; i < GATED_RB; ++i) {
+      const float a0 = warp_sum(dr[i]), b0 = warp_sum(di[i]);
+      if (lane == i) { zr = a0; zi = b0; }
+    }
+    if (lane < nr) {
+      const int row = r0 + lane, c = part * a.bs + j, src = a.src[row];
+      float at, bt;
+      gate_step(zr + a.rb[c], zi + a.ib[c], a.decay[c], us[lane * ld + j], at, bt);
+      const float S = fmaf(at, src >= 0 ? a.S[(size_t)src * a.width + c] : 0.f, bt);
+      a.S[(size_t)a.dst[row] * a.width + c] = S;
+      ((T*)a.out)[(size_t)row * a.width + c] = from_f<T>(S * gelu_tanh_f(to_f<T>(((const T*)a.y)[(size_t)row * a.y_stride + c])));
+    }
+  }
+}
+
+// ---- silu(gate) * up --------------------------------------------------------------------------------------------------------
+template <typename T, int V>
+__global__ void __launch_bounds__(256) silu_mul_kernel(const T* gu, T* out, int ff) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+  if (c >= ff) return;
+  const size_t row = blockIdx.x;
+  float g[V], u[V];
+  load_v<T, V>(gu + row * 2 * ff + c, g);
+  load_v<T, V>(gu + row * 2 * ff + ff + c, u);
+#pragma unroll
+  for (int k = 0; k < V; ++k) g[k] = g[k] * sigmoid_f(g[k]) * u[k];
+  store_v<T, V>(out + row * ff + c, g);
+}
+
+// ---- dispatch ---------------------------------------------------------------------------------------------------------------
+template <typename T, int V>
+static int launch_seam(const SeamArgs& a, int n, cudaStream_t st) {
+  const int vecs = (a.d + V - 1) / V;
+  int nv = 1;
+  while (nv < 8 && (vecs + nv - 1) / nv > 256) nv *= 2;
+  const int threads = ((vecs + nv - 1) / nv + 31) / 32 * 32;
+  if (threads > 512) return (int)cudaErrorInvalidValue;
+  switch (nv) {
+    case 1: return (int)sfb_launch(seam_kernel<T, V, 1>, dim3(n), dim3(threads), 0, st, a);
+    case 2: return (int)sfb_launch(seam_kernel<T, V, 2>, dim3(n), dim3(threads), 0, st, a);
+    case 4: return (int)sfb_launch(seam_kernel<T, V, 4>, dim3(n), dim3(threads), 0, st, a);
+    default: return (int)sfb_launch(seam_kernel<T, V, 8>, dim3(n), dim3(threads), 0, st, a);
+  }
+}
+template <typename T, int V>
+static int launch_conv(const ConvRowsArgs& a, int taps, cudaStream_t st) {
+  const dim3 g((a.C + 128 * V - 1) / (128 * V), (a.n + CONV_RT - 1) / CONV_RT), b(128);
+  switch (taps) {
+    case 1: return (int)sfb_launch(conv_rows_kernel<T, V, 1>, g, b, 0, st, a);
+    case 2: return (int)sfb_launch(conv_rows_kernel<T, V, 2>, g, b, 0, st, a);
+    case 3: return (int)sfb_launch(conv_rows_kernel<T, V, 3>, g, b, 0, st, a);
+    case 4: return (int)sfb_launch(conv_rows_kernel<T, V, 4>, g, b, 0, st, a);
+    case 5: return (int)sfb_launch(conv_rows_kernel<T, V, 5>, g, b, 0, st, a);
+    case 6: return (int)sfb_launch(conv_rows_kernel<T, V, 6>, g, b, 0, st, a);
+    case 7: return (int)sfb_launch(conv_rows_kernel<T, V, 7>, g, b, 0, st, a);
+    case 8: return (int)sfb_launch(conv_rows_kernel<T, V, 8>, g, b, 0, st, a);
+    default: return (int)cudaErrorInvalidValue;
+  }
+}
+
+}  // namespace rows
+}  // namespace sfb
+
+using namespace sfb;
+using namespace sfb::rows;
+
+extern "C" {
+
+// fp32: 1 = float activations, 0 = bf16.  See SeamArgs for the rest; null pointers switch the parts off.
+int sfb_rows_seam(void* x, const void* y, const void* y2, const void* mw, const void* mw2, const void* pw, const void* pb, const void* embed,
+                  const int* tokens, const void* step_vec, void* tap, const void* nw, const void* nb, void* h, const int* row_map,
+                  const void* cw, void* hist, const int* src, const int* dst, int from_embed, int add_embed, int taps, int n, int d,
+                  int vocab, float eps, int fp32, void* status, cudaStream_t stream) {
+  if (n < 1 || d < 1) return (int)cudaErrorInvalidValue;
+  SeamArgs a{(float*)x, y, y2, (const float*)mw, (const float*)mw2, (const float*)pw, (const float*)pb, embed, tokens, (const float*)step_vec,
+             (float*)tap, (const float*)nw, (const float*)nb, h, row_map, (const float*)cw, hist, src, dst, from_embed, add_embed, taps, d,
+             vocab, eps, (Status*)status};
+  if (fp32) return d % 4 ? launch_seam<float, 1>(a, n, stream) : launch_seam<float, 4>(a, n, stream);
+  return d % 4 ? launch_seam<__nv_bfloat16, 1>(a, n, stream) : launch_seam<__nv_bfloat16, 4>(a, n, stream);
+}
+
+int sfb_rows_conv(const void* x, int64_t x_stride, const void* w, const void* bias, void* y, void* hist, const int* row_seg, const int* seg_row0,
+                  const int* seg_len, const int* seg_src, const int* seg_dst, int n, int C, int taps, int residual, int fp32,
+                  cudaStream_t stream) {
+  if (n < 1 || C < 1) return (int)cudaErrorInvalidValue;
+  ConvRowsArgs a{x, x_stride, (const float*)w, (const float*)bias, y, hist, row_seg, seg_row0, seg_len, seg_src, seg_dst, n, C, residual};
+  const bool v4 = C % 4 == 0 && x_stride % 4 == 0 && ((uintptr_t)x % (fp32 ? 16 : 8)) == 0;
+  if (fp32) return v4 ? launch_conv<float, 4>(a, taps, stream) : launch_conv<float, 1>(a, taps, stream);
+  return v4 ? launch_conv<__nv_bfloat16, 4>(a, taps, stream) : launch_conv<__nv_bfloat16, 1>(a, taps, stream);
+}
+
+int sfb_rows_qk_append(const void* proj, int64_t stride, const void* qw, const void* kw, void* q, void* kpool, void* vpool, const int* table,
+                       const int* row_lane, const int* row_pos, int max_pages, int n_pages, int n, int H, int G, int dim, int vdim, float eps,
+                       int fp32, void* status, cudaStream_t stream) {
+  if (n < 1) return (int)cudaErrorInvalidValue;
+  QkAppendArgs a{proj, stride, (const float*)qw, (const float*)kw, q, kpool, vpool, table, row_lane, row_pos, max_pages, n_pages, H, G, dim, vdim,
+                 eps, (Status*)status};
+  const bool v4 = dim % 4 == 0 && vdim % 4 == 0 && stride % 4 == 0;
+  if (fp32) return (int)(v4 ? sfb_launch(qk_append_kernel<float, 4>, dim3(n), dim3(256), 0, stream, a)
+                            : sfb_launch(qk_append_kernel<float, 1>, dim3(n), dim3(256), 0, stream, a));
+  return (int)(v4 ? sfb_launch(qk_append_kernel<__nv_bfloat16, 4>, dim3(n), dim3(256), 0, stream, a)
+                  : sfb_launch(qk_append_kernel<__nv_bfloat16, 1>, dim3(n), dim3(256), 0, stream, a));
+}
+
+// summaries: run the chunk-summary pass first (needed when a segment has more than one chunk)
+int sfb_rows_scan(const void* gates, const void* rb, const void* ib, const void* decay, const void* u, const void* y, int64_t y_stride, void* out,
+                  void* S, void* sums, const int* chunk_seg, const int* chunk_row0, const int* chunk_rows, const int* chunk_first,
+                  const int* seg_src, const int* seg_dst, const int* seg_row0, const int* seg_len, int chunks, int summaries, int n, int width,
+                  int bs, int fp32, cudaStream_t stream) {
+  if (n < 1 || chunks < 1 || chunks > 65535) return (int)cudaErrorInvalidValue;
+  ScanArgs a{(const float*)gates, (const float*)rb, (const float*)ib, (const float*)decay, u, y, y_stride, out, (float*)S, (float2*)sums,
+             chunk_seg, chunk_row0, chunk_rows, chunk_first, seg_src, seg_dst, seg_row0, seg_len, n, width, bs};
+  const dim3 g((width + 127) / 128, chunks), b(128);
+  cudaError_t rc = cudaSuccess;
+  if (summaries) {
+    rc = fp32 ? sfb_launch(scan_kernel<float, false>, g, b, 0, stream, a) : sfb_launch(scan_kernel<__nv_bfloat16, false>, g, b, 0, stream, a);
+    if (rc != cudaSuccess) return (int)rc;
+  }
+  rc = fp32 ? sfb_launch(scan_kernel<float, true>, g, b, 0, stream, a) : sfb_launch(scan_kernel<__nv_bfloat16, true>, g, b, 0, stream, a);
+  return (int)rc;
+}
+
+int sfb_rows_gated_step(const void* x, int64_t x_stride, const void* y, int64_t y_stride, const void* cw, const void* cb, void* hist,
+                        const void* wg, const void* rb, const void* ib, const void* decay, void* S, void* out, const int* src, const int* dst,
+                        int n, int width, int bs, int taps, int fp32, cudaStream_t stream) {
+  if (n < 1 || bs < 1 || width % bs || taps < 1) return (int)cudaErrorInvalidValue;
+  const int parts = width / bs, groups = (n + GATED_RB - 1) / GATED_RB;
+  // enough blocks to fill the machine without repeating the convolution more than needed
+  int tiles = 1;
+  while (tiles < 16 && parts * groups * tiles < 296 && bs / (tiles * 2) >= 8) tiles *= 2;
+  GatedRowArgs a{x, y, x_stride, y_stride, (const float*)cw, (const float*)cb, hist, wg, (const float*)rb, (const float*)ib, (const float*)decay,
+                 (float*)S, out, src, dst, n, width, bs, taps, tiles, (bs + tiles - 1) / tiles};
+  const size_t smem = (size_t)GATED_RB * ((bs + 7) & ~7) * sizeof(float);
+  if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
+  const dim3 g(parts * tiles, groups), b(256);
+  const bool v8 = bs % 8 == 0;
+  if (fp32) return (int)(v8 ? sfb_launch(gated_row_kernel<float, 8>, g, b, smem, stream, a) : sfb_launch(gated_row_kernel<float, 1>, g, b, smem, stream, a));
+  return (int)(v8 ? sfb_launch(gated_row_kernel<__nv_bfloat16, 8>, g, b, smem, stream, a)
+                  : sfb_launch(gated_row_kernel<__nv_bfloat16, 1>, g, b, smem, stream, a));
+}
+
+int sfb_rows_silu_mul(const void* gu, void* out, int n, int ff, int fp32, cudaStream_t stream) {
+  if (n < 1 || ff < 1) return (int)cudaErrorInvalidValue;
+  const int V = ff % 4 ? 1 : 4;
+  const dim3 g(n, (ff + 256 * V - 1) / (256 * V)), b(256);
+  if (fp32) return (int)(V == 4 ? sfb_launch(silu_mul_kernel<float, 4>, g, b, 0, stream, (const float*)gu, (float*)out, ff)
+                                : sfb_launch(silu_mul_kernel<float, 1>, g, b, 0, stream, (const float*)gu, (float*)out, ff));
+  return (int)(V == 4 ? sfb_launch(silu_mul_kernel<__nv_bfloat16, 4>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff)
+                      : sfb_launch(silu_mul_kernel<__nv_bfloat16, 1>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff));
+}
+
+}  // extern "C"

@@ -1,0 +1,78 @@
+// Element access shared by the kernels of the layered decoders (k_rows.cu, k_rows_attn.cu, k_rows_attn_tc.cu): the activation
+// type T is bf16 (serving) or float (every step in true 32-bit); arithmetic is always 32-bit.
+#pragma once
+#include "k_common.cuh"
+
+namespace sfb {
+namespace rows {
+
+template <typename T> __device__ __forceinline__ float to_f(T v);
+template <> __device__ __forceinline__ float to_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T> __device__ __forceinline__ T from_f(float v);
+template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+// V consecutive elements (V = 1 or 4; the address of a group of four is a multiple of its size)
+template <typename T, int V> __device__ __forceinline__ void load_v(const T* p, float* f) {
+  if constexpr (V == 1) {
+    f[0] = to_f<T>(*p);
+  } else if constexpr (sizeof(T) == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+  } else {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
+    f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xffff0000u);
+  }
+}
+template <typename T, int V> __device__ __forceinline__ void store_v(T* p, const float* f) {
+  if constexpr (V == 1) {
+    *p = from_f<T>(f[0]);
+  } else if constexpr (sizeof(T) == 4) {
+    *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  } else {
+    __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
+  }
+}
+// eight consecutive elements, 16-byte aligned groups for bf16, two of them for float
+template <typename T> __device__ __forceinline__ void load8(const T* p, float* f) {
+  if constexpr (sizeof(T) == 4) {
+    load_v<T, 4>(p, f); load_v<T, 4>(p + 4, f + 4);
+  } else {
+    const uint4 v = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { f[2 * i] = __uint_as_float(w[i] << 16); f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u); }
+  }
+}
+
+// Block sum of N values at once; one barrier per call: successive calls alternate between the two halves of `sh`
+// ([2][N * 32] floats), and every thread has read a half before it arrives at the next call's barrier.
+template <int N> __device__ __forceinline__ void block_sums(float (&v)[N], float* sh, int& phase) {
+  const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  float* s = sh + (phase & 1) * (2 * 32);
+  phase ^= 1;
+#pragma unroll
+  for (int k = 0; k < N; ++k) v[k] = warp_sum(v[k]);
+  if (lane == 0) {
+#pragma unroll
+    for (int k = 0; k < N; ++k) s[k * 32 + w] = v[k];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int k = 0; k < N; ++k) {
+    float t = 0.f;
+    for (int i = 0; i < nw; ++i) t += s[k * 32 + i];
+    v[k] = t;
+  }
+}
+
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
+}  // namespace rows
+}  // namespace sfb

@@ -3,6 +3,9 @@
 architecture descriptors."""
 from __future__ import annotations
 
+import importlib
+import json
+import os
 from dataclasses import dataclass
 
 
@@ -23,5 +26,32 @@ MODELS = {m.name: m for m in [
     ModelEntry("qwen3.8-flash-next", "qwen", "oracle", "gated delta-net / KDA linear attention + gated softmax attention + MoE; device rows step on the state kernels", "sparkflash_b200.models.qwen"),
     ModelEntry("inkling-2-small", "inkling", "oracle", "short conv, soft-capped windowed attention and SwiGLU, MoE with expert / intermediate / row splits; device rows step", "sparkflash_b200.models.inkling"),
     ModelEntry("dory-1.0-4b", "dory", "oracle", "latent-recurrence model, loops split over a ring pipeline of ranks", "sparkflash_b200.models.dory"),
+    ModelEntry("fanodra", "fanodra", "device", "gated linear recurrence, alone or beside attention with a distance bias; looped layers, input convolution; layered engine (bf16 or 32-bit)", "sparkflash_b200.models.fanodra"),
     ModelEntry("dflash-block-drafter", "drafter", "oracle", "one-forward block drafter over a ring of captured target features", "sparkflash_b200.models.dflash"),
 ]}
+
+# config.json "architecture" -> (module, class) of the models that run on the layered engine (models/layered.py)
+LAYERED = {"Fanodra": ("sparkflash_b200.models.fanodra", "Fanodra")}
+
+
+def architecture(path: str) -> str:
+    """What a model folder's config.json says it is."""
+    with open(os.path.join(path, "config.json")) as f:
+        d = json.load(f)
+    return d.get("architecture") or d.get("model_type") or (d.get("architectures") or ["unknown"])[0]
+
+
+def layered_class(arch: str):
+    if arch not in LAYERED:
+        raise ValueError(f"architecture {arch!r} does not run on the layered engine; known: {sorted(LAYERED)}")
+    module, cls = LAYERED[arch]
+    return getattr(importlib.import_module(module), cls)
+
+
+def layered_engine(path: str, dtype: str = "bfloat16", device: str = "cuda", max_context: int = 4096, **engine):
+    """The layered engine over the model folder ``path`` (config.json + safetensors)."""
+    import torch
+
+    from .layered import LayeredEngine
+    model = layered_class(architecture(path)).from_dir(path, {"bfloat16": torch.bfloat16, "float32": torch.float32}[dtype], device, max_context)
+    return LayeredEngine(model, max_context=max_context, **engine)

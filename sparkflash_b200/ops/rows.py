@@ -1,0 +1,124 @@
+"""Python faces of the row kernels of the layered decoders (csrc/k_rows*.cu, libsfb_rows.so).
+
+Tensors are on the current CUDA device; activations are bf16 or float32 (the dtype of the first activation tensor chooses the
+kernel), everything that is 32-bit by contract is float32.  Launches go to the current stream and raise on an error code.
+"""
+from __future__ import annotations
+
+from ctypes import c_float, c_int, c_int64, c_void_p
+
+import torch
+
+from .. import _lib
+from .native import _check, _p, _stream
+
+MAX_TAPS = 8
+
+
+def _fp32(t: torch.Tensor) -> c_int:
+    return c_int(1 if t.dtype == torch.float32 else 0)
+
+
+def seam(x, n, *, h=None, y=None, y2=None, merge_w=(None, None), post=(None, None), embed=None, tokens=None, from_embed=False, add_embed=False,
+         step_vec=None, tap=None, norm=(None, None), row_map=None, conv=None, eps=1e-6, status=None):
+    """x += LN(y; post) (y and y2: half the sum of their RMS norms), + embedding, + step_vec; h = LN(x; norm).
+    ``conv``: (weight [taps, d], history, src, dst) applies h + conv(h) on a step of single-row segments."""
+    act = h if h is not None else (y if y is not None else embed)
+    cw, hist, src, dst = conv if conv is not None else (None, None, None, None)
+    _check(_lib.rows().sfb_rows_seam(_p(x), _p(y), _p(y2), _p(merge_w[0]), _p(merge_w[1]), _p(post[0]), _p(post[1]), _p(embed), _p(tokens),
+                                     _p(step_vec), _p(tap), _p(norm[0]), _p(norm[1]), _p(h), _p(row_map), _p(cw), _p(hist), _p(src), _p(dst),
+                                     c_int(from_embed), c_int(add_embed), c_int(cw.shape[0] if cw is not None else 0), c_int(n), c_int(x.shape[1]),
+                                     c_int(embed.shape[0] if embed is not None else 0), c_float(eps), _fp32(act), _p(status), _stream()), "rows_seam")
+
+
+def conv(x, w, bias, y, hist, seg, n, residual):
+    """y = [x +] causal depthwise convolution of x [n, C] over the step's segments."""
+    _check(_lib.rows().sfb_rows_conv(_p(x), c_int64(x.stride(0)), _p(w), _p(bias), _p(y), _p(hist), _p(seg.row_seg), _p(seg.seg_row0), _p(seg.seg_len),
+                                     _p(seg.seg_src), _p(seg.seg_dst), c_int(n), c_int(w.shape[1]), c_int(w.shape[0]), c_int(residual), _fp32(y),
+                                     _stream()), "rows_conv")
+
+
+def qk_append(proj, qw, kw, q, kpool, vpool, table, row_lane, row_pos, n, heads, eps, status):
+    G, dim, vdim = kpool.shape[1], kpool.shape[3], vpool.shape[3]
+    _check(_lib.rows().sfb_rows_qk_append(_p(proj), c_int64(proj.stride(0)), _p(qw), _p(kw), _p(q), _p(kpool), _p(vpool), _p(table), _p(row_lane),
+                                          _p(row_pos), c_int(table.shape[1]), c_int(kpool.shape[0]), c_int(n), c_int(heads), c_int(G), c_int(dim),
+                                          c_int(vdim), c_float(eps), _fp32(q), _p(status), _stream()), "rows_qk_append")
+
+
+def attn(q, kpool, vpool, table, row_lane, row_pos, rows, n_rows, bias, out, part, ml, heads, scale, splits, status):
+    """Exact arm: one block per (row, group of heads, range of pages).  ``rows``: indices of the rows to run, or None for all."""
+    _check(_lib.rows().sfb_rows_attn(_p(q), _p(kpool), _p(vpool), _p(table), _p(row_lane), _p(row_pos), _p(rows), _p(bias),
+                                     c_int64(bias.shape[1] if bias is not None else 0), _p(out), _p(part), _p(ml), c_int(table.shape[1]),
+                                     c_int(kpool.shape[0]), c_int(n_rows), c_int(heads), c_int(kpool.shape[1]), c_int(kpool.shape[3]),
+                                     c_int(vpool.shape[3]), c_int(splits), c_float(scale), _fp32(q), _p(status), _stream()), "rows_attn")
+
+
+def scan(gates, rb, ib, decay, u, y, out, S, sums, seg, n, bs):
+    """Gated recurrence over the step's chunks; ``gates`` [parts, n, 2 bs] pre-activations, y [n, width] view."""
+    _check(_lib.rows().sfb_rows_scan(_p(gates), _p(rb), _p(ib), _p(decay), _p(u), _p(y), c_int64(y.stride(0)), _p(out), _p(S), _p(sums),
+                                     _p(seg.chunk_seg), _p(seg.chunk_row0), _p(seg.chunk_rows), _p(seg.chunk_first), _p(seg.seg_src), _p(seg.seg_dst),
+                                     _p(seg.seg_row0), _p(seg.seg_len), c_int(seg.chunks), c_int(seg.summaries), c_int(n), c_int(S.shape[1]), c_int(bs),
+                                     _fp32(out), _stream()), "rows_scan")
+
+
+def gated_step(x, y, cw, cb, hist, wg, rb, ib, decay, S, out, src, dst, n):
+    """Convolution, gates, recurrence and output gate of single-row segments in one kernel."""
+    _check(_lib.rows().sfb_rows_gated_step(_p(x), c_int64(x.stride(0)), _p(y), c_int64(y.stride(0)), _p(cw), _p(cb), _p(hist), _p(wg), _p(rb), _p(ib),
+                                           _p(decay), _p(S), _p(out), _p(src), _p(dst), c_int(n), c_int(S.shape[1]), c_int(wg.shape[2]),
+                                           c_int(cw.shape[0]), _fp32(out), _stream()), "rows_gated_step")
+
+
+def silu_mul(gate_up, out, n):
+    _check(_lib.rows().sfb_rows_silu_mul(_p(gate_up), _p(out), c_int(n), c_int(out.shape[1]), _fp32(out), _stream()), "rows_silu_mul")
+
+
+def sample(logits, row_pos, temperature, seed, mask, best_val, best_id, n):
+    _check(_lib.rows().sfb_sample(_p(logits), c_int64(logits.stride(0)), _p(row_pos), _p(temperature), _p(seed), _p(mask),
+                                  c_int64(mask.stride(0) if mask is not None else 0), _p(best_val), _p(best_id), c_int(n), c_int(logits.shape[1]),
+                                  c_int(0), _stream()), "sample")
+
+
+def linear(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor | None, out: torch.Tensor) -> torch.Tensor:
+    """out = x w^T (+ b): a library product with 32-bit accumulation."""
+    if b is not None:
+        return torch.addmm(b, x, w.t(), out=out)
+    return torch.mm(x, w.t(), out=out)
+
+
+class exact_matmul:
+    """Library products inside keep 32-bit accumulation throughout: no TF32, no 16-bit partial sums in split reductions."""
+
+    def __enter__(self):
+        m = torch.backends.cuda.matmul
+        self.saved = (m.allow_tf32, m.allow_bf16_reduced_precision_reduction)
+        m.allow_tf32, m.allow_bf16_reduced_precision_reduction = False, False
+
+    def __exit__(self, *exc):
+        m = torch.backends.cuda.matmul
+        m.allow_tf32, m.allow_bf16_reduced_precision_reduction = self.saved
+
+
+def block_gates(u: torch.Tensor, wg: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """Block-diagonal product with a 32-bit result: out [parts, n, 2 bs] = u's part k [n, bs] times wg[k] [2 bs, bs] transposed."""
+    parts, _, bs = wg.shape
+    x = u.view(u.shape[0], parts, bs).transpose(0, 1)
+    if u.dtype == torch.float32:
+        return torch.bmm(x, wg.transpose(1, 2), out=out)
+    return torch.bmm(x, wg.transpose(1, 2), out_dtype=torch.float32, out=out)
+
+
+def attn_blocks(heads: int, kv_heads: int) -> int:
+    """Blocks the exact arm launches per row and range."""
+    rep = heads // kv_heads
+    r = 1 if rep <= 1 else 2 if rep <= 2 else 4 if rep <= 4 else 8
+    return kv_heads * -(-rep // r)
+
+
+def attn_tc_supports(dtype: torch.dtype, dim: int, vdim: int) -> bool:
+    """Shapes the tensor-core arm takes (csrc/k_rows_attn_tc.cu)."""
+    return False
+
+
+def attn_pools(kv, index: int, tc: bool):
+    """(k pool, v pool, tensor maps of both for the tensor-core arm or None) of one attention layer run."""
+    return kv.k[index], kv.v[index], None

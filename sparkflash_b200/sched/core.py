@@ -13,13 +13,15 @@ _declared = False
 
 def _L():
     global _declared
-    L = _lib.host()
+    L = _lib.core()
     if not _declared:
         L.sfb_sched_create.restype = c_void_p
         L.sfb_sched_create.argtypes = [c_int] * 8 + [c_int64]
         L.sfb_sched_destroy.argtypes = [c_void_p]
         L.sfb_sched_set_ring_slack.argtypes = [c_void_p, c_int64]
         L.sfb_sched_set_decoder_tail.argtypes = [c_void_p, c_int]
+        L.sfb_sched_set_pages.argtypes = [c_void_p, c_int, c_int64]
+        L.sfb_sched_lane_rows.argtypes = [c_void_p, c_void_p]
         L.sfb_sched_submit.argtypes = [c_void_p, c_int64, c_void_p, c_int, c_int]
         L.sfb_sched_cancel.argtypes = [c_void_p, c_int64]
         L.sfb_sched_set_drafts.argtypes = [c_void_p, c_int64, c_void_p, c_void_p, c_int]
@@ -67,7 +69,7 @@ STATE_NAMES = ["waiting", "prefill", "decode", "finished", "preempted"]
 class Scheduler:
     def __init__(self, max_lanes=32, queue_depth=64, max_rows=64, prefill_chunk=4096, prefill_chunk_busy=2048,
                  prefix_reuse_min=256, max_context=1048576, spec_depth=5, lane_row_budget=-1):
-        self.max_rows = max_rows
+        self.max_rows, self.max_lanes = max_rows, max_lanes
         self._h = c_void_p(_L().sfb_sched_create(max_lanes, queue_depth, max_rows, prefill_chunk, prefill_chunk_busy,
                                                  prefix_reuse_min, max_context, spec_depth, lane_row_budget))
         self._buf = (c_int64 * (5 * max(max_rows, prefill_chunk)))()
@@ -85,6 +87,16 @@ class Scheduler:
     def set_decoder_tail(self, rows: int) -> None:
         """Prompt rows more than ``rows`` before the prompt's end are planned as kind-3 chunks (cache-owning layers only)."""
         _L().sfb_sched_set_decoder_tail(self._h, rows)
+
+    def set_pages(self, page: int, pages: int) -> None:
+        """The lanes share a pool of ``pages`` cache pages of ``page`` rows: sequences are placed only when their whole length fits."""
+        _L().sfb_sched_set_pages(self._h, page, pages)
+
+    def lane_rows(self) -> list[int]:
+        """Rows every lane holds (running sequences and prefixes kept for reuse)."""
+        out = (c_int64 * self.max_lanes)()
+        _L().sfb_sched_lane_rows(self._h, out)
+        return list(out)
 
     def submit(self, seq_id: int, prompt: list[int], max_new: int) -> int:
         return _L().sfb_sched_submit(self._h, seq_id, _i32(prompt), len(prompt), max_new)

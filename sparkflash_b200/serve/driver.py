@@ -131,6 +131,9 @@ class DeviceDriver(InferenceEngine):
         ring_slack = getattr(engine, "ring_slack", None)
         if ring_slack is not None:
             self.sched.set_ring_slack(ring_slack)
+        self._paged = hasattr(engine, "trim_lanes")      # the engine's lanes share a page pool and follow the scheduler's book
+        if self._paged:
+            self.sched.set_pages(engine.page, engine.n_pages)
         self.capabilities = Capabilities(constrained=getattr(engine, "supports_mask", False), speculative=drafter is not None,
                                          vision=getattr(engine, "supports_vision", False))
         self._inbox: queue.Queue = queue.Queue()
@@ -378,6 +381,10 @@ class DeviceDriver(InferenceEngine):
         elif phase == PHASE_PREFILL and getattr(eng, "supports_headless", False) and not any(
                 self._prefill_completes(self._live[r.seq], rows) for r in rows):
             kw["head"] = False           # no row of this chunk is sampled: skip the vocabulary projection
+        elif phase == PHASE_PREFILL and getattr(eng, "supports_head_last", False):
+            kw["head"] = "last"          # a prefill chunk is one sequence: its last row is the one that is sampled
+        if self._paged:
+            eng.trim_lanes(self.sched.lane_rows())
         out = eng.step([r.token for r in rows], [r.lane for r in rows], [r.pos for r in rows], temps, seeds, **kw)
         out = [int(x) for x in out]
         eng.check_status()
@@ -485,6 +492,38 @@ class DeviceDriver(InferenceEngine):
         if live.req.forced_tokens:
             stats["model_choices"] = list(live.choices[:live.generated])
         self._emit(live, ("finished", reason, stats))
+
+
+class _IdTokenizer:
+    """Stands in where requests carry token ids only."""
+    eos_id = -1
+
+    def token_bytes(self):
+        return []
+
+
+def generate_all(engine, prompts: list[list[int]], max_new: int, temperature: float = 0.0, seed: int = 0, eos_id: int = -1,
+                 drafter=None, **driver_kw) -> list[list[int]]:
+    """Continue several prompts of token ids through the scheduler and the serving loop; returns their tokens in order."""
+    tok = _IdTokenizer()
+    tok.eos_id = eos_id
+    drv = DeviceDriver(engine, tok, queue_depth=len(prompts), drafter=drafter, **driver_kw).start()
+
+    async def one(i, p):
+        out = []
+        async for ev in drv.generate(EngineRequest(f"g{i}", drv.model_id, list(p), max_tokens=max_new, temperature=temperature, seed=seed)):
+            if ev[0] == "token":
+                out.append(ev[1])
+            elif ev[0] == "error":
+                raise RuntimeError(ev[1])
+        return out
+
+    async def everything():
+        return await asyncio.gather(*(one(i, p) for i, p in enumerate(prompts)))
+    try:
+        return asyncio.run(everything())
+    finally:
+        drv.shutdown(1.0)
 
 
 class FakeRowsEngine:

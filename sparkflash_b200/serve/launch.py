@@ -24,6 +24,14 @@ def build_engine(args, settings, rank: int, world: int):
     from ..models.deepseek_v41 import engine as E, prepare as P
     from ..parallel import comm as PC
     torch.cuda.set_device(int(os.environ.get("LOCAL_RANK", rank)))
+    if getattr(args, "model", None):      # a model folder: the layered engine, one GPU
+        if world != 1:
+            raise SystemExit("--model serves on one GPU")
+        from ..models import registry
+        ec = settings.engine
+        ctx = min(ec.max_context, args.max_context)
+        return registry.layered_engine(args.model, args.dtype, max_context=ctx, max_lanes=ec.max_lanes, max_rows=max(ec.max_rows, ec.max_lanes),
+                                       pool_tokens=args.pool_tokens or None, use_graphs=ec.cuda_graphs)
     if args.weights:
         from ..weights.convert import rank_path
         from ..weights.files import load_rank_file
@@ -90,12 +98,13 @@ def run(args) -> int:
         from .driver import DSparkDrafter
         drafter = None
         if settings.engine.speculation:      # the model's own draft stages when the weights carry them, prompt look-up otherwise
-            drafter = DSparkDrafter(settings.engine.spec_depth) if eng.drafter else NgramDrafter(settings.engine.spec_depth)
+            drafter = DSparkDrafter(settings.engine.spec_depth) if getattr(eng, "drafter", False) else NgramDrafter(settings.engine.spec_depth)
         driver = DeviceDriver(eng, tok, model_id=args.model_id, channel=chan, drafter=drafter, queue_depth=settings.engine.queue_depth,
                               prefix_reuse_min=settings.engine.prefix_reuse_min_rows, stall_seconds=settings.engine.stall_secs,
                               decoder_skip=settings.engine.decoder_skip).start()
         engine = driver
-        _boot("engine ready", rank=rank, weights_gb=round(eng.w.nbytes() / 1e9, 2), kv_gb=round(eng.kv.nbytes() / 1e9, 2))
+        weights = eng.w if hasattr(eng, "w") else eng.model
+        _boot("engine ready", rank=rank, weights_gb=round(weights.nbytes() / 1e9, 2), kv_gb=round(eng.kv.nbytes() / 1e9, 2))
         if rank != 0:
             # followers have no HTTP surface: they serve ticks until the channel closes
             while driver.failed is None and chan.alive()[0]:

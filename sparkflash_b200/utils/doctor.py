@@ -20,7 +20,7 @@ def run_checks(nvml=None, need_gpus: int = 1, weights_dir: str | None = None, wo
     out: list[Check] = []
     from .. import _build
     libdir = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "lib")
-    for lib in ("libsfb_cuda.so", "libsfb_host.so"):
+    for lib in ("libsfb_cuda.so", "libsfb_rows.so", "libsfb_host.so", "libsfb_core.so"):
         p = os.path.join(libdir, lib)
         out.append(Check(f"native library {lib}", os.path.exists(p), p if os.path.exists(p) else "missing: run python -m sparkflash_b200._build"))
     out.append(Check("nvcc", shutil.which("nvcc") is not None or os.path.exists("/usr/local/cuda/bin/nvcc"), "needed only to rebuild the kernels", fatal=False))

@@ -101,7 +101,7 @@ def gather(run=_run, paths: list[str] | None = None) -> NodeFacts:
         except OSError as e:
             f.errors.append(f"{p}: {e}")
     lib = Path(__file__).resolve().parent.parent / "lib"
-    f.libraries = {n: (lib / n).is_file() for n in ("libsfb_cuda.so", "libsfb_host.so")}
+    f.libraries = {n: (lib / n).is_file() for n in ("libsfb_cuda.so", "libsfb_rows.so", "libsfb_host.so", "libsfb_core.so")}
     return f
 
 

@@ -28,7 +28,7 @@ _declared = False
 
 def _L():
     global _declared
-    L = _lib.host()
+    L = _lib.core()
     if not _declared:
         L.sfb_weights_last_error.restype = c_char_p
         L.sfb_digest64.restype = c_uint64; L.sfb_digest64.argtypes = [c_void_p, c_uint64]
