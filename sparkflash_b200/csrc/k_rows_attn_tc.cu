@@ -1,0 +1,420 @@
+// Softmax attention over the paged cache for long runs of rows, on tcgen05: score = (q . k) * scale - bias[head][distance],
+// causal, bf16 queries / keys / values, 32-bit scores, softmax and accumulators.
+//
+// One CTA: 256 consecutive query rows of one segment (two halves of 128) x one head.  Key tiles of 128 positions (two cache
+// pages) stream through shared memory by TMA: a (page, head) block is contiguous, so a tile of 64 dims is two box copies.
+//
+//   warps 0-3, 4-7   softmax of half 0 / half 1: one thread per query row (no exchange between threads)
+//   warp 8           issues the MMAs:   S_w = Q_w K^T  (shared x shared),   O_w += P_w V  (P from tensor memory, V MN-major)
+//   warp 9           TMA: the queries once, key and value tiles in two stages each
+//   warps 10-11      stage the tile's window of the bias row (383 distances, four copies shifted by one element each, so that a
+//                    thread reads its row's values, which step down by one per key, as aligned 16-byte words without bank
+//                    conflicts)
+//
+// The halves alternate: while one half's scores are exponentiated the tensor core works for the other.  Tensor memory: S0, S1
+// (128 columns each), O0, O1.  P replaces S in place: the softmax weights stay 32-bit up to the product, which takes them as two
+// bf16 terms (hi in columns 0..63, lo = the remainder in 64..127), so P V sees about 16 mantissa bits.  The output accumulator is
+// rescaled only when a row's maximum grew by more than 2^8.
+//
+// No cluster, no multicast; every wait is bounded and reports through the status word.
+#include <cuda.h>
+
+#include "k_rows.cuh"
+
+namespace sfb {
+namespace rtc {
+
+constexpr int THREADS = 384, ROWS = 256, HALF = 128, KT = 128, PAGE = 64, SLAB = KT * 128;
+constexpr int BW = 392;                       // bias copy stride: 383 values, = 8 mod 32 banks
+constexpr uint32_t SPIN_LIMIT = 1u << 22;
+constexpr float LOG2E = 1.4426950408889634f;
+
+__device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void mbar_init(uint64_t* b, uint32_t count) {
+  asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(b)), "r"(count));
+}
+__device__ __forceinline__ void mbar_arrive(uint64_t* b) { asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(b)) : "memory"); }
+__device__ __forceinline__ void mbar_expect(uint64_t* b, uint32_t bytes) {
+  asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_u32(b)), "r"(bytes) : "memory");
+}
+__device__ __forceinline__ bool mbar_try(uint64_t* b, uint32_t parity) {
+  uint32_t ok;
+  asm volatile("{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\tselp.u32 %0, 1, 0, p;\n\t}"
+               : "=r"(ok) : "r"(smem_u32(b)), "r"(parity) : "memory");
+  return ok != 0;
+}
+// false: the limit ran out, or another role has given up
+__device__ __forceinline__ bool mbar_wait(uint64_t* b, uint32_t parity, volatile int* dead) {
+  for (uint32_t i = 0; i < SPIN_LIMIT; ++i) {
+    if (mbar_try(b, parity)) return true;
+    if (i > 4096) {
+      if (*dead) return false;
+      __nanosleep(64);
+    }
+  }
+  *dead = 1;
+  return false;
+}
+__device__ __forceinline__ void tma2d(void* dst, const CUtensorMap* map, int x, int y, uint64_t* bar) {
+  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];"
+               ::"r"(smem_u32(dst)), "l"(map), "r"(x), "r"(y), "r"(smem_u32(bar)) : "memory");
+}
+__device__ __forceinline__ void fence_before() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
+__device__ __forceinline__ void fence_after() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
+__device__ __forceinline__ void commit(uint64_t* b) {
+  asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(b)) : "memory");
+}
+__device__ __forceinline__ void mma_ss(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t acc) {
+  asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+               ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(acc) : "memory");
+}
+// A from tensor memory: lane = row, one 32-bit column per two consecutive k
+__device__ __forceinline__ void mma_ts(uint32_t d, uint32_t a, uint64_t b, uint32_t idesc, uint32_t acc) {
+  asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+               ::"r"(d), "r"(a), "l"(b), "r"(idesc), "r"(acc) : "memory");
+}
+__device__ __forceinline__ void ld32(uint32_t t, float* f) {
+  uint32_t* v = reinterpret_cast<uint32_t*>(f);
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,"
+      "%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"
+      : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]), "=r"(v[9]),
+        "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15]), "=r"(v[16]), "=r"(v[17]), "=r"(v[18]), "=r"(v[19]),
+        "=r"(v[20]), "=r"(v[21]), "=r"(v[22]), "=r"(v[23]), "=r"(v[24]), "=r"(v[25]), "=r"(v[26]), "=r"(v[27]), "=r"(v[28]), "=r"(v[29]),
+        "=r"(v[30]), "=r"(v[31])
+      : "r"(t) : "memory");
+}
+__device__ __forceinline__ void ld16(uint32_t t, float* f) {
+  uint32_t* v = reinterpret_cast<uint32_t*>(f);
+  asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+               : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]), "=r"(v[8]), "=r"(v[9]),
+                 "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
+               : "r"(t) : "memory");
+}
+__device__ __forceinline__ void st16(uint32_t t, const uint32_t* v) {
+  asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
+               ::"r"(t), "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]), "r"(v[9]),
+                 "r"(v[10]), "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15]) : "memory");
+}
+__device__ __forceinline__ void wait_ld() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
+__device__ __forceinline__ void wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// 128-byte swizzled tile.  K-major: 128-byte rows, 8-row groups 1024 bytes apart.  MN-major: 64 MN elements per 128-byte row, one
+// row per k, 8-k groups 1024 bytes apart, 64-element MN blocks `lbo` bytes apart.
+__device__ __forceinline__ uint64_t desc(uint32_t saddr, uint32_t lbo) {
+  return (uint64_t)((saddr >> 4) & 0x3fff) | (uint64_t)((lbo >> 4) & 0x3fff) << 16 | (uint64_t)(1024 >> 4) << 32 | (uint64_t)1 << 46 |
+         (uint64_t)2 << 61;
+}
+// kind::f16: bf16 operands, 32-bit accumulator, M = 128
+__device__ __forceinline__ uint32_t idesc(int N, int b_mn) {
+  return 1u << 4 | 1u << 7 | 1u << 10 | (uint32_t)b_mn << 16 | (uint32_t)(N >> 3) << 17 | (128u >> 4) << 24;
+}
+
+struct Args {
+  const int* tiles;          // (row0, rows) pairs
+  const int* table;
+  const int *row_lane, *row_pos;
+  const float* bias;         // [H, bias_len] or null
+  int64_t bias_len;
+  __nv_bfloat16* out;        // [n, H vdim]
+  int max_pages, n_pages, H, G, dim, vdim;
+  float scale;
+  Status* status;
+};
+
+template <int DS, int VS>    // 64-element slabs of a query / key row and of a value row
+struct Smem {
+  alignas(1024) uint8_t q[2 * DS * SLAB];
+  alignas(1024) uint8_t k[2 * DS * SLAB];
+  alignas(1024) uint8_t v[2 * VS * SLAB];
+  alignas(16) float bias[2 * 4 * BW];
+  alignas(8) uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], p_full[2], pv_done[2], b_full[2], b_empty[2];
+  uint32_t tmem;
+  int dead;
+};
+
+template <int DS, int VS>
+__global__ void __launch_bounds__(THREADS, 1)
+attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv, Args a) {
+  extern __shared__ uint8_t raw[];
+  Smem<DS, VS>& S = *reinterpret_cast<Smem<DS, VS>*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  volatile int* dead = &S.dead;
+  if (tid == 0) {
+    S.dead = 0;
+    mbar_init(&S.q_full, 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&S.k_full[i], 1); mbar_init(&S.k_empty[i], 1); mbar_init(&S.v_full[i], 1); mbar_init(&S.v_empty[i], 1);
+      mbar_init(&S.s_full[i], 1); mbar_init(&S.p_full[i], HALF); mbar_init(&S.pv_done[i], 1);
+      mbar_init(&S.b_full[i], 64); mbar_init(&S.b_empty[i], ROWS);
+    }
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (warp == 8) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], 512;" ::"r"(smem_u32(&S.tmem)) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
+  pdl_launch_dependents();
+  fence_before();
+  __syncthreads();
+  fence_after();
+  pdl_wait();
+  const uint32_t tmem = S.tmem;
+  const int h = blockIdx.x, g = h / (a.H / a.G);
+  const int row0 = a.tiles[2 * blockIdx.y], rows = a.tiles[2 * blockIdx.y + 1];
+  const int pos0 = a.row_pos[row0];
+  // key tiles of each half: up to the position of its last row that exists (a half without rows has none)
+  const int n0 = (pos0 + min(rows, HALF) - 1) / KT + 1;
+  const int n1 = rows > HALF ? (pos0 + rows - 1) / KT + 1 : 0;
+  const int nt = max(n0, n1);
+  const int* tab = a.table + (size_t)a.row_lane[row0] * a.max_pages;
+
+  if (warp == 9) {
+    if (elect_one()) {
+      const int last_page = (pos0 + rows - 1) / PAGE;
+      mbar_expect(&S.q_full, 2 * DS * SLAB);
+      for (int w = 0; w < 2; ++w)
+        for (int s = 0; s < DS; ++s) tma2d(S.q + (w * DS + s) * SLAB, &mq, h * a.dim + 64 * s, row0 + w * HALF, &S.q_full);
+      int issued = 0;
+      for (int j = 0; j < nt; ++j) {
+        const int st = j & 1, ph = (j >> 1) & 1;
+        int y[2];
+        for (int f = 0; f < 2; ++f) {
+          const int p = min(2 * j + f, last_page);        // past the last page: any finite page, its keys are masked
+          int page = tab[p];
+          if (page < 0 || page >= a.n_pages) { status_set(a.status, ST_BOUNDS, 63, page, a.n_pages); page = 0; }
+          y[f] = (page * a.G + g) * PAGE;
+        }
+        if (!mbar_wait(&S.k_empty[st], ph ^ 1, dead)) break;
+        mbar_expect(&S.k_full[st], DS * SLAB);
+        for (int s = 0; s < DS; ++s)
+          for (int f = 0; f < 2; ++f) tma2d(S.k + (st * DS + s) * SLAB + f * (SLAB / 2), &mk, 64 * s, y[f], &S.k_full[st]);
+        issued = 2 * j + 1;
+        if (!mbar_wait(&S.v_empty[st], ph ^ 1, dead)) break;
+        mbar_expect(&S.v_full[st], VS * SLAB);
+        for (int s = 0; s < VS; ++s)
+          for (int f = 0; f < 2; ++f) tma2d(S.v + (st * VS + s) * SLAB + f * (SLAB / 2), &mv, 64 * s, y[f], &S.v_full[st]);
+        issued = 2 * j + 2;
+      }
+      if (*dead) {               // nobody may have waited for the copies in flight: do so, with a limit, before the CTA ends
+        for (int c = max(0, issued - 4); c < issued; ++c) {
+          uint64_t* b = (c & 1) ? &S.v_full[(c >> 1) & 1] : &S.k_full[(c >> 1) & 1];
+          for (int i = 0; i < 100000 && !mbar_try(b, (c >> 2) & 1); ++i) __nanosleep(64);
+        }
+        for (int i = 0; i < 100000 && !mbar_try(&S.q_full, 0); ++i) __nanosleep(64);
+      }
+    }
+  } else if (warp == 8) {
+    if (elect_one()) {
+      const int ks = (a.dim + 15) / 16, nv = (a.vdim + 15) / 16 * 16;
+      const uint32_t id_s = idesc(KT, 0), id_o = idesc(nv, 1);
+      const uint32_t qb = smem_u32(S.q), kb = smem_u32(S.k), vb = smem_u32(S.v);
+      bool ok = mbar_wait(&S.q_full, 0, dead);
+      for (int j = 0; ok && j <= nt; ++j) {
+        const int st = j & 1, ph = (j >> 1) & 1, sp = (j - 1) & 1, pp = ((j - 1) >> 1) & 1;
+        if (j < nt) ok = mbar_wait(&S.k_full[st], ph, dead);
+        if (ok && j > 0) ok = mbar_wait(&S.v_full[sp], pp, dead);
+        for (int w = 0; ok && w < 2; ++w) {
+          const int nw = w ? n1 : n0;
+          const uint32_t ts = tmem + w * 128, to = tmem + 256 + w * 128;
+          if (j > 0 && j - 1 < nw) {
+            ok = mbar_wait(&S.p_full[w], (j - 1) & 1, dead);
+            if (!ok) break;
+            fence_after();
+            for (int t = 0; t < 16; ++t)       // eight k-steps of the hi term, then of the lo term
+              mma_ts(to, ts + t * 8, desc(vb + sp * VS * SLAB + (t & 7) * 2048, SLAB), id_o, (j > 1 || t > 0) ? 1u : 0u);
+            commit(&S.pv_done[w]);
+          }
+          if (j < nw) {
+            // S overwrites P: the products that read it must be done
+            if (j > 0) ok = mbar_wait(&S.pv_done[w], (j - 1) & 1, dead);
+            if (!ok) break;
+            fence_after();
+            for (int t = 0; t < ks; ++t)
+              mma_ss(ts, desc(qb + (w * DS + (t >> 2)) * SLAB + (t & 3) * 32, 16), desc(kb + (st * DS + (t >> 2)) * SLAB + (t & 3) * 32, 16), id_s,
+                     t ? 1u : 0u);
+            commit(&S.s_full[w]);
+          }
+        }
+        if (!ok) break;
+        if (j < nt) commit(&S.k_empty[st]);
+        if (j > 0) commit(&S.v_empty[sp]);
+      }
+      if (ok) mbar_wait(&S.v_empty[(nt - 1) & 1], ((nt - 1) >> 1) & 1, dead);     // no arrival may be under way when the CTA ends
+    }
+  } else if (warp >= 10) {
+    const int t = tid - 320;
+    const float* brow = a.bias ? a.bias + (size_t)h * a.bias_len : nullptr;
+    for (int j = 0; j < nt; ++j) {
+      const int st = j & 1, ph = (j >> 1) & 1;
+      if (!mbar_wait(&S.b_empty[st], ph ^ 1, dead)) break;
+      float* dst = S.bias + st * 4 * BW;
+      const int d0 = pos0 - j * KT - 127;
+      for (int i = t; i < 384; i += 64) {
+        const int d = d0 + i;
+        const float v = (brow && d >= 0 && d < a.bias_len) ? brow[d] * LOG2E : 0.f;
+#pragma unroll
+        for (int s = 0; s < 4; ++s)
+          if (i >= s) dst[s * BW + i - s] = v;
+      }
+      mbar_arrive(&S.b_full[st]);
+    }
+  } else {
+    const int w = warp >> 2, r = (warp & 3) * 32 + lane, nw = w ? n1 : n0;
+    const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
+    const uint32_t ts = tmem + w * 128 + lanes, to = tmem + 256 + w * 128 + lanes;
+    const int pos = pos0 + w * HALF + r, rr = w * HALF + r, shift = rr & 3;
+    const float sl2 = a.scale * LOG2E;
+    float m = -INFINITY, l = 0.f;
+    bool ok = true;
+    for (int j = 0; j < nt; ++j) {
+      const int st = j & 1, ph = (j >> 1) & 1;
+      ok = mbar_wait(&S.b_full[st], ph, dead);
+      if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+      if (j >= nw) { mbar_arrive(&S.b_empty[st]); continue; }
+      ok = mbar_wait(&S.s_full[w], j & 1, dead);
+      if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+      fence_after();
+      float s[KT];
+      ld32(ts, s); ld32(ts + 32, s + 32); ld32(ts + 64, s + 64); ld32(ts + 96, s + 96);
+      wait_ld();
+      const float* bp = S.bias + st * 4 * BW + shift * BW + (rr + 124 - shift);
+#pragma unroll
+      for (int q = 0; q < KT / 4; ++q) {
+        const float4 b = *reinterpret_cast<const float4*>(bp - 4 * q);
+        s[4 * q] = fmaf(s[4 * q], sl2, -b.w);
+        s[4 * q + 1] = fmaf(s[4 * q + 1], sl2, -b.z);
+        s[4 * q + 2] = fmaf(s[4 * q + 2], sl2, -b.y);
+        s[4 * q + 3] = fmaf(s[4 * q + 3], sl2, -b.x);
+      }
+      mbar_arrive(&S.b_empty[st]);
+      const int vis = pos - j * KT;                  // keys 0 .. vis of the tile are visible
+      if (j * KT + KT - 1 > pos0 + w * HALF) {
+#pragma unroll
+        for (int c = 0; c < KT; ++c) s[c] = c <= vis ? s[c] : -INFINITY;
+      }
+      float mx[4] = {s[0], s[1], s[2], s[3]};
+#pragma unroll
+      for (int c = 4; c < KT; ++c) mx[c & 3] = fmaxf(mx[c & 3], s[c]);
+      float m_new = fmaxf(m, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])));
+      if (j > 0 && m_new - m <= 8.f) m_new = m;      // key 0 is visible to every row, so m is finite from the first tile on
+      const float corr = ex2(m - m_new);
+      float ls[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int q = 0; q < 4; ++q) {
+        uint32_t hi[16], lo[16];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float p0 = ex2(s[q * 32 + 2 * i] - m_new), p1 = ex2(s[q * 32 + 2 * i + 1] - m_new);
+          ls[i & 3] += p0 + p1;
+          const __nv_bfloat162 hb = __floats2bfloat162_rn(p0, p1);
+          hi[i] = *reinterpret_cast<const uint32_t*>(&hb);
+          const __nv_bfloat162 lb = __floats2bfloat162_rn(p0 - __uint_as_float(hi[i] << 16), p1 - __uint_as_float(hi[i] & 0xffff0000u));
+          lo[i] = *reinterpret_cast<const uint32_t*>(&lb);
+        }
+        st16(ts + q * 16, hi);
+        st16(ts + 64 + q * 16, lo);
+      }
+      if (j > 0 && __any_sync(0xffffffffu, corr != 1.f)) {
+        for (int c = 0; c < VS * 64; c += 16) {
+          float o[16];
+          ld16(to + c, o);
+          wait_ld();
+#pragma unroll
+          for (int i = 0; i < 16; ++i) o[i] *= corr;
+          st16(to + c, reinterpret_cast<const uint32_t*>(o));
+        }
+      }
+      wait_st();
+      l = l * corr + (ls[0] + ls[1]) + (ls[2] + ls[3]);
+      m = m_new;
+      fence_before();
+      mbar_arrive(&S.p_full[w]);
+    }
+    if (ok && nw > 0) {
+      ok = mbar_wait(&S.pv_done[w], (nw - 1) & 1, dead);
+      if (__all_sync(0xffffffffu, ok)) {
+        fence_after();
+        const float inv = 1.f / l;
+        const bool valid = rr < rows;
+        __nv_bfloat16* o = a.out + ((size_t)(row0 + rr) * a.H + h) * a.vdim;
+        for (int c = 0; c < a.vdim; c += 16) {
+          float f[16];
+          ld16(to + c, f);
+          wait_ld();
+          uint32_t u[8];
+#pragma unroll
+          for (int i = 0; i < 8; ++i) {
+            const __nv_bfloat162 t = __floats2bfloat162_rn(f[2 * i] * inv, f[2 * i + 1] * inv);
+            u[i] = *reinterpret_cast<const uint32_t*>(&t);
+          }
+          if (valid) {             // vdim is a multiple of eight: whole 16-byte words
+            *reinterpret_cast<uint4*>(o + c) = make_uint4(u[0], u[1], u[2], u[3]);
+            if (c + 8 < a.vdim) *reinterpret_cast<uint4*>(o + c + 8) = make_uint4(u[4], u[5], u[6], u[7]);
+          }
+        }
+      }
+    }
+  }
+  fence_before();
+  __syncthreads();
+  if (tid == 0 && *dead) status_set(a.status, ST_TIMEOUT, 64, blockIdx.x, blockIdx.y);
+  if (warp == 8) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, 512;" ::"r"(tmem) : "memory");
+}
+
+typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
+                             const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+
+template <int DS, int VS>
+static int launch(const CUtensorMap* mq, const CUtensorMap* mk, const CUtensorMap* mv, const Args& a, int n_tiles, cudaStream_t st) {
+  const size_t smem = sizeof(Smem<DS, VS>) + 1024;
+  static bool done = false;
+  if (!done) {
+    const cudaError_t e = cudaFuncSetAttribute(attn_run_kernel<DS, VS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    done = true;
+  }
+  return (int)sfb_launch(attn_run_kernel<DS, VS>, dim3(a.H, n_tiles), dim3(THREADS), smem, st, *mq, *mk, *mv, a);
+}
+
+}  // namespace rtc
+}  // namespace sfb
+
+using namespace sfb;
+using namespace sfb::rtc;
+
+extern "C" {
+
+// 2-D bf16 map over [rows, cols] (row stride in bytes, a multiple of 16) with a 128-byte swizzled box of 64 columns x box_rows; columns
+// past the row's end read as zero.  0, a CUresult, or -1 without the driver entry point.
+int sfb_rows_tmap(void* out_map, const void* base, int64_t rows, int64_t cols, int64_t row_bytes, int box_rows) {
+  static EncodeFn fn = nullptr;
+  if (!fn) {
+    void* p = nullptr;
+    cudaDriverEntryPointQueryResult q;
+    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault, &q) == cudaSuccess && q == cudaDriverEntryPointSuccess) fn = (EncodeFn)p;
+  }
+  if (!fn) return -1;
+  cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)row_bytes};
+  cuuint32_t box[2] = {64u, (cuuint32_t)box_rows}, estr[2] = {1u, 1u};
+  return (int)fn((CUtensorMap*)out_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
+                 CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+}
+
+// mq: queries [rows, H dim], box 128 rows; mk, mv: pools [pages G 64, dim / vdim], box 64 rows.  dim and vdim: multiples of 8 up to 128.
+int sfb_rows_attn_tc(const void* mq, const void* mk, const void* mv, const int* table, const int* row_lane, const int* row_pos, const int* tiles,
+                     int n_tiles, const void* bias, int64_t bias_len, void* out, int max_pages, int n_pages, int H, int G, int dim, int vdim,
+                     float scale, void* status, cudaStream_t stream) {
+  if (n_tiles < 1 || n_tiles > 65535 || G < 1 || H % G || dim % 8 || vdim % 8 || dim < 8 || dim > 128 || vdim < 8 || vdim > 128)
+    return (int)cudaErrorInvalidValue;
+  Args a{tiles, table, row_lane, row_pos, (const float*)bias, bias_len, (__nv_bfloat16*)out, max_pages, n_pages, H, G, dim, vdim, scale, (Status*)status};
+  const CUtensorMap *q = (const CUtensorMap*)mq, *k = (const CUtensorMap*)mk, *v = (const CUtensorMap*)mv;
+  if (dim <= 64) return vdim <= 64 ? launch<1, 1>(q, k, v, a, n_tiles, stream) : launch<1, 2>(q, k, v, a, n_tiles, stream);
+  return vdim <= 64 ? launch<2, 1>(q, k, v, a, n_tiles, stream) : launch<2, 2>(q, k, v, a, n_tiles, stream);
+}
+
+}  // extern "C"

@@ -5,6 +5,7 @@ kernel), everything that is 32-bit by contract is float32.  Launches go to the c
 """
 from __future__ import annotations
 
+import ctypes
 from ctypes import c_float, c_int, c_int64, c_void_p
 
 import torch
@@ -116,9 +117,40 @@ def attn_blocks(heads: int, kv_heads: int) -> int:
 
 def attn_tc_supports(dtype: torch.dtype, dim: int, vdim: int) -> bool:
     """Shapes the tensor-core arm takes (csrc/k_rows_attn_tc.cu)."""
-    return False
+    return dtype == torch.bfloat16 and dim % 8 == 0 and vdim % 8 == 0 and max(dim, vdim) <= 128
+
+
+class TensorMap:
+    """A 2-D TMA map over a bf16 tensor seen as [rows, cols], boxes of 64 columns x ``box`` rows."""
+
+    def __init__(self, t: torch.Tensor, rows: int, cols: int, box: int):
+        self._raw = (ctypes.c_uint8 * 192)()
+        self.ptr = c_void_p((ctypes.addressof(self._raw) + 63) & ~63)
+        rc = _lib.rows().sfb_rows_tmap(self.ptr, c_void_p(t.data_ptr()), c_int64(rows), c_int64(cols), c_int64(cols * 2), c_int(box))
+        if rc:
+            raise RuntimeError(f"tensor map over [{rows}, {cols}]: error {rc}")
 
 
 def attn_pools(kv, index: int, tc: bool):
     """(k pool, v pool, tensor maps of both for the tensor-core arm or None) of one attention layer run."""
-    return kv.k[index], kv.v[index], None
+    k, v = kv.k[index], kv.v[index]
+    maps = None
+    if tc and k.is_cuda:
+        maps = tuple(TensorMap(t, t.shape[0] * t.shape[1] * t.shape[2], t.shape[3], 64) for t in (k, v))
+    return k, v, maps
+
+
+_query_maps: dict[tuple, TensorMap] = {}
+
+
+def attn_tc(q, kv, table, row_lane, row_pos, tiles, n_tiles, bias, out, heads, scale, status):
+    """Tensor-core arm over runs of rows: ``tiles`` are (row0, rows <= 256) pairs, each inside one segment; kv from attn_pools."""
+    k, v, (mk, mv) = kv
+    key = (q.data_ptr(), q.untyped_storage().nbytes(), q.shape[1])
+    mq = _query_maps.get(key)
+    if mq is None:        # over the whole scratch buffer, so that one map serves every step
+        mq = _query_maps[key] = TensorMap(q, q.untyped_storage().nbytes() // (2 * q.shape[1]), q.shape[1], 128)
+    _check(_lib.rows().sfb_rows_attn_tc(mq.ptr, mk.ptr, mv.ptr, _p(table), _p(row_lane), _p(row_pos), _p(tiles), c_int(n_tiles), _p(bias),
+                                        c_int64(bias.shape[1] if bias is not None else 0), _p(out), c_int(table.shape[1]), c_int(k.shape[0]),
+                                        c_int(heads), c_int(k.shape[1]), c_int(k.shape[3]), c_int(v.shape[3]), c_float(scale), _p(status), _stream()),
+           "rows_attn_tc")

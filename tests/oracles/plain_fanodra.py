@@ -145,3 +145,70 @@ def forward(w, cfg, tokens, dtype=torch.float64, taps=None):
             taps.append(x.clone())
     x = layer_norm(x, w["final.norm"], w["final.norm.b"], cfg["norm"]["eps"])
     return x @ w["embed"].T
+
+
+# ---- small random models ---------------------------------------------------------------------------------------------
+def recurrent(width, blocks, conv):
+    return {"width": width, "blocks": blocks, "conv": conv}
+
+
+def attending(heads, kv_heads, dim, vdim, scale):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale}
+
+
+def make_config(vocab, width, taps, layers, loop=None, eps=1e-5):
+    """layers: ("rglru", recurrent(...), ff or None) or ("parallel", attending(...), recurrent(...), ff or None)."""
+    out = []
+    for L in layers:
+        mixer = L[1] if L[0] == "rglru" else {"left": L[1], "right": L[2]}
+        out.append({"type": L[0], "mixer": mixer, "mlp": {"kind": "dense", "ff": L[-1]} if L[-1] else None})
+    return {"architecture": "Fanodra", "vocab": vocab, "width": width, "canon": {"taps": taps}, "norm": {"eps": eps}, "layers": out,
+            "loop": dict(zip(("start", "stop", "times"), loop)) if loop else None}
+
+
+def make_weights(cfg, seed=0):
+    """Random bf16 tensors; every norm weight, bias, tap and gate differs from 1 and 0, so that leaving one out shows."""
+    g = torch.Generator().manual_seed(seed)
+    w, d = {}, cfg["width"]
+
+    def put(name, *shape, s=None, mean=0.0):
+        w[name] = (mean + torch.randn(*shape, generator=g) * (shape[-1] ** -0.5 if s is None else s)).to(torch.bfloat16)
+
+    def norm(name):
+        put(name, d, s=0.3, mean=1.0)
+        put(name + ".b", d, s=0.3)
+
+    def rec(p, m):
+        n, b = m["width"], m["blocks"]
+        for k in ("y", "x"):
+            put(p + k, n, d); put(p + k + ".b", n, s=0.3)
+        put(p + "conv", n, m["conv"], s=0.6); put(p + "conv.b", n, s=0.3)
+        for k in ("ra", "ri"):
+            put(p + k, b, n // b, n // b); put(p + k + ".b", b, n // b, s=0.5)
+        put(p + "lam", n, s=2.0, mean=-4.0)          # decays from a few tokens to thousands
+        put(p + "o", d, n)
+    put("embed", cfg["vocab"], d, s=1.0)
+    norm("final.norm")
+    if cfg.get("loop"):
+        put("loop.step", cfg["loop"]["times"], d, s=0.5)
+    for i, L in enumerate(cfg["layers"]):
+        p = f"l{i}."
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if L["mlp"] else ()):
+            norm(p + n)
+        put(p + "canon1", d, cfg["canon"]["taps"], s=0.4)
+        if L["type"] == "rglru":
+            rec(p + "mix.", L["mixer"])
+        else:
+            m, q = L["mixer"]["left"], p + "mix.left."
+            for n, rows in (("q", m["heads"] * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", m["kv_heads"] * m["vdim"])):
+                put(q + n, rows, d); put(q + n + ".b", rows, s=0.3)
+            put(q + "q.norm", m["heads"] * m["dim"], s=0.3, mean=1.5); put(q + "k.norm", m["kv_heads"] * m["dim"], s=0.3, mean=1.5)
+            w[q + "r1"] = (0.1 + torch.rand(m["heads"], generator=g)).to(torch.bfloat16)
+            w[q + "r2"] = (0.05 + 2 * torch.rand(m["heads"], generator=g)).to(torch.bfloat16)
+            put(q + "o", d, m["heads"] * m["vdim"]); put(q + "o.b", d, s=0.3)
+            put(q + "out", d, s=0.3, mean=1.0)
+            rec(p + "mix.right.", L["mixer"]["right"])
+            put(p + "mix.right.out", d, s=0.3, mean=1.0)
+        if L["mlp"]:
+            put(p + "mlp.gate", L["mlp"]["ff"], d); put(p + "mlp.up", L["mlp"]["ff"], d); put(p + "mlp.down", d, L["mlp"]["ff"])
+    return w
