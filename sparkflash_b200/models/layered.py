@@ -80,6 +80,8 @@ class LayeredEngine:
         """``pool_tokens``: tokens all lanes together may hold (each lane rounded up to pages); by default every lane can be full."""
         self.model, self.cfg = model, model.cfg
         self.dev = torch.device(model.device)
+        if self.dev.type == "cuda" and self.dev.index is None:       # the serving thread selects it by number
+            self.dev = torch.device("cuda", torch.cuda.current_device())
         self.max_lanes, self.max_context, self.max_rows = max_lanes, max_context, max_rows
         if not 0 < max_rows <= 65535:
             raise ValueError("max_rows must be in 1..65535")

@@ -187,7 +187,7 @@ def make_weights(cfg, seed=0):
             put(p + k, b, n // b, n // b); put(p + k + ".b", b, n // b, s=0.5)
         put(p + "lam", n, s=2.0, mean=-4.0)          # decays from a few tokens to thousands
         put(p + "o", d, n)
-    put("embed", cfg["vocab"], d, s=1.0)
+    put("embed", cfg["vocab"], d, s=0.2)          # small, so that greedy decoding does not just repeat its input
     norm("final.norm")
     if cfg.get("loop"):
         put("loop.step", cfg["loop"]["times"], d, s=0.5)
