@@ -7,7 +7,7 @@
 //   conv       causal depthwise convolution with carried inputs, optionally added to its input, optionally with a bias.
 //   qk_append  RMS norm over a whole query / key projection, keys and values into the paged cache.
 //   gated scan real-gated linear recurrence S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t with a = exp(-c r softplus(lam)):
-//              a chunk summary kernel and an output kernel for prompts, one fused kernel (convolution, gates, recurrence,
+//              two passes over chunks of rows for prompts, one fused kernel (convolution, gates, recurrence,
 //              output gate) for single rows.
 //   silu_mul   silu(gate) * up.
 //
@@ -41,15 +41,65 @@ struct SeamArgs {
   Status* status;
 };
 
+// Mean and sum of squared deviations of a row held as x[NV][V] per thread (`mine` = how many of them exist, `wcnt` = the warp's
+// total): each warp takes both about its own mean, then the warps' pairs are combined - one barrier.
+template <int V, int NV>
+__device__ __forceinline__ void row_moments(const float (&x)[NV][V], int c0, int step, int d, float wcnt, float* sh, int& phase, float& mu, float& m2) {
+  const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  float* s = sh + (phase & 1) * 96;
+  phase ^= 1;
+  float t = 0.f, q = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+    if (c0 + i * step < d) {
+#pragma unroll
+      for (int k = 0; k < V; ++k) t += x[i][k];
+    }
+  t = warp_sum(t);
+  const float wm = wcnt > 0.f ? t / wcnt : 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i)
+    if (c0 + i * step < d) {
+#pragma unroll
+      for (int k = 0; k < V; ++k) { const float e = x[i][k] - wm; q += e * e; }
+    }
+  q = warp_sum(q);
+  if (lane == 0) { s[w] = t; s[32 + w] = q; s[64 + w] = wcnt; }
+  __syncthreads();
+  t = 0.f;
+  for (int i = 0; i < nw; ++i) t += s[i];
+  mu = t / (float)d;
+  m2 = 0.f;
+  for (int i = 0; i < nw; ++i) {
+    const float c = s[64 + i], e = (c > 0.f ? s[i] / c : 0.f) - mu;
+    m2 += s[32 + i] + c * e * e;
+  }
+}
+
 template <typename T, int V, int NV>
 __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
-  __shared__ float sh[2 * 2 * 32];
-  int phase = 0;
+  __shared__ float sh[2 * 96], sh2[2 * 2 * 32];
+  int phase = 0, phase2 = 0;
+  const int d = a.d, step = blockDim.x * V, c0 = threadIdx.x * V;
+  const float inv_d = 1.f / (float)d;
+  constexpr bool AHEAD = NV <= 2;      // the weights of a short row are requested before the previous kernel has finished
+  float pw[NV][V], pb[NV][V], nw[NV][V], nb[NV][V];
+  if constexpr (AHEAD) {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = c0 + i * step;
+      if (c >= d) continue;
+      if (a.y) { load_v<float, V>(a.pw + c, pw[i]); load_v<float, V>(a.pb + c, pb[i]); }
+      if (a.nw) { load_v<float, V>(a.nw + c, nw[i]); load_v<float, V>(a.nb + c, nb[i]); }
+    }
+  }
   pdl_launch_dependents();
   pdl_wait();
   const int out_row = blockIdx.x, row = a.row_map ? a.row_map[out_row] : out_row;
-  const int d = a.d, step = blockDim.x * V, c0 = threadIdx.x * V;
-  const float inv_d = 1.f / (float)d;
+  int mine = 0;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) mine += max(0, min(V, d - (c0 + i * step)));
+  const float wcnt = warp_sum((float)mine);
   float x[NV][V], e[NV][V];
   const bool want_embed = a.from_embed || a.add_embed;
   if (want_embed) {
@@ -69,8 +119,8 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
   if (a.y) {
     float y[NV][V];
     const T* yr = (const T*)a.y + (size_t)row * d;
-    float s[2] = {0.f, 0.f};
     if (a.y2) {
+      float s[2] = {0.f, 0.f};
       const T* zr = (const T*)a.y2 + (size_t)row * d;
       float z[NV][V];
 #pragma unroll
@@ -81,7 +131,7 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
 #pragma unroll
           for (int k = 0; k < V; ++k) { s[0] += y[i][k] * y[i][k]; s[1] += z[i][k] * z[i][k]; }
         }
-      block_sums<2>(s, sh, phase);
+      block_sums<2>(s, sh2, phase2);
       const float r0 = 0.5f / sqrtf(s[0] * inv_d + a.eps), r1 = 0.5f / sqrtf(s[1] * inv_d + a.eps);
 #pragma unroll
       for (int i = 0; i < NV; ++i)
@@ -97,31 +147,18 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
       for (int i = 0; i < NV; ++i)
         if (c0 + i * step < d) load_v<T, V>(yr + c0 + i * step, y[i]);
     }
-    float m[1] = {0.f}, q[1] = {0.f};
+    float mu, m2;
+    row_moments<V, NV>(y, c0, step, d, wcnt, sh, phase, mu, m2);
+    const float rs = 1.f / sqrtf(m2 * inv_d + a.eps);
 #pragma unroll
     for (int i = 0; i < NV; ++i)
       if (c0 + i * step < d) {
+        if constexpr (!AHEAD) {
+          load_v<float, V>(a.pw + c0 + i * step, pw[i]);
+          load_v<float, V>(a.pb + c0 + i * step, pb[i]);
+        }
 #pragma unroll
-        for (int k = 0; k < V; ++k) m[0] += y[i][k];
-      }
-    block_sums<1>(m, sh, phase);
-    const float mu = m[0] * inv_d;
-#pragma unroll
-    for (int i = 0; i < NV; ++i)
-      if (c0 + i * step < d) {
-#pragma unroll
-        for (int k = 0; k < V; ++k) { const float t = y[i][k] - mu; q[0] += t * t; }
-      }
-    block_sums<1>(q, sh, phase);
-    const float rs = 1.f / sqrtf(q[0] * inv_d + a.eps);
-#pragma unroll
-    for (int i = 0; i < NV; ++i)
-      if (c0 + i * step < d) {
-        float w[V], b[V];
-        load_v<float, V>(a.pw + c0 + i * step, w);
-        load_v<float, V>(a.pb + c0 + i * step, b);
-#pragma unroll
-        for (int k = 0; k < V; ++k) x[i][k] += (y[i][k] - mu) * rs * w[k] + b[k];
+        for (int k = 0; k < V; ++k) x[i][k] += (y[i][k] - mu) * rs * pw[i][k] + pb[i][k];
         if (a.tap) store_v<float, V>(a.tap + (size_t)row * d + c0 + i * step, x[i]);
       }
   }
@@ -144,23 +181,9 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
       store_v<float, V>(xr + c0 + i * step, x[i]);
     }
   if (!a.nw) return;
-  float m[1] = {0.f}, q[1] = {0.f};
-#pragma unroll
-  for (int i = 0; i < NV; ++i)
-    if (c0 + i * step < d) {
-#pragma unroll
-      for (int k = 0; k < V; ++k) m[0] += x[i][k];
-    }
-  block_sums<1>(m, sh, phase);
-  const float mu = m[0] * inv_d;
-#pragma unroll
-  for (int i = 0; i < NV; ++i)
-    if (c0 + i * step < d) {
-#pragma unroll
-      for (int k = 0; k < V; ++k) { const float t = x[i][k] - mu; q[0] += t * t; }
-    }
-  block_sums<1>(q, sh, phase);
-  const float rs = 1.f / sqrtf(q[0] * inv_d + a.eps);
+  float mu, m2;
+  row_moments<V, NV>(x, c0, step, d, wcnt, sh, phase, mu, m2);
+  const float rs = 1.f / sqrtf(m2 * inv_d + a.eps);
   T* hr = (T*)a.h + (size_t)out_row * d;
   const int W = a.taps - 1;
   const int src = a.cw ? a.src[row] : -1;
@@ -170,11 +193,10 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
   for (int i = 0; i < NV; ++i) {
     const int c = c0 + i * step;
     if (c >= d) continue;
-    float w[V], b[V], o[V];
-    load_v<float, V>(a.nw + c, w);
-    load_v<float, V>(a.nb + c, b);
+    float o[V];
+    if constexpr (!AHEAD) { load_v<float, V>(a.nw + c, nw[i]); load_v<float, V>(a.nb + c, nb[i]); }
 #pragma unroll
-    for (int k = 0; k < V; ++k) o[k] = (x[i][k] - mu) * rs * w[k] + b[k];
+    for (int k = 0; k < V; ++k) o[k] = (x[i][k] - mu) * rs * nw[i][k] + nb[i][k];
     if (a.cw) {
       // the convolution sees the norm's output at activation precision, as the many-row kernel does
       float acc[V], t[V];
@@ -183,6 +205,7 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
       load_v<float, V>(a.cw + (size_t)W * d + c, t);
 #pragma unroll
       for (int k = 0; k < V; ++k) acc[k] = t[k] * o[k];
+#pragma unroll 4
       for (int j = 0; j < W; ++j) {
         float g[V];
         if (hs) load_v<T, V>(hs + (size_t)j * d + c, g);
@@ -348,7 +371,7 @@ __global__ void __launch_bounds__(256) qk_append_kernel(QkAppendArgs a) {
 
 // ---- real-gated linear recurrence -------------------------------------------------------------------------------------------
 struct ScanArgs {
-  const float* gates;       // [blocks, n, 2 bs]: pre-activations of r, then of i
+  const float* gates;       // [blocks, n, 2 bs]: pre-activations of r, then of i; the two-pass form leaves a and b there
   const float *rb, *ib;     // [width] gate biases
   const float* decay;       // [width] c * softplus(lam)
   const void* u;            // [n, width] (T)
@@ -362,31 +385,44 @@ struct ScanArgs {
   int n, width, bs;
 };
 
-// decay a and input b of one step from the gate pre-activations; sqrt(1 - a^2) through expm1, which keeps its digits near a = 1
-__device__ __forceinline__ void gate_step(float zr, float zi, float decay, float u, float& a, float& b) {
-  const float la = -decay * sigmoid_f(zr);
+// exp, reciprocal and square root of the gates, all 32-bit: library-accurate with float activations; with bf16 activations the
+// hardware approximations (relative error below 2^-21), whose error is far below the rounding of u
+template <typename T> __device__ __forceinline__ float gate_sigmoid(float z) {
+  if constexpr (sizeof(T) == 4) return sigmoid_f(z);
+  else return __fdividef(1.f, 1.f + __expf(-z));
+}
+// 1 - exp(t) for t <= 0: a polynomial near 0, where 1 - exp would cancel (Taylor, remainder below 2^-25 of the result)
+__device__ __forceinline__ float one_minus_exp(float t, float e) {
+  float p = 1.f / 40320.f;
+  p = fmaf(p, t, 1.f / 5040.f); p = fmaf(p, t, 1.f / 720.f); p = fmaf(p, t, 1.f / 120.f); p = fmaf(p, t, 1.f / 24.f);
+  p = fmaf(p, t, 1.f / 6.f); p = fmaf(p, t, 0.5f); p = fmaf(p, t, 1.f);
+  return t > -0.5f ? -t * p : 1.f - e;
+}
+// decay a and input b of one step from the gate pre-activations
+template <typename T> __device__ __forceinline__ void gate_step(float zr, float zi, float decay, float u, float& a, float& b) {
+  const float la = -decay * gate_sigmoid<T>(zr);
   a = expf(la);
-  b = sqrtf(-expm1f(2.f * la)) * (sigmoid_f(zi) * u);
+  const float m = one_minus_exp(2.f * la, a * a);
+  b = sqrtf(m) * (gate_sigmoid<T>(zi) * u);
+}
+template <typename T> __device__ __forceinline__ float gate_gelu(float z) {
+  if constexpr (sizeof(T) == 4) return gelu_tanh_f(z);
+  else {   // 0.5 (1 + tanh(k)) = sigmoid(2 k)
+    const float k = 1.5957691216057308f * (z + 0.044715f * z * z * z);
+    return z * gate_sigmoid<T>(k);
+  }
 }
 
-template <typename T, bool OUT>
-__global__ void __launch_bounds__(128) scan_kernel(ScanArgs a) {
+// One chunk per segment: gates, recurrence and output gate in one pass.
+template <typename T>
+__global__ void __launch_bounds__(128) scan_short_kernel(ScanArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= a.width) return;
-  const int ch = blockIdx.y, seg = a.chunk_seg[ch], row0 = a.chunk_row0[ch], rows = a.chunk_rows[ch], first = a.chunk_first[ch];
-  const bool last = row0 + rows == a.seg_row0[seg] + a.seg_len[seg];
-  if (!OUT && last) return;                 // nobody reads the last chunk's summary
-  float S = 0.f, P = 1.f;
-  if (OUT) {
-    const int src = a.seg_src[seg];
-    if (src >= 0) S = a.S[(size_t)src * a.width + c];
-    for (int k = first; k < ch; ++k) {
-      const float2 t = a.sums[(size_t)k * a.width + c];
-      S = fmaf(t.x, S, t.y);
-    }
-  }
+  const int ch = blockIdx.y, seg = a.chunk_seg[ch], row0 = a.chunk_row0[ch], rows = a.chunk_rows[ch];
+  const int src = a.seg_src[seg];
+  float S = src >= 0 ? a.S[(size_t)src * a.width + c] : 0.f;
   const int b = c / a.bs, j = c - b * a.bs;
   const float* g = a.gates + ((size_t)b * a.n + row0) * 2 * a.bs + j;
   const T* U = (const T*)a.u + (size_t)row0 * a.width + c;
@@ -396,13 +432,89 @@ __global__ void __launch_bounds__(128) scan_kernel(ScanArgs a) {
 #pragma unroll 4
   for (int t = 0; t < rows; ++t) {
     float at, bt;
-    gate_step(g[(size_t)t * 2 * a.bs] + rb, g[(size_t)t * 2 * a.bs + a.bs] + ib, dec, to_f<T>(U[(size_t)t * a.width]), at, bt);
+    gate_step<T>(g[(size_t)t * 2 * a.bs] + rb, g[(size_t)t * 2 * a.bs + a.bs] + ib, dec, to_f<T>(U[(size_t)t * a.width]), at, bt);
     S = fmaf(at, S, bt);
-    if (OUT) O[(size_t)t * a.width] = from_f<T>(S * gelu_tanh_f(to_f<T>(Y[(size_t)t * a.y_stride])));
-    else P *= at;
+    O[(size_t)t * a.width] = from_f<T>(S * gate_gelu<T>(to_f<T>(Y[(size_t)t * a.y_stride])));
   }
-  if (!OUT) a.sums[(size_t)ch * a.width + c] = make_float2(P, S);
-  else if (last) a.S[(size_t)a.seg_dst[seg] * a.width + c] = S;
+  a.S[(size_t)a.seg_dst[seg] * a.width + c] = S;
+}
+
+// Longer segments, pass 1: (a, b) of every step, in place of the gate pre-activations, and every chunk's summary.
+constexpr int SCAN_T = 8;    // rows whose loads are in flight together
+template <typename T>
+__global__ void __launch_bounds__(128) scan_gates_kernel(ScanArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= a.width) return;
+  const int ch = blockIdx.y, row0 = a.chunk_row0[ch], rows = a.chunk_rows[ch];
+  const int b = c / a.bs, j = c - b * a.bs;
+  float* g = const_cast<float*>(a.gates) + ((size_t)b * a.n + row0) * 2 * a.bs + j;
+  const T* U = (const T*)a.u + (size_t)row0 * a.width + c;
+  const float rb = a.rb[c], ib = a.ib[c], dec = a.decay[c];
+  float S = 0.f, P = 1.f;
+  for (int t0 = 0; t0 < rows; t0 += SCAN_T) {
+    float zr[SCAN_T], zi[SCAN_T], u[SCAN_T];
+#pragma unroll
+    for (int i = 0; i < SCAN_T; ++i)
+      if (t0 + i < rows) {
+        const float* gp = g + (size_t)(t0 + i) * 2 * a.bs;
+        zr[i] = gp[0]; zi[i] = gp[a.bs]; u[i] = to_f<T>(U[(size_t)(t0 + i) * a.width]);
+      }
+#pragma unroll
+    for (int i = 0; i < SCAN_T; ++i)
+      if (t0 + i < rows) {
+        float at, bt;
+        gate_step<T>(zr[i] + rb, zi[i] + ib, dec, u[i], at, bt);
+        float* gp = g + (size_t)(t0 + i) * 2 * a.bs;
+        gp[0] = at; gp[a.bs] = bt;
+        S = fmaf(at, S, bt);
+        P *= at;
+      }
+  }
+  a.sums[(size_t)ch * a.width + c] = make_float2(P, S);
+}
+
+// Pass 2: the chunk's start from the summaries before it, then the recurrence and the output gate.
+template <typename T>
+__global__ void __launch_bounds__(128) scan_apply_kernel(ScanArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c >= a.width) return;
+  const int ch = blockIdx.y, seg = a.chunk_seg[ch], row0 = a.chunk_row0[ch], rows = a.chunk_rows[ch], first = a.chunk_first[ch];
+  const int src = a.seg_src[seg];
+  float S = src >= 0 ? a.S[(size_t)src * a.width + c] : 0.f;
+  const float2* sums = a.sums + c;
+  int k = first;
+  for (; k + 8 <= ch; k += 8) {
+    float2 t[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) t[i] = sums[(size_t)(k + i) * a.width];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) S = fmaf(t[i].x, S, t[i].y);
+  }
+  for (; k < ch; ++k) { const float2 t = sums[(size_t)k * a.width]; S = fmaf(t.x, S, t.y); }
+  const int b = c / a.bs, j = c - b * a.bs;
+  const float* g = a.gates + ((size_t)b * a.n + row0) * 2 * a.bs + j;
+  const T* Y = (const T*)a.y + (size_t)row0 * a.y_stride + c;
+  T* O = (T*)a.out + (size_t)row0 * a.width + c;
+  for (int t0 = 0; t0 < rows; t0 += SCAN_T) {
+    float at[SCAN_T], bt[SCAN_T], y[SCAN_T];
+#pragma unroll
+    for (int i = 0; i < SCAN_T; ++i)
+      if (t0 + i < rows) {
+        const float* gp = g + (size_t)(t0 + i) * 2 * a.bs;
+        at[i] = gp[0]; bt[i] = gp[a.bs]; y[i] = to_f<T>(Y[(size_t)(t0 + i) * a.y_stride]);
+      }
+#pragma unroll
+    for (int i = 0; i < SCAN_T; ++i)
+      if (t0 + i < rows) {
+        S = fmaf(at[i], S, bt[i]);
+        O[(size_t)(t0 + i) * a.width] = from_f<T>(S * gate_gelu<T>(y[i]));
+      }
+  }
+  if (row0 + rows == a.seg_row0[seg] + a.seg_len[seg]) a.S[(size_t)a.seg_dst[seg] * a.width + c] = S;
 }
 
 // Single-row segments: convolution, gates, recurrence and output gate of one part of the width in one kernel.
@@ -477,10 +589,10 @@ __global__ void __launch_bounds__(256) gated_row_kernel(GatedRowArgs a) {
     if (lane < nr) {
       const int row = r0 + lane, c = part * a.bs + j, src = a.src[row];
       float at, bt;
-      gate_step(zr + a.rb[c], zi + a.ib[c], a.decay[c], us[lane * ld + j], at, bt);
+      gate_step<T>(zr + a.rb[c], zi + a.ib[c], a.decay[c], us[lane * ld + j], at, bt);
       const float S = fmaf(at, src >= 0 ? a.S[(size_t)src * a.width + c] : 0.f, bt);
       a.S[(size_t)a.dst[row] * a.width + c] = S;
-      ((T*)a.out)[(size_t)row * a.width + c] = from_f<T>(S * gelu_tanh_f(to_f<T>(((const T*)a.y)[(size_t)row * a.y_stride + c])));
+      ((T*)a.out)[(size_t)row * a.width + c] = from_f<T>(S * gate_gelu<T>(to_f<T>(((const T*)a.y)[(size_t)row * a.y_stride + c])));
     }
   }
 }
@@ -576,7 +688,7 @@ int sfb_rows_qk_append(const void* proj, int64_t stride, const void* qw, const v
                   : sfb_launch(qk_append_kernel<__nv_bfloat16, 1>, dim3(n), dim3(256), 0, stream, a));
 }
 
-// summaries: run the chunk-summary pass first (needed when a segment has more than one chunk)
+// summaries: a segment has more than one chunk (two passes; the gates are overwritten); otherwise one pass
 int sfb_rows_scan(const void* gates, const void* rb, const void* ib, const void* decay, const void* u, const void* y, int64_t y_stride, void* out,
                   void* S, void* sums, const int* chunk_seg, const int* chunk_row0, const int* chunk_rows, const int* chunk_first,
                   const int* seg_src, const int* seg_dst, const int* seg_row0, const int* seg_len, int chunks, int summaries, int n, int width,
@@ -585,12 +697,11 @@ int sfb_rows_scan(const void* gates, const void* rb, const void* ib, const void*
   ScanArgs a{(const float*)gates, (const float*)rb, (const float*)ib, (const float*)decay, u, y, y_stride, out, (float*)S, (float2*)sums,
              chunk_seg, chunk_row0, chunk_rows, chunk_first, seg_src, seg_dst, seg_row0, seg_len, n, width, bs};
   const dim3 g((width + 127) / 128, chunks), b(128);
-  cudaError_t rc = cudaSuccess;
-  if (summaries) {
-    rc = fp32 ? sfb_launch(scan_kernel<float, false>, g, b, 0, stream, a) : sfb_launch(scan_kernel<__nv_bfloat16, false>, g, b, 0, stream, a);
-    if (rc != cudaSuccess) return (int)rc;
-  }
-  rc = fp32 ? sfb_launch(scan_kernel<float, true>, g, b, 0, stream, a) : sfb_launch(scan_kernel<__nv_bfloat16, true>, g, b, 0, stream, a);
+  if (!summaries)
+    return (int)(fp32 ? sfb_launch(scan_short_kernel<float>, g, b, 0, stream, a) : sfb_launch(scan_short_kernel<__nv_bfloat16>, g, b, 0, stream, a));
+  cudaError_t rc = fp32 ? sfb_launch(scan_gates_kernel<float>, g, b, 0, stream, a) : sfb_launch(scan_gates_kernel<__nv_bfloat16>, g, b, 0, stream, a);
+  if (rc != cudaSuccess) return (int)rc;
+  rc = fp32 ? sfb_launch(scan_apply_kernel<float>, g, b, 0, stream, a) : sfb_launch(scan_apply_kernel<__nv_bfloat16>, g, b, 0, stream, a);
   return (int)rc;
 }
 

@@ -1,0 +1,149 @@
+// Matrix products of one to four rows, bf16 weights streamed once: out = x W^T (+ bias), to bf16 or 32-bit, or silu(x Wg^T) * (x Wu^T)
+// with gate and up stacked.  Paced by memory: a warp (or two, four, eight of them, each on a share of K) owns two weight rows, whose first
+// 16-byte words are requested before the previous kernel has finished - weights do not depend on it; x sits in shared memory.
+#include "k_rows.cuh"
+
+namespace sfb {
+namespace rgemv {
+
+constexpr int U = 4;          // 256-element steps of K in flight per weight row
+
+struct Args {
+  const __nv_bfloat16* w;     // [M, K] ([2 M, K] with silu: gate rows, then up rows)
+  const __nv_bfloat16* x;     // [n, K]
+  const __nv_bfloat16* bias;  // [M] or null
+  void* out;                  // [n, M] bf16 (or float)
+  int M, K, n, wk, f32, silu;
+};
+
+template <int N>
+__global__ void __launch_bounds__(256) gemv_kernel(Args a) {
+  extern __shared__ __align__(16) uint8_t raw[];
+  __shared__ float part[8][2][N];
+  __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(raw);      // [N][K]
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int groups = 8 / a.wk, g = warp / a.wk, pk = warp % a.wk;
+  const int o = blockIdx.x * groups + g;
+  const int r0 = a.silu ? o : 2 * o, r1 = a.silu ? o + a.M : 2 * o + 1;
+  const bool v0 = a.silu ? o < a.M : r0 < a.M, v1 = a.silu ? o < a.M : r1 < a.M;
+  const int steps = (a.K + 255) / 256, mine = steps > pk ? (steps - pk + a.wk - 1) / a.wk : 0;
+  const uint4* w0 = reinterpret_cast<const uint4*>(a.w + (size_t)r0 * a.K);
+  const uint4* w1 = reinterpret_cast<const uint4*>(a.w + (size_t)r1 * a.K);
+  uint4 c0[U], c1[U];
+  auto fetch = [&](int s, uint4& d0, uint4& d1) {
+    const int k = (pk + s * a.wk) * 32 + lane;                    // 16-byte word of the row
+    const bool in = s < mine && k * 8 < a.K;
+    d0 = in && v0 ? ldg_nc(w0 + k) : make_uint4(0u, 0u, 0u, 0u);
+    d1 = in && v1 ? ldg_nc(w1 + k) : make_uint4(0u, 0u, 0u, 0u);
+  };
+#pragma unroll
+  for (int i = 0; i < U; ++i) fetch(i, c0[i], c1[i]);
+  pdl_launch_dependents();
+  pdl_wait();
+  const int words = a.K / 8;
+  for (int i = tid; i < N * words; i += 256) {
+    const int r = i / words;
+    reinterpret_cast<uint4*>(xs)[i] = r < a.n ? reinterpret_cast<const uint4*>(a.x)[i] : make_uint4(0u, 0u, 0u, 0u);
+  }
+  __syncthreads();
+  float acc[2][N];
+#pragma unroll
+  for (int i = 0; i < N; ++i) acc[0][i] = acc[1][i] = 0.f;
+  for (int s0 = 0; s0 < mine; s0 += U) {
+    uint4 n0[U], n1[U];
+#pragma unroll
+    for (int i = 0; i < U; ++i) fetch(s0 + U + i, n0[i], n1[i]);
+#pragma unroll
+    for (int i = 0; i < U; ++i) {
+      const int k = (pk + (s0 + i) * a.wk) * 32 + lane;
+      if (s0 + i >= mine || k * 8 >= a.K) continue;
+      const uint32_t p[4] = {c0[i].x, c0[i].y, c0[i].z, c0[i].w}, q[4] = {c1[i].x, c1[i].y, c1[i].z, c1[i].w};
+#pragma unroll
+      for (int r = 0; r < N; ++r) {
+        const uint4 xv = reinterpret_cast<const uint4*>(xs)[r * words + k];
+        const uint32_t xw[4] = {xv.x, xv.y, xv.z, xv.w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float x0 = __uint_as_float(xw[j] << 16), x1 = __uint_as_float(xw[j] & 0xffff0000u);
+          acc[0][r] = fmaf(__uint_as_float(p[j] << 16), x0, acc[0][r]);
+          acc[0][r] = fmaf(__uint_as_float(p[j] & 0xffff0000u), x1, acc[0][r]);
+          acc[1][r] = fmaf(__uint_as_float(q[j] << 16), x0, acc[1][r]);
+          acc[1][r] = fmaf(__uint_as_float(q[j] & 0xffff0000u), x1, acc[1][r]);
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < U; ++i) { c0[i] = n0[i]; c1[i] = n1[i]; }
+  }
+#pragma unroll
+  for (int r = 0; r < N; ++r) {
+    acc[0][r] = warp_sum(acc[0][r]);
+    acc[1][r] = warp_sum(acc[1][r]);
+  }
+  if (a.wk > 1) {
+    if (lane == 0) {
+#pragma unroll
+      for (int r = 0; r < N; ++r) { part[warp][0][r] = acc[0][r]; part[warp][1][r] = acc[1][r]; }
+    }
+    __syncthreads();
+    if (pk == 0) {
+      for (int k = 1; k < a.wk; ++k) {
+#pragma unroll
+        for (int r = 0; r < N; ++r) { acc[0][r] += part[warp + k][0][r]; acc[1][r] += part[warp + k][1][r]; }
+      }
+    }
+  }
+  if (pk == 0 && lane < a.n) {
+    float s0 = acc[0][0], s1 = acc[1][0];
+#pragma unroll
+    for (int r = 1; r < N; ++r)
+      if (lane == r) { s0 = acc[0][r]; s1 = acc[1][r]; }
+    const size_t at = (size_t)lane * a.M;
+    if (a.silu) {
+      if (v0) ((__nv_bfloat16*)a.out)[at + o] = __float2bfloat16_rn(s0 * rows::sigmoid_f(s0) * s1);
+    } else {
+      if (a.bias) { if (v0) s0 += __bfloat162float(a.bias[r0]); if (v1) s1 += __bfloat162float(a.bias[r1]); }
+      if (a.f32) {
+        if (v0) ((float*)a.out)[at + r0] = s0;
+        if (v1) ((float*)a.out)[at + r1] = s1;
+      } else {
+        if (v0) ((__nv_bfloat16*)a.out)[at + r0] = __float2bfloat16_rn(s0);
+        if (v1) ((__nv_bfloat16*)a.out)[at + r1] = __float2bfloat16_rn(s1);
+      }
+    }
+  }
+}
+
+template <int N>
+static int launch(const Args& a, int blocks, cudaStream_t st) {
+  const size_t smem = (size_t)N * a.K * 2;
+  static size_t granted = 40 * 1024;
+  if (smem > granted) {
+    const cudaError_t e = cudaFuncSetAttribute(gemv_kernel<N>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    granted = smem;
+  }
+  return (int)sfb_launch(gemv_kernel<N>, dim3(blocks), dim3(256), smem, st, a);
+}
+
+}  // namespace rgemv
+}  // namespace sfb
+
+using namespace sfb;
+using namespace sfb::rgemv;
+
+extern "C" {
+
+// n <= 4 rows, K a multiple of 8, n K bounded by shared memory (4 K rows of 200 KB).  silu: w holds 2 M rows, out [n, M].
+int sfb_rows_gemv(const void* w, const void* x, const void* bias, void* out, int n, int M, int K, int f32, int silu, cudaStream_t stream) {
+  const int N = n <= 1 ? 1 : n <= 2 ? 2 : 4;
+  if (n < 1 || n > 4 || M < 1 || K < 8 || K % 8 || (size_t)N * K * 2 > 200 * 1024) return (int)cudaErrorInvalidValue;
+  const int pairs = silu ? M : (M + 1) / 2, steps = (K + 255) / 256;
+  int wk = 1;
+  while (wk < 8 && (long long)pairs * wk / 8 < 592 && steps / (wk * 2) >= 2) wk *= 2;
+  const int blocks = (pairs + 8 / wk - 1) / (8 / wk);
+  Args a{(const __nv_bfloat16*)w, (const __nv_bfloat16*)x, (const __nv_bfloat16*)bias, out, M, K, n, wk, f32, silu};
+  return N == 1 ? launch<1>(a, blocks, stream) : N == 2 ? launch<2>(a, blocks, stream) : launch<4>(a, blocks, stream);
+}
+
+}  // extern "C"

@@ -232,7 +232,7 @@ class Fanodra:
             elif isinstance(o, dict):
                 todo += o.values()
             elif type(o).__module__.startswith("sparkflash_b200.models"):
-                todo += vars(o).values()
+                todo += [v for k, v in vars(o).items() if k not in ("engine", "run_state")]
         return total
 
     # ---- layered engine -----------------------------------------------------------------------------------------------
@@ -299,6 +299,4 @@ class Fanodra:
             return None
         V = self.vocab
         out = s.scratch.get("logits", s.nhead, V) if s.single else torch.empty((s.nhead, V), dtype=torch.float32, device=x.device)
-        if self.dtype == torch.float32:
-            return torch.mm(hf, self.embed.t(), out=out)
-        return torch.mm(hf, self.embed.t(), out_dtype=torch.float32, out=out)
+        return R.head(hf, self.embed, out)

@@ -54,6 +54,7 @@ class BiasedAttention:
         self.bias = log_distance_bias(w.f32("r1"), w.f32("r2"), max_context, w.device)
         self.wo, self.bo = w.act("o"), w.act("o.b")
         self.tc = R.attn_tc_supports(self.wo.dtype, self.dim, self.vdim)
+        self.stream = R.attn_stream_supports(self.wo.dtype, self.dim, self.vdim)
 
     PROJ, PROJ_BIAS = ("q", "k", "v"), ("q.b", "k.b", "v.b")
 
@@ -64,6 +65,8 @@ class BiasedAttention:
         # partial outputs of split rows: rows x heads x ranges, bounded by the blocks of one launch (see LayeredEngine.splits)
         per = self.H // R.attn_blocks(self.H, self.G)
         parts = max(1, per) * 1024 + self.H * 64
+        if self.stream:
+            parts = max(parts, 2 * R.STREAM_CTAS * R.attn_stream_heads(self.H, self.G, self.dim))
         e.scratch.reserve("attn_part", parts * self.vdim, torch.float32)
         e.scratch.reserve("attn_ml", parts * 2, torch.float32)
 
@@ -75,7 +78,10 @@ class BiasedAttention:
         R.qk_append(proj, self.q_norm, self.k_norm, q, k, v, s.table, s.row_lane, s.row_pos, n, self.H, self.eps, s.status)
         if s.ntiles:
             R.attn_tc(q, kv, s.table, s.row_lane, s.row_pos, s.tiles, s.ntiles, self.bias, o, self.H, self.scale, s.status)
-        if s.short:
+        if s.short and self.stream and s.short <= R.STREAM_ROWS:
+            R.attn_stream(q, k, v, s.table, s.row_lane, s.row_pos, s.short_rows, s.short, self.bias, o, s.scratch.buf["attn_part"],
+                          s.scratch.buf["attn_ml"], self.H, self.scale, s.short * s.pages, s.status)
+        elif s.short:
             blocks = R.attn_blocks(self.H, self.G)
             sp = s.engine.splits(s, s.short, blocks)
             part = s.scratch.buf["attn_part"] if sp > 1 else None
@@ -188,7 +194,5 @@ class DenseFF:
         e.scratch.reserve("ff_act", e.max_rows * self.ff, self.w_in.dtype)
 
     def run(self, s, h):
-        gu = R.linear(h, self.w_in, None, s.scratch.get("proj", s.n, 2 * self.ff))
-        act = s.scratch.get("ff_act", s.n, self.ff)
-        R.silu_mul(gu, act, s.n)
+        act = R.gated_linear(h, self.w_in, s.scratch.get("proj", s.n, 2 * self.ff), s.scratch.get("ff_act", s.n, self.ff))
         return R.linear(act, self.w_out, None, s.scratch.get("y", s.n, h.shape[1]))

@@ -11,6 +11,7 @@ from ctypes import c_float, c_int, c_int64, c_void_p
 import torch
 
 from .. import _lib
+from ..runtime.segments import note
 from .native import _check, _p, _stream
 
 MAX_TAPS = 8
@@ -79,11 +80,40 @@ def sample(logits, row_pos, temperature, seed, mask, best_val, best_id, n):
                                   c_int(0), _stream()), "sample")
 
 
+GEMV_ROWS = 4
+
+
+def _gemv_takes(x: torch.Tensor) -> bool:
+    n, K = x.shape
+    return x.dtype == torch.bfloat16 and n <= GEMV_ROWS and K % 8 == 0 and (n if n < 3 else 4) * K * 2 <= 200 * 1024
+
+
+def _gemv(x, w, b, out, silu: bool) -> None:
+    _check(_lib.rows().sfb_rows_gemv(_p(w), _p(x), _p(b), _p(out), c_int(x.shape[0]), c_int(out.shape[1]), c_int(x.shape[1]),
+                                     c_int(out.dtype == torch.float32), c_int(silu), _stream()), "rows_gemv")
+
+
 def linear(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor | None, out: torch.Tensor) -> torch.Tensor:
-    """out = x w^T (+ b): a library product with 32-bit accumulation."""
+    """out = x w^T (+ b) with 32-bit accumulation: up to four bf16 rows by the streaming kernel, a library product otherwise."""
+    if _gemv_takes(x):
+        _gemv(x, w, b, out, False)
+        return out
     if b is not None:
-        return torch.addmm(b, x, w.t(), out=out)
-    return torch.mm(x, w.t(), out=out)
+        torch.addmm(b, x, w.t(), out=out)
+    else:
+        torch.mm(x, w.t(), out=out)
+    note("linear")
+    return out
+
+
+def gated_linear(x: torch.Tensor, w: torch.Tensor, scratch: torch.Tensor | None, out: torch.Tensor) -> torch.Tensor:
+    """out = silu(x wg^T) * (x wu^T), w = wg stacked on wu; ``scratch`` [n, 2 ff] holds both products where they are not fused."""
+    if _gemv_takes(x):
+        _gemv(x, w, None, out, True)
+        return out
+    linear(x, w, None, scratch)
+    silu_mul(scratch, out, x.shape[0])
+    return out
 
 
 class exact_matmul:
@@ -104,8 +134,24 @@ def block_gates(u: torch.Tensor, wg: torch.Tensor, out: torch.Tensor) -> torch.T
     parts, _, bs = wg.shape
     x = u.view(u.shape[0], parts, bs).transpose(0, 1)
     if u.dtype == torch.float32:
-        return torch.bmm(x, wg.transpose(1, 2), out=out)
-    return torch.bmm(x, wg.transpose(1, 2), out_dtype=torch.float32, out=out)
+        torch.bmm(x, wg.transpose(1, 2), out=out)
+    else:
+        torch.bmm(x, wg.transpose(1, 2), out_dtype=torch.float32, out=out)
+    note("block_gates")
+    return out
+
+
+def head(x: torch.Tensor, embed: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """32-bit logits of x [rows, width] against the tied table."""
+    if _gemv_takes(x):
+        _gemv(x, embed, None, out, False)
+        return out
+    if x.dtype == torch.float32:
+        torch.mm(x, embed.t(), out=out)
+    else:
+        torch.mm(x, embed.t(), out_dtype=torch.float32, out=out)
+    note("head")
+    return out
 
 
 def attn_blocks(heads: int, kv_heads: int) -> int:
@@ -113,6 +159,31 @@ def attn_blocks(heads: int, kv_heads: int) -> int:
     rep = heads // kv_heads
     r = 1 if rep <= 1 else 2 if rep <= 2 else 4 if rep <= 4 else 8
     return kv_heads * -(-rep // r)
+
+
+STREAM_CTAS = 592          # most CTAs of the streaming arm (csrc/k_rows_attn_dec.cu)
+STREAM_ROWS = 1024
+
+
+def attn_stream_heads(heads: int, kv_heads: int, dim: int) -> int:
+    """Query heads the streaming arm handles per pass over a key head's pages."""
+    rep = heads // kv_heads
+    r = 1 if rep <= 1 else 2 if rep <= 2 else 4
+    return min(r, 2) if dim > 128 else r
+
+
+def attn_stream_supports(dtype: torch.dtype, dim: int, vdim: int) -> bool:
+    return dtype == torch.bfloat16 and dim in (32, 64, 96, 128, 256) and vdim % 32 == 0 and vdim <= 256
+
+
+def attn_stream(q, kpool, vpool, table, row_lane, row_pos, rows, n_rows, bias, out, part, ml, heads, scale, page_bound, status):
+    """Single rows, bf16: the pages of all rows cut evenly over the machine.  ``page_bound``: at least the sum of the rows' pages."""
+    G, dim, vdim = kpool.shape[1], kpool.shape[3], vpool.shape[3]
+    _check(_lib.rows().sfb_rows_attn_stream(_p(q), _p(kpool), _p(vpool), _p(table), _p(row_lane), _p(row_pos), _p(rows), _p(bias),
+                                            c_int64(bias.shape[1] if bias is not None else 0), _p(out), _p(part), _p(ml), c_int(table.shape[1]),
+                                            c_int(kpool.shape[0]), c_int(n_rows), c_int(heads), c_int(G), c_int(dim), c_int(vdim),
+                                            c_int(attn_stream_heads(heads, G, dim)), c_int(page_bound), c_float(scale), _p(status), _stream()),
+           "rows_attn_stream")
 
 
 def attn_tc_supports(dtype: torch.dtype, dim: int, vdim: int) -> bool:

@@ -125,9 +125,9 @@ def test_gated_recurrence_chunks_and_single_rows(dt, parts, bs, taps):
         n = len(x)
         u, o, gates = torch.empty_like(x), torch.empty_like(x), torch.empty(parts, n, 2 * bs, device="cuda")
         R.conv(x, W, B, u, hist, seg, n, residual=False)
-        with R.exact_matmul():
-            R.block_gates(u, wg, gates)
-        for _ in range(2):
+        for _ in range(2):          # a repeated launch gives the same result
+            with R.exact_matmul():
+                R.block_gates(u, wg, gates)
             R.scan(gates, RB, IB, decay, u, y, o, S, sums, seg, n, bs)
         return o.float().cpu()
     # a prompt portion of both lanes (several chunks), then single rows through the fused kernel, then a portion again
@@ -196,6 +196,20 @@ def _run_exact(case, rows, splits):
     return out.float().cpu()
 
 
+def _run_stream(case, rows, picked=None, slack=0):
+    """rows: (lane, position) pairs; ``picked``: run only these of them."""
+    q = torch.stack([case.q[a][p] for a, p in rows]).to("cuda", case.dt)
+    out = torch.full((len(rows), case.H * case.vdim), 9.0, dtype=case.dt, device="cuda")
+    n = 2 * R.STREAM_CTAS * R.attn_stream_heads(case.H, case.G, case.dim)
+    part, ml, st = torch.full((n * case.vdim,), float("nan"), device="cuda"), torch.full((n * 2,), float("nan"), device="cuda"), _status()
+    run = range(len(rows)) if picked is None else picked
+    R.attn_stream(q, case.kv.k[0], case.kv.v[0], case.kv.table, _i32([a for a, _ in rows]), _i32([p for _, p in rows]),
+                  None if picked is None else _i32(picked), len(run), case.bias, out, part, ml, case.H, case.scale,
+                  slack + sum(rows[i][1] // PAGE + 1 for i in run), st)
+    assert st.tolist()[0] == 0, st.tolist()
+    return out.float().cpu()
+
+
 def _run_tiles(case, runs):
     """runs: (lane, first position, rows) segments through the tensor-core arm."""
     lanes = [a for a, _, m in runs for _ in range(m)]
@@ -242,27 +256,46 @@ def test_tensor_core_attention_runs_match_the_equations(H, G, dim, vdim):
             assert (o - want[a][p:p + m]).abs().max() < 0.02, (runs, a, (o - want[a][p:p + m]).abs().max())
 
 
-@pytest.mark.parametrize("arm", ["exact32", "exact16", "tiles"])
+@pytest.mark.parametrize("H,G,dim,vdim", [(4, 4, 64, 64), (4, 2, 128, 128), (5, 1, 32, 96), (3, 1, 96, 32), (2, 1, 256, 256), (7, 1, 64, 160), (2, 2, 128, 64)])
+def test_streamed_attention_of_rows_of_many_lengths(H, G, dim, vdim):
+    case = _attention_case(torch.bfloat16, H, G, dim, vdim, [1, 64, 65, 1000, 300])
+    _fill(case)
+    want = [_want(case, a) for a in range(5)]
+    many = [(a, p) for a, n in enumerate((1, 64, 65, 1000, 300)) for p in {0, n - 1, n // 2, max(0, n - 7), min(63, n - 1), min(64, n - 1)}]
+    for rows in ([(3, 999)], [(0, 0)], [(0, 0), (3, 640)], [(2, 64), (1, 63), (1, 0)], many, many * 9):
+        for slack in (0, 5000):                     # few CTAs, or as many as the machine takes
+            got = _run_stream(case, rows, slack=slack)
+            for (a, p), row in zip(rows, got):
+                assert (row - want[a][p]).abs().max() < 0.03, (a, p, len(rows), slack)
+    got = _run_stream(case, many, picked=[5, 1, 8])
+    for i in (5, 1, 8):
+        assert (got[i] - want[many[i][0]][many[i][1]]).abs().max() < 0.03
+    assert (got[0] == 9).all()                      # rows that are not picked are left alone
+
+
+@pytest.mark.parametrize("arm", ["exact32", "exact16", "stream", "tiles"])
 def test_one_far_key_stands_out(arm):
     """One query's score against one key is far above the rest: its value must come back, wherever the key lies."""
     dt = torch.float32 if arm == "exact32" else torch.bfloat16
+    _run_rows = (lambda c, rows, _: _run_stream(c, rows)) if arm == "stream" else _run_exact
+    VD = 32
     for key in (0, 1, 63, 64, 65, 127, 128, 255, 256, 383, 384, 510, 511):
-        case = _attention_case(dt, 2, 1, 32, 16, [512], seed=key, scale=1.0)
+        case = _attention_case(dt, 2, 1, 32, VD, [512], seed=key, scale=1.0)
         q = 511 if key % 2 else max(key, 480)
         case.k[0][key] = 0
         case.k[0][key, :4] = 6.0
         case.q[0][:, :] *= 0.1
         case.q[0][q].view(2, 32)[:, :4] = 3.0                   # score 72 against the key, a few at most against any other
         _fill(case)
-        got = _run_tiles(case, [(0, 400, 112)])[q - 400] if arm == "tiles" else _run_exact(case, [(0, q)], 3)[0]
-        assert (got.view(2, 16) - case.v[0][key]).abs().max() < 0.02, (arm, key)
+        got = _run_tiles(case, [(0, 400, 112)])[q - 400] if arm == "tiles" else _run_rows(case, [(0, q)], 3)[0]
+        assert (got.view(2, VD) - case.v[0][key]).abs().max() < 0.02, (arm, key)
         # the row before the key does not see it
         if 0 < key < 511 and arm != "tiles":
             case.q[0][key - 1].view(2, 32)[:, :4] = 3.0
-            assert (_run_exact(case, [(0, key - 1)], 2)[0].view(2, 16) - case.v[0][key]).abs().max() > 0.5
+            assert (_run_rows(case, [(0, key - 1)], 2)[0].view(2, VD) - case.v[0][key]).abs().max() > 0.5
         if arm == "tiles" and key > 460:
             case.q[0][key - 1].view(2, 32)[:, :4] = 3.0
-            assert (_run_tiles(case, [(0, 400, 112)])[key - 1 - 400].view(2, 16) - case.v[0][key]).abs().max() > 0.5
+            assert (_run_tiles(case, [(0, 400, 112)])[key - 1 - 400].view(2, VD) - case.v[0][key]).abs().max() > 0.5
 
 
 def test_large_scores_and_rising_maxima():
@@ -275,7 +308,8 @@ def test_large_scores_and_rising_maxima():
     _fill(case)
     want = _want(case, 0)
     assert (_run_tiles(case, [(0, 0, 600)]) - want).abs().max() < 0.02
-    assert (_run_exact(case, [(0, p) for p in (63, 200, 599)], 4) - want[[63, 200, 599]]).abs().max() < 0.02
+    for run in (lambda r: _run_exact(case, r, 4), lambda r: _run_stream(case, r)):
+        assert (run([(0, p) for p in (63, 200, 599)]) - want[[63, 200, 599]]).abs().max() < 0.02
 
 
 @pytest.mark.parametrize("dt", DTYPES)
@@ -299,3 +333,22 @@ def test_query_key_norm_covers_the_whole_projection(dt, H, G, dim, vdim):
         page = kv.pages[1][p // PAGE]
         assert (kv.k[0][page, :, p % PAGE].float().cpu() - k[i]).abs().max() < 2 * _tol(dt)
         assert torch.equal(kv.v[0][page, :, p % PAGE].float().cpu(), v[i])
+
+
+@pytest.mark.parametrize("M,K", [(40, 64), (33, 24), (2048, 2048), (96, 5128), (4100, 512)])
+def test_few_row_products(M, K):
+    g = torch.Generator().manual_seed(M)
+    for n in (1, 2, 3, 4):
+        x, w, b = torch.randn(n, K, generator=g).bfloat16(), (torch.randn(M, K, generator=g) * K ** -0.5).bfloat16(), torch.randn(M, generator=g).bfloat16()
+        want = x.double() @ w.double().T
+        out = torch.zeros(n, M, dtype=torch.bfloat16, device="cuda")
+        assert R._gemv_takes(x)
+        R.linear(x.cuda(), w.cuda(), b.cuda(), out)
+        assert (out.cpu().double() - want - b.double()).abs().max() < 0.04
+        logits = torch.zeros(n, M, device="cuda")
+        R.head(x.cuda(), w.cuda(), logits)
+        assert (logits.cpu().double() - want).abs().max() < 1e-4
+        if M % 2 == 0:
+            act = torch.zeros(n, M // 2, dtype=torch.bfloat16, device="cuda")
+            R.gated_linear(x.cuda(), w.cuda(), None, act)
+            assert (act.cpu().double() - P.silu(want[:, :M // 2]) * want[:, M // 2:]).abs().max() < 0.08
