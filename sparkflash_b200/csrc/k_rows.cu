@@ -41,10 +41,11 @@ struct SeamArgs {
   Status* status;
 };
 
-// Mean and sum of squared deviations of a row held as x[NV][V] per thread (`mine` = how many of them exist, `wcnt` = the warp's
-// total): each warp takes both about its own mean, then the warps' pairs are combined - one barrier.
+// Mean and sum of squared deviations of a row held as x[NV][V] per thread (`wcnt` = how many of the elements are this warp's):
+// each warp takes both about its own mean, then the warps' pairs are combined - one barrier.
 template <int V, int NV>
-__device__ __forceinline__ void row_moments(const float (&x)[NV][V], int c0, int step, int d, float wcnt, float* sh, int& phase, float& mu, float& m2) {
+__device__ __forceinline__ void row_moments(const float (&x)[NV][V], int c0, int step, int d, float wcnt, float winv, float inv_d, float* sh, int& phase,
+                                            float& mu, float& m2) {
   const int lane = threadIdx.x & 31, w = threadIdx.x >> 5, nw = blockDim.x >> 5;
   float* s = sh + (phase & 1) * 96;
   phase ^= 1;
@@ -55,8 +56,7 @@ __device__ __forceinline__ void row_moments(const float (&x)[NV][V], int c0, int
 #pragma unroll
       for (int k = 0; k < V; ++k) t += x[i][k];
     }
-  t = warp_sum(t);
-  const float wm = wcnt > 0.f ? t / wcnt : 0.f;
+  const float wm = warp_sum(t) * winv;
 #pragma unroll
   for (int i = 0; i < NV; ++i)
     if (c0 + i * step < d) {
@@ -64,26 +64,25 @@ __device__ __forceinline__ void row_moments(const float (&x)[NV][V], int c0, int
       for (int k = 0; k < V; ++k) { const float e = x[i][k] - wm; q += e * e; }
     }
   q = warp_sum(q);
-  if (lane == 0) { s[w] = t; s[32 + w] = q; s[64 + w] = wcnt; }
+  if (lane == 0) { s[w] = wm; s[32 + w] = q; s[64 + w] = wcnt; }
   __syncthreads();
-  t = 0.f;
-  for (int i = 0; i < nw; ++i) t += s[i];
-  mu = t / (float)d;
-  m2 = 0.f;
-  for (int i = 0; i < nw; ++i) {
-    const float c = s[64 + i], e = (c > 0.f ? s[i] / c : 0.f) - mu;
-    m2 += s[32 + i] + c * e * e;
-  }
+  mu = m2 = 0.f;
+  for (int i = 0; i < nw; ++i) mu += s[i] * s[64 + i];
+  mu *= inv_d;
+  for (int i = 0; i < nw; ++i) { const float e = s[i] - mu; m2 += s[32 + i] + s[64 + i] * e * e; }
 }
 
-template <typename T, int V, int NV>
+// AHEAD (few rows): weights and the convolution's carried inputs are requested before they are needed, the former before the
+// previous kernel has finished; with many rows that only costs registers.
+template <typename T, int V, int NV, bool AHEAD>
 __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
   __shared__ float sh[2 * 96], sh2[2 * 2 * 32];
   int phase = 0, phase2 = 0;
   const int d = a.d, step = blockDim.x * V, c0 = threadIdx.x * V;
   const float inv_d = 1.f / (float)d;
-  constexpr bool AHEAD = NV <= 2;      // the weights of a short row are requested before the previous kernel has finished
-  float pw[NV][V], pb[NV][V], nw[NV][V], nb[NV][V];
+  constexpr int TW = AHEAD ? 4 : 1;      // taps held ahead
+  float pw[NV][V], pb[NV][V], nw[NV][V], nb[NV][V], cw[TW][NV][V], cg[TW][NV][V];
+  const bool ahead_conv = AHEAD && a.cw && a.taps <= TW;
   if constexpr (AHEAD) {
 #pragma unroll
     for (int i = 0; i < NV; ++i) {
@@ -91,6 +90,11 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
       if (c >= d) continue;
       if (a.y) { load_v<float, V>(a.pw + c, pw[i]); load_v<float, V>(a.pb + c, pb[i]); }
       if (a.nw) { load_v<float, V>(a.nw + c, nw[i]); load_v<float, V>(a.nb + c, nb[i]); }
+      if (ahead_conv) {
+#pragma unroll
+        for (int j = 0; j < TW; ++j)
+          if (j < a.taps) load_v<float, V>(a.cw + (size_t)j * d + c, cw[j][i]);
+      }
     }
   }
   pdl_launch_dependents();
@@ -99,7 +103,25 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
   int mine = 0;
 #pragma unroll
   for (int i = 0; i < NV; ++i) mine += max(0, min(V, d - (c0 + i * step)));
-  const float wcnt = warp_sum((float)mine);
+  const float wcnt = warp_sum((float)mine), winv = wcnt > 0.f ? 1.f / wcnt : 0.f;
+  const int W = a.taps - 1;
+  const int src = a.cw ? a.src[row] : -1;
+  T* hd = a.cw ? (T*)a.hist + (size_t)a.dst[row] * W * d : nullptr;
+  const T* hs = src >= 0 ? (const T*)a.hist + (size_t)src * W * d : nullptr;
+  if constexpr (AHEAD) {
+    if (ahead_conv) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+#pragma unroll
+        for (int j = 0; j < TW - 1; ++j) {
+          if (j < W && hs && c0 + i * step < d) load_v<T, V>(hs + (size_t)j * d + c0 + i * step, cg[j][i]);
+          else {
+#pragma unroll
+            for (int k = 0; k < V; ++k) cg[j][i][k] = 0.f;
+          }
+        }
+    }
+  }
   float x[NV][V], e[NV][V];
   const bool want_embed = a.from_embed || a.add_embed;
   if (want_embed) {
@@ -148,7 +170,7 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
         if (c0 + i * step < d) load_v<T, V>(yr + c0 + i * step, y[i]);
     }
     float mu, m2;
-    row_moments<V, NV>(y, c0, step, d, wcnt, sh, phase, mu, m2);
+    row_moments<V, NV>(y, c0, step, d, wcnt, winv, inv_d, sh, phase, mu, m2);
     const float rs = 1.f / sqrtf(m2 * inv_d + a.eps);
 #pragma unroll
     for (int i = 0; i < NV; ++i)
@@ -182,13 +204,9 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
     }
   if (!a.nw) return;
   float mu, m2;
-  row_moments<V, NV>(x, c0, step, d, wcnt, sh, phase, mu, m2);
+  row_moments<V, NV>(x, c0, step, d, wcnt, winv, inv_d, sh, phase, mu, m2);
   const float rs = 1.f / sqrtf(m2 * inv_d + a.eps);
   T* hr = (T*)a.h + (size_t)out_row * d;
-  const int W = a.taps - 1;
-  const int src = a.cw ? a.src[row] : -1;
-  T* hd = a.cw ? (T*)a.hist + (size_t)a.dst[row] * W * d : nullptr;
-  const T* hs = src >= 0 ? (const T*)a.hist + (size_t)src * W * d : nullptr;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int c = c0 + i * step;
@@ -202,6 +220,26 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
       float acc[V], t[V];
 #pragma unroll
       for (int k = 0; k < V; ++k) o[k] = to_f<T>(from_f<T>(o[k]));
+      if (ahead_conv) {
+#pragma unroll
+        for (int k = 0; k < V; ++k) acc[k] = 0.f;
+#pragma unroll
+        for (int j = 0; j < TW; ++j) {
+          if (j < W) {
+#pragma unroll
+            for (int k = 0; k < V; ++k) acc[k] += cw[j][i][k] * cg[j][i][k];
+            if (j > 0) store_v<T, V>(hd + (size_t)(j - 1) * d + c, cg[j][i]);
+          } else if (j == W) {
+#pragma unroll
+            for (int k = 0; k < V; ++k) acc[k] += cw[j][i][k] * o[k];
+          }
+        }
+        if (W > 0) store_v<T, V>(hd + (size_t)(W - 1) * d + c, o);
+#pragma unroll
+        for (int k = 0; k < V; ++k) o[k] += acc[k];
+        store_v<T, V>(hr + c, o);
+        continue;
+      }
       load_v<float, V>(a.cw + (size_t)W * d + c, t);
 #pragma unroll
       for (int k = 0; k < V; ++k) acc[k] = t[k] * o[k];
@@ -379,10 +417,11 @@ struct ScanArgs {
   int64_t y_stride;
   void* out;                // [n, width] (T)
   float* S;                 // [slots, width]
-  float2* sums;             // [chunks, width] (product of a, end value from a zero start)
+  float2* sums;             // [chunks, width] (product of a, end value from a zero start), then (start state, -)
   const int *chunk_seg, *chunk_row0, *chunk_rows, *chunk_first;   // chunk_first: first chunk of the same segment
   const int *seg_src, *seg_dst, *seg_row0, *seg_len;
-  int n, width, bs;
+  int* tickets;             // one per 128 channels, zero between launches
+  int n, width, bs, chunks;
 };
 
 // exp, reciprocal and square root of the gates, all 32-bit: library-accurate with float activations; with bf16 activations the
@@ -401,9 +440,15 @@ __device__ __forceinline__ float one_minus_exp(float t, float e) {
 // decay a and input b of one step from the gate pre-activations
 template <typename T> __device__ __forceinline__ void gate_step(float zr, float zi, float decay, float u, float& a, float& b) {
   const float la = -decay * gate_sigmoid<T>(zr);
-  a = expf(la);
+  if constexpr (sizeof(T) == 4) a = expf(la);
+  else a = __expf(la);
   const float m = one_minus_exp(2.f * la, a * a);
-  b = sqrtf(m) * (gate_sigmoid<T>(zi) * u);
+  if constexpr (sizeof(T) == 4) b = sqrtf(m) * (gate_sigmoid<T>(zi) * u);
+  else {
+    float r;
+    asm("sqrt.approx.f32 %0, %1;" : "=f"(r) : "f"(m));
+    b = r * (gate_sigmoid<T>(zi) * u);
+  }
 }
 template <typename T> __device__ __forceinline__ float gate_gelu(float z) {
   if constexpr (sizeof(T) == 4) return gelu_tanh_f(z);
@@ -439,14 +484,11 @@ __global__ void __launch_bounds__(128) scan_short_kernel(ScanArgs a) {
   a.S[(size_t)a.seg_dst[seg] * a.width + c] = S;
 }
 
-// Longer segments, pass 1: (a, b) of every step, in place of the gate pre-activations, and every chunk's summary.
+// Longer segments, pass 1: (a, b) of every step, in place of the gate pre-activations, and every chunk's summary; the last CTA of a
+// column to arrive (a ticket, nobody waits) turns the column's summaries into the chunks' start states and writes the final states.
 constexpr int SCAN_T = 8;    // rows whose loads are in flight together
 template <typename T>
-__global__ void __launch_bounds__(128) scan_gates_kernel(ScanArgs a) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
-  if (c >= a.width) return;
+__device__ __forceinline__ void chunk_gates(const ScanArgs& a, int c) {
   const int ch = blockIdx.y, row0 = a.chunk_row0[ch], rows = a.chunk_rows[ch];
   const int b = c / a.bs, j = c - b * a.bs;
   float* g = const_cast<float*>(a.gates) + ((size_t)b * a.n + row0) * 2 * a.bs + j;
@@ -475,38 +517,70 @@ __global__ void __launch_bounds__(128) scan_gates_kernel(ScanArgs a) {
   a.sums[(size_t)ch * a.width + c] = make_float2(P, S);
 }
 
-// Pass 2: the chunk's start from the summaries before it, then the recurrence and the output gate.
+template <typename T>
+__global__ void __launch_bounds__(128) scan_gates_kernel(ScanArgs a) {
+  __shared__ int last;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int c = blockIdx.x * blockDim.x + threadIdx.x;
+  if (c < a.width) chunk_gates<T>(a, c);
+  __threadfence();
+  __syncthreads();
+  if (threadIdx.x == 0) last = atomicAdd(a.tickets + blockIdx.x, 1) == a.chunks - 1;
+  __syncthreads();
+  if (!last) return;
+  if (threadIdx.x == 0) a.tickets[blockIdx.x] = 0;      // for the next launch
+  __threadfence();
+  if (c >= a.width) return;
+  constexpr int B = 16;
+  float S = 0.f;
+  for (int k0 = 0; k0 < a.chunks; k0 += B) {
+    float2 t[B];
+    int first[B + 1];                      // chunk k + 1 begins a segment: chunk k ends one
+#pragma unroll
+    for (int i = 0; i < B; ++i)
+      if (k0 + i < a.chunks) t[i] = __ldcg(a.sums + (size_t)(k0 + i) * a.width + c);
+#pragma unroll
+    for (int i = 0; i <= B; ++i) first[i] = k0 + i < a.chunks ? a.chunk_first[k0 + i] : k0 + i;
+#pragma unroll
+    for (int i = 0; i < B; ++i) {
+      const int k = k0 + i;
+      if (k >= a.chunks) break;
+      if (first[i] == k) {
+        const int src = a.seg_src[a.chunk_seg[k]];
+        S = src >= 0 ? a.S[(size_t)src * a.width + c] : 0.f;
+      }
+      a.sums[(size_t)k * a.width + c].x = S;
+      S = fmaf(t[i].x, S, t[i].y);
+      if (first[i + 1] == k + 1) a.S[(size_t)a.seg_dst[a.chunk_seg[k]] * a.width + c] = S;
+    }
+  }
+}
+
+// Pass 2: the recurrence from the chunk's start state, and the output gate.
 template <typename T>
 __global__ void __launch_bounds__(128) scan_apply_kernel(ScanArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= a.width) return;
-  const int ch = blockIdx.y, seg = a.chunk_seg[ch], row0 = a.chunk_row0[ch], rows = a.chunk_rows[ch], first = a.chunk_first[ch];
-  const int src = a.seg_src[seg];
-  float S = src >= 0 ? a.S[(size_t)src * a.width + c] : 0.f;
-  const float2* sums = a.sums + c;
-  int k = first;
-  for (; k + 8 <= ch; k += 8) {
-    float2 t[8];
-#pragma unroll
-    for (int i = 0; i < 8; ++i) t[i] = sums[(size_t)(k + i) * a.width];
-#pragma unroll
-    for (int i = 0; i < 8; ++i) S = fmaf(t[i].x, S, t[i].y);
-  }
-  for (; k < ch; ++k) { const float2 t = sums[(size_t)k * a.width]; S = fmaf(t.x, S, t.y); }
+  const int ch = blockIdx.y, row0 = a.chunk_row0[ch], rows = a.chunk_rows[ch];
+  float S = a.sums[(size_t)ch * a.width + c].x;
   const int b = c / a.bs, j = c - b * a.bs;
   const float* g = a.gates + ((size_t)b * a.n + row0) * 2 * a.bs + j;
   const T* Y = (const T*)a.y + (size_t)row0 * a.y_stride + c;
   T* O = (T*)a.out + (size_t)row0 * a.width + c;
-  for (int t0 = 0; t0 < rows; t0 += SCAN_T) {
-    float at[SCAN_T], bt[SCAN_T], y[SCAN_T];
+  float at[SCAN_T], bt[SCAN_T], y[SCAN_T];
+  auto fetch = [&](int t0) {
 #pragma unroll
     for (int i = 0; i < SCAN_T; ++i)
       if (t0 + i < rows) {
         const float* gp = g + (size_t)(t0 + i) * 2 * a.bs;
         at[i] = gp[0]; bt[i] = gp[a.bs]; y[i] = to_f<T>(Y[(size_t)(t0 + i) * a.y_stride]);
       }
+  };
+  for (int t0 = 0; t0 < rows; t0 += SCAN_T) {
+    fetch(t0);
 #pragma unroll
     for (int i = 0; i < SCAN_T; ++i)
       if (t0 + i < rows) {
@@ -514,7 +588,6 @@ __global__ void __launch_bounds__(128) scan_apply_kernel(ScanArgs a) {
         O[(size_t)(t0 + i) * a.width] = from_f<T>(S * gate_gelu<T>(y[i]));
       }
   }
-  if (row0 + rows == a.seg_row0[seg] + a.seg_len[seg]) a.S[(size_t)a.seg_dst[seg] * a.width + c] = S;
 }
 
 // Single-row segments: convolution, gates, recurrence and output gate of one part of the width in one kernel.
@@ -535,13 +608,22 @@ struct GatedRowArgs {
 constexpr int GATED_RB = 4;
 
 template <typename T, int V>
-__global__ void __launch_bounds__(256) gated_row_kernel(GatedRowArgs a) {
+__global__ void __launch_bounds__(256, 2) gated_row_kernel(GatedRowArgs a) {
   extern __shared__ float us[];             // [RB][bs rounded up to 8]
-  pdl_launch_dependents();
-  pdl_wait();
   const int part = blockIdx.x / a.tiles, tile = blockIdx.x % a.tiles;
   const int r0 = blockIdx.y * GATED_RB, nr = min(GATED_RB, a.n - r0);
   const int W = a.taps - 1, ld = (a.bs + 7) & ~7;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int j0 = tile * a.per_tile + warp, j1 = min((tile + 1) * a.per_tile, a.bs);
+  // the first weight rows are requested before the previous kernel has finished: they do not depend on it
+  float wr0[V], wi0[V];
+  const bool pre = V == 8 && j0 < j1 && lane * V < a.bs;
+  if (pre) {
+    const T* w = (const T*)a.wg + ((size_t)part * 2 * a.bs + j0) * a.bs + lane * V;
+    if constexpr (V == 8) { load8<T>(w, wr0); load8<T>(w + (size_t)a.bs * a.bs, wi0); }
+  }
+  pdl_launch_dependents();
+  pdl_wait();
   for (int idx = threadIdx.x; idx < GATED_RB * a.bs; idx += blockDim.x) {
     const int i = idx / a.bs, j = idx - i * a.bs, c = part * a.bs + j;
     float acc = 0.f;
@@ -562,9 +644,7 @@ __global__ void __launch_bounds__(256) gated_row_kernel(GatedRowArgs a) {
     us[i * ld + j] = acc;
   }
   __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int j1 = min((tile + 1) * a.per_tile, a.bs);
-  for (int j = tile * a.per_tile + warp; j < j1; j += 8) {
+  for (int j = j0; j < j1; j += 8) {
     const T* wr = (const T*)a.wg + ((size_t)part * 2 * a.bs + j) * a.bs;
     const T* wi = wr + (size_t)a.bs * a.bs;
     float dr[GATED_RB], di[GATED_RB];
@@ -572,7 +652,10 @@ __global__ void __launch_bounds__(256) gated_row_kernel(GatedRowArgs a) {
     for (int i = 0; i < GATED_RB; ++i) dr[i] = di[i] = 0.f;
     for (int k = lane * V; k < a.bs; k += 32 * V) {
       float fr[V], fi[V];
-      if constexpr (V == 8) { load8<T>(wr + k, fr); load8<T>(wi + k, fi); }
+      if (V == 8 && j == j0 && k == lane * V) {
+#pragma unroll
+        for (int v = 0; v < V; ++v) { fr[v] = wr0[v]; fi[v] = wi0[v]; }
+      } else if constexpr (V == 8) { load8<T>(wr + k, fr); load8<T>(wi + k, fi); }
       else { load_v<T, 1>(wr + k, fr); load_v<T, 1>(wi + k, fi); }
 #pragma unroll
       for (int i = 0; i < GATED_RB; ++i) {
@@ -617,15 +700,17 @@ __global__ void __launch_bounds__(256) silu_mul_kernel(const T* gu, T* out, int 
 template <typename T, int V>
 static int launch_seam(const SeamArgs& a, int n, cudaStream_t st) {
   const int vecs = (a.d + V - 1) / V;
-  int nv = 1;
-  while (nv < 8 && (vecs + nv - 1) / nv > 256) nv *= 2;
+  const bool few = n <= 296;
+  int nv = 1;                              // few rows: many threads per row; many rows: more of the row per thread
+  while (nv < 8 && (vecs + nv - 1) / nv > (few ? 256 : nv < 4 ? 128 : 256)) nv *= 2;
   const int threads = ((vecs + nv - 1) / nv + 31) / 32 * 32;
   if (threads > 512) return (int)cudaErrorInvalidValue;
+  const dim3 g(n), b(threads);
   switch (nv) {
-    case 1: return (int)sfb_launch(seam_kernel<T, V, 1>, dim3(n), dim3(threads), 0, st, a);
-    case 2: return (int)sfb_launch(seam_kernel<T, V, 2>, dim3(n), dim3(threads), 0, st, a);
-    case 4: return (int)sfb_launch(seam_kernel<T, V, 4>, dim3(n), dim3(threads), 0, st, a);
-    default: return (int)sfb_launch(seam_kernel<T, V, 8>, dim3(n), dim3(threads), 0, st, a);
+    case 1: return (int)(few ? sfb_launch(seam_kernel<T, V, 1, true>, g, b, 0, st, a) : sfb_launch(seam_kernel<T, V, 1, false>, g, b, 0, st, a));
+    case 2: return (int)(few ? sfb_launch(seam_kernel<T, V, 2, true>, g, b, 0, st, a) : sfb_launch(seam_kernel<T, V, 2, false>, g, b, 0, st, a));
+    case 4: return (int)sfb_launch(seam_kernel<T, V, 4, false>, g, b, 0, st, a);
+    default: return (int)sfb_launch(seam_kernel<T, V, 8, false>, g, b, 0, st, a);
   }
 }
 template <typename T, int V>
@@ -690,12 +775,12 @@ int sfb_rows_qk_append(const void* proj, int64_t stride, const void* qw, const v
 
 // summaries: a segment has more than one chunk (two passes; the gates are overwritten); otherwise one pass
 int sfb_rows_scan(const void* gates, const void* rb, const void* ib, const void* decay, const void* u, const void* y, int64_t y_stride, void* out,
-                  void* S, void* sums, const int* chunk_seg, const int* chunk_row0, const int* chunk_rows, const int* chunk_first,
+                  void* S, void* sums, void* tickets, const int* chunk_seg, const int* chunk_row0, const int* chunk_rows, const int* chunk_first,
                   const int* seg_src, const int* seg_dst, const int* seg_row0, const int* seg_len, int chunks, int summaries, int n, int width,
                   int bs, int fp32, cudaStream_t stream) {
   if (n < 1 || chunks < 1 || chunks > 65535) return (int)cudaErrorInvalidValue;
   ScanArgs a{(const float*)gates, (const float*)rb, (const float*)ib, (const float*)decay, u, y, y_stride, out, (float*)S, (float2*)sums,
-             chunk_seg, chunk_row0, chunk_rows, chunk_first, seg_src, seg_dst, seg_row0, seg_len, n, width, bs};
+             chunk_seg, chunk_row0, chunk_rows, chunk_first, seg_src, seg_dst, seg_row0, seg_len, (int*)tickets, n, width, bs, chunks};
   const dim3 g((width + 127) / 128, chunks), b(128);
   if (!summaries)
     return (int)(fp32 ? sfb_launch(scan_short_kernel<float>, g, b, 0, stream, a) : sfb_launch(scan_short_kernel<__nv_bfloat16>, g, b, 0, stream, a));
@@ -712,7 +797,7 @@ int sfb_rows_gated_step(const void* x, int64_t x_stride, const void* y, int64_t 
   const int parts = width / bs, groups = (n + GATED_RB - 1) / GATED_RB;
   // enough blocks to fill the machine without repeating the convolution more than needed
   int tiles = 1;
-  while (tiles < 16 && parts * groups * tiles < 296 && bs / (tiles * 2) >= 8) tiles *= 2;
+  while (tiles < 16 && parts * groups * tiles < 148 && bs / (tiles * 2) >= 8) tiles *= 2;
   GatedRowArgs a{x, y, x_stride, y_stride, (const float*)cw, (const float*)cb, hist, wg, (const float*)rb, (const float*)ib, (const float*)decay,
                  (float*)S, out, src, dst, n, width, bs, taps, tiles, (bs + tiles - 1) / tiles};
   const size_t smem = (size_t)GATED_RB * ((bs + 7) & ~7) * sizeof(float);

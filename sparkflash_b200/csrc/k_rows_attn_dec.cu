@@ -326,19 +326,45 @@ __global__ void __launch_bounds__(128) attn_stream_merge_kernel(Args a) {
   if (c0 == c1) return;
   const int h0 = (u / a.hgroups) * rep + (u % a.hgroups) * R, nh = min(R, rep - (u % a.hgroups) * R);
   const int row = a.rows ? a.rows[r] : r;
-  for (int x = threadIdx.x; x < nh * a.vdim; x += 128) {
-    const int k = x / a.vdim, v = x - k * a.vdim;
-    float m = -INFINITY, l = 0.f, o = 0.f;
-#pragma unroll 4
-    for (int c = c0; c <= c1; ++c) m = fmaxf(m, a.ml[((size_t)(2 * c + (start > c * per)) * R + k) * 2]);
-#pragma unroll 4
-    for (int c = c0; c <= c1; ++c) {
-      const size_t s = (size_t)(2 * c + (start > c * per)) * R + k;
+  // weight of every partial: one warp per head, lanes over the partials
+  extern __shared__ float wts[];             // [R][partials]
+  __shared__ float lsum[R];
+  const int parts = c1 - c0 + 1, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int k = warp; k < nh; k += 4) {
+    float m = -INFINITY, l = 0.f;
+    for (int c = lane; c < parts; c += 32) m = fmaxf(m, a.ml[((size_t)(2 * (c0 + c) + (start > (c0 + c) * per)) * R + k) * 2]);
+    m = warp_max(m);
+    for (int c = lane; c < parts; c += 32) {
+      const size_t s = (size_t)(2 * (c0 + c) + (start > (c0 + c) * per)) * R + k;
       const float f = ex2(a.ml[2 * s] - m);
+      wts[k * parts + c] = f;
       l += a.ml[2 * s + 1] * f;
-      o += a.part[s * a.vdim + v] * f;
     }
-    a.out[((size_t)row * a.H + h0 + k) * a.vdim + v] = __float2bfloat16_rn(o / l);
+    l = warp_sum(l);
+    if (lane == 0) lsum[k] = l;
+  }
+  __syncthreads();
+  // a warp takes every fourth partial, a lane four dims of it; the warps' sums meet in shared memory
+  __shared__ float4 red[4][R * 64];
+  const int quads = nh * a.vdim / 4;
+  for (int x = lane; x < quads; x += 32) {
+    const int k = x / (a.vdim / 4), v = (x - k * (a.vdim / 4)) * 4;
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+    for (int c = warp; c < parts; c += 4) {
+      const float4 p = *reinterpret_cast<const float4*>(a.part + ((size_t)(2 * (c0 + c) + (start > (c0 + c) * per)) * R + k) * a.vdim + v);
+      const float w = wts[k * parts + c];
+      o.x += p.x * w; o.y += p.y * w; o.z += p.z * w; o.w += p.w * w;
+    }
+    red[warp][x] = o;
+  }
+  __syncthreads();
+  for (int x = threadIdx.x; x < quads; x += 128) {
+    const int k = x / (a.vdim / 4), v = (x - k * (a.vdim / 4)) * 4;
+    const float inv = 1.f / lsum[k];
+    const float4 p = red[0][x], q = red[1][x], r2 = red[2][x], t = red[3][x];
+    const float f[4] = {(p.x + q.x + r2.x + t.x) * inv, (p.y + q.y + r2.y + t.y) * inv, (p.z + q.z + r2.z + t.z) * inv, (p.w + q.w + r2.w + t.w) * inv};
+    rows::store_v<__nv_bfloat16, 4>(a.out + ((size_t)row * a.H + h0 + k) * a.vdim + v, f);
   }
 }
 
@@ -366,7 +392,7 @@ static int launch(Args a, int max_total, cudaStream_t st) {
   if (pages < (long long)a.ctas * MIN_PAGES) a.ctas = (int)((pages + MIN_PAGES - 1) / MIN_PAGES);
   const int rc = (int)sfb_launch(attn_stream_kernel<KC, NVV, R>, dim3(a.ctas), dim3(THREADS), smem, st, a);
   if (rc) return rc;
-  return (int)sfb_launch(attn_stream_merge_kernel<R>, dim3(a.G * a.hgroups, a.n_rows), dim3(128), 0, st, a);
+  return (int)sfb_launch(attn_stream_merge_kernel<R>, dim3(a.G * a.hgroups, a.n_rows), dim3(128), (size_t)R * a.ctas * sizeof(float), st, a);
 }
 template <int KC, int R>
 static int launch_v(const Args& a, int max_total, cudaStream_t st) {

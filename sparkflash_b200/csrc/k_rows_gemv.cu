@@ -17,27 +17,32 @@ struct Args {
 };
 
 template <int N>
-__global__ void __launch_bounds__(256) gemv_kernel(Args a) {
+__global__ void __launch_bounds__(256, 2) gemv_kernel(Args a) {
   extern __shared__ __align__(16) uint8_t raw[];
-  __shared__ float part[8][2][N];
+  __shared__ float part[2][8][2][N];
   __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(raw);      // [N][K]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int groups = 8 / a.wk, g = warp / a.wk, pk = warp % a.wk;
-  const int o = blockIdx.x * groups + g;
-  const int r0 = a.silu ? o : 2 * o, r1 = a.silu ? o + a.M : 2 * o + 1;
-  const bool v0 = a.silu ? o < a.M : r0 < a.M, v1 = a.silu ? o < a.M : r1 < a.M;
-  const int steps = (a.K + 255) / 256, mine = steps > pk ? (steps - pk + a.wk - 1) / a.wk : 0;
-  const uint4* w0 = reinterpret_cast<const uint4*>(a.w + (size_t)r0 * a.K);
-  const uint4* w1 = reinterpret_cast<const uint4*>(a.w + (size_t)r1 * a.K);
+  const int outs = a.silu ? a.M : (a.M + 1) / 2;                 // pairs of weight rows
+  const int stride = gridDim.x * groups, first = blockIdx.x * groups;
+  const int rounds = first < outs ? (outs - first + stride - 1) / stride : 0;      // the same for every warp of the block
+  const int steps = (a.K + 255) / 256, mine = (steps + a.wk - 1) / a.wk, batches = (mine + U - 1) / U;
   uint4 c0[U], c1[U];
-  auto fetch = [&](int s, uint4& d0, uint4& d1) {
-    const int k = (pk + s * a.wk) * 32 + lane;                    // 16-byte word of the row
-    const bool in = s < mine && k * 8 < a.K;
-    d0 = in && v0 ? ldg_nc(w0 + k) : make_uint4(0u, 0u, 0u, 0u);
-    d1 = in && v1 ? ldg_nc(w1 + k) : make_uint4(0u, 0u, 0u, 0u);
-  };
+  // batch b of the warp's pair in round t (the stream of batches runs on over the rounds)
+  auto fetch = [&](int t, int b) {
+    const int o = first + t * stride + g;
+    const bool v0 = a.silu ? o < a.M : 2 * o < a.M, v1 = a.silu ? o < a.M : 2 * o + 1 < a.M;
+    const uint4* w0 = reinterpret_cast<const uint4*>(a.w + (size_t)(a.silu ? o : 2 * o) * a.K);
+    const uint4* w1 = reinterpret_cast<const uint4*>(a.w + (size_t)(a.silu ? o + a.M : 2 * o + 1) * a.K);
 #pragma unroll
-  for (int i = 0; i < U; ++i) fetch(i, c0[i], c1[i]);
+    for (int i = 0; i < U; ++i) {
+      const int k = (pk + (b * U + i) * a.wk) * 32 + lane;       // 16-byte word of the row
+      const bool in = t < rounds && k * 8 < a.K;
+      c0[i] = in && v0 ? ldg_nc(w0 + k) : make_uint4(0u, 0u, 0u, 0u);
+      c1[i] = in && v1 ? ldg_nc(w1 + k) : make_uint4(0u, 0u, 0u, 0u);
+    }
+  };
+  fetch(0, 0);
   pdl_launch_dependents();
   pdl_wait();
   const int words = a.K / 8;
@@ -49,68 +54,74 @@ __global__ void __launch_bounds__(256) gemv_kernel(Args a) {
   float acc[2][N];
 #pragma unroll
   for (int i = 0; i < N; ++i) acc[0][i] = acc[1][i] = 0.f;
-  for (int s0 = 0; s0 < mine; s0 += U) {
-    uint4 n0[U], n1[U];
+  for (int t = 0; t < rounds; ++t) {
+    for (int b = 0; b < batches; ++b) {
+      uint4 d0[U], d1[U];
 #pragma unroll
-    for (int i = 0; i < U; ++i) fetch(s0 + U + i, n0[i], n1[i]);
+      for (int i = 0; i < U; ++i) { d0[i] = c0[i]; d1[i] = c1[i]; }
+      if (b + 1 < batches) fetch(t, b + 1);
+      else fetch(t + 1, 0);
 #pragma unroll
-    for (int i = 0; i < U; ++i) {
-      const int k = (pk + (s0 + i) * a.wk) * 32 + lane;
-      if (s0 + i >= mine || k * 8 >= a.K) continue;
-      const uint32_t p[4] = {c0[i].x, c0[i].y, c0[i].z, c0[i].w}, q[4] = {c1[i].x, c1[i].y, c1[i].z, c1[i].w};
+      for (int i = 0; i < U; ++i) {
+        const int k = (pk + (b * U + i) * a.wk) * 32 + lane;
+        if (k * 8 >= a.K) continue;
+        const uint32_t p[4] = {d0[i].x, d0[i].y, d0[i].z, d0[i].w}, q[4] = {d1[i].x, d1[i].y, d1[i].z, d1[i].w};
 #pragma unroll
-      for (int r = 0; r < N; ++r) {
-        const uint4 xv = reinterpret_cast<const uint4*>(xs)[r * words + k];
-        const uint32_t xw[4] = {xv.x, xv.y, xv.z, xv.w};
+        for (int r = 0; r < N; ++r) {
+          const uint4 xv = reinterpret_cast<const uint4*>(xs)[r * words + k];
+          const uint32_t xw[4] = {xv.x, xv.y, xv.z, xv.w};
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          const float x0 = __uint_as_float(xw[j] << 16), x1 = __uint_as_float(xw[j] & 0xffff0000u);
-          acc[0][r] = fmaf(__uint_as_float(p[j] << 16), x0, acc[0][r]);
-          acc[0][r] = fmaf(__uint_as_float(p[j] & 0xffff0000u), x1, acc[0][r]);
-          acc[1][r] = fmaf(__uint_as_float(q[j] << 16), x0, acc[1][r]);
-          acc[1][r] = fmaf(__uint_as_float(q[j] & 0xffff0000u), x1, acc[1][r]);
+          for (int j = 0; j < 4; ++j) {
+            const float x0 = __uint_as_float(xw[j] << 16), x1 = __uint_as_float(xw[j] & 0xffff0000u);
+            acc[0][r] = fmaf(__uint_as_float(p[j] << 16), x0, acc[0][r]);
+            acc[0][r] = fmaf(__uint_as_float(p[j] & 0xffff0000u), x1, acc[0][r]);
+            acc[1][r] = fmaf(__uint_as_float(q[j] << 16), x0, acc[1][r]);
+            acc[1][r] = fmaf(__uint_as_float(q[j] & 0xffff0000u), x1, acc[1][r]);
+          }
         }
       }
     }
 #pragma unroll
-    for (int i = 0; i < U; ++i) { c0[i] = n0[i]; c1[i] = n1[i]; }
-  }
-#pragma unroll
-  for (int r = 0; r < N; ++r) {
-    acc[0][r] = warp_sum(acc[0][r]);
-    acc[1][r] = warp_sum(acc[1][r]);
-  }
-  if (a.wk > 1) {
-    if (lane == 0) {
-#pragma unroll
-      for (int r = 0; r < N; ++r) { part[warp][0][r] = acc[0][r]; part[warp][1][r] = acc[1][r]; }
+    for (int r = 0; r < N; ++r) {
+      acc[0][r] = warp_sum(acc[0][r]);
+      acc[1][r] = warp_sum(acc[1][r]);
     }
-    __syncthreads();
-    if (pk == 0) {
-      for (int k = 1; k < a.wk; ++k) {
+    if (a.wk > 1) {
+      if (lane == 0) {
 #pragma unroll
-        for (int r = 0; r < N; ++r) { acc[0][r] += part[warp + k][0][r]; acc[1][r] += part[warp + k][1][r]; }
+        for (int r = 0; r < N; ++r) { part[t & 1][warp][0][r] = acc[0][r]; part[t & 1][warp][1][r] = acc[1][r]; }
+      }
+      __syncthreads();       // the other half of `part` was read before this round's barrier
+      if (pk == 0) {
+        for (int k = 1; k < a.wk; ++k) {
+#pragma unroll
+          for (int r = 0; r < N; ++r) { acc[0][r] += part[t & 1][warp + k][0][r]; acc[1][r] += part[t & 1][warp + k][1][r]; }
+        }
       }
     }
-  }
-  if (pk == 0 && lane < a.n) {
-    float s0 = acc[0][0], s1 = acc[1][0];
+    if (pk == 0 && lane < a.n) {
+      float s0 = acc[0][0], s1 = acc[1][0];
 #pragma unroll
-    for (int r = 1; r < N; ++r)
-      if (lane == r) { s0 = acc[0][r]; s1 = acc[1][r]; }
-    const size_t at = (size_t)lane * a.M;
-    if (a.silu) {
-      if (v0) ((__nv_bfloat16*)a.out)[at + o] = __float2bfloat16_rn(s0 * rows::sigmoid_f(s0) * s1);
-    } else {
-      if (a.bias) { if (v0) s0 += __bfloat162float(a.bias[r0]); if (v1) s1 += __bfloat162float(a.bias[r1]); }
-      if (a.f32) {
-        if (v0) ((float*)a.out)[at + r0] = s0;
-        if (v1) ((float*)a.out)[at + r1] = s1;
+      for (int r = 1; r < N; ++r)
+        if (lane == r) { s0 = acc[0][r]; s1 = acc[1][r]; }
+      const int o = first + t * stride + g;
+      const size_t at = (size_t)lane * a.M;
+      if (a.silu) {
+        if (o < a.M) ((__nv_bfloat16*)a.out)[at + o] = __float2bfloat16_rn(s0 * rows::sigmoid_f(s0) * s1);
       } else {
-        if (v0) ((__nv_bfloat16*)a.out)[at + r0] = __float2bfloat16_rn(s0);
-        if (v1) ((__nv_bfloat16*)a.out)[at + r1] = __float2bfloat16_rn(s1);
+        const int r0 = 2 * o, r1 = r0 + 1;
+        if (a.bias) { if (r0 < a.M) s0 += __bfloat162float(a.bias[r0]); if (r1 < a.M) s1 += __bfloat162float(a.bias[r1]); }
+        if (a.f32) {
+          if (r0 < a.M) ((float*)a.out)[at + r0] = s0;
+          if (r1 < a.M) ((float*)a.out)[at + r1] = s1;
+        } else {
+          if (r0 < a.M) ((__nv_bfloat16*)a.out)[at + r0] = __float2bfloat16_rn(s0);
+          if (r1 < a.M) ((__nv_bfloat16*)a.out)[at + r1] = __float2bfloat16_rn(s1);
+        }
       }
     }
+#pragma unroll
+    for (int r = 0; r < N; ++r) acc[0][r] = acc[1][r] = 0.f;
   }
 }
 
@@ -139,9 +150,9 @@ int sfb_rows_gemv(const void* w, const void* x, const void* bias, void* out, int
   const int N = n <= 1 ? 1 : n <= 2 ? 2 : 4;
   if (n < 1 || n > 4 || M < 1 || K < 8 || K % 8 || (size_t)N * K * 2 > 200 * 1024) return (int)cudaErrorInvalidValue;
   const int pairs = silu ? M : (M + 1) / 2, steps = (K + 255) / 256;
-  int wk = 1;
-  while (wk < 8 && (long long)pairs * wk / 8 < 592 && steps / (wk * 2) >= 2) wk *= 2;
-  const int blocks = (pairs + 8 / wk - 1) / (8 / wk);
+  int wk = 1;              // enough pairs of rows for every SM, at least a batch of K per warp
+  while (wk < 8 && (long long)pairs * wk / 8 < 296 && steps / (wk * 2) >= 2) wk *= 2;
+  const int needed = (pairs + 8 / wk - 1) / (8 / wk), blocks = needed < 296 ? needed : 296;
   Args a{(const __nv_bfloat16*)w, (const __nv_bfloat16*)x, (const __nv_bfloat16*)bias, out, M, K, n, wk, f32, silu};
   return N == 1 ? launch<1>(a, blocks, stream) : N == 2 ? launch<2>(a, blocks, stream) : launch<4>(a, blocks, stream);
 }

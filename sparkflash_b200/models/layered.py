@@ -91,7 +91,7 @@ class LayeredEngine:
         self.state = StateSlots(max_lanes, self.dev)
         self.scratch = Scratch(self.dev)
         self.status = torch.zeros((4,), dtype=torch.int32, device=self.dev)
-        self.chunk_rows = 32 if max_rows <= 2048 else 64
+        self.chunk_rows = 32          # rows of a scan chunk
         self.use_graphs = use_graphs
         model.bind(self)
         self.scratch.reserve("logits", max_lanes * model.vocab, torch.float32)

@@ -118,7 +118,7 @@ def test_gated_recurrence_chunks_and_single_rows(dt, parts, bs, taps):
     decay = c(8 * P.softplus(lam.double()))
     S, hist = torch.full((4, width), 5.0, device="cuda"), torch.full((4, taps - 1, width), 5.0, dtype=dt, device="cuda")
     W, B, RB, IB = c(cw.t()), c(cb), c(rb.reshape(-1)), c(ib.reshape(-1))
-    sums = torch.zeros(64 * 2 * width, device="cuda")
+    sums, tickets = torch.zeros(64 * 2 * width, device="cuda"), torch.zeros(-(-width // 128), dtype=torch.int32, device="cuda")
 
     def many(parts_x, parts_y, seg):
         x, y = c(torch.cat(parts_x), dt), c(torch.cat(parts_y), dt)
@@ -128,7 +128,7 @@ def test_gated_recurrence_chunks_and_single_rows(dt, parts, bs, taps):
         for _ in range(2):          # a repeated launch gives the same result
             with R.exact_matmul():
                 R.block_gates(u, wg, gates)
-            R.scan(gates, RB, IB, decay, u, y, o, S, sums, seg, n, bs)
+            R.scan(gates, RB, IB, decay, u, y, o, S, sums, tickets, seg, n, bs)
         return o.float().cpu()
     # a prompt portion of both lanes (several chunks), then single rows through the fused kernel, then a portion again
     a = [11, 2]
