@@ -75,7 +75,7 @@ __device__ __forceinline__ void row_moments(const float (&x)[NV][V], int c0, int
 // AHEAD (few rows): weights and the convolution's carried inputs are requested before they are needed, the former before the
 // previous kernel has finished; with many rows that only costs registers.
 template <typename T, int V, int NV, bool AHEAD>
-__global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
+__global__ void __launch_bounds__(NV < 8 ? 256 : 512, !AHEAD && NV == 4 ? 4 : 1) seam_kernel(SeamArgs a) {
   __shared__ float sh[2 * 96], sh2[2 * 2 * 32];
   int phase = 0, phase2 = 0;
   const int d = a.d, step = blockDim.x * V, c0 = threadIdx.x * V;
@@ -122,15 +122,12 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
         }
     }
   }
-  float x[NV][V], e[NV][V];
-  const bool want_embed = a.from_embed || a.add_embed;
-  if (want_embed) {
+  float x[NV][V];
+  const T* er = nullptr;
+  if (a.from_embed || a.add_embed) {
     int tok = a.tokens[row];
     if (tok < 0 || tok >= a.vocab) { if (threadIdx.x == 0) status_set(a.status, ST_BOUNDS, 60, tok, a.vocab); tok = 0; }
-    const T* er = (const T*)a.embed + (size_t)tok * d;
-#pragma unroll
-    for (int i = 0; i < NV; ++i)
-      if (c0 + i * step < d) load_v<T, V>(er + c0 + i * step, e[i]);
+    er = (const T*)a.embed + (size_t)tok * d;
   }
   float* xr = a.x + (size_t)row * d;
   if (!a.from_embed) {
@@ -144,25 +141,26 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
     if (a.y2) {
       float s[2] = {0.f, 0.f};
       const T* zr = (const T*)a.y2 + (size_t)row * d;
-      float z[NV][V];
 #pragma unroll
       for (int i = 0; i < NV; ++i)
         if (c0 + i * step < d) {
+          float z[V];
           load_v<T, V>(yr + c0 + i * step, y[i]);
-          load_v<T, V>(zr + c0 + i * step, z[i]);
+          load_v<T, V>(zr + c0 + i * step, z);
 #pragma unroll
-          for (int k = 0; k < V; ++k) { s[0] += y[i][k] * y[i][k]; s[1] += z[i][k] * z[i][k]; }
+          for (int k = 0; k < V; ++k) { s[0] += y[i][k] * y[i][k]; s[1] += z[k] * z[k]; }
         }
       block_sums<2>(s, sh2, phase2);
       const float r0 = 0.5f / sqrtf(s[0] * inv_d + a.eps), r1 = 0.5f / sqrtf(s[1] * inv_d + a.eps);
 #pragma unroll
       for (int i = 0; i < NV; ++i)
         if (c0 + i * step < d) {
-          float w0[V], w1[V];
+          float w0[V], w1[V], z[V];
+          load_v<T, V>(zr + c0 + i * step, z);           // again, out of L1
           load_v<float, V>(a.mw + c0 + i * step, w0);
           load_v<float, V>(a.mw2 + c0 + i * step, w1);
 #pragma unroll
-          for (int k = 0; k < V; ++k) y[i][k] = y[i][k] * r0 * w0[k] + z[i][k] * r1 * w1[k];
+          for (int k = 0; k < V; ++k) y[i][k] = y[i][k] * r0 * w0[k] + z[k] * r1 * w1[k];
         }
     } else {
 #pragma unroll
@@ -176,23 +174,26 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512) seam_kernel(SeamArgs a) {
     for (int i = 0; i < NV; ++i)
       if (c0 + i * step < d) {
         if constexpr (!AHEAD) {
-          load_v<float, V>(a.pw + c0 + i * step, pw[i]);
-          load_v<float, V>(a.pb + c0 + i * step, pb[i]);
-        }
+          float w[V], b[V];
+          load_v<float, V>(a.pw + c0 + i * step, w);
+          load_v<float, V>(a.pb + c0 + i * step, b);
 #pragma unroll
-        for (int k = 0; k < V; ++k) x[i][k] += (y[i][k] - mu) * rs * pw[i][k] + pb[i][k];
+          for (int k = 0; k < V; ++k) x[i][k] += (y[i][k] - mu) * rs * w[k] + b[k];
+        } else {
+#pragma unroll
+          for (int k = 0; k < V; ++k) x[i][k] += (y[i][k] - mu) * rs * pw[i][k] + pb[i][k];
+        }
         if (a.tap) store_v<float, V>(a.tap + (size_t)row * d + c0 + i * step, x[i]);
       }
   }
 #pragma unroll
   for (int i = 0; i < NV; ++i)
     if (c0 + i * step < d) {
-      if (a.from_embed) {
+      if (er) {
+        float e[V];
+        load_v<T, V>(er + c0 + i * step, e);
 #pragma unroll
-        for (int k = 0; k < V; ++k) x[i][k] = e[i][k];
-      } else if (a.add_embed) {
-#pragma unroll
-        for (int k = 0; k < V; ++k) x[i][k] += e[i][k];
+        for (int k = 0; k < V; ++k) x[i][k] = a.from_embed ? e[k] : x[i][k] + e[k];
       }
       if (a.step_vec) {
         float sv[V];
@@ -532,7 +533,7 @@ __global__ void __launch_bounds__(128) scan_gates_kernel(ScanArgs a) {
   if (threadIdx.x == 0) a.tickets[blockIdx.x] = 0;      // for the next launch
   __threadfence();
   if (c >= a.width) return;
-  constexpr int B = 16;
+  constexpr int B = 8;
   float S = 0.f;
   for (int k0 = 0; k0 < a.chunks; k0 += B) {
     float2 t[B];

@@ -1,20 +1,20 @@
 // Softmax attention over the paged cache for long runs of rows, on tcgen05: score = (q . k) * scale - bias[head][distance],
 // causal, bf16 queries / keys / values, 32-bit scores, softmax and accumulators.
 //
-// One CTA: 256 consecutive query rows of one segment (two halves of 128) x one head.  Key tiles of 128 positions (two cache
-// pages) stream through shared memory by TMA: a (page, head) block is contiguous, so a tile of 64 dims is two box copies.
+// One CTA: 256 consecutive query rows of one segment (two halves of 128) x one head.  Key tiles of one cache page (64 positions)
+// stream through shared memory by TMA: a (page, head) block is contiguous, so 64 dims of a tile are one box copy.
 //
 //   warps 0-3, 4-7   softmax of half 0 / half 1: one thread per query row (no exchange between threads)
-//   warp 8           issues the MMAs:   S_w = Q_w K^T  (shared x shared),   O_w += P_w V  (P from tensor memory, V MN-major)
-//   warp 9           TMA: the queries once, key and value tiles in two stages each
-//   warps 10-11      stage the tile's window of the bias row (383 distances, four copies shifted by one element each, so that a
-//                    thread reads its row's values, which step down by one per key, as aligned 16-byte words without bank
+//   warps 8, 10      issue the MMAs of half 0 / half 1:   S = Q K^T (shared x shared),   O += P V (P from tensor memory, V MN-major)
+//   warp 9           TMA: the queries once, key and value tiles through a ring of stages
+//   warp 11          stages the tile's window of the bias row (319 distances, four copies shifted by one element each, so that a
+//                    thread reads its row's values, one distance down per key, as aligned 16-byte words without bank
 //                    conflicts)
 //
-// The halves alternate: while one half's scores are exponentiated the tensor core works for the other.  Tensor memory: S0, S1
-// (128 columns each), O0, O1.  P replaces S in place: the softmax weights stay 32-bit up to the product, which takes them as two
-// bf16 terms (hi in columns 0..63, lo = the remainder in 64..127), so P V sees about 16 mantissa bits.  The output accumulator is
-// rescaled only when a row's maximum grew by more than 2^8.
+// Tensor memory: S0, S1 (64 columns each), P0, P1 (64 columns each), O0, O1 (128 each).  S and P are separate, so the next tile's
+// scores are computed while this tile's are exponentiated.  The softmax weights stay 32-bit up to the product, which takes them as
+// two bf16 terms (hi = the upper half of the float in columns 0..31, lo = the remainder in 32..63): P V sees 16 mantissa bits.
+// The output accumulator is rescaled only when a row's maximum grew by more than 2^8.
 //
 // No cluster, no multicast; every wait is bounded and reports through the status word.
 #include <cuda.h>
@@ -24,8 +24,8 @@
 namespace sfb {
 namespace rtc {
 
-constexpr int THREADS = 384, ROWS = 256, HALF = 128, KT = 128, PAGE = 64, SLAB = KT * 128;
-constexpr int BW = 392;                       // bias copy stride: 383 values, = 8 mod 32 banks
+constexpr int THREADS = 384, ROWS = 256, HALF = 128, KT = 64, QSLAB = HALF * 128, SLAB = KT * 128, ST = 4, BST = 4;
+constexpr int BW = 328;                       // bias copy stride: 319 values, = 8 mod 32 banks
 constexpr uint32_t SPIN_LIMIT = 1u << 22;
 constexpr float LOG2E = 1.4426950408889634f;
 
@@ -98,6 +98,20 @@ __device__ __forceinline__ void st16(uint32_t t, const uint32_t* v) {
 }
 __device__ __forceinline__ void wait_ld() { asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory"); }
 __device__ __forceinline__ void wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+// two 32-bit operations in one instruction
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+  float2 d;
+  asm("{\n\t.reg .b64 a, b, c, d;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tmov.b64 c, {%6, %7};\n\tfma.rn.f32x2 d, a, b, c;\n\t"
+      "mov.b64 {%0, %1}, d;\n\t}"
+      : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y), "f"(c.x), "f"(c.y));
+  return d;
+}
+__device__ __forceinline__ float2 add2(float2 a, float2 b) {
+  float2 d;
+  asm("{\n\t.reg .b64 a, b, d;\n\tmov.b64 a, {%2, %3};\n\tmov.b64 b, {%4, %5};\n\tadd.rn.f32x2 d, a, b;\n\tmov.b64 {%0, %1}, d;\n\t}"
+      : "=f"(d.x), "=f"(d.y) : "f"(a.x), "f"(a.y), "f"(b.x), "f"(b.y));
+  return d;
+}
 __device__ __forceinline__ float ex2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -128,11 +142,11 @@ struct Args {
 
 template <int DS, int VS>    // 64-element slabs of a query / key row and of a value row
 struct Smem {
-  alignas(1024) uint8_t q[2 * DS * SLAB];
-  alignas(1024) uint8_t k[2 * DS * SLAB];
-  alignas(1024) uint8_t v[2 * VS * SLAB];
-  alignas(16) float bias[2 * 4 * BW];
-  alignas(8) uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], p_full[2], pv_done[2], b_full[2], b_empty[2];
+  alignas(1024) uint8_t q[2 * DS * QSLAB];
+  alignas(1024) uint8_t k[ST * DS * SLAB];
+  alignas(1024) uint8_t v[ST * VS * SLAB];
+  alignas(16) float bias[BST * 4 * BW];
+  alignas(8) uint64_t q_full, k_full[ST], k_empty[ST], v_full[ST], v_empty[ST], s_full[2], s_free[2], p_full[2], pv_done[2], b_full[BST], b_empty[BST];
   uint32_t tmem;
   int dead;
 };
@@ -147,11 +161,11 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
   if (tid == 0) {
     S.dead = 0;
     mbar_init(&S.q_full, 1);
+    for (int i = 0; i < ST; ++i) { mbar_init(&S.k_full[i], 1); mbar_init(&S.k_empty[i], 2); mbar_init(&S.v_full[i], 1); mbar_init(&S.v_empty[i], 2); }
     for (int i = 0; i < 2; ++i) {
-      mbar_init(&S.k_full[i], 1); mbar_init(&S.k_empty[i], 1); mbar_init(&S.v_full[i], 1); mbar_init(&S.v_empty[i], 1);
-      mbar_init(&S.s_full[i], 1); mbar_init(&S.p_full[i], HALF); mbar_init(&S.pv_done[i], 1);
-      mbar_init(&S.b_full[i], 64); mbar_init(&S.b_empty[i], ROWS);
+      mbar_init(&S.s_full[i], 1); mbar_init(&S.s_free[i], HALF); mbar_init(&S.p_full[i], HALF); mbar_init(&S.pv_done[i], 1);
     }
+    for (int i = 0; i < BST; ++i) { mbar_init(&S.b_full[i], 32); mbar_init(&S.b_empty[i], ROWS); }
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
   if (warp == 8) {
@@ -175,104 +189,114 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
 
   if (warp == 9) {
     if (elect_one()) {
-      const int last_page = (pos0 + rows - 1) / PAGE;
-      mbar_expect(&S.q_full, 2 * DS * SLAB);
+      mbar_expect(&S.q_full, 2 * DS * QSLAB);
       for (int w = 0; w < 2; ++w)
-        for (int s = 0; s < DS; ++s) tma2d(S.q + (w * DS + s) * SLAB, &mq, h * a.dim + 64 * s, row0 + w * HALF, &S.q_full);
+        for (int s = 0; s < DS; ++s) tma2d(S.q + (w * DS + s) * QSLAB, &mq, h * a.dim + 64 * s, row0 + w * HALF, &S.q_full);
       int issued = 0;
       for (int j = 0; j < nt; ++j) {
-        const int st = j & 1, ph = (j >> 1) & 1;
-        int y[2];
-        for (int f = 0; f < 2; ++f) {
-          const int p = min(2 * j + f, last_page);        // past the last page: any finite page, its keys are masked
-          int page = tab[p];
-          if (page < 0 || page >= a.n_pages) { status_set(a.status, ST_BOUNDS, 63, page, a.n_pages); page = 0; }
-          y[f] = (page * a.G + g) * PAGE;
-        }
+        const int st = j % ST, ph = (j / ST) & 1;
+        int page = tab[j];
+        if (page < 0 || page >= a.n_pages) { status_set(a.status, ST_BOUNDS, 63, page, a.n_pages); page = 0; }
+        const int y = (page * a.G + g) * KT;
         if (!mbar_wait(&S.k_empty[st], ph ^ 1, dead)) break;
         mbar_expect(&S.k_full[st], DS * SLAB);
-        for (int s = 0; s < DS; ++s)
-          for (int f = 0; f < 2; ++f) tma2d(S.k + (st * DS + s) * SLAB + f * (SLAB / 2), &mk, 64 * s, y[f], &S.k_full[st]);
+        for (int s = 0; s < DS; ++s) tma2d(S.k + (st * DS + s) * SLAB, &mk, 64 * s, y, &S.k_full[st]);
         issued = 2 * j + 1;
         if (!mbar_wait(&S.v_empty[st], ph ^ 1, dead)) break;
         mbar_expect(&S.v_full[st], VS * SLAB);
-        for (int s = 0; s < VS; ++s)
-          for (int f = 0; f < 2; ++f) tma2d(S.v + (st * VS + s) * SLAB + f * (SLAB / 2), &mv, 64 * s, y[f], &S.v_full[st]);
+        for (int s = 0; s < VS; ++s) tma2d(S.v + (st * VS + s) * SLAB, &mv, 64 * s, y, &S.v_full[st]);
         issued = 2 * j + 2;
       }
       if (*dead) {               // nobody may have waited for the copies in flight: do so, with a limit, before the CTA ends
-        for (int c = max(0, issued - 4); c < issued; ++c) {
-          uint64_t* b = (c & 1) ? &S.v_full[(c >> 1) & 1] : &S.k_full[(c >> 1) & 1];
-          for (int i = 0; i < 100000 && !mbar_try(b, (c >> 2) & 1); ++i) __nanosleep(64);
+        for (int c = max(0, issued - 2 * ST); c < issued; ++c) {
+          const int j = c >> 1;
+          uint64_t* b = (c & 1) ? &S.v_full[j % ST] : &S.k_full[j % ST];
+          for (int i = 0; i < 100000 && !mbar_try(b, (j / ST) & 1); ++i) __nanosleep(64);
         }
         for (int i = 0; i < 100000 && !mbar_try(&S.q_full, 0); ++i) __nanosleep(64);
       }
     }
-  } else if (warp == 8) {
+  } else if (warp == 8 || warp == 10) {
     if (elect_one()) {
+      const int w = warp == 10, nw = w ? n1 : n0;
       const int ks = (a.dim + 15) / 16, nv = (a.vdim + 15) / 16 * 16;
       const uint32_t id_s = idesc(KT, 0), id_o = idesc(nv, 1);
-      const uint32_t qb = smem_u32(S.q), kb = smem_u32(S.k), vb = smem_u32(S.v);
+      const uint32_t ts = tmem + w * 64, tp = tmem + 128 + w * 64, to = tmem + 256 + w * 128;
+      const uint32_t vb = smem_u32(S.v);
+      const uint64_t dq = desc(smem_u32(S.q) + w * DS * QSLAB, 16), dk = desc(smem_u32(S.k), 16), dv = desc(vb, SLAB);
+      auto scores = [&](int j) {          // descriptors step in units of 16 bytes
+        const uint64_t kd = dk + (uint64_t)((j % ST) * DS * (SLAB >> 4));
+#pragma unroll
+        for (int t = 0; t < DS * 4; ++t)
+          if (t < ks) mma_ss(ts, dq + (t >> 2) * (QSLAB >> 4) + (t & 3) * 2, kd + (t >> 2) * (SLAB >> 4) + (t & 3) * 2, id_s, t ? 1u : 0u);
+        commit(&S.s_full[w]);
+        commit(&S.k_empty[j % ST]);
+      };
       bool ok = mbar_wait(&S.q_full, 0, dead);
-      for (int j = 0; ok && j <= nt; ++j) {
-        const int st = j & 1, ph = (j >> 1) & 1, sp = (j - 1) & 1, pp = ((j - 1) >> 1) & 1;
-        if (j < nt) ok = mbar_wait(&S.k_full[st], ph, dead);
-        if (ok && j > 0) ok = mbar_wait(&S.v_full[sp], pp, dead);
-        for (int w = 0; ok && w < 2; ++w) {
-          const int nw = w ? n1 : n0;
-          const uint32_t ts = tmem + w * 128, to = tmem + 256 + w * 128;
-          if (j > 0 && j - 1 < nw) {
-            ok = mbar_wait(&S.p_full[w], (j - 1) & 1, dead);
-            if (!ok) break;
-            fence_after();
-            for (int t = 0; t < 16; ++t)       // eight k-steps of the hi term, then of the lo term
-              mma_ts(to, ts + t * 8, desc(vb + sp * VS * SLAB + (t & 7) * 2048, SLAB), id_o, (j > 1 || t > 0) ? 1u : 0u);
-            commit(&S.pv_done[w]);
-          }
-          if (j < nw) {
-            // S overwrites P: the products that read it must be done
-            if (j > 0) ok = mbar_wait(&S.pv_done[w], (j - 1) & 1, dead);
-            if (!ok) break;
-            fence_after();
-            for (int t = 0; t < ks; ++t)
-              mma_ss(ts, desc(qb + (w * DS + (t >> 2)) * SLAB + (t & 3) * 32, 16), desc(kb + (st * DS + (t >> 2)) * SLAB + (t & 3) * 32, 16), id_s,
-                     t ? 1u : 0u);
-            commit(&S.s_full[w]);
-          }
+      for (int j = 0; ok && j < nt; ++j) {
+        const int st = j % ST, ph = (j / ST) & 1;
+        if (j == 0 && nw > 0) {
+          if (!(ok = mbar_wait(&S.k_full[0], 0, dead))) break;
+          fence_after();
+          scores(0);
         }
-        if (!ok) break;
-        if (j < nt) commit(&S.k_empty[st]);
-        if (j > 0) commit(&S.v_empty[sp]);
+        if (j + 1 < nw) {                 // the next tile's scores as soon as this tile's have been read
+          ok = mbar_wait(&S.k_full[(j + 1) % ST], ((j + 1) / ST) & 1, dead) && mbar_wait(&S.s_free[w], j & 1, dead);
+          if (!ok) break;
+          fence_after();
+          scores(j + 1);
+        }
+        if (j < nw) {
+          ok = mbar_wait(&S.v_full[st], ph, dead) && mbar_wait(&S.p_full[w], j & 1, dead);
+          if (!ok) break;
+          fence_after();
+          const uint64_t vd = dv + (uint64_t)(st * VS * (SLAB >> 4));
+#pragma unroll
+          for (int t = 0; t < 8; ++t)     // four k-steps of the hi term, then of the lo term
+            mma_ts(to, tp + t * 8, vd + (t & 3) * (2048 >> 4), id_o, (j | t) ? 1u : 0u);
+          commit(&S.pv_done[w]);
+          commit(&S.v_empty[st]);
+        } else {                          // a tile that only the other half uses
+          ok = mbar_wait(&S.k_full[st], ph, dead) && mbar_wait(&S.v_full[st], ph, dead);
+          if (!ok) break;
+          mbar_arrive(&S.k_empty[st]);
+          mbar_arrive(&S.v_empty[st]);
+        }
       }
-      if (ok) mbar_wait(&S.v_empty[(nt - 1) & 1], ((nt - 1) >> 1) & 1, dead);     // no arrival may be under way when the CTA ends
+      // no arrival may be under way when the CTA ends: every stage's last use has been released
+      for (int j = max(0, nt - ST); ok && j < nt; ++j)
+        ok = mbar_wait(&S.k_empty[j % ST], (j / ST) & 1, dead) && mbar_wait(&S.v_empty[j % ST], (j / ST) & 1, dead);
     }
-  } else if (warp >= 10) {
-    const int t = tid - 320;
+  } else if (warp == 11) {
     const float* brow = a.bias ? a.bias + (size_t)h * a.bias_len : nullptr;
     for (int j = 0; j < nt; ++j) {
-      const int st = j & 1, ph = (j >> 1) & 1;
+      const int st = j % BST, ph = (j / BST) & 1;
+      float v[10];                         // requested before the buffer is free
+      const int d0 = pos0 + ROWS - 1 - j * KT;         // the window's entries step down in distance, as a row's keys do
+#pragma unroll
+      for (int i = 0; i < 10; ++i) {
+        const int d = d0 - i * 32 - lane;
+        v[i] = (brow && d >= 0 && d < a.bias_len) ? -brow[d] * LOG2E : 0.f;
+      }
       if (!mbar_wait(&S.b_empty[st], ph ^ 1, dead)) break;
       float* dst = S.bias + st * 4 * BW;
-      const int d0 = pos0 - j * KT - 127;
-      for (int i = t; i < 384; i += 64) {
-        const int d = d0 + i;
-        const float v = (brow && d >= 0 && d < a.bias_len) ? brow[d] * LOG2E : 0.f;
+#pragma unroll
+      for (int i = 0; i < 10; ++i)
 #pragma unroll
         for (int s = 0; s < 4; ++s)
-          if (i >= s) dst[s * BW + i - s] = v;
-      }
+          if (i * 32 + lane >= s) dst[s * BW + i * 32 + lane - s] = v[i];
       mbar_arrive(&S.b_full[st]);
     }
   } else {
     const int w = warp >> 2, r = (warp & 3) * 32 + lane, nw = w ? n1 : n0;
     const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
-    const uint32_t ts = tmem + w * 128 + lanes, to = tmem + 256 + w * 128 + lanes;
-    const int pos = pos0 + w * HALF + r, rr = w * HALF + r, shift = rr & 3;
+    const uint32_t ts = tmem + w * 64 + lanes, tp = tmem + 128 + w * 64 + lanes, to = tmem + 256 + w * 128 + lanes;
+    const int pos = pos0 + w * HALF + r, rr = w * HALF + r, shift = (ROWS - 1 - rr) & 3;
     const float sl2 = a.scale * LOG2E;
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = 0; j < nt; ++j) {
-      const int st = j & 1, ph = (j >> 1) & 1;
+      const int st = j % BST, ph = (j / BST) & 1;
       ok = mbar_wait(&S.b_full[st], ph, dead);
       if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
       if (j >= nw) { mbar_arrive(&S.b_empty[st]); continue; }
@@ -280,16 +304,17 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
       if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
       fence_after();
       float s[KT];
-      ld32(ts, s); ld32(ts + 32, s + 32); ld32(ts + 64, s + 64); ld32(ts + 96, s + 96);
+      ld32(ts, s); ld32(ts + 32, s + 32);
       wait_ld();
-      const float* bp = S.bias + st * 4 * BW + shift * BW + (rr + 124 - shift);
+      fence_before();
+      mbar_arrive(&S.s_free[w]);
+      const float* bp = S.bias + st * 4 * BW + shift * BW + (ROWS - 1 - rr - shift);
 #pragma unroll
       for (int q = 0; q < KT / 4; ++q) {
-        const float4 b = *reinterpret_cast<const float4*>(bp - 4 * q);
-        s[4 * q] = fmaf(s[4 * q], sl2, -b.w);
-        s[4 * q + 1] = fmaf(s[4 * q + 1], sl2, -b.z);
-        s[4 * q + 2] = fmaf(s[4 * q + 2], sl2, -b.y);
-        s[4 * q + 3] = fmaf(s[4 * q + 3], sl2, -b.x);
+        const float4 b = *reinterpret_cast<const float4*>(bp + 4 * q);
+        const float2 x = fma2(make_float2(s[4 * q], s[4 * q + 1]), make_float2(sl2, sl2), make_float2(b.x, b.y));
+        const float2 y = fma2(make_float2(s[4 * q + 2], s[4 * q + 3]), make_float2(sl2, sl2), make_float2(b.z, b.w));
+        s[4 * q] = x.x; s[4 * q + 1] = x.y; s[4 * q + 2] = y.x; s[4 * q + 3] = y.y;
       }
       mbar_arrive(&S.b_empty[st]);
       const int vis = pos - j * KT;                  // keys 0 .. vis of the tile are visible
@@ -303,22 +328,26 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
       float m_new = fmaxf(m, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])));
       if (j > 0 && m_new - m <= 8.f) m_new = m;      // key 0 is visible to every row, so m is finite from the first tile on
       const float corr = ex2(m - m_new);
-      float ls[4] = {0.f, 0.f, 0.f, 0.f};
+      float2 ls[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
+      const float2 mneg = make_float2(-m_new, -m_new);
+      uint32_t hi[KT / 2], lo[KT / 2];
 #pragma unroll
-      for (int q = 0; q < 4; ++q) {
-        uint32_t hi[16], lo[16];
-#pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          const float p0 = ex2(s[q * 32 + 2 * i] - m_new), p1 = ex2(s[q * 32 + 2 * i + 1] - m_new);
-          ls[i & 3] += p0 + p1;
-          const __nv_bfloat162 hb = __floats2bfloat162_rn(p0, p1);
-          hi[i] = *reinterpret_cast<const uint32_t*>(&hb);
-          const __nv_bfloat162 lb = __floats2bfloat162_rn(p0 - __uint_as_float(hi[i] << 16), p1 - __uint_as_float(hi[i] & 0xffff0000u));
-          lo[i] = *reinterpret_cast<const uint32_t*>(&lb);
-        }
-        st16(ts + q * 16, hi);
-        st16(ts + 64 + q * 16, lo);
+      for (int i = 0; i < KT / 2; ++i) {
+        const float2 t = add2(make_float2(s[2 * i], s[2 * i + 1]), mneg);
+        const float p0 = ex2(t.x), p1 = ex2(t.y);
+        ls[i & 1] = add2(ls[i & 1], make_float2(p0, p1));
+        hi[i] = __byte_perm(__float_as_uint(p0), __float_as_uint(p1), 0x7632);      // the upper halves
+        const float2 rest = add2(make_float2(p0, p1), make_float2(__uint_as_float((__float_as_uint(p0) & 0xffff0000u) ^ 0x80000000u),
+                                                                  __uint_as_float((__float_as_uint(p1) & 0xffff0000u) ^ 0x80000000u)));
+        const __nv_bfloat162 lb = __floats2bfloat162_rn(rest.x, rest.y);
+        lo[i] = *reinterpret_cast<const uint32_t*>(&lb);
       }
+      if (j > 0) {                         // P and O are free once the previous tile's product is done
+        ok = mbar_wait(&S.pv_done[w], (j - 1) & 1, dead);
+        if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+        fence_after();
+      }
+      st16(tp, hi); st16(tp + 16, hi + 16); st16(tp + 32, lo); st16(tp + 48, lo + 16);
       if (j > 0 && __any_sync(0xffffffffu, corr != 1.f)) {
         for (int c = 0; c < VS * 64; c += 16) {
           float o[16];
@@ -330,7 +359,7 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
         }
       }
       wait_st();
-      l = l * corr + (ls[0] + ls[1]) + (ls[2] + ls[3]);
+      l = l * corr + (ls[0].x + ls[0].y) + (ls[1].x + ls[1].y);
       m = m_new;
       fence_before();
       mbar_arrive(&S.p_full[w]);
