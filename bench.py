@@ -48,6 +48,23 @@ def reference_arm() -> None:
                                      "no cargo/rustc offline, kernels are sm_121a-only mma.sync forms"}))
 
 
+def design_arm(args) -> None:
+    """--design: one GPU, synthetic token ids, random weights."""
+    import torch
+    from sparkflash_b200.utils import layered_bench as LB
+    torch.cuda.set_device(0)
+    sampler = ClockSampler(0)
+    sampler.start()
+    time.sleep(1.0)
+    sampler.mark()
+    sizes = LB.run(args.design_sizes.split(","), args.steps)
+    first = sizes[args.design_sizes.split(",")[-1]]["throughput"]
+    print(json.dumps({"metric": f"{args.design}: decode tok/s, 16 streams, {args.design_sizes.split(',')[-1]}", "value": first["decode_16"]["tok_s"],
+                      "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": 3, "higher_is_better": True, "dtype": "bf16, 32-bit residual / norms / "
+                      "scores / recurrence", "data": "synthetic token ids, random weights", "l2": "every step streams more than L2 holds",
+                      "clocks": sampler.stop(), "sizes": sizes}))
+
+
 class ClockSampler:
     def __init__(self, gpu_index: int):
         self.proc = None
@@ -493,9 +510,15 @@ def main() -> None:
     ap.add_argument("--prefill-chunk", type=int, default=4096, help="rows per prompt chunk (the reference prefills 4,096-row chunks)")
     ap.add_argument("--no-mtp", action="store_true", help="skip the DSpark draft-path section")
     ap.add_argument("--no-ep", action="store_true", help="skip the expert-parallel section (2+ GPUs)")
+    ap.add_argument("--design", default="", choices=["", "fanodra"], help="benchmark a layered design instead of the headline model: prefill and "
+                    "decode throughput and per-kernel roofline fractions, beside the closest model (one JSON line)")
+    ap.add_argument("--design-sizes", default="w1024,w2048,w4096", help="sizes of --design (sparkflash_b200/utils/layered_bench.py)")
     args = ap.parse_args()
     if args.impl == "reference":
         reference_arm()
+        return
+    if args.design:
+        design_arm(args)
         return
     args.warmup = max(args.warmup, 3)
     args.reps = max(args.reps, 1)

@@ -145,27 +145,121 @@ def work(cfg: FanodraConfig, n: int, ctx: int, head_rows: int, decode: bool) -> 
     return out
 
 
-def kernel_table(name: str, rows: int = 4096, ctx: int = 8192) -> list[dict]:
-    """Roofline fractions per kernel of one prompt portion (the last ``rows`` of ``ctx`` positions), event after every launch."""
+def _fractions(timings: list[list[tuple[str, float]]], wk: dict[str, roofline.ClassWork]) -> list[dict]:
+    """Median over repetitions of every launch name's total, beside its roofline time."""
+    by: dict[str, list[float]] = {}
+    for rep in timings:
+        one: dict[str, float] = {}
+        for nm, us in rep:
+            one[nm] = one.get(nm, 0.0) + us
+        for nm, us in one.items():
+            by.setdefault(nm, []).append(us)
+    pk, out = roofline.peaks(), []
+    for nm, ts in sorted(by.items(), key=lambda kv: -statistics.median(kv[1])):
+        us, k = statistics.median(ts), wk.get(nm)
+        row = {"kernel": nm, "us": round(us, 1)}
+        if k is not None and (k.bytes or k.flops):
+            mem, cmp = k.bytes / pk["hbm_gbs"] * 1e-3, k.flops / pk["bf16_tflops_sustained"] * 1e-6
+            row.update(roofline_us=round(max(mem, cmp), 1), bound="memory" if mem >= cmp else "compute", fraction=round(max(mem, cmp) / us, 3))
+        out.append(row)
+    return out
+
+
+def kernel_table(name: str, rows: int = 4096, ctx: int = 8192, reps: int = 5) -> list[dict]:
+    """Roofline fractions per kernel of one prompt portion (the last ``rows`` of ``ctx`` positions)."""
     eng = engine(name, 1, ctx + 64, rows)
     ids = torch.randint(0, eng.model.vocab, (ctx,), generator=torch.Generator().manual_seed(0)).tolist()
     for a in range(0, ctx - rows, rows):
         eng.step(ids[a:a + rows], [0] * rows, list(range(a, a + rows)), head=False)
-    call = (ids[ctx - rows:], [0] * rows, list(range(ctx - rows, ctx)))
-    best: dict[str, list[float]] = {}
-    for _ in range(5):
+    call, ts = (ids[ctx - rows:], [0] * rows, list(range(ctx - rows, ctx))), []
+    for _ in range(reps + 1):
         eng.state.lanes[0].rows = ctx - rows
-        by: dict[str, list[float]] = {}
-        for nm, us in roofline.timed_step(eng, *call, head="last"):
-            by.setdefault(nm, []).append(us)
-        for nm, ts in by.items():
-            best.setdefault(nm, []).append(sum(ts))
+        ts.append(roofline.timed_step(eng, *call, lead_cycles=60_000_000, head="last"))
     eng.check_status()
-    wk, pk, table = work(eng.cfg, rows, ctx, 1, False), roofline.peaks(), []
-    for nm, ts in sorted(best.items(), key=lambda kv: -min(kv[1])):
-        us, k = min(ts), wk.get(nm, roofline.ClassWork())
-        mem, cmp = k.bytes / pk["hbm_gbs"] * 1e-3, k.flops / pk["bf16_tflops_sustained"] * 1e-6
-        table.append({"kernel": nm, "us": round(us, 1), "roofline_us": round(max(mem, cmp), 1), "bound": "memory" if mem >= cmp else "compute",
-                      "fraction": round(max(mem, cmp) / us, 3)})
+    cfg = eng.cfg
     eng.close()
-    return table
+    return _fractions(ts[1:], work(cfg, rows, ctx, 1, False))
+
+
+def decode_table(name: str, n: int = 16, ctx: int = 8192, reps: int = 5) -> list[dict]:
+    """The same of a decode step of n rows against ``ctx`` cached tokens each."""
+    eng = engine(name, n, ctx + 64, 4096)
+    eng.use_graphs = False
+    ids = torch.randint(0, eng.model.vocab, (ctx,), generator=torch.Generator().manual_seed(0)).tolist()
+    for lane in range(n):
+        for a in range(0, ctx, 4096):
+            b = min(ctx, a + 4096)
+            eng.step(ids[a:b], [lane] * (b - a), list(range(a, b)), head=False)
+    ts = [roofline.timed_step(eng, [5] * n, list(range(n)), [ctx + i] * n, lead_cycles=30_000_000) for i in range(reps + 1)]
+    eng.check_status()
+    cfg = eng.cfg
+    eng.close()
+    wk = work(cfg, n, ctx, n, True)
+    if n <= 4:           # the streaming products take the projections and the head, gate and up fused with their activation
+        wk["rows_gemv"] = roofline.ClassWork(wk["linear"].bytes + wk["head"].bytes, wk["linear"].flops + wk["head"].flops)
+    wk["rows_attn_stream"] = wk["rows_attn"]
+    return _fractions(ts[1:], wk)
+
+
+# ---- the closest model of the package: models/qwen.py ------------------------------------------------------------------
+def closest(name: str, rows: int = 256, lanes: int = 4, steps: int = 3) -> dict:
+    """models/qwen.py at the same width, depth, head sizes and active feed-forward width (one expert plus the shared one): tok/s of
+    its rows step, and its recurrence and convolution kernels alone on ``kernel_rows`` rows beside their rooflines."""
+    from ..models import linear_attn as LA
+    from ..models import qwen as Q
+    w, n, H, G, dim, _, _, _, ff, vocab, _ = SIZES[name]
+    c = Q.HybridConfig(vocab=vocab, d=w, layers=n, heads=H, head_dim=dim, lin_heads=H, dk=dim, dv=dim, experts=1, top_k=1, inter=ff // 2)
+    torch.manual_seed(0)
+    weights = {k: torch.randn_like(v, device="cuda") * v.shape[-1] ** -0.5 for k, v in _meta_weights(c).items()}
+    eng = Q.HybridEngine(c, weights, lanes=lanes, max_context=rows + 64)
+    ids = list(range(rows))
+    out = {}
+    ms = timed(lambda: eng.step(ids, [0] * rows, ids), 1, warm=1)
+    out["prefill"] = {"tok_s": rows / ms * 1e3, "rows": rows}
+    for m in (1, lanes):
+        ms = timed(lambda: eng.step([5] * m, list(range(m)), [rows] * m), steps, warm=1)
+        out[f"decode_{m}"] = {"tok_s": m / ms * 1e3, "context": rows}
+    del eng, weights
+    kr, pk = 4096, roofline.peaks()
+    r = lambda *s: torch.randn(*s, device="cuda")
+    st, cv = LA.DeltaState(1, H, dim, dim), LA.ConvState(1, H * 3 * dim, 4)
+    q, k, v, a, b = r(kr, H, dim), torch.nn.functional.normalize(r(kr, H, dim), dim=-1), r(kr, H, dim), torch.rand(kr, H, device="cuda"), torch.rand(kr, H, device="cuda")
+    x, cw = r(kr, H * 3 * dim).bfloat16(), r(H * 3 * dim, 4)
+    for nm, fn, nbytes in (("delta_rule", lambda: st.step(q, k, v, a, b, [0] * kr), kr * H * dim * 16.0), ("short_conv", lambda: cv.step(x, cw, [0] * kr), x.numel() * 4.0)):
+        us, roof = timed(fn, 3, warm=1) * 1e3, nbytes / pk["hbm_gbs"] * 1e-3
+        out[nm] = {"rows": kr, "us": round(us, 1), "roofline_us": round(roof, 1), "fraction": round(roof / us, 4)}
+    qq, kc = r(H, dim), r(8192, H, dim)
+
+    def row_attention():       # what the hybrid's step does per row and full-attention layer
+        s = torch.einsum("hd,shd->hs", qq, kc) * dim ** -0.5
+        return torch.einsum("hs,shd->hd", torch.softmax(s, -1), kc)
+    flush = torch.empty(64 << 20, device="cuda")
+    us, roof = timed(row_attention, 5, flush=flush) * 1e3, 2 * kc.numel() * 4 / pk["hbm_gbs"] * 1e-3
+    out["row_attention"] = {"context": 8192, "us": round(us, 1), "roofline_us": round(roof, 1), "fraction": round(roof / us, 4)}
+    h, wt = r(kr, w), r(ff, w)
+    us, roof = timed(lambda: h @ wt.t(), 5) * 1e3, 2.0 * kr * w * ff / pk["bf16_tflops_sustained"] * 1e-6
+    out["projection_32bit"] = {"rows": kr, "us": round(us, 1), "roofline_us": round(roof, 1), "fraction": round(roof / us, 4)}
+    return out
+
+
+def _meta_weights(c):
+    """Shapes of a hybrid model's weights without filling them on the host."""
+    from ..models import qwen as Q
+    real = torch.randn
+    try:
+        torch.randn = lambda *s, generator=None, **kw: torch.empty(*s, device="meta")
+        with torch.device("meta"):
+            return Q.init_weights(c)
+    finally:
+        torch.randn = real
+
+
+def run(sizes: list[str], steps: int, compare: bool = True) -> dict:
+    out = {}
+    for name in sizes:
+        out[name] = {"throughput": throughput(name, steps=steps), "prefill_kernels": kernel_table(name), "decode16_kernels": decode_table(name, 16),
+                     "decode1_kernels": decode_table(name, 1)}
+        if compare:
+            out[name]["closest_model"] = closest(name)
+        torch.cuda.empty_cache()
+    return out

@@ -70,13 +70,17 @@ class _TimedLog(segments.LaunchLog):
         self.events.append(e)
 
 
-def timed_step(engine, tokens, lanes, positions, **kw) -> list[tuple[str, float]]:
-    """One eager step (the engine must have been built with ``use_graphs=False``) with an event after every launch."""
+def timed_step(engine, tokens, lanes, positions, lead_cycles: int = 0, **kw) -> list[tuple[str, float]]:
+    """One eager step (the engine must have been built with ``use_graphs=False``) with an event after every launch.
+    ``lead_cycles``: keep the GPU busy that long first, so that the host queues the whole step ahead of it and the times hold no
+    gaps between launches."""
     start = torch.cuda.Event(enable_timing=True)
     log = _TimedLog()
     prev = segments.install(log)
     try:
         torch.cuda.synchronize()
+        if lead_cycles:
+            torch.cuda._sleep(lead_cycles)
         start.record()
         engine.step(tokens, lanes, positions, **kw)
         torch.cuda.synchronize()
