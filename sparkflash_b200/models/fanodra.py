@@ -13,6 +13,7 @@ from __future__ import annotations
 
 import json
 import os
+import warnings
 from dataclasses import dataclass, field
 
 import torch
@@ -194,7 +195,7 @@ class Fanodra:
                 raise ValueError(f"{name}: shape {tuple(tensors[name].shape)}, expected {shape}")
         extra = set(tensors) - set(cfg.shapes())
         if extra:
-            raise ValueError(f"checkpoint has tensors the configuration does not: {sorted(extra)[:4]}")
+            warnings.warn(f"checkpoint tensors that the configuration does not use: {sorted(extra)[:4]}")
         self.cfg, self.vocab, self.width, self.dtype, self.device = cfg, cfg.vocab, cfg.width, dtype, device
         self.layers = [_Layer(tensors, i, spec, cfg, dtype, device, max_context) for i, spec in enumerate(cfg.layers)]
         top = W(tensors, "", dtype, device)

@@ -78,7 +78,7 @@ class LayeredEngine:
     def __init__(self, model, max_lanes: int = 4, max_context: int = 4096, max_rows: int = 1024, pool_tokens: int | None = None,
                  use_graphs: bool = True):
         """``pool_tokens``: tokens all lanes together may hold (each lane rounded up to pages); by default every lane can be full."""
-        self.model, self.cfg = model, model.cfg
+        self.model, self.cfg, self.vocab = model, model.cfg, model.vocab
         self.dev = torch.device(model.device)
         if self.dev.type == "cuda" and self.dev.index is None:       # the serving thread selects it by number
             self.dev = torch.device("cuda", torch.cuda.current_device())

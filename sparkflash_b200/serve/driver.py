@@ -189,6 +189,9 @@ class DeviceDriver(InferenceEngine):
 
     def validate(self, req: EngineRequest) -> None:
         super().validate(req)
+        vocab = getattr(self.engine, "vocab", None)
+        if vocab is not None and req.prompt_tokens and max(req.prompt_tokens) >= vocab:
+            raise ApiError(400, f"the tokenizer produced token {max(req.prompt_tokens)}, the model has {vocab}", "invalid_request_error", "messages")
         if (req.top_p < 1.0 or req.top_k > 0) and not getattr(self.engine, "supports_filter", False):
             raise ApiError(400, "top_p / top_k need the candidate filter, which this engine build does not have",
                            "unsupported_parameter", "top_p")

@@ -262,3 +262,49 @@ def test_replay_writes_the_wanted_logits(tmp_path):
     for i, want in ((0, A[[0, 63]]), (1, A[[64]]), (2, B[[69, 6]]), (3, A[[89]])):
         assert error(read(i), want) < 2e-4
     assert not (tmp_path / "4.f32").exists()
+
+
+def test_small_engines_and_a_pool_of_one_page():
+    """A portion as large as the whole engine (fewer rows than a query tile), in bf16 through the tensor-core attention."""
+    toks = tokens("once", 64)
+    eng = engine("once", torch.bfloat16, max_lanes=1, max_context=64, max_rows=64)
+    assert error(feed(eng, 0, toks, 0, [40, 24]), expected("once", toks)) < TOL[torch.bfloat16]
+    eng.release_lane(0)
+    assert error(feed(eng, 0, toks, 0, [64]), expected("once", toks)) < TOL[torch.bfloat16]
+    with pytest.raises(ValueError, match="beyond the context"):
+        eng.step([1], [0], [64])
+    with pytest.raises(ValueError, match="vocabulary"):
+        eng.step([128], [0], [0])
+
+
+def test_command_line_and_serving_builders(tmp_path, capsys):
+    import asyncio
+    from sparkflash_b200 import cli
+    from sparkflash_b200.config import Settings
+    from sparkflash_b200.serve import launch
+    from sparkflash_b200.serve.driver import DeviceDriver
+    from sparkflash_b200.serve.engine_api import ApiError, EngineRequest
+    from sparkflash_b200.serve.tokenizer import load_tokenizer
+    from sparkflash_b200.weights.files import write_safetensors
+    (tmp_path / "config.json").write_text(json.dumps(CONFIGS["gen"]))
+    write_safetensors(str(tmp_path / "model.safetensors"), weights("gen"))
+    a, b = list(tokens("gen", 9)), list(tokens("gen", 14, 1))
+    assert cli.main(["generate", "--model", str(tmp_path), "--dtype", "float32", "--max-new", "6", "--max-context", "128", "--max-rows", "64",
+                     "--tokens", ",".join(map(str, a)), "--tokens", ",".join(map(str, b))]) == 0
+    got = [json.loads(x)["tokens"] for x in capsys.readouterr().out.splitlines() if x.startswith("{")]
+    assert got == [greedy("gen", a, 6), greedy("gen", b, 6)]
+    st = Settings()
+    st.engine.max_lanes = 2
+    args = types.SimpleNamespace(model=str(tmp_path), dtype="float32", max_context=128, pool_tokens=256, weights=None, synthetic=None)
+    eng = launch.build_engine(args, st, 0, 1)
+    tok = load_tokenizer(None, eng.cfg.vocab_size)
+    drv = DeviceDriver(eng, tok, model_id="m", eos_id=-1).start()
+    try:
+        with pytest.raises(ApiError):
+            drv.validate(EngineRequest("x", "m", [eng.vocab], max_tokens=4))
+
+        async def ask():
+            return [e[1] async for e in drv.generate(EngineRequest("r", "m", a, max_tokens=6, temperature=0.0)) if e[0] == "token"]
+        assert asyncio.run(ask()) == greedy("gen", a, 6)
+    finally:
+        drv.shutdown(1.0)
