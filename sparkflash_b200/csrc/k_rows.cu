@@ -7,7 +7,7 @@
 //   conv       causal depthwise convolution with carried inputs, optionally added to its input, optionally with a bias.
 //   qk_append  RMS norm over a whole query / key projection, keys and values into the paged cache.
 //   gated scan real-gated linear recurrence S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t with a = exp(-c r softplus(lam)):
-//              two passes over chunks of rows for prompts, one fused kernel (convolution, gates, recurrence,
+//              two passes over chunks of rows for prompts (the chunks' start states in between), one fused kernel (convolution, gates, recurrence,
 //              output gate) for single rows.
 //   silu_mul   silu(gate) * up.
 //
@@ -421,7 +421,6 @@ struct ScanArgs {
   float2* sums;             // [chunks, width] (product of a, end value from a zero start), then (start state, -)
   const int *chunk_seg, *chunk_row0, *chunk_rows, *chunk_first;   // chunk_first: first chunk of the same segment
   const int *seg_src, *seg_dst, *seg_row0, *seg_len;
-  int* tickets;             // one per 128 channels, zero between launches
   int n, width, bs, chunks;
 };
 
@@ -485,8 +484,7 @@ __global__ void __launch_bounds__(128) scan_short_kernel(ScanArgs a) {
   a.S[(size_t)a.seg_dst[seg] * a.width + c] = S;
 }
 
-// Longer segments, pass 1: (a, b) of every step, in place of the gate pre-activations, and every chunk's summary; the last CTA of a
-// column to arrive (a ticket, nobody waits) turns the column's summaries into the chunks' start states and writes the final states.
+// Longer segments, pass 1: (a, b) of every step, in place of the gate pre-activations, and every chunk's summary.
 constexpr int SCAN_T = 8;    // rows whose loads are in flight together
 template <typename T>
 __device__ __forceinline__ void chunk_gates(const ScanArgs& a, int c) {
@@ -520,40 +518,58 @@ __device__ __forceinline__ void chunk_gates(const ScanArgs& a, int c) {
 
 template <typename T>
 __global__ void __launch_bounds__(128) scan_gates_kernel(ScanArgs a) {
-  __shared__ int last;
   pdl_launch_dependents();
   pdl_wait();
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c < a.width) chunk_gates<T>(a, c);
-  __threadfence();
-  __syncthreads();
-  if (threadIdx.x == 0) last = atomicAdd(a.tickets + blockIdx.x, 1) == a.chunks - 1;
-  __syncthreads();
-  if (!last) return;
-  if (threadIdx.x == 0) a.tickets[blockIdx.x] = 0;      // for the next launch
-  __threadfence();
-  if (c >= a.width) return;
-  constexpr int B = 8;
-  float S = 0.f;
-  for (int k0 = 0; k0 < a.chunks; k0 += B) {
-    float2 t[B];
-    int first[B + 1];                      // chunk k + 1 begins a segment: chunk k ends one
+}
+
+// Start state of every chunk and the segments' final states.  A chunk maps its start state S to P S + E; these maps compose, so a
+// column's chunks are shared by START_G threads: each composes its own run of chunks, takes its start from the runs before it,
+// and goes over its run again.
+constexpr int START_G = 16, START_B = 8;
+__global__ void __launch_bounds__(32 * START_G) scan_starts_kernel(ScanArgs a) {
+  __shared__ float mp[START_G][32], me[START_G][32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int x = threadIdx.x, g = threadIdx.y, c = blockIdx.x * 32 + x;
+  const bool on = c < a.width;
+  const int per = (a.chunks + START_G - 1) / START_G, k0 = g * per, k1 = min(k0 + per, a.chunks);
+  float2 t[START_B];
+  float P = 1.f, E = 0.f;
+  for (int pass = 0; pass < 2; ++pass) {
+    float S = 0.f;
+    if (pass) {
+      for (int q = 0; q < g; ++q) S = fmaf(mp[q][x], S, me[q][x]);
+    }
+    for (int kb = k0; kb < k1; kb += START_B) {
+      int seg[START_B + 1];
+      if (pass == 0 || per > START_B) {
 #pragma unroll
-    for (int i = 0; i < B; ++i)
-      if (k0 + i < a.chunks) t[i] = __ldcg(a.sums + (size_t)(k0 + i) * a.width + c);
-#pragma unroll
-    for (int i = 0; i <= B; ++i) first[i] = k0 + i < a.chunks ? a.chunk_first[k0 + i] : k0 + i;
-#pragma unroll
-    for (int i = 0; i < B; ++i) {
-      const int k = k0 + i;
-      if (k >= a.chunks) break;
-      if (first[i] == k) {
-        const int src = a.seg_src[a.chunk_seg[k]];
-        S = src >= 0 ? a.S[(size_t)src * a.width + c] : 0.f;
+        for (int i = 0; i < START_B; ++i)
+          if (on && kb + i < k1) t[i] = a.sums[(size_t)(kb + i) * a.width + c];
       }
-      a.sums[(size_t)k * a.width + c].x = S;
-      S = fmaf(t[i].x, S, t[i].y);
-      if (first[i + 1] == k + 1) a.S[(size_t)a.seg_dst[a.chunk_seg[k]] * a.width + c] = S;
+#pragma unroll
+      for (int i = 0; i <= START_B; ++i) seg[i] = kb + i < a.chunks ? a.chunk_first[kb + i] : kb + i;      // its own index: a segment begins
+#pragma unroll
+      for (int i = 0; i < START_B; ++i) {
+        const int k = kb + i;
+        if (k >= k1 || !on) break;
+        if (seg[i] == k) {
+          const int src = a.seg_src[a.chunk_seg[k]];
+          S = src >= 0 ? a.S[(size_t)src * a.width + c] : 0.f;
+          P = 0.f; E = S;
+        }
+        if (pass) a.sums[(size_t)k * a.width + c].x = S;
+        S = fmaf(t[i].x, S, t[i].y);
+        P *= t[i].x;
+        E = fmaf(t[i].x, E, t[i].y);
+        if (pass && seg[i + 1] == k + 1) a.S[(size_t)a.seg_dst[a.chunk_seg[k]] * a.width + c] = S;
+      }
+    }
+    if (!pass) {
+      mp[g][x] = P; me[g][x] = E;
+      __syncthreads();
     }
   }
 }
@@ -621,7 +637,7 @@ __global__ void __launch_bounds__(256, 2) gated_row_kernel(GatedRowArgs a) {
   const bool pre = V == 8 && j0 < j1 && lane * V < a.bs;
   if (pre) {
     const T* w = (const T*)a.wg + ((size_t)part * 2 * a.bs + j0) * a.bs + lane * V;
-    if constexpr (V == 8) { load8<T>(w, wr0); load8<T>(w + (size_t)a.bs * a.bs, wi0); }
+    if constexpr (V == 8) { load_v<T, 8>(w, wr0); load_v<T, 8>(w + (size_t)a.bs * a.bs, wi0); }
   }
   pdl_launch_dependents();
   pdl_wait();
@@ -656,7 +672,7 @@ __global__ void __launch_bounds__(256, 2) gated_row_kernel(GatedRowArgs a) {
       if (V == 8 && j == j0 && k == lane * V) {
 #pragma unroll
         for (int v = 0; v < V; ++v) { fr[v] = wr0[v]; fi[v] = wi0[v]; }
-      } else if constexpr (V == 8) { load8<T>(wr + k, fr); load8<T>(wi + k, fi); }
+      } else if constexpr (V == 8) { load_v<T, 8>(wr + k, fr); load_v<T, 8>(wi + k, fi); }
       else { load_v<T, 1>(wr + k, fr); load_v<T, 1>(wi + k, fi); }
 #pragma unroll
       for (int i = 0; i < GATED_RB; ++i) {
@@ -693,7 +709,7 @@ __global__ void __launch_bounds__(256) silu_mul_kernel(const T* gu, T* out, int 
   load_v<T, V>(gu + row * 2 * ff + c, g);
   load_v<T, V>(gu + row * 2 * ff + ff + c, u);
 #pragma unroll
-  for (int k = 0; k < V; ++k) g[k] = g[k] * sigmoid_f(g[k]) * u[k];
+  for (int k = 0; k < V; ++k) g[k] = g[k] * gate_sigmoid<T>(g[k]) * u[k];
   store_v<T, V>(out + row * ff + c, g);
 }
 
@@ -768,6 +784,8 @@ int sfb_rows_qk_append(const void* proj, int64_t stride, const void* qw, const v
   QkAppendArgs a{proj, stride, (const float*)qw, (const float*)kw, q, kpool, vpool, table, row_lane, row_pos, max_pages, n_pages, H, G, dim, vdim,
                  eps, (Status*)status};
   const bool v4 = dim % 4 == 0 && vdim % 4 == 0 && stride % 4 == 0;
+  if (!fp32 && dim % 8 == 0 && vdim % 8 == 0 && stride % 8 == 0)
+    return (int)sfb_launch(qk_append_kernel<__nv_bfloat16, 8>, dim3(n), dim3(256), 0, stream, a);
   if (fp32) return (int)(v4 ? sfb_launch(qk_append_kernel<float, 4>, dim3(n), dim3(256), 0, stream, a)
                             : sfb_launch(qk_append_kernel<float, 1>, dim3(n), dim3(256), 0, stream, a));
   return (int)(v4 ? sfb_launch(qk_append_kernel<__nv_bfloat16, 4>, dim3(n), dim3(256), 0, stream, a)
@@ -776,16 +794,18 @@ int sfb_rows_qk_append(const void* proj, int64_t stride, const void* qw, const v
 
 // summaries: a segment has more than one chunk (two passes; the gates are overwritten); otherwise one pass
 int sfb_rows_scan(const void* gates, const void* rb, const void* ib, const void* decay, const void* u, const void* y, int64_t y_stride, void* out,
-                  void* S, void* sums, void* tickets, const int* chunk_seg, const int* chunk_row0, const int* chunk_rows, const int* chunk_first,
+                  void* S, void* sums, const int* chunk_seg, const int* chunk_row0, const int* chunk_rows, const int* chunk_first,
                   const int* seg_src, const int* seg_dst, const int* seg_row0, const int* seg_len, int chunks, int summaries, int n, int width,
                   int bs, int fp32, cudaStream_t stream) {
   if (n < 1 || chunks < 1 || chunks > 65535) return (int)cudaErrorInvalidValue;
   ScanArgs a{(const float*)gates, (const float*)rb, (const float*)ib, (const float*)decay, u, y, y_stride, out, (float*)S, (float2*)sums,
-             chunk_seg, chunk_row0, chunk_rows, chunk_first, seg_src, seg_dst, seg_row0, seg_len, (int*)tickets, n, width, bs, chunks};
+             chunk_seg, chunk_row0, chunk_rows, chunk_first, seg_src, seg_dst, seg_row0, seg_len, n, width, bs, chunks};
   const dim3 g((width + 127) / 128, chunks), b(128);
   if (!summaries)
     return (int)(fp32 ? sfb_launch(scan_short_kernel<float>, g, b, 0, stream, a) : sfb_launch(scan_short_kernel<__nv_bfloat16>, g, b, 0, stream, a));
   cudaError_t rc = fp32 ? sfb_launch(scan_gates_kernel<float>, g, b, 0, stream, a) : sfb_launch(scan_gates_kernel<__nv_bfloat16>, g, b, 0, stream, a);
+  if (rc != cudaSuccess) return (int)rc;
+  rc = sfb_launch(scan_starts_kernel, dim3((width + 31) / 32), dim3(32, START_G), 0, stream, a);
   if (rc != cudaSuccess) return (int)rc;
   rc = fp32 ? sfb_launch(scan_apply_kernel<float>, g, b, 0, stream, a) : sfb_launch(scan_apply_kernel<__nv_bfloat16>, g, b, 0, stream, a);
   return (int)rc;
@@ -812,10 +832,11 @@ int sfb_rows_gated_step(const void* x, int64_t x_stride, const void* y, int64_t 
 
 int sfb_rows_silu_mul(const void* gu, void* out, int n, int ff, int fp32, cudaStream_t stream) {
   if (n < 1 || ff < 1) return (int)cudaErrorInvalidValue;
-  const int V = ff % 4 ? 1 : 4;
+  const int V = ff % 4 ? 1 : (fp32 || ff % 8) ? 4 : 8;
   const dim3 g(n, (ff + 256 * V - 1) / (256 * V)), b(256);
   if (fp32) return (int)(V == 4 ? sfb_launch(silu_mul_kernel<float, 4>, g, b, 0, stream, (const float*)gu, (float*)out, ff)
                                 : sfb_launch(silu_mul_kernel<float, 1>, g, b, 0, stream, (const float*)gu, (float*)out, ff));
+  if (V == 8) return (int)sfb_launch(silu_mul_kernel<__nv_bfloat16, 8>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff);
   return (int)(V == 4 ? sfb_launch(silu_mul_kernel<__nv_bfloat16, 4>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff)
                       : sfb_launch(silu_mul_kernel<__nv_bfloat16, 1>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff));
 }

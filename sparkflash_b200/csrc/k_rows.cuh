@@ -13,10 +13,17 @@ template <typename T> __device__ __forceinline__ T from_f(float v);
 template <> __device__ __forceinline__ float from_f<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
-// V consecutive elements (V = 1 or 4; the address of a group of four is a multiple of its size)
+// V consecutive elements (V = 1, 4 or 8; the address of a group is a multiple of its size, at most 16 bytes)
 template <typename T, int V> __device__ __forceinline__ void load_v(const T* p, float* f) {
   if constexpr (V == 1) {
     f[0] = to_f<T>(*p);
+  } else if constexpr (V == 8 && sizeof(T) == 2) {
+    const uint4 v = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { f[2 * i] = __uint_as_float(w[i] << 16); f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u); }
+  } else if constexpr (V == 8) {
+    load_v<T, 4>(p, f); load_v<T, 4>(p + 4, f + 4);
   } else if constexpr (sizeof(T) == 4) {
     const float4 v = *reinterpret_cast<const float4*>(p);
     f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
@@ -29,6 +36,13 @@ template <typename T, int V> __device__ __forceinline__ void load_v(const T* p, 
 template <typename T, int V> __device__ __forceinline__ void store_v(T* p, const float* f) {
   if constexpr (V == 1) {
     *p = from_f<T>(f[0]);
+  } else if constexpr (V == 8 && sizeof(T) == 2) {
+    uint32_t w[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { const __nv_bfloat162 t = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]); w[i] = *reinterpret_cast<const uint32_t*>(&t); }
+    *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]);
+  } else if constexpr (V == 8) {
+    store_v<T, 4>(p, f); store_v<T, 4>(p + 4, f + 4);
   } else if constexpr (sizeof(T) == 4) {
     *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
   } else {
@@ -36,18 +50,6 @@ template <typename T, int V> __device__ __forceinline__ void store_v(T* p, const
     *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<uint32_t*>(&a), *reinterpret_cast<uint32_t*>(&b));
   }
 }
-// eight consecutive elements, 16-byte aligned groups for bf16, two of them for float
-template <typename T> __device__ __forceinline__ void load8(const T* p, float* f) {
-  if constexpr (sizeof(T) == 4) {
-    load_v<T, 4>(p, f); load_v<T, 4>(p + 4, f + 4);
-  } else {
-    const uint4 v = *reinterpret_cast<const uint4*>(p);
-    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) { f[2 * i] = __uint_as_float(w[i] << 16); f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u); }
-  }
-}
-
 // Block sum of N values at once; one barrier per call: successive calls alternate between the two halves of `sh`
 // ([2][N * 32] floats), and every thread has read a half before it arrives at the next call's barrier.
 template <int N> __device__ __forceinline__ void block_sums(float (&v)[N], float* sh, int& phase) {

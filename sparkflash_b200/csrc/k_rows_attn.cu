@@ -120,7 +120,7 @@ __global__ void __launch_bounds__(ATHREADS) attn_rows_kernel(AttnRowsArgs a) {
       for (int r = 0; r < R; ++r) dot[r] = 0.f;
       for (int c = half * 8; c < dim8; c += 16) {
         float kf[8];
-        load8<T>(kr + c, kf);
+        load_v<T, 8>(kr + c, kf);
 #pragma unroll
         for (int r = 0; r < R; ++r) {
           const float4 q0 = *reinterpret_cast<const float4*>(qs + r * dim8 + c), q1 = *reinterpret_cast<const float4*>(qs + r * dim8 + c + 4);

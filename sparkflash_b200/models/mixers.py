@@ -111,7 +111,6 @@ class GatedRecurrence:
         e.scratch.reserve("rec_u", n * self.width, dt)
         e.scratch.reserve("rec_o", n * self.width, dt)
         e.scratch.reserve("rec_gates", n * 2 * self.width, torch.float32)
-        e.scratch.reserve("rec_tickets", -(-self.width // 128), torch.int32)
         e.scratch.reserve("rec_sums", (-(-n // e.chunk_rows) + e.max_lanes) * 2 * self.width, torch.float32)
 
     def states(self, e, tag: str):
@@ -130,7 +129,7 @@ class GatedRecurrence:
             R.conv(x, self.cw, self.cb, u, hist, s, n, residual=False)
             gates = s.scratch.get("rec_gates", self.parts, n, 2 * self.bs)
             R.block_gates(u, self.wg, gates)
-            R.scan(gates, self.rb, self.ib, self.decay, u, y, o, S, s.scratch.buf["rec_sums"], s.scratch.buf["rec_tickets"], s, n, self.bs)
+            R.scan(gates, self.rb, self.ib, self.decay, u, y, o, S, s.scratch.buf["rec_sums"], s, n, self.bs)
         return R.linear(o, self.wo, None, out)
 
 

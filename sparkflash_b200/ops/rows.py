@@ -55,10 +55,9 @@ def attn(q, kpool, vpool, table, row_lane, row_pos, rows, n_rows, bias, out, par
                                      c_int(vpool.shape[3]), c_int(splits), c_float(scale), _fp32(q), _p(status), _stream()), "rows_attn")
 
 
-def scan(gates, rb, ib, decay, u, y, out, S, sums, tickets, seg, n, bs):
-    """Gated recurrence over the step's chunks; ``gates`` [parts, n, 2 bs] pre-activations (overwritten), y [n, width] view,
-    ``tickets`` [ceil(width / 128)] int32 zeros (left zero)."""
-    _check(_lib.rows().sfb_rows_scan(_p(gates), _p(rb), _p(ib), _p(decay), _p(u), _p(y), c_int64(y.stride(0)), _p(out), _p(S), _p(sums), _p(tickets),
+def scan(gates, rb, ib, decay, u, y, out, S, sums, seg, n, bs):
+    """Gated recurrence over the step's chunks; ``gates`` [parts, n, 2 bs] pre-activations (overwritten), y [n, width] view."""
+    _check(_lib.rows().sfb_rows_scan(_p(gates), _p(rb), _p(ib), _p(decay), _p(u), _p(y), c_int64(y.stride(0)), _p(out), _p(S), _p(sums),
                                      _p(seg.chunk_seg), _p(seg.chunk_row0), _p(seg.chunk_rows), _p(seg.chunk_first), _p(seg.seg_src), _p(seg.seg_dst),
                                      _p(seg.seg_row0), _p(seg.seg_len), c_int(seg.chunks), c_int(seg.summaries), c_int(n), c_int(S.shape[1]), c_int(bs),
                                      _fp32(out), _stream()), "rows_scan")

@@ -118,7 +118,7 @@ def test_gated_recurrence_chunks_and_single_rows(dt, parts, bs, taps):
     decay = c(8 * P.softplus(lam.double()))
     S, hist = torch.full((4, width), 5.0, device="cuda"), torch.full((4, taps - 1, width), 5.0, dtype=dt, device="cuda")
     W, B, RB, IB = c(cw.t()), c(cb), c(rb.reshape(-1)), c(ib.reshape(-1))
-    sums, tickets = torch.zeros(64 * 2 * width, device="cuda"), torch.zeros(-(-width // 128), dtype=torch.int32, device="cuda")
+    sums = torch.zeros(64 * 2 * width, device="cuda")
 
     def many(parts_x, parts_y, seg):
         x, y = c(torch.cat(parts_x), dt), c(torch.cat(parts_y), dt)
@@ -128,7 +128,7 @@ def test_gated_recurrence_chunks_and_single_rows(dt, parts, bs, taps):
         for _ in range(2):          # a repeated launch gives the same result
             with R.exact_matmul():
                 R.block_gates(u, wg, gates)
-            R.scan(gates, RB, IB, decay, u, y, o, S, sums, tickets, seg, n, bs)
+            R.scan(gates, RB, IB, decay, u, y, o, S, sums, seg, n, bs)
         return o.float().cpu()
     # a prompt portion of both lanes (several chunks), then single rows through the fused kernel, then a portion again
     a = [11, 2]
@@ -146,6 +146,33 @@ def test_gated_recurrence_chunks_and_single_rows(dt, parts, bs, taps):
         got[k].append(p)
     for k in range(2):
         assert (torch.cat(got[k]) - want[k]).abs().max() < 2 * _tol(dt)
+
+
+def test_recurrence_over_many_chunks_and_segments():
+    """More chunks than one thread of the start-state kernel takes at once; slow and fast decays; segments of one and of many chunks."""
+    g = torch.Generator().manual_seed(2)
+    lens, width = [1, 700, 4, 37, 300], 40
+    n = sum(lens)
+    seg = _segs(lens, [-1, 3, 4, -1, 8], [0, 2, 5, 6, 9])
+    u, y = torch.randn(n, width, generator=g), torch.randn(n, width, generator=g)
+    z, lam = torch.randn(2, n, width, generator=g), torch.linspace(-9, 1, width)
+    S = torch.randn(10, width, generator=g)
+    want, at = [], 0
+    for k, m in enumerate(lens):
+        r, i = torch.sigmoid(z[0, at:at + m].double()), torch.sigmoid(z[1, at:at + m].double())
+        s0 = S[[-1, 3, 4, -1, 8][k]].double() if k in (1, 2, 4) else None
+        want.append(P.gated_recurrence(u[at:at + m].double(), r, i, lam.double(), s0))
+        at += m
+    Sd, out = S.cuda(), torch.zeros(n, width, device="cuda")
+    gates = torch.cat([z[0], z[1]], -1).view(1, n, 2 * width).cuda()
+    zero = torch.zeros(width, device="cuda")
+    R.scan(gates, zero, zero, (8 * P.softplus(lam.double())).float().cuda(), u.cuda(), y.cuda(), out, Sd, torch.zeros(2 * seg.chunks * width, device="cuda"),
+           seg, n, width)
+    ref = torch.cat(want)
+    assert (out.cpu() - ref.float() * P.gelu_tanh(y)).abs().max() < 2e-4 * ref.abs().max()
+    for k, dst in enumerate((0, 2, 5, 6, 9)):
+        assert (Sd[dst].cpu() - want[k][-1].float()).abs().max() < 2e-4 * ref.abs().max()
+    assert torch.equal(Sd[[1, 3, 4, 7, 8]].cpu(), S[[1, 3, 4, 7, 8]])
 
 
 def _attention_case(dt, H, G, dim, vdim, lens, seed=0, scale=0.2):
