@@ -29,6 +29,8 @@ CONFIGS = {
     "loops": P.make_config(90, 80, 3, [("rglru", P.recurrent(40, 1, 2), 48), ("parallel", P.attending(5, 5, 24, 48, 0.2), P.recurrent(32, 2, 3), 40)],
                            loop=(1, 2, 4)),
 }
+# recurrence only: no attention anywhere; the first layer looped, the same state shapes in every pass
+CONFIGS["rec"] = P.make_config(97, 48, 4, [("rglru", P.recurrent(56, 7, 4), None), ("rglru", P.recurrent(32, 1, 8), 36)], loop=(0, 1, 3))
 CONFIGS["gen"] = CONFIGS["loops"]       # for greedy decoding: no constant directions in the residual, so that the text varies
 TOL = {torch.float32: 2e-4, torch.bfloat16: 0.12}      # rms of the logits' difference over the logits' spread
 
@@ -78,7 +80,7 @@ def feed(eng, lane, toks, at, cuts):
 
 
 @pytest.mark.parametrize("dt", list(TOL))
-@pytest.mark.parametrize("name", ["mid", "odd", "once", "loops"])
+@pytest.mark.parametrize("name", ["mid", "odd", "once", "loops", "rec"])
 def test_whole_prompt_and_layers(name, dt):
     toks = tokens(name, 333)
     eng = engine(name, dt)
@@ -92,7 +94,7 @@ def test_whole_prompt_and_layers(name, dt):
     assert error(feed(eng, 0, toks, 0, [333]), expected(name, toks)) < TOL[dt]
 
 
-@pytest.mark.parametrize("name", ["mid", "odd", "once", "loops"])
+@pytest.mark.parametrize("name", ["mid", "odd", "once", "loops", "rec"])
 def test_portions_and_token_by_token_match_the_whole(name):
     toks = tokens(name, 200)
     want = expected(name, toks)
