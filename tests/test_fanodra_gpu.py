@@ -32,6 +32,7 @@ CONFIGS = {
 # recurrence only: no attention anywhere; the first layer looped, the same state shapes in every pass
 CONFIGS["rec"] = P.make_config(97, 48, 4, [("rglru", P.recurrent(56, 7, 4), None), ("rglru", P.recurrent(32, 1, 8), 36)], loop=(0, 1, 3))
 CONFIGS["gen"] = CONFIGS["loops"]       # for greedy decoding: no constant directions in the residual, so that the text varies
+CONFIGS["far"] = CONFIGS["mid"]         # for far keys: sharp scores and hardly any distance bias
 TOL = {torch.float32: 2e-4, torch.bfloat16: 0.12}      # rms of the logits' difference over the logits' spread
 
 
@@ -43,6 +44,12 @@ def weights(name):
             if k.endswith(".b") and "norm" in k or k.startswith("loop"):
                 w[k] = torch.zeros_like(w[k])
         w["embed"] = w["embed"] * 0.25
+    if name == "far":
+        for k in w:
+            if k.endswith(".q.norm"):
+                w[k] = w[k] * 2
+            if k.endswith(".r1"):
+                w[k] = w[k] * 0.02
     return w
 
 
@@ -106,6 +113,21 @@ def test_portions_and_token_by_token_match_the_whole(name):
             got = feed(eng, lane, toks, 0, cuts)
             assert error(got, ref) < (2e-4 if dt == torch.float32 else 0.08), (dt, cuts[:4], error(got, ref))
             assert error(got, want) < TOL[dt]
+
+
+@pytest.mark.parametrize("dt", list(TOL))
+@pytest.mark.parametrize("n,key", [(300, 0), (300, 1), (300, 63), (300, 64), (257, 128), (321, 255)])
+def test_a_far_token_reaches_prompt_and_decoded_rows(n, key, dt):
+    """One token changed long before the row: the change of the logits is the plain implementation's, in a portion and decoded."""
+    a = list(tokens("far", n))
+    b = list(a)
+    b[key] = (b[key] + 17) % 203
+    eng = engine("far", dt)
+    want = expected("far", tuple(b))[-1] - expected("far", tuple(a))[-1]
+    for cuts in ([n], [n - 40] + [1] * 40, [50, n - 52, 2]):
+        got = feed(eng, 0, b, 0, cuts)[-1] - feed(eng, 1, a, 0, cuts)[-1]
+        rel = ((got - want).pow(2).mean() / want.pow(2).mean()).sqrt().item()
+        assert rel < (0.02 if dt == torch.float32 else 0.6), (cuts[:2], rel, want.pow(2).mean().sqrt())
 
 
 @pytest.mark.parametrize("dt", list(TOL))
