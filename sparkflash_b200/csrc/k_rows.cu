@@ -3,13 +3,15 @@
 //
 //   seam       residual += norm(sublayer output), then the next sublayer's norm, in one pass over a row; options: the output is
 //              half the sum of two branches with an RMS norm each; the row starts from the embedding table; a loop pass adds
-//              the embedding output and a vector; a step of single-row segments also applies the input convolution.
-//   conv       causal depthwise convolution with carried inputs, optionally added to its input, optionally with a bias.
+//              the embedding output and a vector; a step of single-row segments also applies the input convolution; the embedding is
+//              scaled; without a next norm h is the residual at activation precision.
+//   conv       causal depthwise convolution with carried inputs, optionally added to its input or followed by silu, optionally with a
+//              bias.
 //   qk_append  RMS norm over a whole query / key projection, keys and values into the paged cache.
 //   gated scan real-gated linear recurrence S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t with a = exp(-c r softplus(lam)):
 //              two passes over chunks of rows for prompts (the chunks' start states in between), one fused kernel (convolution, gates, recurrence,
 //              output gate) for single rows.
-//   silu_mul   silu(gate) * up.
+//   act_mul    act(gate) * up, act = silu or the tanh form of gelu.
 //
 // Recurrent state (scan state, convolution inputs) has two versions per lane.  A segment reads version `src` (-1: zeros) and
 // writes version `dst`, so every block of a launch sees the state before the step, a replayed graph repeats the same result,
@@ -30,14 +32,14 @@ struct SeamArgs {
   const int* tokens;        // [rows]
   const float* step_vec;    // [d] or null: added after the update
   float* tap;               // [rows, d] or null: the residual right after the update
-  const float *nw, *nb;     // next norm, or null: none
-  void* h;                  // [rows, d] (T) its output
+  const float *nw, *nb;     // next norm, or null: h is the residual itself
+  void* h;                  // [rows, d] (T) its output, or null
   const int* row_map;       // null: row = block; otherwise the residual row of output row `block`
   const float* cw;          // [taps, d] input convolution, or null
   void* hist;               // [slots, taps - 1, d] (T)
   const int *src, *dst;     // [rows] state versions of single-row segments
   int from_embed, add_embed, taps, d, vocab;
-  float eps;
+  float eps, embed_scale;
   Status* status;
 };
 
@@ -193,7 +195,7 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512, !AHEAD && NV == 4 ? 4 : 1)
         float e[V];
         load_v<T, V>(er + c0 + i * step, e);
 #pragma unroll
-        for (int k = 0; k < V; ++k) x[i][k] = a.from_embed ? e[k] : x[i][k] + e[k];
+        for (int k = 0; k < V; ++k) x[i][k] = a.from_embed ? e[k] * a.embed_scale : fmaf(e[k], a.embed_scale, x[i][k]);
       }
       if (a.step_vec) {
         float sv[V];
@@ -202,6 +204,7 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512, !AHEAD && NV == 4 ? 4 : 1)
         for (int k = 0; k < V; ++k) x[i][k] += sv[k];
       }
       store_v<float, V>(xr + c0 + i * step, x[i]);
+      if (!a.nw && a.h) store_v<T, V>((T*)a.h + (size_t)out_row * d + c0 + i * step, x[i]);
     }
   if (!a.nw) return;
   float mu, m2;
@@ -274,7 +277,7 @@ struct ConvRowsArgs {
   void* y;                  // [n, C] (T)
   void* hist;               // [slots, taps - 1, C] (T), oldest first
   const int *row_seg, *seg_row0, *seg_len, *seg_src, *seg_dst;
-  int n, C, residual;       // residual: y = x + conv(x)
+  int n, C, mode;           // 1: y = x + conv(x), 2: y = silu(conv(x))
 };
 constexpr int CONV_RT = 8;  // rows per block: their loads are all in flight before the first product
 
@@ -332,7 +335,7 @@ __global__ void __launch_bounds__(128) conv_rows_kernel(ConvRowsArgs a) {
       float acc = bias[k] + w[W][k] * in[i][k];
 #pragma unroll
       for (int j = 0; j < W; ++j) acc += w[j][k] * win[j][k];
-      o[k] = a.residual ? in[i][k] + acc : acc;
+      o[k] = a.mode == 1 ? in[i][k] + acc : a.mode == 2 ? acc * gate_sigmoid<T>(acc) : acc;
     }
     store_v<T, V>((T*)a.y + (size_t)r * a.C + c, o);
 #pragma unroll
@@ -424,12 +427,6 @@ struct ScanArgs {
   int n, width, bs, chunks;
 };
 
-// exp, reciprocal and square root of the gates, all 32-bit: library-accurate with float activations; with bf16 activations the
-// hardware approximations (relative error below 2^-21), whose error is far below the rounding of u
-template <typename T> __device__ __forceinline__ float gate_sigmoid(float z) {
-  if constexpr (sizeof(T) == 4) return sigmoid_f(z);
-  else return __fdividef(1.f, 1.f + __expf(-z));
-}
 // 1 - exp(t) for t <= 0: a polynomial near 0, where 1 - exp would cancel (Taylor, remainder below 2^-25 of the result)
 __device__ __forceinline__ float one_minus_exp(float t, float e) {
   float p = 1.f / 40320.f;
@@ -450,14 +447,6 @@ template <typename T> __device__ __forceinline__ void gate_step(float zr, float 
     b = r * (gate_sigmoid<T>(zi) * u);
   }
 }
-template <typename T> __device__ __forceinline__ float gate_gelu(float z) {
-  if constexpr (sizeof(T) == 4) return gelu_tanh_f(z);
-  else {   // 0.5 (1 + tanh(k)) = sigmoid(2 k)
-    const float k = 1.5957691216057308f * (z + 0.044715f * z * z * z);
-    return z * gate_sigmoid<T>(k);
-  }
-}
-
 // One chunk per segment: gates, recurrence and output gate in one pass.
 template <typename T>
 __global__ void __launch_bounds__(128) scan_short_kernel(ScanArgs a) {
@@ -697,9 +686,9 @@ __global__ void __launch_bounds__(256, 2) gated_row_kernel(GatedRowArgs a) {
   }
 }
 
-// ---- silu(gate) * up --------------------------------------------------------------------------------------------------------
+// ---- act(gate) * up --------------------------------------------------------------------------------------------------------
 template <typename T, int V>
-__global__ void __launch_bounds__(256) silu_mul_kernel(const T* gu, T* out, int ff) {
+__global__ void __launch_bounds__(256) act_mul_kernel(const T* gu, T* out, int ff, int act) {
   pdl_launch_dependents();
   pdl_wait();
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
@@ -709,7 +698,7 @@ __global__ void __launch_bounds__(256) silu_mul_kernel(const T* gu, T* out, int 
   load_v<T, V>(gu + row * 2 * ff + c, g);
   load_v<T, V>(gu + row * 2 * ff + ff + c, u);
 #pragma unroll
-  for (int k = 0; k < V; ++k) g[k] = g[k] * gate_sigmoid<T>(g[k]) * u[k];
+  for (int k = 0; k < V; ++k) g[k] = (act == ACT_GELU ? gate_gelu<T>(g[k]) : g[k] * gate_sigmoid<T>(g[k])) * u[k];
   store_v<T, V>(out + row * ff + c, g);
 }
 
@@ -758,20 +747,20 @@ extern "C" {
 int sfb_rows_seam(void* x, const void* y, const void* y2, const void* mw, const void* mw2, const void* pw, const void* pb, const void* embed,
                   const int* tokens, const void* step_vec, void* tap, const void* nw, const void* nb, void* h, const int* row_map,
                   const void* cw, void* hist, const int* src, const int* dst, int from_embed, int add_embed, int taps, int n, int d,
-                  int vocab, float eps, int fp32, void* status, cudaStream_t stream) {
+                  int vocab, float eps, float embed_scale, int fp32, void* status, cudaStream_t stream) {
   if (n < 1 || d < 1) return (int)cudaErrorInvalidValue;
   SeamArgs a{(float*)x, y, y2, (const float*)mw, (const float*)mw2, (const float*)pw, (const float*)pb, embed, tokens, (const float*)step_vec,
              (float*)tap, (const float*)nw, (const float*)nb, h, row_map, (const float*)cw, hist, src, dst, from_embed, add_embed, taps, d,
-             vocab, eps, (Status*)status};
+             vocab, eps, embed_scale, (Status*)status};
   if (fp32) return d % 4 ? launch_seam<float, 1>(a, n, stream) : launch_seam<float, 4>(a, n, stream);
   return d % 4 ? launch_seam<__nv_bfloat16, 1>(a, n, stream) : launch_seam<__nv_bfloat16, 4>(a, n, stream);
 }
 
 int sfb_rows_conv(const void* x, int64_t x_stride, const void* w, const void* bias, void* y, void* hist, const int* row_seg, const int* seg_row0,
-                  const int* seg_len, const int* seg_src, const int* seg_dst, int n, int C, int taps, int residual, int fp32,
+                  const int* seg_len, const int* seg_src, const int* seg_dst, int n, int C, int taps, int mode, int fp32,
                   cudaStream_t stream) {
   if (n < 1 || C < 1) return (int)cudaErrorInvalidValue;
-  ConvRowsArgs a{x, x_stride, (const float*)w, (const float*)bias, y, hist, row_seg, seg_row0, seg_len, seg_src, seg_dst, n, C, residual};
+  ConvRowsArgs a{x, x_stride, (const float*)w, (const float*)bias, y, hist, row_seg, seg_row0, seg_len, seg_src, seg_dst, n, C, mode};
   const bool v4 = C % 4 == 0 && x_stride % 4 == 0 && ((uintptr_t)x % (fp32 ? 16 : 8)) == 0;
   if (fp32) return v4 ? launch_conv<float, 4>(a, taps, stream) : launch_conv<float, 1>(a, taps, stream);
   return v4 ? launch_conv<__nv_bfloat16, 4>(a, taps, stream) : launch_conv<__nv_bfloat16, 1>(a, taps, stream);
@@ -830,15 +819,15 @@ int sfb_rows_gated_step(const void* x, int64_t x_stride, const void* y, int64_t 
                   : sfb_launch(gated_row_kernel<__nv_bfloat16, 1>, g, b, smem, stream, a));
 }
 
-int sfb_rows_silu_mul(const void* gu, void* out, int n, int ff, int fp32, cudaStream_t stream) {
+int sfb_rows_act_mul(const void* gu, void* out, int n, int ff, int act, int fp32, cudaStream_t stream) {
   if (n < 1 || ff < 1) return (int)cudaErrorInvalidValue;
   const int V = ff % 4 ? 1 : (fp32 || ff % 8) ? 4 : 8;
   const dim3 g(n, (ff + 256 * V - 1) / (256 * V)), b(256);
-  if (fp32) return (int)(V == 4 ? sfb_launch(silu_mul_kernel<float, 4>, g, b, 0, stream, (const float*)gu, (float*)out, ff)
-                                : sfb_launch(silu_mul_kernel<float, 1>, g, b, 0, stream, (const float*)gu, (float*)out, ff));
-  if (V == 8) return (int)sfb_launch(silu_mul_kernel<__nv_bfloat16, 8>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff);
-  return (int)(V == 4 ? sfb_launch(silu_mul_kernel<__nv_bfloat16, 4>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff)
-                      : sfb_launch(silu_mul_kernel<__nv_bfloat16, 1>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff));
+  if (fp32) return (int)(V == 4 ? sfb_launch(act_mul_kernel<float, 4>, g, b, 0, stream, (const float*)gu, (float*)out, ff, act)
+                                : sfb_launch(act_mul_kernel<float, 1>, g, b, 0, stream, (const float*)gu, (float*)out, ff, act));
+  if (V == 8) return (int)sfb_launch(act_mul_kernel<__nv_bfloat16, 8>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff, act);
+  return (int)(V == 4 ? sfb_launch(act_mul_kernel<__nv_bfloat16, 4>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff, act)
+                      : sfb_launch(act_mul_kernel<__nv_bfloat16, 1>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff, act));
 }
 
 }  // extern "C"

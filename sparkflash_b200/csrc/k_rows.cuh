@@ -76,5 +76,22 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
+
+constexpr int ACT_SILU = 1, ACT_GELU = 2;      // activations of the gated products
+
+// exp, reciprocal and square root of the gates, all 32-bit: library-accurate with float activations; with bf16 activations the
+// hardware approximations (relative error below 2^-21), whose error is far below the rounding of u
+template <typename T> __device__ __forceinline__ float gate_sigmoid(float z) {
+  if constexpr (sizeof(T) == 4) return sigmoid_f(z);
+  else return __fdividef(1.f, 1.f + __expf(-z));
+}
+template <typename T> __device__ __forceinline__ float gate_gelu(float z) {
+  if constexpr (sizeof(T) == 4) return gelu_tanh_f(z);
+  else {   // 0.5 (1 + tanh(k)) = sigmoid(2 k)
+    const float k = 1.5957691216057308f * (z + 0.044715f * z * z * z);
+    return z * gate_sigmoid<T>(k);
+  }
+}
+
 }  // namespace rows
 }  // namespace sfb

@@ -1,7 +1,7 @@
 // Softmax attention over the paged cache for single rows and short runs of rows (k_rows_attn_tc.cu takes long runs), in bf16
-// or true 32-bit, any head sizes: score = (q . k) * scale - bias[head][distance], causal.
+// or true 32-bit, any head sizes: score = (q . k) * scale - bias[head][distance], causal, the last `window` positions.
 //
-// The bias is a table over the distance i - j ([heads, table length], 32-bit), so any distance-only bias is one row of
+// Values may be the first columns of the keys (vpool null): then only key pages are read.  The bias is a table over the distance i - j ([heads, table length], 32-bit), so any distance-only bias is one row of
 // numbers per head; null: none.
 //
 // One block: one row x up to R query heads that share a key/value head x one range of pages.  A page (64 keys) is staged in
@@ -25,6 +25,8 @@ struct AttnRowsArgs {
   float* part;              // [launch rows, H, splits, vdim]
   float* ml;                // [launch rows, H, splits, 2]
   int max_pages, n_pages, H, G, dim, vdim, splits, hgroups, stages;
+  int window;               // keys a row sees: itself and the window - 1 before it
+  int compact;              // q and out hold the launch's rows one after another
   int ldk, ldv;             // shared-memory row strides in elements
   float scale;
   Status* status;
@@ -68,13 +70,14 @@ __global__ void __launch_bounds__(ATHREADS) attn_rows_kernel(AttnRowsArgs a) {
   const int rep = a.H / a.G, h0 = g * rep + hg * R, nh = min(R, rep - hg * R);
   const int row = a.rows ? a.rows[blockIdx.y] : blockIdx.y;
   const int pos = a.row_pos[row], lane_id = a.row_lane[row];
-  const int pages = pos / AP + 1, per = (pages + a.splits - 1) / a.splits;
-  const int p0 = blockIdx.z * per, p1 = min(p0 + per, pages);
+  const int first = max(0, pos - a.window + 1) / AP, pages = pos / AP + 1 - first, per = (pages + a.splits - 1) / a.splits;
+  const int p0 = first + blockIdx.z * per, p1 = min(p0 + per, first + pages);
+  const size_t io = a.compact ? blockIdx.y : row;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int dim8 = (a.dim + 7) & ~7;
   T* kt = reinterpret_cast<T*>(smem);
-  T* vt = kt + (size_t)a.stages * AP * a.ldk;
-  float* qs = reinterpret_cast<float*>(vt + (size_t)a.stages * AP * a.ldv);   // [R][dim8]
+  T* vt = a.vpool ? kt + (size_t)a.stages * AP * a.ldk : kt;
+  float* qs = reinterpret_cast<float*>(kt + (size_t)a.stages * AP * (a.ldk + (a.vpool ? a.ldv : 0)));   // [R][dim8]
   float* ps = qs + R * dim8;                                                  // [R][64]
   float* fac = ps + R * AP;                                                   // [R] rescale of the running output
   float* msum = fac + R;                                                      // [R][2]
@@ -94,13 +97,13 @@ __global__ void __launch_bounds__(ATHREADS) attn_rows_kernel(AttnRowsArgs a) {
     if (page < 0 || page >= a.n_pages) { if (tid == 0) status_set(a.status, ST_BOUNDS, 62, page, a.n_pages); page = 0; }
     const int s = (p - p0) % a.stages;
     stage_page<T>(kt + (size_t)s * AP * a.ldk, (const T*)a.kpool + ((size_t)page * a.G + g) * AP * a.dim, a.dim, a.ldk);
-    stage_page<T>(vt + (size_t)s * AP * a.ldv, (const T*)a.vpool + ((size_t)page * a.G + g) * AP * a.vdim, a.vdim, a.ldv);
+    if (a.vpool) stage_page<T>(vt + (size_t)s * AP * a.ldv, (const T*)a.vpool + ((size_t)page * a.G + g) * AP * a.vdim, a.vdim, a.ldv);
   };
   if (p0 < p1) stage(p0);
   asm volatile("cp.async.commit_group;" ::: "memory");
   for (int i = tid; i < R * dim8; i += ATHREADS) {
     const int r = i / dim8, c = i - r * dim8;
-    qs[i] = (r < nh && c < a.dim) ? to_f<T>(((const T*)a.q)[(size_t)row * a.H * a.dim + (size_t)(h0 + r) * a.dim + c]) * a.scale : 0.f;
+    qs[i] = (r < nh && c < a.dim) ? to_f<T>(((const T*)a.q)[io * a.H * a.dim + (size_t)(h0 + r) * a.dim + c]) * a.scale : 0.f;
   }
   for (int p = p0; p < p1; ++p) {
     if (a.stages > 1) {
@@ -133,7 +136,7 @@ __global__ void __launch_bounds__(ATHREADS) attn_rows_kernel(AttnRowsArgs a) {
         dot[r] += __shfl_xor_sync(0xffffffffu, dot[r], 1);
         if (half == (r & 1) && r < nh) {
           float v = -INFINITY;
-          if (dist >= 0) v = a.bias ? dot[r] - a.bias[(size_t)(h0 + r) * a.bias_len + dist] : dot[r];
+          if (dist >= 0 && dist < a.window) v = a.bias ? dot[r] - a.bias[(size_t)(h0 + r) * a.bias_len + dist] : dot[r];
           ps[r * AP + key] = v;
         }
       }
@@ -144,7 +147,7 @@ __global__ void __launch_bounds__(ATHREADS) attn_rows_kernel(AttnRowsArgs a) {
       const int r = warp + i * 4;
       if (r < nh) {
         const float s0 = ps[r * AP + lane], s1 = ps[r * AP + 32 + lane];
-        const float m_new = fmaxf(m_run[i], warp_max(fmaxf(s0, s1)));      // key 0 of the first page is always visible
+        const float m_new = fmaxf(m_run[i], warp_max(fmaxf(s0, s1)));      // every page of the range holds a visible key
         const float e0 = expf(s0 - m_new), e1 = expf(s1 - m_new);
         const float corr = expf(m_run[i] - m_new);
         ps[r * AP + lane] = e0; ps[r * AP + 32 + lane] = e1;
@@ -199,7 +202,7 @@ __global__ void __launch_bounds__(ATHREADS) attn_rows_kernel(AttnRowsArgs a) {
     const int r = i / a.vdim, v = i - r * a.vdim;
     float t = 0.f;
     for (int k = 0; k < groups; ++k) t += red[((size_t)k * R + r) * cols * 4 + v];
-    if (a.splits == 1) ((T*)a.out)[((size_t)row * a.H + h0 + r) * a.vdim + v] = from_f<T>(t / msum[2 * r + 1]);
+    if (a.splits == 1) ((T*)a.out)[(io * a.H + h0 + r) * a.vdim + v] = from_f<T>(t / msum[2 * r + 1]);
     else a.part[(((size_t)blockIdx.y * a.H + h0 + r) * a.splits + blockIdx.z) * a.vdim + v] = t;
   }
   if (a.splits > 1 && tid < 2 * nh) a.ml[(((size_t)blockIdx.y * a.H + h0 + (tid >> 1)) * a.splits + blockIdx.z) * 2 + (tid & 1)] = msum[tid];
@@ -210,7 +213,7 @@ template <typename T>
 __global__ void __launch_bounds__(128) attn_rows_merge_kernel(AttnRowsArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  const int h = blockIdx.x, row = a.rows ? a.rows[blockIdx.y] : blockIdx.y;
+  const int h = blockIdx.x, row = a.rows && !a.compact ? a.rows[blockIdx.y] : blockIdx.y;
   const float* ml = a.ml + ((size_t)blockIdx.y * a.H + h) * a.splits * 2;
   const float* part = a.part + ((size_t)blockIdx.y * a.H + h) * a.splits * a.vdim;
   float m = -INFINITY, l = 0.f;
@@ -229,15 +232,15 @@ static int launch_attn(AttnRowsArgs a, int n_rows, cudaStream_t st) {
   // rows of shared memory: a whole number of 16-byte units, two more than a multiple of eight, so that the two lanes of
   // four neighbouring keys read eight different bank groups
   auto ld = [&](int w) { const int u = (((w + 7) & ~7) + unit - 1) / unit; return ((u + 7) / 8 * 8 + 2) * unit; };
-  a.ldk = ld(a.dim); a.ldv = ld(a.vdim);
+  a.ldk = ld(a.dim); a.ldv = a.vpool ? ld(a.vdim) : a.ldk;
   const int rep = a.H / a.G, cols = (a.vdim + 3) / 4, groups = ATHREADS / cols;
   a.hgroups = (rep + R - 1) / R;
-  const size_t tile = (size_t)AP * (a.ldk + a.ldv) * sizeof(T);
+  const size_t tile = (size_t)AP * (a.ldk + (a.vpool ? a.ldv : 0)) * sizeof(T);
   const size_t extra = ((size_t)R * ((a.dim + 7) & ~7) + R * AP + 3 * R) * sizeof(float);
   const size_t red = (size_t)groups * R * cols * 4 * sizeof(float);
   a.stages = 2 * tile + extra <= 100 * 1024 ? 2 : 1;
   const size_t smem = a.stages * tile + extra;
-  if (tile < red || smem > 227 * 1024) return (int)cudaErrorInvalidValue;      // the final reduction reuses the tiles
+  if (a.stages * tile < red || smem > 227 * 1024) return (int)cudaErrorInvalidValue;      // the final reduction reuses the tiles
   static size_t granted = 0;
   if (smem > granted) {
     const cudaError_t e = cudaFuncSetAttribute(attn_rows_kernel<T, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -268,12 +271,13 @@ extern "C" {
 
 int sfb_rows_attn(const void* q, const void* kpool, const void* vpool, const int* table, const int* row_lane, const int* row_pos,
                   const int* rows, const void* bias, int64_t bias_len, void* out, void* part, void* ml, int max_pages, int n_pages,
-                  int n_rows, int H, int G, int dim, int vdim, int splits, float scale, int fp32, void* status, cudaStream_t stream) {
-  if (n_rows < 1 || n_rows > 65535 || G < 1 || H % G || vdim > 4 * ATHREADS || dim < 1 || vdim < 1 || splits < 1) return (int)cudaErrorInvalidValue;
+                  int n_rows, int H, int G, int dim, int vdim, int splits, int window, int compact, float scale, int fp32, void* status, cudaStream_t stream) {
+  if (n_rows < 1 || n_rows > 65535 || G < 1 || H % G || vdim > 4 * ATHREADS || dim < 1 || vdim < 1 || splits < 1 || window < 1 || (!vpool && vdim > dim)) return (int)cudaErrorInvalidValue;
   AttnRowsArgs a{};
   a.q = q; a.kpool = kpool; a.vpool = vpool; a.table = table; a.row_lane = row_lane; a.row_pos = row_pos; a.rows = rows;
   a.bias = (const float*)bias; a.bias_len = bias_len; a.out = out; a.part = (float*)part; a.ml = (float*)ml; a.max_pages = max_pages;
   a.n_pages = n_pages; a.H = H; a.G = G; a.dim = dim; a.vdim = vdim; a.splits = splits; a.scale = scale; a.status = (Status*)status;
+  a.window = window; a.compact = compact;
   return fp32 ? launch_attn_r<float>(a, n_rows, stream) : launch_attn_r<__nv_bfloat16>(a, n_rows, stream);
 }
 

@@ -1,5 +1,5 @@
 // Softmax attention over the paged cache for long runs of rows, on tcgen05: score = (q . k) * scale - bias[head][distance],
-// causal, bf16 queries / keys / values, 32-bit scores, softmax and accumulators.
+// causal, the last `window` positions, bf16 queries / keys / values, 32-bit scores, softmax and accumulators.
 //
 // One CTA: 256 consecutive query rows of one segment (two halves of 128) x one head.  Key tiles of one cache page (64 positions)
 // stream through shared memory by TMA: a (page, head) block is contiguous, so 64 dims of a tile are one box copy.
@@ -16,6 +16,10 @@
 // two bf16 terms (hi = the upper half of the float in columns 0..31, lo = the remainder in 32..63): P V sees 16 mantissa bits.
 // The output accumulator is rescaled only when a row's maximum grew by more than 2^8.
 //
+// Keys come from the page pool through the page table, or (`offs`) from rows that were multiplied out for this step: page p of a
+// tile's lane is then page p + offs[tile], heads k_head rows apart.  A key may have a second part that all heads share (template RS:
+// its own map, one 64-element slab), matched by the last columns of the head's query; there is no bias then.
+//
 // No cluster, no multicast; every wait is bounded and reports through the status word.
 #include <cuda.h>
 
@@ -24,7 +28,7 @@
 namespace sfb {
 namespace rtc {
 
-constexpr int THREADS = 384, ROWS = 256, HALF = 128, KT = 64, QSLAB = HALF * 128, SLAB = KT * 128, ST = 4, BST = 4;
+constexpr int THREADS = 384, ROWS = 256, HALF = 128, KT = 64, QSLAB = HALF * 128, SLAB = KT * 128, BST = 4;
 constexpr int BW = 328;                       // bias copy stride: 319 values, = 8 mod 32 banks
 constexpr uint32_t SPIN_LIMIT = 1u << 22;
 constexpr float LOG2E = 1.4426950408889634f;
@@ -132,30 +136,37 @@ struct Args {
   const int* tiles;          // (row0, rows) pairs
   const int* table;
   const int *row_lane, *row_pos;
+  const int* offs;           // page offset of every tile, or null: through the table
   const float* bias;         // [H, bias_len] or null
   int64_t bias_len;
   __nv_bfloat16* out;        // [n, H vdim]
-  int max_pages, n_pages, H, G, dim, vdim;
+  int max_pages, n_pages, H, G, dim, vdim, rot;    // n_pages: of the pool, or of the rows multiplied out
+  int k_page, k_head;        // rows between the pages and between the heads of the keys and values
+  int window;
   float scale;
   Status* status;
 };
 
-template <int DS, int VS>    // 64-element slabs of a query / key row and of a value row
+template <int DS, int VS, int RS>    // 64-element slabs of a query / key row, of a value row, and of the shared key part
 struct Smem {
-  alignas(1024) uint8_t q[2 * DS * QSLAB];
-  alignas(1024) uint8_t k[ST * DS * SLAB];
+  static constexpr int ST = RS ? 3 : 4, QS = DS + RS;
+  alignas(1024) uint8_t q[2 * QS * QSLAB];
+  alignas(1024) uint8_t k[ST * QS * SLAB];
   alignas(1024) uint8_t v[ST * VS * SLAB];
-  alignas(16) float bias[BST * 4 * BW];
+  alignas(16) float bias[RS ? 4 : BST * 4 * BW];
   alignas(8) uint64_t q_full, k_full[ST], k_empty[ST], v_full[ST], v_empty[ST], s_full[2], s_free[2], p_full[2], pv_done[2], b_full[BST], b_empty[BST];
   uint32_t tmem;
   int dead;
 };
 
-template <int DS, int VS>
+template <int DS, int VS, int RS>
 __global__ void __launch_bounds__(THREADS, 1)
-attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv, Args a) {
+attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv,
+                const __grid_constant__ CUtensorMap mr, Args a) {
   extern __shared__ uint8_t raw[];
-  Smem<DS, VS>& S = *reinterpret_cast<Smem<DS, VS>*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
+  using SM = Smem<DS, VS, RS>;
+  constexpr int ST = SM::ST, QS = SM::QS;
+  SM& S = *reinterpret_cast<SM*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   volatile int* dead = &S.dead;
   if (tid == 0) {
@@ -182,25 +193,29 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
   const int row0 = a.tiles[2 * blockIdx.y], rows = a.tiles[2 * blockIdx.y + 1];
   const int pos0 = a.row_pos[row0];
   // key tiles of each half: up to the position of its last row that exists (a half without rows has none)
-  const int n0 = (pos0 + min(rows, HALF) - 1) / KT + 1;
-  const int n1 = rows > HALF ? (pos0 + rows - 1) / KT + 1 : 0;
+  const int j0 = max(0, pos0 - a.window + 1) / KT;           // tiles before the first row's window are not visited
+  const int n0 = (pos0 + min(rows, HALF) - 1) / KT + 1 - j0;
+  const int n1 = rows > HALF ? (pos0 + rows - 1) / KT + 1 - j0 : 0;
   const int nt = max(n0, n1);
-  const int* tab = a.table + (size_t)a.row_lane[row0] * a.max_pages;
+  const int* tab = a.offs ? nullptr : a.table + (size_t)a.row_lane[row0] * a.max_pages + j0;
+  const int off = a.offs ? a.offs[blockIdx.y] + j0 : 0;
 
   if (warp == 9) {
     if (elect_one()) {
-      mbar_expect(&S.q_full, 2 * DS * QSLAB);
+      mbar_expect(&S.q_full, 2 * QS * QSLAB);
       for (int w = 0; w < 2; ++w)
-        for (int s = 0; s < DS; ++s) tma2d(S.q + (w * DS + s) * QSLAB, &mq, h * a.dim + 64 * s, row0 + w * HALF, &S.q_full);
+        for (int s = 0; s < QS; ++s)
+          tma2d(S.q + (w * QS + s) * QSLAB, &mq, h * (a.dim + a.rot) + (s < DS ? 64 * s : a.dim), row0 + w * HALF, &S.q_full);
       int issued = 0;
       for (int j = 0; j < nt; ++j) {
         const int st = j % ST, ph = (j / ST) & 1;
-        int page = tab[j];
+        int page = a.offs ? off + j : tab[j];
         if (page < 0 || page >= a.n_pages) { status_set(a.status, ST_BOUNDS, 63, page, a.n_pages); page = 0; }
-        const int y = (page * a.G + g) * KT;
+        const int y = page * a.k_page + g * a.k_head;
         if (!mbar_wait(&S.k_empty[st], ph ^ 1, dead)) break;
-        mbar_expect(&S.k_full[st], DS * SLAB);
-        for (int s = 0; s < DS; ++s) tma2d(S.k + (st * DS + s) * SLAB, &mk, 64 * s, y, &S.k_full[st]);
+        mbar_expect(&S.k_full[st], QS * SLAB);
+        for (int s = 0; s < DS; ++s) tma2d(S.k + (st * QS + s) * SLAB, &mk, 64 * s, y, &S.k_full[st]);
+        if constexpr (RS > 0) tma2d(S.k + (st * QS + DS) * SLAB, &mr, 0, page * KT, &S.k_full[st]);
         issued = 2 * j + 1;
         if (!mbar_wait(&S.v_empty[st], ph ^ 1, dead)) break;
         mbar_expect(&S.v_full[st], VS * SLAB);
@@ -219,16 +234,16 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
   } else if (warp == 8 || warp == 10) {
     if (elect_one()) {
       const int w = warp == 10, nw = w ? n1 : n0;
-      const int ks = (a.dim + 15) / 16, nv = (a.vdim + 15) / 16 * 16;
+      const int ks = (a.dim + 15) / 16, rs = (a.rot + 15) / 16, nv = (a.vdim + 15) / 16 * 16;
       const uint32_t id_s = idesc(KT, 0), id_o = idesc(nv, 1);
       const uint32_t ts = tmem + w * 64, tp = tmem + 128 + w * 64, to = tmem + 256 + w * 128;
       const uint32_t vb = smem_u32(S.v);
-      const uint64_t dq = desc(smem_u32(S.q) + w * DS * QSLAB, 16), dk = desc(smem_u32(S.k), 16), dv = desc(vb, SLAB);
+      const uint64_t dq = desc(smem_u32(S.q) + w * QS * QSLAB, 16), dk = desc(smem_u32(S.k), 16), dv = desc(vb, SLAB);
       auto scores = [&](int j) {          // descriptors step in units of 16 bytes
-        const uint64_t kd = dk + (uint64_t)((j % ST) * DS * (SLAB >> 4));
+        const uint64_t kd = dk + (uint64_t)((j % ST) * QS * (SLAB >> 4));
 #pragma unroll
-        for (int t = 0; t < DS * 4; ++t)
-          if (t < ks) mma_ss(ts, dq + (t >> 2) * (QSLAB >> 4) + (t & 3) * 2, kd + (t >> 2) * (SLAB >> 4) + (t & 3) * 2, id_s, t ? 1u : 0u);
+        for (int t = 0; t < QS * 4; ++t)
+          if (t < DS * 4 ? t < ks : t - DS * 4 < rs) mma_ss(ts, dq + (t >> 2) * (QSLAB >> 4) + (t & 3) * 2, kd + (t >> 2) * (SLAB >> 4) + (t & 3) * 2, id_s, t ? 1u : 0u);
         commit(&S.s_full[w]);
         commit(&S.k_empty[j % ST]);
       };
@@ -268,6 +283,7 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
         ok = mbar_wait(&S.k_empty[j % ST], (j / ST) & 1, dead) && mbar_wait(&S.v_empty[j % ST], (j / ST) & 1, dead);
     }
   } else if (warp == 11) {
+    if constexpr (RS == 0) {
     const float* brow = a.bias ? a.bias + (size_t)h * a.bias_len : nullptr;
     for (int j = 0; j < nt; ++j) {
       const int st = j % BST, ph = (j / BST) & 1;
@@ -287,6 +303,7 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
           if (i * 32 + lane >= s) dst[s * BW + i * 32 + lane - s] = v[i];
       mbar_arrive(&S.b_full[st]);
     }
+    }
   } else {
     const int w = warp >> 2, r = (warp & 3) * 32 + lane, nw = w ? n1 : n0;
     const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
@@ -297,9 +314,14 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
     bool ok = true;
     for (int j = 0; j < nt; ++j) {
       const int st = j % BST, ph = (j / BST) & 1;
-      ok = mbar_wait(&S.b_full[st], ph, dead);
-      if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
-      if (j >= nw) { mbar_arrive(&S.b_empty[st]); continue; }
+      if constexpr (RS == 0) {
+        ok = mbar_wait(&S.b_full[st], ph, dead);
+        if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
+      }
+      if (j >= nw) {
+        if constexpr (RS == 0) mbar_arrive(&S.b_empty[st]);
+        continue;
+      }
       ok = mbar_wait(&S.s_full[w], j & 1, dead);
       if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
       fence_after();
@@ -308,28 +330,29 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
       wait_ld();
       fence_before();
       mbar_arrive(&S.s_free[w]);
-      const float* bp = S.bias + st * 4 * BW + shift * BW + (ROWS - 1 - rr - shift);
+      const float* bp = S.bias + (RS ? 0 : st * 4 * BW + shift * BW + (ROWS - 1 - rr - shift));
 #pragma unroll
       for (int q = 0; q < KT / 4; ++q) {
-        const float4 b = *reinterpret_cast<const float4*>(bp + 4 * q);
+        const float4 b = RS ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(bp + 4 * q);
         const float2 x = fma2(make_float2(s[4 * q], s[4 * q + 1]), make_float2(sl2, sl2), make_float2(b.x, b.y));
         const float2 y = fma2(make_float2(s[4 * q + 2], s[4 * q + 3]), make_float2(sl2, sl2), make_float2(b.z, b.w));
         s[4 * q] = x.x; s[4 * q + 1] = x.y; s[4 * q + 2] = y.x; s[4 * q + 3] = y.y;
       }
-      mbar_arrive(&S.b_empty[st]);
-      const int vis = pos - j * KT;                  // keys 0 .. vis of the tile are visible
-      if (j * KT + KT - 1 > pos0 + w * HALF) {
+      if constexpr (RS == 0) mbar_arrive(&S.b_empty[st]);
+      const int k0 = (j0 + j) * KT, vis = pos - k0, out = vis - a.window;      // keys out + 1 .. vis of the tile are visible
+      if (k0 + KT - 1 > pos0 + w * HALF || k0 <= pos0 + w * HALF + HALF - 1 - a.window) {
 #pragma unroll
-        for (int c = 0; c < KT; ++c) s[c] = c <= vis ? s[c] : -INFINITY;
+        for (int c = 0; c < KT; ++c) s[c] = c <= vis && c > out ? s[c] : -INFINITY;
       }
       float mx[4] = {s[0], s[1], s[2], s[3]};
 #pragma unroll
       for (int c = 4; c < KT; ++c) mx[c & 3] = fmaxf(mx[c & 3], s[c]);
       float m_new = fmaxf(m, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])));
-      if (j > 0 && m_new - m <= 8.f) m_new = m;      // key 0 is visible to every row, so m is finite from the first tile on
-      const float corr = ex2(m - m_new);
+      if (j > 0 && m_new - m <= 8.f) m_new = m;
+      const float ref = m_new == -INFINITY ? 0.f : m_new;      // no visible key yet
+      const float corr = ex2(m - ref);
       float2 ls[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
-      const float2 mneg = make_float2(-m_new, -m_new);
+      const float2 mneg = make_float2(-ref, -ref);
       uint32_t hi[KT / 2], lo[KT / 2];
 #pragma unroll
       for (int i = 0; i < KT / 2; ++i) {
@@ -398,16 +421,16 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
 typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
                              const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
-template <int DS, int VS>
-static int launch(const CUtensorMap* mq, const CUtensorMap* mk, const CUtensorMap* mv, const Args& a, int n_tiles, cudaStream_t st) {
-  const size_t smem = sizeof(Smem<DS, VS>) + 1024;
+template <int DS, int VS, int RS>
+static int launch(const CUtensorMap* mq, const CUtensorMap* mk, const CUtensorMap* mv, const CUtensorMap* mr, const Args& a, int n_tiles, cudaStream_t st) {
+  const size_t smem = sizeof(Smem<DS, VS, RS>) + 1024;
   static bool done = false;
   if (!done) {
-    const cudaError_t e = cudaFuncSetAttribute(attn_run_kernel<DS, VS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const cudaError_t e = cudaFuncSetAttribute(attn_run_kernel<DS, VS, RS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     done = true;
   }
-  return (int)sfb_launch(attn_run_kernel<DS, VS>, dim3(a.H, n_tiles), dim3(THREADS), smem, st, *mq, *mk, *mv, a);
+  return (int)sfb_launch(attn_run_kernel<DS, VS, RS>, dim3(a.H, n_tiles), dim3(THREADS), smem, st, *mq, *mk, *mv, *mr, a);
 }
 
 }  // namespace rtc
@@ -434,16 +457,24 @@ int sfb_rows_tmap(void* out_map, const void* base, int64_t rows, int64_t cols, i
                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
 }
 
-// mq: queries [rows, H dim], box 128 rows; mk, mv: pools [pages G 64, dim / vdim], box 64 rows.  dim and vdim: multiples of 8 up to 128.
-int sfb_rows_attn_tc(const void* mq, const void* mk, const void* mv, const int* table, const int* row_lane, const int* row_pos, const int* tiles,
-                     int n_tiles, const void* bias, int64_t bias_len, void* out, int max_pages, int n_pages, int H, int G, int dim, int vdim,
-                     float scale, void* status, cudaStream_t stream) {
-  if (n_tiles < 1 || n_tiles > 65535 || G < 1 || H % G || dim % 8 || vdim % 8 || dim < 8 || dim > 128 || vdim < 8 || vdim > 128)
+// mq: queries [rows, H (dim + rot)], box 128 rows; mk, mv: keys and values [rows, dim / vdim], box 64 rows, page p of head g at row
+// p k_page + g k_head (through the page table, or p + offs[tile]); mr: the shared key part [rows, rot] or null.  dim and vdim: multiples
+// of 8 up to 128; rot: a multiple of 8 up to 64.
+int sfb_rows_attn_tc(const void* mq, const void* mk, const void* mv, const void* mr, const int* table, const int* row_lane, const int* row_pos,
+                     const int* tiles, const int* offs, int n_tiles, const void* bias, int64_t bias_len, void* out, int max_pages, int n_pages, int H, int G,
+                     int dim, int vdim, int rot, int k_page, int k_head, int window, float scale, void* status, cudaStream_t stream) {
+  if (n_tiles < 1 || n_tiles > 65535 || G < 1 || H % G || dim % 8 || vdim % 8 || dim < 8 || dim > 128 || vdim < 8 || vdim > 128 || rot % 8 || rot > 64 ||
+      (rot > 0) != (mr != nullptr) || (rot && bias) || window < 1)
     return (int)cudaErrorInvalidValue;
-  Args a{tiles, table, row_lane, row_pos, (const float*)bias, bias_len, (__nv_bfloat16*)out, max_pages, n_pages, H, G, dim, vdim, scale, (Status*)status};
-  const CUtensorMap *q = (const CUtensorMap*)mq, *k = (const CUtensorMap*)mk, *v = (const CUtensorMap*)mv;
-  if (dim <= 64) return vdim <= 64 ? launch<1, 1>(q, k, v, a, n_tiles, stream) : launch<1, 2>(q, k, v, a, n_tiles, stream);
-  return vdim <= 64 ? launch<2, 1>(q, k, v, a, n_tiles, stream) : launch<2, 2>(q, k, v, a, n_tiles, stream);
+  Args a{tiles, table, row_lane, row_pos, offs, (const float*)bias, bias_len, (__nv_bfloat16*)out, max_pages, n_pages, H, G, dim, vdim, rot, k_page, k_head,
+         window, scale, (Status*)status};
+  const CUtensorMap *q = (const CUtensorMap*)mq, *k = (const CUtensorMap*)mk, *v = (const CUtensorMap*)mv, *r = mr ? (const CUtensorMap*)mr : k;
+  if (rot) {
+    if (dim <= 64) return vdim <= 64 ? launch<1, 1, 1>(q, k, v, r, a, n_tiles, stream) : launch<1, 2, 1>(q, k, v, r, a, n_tiles, stream);
+    return vdim <= 64 ? launch<2, 1, 1>(q, k, v, r, a, n_tiles, stream) : launch<2, 2, 1>(q, k, v, r, a, n_tiles, stream);
+  }
+  if (dim <= 64) return vdim <= 64 ? launch<1, 1, 0>(q, k, v, r, a, n_tiles, stream) : launch<1, 2, 0>(q, k, v, r, a, n_tiles, stream);
+  return vdim <= 64 ? launch<2, 1, 0>(q, k, v, r, a, n_tiles, stream) : launch<2, 2, 0>(q, k, v, r, a, n_tiles, stream);
 }
 
 }  // extern "C"

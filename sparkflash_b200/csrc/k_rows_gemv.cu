@@ -1,4 +1,4 @@
-// Matrix products of one to four rows, bf16 weights streamed once: out = x W^T (+ bias), to bf16 or 32-bit, or silu(x Wg^T) * (x Wu^T)
+// Matrix products of one to four rows, bf16 weights streamed once: out = x W^T (+ bias), to bf16 or 32-bit, or act(x Wg^T) * (x Wu^T)
 // with gate and up stacked.  Paced by memory: a warp (or two, four, eight of them, each on a share of K) owns two weight rows, whose first
 // 16-byte words are requested before the previous kernel has finished - weights do not depend on it; x sits in shared memory.
 #include "k_rows.cuh"
@@ -9,11 +9,11 @@ namespace rgemv {
 constexpr int U = 4;          // 256-element steps of K in flight per weight row
 
 struct Args {
-  const __nv_bfloat16* w;     // [M, K] ([2 M, K] with silu: gate rows, then up rows)
+  const __nv_bfloat16* w;     // [M, K] ([2 M, K] with act: gate rows, then up rows)
   const __nv_bfloat16* x;     // [n, K]
   const __nv_bfloat16* bias;  // [M] or null
   void* out;                  // [n, M] bf16 (or float)
-  int M, K, n, wk, f32, silu;
+  int M, K, n, wk, f32, act;
 };
 
 template <int N>
@@ -23,7 +23,7 @@ __global__ void __launch_bounds__(256, 2) gemv_kernel(Args a) {
   __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(raw);      // [N][K]
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int groups = 8 / a.wk, g = warp / a.wk, pk = warp % a.wk;
-  const int outs = a.silu ? a.M : (a.M + 1) / 2;                 // pairs of weight rows
+  const int outs = a.act ? a.M : (a.M + 1) / 2;                 // pairs of weight rows
   const int stride = gridDim.x * groups, first = blockIdx.x * groups;
   const int rounds = first < outs ? (outs - first + stride - 1) / stride : 0;      // the same for every warp of the block
   const int steps = (a.K + 255) / 256, mine = (steps + a.wk - 1) / a.wk, batches = (mine + U - 1) / U;
@@ -31,9 +31,9 @@ __global__ void __launch_bounds__(256, 2) gemv_kernel(Args a) {
   // batch b of the warp's pair in round t (the stream of batches runs on over the rounds)
   auto fetch = [&](int t, int b) {
     const int o = first + t * stride + g;
-    const bool v0 = a.silu ? o < a.M : 2 * o < a.M, v1 = a.silu ? o < a.M : 2 * o + 1 < a.M;
-    const uint4* w0 = reinterpret_cast<const uint4*>(a.w + (size_t)(a.silu ? o : 2 * o) * a.K);
-    const uint4* w1 = reinterpret_cast<const uint4*>(a.w + (size_t)(a.silu ? o + a.M : 2 * o + 1) * a.K);
+    const bool v0 = a.act ? o < a.M : 2 * o < a.M, v1 = a.act ? o < a.M : 2 * o + 1 < a.M;
+    const uint4* w0 = reinterpret_cast<const uint4*>(a.w + (size_t)(a.act ? o : 2 * o) * a.K);
+    const uint4* w1 = reinterpret_cast<const uint4*>(a.w + (size_t)(a.act ? o + a.M : 2 * o + 1) * a.K);
 #pragma unroll
     for (int i = 0; i < U; ++i) {
       const int k = (pk + (b * U + i) * a.wk) * 32 + lane;       // 16-byte word of the row
@@ -106,8 +106,8 @@ __global__ void __launch_bounds__(256, 2) gemv_kernel(Args a) {
         if (lane == r) { s0 = acc[0][r]; s1 = acc[1][r]; }
       const int o = first + t * stride + g;
       const size_t at = (size_t)lane * a.M;
-      if (a.silu) {
-        if (o < a.M) ((__nv_bfloat16*)a.out)[at + o] = __float2bfloat16_rn(s0 * rows::sigmoid_f(s0) * s1);
+      if (a.act) {
+        if (o < a.M) ((__nv_bfloat16*)a.out)[at + o] = __float2bfloat16_rn((a.act == rows::ACT_GELU ? rows::gelu_tanh_f(s0) : s0 * rows::sigmoid_f(s0)) * s1);
       } else {
         const int r0 = 2 * o, r1 = r0 + 1;
         if (a.bias) { if (r0 < a.M) s0 += __bfloat162float(a.bias[r0]); if (r1 < a.M) s1 += __bfloat162float(a.bias[r1]); }
@@ -145,15 +145,15 @@ using namespace sfb::rgemv;
 
 extern "C" {
 
-// n <= 4 rows, K a multiple of 8, n K bounded by shared memory (4 K rows of 200 KB).  silu: w holds 2 M rows, out [n, M].
-int sfb_rows_gemv(const void* w, const void* x, const void* bias, void* out, int n, int M, int K, int f32, int silu, cudaStream_t stream) {
+// n <= 4 rows, K a multiple of 8, n K bounded by shared memory (4 K rows of 200 KB).  act (1 silu, 2 gelu): w holds 2 M rows, out [n, M].
+int sfb_rows_gemv(const void* w, const void* x, const void* bias, void* out, int n, int M, int K, int f32, int act, cudaStream_t stream) {
   const int N = n <= 1 ? 1 : n <= 2 ? 2 : 4;
   if (n < 1 || n > 4 || M < 1 || K < 8 || K % 8 || (size_t)N * K * 2 > 200 * 1024) return (int)cudaErrorInvalidValue;
-  const int pairs = silu ? M : (M + 1) / 2, steps = (K + 255) / 256;
+  const int pairs = act ? M : (M + 1) / 2, steps = (K + 255) / 256;
   int wk = 1;              // enough pairs of rows for every SM, at least a batch of K per warp
   while (wk < 8 && (long long)pairs * wk / 8 < 296 && steps / (wk * 2) >= 2) wk *= 2;
   const int needed = (pairs + 8 / wk - 1) / (8 / wk), blocks = needed < 296 ? needed : 296;
-  Args a{(const __nv_bfloat16*)w, (const __nv_bfloat16*)x, (const __nv_bfloat16*)bias, out, M, K, n, wk, f32, silu};
+  Args a{(const __nv_bfloat16*)w, (const __nv_bfloat16*)x, (const __nv_bfloat16*)bias, out, M, K, n, wk, f32, act};
   return N == 1 ? launch<1>(a, blocks, stream) : N == 2 ? launch<2>(a, blocks, stream) : launch<4>(a, blocks, stream);
 }
 

@@ -1,0 +1,199 @@
+// Row kernels of latent attention (models/mixers.py): keys and values of all heads are products of one cached vector per token, the
+// RMS-normed latent c, beside one rotated key part that the heads share.
+//
+//   latent_append  norm of the latent, rotation of the shared key part (both to the page pool) and of every head's rotated query part
+//                  (in place), pairs (2i, 2i + 1)
+//   head_proj      out[row][h] = x[row][h] W[h] for few rows, W [H, K, M]: the query into the latent space, and the attention output
+//                  out of it
+//   gather_pages   pages of the pool -> consecutive rows (the keys of a prompt portion, before they are multiplied out)
+#include "k_rows.cuh"
+
+namespace sfb {
+namespace rows {
+
+struct LatentArgs {
+  void* proj;               // [n, stride] (T): q [H, dim + rot], then latent [rank], shared key part [rot]
+  int64_t stride;
+  const float* w;           // [rank]
+  const float2* cs;         // [positions, rot / 2] (cos, sin)
+  void* pool;               // [pages, 64, rank + rot] (T)
+  const int* table;
+  const int *row_lane, *row_pos;
+  int max_pages, n_pages, H, dim, rot, rank;
+  float eps;
+  Status* status;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(128) latent_append_kernel(LatentArgs a) {
+  __shared__ float sh[2 * 2 * 32];
+  int phase = 0;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x, pos = a.row_pos[row], qd = a.dim + a.rot, half = a.rot >> 1;
+  T* p = (T*)a.proj + (size_t)row * a.stride;
+  T* c = p + (size_t)a.H * qd;
+  const float2* cs = a.cs + (size_t)pos * half;
+  float s[1] = {0.f};
+  for (int i = threadIdx.x; i < a.rank; i += 128) { const float f = to_f<T>(c[i]); s[0] += f * f; }
+  for (int i = threadIdx.x; i < a.H * half; i += 128) {
+    const int h = i / half, k = i - h * half;
+    T* x = p + (size_t)h * qd + a.dim + 2 * k;
+    const float u = to_f<T>(x[0]), v = to_f<T>(x[1]);
+    const float2 t = cs[k];
+    x[0] = from_f<T>(u * t.x - v * t.y);
+    x[1] = from_f<T>(v * t.x + u * t.y);
+  }
+  block_sums<1>(s, sh, phase);
+  const float r = 1.f / sqrtf(s[0] / (float)a.rank + a.eps);
+  const int page = a.table[(size_t)a.row_lane[row] * a.max_pages + pos / 64];
+  if (page < 0 || page >= a.n_pages) {
+    if (threadIdx.x == 0) status_set(a.status, ST_BOUNDS, 67, page, a.n_pages);
+    return;
+  }
+  T* o = (T*)a.pool + ((size_t)page * 64 + pos % 64) * (a.rank + a.rot);
+  for (int i = threadIdx.x; i < a.rank; i += 128) o[i] = from_f<T>(to_f<T>(c[i]) * r * a.w[i]);
+  for (int k = threadIdx.x; k < half; k += 128) {
+    const float u = to_f<T>(c[a.rank + 2 * k]), v = to_f<T>(c[a.rank + 2 * k + 1]);
+    const float2 t = cs[k];
+    o[a.rank + 2 * k] = from_f<T>(u * t.x - v * t.y);
+    o[a.rank + 2 * k + 1] = from_f<T>(v * t.x + u * t.y);
+  }
+}
+
+struct HeadProjArgs {
+  const void* x;            // (T) x of (row, head): row * x_row + head * x_head elements in
+  int64_t x_row, x_head;
+  const void* w;            // [H, K, M] (T)
+  void* out;                // (T)
+  int64_t out_row, out_head;
+  const int* rows;          // row of x (x_list) or of out (out_list) for every launch row, or null: identity
+  int x_list, out_list, n, K, M, tail;      // tail: elements after x's K that are copied after out's M
+};
+constexpr int HP_M = 128, HP_R = 4, HP_T = 128;      // outputs and rows per block; 16 threads x 8 outputs, 8 shares of K
+
+template <typename T, int V>
+__global__ void __launch_bounds__(HP_T) head_proj_kernel(HeadProjArgs a) {
+  extern __shared__ __align__(16) float sm[];          // x [HP_R][K], then partials [8][HP_R][HP_M]
+  float* xs = sm;
+  float* red = sm + HP_R * a.K;
+  const int tid = threadIdx.x, mg = tid & 15, kg = tid >> 4;
+  const int mt = (a.M + HP_M - 1) / HP_M, h = blockIdx.x / mt, m0 = (blockIdx.x % mt) * HP_M + mg * 8;
+  const int r0 = blockIdx.y * HP_R, nr = min(HP_R, a.n - r0);
+  pdl_launch_dependents();
+  pdl_wait();
+  for (int i = tid; i < HP_R * a.K; i += HP_T) {
+    const int r = i / a.K, k = i - r * a.K;
+    float f = 0.f;
+    if (r < nr) {
+      const int row = a.rows && a.x_list ? a.rows[r0 + r] : r0 + r;
+      f = to_f<T>(((const T*)a.x)[(size_t)row * a.x_row + (size_t)h * a.x_head + k]);
+    }
+    xs[i] = f;
+  }
+  if (a.tail && blockIdx.x % mt == 0) {
+    for (int i = tid; i < nr * a.tail; i += HP_T) {
+      const int r = i / a.tail, k = i - r * a.tail;
+      const int xr = a.rows && a.x_list ? a.rows[r0 + r] : r0 + r, orow = a.rows && a.out_list ? a.rows[r0 + r] : r0 + r;
+      ((T*)a.out)[(size_t)orow * a.out_row + (size_t)h * a.out_head + a.M + k] = ((const T*)a.x)[(size_t)xr * a.x_row + (size_t)h * a.x_head + a.K + k];
+    }
+  }
+  __syncthreads();
+  float acc[HP_R][8];
+#pragma unroll
+  for (int r = 0; r < HP_R; ++r)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) acc[r][j] = 0.f;
+  const T* w = (const T*)a.w + (size_t)h * a.K * a.M + m0;
+  if (m0 < a.M) {
+#pragma unroll 8
+    for (int k = kg; k < a.K; k += 8) {
+      float f[8];
+      if constexpr (V == 8) load_v<T, 8>(w + (size_t)k * a.M, f);
+      else {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) f[j] = m0 + j < a.M ? to_f<T>(w[(size_t)k * a.M + j]) : 0.f;
+      }
+#pragma unroll
+      for (int r = 0; r < HP_R; ++r) {
+        const float xv = xs[r * a.K + k];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) acc[r][j] = fmaf(xv, f[j], acc[r][j]);
+      }
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < HP_R; ++r) {
+    *reinterpret_cast<float4*>(red + ((size_t)kg * HP_R + r) * HP_M + mg * 8) = make_float4(acc[r][0], acc[r][1], acc[r][2], acc[r][3]);
+    *reinterpret_cast<float4*>(red + ((size_t)kg * HP_R + r) * HP_M + mg * 8 + 4) = make_float4(acc[r][4], acc[r][5], acc[r][6], acc[r][7]);
+  }
+  __syncthreads();
+  const int m = (blockIdx.x % mt) * HP_M + tid;
+  if (m < a.M)
+    for (int r = 0; r < nr; ++r) {
+      float t = 0.f;
+#pragma unroll
+      for (int q = 0; q < 8; ++q) t += red[((size_t)q * HP_R + r) * HP_M + tid];
+      const int row = a.rows && a.out_list ? a.rows[r0 + r] : r0 + r;
+      ((T*)a.out)[(size_t)row * a.out_row + (size_t)h * a.out_head + m] = from_f<T>(t);
+    }
+}
+
+__global__ void __launch_bounds__(256) gather_pages_kernel(const uint4* pool, const int* pages, uint4* out, int words, int n_pages, Status* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  int page = pages[blockIdx.x];
+  if (page < 0 || page >= n_pages) { if (threadIdx.x == 0) status_set(status, ST_BOUNDS, 68, page, n_pages); page = 0; }
+  const uint4* s = pool + (size_t)page * words;
+  uint4* d = out + (size_t)blockIdx.x * words;
+#pragma unroll 4
+  for (int i = blockIdx.y * 256 + threadIdx.x; i < words; i += gridDim.y * 256) d[i] = s[i];
+}
+
+template <typename T, int V>
+static int launch_head_proj(const HeadProjArgs& a, int H, cudaStream_t st) {
+  const size_t smem = ((size_t)HP_R * a.K + (size_t)8 * HP_R * HP_M) * sizeof(float);
+  static size_t granted = 48 * 1024;
+  if (smem > granted) {
+    const cudaError_t e = cudaFuncSetAttribute(head_proj_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    granted = smem;
+  }
+  return (int)sfb_launch(head_proj_kernel<T, V>, dim3(H * ((a.M + HP_M - 1) / HP_M), (a.n + HP_R - 1) / HP_R), dim3(HP_T), smem, st, a);
+}
+
+}  // namespace rows
+}  // namespace sfb
+
+using namespace sfb;
+using namespace sfb::rows;
+
+extern "C" {
+
+int sfb_rows_latent_append(void* proj, int64_t stride, const void* w, const void* cs, void* pool, const int* table, const int* row_lane, const int* row_pos,
+                           int max_pages, int n_pages, int n, int H, int dim, int rot, int rank, float eps, int fp32, void* status, cudaStream_t stream) {
+  if (n < 1 || H < 1 || dim < 1 || rot < 0 || rot % 2 || rank < 1) return (int)cudaErrorInvalidValue;
+  LatentArgs a{proj, stride, (const float*)w, (const float2*)cs, pool, table, row_lane, row_pos, max_pages, n_pages, H, dim, rot, rank, eps, (Status*)status};
+  return (int)(fp32 ? sfb_launch(latent_append_kernel<float>, dim3(n), dim3(128), 0, stream, a)
+                    : sfb_launch(latent_append_kernel<__nv_bfloat16>, dim3(n), dim3(128), 0, stream, a));
+}
+
+// list: 0 = rows ignored, 1 = it names x's rows, 2 = it names out's rows
+int sfb_rows_head_proj(const void* x, int64_t x_row, int64_t x_head, const void* w, void* out, int64_t out_row, int64_t out_head, const int* rows, int list,
+                       int n, int H, int K, int M, int tail, int fp32, cudaStream_t stream) {
+  if (n < 1 || n > 65535 * HP_R || H < 1 || K < 1 || M < 1 || K > 8192) return (int)cudaErrorInvalidValue;
+  HeadProjArgs a{x, x_row, x_head, w, out, out_row, out_head, list ? rows : nullptr, list == 1, list == 2, n, K, M, tail};
+  const bool v8 = M % 8 == 0;
+  if (fp32) return v8 ? launch_head_proj<float, 8>(a, H, stream) : launch_head_proj<float, 1>(a, H, stream);
+  return v8 ? launch_head_proj<__nv_bfloat16, 8>(a, H, stream) : launch_head_proj<__nv_bfloat16, 1>(a, H, stream);
+}
+
+// bytes of a page: a multiple of 16
+int sfb_rows_gather_pages(const void* pool, const int* pages, void* out, int count, int64_t page_bytes, int n_pages, void* status, cudaStream_t stream) {
+  if (count < 1 || page_bytes < 16 || page_bytes % 16) return (int)cudaErrorInvalidValue;
+  const int words = (int)(page_bytes / 16);
+  return (int)sfb_launch(gather_pages_kernel, dim3(count, min(8, (words + 1023) / 1024)), dim3(256), 0, stream, (const uint4*)pool, pages, (uint4*)out, words,
+                         n_pages, (Status*)status);
+}
+
+}  // extern "C"

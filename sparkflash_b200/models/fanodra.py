@@ -11,29 +11,20 @@ ops/rows.py; lanes, cache, state, batching and sampling are models/layered.py.
 """
 from __future__ import annotations
 
-import json
-import os
-import warnings
 from dataclasses import dataclass, field
 
 import torch
 
 from ..ops import rows as R
+from .layered import CONFIG_META, LayeredModel, check_keys
 from .mixers import DenseFF, ParallelMixer, RecurrentMixer, W
 
 ARCHITECTURE = "Fanodra"
 DECAY_C = 8.0             # log a = -DECAY_C * r * softplus(lam)
 
 _TOP = {"architecture", "vocab", "width", "norm", "canon", "layers", "loop"}
-_META = {"model_type", "architectures", "dtype", "torch_dtype", "transformers_version", "name", "bos_token_id", "eos_token_id", "pad_token_id"}
 _REC = {"width", "blocks", "conv"}
 _ATT = {"heads", "kv_heads", "dim", "vdim", "scale"}
-
-
-def _keys(d: dict, want: set, where: str, optional: set = frozenset()) -> None:
-    missing, extra = want - set(d) - optional, set(d) - want - optional
-    if missing or extra:
-        raise ValueError(f"config.json: {where}: missing {sorted(missing)}, unknown {sorted(extra)}")
 
 
 @dataclass
@@ -62,36 +53,36 @@ class FanodraConfig:
 
     @classmethod
     def from_dict(cls, d: dict) -> "FanodraConfig":
-        _keys(d, _TOP, "top level", _META | {"loop"})
+        check_keys(d, _TOP, "top level", CONFIG_META | {"loop"})
         if d["architecture"] != ARCHITECTURE:
             raise ValueError(f"config.json: architecture {d['architecture']!r} is not {ARCHITECTURE}")
-        _keys(d["norm"], {"eps"}, "norm")
-        _keys(d["canon"], {"taps"}, "canon")
+        check_keys(d["norm"], {"eps"}, "norm")
+        check_keys(d["canon"], {"taps"}, "canon")
         layers = []
         for i, L in enumerate(d["layers"]):
-            _keys(L, {"type", "mixer", "mlp"}, f"layer {i}", {"mlp"})
+            check_keys(L, {"type", "mixer", "mlp"}, f"layer {i}", {"mlp"})
             m = L["mixer"]
             if L["type"] == "parallel":
-                _keys(m, {"left", "right"}, f"layer {i} mixer")
-                _keys(m["left"], _ATT, f"layer {i} left")
+                check_keys(m, {"left", "right"}, f"layer {i} mixer")
+                check_keys(m["left"], _ATT, f"layer {i} left")
                 if m["left"]["heads"] % m["left"]["kv_heads"]:
                     raise ValueError(f"layer {i}: heads must be a multiple of kv_heads")
             elif L["type"] != "rglru":
                 raise ValueError(f"layer {i}: unknown type {L['type']!r}")
             rec = m["right"] if L["type"] == "parallel" else m
-            _keys(rec, _REC, f"layer {i} recurrence")
+            check_keys(rec, _REC, f"layer {i} recurrence")
             if rec["width"] % rec["blocks"]:
                 raise ValueError(f"layer {i}: recurrence width must be a multiple of blocks")
             if not 1 <= rec["conv"] <= R.MAX_TAPS:
                 raise ValueError(f"layer {i}: convolutions of 1..{R.MAX_TAPS} taps are implemented")
             ff = L.get("mlp")
             if ff is not None:
-                _keys(ff, {"kind", "ff"}, f"layer {i} mlp")
+                check_keys(ff, {"kind", "ff"}, f"layer {i} mlp")
                 if ff["kind"] != "dense":
                     raise ValueError(f"layer {i}: unknown mlp kind {ff['kind']!r}")
             layers.append(LayerSpec(L["type"], m, ff["ff"] if ff is not None else None))
         loop = d.get("loop") or {"start": 0, "stop": 0, "times": 0}
-        _keys(loop, {"start", "stop", "times"}, "loop")
+        check_keys(loop, {"start", "stop", "times"}, "loop")
         if loop["times"] and not 0 <= loop["start"] < loop["stop"] <= len(layers):
             raise ValueError("config.json: loop range outside the layers")
         if not 1 <= d["canon"]["taps"] <= R.MAX_TAPS:
@@ -181,22 +172,14 @@ class _Layer:
         self.canon = w.taps("canon1")
 
 
-class Fanodra:
+class Fanodra(LayeredModel):
     """The model as models/layered.py drives it."""
+
+    config_class = FanodraConfig
 
     def __init__(self, cfg: FanodraConfig, tensors: dict[str, torch.Tensor], dtype: torch.dtype = torch.bfloat16, device="cuda",
                  max_context: int = 4096):
-        if dtype not in (torch.bfloat16, torch.float32):
-            raise ValueError("activation type must be bfloat16 or float32")
-        for name, shape in cfg.shapes().items():
-            if name not in tensors:
-                raise ValueError(f"checkpoint lacks {name}")
-            if tuple(tensors[name].shape) != shape:
-                raise ValueError(f"{name}: shape {tuple(tensors[name].shape)}, expected {shape}")
-        extra = set(tensors) - set(cfg.shapes())
-        if extra:
-            warnings.warn(f"checkpoint tensors that the configuration does not use: {sorted(extra)[:4]}")
-        self.cfg, self.vocab, self.width, self.dtype, self.device = cfg, cfg.vocab, cfg.width, dtype, device
+        self._load(cfg, tensors, dtype, device)
         self.layers = [_Layer(tensors, i, spec, cfg, dtype, device, max_context) for i, spec in enumerate(cfg.layers)]
         top = W(tensors, "", dtype, device)
         self.embed = top.act("embed")
@@ -205,36 +188,6 @@ class Fanodra:
         self.order = cfg.runs()
         self.kv_runs = [self.layers[i].mixer.kv_run for i, _ in self.order if self.layers[i].mixer.kv_run is not None]
         self.tc_attention = any(L.mixer.att.tc for L in self.layers if isinstance(L.mixer, ParallelMixer))
-
-    @classmethod
-    def from_dir(cls, path: str, dtype: torch.dtype = torch.bfloat16, device="cuda", max_context: int = 4096) -> "Fanodra":
-        from ..weights.files import load_checkpoint_dir
-        with open(os.path.join(path, "config.json")) as f:
-            cfg = FanodraConfig.from_dict(json.load(f))
-        tensors, files = load_checkpoint_dir(path)
-        model = cls(cfg, tensors, dtype, device, max_context)
-        if torch.device(device).type == "cuda":
-            torch.cuda.synchronize()          # the copies out of the mapped files have been made
-        for f in files:
-            f.close()
-        return model
-
-    def nbytes(self) -> int:
-        seen, total, todo = set(), 0, [self]
-        while todo:
-            o = todo.pop()
-            if id(o) in seen:
-                continue
-            seen.add(id(o))
-            if isinstance(o, torch.Tensor):
-                total += o.numel() * o.element_size()
-            elif isinstance(o, (list, tuple)):
-                todo += o
-            elif isinstance(o, dict):
-                todo += o.values()
-            elif type(o).__module__.startswith("sparkflash_b200.models"):
-                todo += [v for k, v in vars(o).items() if k not in ("engine", "run_state")]
-        return total
 
     # ---- layered engine -----------------------------------------------------------------------------------------------
     def bind(self, e) -> None:
@@ -274,7 +227,7 @@ class Fanodra:
                 return h
             R.seam(x, n, h=h, norm=L.norm["norm1"], **self._begin(r), **update, **common)
             hc = s.scratch.get("hc", n, d)
-            R.conv(h, L.canon, None, hc, st["canon"], s, n, residual=True)
+            R.conv(h, L.canon, None, hc, st["canon"], s, n, R.CONV_RESIDUAL)
             return hc
         h_in = enter(0, from_embed=True)
         for r, (i, _) in enumerate(self.order):

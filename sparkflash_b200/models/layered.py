@@ -7,12 +7,18 @@ row selection and the sampler - and speaks the contract of serve/driver.py.  A m
 
     vocab, width, dtype, device        sizes; ``dtype`` is the activation type (bfloat16, or float32 for true 32-bit)
     kv_runs                            (kv_heads, dim, vdim) of every attention layer run
+    tc_attention, tc_state             long runs of rows go to the tensor-core arms of attention / of the matrix-state recurrence
+    windows                            window lengths whose keys are multiplied out for a step's long runs
     bind(engine)                       reserve scratch, register state tensors
     forward(step) -> [head rows, vocab] float32 logits (None without a head)
 
-and writes no loop, cache or batching of its own (models/fanodra.py is one).
+and writes no loop, cache or batching of its own (models/fanodra.py and models/gudutar.py are two; ``LayeredModel`` has what they share).
 """
 from __future__ import annotations
+
+import json
+import os
+import warnings
 
 import torch
 
@@ -23,6 +29,7 @@ from ..ops.sampling import candidate_choice
 
 TC_MIN_ROWS = 32          # runs of at least this many rows go to the tensor-core attention (csrc/k_rows_attn_tc.cu)
 TC_TILE = 256             # query rows per block there
+STATE_CHUNK = 128         # rows of a chunk of the tensor-core recurrence (csrc/k_rows_state_tc.cu)
 TARGET_BLOCKS = 592       # blocks that fill the machine (148 SMs x 4): how far a row's keys are split
 MAX_SPLITS = 64
 
@@ -61,10 +68,76 @@ class Step:
 
     rows: ``tokens``, ``row_pos``, ``row_lane``, ``row_seg``; segments: ``seg_row0``, ``seg_len``, ``seg_src``, ``seg_dst``;
     scan chunks: ``chunk_*``; attention: ``short_rows`` (rows for the exact arm, None = all), ``tiles`` ((row0, rows) pairs of
-    the tensor-core arm, longest first); head: ``head_rows`` (None = all rows, in order)."""
+    the tensor-core arm, longest first); matrix-state recurrence: ``short_segs`` (segments for the row arm, None = all, ``nshort`` of
+    them), ``long_*`` (``nchunks`` chunks of the ``nlong`` others, see _stage); ``expand``: per window the pages whose keys the
+    tensor-core arm needs, how many they are, and every tile's page offset among them; head: ``head_rows`` (None = all rows, in order)."""
 
     single = False            # every segment is one row (a decode step)
     taps: list | None = None  # debug: collects the residual after every layer run
+
+
+class LayeredModel:
+    """What the models of the engine share: a checkpoint of named tensors whose shapes the configuration knows."""
+
+    config_class: type
+    tc_attention = False
+    tc_state = False
+    windows: tuple[int, ...] = ()
+
+    def _load(self, cfg, tensors: dict[str, torch.Tensor], dtype: torch.dtype, device) -> None:
+        if dtype not in (torch.bfloat16, torch.float32):
+            raise ValueError("activation type must be bfloat16 or float32")
+        shapes = cfg.shapes()
+        for name, shape in shapes.items():
+            if name not in tensors:
+                raise ValueError(f"checkpoint lacks {name}")
+            if tuple(tensors[name].shape) != shape:
+                raise ValueError(f"{name}: shape {tuple(tensors[name].shape)}, expected {shape}")
+        extra = set(tensors) - set(shapes)
+        if extra:
+            warnings.warn(f"checkpoint tensors that the configuration does not use: {sorted(extra)[:4]}")
+        self.cfg, self.vocab, self.width, self.dtype, self.device = cfg, cfg.vocab, cfg.width, dtype, device
+
+    @classmethod
+    def from_dir(cls, path: str, dtype: torch.dtype = torch.bfloat16, device="cuda", max_context: int = 4096):
+        from ..weights.files import load_checkpoint_dir
+        with open(os.path.join(path, "config.json")) as f:
+            cfg = cls.config_class.from_dict(json.load(f))
+        tensors, files = load_checkpoint_dir(path)
+        model = cls(cfg, tensors, dtype, device, max_context)
+        if torch.device(device).type == "cuda":
+            torch.cuda.synchronize()          # the copies out of the mapped files have been made
+        for f in files:
+            f.close()
+        return model
+
+    def nbytes(self) -> int:
+        seen, total, todo = set(), 0, [self]
+        while todo:
+            o = todo.pop()
+            if id(o) in seen:
+                continue
+            seen.add(id(o))
+            if isinstance(o, torch.Tensor):
+                total += o.numel() * o.element_size()
+            elif isinstance(o, (list, tuple)):
+                todo += o
+            elif isinstance(o, dict):
+                todo += o.values()
+            elif type(o).__module__.startswith("sparkflash_b200.models"):
+                todo += [v for k, v in vars(o).items() if k not in ("engine", "run_state")]
+        return total
+
+
+def check_keys(d: dict, want: set, where: str, optional: set = frozenset()) -> None:
+    """A part of config.json has exactly these keys: what is not implemented is refused."""
+    missing, extra = want - set(d) - optional, set(d) - want - optional
+    if missing or extra:
+        raise ValueError(f"config.json: {where}: missing {sorted(missing)}, unknown {sorted(extra)}")
+
+
+# keys of a config.json that do not describe the computation
+CONFIG_META = {"model_type", "architectures", "dtype", "torch_dtype", "transformers_version", "name", "bos_token_id", "eos_token_id", "pad_token_id"}
 
 
 class LayeredEngine:
@@ -96,7 +169,7 @@ class LayeredEngine:
         model.bind(self)
         self.scratch.reserve("logits", max_lanes * model.vocab, torch.float32)
         self.scratch.allocate()
-        self._cap = 20 * max_rows + 64
+        self._cap = 22 * max_rows + 64 + len(model.windows) * (self.n_pages + max_rows)
         cuda = self.dev.type == "cuda"
         self._host = torch.zeros((self._cap,), dtype=torch.int32, pin_memory=cuda)
         self._np = self._host.numpy()
@@ -173,7 +246,8 @@ class LayeredEngine:
         n = len(rows_tok)
         if n > self.max_rows:
             raise ValueError(f"{n} rows with the ones to run again, at most {self.max_rows}")
-        s.n, s.nseg, s.single = n, len(segs), len(segs) == n
+        s.n, s.nseg, s.single, model = n, len(segs), len(segs) == n, self.model
+        s.nlong, s.nchunks, s.nshort, s.expand = 0, 0, len(segs), {}
         hrows = [back[i] for i in heads]
         s.nhead = len(hrows)
         all_heads = hrows == list(range(n))
@@ -198,7 +272,7 @@ class LayeredEngine:
             s.chunks, s.summaries = len(cs), int(len(cs) > len(segs))
             short, tiles = [], []
             for k in range(len(segs)):
-                if self.model.tc_attention and length[k] >= TC_MIN_ROWS:
+                if model.tc_attention and length[k] >= TC_MIN_ROWS:
                     tiles += [(rows_pos[row0[k] + r], row0[k] + r, min(TC_TILE, length[k] - r)) for r in range(0, length[k], TC_TILE)]
                 else:
                     short += range(row0[k], row0[k] + length[k])
@@ -207,6 +281,27 @@ class LayeredEngine:
             put("tiles", [x for _, r, m in tiles for x in (r, m)])
             if tiles:
                 put("short_rows", short)
+            if model.windows and tiles:
+                for w in model.windows:
+                    pages, base = [], {}
+                    for k in range(len(segs)):
+                        if length[k] >= TC_MIN_ROWS:
+                            p0 = rows_pos[row0[k]]
+                            lo, hi = max(0, p0 - w + 1) // PAGE, (p0 + length[k] - 1) // PAGE + 1
+                            base[k] = len(pages) - lo
+                            pages += self.kv.pages[segs[k][0]][lo:hi]
+                    put(f"pages{w}", pages)
+                    put(f"offs{w}", [base[rows_seg[r]] for _, r, _ in tiles])
+            if model.tc_state:
+                long = [k for k in range(len(segs)) if length[k] >= TC_MIN_ROWS]
+                put("short_segs", [k for k in range(len(segs)) if length[k] < TC_MIN_ROWS])
+                chunks, first = [], []
+                for k in long:
+                    first.append(len(chunks))
+                    chunks += [(row0[k] + r, min(STATE_CHUNK, length[k] - r)) for r in range(0, length[k], STATE_CHUNK)]
+                put("long_seg", long); put("long_first", first + [len(chunks)])
+                put("long_row0", [c[0] for c in chunks]); put("long_rows", [c[1] for c in chunks])
+                s.nlong, s.nchunks, s.nshort = len(long), len(chunks), len(segs) - len(long)
         self._meta[:at].copy_(self._host[:at], non_blocking=True)
         self.kv.upload()
         if self._event is not None:
@@ -218,6 +313,9 @@ class LayeredEngine:
             s.seg_len = s.chunk_rows = self._ones[:n]
         if "short_rows" not in views:
             s.short_rows = None
+        if "short_segs" not in views:
+            s.short_segs = None
+        s.expand = {w: (getattr(s, f"pages{w}"), views[f"pages{w}"][1], getattr(s, f"offs{w}")) for w in model.windows if f"pages{w}" in views}
         if all_heads:
             s.head_rows = None
         s.seed, s.temp = s.seed.view(torch.int64), s.temp.view(torch.float32)
@@ -312,9 +410,18 @@ class LayeredEngine:
         torch.cuda.synchronize()
         self.graphs.clear()
 
-    def splits(self, s: Step, rows: int, blocks_per_row: int) -> int:
+    def short_rows(self, tc: bool) -> int:
+        """Most rows of a step that do not go to the tensor-core arm."""
+        return self.max_lanes * TC_MIN_ROWS if tc else self.max_rows
+
+    def expanded_rows(self, window: int) -> int:
+        """Most positions whose keys the long runs of a step need: their own and a window before each run, in whole pages."""
+        runs = min(self.max_lanes, max(1, self.max_rows // TC_MIN_ROWS))
+        return PAGE * min(self.n_pages, self.max_rows // PAGE + runs * (window // PAGE + 3))
+
+    def splits(self, s: Step, rows: int, blocks_per_row: int, window: int = 2 ** 31 - 1) -> int:
         """Ranges a row's pages are cut into so that ``rows`` single rows fill the machine."""
-        return max(1, min(s.pages, MAX_SPLITS, TARGET_BLOCKS // max(1, rows * blocks_per_row)))
+        return max(1, min(s.pages, window // PAGE + 2, MAX_SPLITS, TARGET_BLOCKS // max(1, rows * blocks_per_row)))
 
     def generate(self, prompt: list[int], n_new: int, lane: int = 0, temperature: float = 0.0, seed: int = 0, chunk: int | None = None):
         """Prefill ``prompt`` in portions of ``chunk`` rows, then decode ``n_new`` tokens one row at a time."""

@@ -1,5 +1,6 @@
 """Sublayers of the layered decoders (models/layered.py): attention with a distance bias, the real-gated linear recurrence, two
-mixers side by side, and the dense gated feed-forward.  Each takes its sizes and constants as arguments, reads its weights by
+mixers side by side, matrix-state recurrences (state-space duality, retention), latent attention in a window, and the dense gated
+feed-forward.  Each takes its sizes and constants as arguments, reads its weights by
 name, keeps its caches in the engine's page pool or state slots, and runs on a step's rows through the kernels of ops/rows.py.
 
 A sublayer is built once per layer (``weights``) and bound once per run of the layer (``bind_run``): a looped layer shares its
@@ -24,9 +25,12 @@ class W:
     def sub(self, name: str) -> "W":
         return W(self.t, self.p + name, self.dtype, self.device)
 
-    def act(self, *names: str) -> torch.Tensor:
-        """One matrix out of several, stacked along the output dimension."""
-        return torch.cat([self.t[self.p + n] for n in names], 0).to(self.device, self.dtype).contiguous()
+    def act(self, *names: str, pad: int = 1) -> torch.Tensor:
+        """One matrix out of several, stacked along the output dimension; zero rows up to a multiple of ``pad``."""
+        t = torch.cat([self.t[self.p + n] for n in names], 0).to(self.device, self.dtype)
+        if t.shape[0] % pad:
+            t = torch.cat([t, t.new_zeros(pad - t.shape[0] % pad, *t.shape[1:])], 0)
+        return t.contiguous()
 
     def f32(self, name: str) -> torch.Tensor:
         return self.t[self.p + name].to(self.device, torch.float32).contiguous()
@@ -126,7 +130,7 @@ class GatedRecurrence:
             R.gated_step(x, y, self.cw, self.cb, hist, self.wg, self.rb, self.ib, self.decay, S, o, s.seg_src, s.seg_dst, n)
         else:
             u = s.scratch.get("rec_u", n, self.width)
-            R.conv(x, self.cw, self.cb, u, hist, s, n, residual=False)
+            R.conv(x, self.cw, self.cb, u, hist, s, n)
             gates = s.scratch.get("rec_gates", self.parts, n, 2 * self.bs)
             R.block_gates(u, self.wg, gates)
             R.scan(gates, self.rb, self.ib, self.decay, u, y, o, S, s.scratch.buf["rec_sums"], s, n, self.bs)
@@ -182,10 +186,178 @@ class ParallelMixer:
         return y, y2
 
 
-class DenseFF:
-    """W_down (silu(W_gate h) * (W_up h)) with gate and up in one product."""
+def rotation_table(base: float, dims: int, length: int, device) -> torch.Tensor:
+    """[length, dims / 2, 2]: cosine and sine of p base^(-2 i / dims), evaluated in 64-bit and rounded once."""
+    f = torch.tensor([base ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64)
+    a = torch.arange(length, dtype=torch.float64)[:, None] * f
+    return torch.stack([a.cos(), a.sin()], -1).to(torch.float32).to(device).contiguous()
 
-    def __init__(self, w: W):
+
+class MatrixState:
+    """S_t = a_t S_(t-1) + w_t k_t v_t^T, y_t = S_t^T q_t + D v_t: one 32-bit state [P, N] and one decay per head, q and k shared by
+    groups of heads.  Decay and input weight come from a step size per token (a = exp(A dt), w = dt), or the decay is a constant."""
+
+    def __init__(self, heads: int, groups: int, n: int, p: int, decay: torch.Tensor, dt_bias=None, skip=None, rot=None, rot_dims: int = 0,
+                 k_scale: float = 1.0):
+        self.H, self.G, self.N, self.P = heads, groups, n, p
+        self.decay, self.dt_bias, self.skip, self.rot, self.rot_dims, self.k_scale = decay, dt_bias, skip, rot, rot_dims, k_scale
+        self.tc = False
+
+    def state(self, e, tag: str) -> torch.Tensor:
+        return e.state.add(tag, (self.H, self.P, R.state_pad(self.N)), torch.float32)
+
+    def reserve(self, e, dtype) -> None:
+        pass
+
+    def run(self, s, q, k, v, dt, S, y, conv=None) -> None:
+        R.state_rows(q, k, v, dt, self.dt_bias, self.decay, self.skip, self.rot, self.rot_dims, self.k_scale, s.row_pos, y, S, self.N, self.G, s.short_segs,
+                     s.nshort, s, conv)
+
+
+class StateSpaceMixer:
+    """Mamba-2 (Dao & Gu, "Transformers are SSMs: Generalized Models and Efficient Algorithms Through Structured State Space Duality"):
+    z | x | B | C | dt = W_in h; x, B, C through a causal convolution and silu; the matrix-state recurrence with k = B, v = x, q = C; silu(z)
+    gate, RMS norm in equal parts, W_o."""
+
+    def __init__(self, w: W, spec: dict, eps: float):
+        H, P, N, G = spec["heads"], spec["vdim"], spec["state"], spec["groups"]
+        self.inner, self.bc, self.taps, self.eps, self.part = H * P, G * N, spec["conv"], eps, H * P // spec["norm_groups"]
+        self.channels = self.inner + 2 * self.bc
+        self.w_in, self.w_out = w.act("in", pad=8), w.act("o")
+        self.cw, self.cb, self.norm = w.taps("conv"), w.f32("conv.b"), w.f32("norm")
+        A = -torch.exp(w.t[w.p + "A_log"].to(w.device, torch.float64)).to(torch.float32)
+        self.core = MatrixState(H, G, N, P, A.contiguous(), w.f32("dt_bias"), w.f32("D"))
+        self.merge, self.kv_run = (None, None), None
+
+    def reserve(self, e) -> None:
+        n, dt = e.max_rows, self.w_in.dtype
+        e.scratch.reserve("proj", n * self.w_in.shape[0], dt)
+        e.scratch.reserve("mix_u", n * self.channels, dt)
+        e.scratch.reserve("mix_y", n * self.inner, dt)
+        e.scratch.reserve("mix_o", n * self.inner, dt)
+        self.core.reserve(e, dt)
+
+    def bind_run(self, e, tag: str, kv_index):
+        return {"conv": e.state.add(tag + ".conv", (self.taps - 1, self.channels), self.w_in.dtype), "S": self.core.state(e, tag + ".S")}
+
+    def run(self, s, h, run):
+        n, i, bc = s.n, self.inner, self.bc
+        proj = R.linear(h, self.w_in, None, s.scratch.get("proj", n, self.w_in.shape[0]))
+        z, u, dt = proj[:, :i], proj[:, i:i + self.channels], proj[:, i + self.channels:]
+        y = s.scratch.get("mix_y", n, i)
+        conv = (self.cw, self.cb, run["conv"], (i + bc, i, 0)) if s.single else None
+        if conv is None:
+            raw, u = u, s.scratch.get("mix_u", n, self.channels)
+            R.conv(raw, self.cw, self.cb, u, run["conv"], s, n, R.CONV_SILU)
+        self.core.run(s, u[:, i + bc:], u[:, i:i + bc], u[:, :i], dt, run["S"], y, conv)
+        o = s.scratch.get("mix_o", n, i)
+        R.gated_norm(y, z, self.norm, o, self.part, True, self.eps)
+        return R.linear(o, self.w_out, None, s.scratch.get("y", n, h.shape[1])), None
+
+
+class RetentionMixer:
+    """Retention (Sun et al., "Retentive Network: A Successor to Transformer for Large Language Models"): rotated queries and keys, a
+    fixed decay per head, no softmax; every head's output over its RMS, silu(W_g h) gate, W_o."""
+
+    PROJ = ("q", "k", "v", "g")
+
+    def __init__(self, w: W, spec: dict, eps: float, max_context: int):
+        H, N, P, rot = spec["heads"], spec["dim"], spec["vdim"], spec["rot"]
+        self.inner, self.qk, self.P, self.eps = H * P, H * N, P, eps
+        self.w_in, self.w_out = w.act(*self.PROJ, pad=8), w.act("o")
+        decay = torch.tensor(spec["decay"], dtype=torch.float64).to(w.device, torch.float32)
+        self.core = MatrixState(H, H, N, P, decay, rot=rotation_table(rot["base"], rot["dims"], max_context, w.device), rot_dims=rot["dims"],
+                                k_scale=N ** -0.5)
+        self.merge, self.kv_run = (None, None), None
+
+    def reserve(self, e) -> None:
+        n, dt = e.max_rows, self.w_in.dtype
+        e.scratch.reserve("proj", n * self.w_in.shape[0], dt)
+        e.scratch.reserve("mix_y", n * self.inner, dt)
+        e.scratch.reserve("mix_o", n * self.inner, dt)
+        self.core.reserve(e, dt)
+
+    def bind_run(self, e, tag: str, kv_index):
+        return {"S": self.core.state(e, tag + ".S")}
+
+    def run(self, s, h, run):
+        n, i, qk = s.n, self.inner, self.qk
+        proj = R.linear(h, self.w_in, None, s.scratch.get("proj", n, self.w_in.shape[0]))
+        y, o = s.scratch.get("mix_y", n, i), s.scratch.get("mix_o", n, i)
+        self.core.run(s, proj[:, :qk], proj[:, qk:2 * qk], proj[:, 2 * qk:2 * qk + i], None, run["S"], y)
+        R.gated_norm(y, proj[:, 2 * qk + i:2 * qk + 2 * i], None, o, self.P, False, self.eps)
+        return R.linear(o, self.w_out, None, s.scratch.get("y", n, h.shape[1])), None
+
+
+class LatentAttention:
+    """Attention whose keys and values are products of one cached vector per token (DeepSeek-AI, "DeepSeek-V2: A Strong, Economical, and
+    Efficient Mixture-of-Experts Language Model"): the RMS-normed latent c, beside one rotated key part that the heads share.  A
+    position sees the last ``window`` ones.  Single rows and short runs score in the latent space (W_uk on the query, W_uv on the output);
+    long runs multiply the window's keys and values out and take the tensor-core attention."""
+
+    PROJ = ("q", "dkv")
+
+    def __init__(self, w: W, spec: dict, eps: float, max_context: int):
+        self.H, self.dim, self.rot, self.vdim, self.rank = spec["heads"], spec["dim"], spec["rot_dim"], spec["vdim"], spec["kv_rank"]
+        self.scale, self.eps, self.window = float(spec["scale"]), eps, min(int(spec["mask"]["size"]), max_context)
+        self.w_in, self.w_out, self.norm = w.act(*self.PROJ, pad=8), w.act("o"), w.f32("dkv.norm")
+        self.uk = w.act("uk").view(self.H, self.dim, self.rank)
+        self.uv = w.act("uv").view(self.H, self.vdim, self.rank).transpose(1, 2).contiguous()       # [H, rank, vdim]
+        self.cs = rotation_table(spec["rot"]["base"], self.rot, max_context, w.device)
+        self.tc = R.latent_tc_supports(w.dtype, self.dim, self.rot, self.vdim, self.rank)
+        self.merge, self.kv_run = (None, None), (1, self.rank + self.rot, 0)
+
+    def reserve(self, e) -> None:
+        n, dt, key = e.max_rows, self.w_in.dtype, self.rank + self.rot
+        e.scratch.reserve("proj", n * self.w_in.shape[0], dt)
+        e.scratch.reserve("mix_o", n * self.H * self.vdim, dt)
+        short = min(n, e.short_rows(self.tc))
+        e.scratch.reserve("lat_q", short * self.H * key, dt)
+        e.scratch.reserve("lat_o", short * self.H * self.rank, dt)
+        parts = max(1, self.H // R.attn_blocks(self.H, 1)) * 1024 + self.H * 64
+        e.scratch.reserve("attn_part", parts * self.rank, torch.float32)
+        e.scratch.reserve("attn_ml", parts * 2, torch.float32)
+        if self.tc:
+            m = e.expanded_rows(self.window)
+            e.scratch.reserve("lat_rows", m * key, dt)
+            e.scratch.reserve("lat_k", m * self.H * self.dim, dt)
+            e.scratch.reserve("lat_v", m * self.H * self.vdim, dt)
+
+    def bind_run(self, e, tag: str, kv_index):
+        return {"kv": e.kv.k[kv_index]}
+
+    def run(self, s, h, run):
+        n, H, dim, rot, key, pool = s.n, self.H, self.dim, self.rot, self.rank + self.rot, run["kv"]
+        proj = R.linear(h, self.w_in, None, s.scratch.get("proj", n, self.w_in.shape[0]))
+        R.latent_append(proj, self.norm, self.cs, pool, s.table, s.row_lane, s.row_pos, n, H, dim, rot, self.rank, self.eps, s.status)
+        o = s.scratch.get("mix_o", n, H * self.vdim)
+        if s.ntiles:
+            pages, count, offs = s.expand[self.window]
+            m = count * 64
+            rows = s.scratch.get("lat_rows", m, key)
+            kx, vx = s.scratch.get("lat_k", H, m, dim), s.scratch.get("lat_v", H, m, self.vdim)
+            R.gather_pages(pool, pages, rows, count, s.status)
+            R.expand(rows[:, :self.rank], self.uk.transpose(1, 2), kx)
+            R.expand(rows[:, :self.rank], self.uv, vx)
+            R.latent_attn_tc(proj, proj.shape[1], kx, vx, rows, self.rank, s.row_pos, s.tiles, offs, s.ntiles, o, H, dim, rot, self.vdim, self.window,
+                             self.scale, s.status)
+        if s.short:
+            m = s.short
+            q, c = s.scratch.get("lat_q", m, H * key), s.scratch.get("lat_o", m, H * self.rank)
+            R.head_proj(proj, dim + rot, self.uk, q, key, m, s.short_rows, 1, rot)
+            blocks = R.attn_blocks(H, 1)
+            sp = s.engine.splits(s, m, blocks, self.window)
+            part, ml = (s.scratch.buf["attn_part"], s.scratch.buf["attn_ml"]) if sp > 1 else (None, None)
+            R.attn(q, pool, None, s.table, s.row_lane, s.row_pos, s.short_rows, m, None, c, part, ml, H, self.scale, sp, s.status, self.window, self.rank, True)
+            R.head_proj(c, self.rank, self.uv, o, self.vdim, m, s.short_rows, 2)
+        return R.linear(o, self.w_out, None, s.scratch.get("y", n, h.shape[1])), None
+
+
+class DenseFF:
+    """W_down (act(W_gate h) * (W_up h)) with gate and up in one product; act: silu, or gelu_tanh."""
+
+    def __init__(self, w: W, act: str = "silu"):
+        self.act = act
         self.w_in, self.w_out = w.act("gate", "up"), w.act("down")
         self.ff = self.w_out.shape[1]
 
@@ -194,5 +366,5 @@ class DenseFF:
         e.scratch.reserve("ff_act", e.max_rows * self.ff, self.w_in.dtype)
 
     def run(self, s, h):
-        act = R.gated_linear(h, self.w_in, s.scratch.get("proj", s.n, 2 * self.ff), s.scratch.get("ff_act", s.n, self.ff))
+        act = R.gated_linear(h, self.w_in, s.scratch.get("proj", s.n, 2 * self.ff), s.scratch.get("ff_act", s.n, self.ff), self.act)
         return R.linear(act, self.w_out, None, s.scratch.get("y", s.n, h.shape[1]))

@@ -27,11 +27,12 @@ MODELS = {m.name: m for m in [
     ModelEntry("inkling-2-small", "inkling", "oracle", "short conv, soft-capped windowed attention and SwiGLU, MoE with expert / intermediate / row splits; device rows step", "sparkflash_b200.models.inkling"),
     ModelEntry("dory-1.0-4b", "dory", "oracle", "latent-recurrence model, loops split over a ring pipeline of ranks", "sparkflash_b200.models.dory"),
     ModelEntry("fanodra", "fanodra", "device", "gated linear recurrence, alone or beside attention with a distance bias; looped layers, input convolution; layered engine (bf16 or 32-bit)", "sparkflash_b200.models.fanodra"),
+    ModelEntry("gudutar", "gudutar", "device", "state-space duality, retention and latent attention in a window; norms on sublayer outputs, layers that share weights; layered engine (bf16 or 32-bit)", "sparkflash_b200.models.gudutar"),
     ModelEntry("dflash-block-drafter", "drafter", "oracle", "one-forward block drafter over a ring of captured target features", "sparkflash_b200.models.dflash"),
 ]}
 
 # config.json "architecture" -> (module, class) of the models that run on the layered engine (models/layered.py)
-LAYERED = {"Fanodra": ("sparkflash_b200.models.fanodra", "Fanodra")}
+LAYERED = {"Fanodra": ("sparkflash_b200.models.fanodra", "Fanodra"), "Gudutar": ("sparkflash_b200.models.gudutar", "Gudutar")}
 
 
 def architecture(path: str) -> str:

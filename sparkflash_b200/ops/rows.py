@@ -22,21 +22,24 @@ def _fp32(t: torch.Tensor) -> c_int:
 
 
 def seam(x, n, *, h=None, y=None, y2=None, merge_w=(None, None), post=(None, None), embed=None, tokens=None, from_embed=False, add_embed=False,
-         step_vec=None, tap=None, norm=(None, None), row_map=None, conv=None, eps=1e-6, status=None):
-    """x += LN(y; post) (y and y2: half the sum of their RMS norms), + embedding, + step_vec; h = LN(x; norm).
+         step_vec=None, tap=None, norm=(None, None), row_map=None, conv=None, eps=1e-6, status=None, embed_scale=1.0):
+    """x += LN(y; post) (y and y2: half the sum of their RMS norms), + embedding * embed_scale, + step_vec; h = LN(x; norm), or x itself.
     ``conv``: (weight [taps, d], history, src, dst) applies h + conv(h) on a step of single-row segments."""
     act = h if h is not None else (y if y is not None else embed)
     cw, hist, src, dst = conv if conv is not None else (None, None, None, None)
     _check(_lib.rows().sfb_rows_seam(_p(x), _p(y), _p(y2), _p(merge_w[0]), _p(merge_w[1]), _p(post[0]), _p(post[1]), _p(embed), _p(tokens),
                                      _p(step_vec), _p(tap), _p(norm[0]), _p(norm[1]), _p(h), _p(row_map), _p(cw), _p(hist), _p(src), _p(dst),
                                      c_int(from_embed), c_int(add_embed), c_int(cw.shape[0] if cw is not None else 0), c_int(n), c_int(x.shape[1]),
-                                     c_int(embed.shape[0] if embed is not None else 0), c_float(eps), _fp32(act), _p(status), _stream()), "rows_seam")
+                                     c_int(embed.shape[0] if embed is not None else 0), c_float(eps), c_float(embed_scale), _fp32(act), _p(status), _stream()), "rows_seam")
 
 
-def conv(x, w, bias, y, hist, seg, n, residual):
-    """y = [x +] causal depthwise convolution of x [n, C] over the step's segments."""
+CONV_PLAIN, CONV_RESIDUAL, CONV_SILU = 0, 1, 2
+
+
+def conv(x, w, bias, y, hist, seg, n, mode=CONV_PLAIN):
+    """y = causal depthwise convolution of x [n, C] over the step's segments (+ x, or followed by silu)."""
     _check(_lib.rows().sfb_rows_conv(_p(x), c_int64(x.stride(0)), _p(w), _p(bias), _p(y), _p(hist), _p(seg.row_seg), _p(seg.seg_row0), _p(seg.seg_len),
-                                     _p(seg.seg_src), _p(seg.seg_dst), c_int(n), c_int(w.shape[1]), c_int(w.shape[0]), c_int(residual), _fp32(y),
+                                     _p(seg.seg_src), _p(seg.seg_dst), c_int(n), c_int(w.shape[1]), c_int(w.shape[0]), c_int(mode), _fp32(y),
                                      _stream()), "rows_conv")
 
 
@@ -47,12 +50,18 @@ def qk_append(proj, qw, kw, q, kpool, vpool, table, row_lane, row_pos, n, heads,
                                           c_int(vdim), c_float(eps), _fp32(q), _p(status), _stream()), "rows_qk_append")
 
 
-def attn(q, kpool, vpool, table, row_lane, row_pos, rows, n_rows, bias, out, part, ml, heads, scale, splits, status):
-    """Exact arm: one block per (row, group of heads, range of pages).  ``rows``: indices of the rows to run, or None for all."""
+NO_WINDOW = 2 ** 31 - 1
+
+
+def attn(q, kpool, vpool, table, row_lane, row_pos, rows, n_rows, bias, out, part, ml, heads, scale, splits, status, window=NO_WINDOW, vdim=None,
+         compact=False):
+    """Exact arm: one block per (row, group of heads, range of pages).  ``rows``: indices of the rows to run, or None for all.
+    ``vpool`` None: values are the first ``vdim`` columns of the keys.  ``compact``: q and out hold only the rows of the launch."""
     _check(_lib.rows().sfb_rows_attn(_p(q), _p(kpool), _p(vpool), _p(table), _p(row_lane), _p(row_pos), _p(rows), _p(bias),
                                      c_int64(bias.shape[1] if bias is not None else 0), _p(out), _p(part), _p(ml), c_int(table.shape[1]),
                                      c_int(kpool.shape[0]), c_int(n_rows), c_int(heads), c_int(kpool.shape[1]), c_int(kpool.shape[3]),
-                                     c_int(vpool.shape[3]), c_int(splits), c_float(scale), _fp32(q), _p(status), _stream()), "rows_attn")
+                                     c_int(vdim or vpool.shape[3]), c_int(splits), c_int(window), c_int(compact), c_float(scale), _fp32(q), _p(status), _stream()),
+           "rows_attn")
 
 
 def scan(gates, rb, ib, decay, u, y, out, S, sums, seg, n, bs):
@@ -70,8 +79,66 @@ def gated_step(x, y, cw, cb, hist, wg, rb, ib, decay, S, out, src, dst, n):
                                            c_int(cw.shape[0]), _fp32(out), _stream()), "rows_gated_step")
 
 
-def silu_mul(gate_up, out, n):
-    _check(_lib.rows().sfb_rows_silu_mul(_p(gate_up), _p(out), c_int(n), c_int(out.shape[1]), _fp32(out), _stream()), "rows_silu_mul")
+ACT = {"silu": 1, "gelu_tanh": 2}
+
+
+def act_mul(gate_up, out, n, act="silu"):
+    _check(_lib.rows().sfb_rows_act_mul(_p(gate_up), _p(out), c_int(n), c_int(out.shape[1]), c_int(ACT[act]), _fp32(out), _stream()), "rows_act_mul")
+
+
+def _strides(t) -> tuple:
+    return (_p(t), c_int64(t.stride(0))) if t is not None else (None, c_int64(0))
+
+
+def state_rows(q, k, v, dt, dt_bias, a, D, rot, rot_dims, k_scale, row_pos, y, S, N, groups, segs, n_segs, seg, conv=None):
+    """S = a S + w k v^T, y = S^T q + D v, one block per (segment, head, tile of value dims); q, k, v, dt: [n, .] views.
+    ``rot``: [positions, rot_dims / 2, 2] or None.  ``conv``: (weight [taps, C], bias, history, first channels of q, k, v) where every
+    segment is one row and q, k, v are the inputs of a convolution with silu.  ``segs``: segments to run, or None for all."""
+    _, H, P, Np = S.shape
+    cw, cb, hist, ch = conv if conv is not None else (None, None, None, (0, 0, 0))
+    _check(_lib.rows().sfb_rows_state(*_strides(q), *_strides(k), *_strides(v), *_strides(dt), _p(dt_bias), _p(a), _p(D), _p(rot), _p(row_pos), _p(y), _p(S),
+                                      _p(cw), _p(cb), _p(hist), _p(segs), _p(seg.seg_row0), _p(seg.seg_len), _p(seg.seg_src), _p(seg.seg_dst),
+                                      c_int(n_segs), c_int(rot_dims), c_int(cw.shape[0] if cw is not None else 0),
+                                      c_int(cw.shape[1] if cw is not None else 0), *map(c_int, ch), c_int(H), c_int(groups), c_int(N), c_int(P),
+                                      c_int(Np), c_float(k_scale), _fp32(y), _stream()), "rows_state")
+
+
+STATE_PADS = tuple(range(32, 257, 32)) + (384, 512)
+
+
+def state_pad(n: int) -> int:
+    """Length of a stored state column of ``n`` elements."""
+    for p in STATE_PADS:
+        if n <= p:
+            return p
+    raise ValueError(f"states of {n} rows are beyond the {STATE_PADS[-1]} implemented")
+
+
+def gated_norm(y, gate, w, out, part, before, eps):
+    """RMS norm of equal parts of a row, times silu(gate): ``before`` the norm, or after it; optional weight."""
+    _check(_lib.rows().sfb_rows_gated_norm(_p(y), *_strides(gate), _p(w), _p(out), c_int(y.shape[0]), c_int(y.shape[1]), c_int(part), c_int(before),
+                                           c_float(eps), _fp32(y), _stream()), "rows_gated_norm")
+
+
+def latent_append(proj, w, cs, pool, table, row_lane, row_pos, n, heads, dim, rot, rank, eps, status):
+    """Norm and rotation of q | latent | shared key part in ``proj``: queries in place, the rest to the pool [pages, 1, 64, rank + rot]."""
+    _check(_lib.rows().sfb_rows_latent_append(*_strides(proj), _p(w), _p(cs), _p(pool), _p(table), _p(row_lane), _p(row_pos), c_int(table.shape[1]),
+                                              c_int(pool.shape[0]), c_int(n), c_int(heads), c_int(dim), c_int(rot), c_int(rank), c_float(eps), _fp32(pool),
+                                              _p(status), _stream()), "rows_latent_append")
+
+
+def head_proj(x, x_head, w, out, out_head, n, rows=None, lists=0, tail=0):
+    """out[row][h] = x[row][h] w[h], w [heads, K, M]; heads ``x_head`` / ``out_head`` elements apart.  ``rows`` names rows of x (lists=1) or
+    of out (lists=2); ``tail`` elements behind x's K are copied behind out's M."""
+    H, K, M = w.shape
+    _check(_lib.rows().sfb_rows_head_proj(*_strides(x), c_int64(x_head), _p(w), *_strides(out), c_int64(out_head), _p(rows), c_int(lists if rows is not None else 0),
+                                          c_int(n), c_int(H), c_int(K), c_int(M), c_int(tail), _fp32(w), _stream()), "rows_head_proj")
+
+
+def gather_pages(pool, pages, out, count, status):
+    nbytes = pool.stride(0) * pool.element_size()
+    _check(_lib.rows().sfb_rows_gather_pages(_p(pool), _p(pages), _p(out), c_int(count), c_int64(nbytes), c_int(pool.shape[0]), _p(status), _stream()),
+           "rows_gather_pages")
 
 
 def sample(logits, row_pos, temperature, seed, mask, best_val, best_id, n):
@@ -88,15 +155,15 @@ def _gemv_takes(x: torch.Tensor) -> bool:
     return x.dtype == torch.bfloat16 and n <= GEMV_ROWS and K % 8 == 0 and (n if n < 3 else 4) * K * 2 <= 200 * 1024
 
 
-def _gemv(x, w, b, out, silu: bool) -> None:
+def _gemv(x, w, b, out, act: int = 0) -> None:
     _check(_lib.rows().sfb_rows_gemv(_p(w), _p(x), _p(b), _p(out), c_int(x.shape[0]), c_int(out.shape[1]), c_int(x.shape[1]),
-                                     c_int(out.dtype == torch.float32), c_int(silu), _stream()), "rows_gemv")
+                                     c_int(out.dtype == torch.float32), c_int(act), _stream()), "rows_gemv")
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor | None, out: torch.Tensor) -> torch.Tensor:
     """out = x w^T (+ b) with 32-bit accumulation: up to four bf16 rows by the streaming kernel, a library product otherwise."""
     if _gemv_takes(x):
-        _gemv(x, w, b, out, False)
+        _gemv(x, w, b, out)
         return out
     if b is not None:
         torch.addmm(b, x, w.t(), out=out)
@@ -106,13 +173,13 @@ def linear(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor | None, out: torch.
     return out
 
 
-def gated_linear(x: torch.Tensor, w: torch.Tensor, scratch: torch.Tensor | None, out: torch.Tensor) -> torch.Tensor:
-    """out = silu(x wg^T) * (x wu^T), w = wg stacked on wu; ``scratch`` [n, 2 ff] holds both products where they are not fused."""
+def gated_linear(x: torch.Tensor, w: torch.Tensor, scratch: torch.Tensor | None, out: torch.Tensor, act: str = "silu") -> torch.Tensor:
+    """out = act(x wg^T) * (x wu^T), w = wg stacked on wu; ``scratch`` [n, 2 ff] holds both products where they are not fused."""
     if _gemv_takes(x):
-        _gemv(x, w, None, out, True)
+        _gemv(x, w, None, out, ACT[act])
         return out
     linear(x, w, None, scratch)
-    silu_mul(scratch, out, x.shape[0])
+    act_mul(scratch, out, x.shape[0], act)
     return out
 
 
@@ -142,9 +209,9 @@ def block_gates(u: torch.Tensor, wg: torch.Tensor, out: torch.Tensor) -> torch.T
 
 
 def head(x: torch.Tensor, embed: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """32-bit logits of x [rows, width] against the tied table."""
+    """32-bit logits of x [rows, width] against the output table."""
     if _gemv_takes(x):
-        _gemv(x, embed, None, out, False)
+        _gemv(x, embed, None, out)
         return out
     if x.dtype == torch.float32:
         torch.mm(x, embed.t(), out=out)
@@ -192,12 +259,13 @@ def attn_tc_supports(dtype: torch.dtype, dim: int, vdim: int) -> bool:
 
 
 class TensorMap:
-    """A 2-D TMA map over a bf16 tensor seen as [rows, cols], boxes of 64 columns x ``box`` rows."""
+    """A 2-D TMA map over a bf16 tensor seen as [rows, cols] with rows ``stride`` elements apart (cols by default), from element
+    ``first`` on; boxes of 64 columns x ``box`` rows."""
 
-    def __init__(self, t: torch.Tensor, rows: int, cols: int, box: int):
+    def __init__(self, t: torch.Tensor, rows: int, cols: int, box: int, stride: int | None = None, first: int = 0):
         self._raw = (ctypes.c_uint8 * 192)()
         self.ptr = c_void_p((ctypes.addressof(self._raw) + 63) & ~63)
-        rc = _lib.rows().sfb_rows_tmap(self.ptr, c_void_p(t.data_ptr()), c_int64(rows), c_int64(cols), c_int64(cols * 2), c_int(box))
+        rc = _lib.rows().sfb_rows_tmap(self.ptr, c_void_p(t.data_ptr() + 2 * first), c_int64(rows), c_int64(cols), c_int64((stride or cols) * 2), c_int(box))
         if rc:
             raise RuntimeError(f"tensor map over [{rows}, {cols}]: error {rc}")
 
@@ -211,17 +279,49 @@ def attn_pools(kv, index: int, tc: bool):
     return k, v, maps
 
 
-_query_maps: dict[tuple, TensorMap] = {}
+_maps: dict[tuple, TensorMap] = {}
+
+
+def tensor_map(t: torch.Tensor, cols: int, box: int, stride: int | None = None, first: int = 0) -> TensorMap:
+    """The map over all of ``t``'s storage, kept, so that one map serves every step over a scratch buffer."""
+    stride = stride or cols
+    total = t.untyped_storage().nbytes() // 2
+    key = (t.untyped_storage().data_ptr(), total, cols, box, stride, first)
+    m = _maps.get(key)
+    if m is None:
+        base = t if t.storage_offset() == 0 else torch.empty(0, dtype=t.dtype, device=t.device).set_(t.untyped_storage())
+        m = _maps[key] = TensorMap(base, (total - first - cols) // stride + 1, cols, box, stride, first)
+    return m
 
 
 def attn_tc(q, kv, table, row_lane, row_pos, tiles, n_tiles, bias, out, heads, scale, status):
     """Tensor-core arm over runs of rows: ``tiles`` are (row0, rows <= 256) pairs, each inside one segment; kv from attn_pools."""
     k, v, (mk, mv) = kv
-    key = (q.data_ptr(), q.untyped_storage().nbytes(), q.shape[1])
-    mq = _query_maps.get(key)
-    if mq is None:        # over the whole scratch buffer, so that one map serves every step
-        mq = _query_maps[key] = TensorMap(q, q.untyped_storage().nbytes() // (2 * q.shape[1]), q.shape[1], 128)
-    _check(_lib.rows().sfb_rows_attn_tc(mq.ptr, mk.ptr, mv.ptr, _p(table), _p(row_lane), _p(row_pos), _p(tiles), c_int(n_tiles), _p(bias),
+    mq = tensor_map(q, q.shape[1], 128)
+    G = k.shape[1]
+    _check(_lib.rows().sfb_rows_attn_tc(mq.ptr, mk.ptr, mv.ptr, None, _p(table), _p(row_lane), _p(row_pos), _p(tiles), None, c_int(n_tiles), _p(bias),
                                         c_int64(bias.shape[1] if bias is not None else 0), _p(out), c_int(table.shape[1]), c_int(k.shape[0]),
-                                        c_int(heads), c_int(k.shape[1]), c_int(k.shape[3]), c_int(v.shape[3]), c_float(scale), _p(status), _stream()),
-           "rows_attn_tc")
+                                        c_int(heads), c_int(G), c_int(k.shape[3]), c_int(v.shape[3]), c_int(0), c_int(G * 64), c_int(64),
+                                        c_int(NO_WINDOW), c_float(scale), _p(status), _stream()), "rows_attn_tc")
+
+
+def latent_tc_supports(dtype: torch.dtype, dim: int, rot: int, vdim: int, rank: int) -> bool:
+    return attn_tc_supports(dtype, dim, vdim) and rot % 8 == 0 and 0 < rot <= 64 and rank % 8 == 0
+
+
+def expand(c: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """out [heads, rows, M] = c [rows, K] times w [heads, K, M] of every head."""
+    torch.bmm(c.unsqueeze(0).expand(w.shape[0], -1, -1), w, out=out)
+    note("linear")
+    return out
+
+
+def latent_attn_tc(q, q_stride, kx, vx, rows, rank, row_pos, tiles, offs, n_tiles, out, heads, dim, rot, vdim, window, scale, status):
+    """Tensor-core arm over keys kx [heads, m, dim] and values vx [heads, m, vdim] that were multiplied out, and the shared key part: the
+    last columns of ``rows`` [m, rank + rot].  q: [n, q_stride] with a head's dim + rot columns side by side."""
+    m = kx.shape[1]
+    mq, mk, mv = tensor_map(q, heads * (dim + rot), 128, q_stride), tensor_map(kx, dim, 64), tensor_map(vx, vdim, 64)
+    mr = tensor_map(rows, rot, 64, rank + rot, rank)
+    _check(_lib.rows().sfb_rows_attn_tc(mq.ptr, mk.ptr, mv.ptr, mr.ptr, None, None, _p(row_pos), _p(tiles), _p(offs), c_int(n_tiles), None, c_int64(0),
+                                        _p(out), c_int(0), c_int(m // 64), c_int(heads), c_int(heads), c_int(dim), c_int(vdim), c_int(rot), c_int(64),
+                                        c_int(m), c_int(window), c_float(scale), _p(status), _stream()), "rows_attn_tc")

@@ -102,7 +102,7 @@ def work(cfg: FanodraConfig, n: int, ctx: int, head_rows: int, decode: bool) -> 
     """Bytes that must move and FLOPs that must be done by a step of n rows that ends at ``ctx`` cached positions (prefill: one
     segment; decode: one row in each of n lanes), per launch name."""
     d, W = cfg.width, roofline.ClassWork
-    out = {k: W() for k in ("rows_seam", "rows_conv", "rows_scan", "rows_gated_step", "rows_qk_append", "rows_attn", "rows_attn_tc", "rows_silu_mul",
+    out = {k: W() for k in ("rows_seam", "rows_conv", "rows_scan", "rows_gated_step", "rows_qk_append", "rows_attn", "rows_attn_tc", "rows_act_mul",
                             "linear", "block_gates", "head")}
 
     def linear(k, m):
@@ -138,7 +138,7 @@ def work(cfg: FanodraConfig, n: int, ctx: int, head_rows: int, decode: bool) -> 
         if L.ff is not None:
             linear(d, 2 * L.ff)
             linear(L.ff, d)
-            out["rows_silu_mul"].bytes += n * L.ff * 6.0
+            out["rows_act_mul"].bytes += n * L.ff * 6.0
             out["rows_seam"].bytes += n * d * 12.0
     out["head"].flops += 2.0 * head_rows * cfg.vocab * d
     out["head"].bytes += 2.0 * cfg.vocab * d

@@ -88,14 +88,14 @@ def test_conv_portions_carry_their_inputs(dt, taps, C):
         x = torch.cat(parts).to("cuda", dt)
         y = torch.empty_like(x)
         for _ in range(2):          # a repeated launch gives the same result
-            R.conv(x, W, B, y, hist, seg, len(x), residual=False)
+            R.conv(x, W, B, y, hist, seg, len(x))
         for k, p in zip(live, y.float().cpu().split([len(p) for p in parts])):
             got[k].append(p); ver[k] ^= 1
     for k in range(3):
         assert (torch.cat(got[k]) - P.causal_conv(xs[k], w, b)).abs().max() < 2 * _tol(dt)
     x = xs[0].to("cuda", dt)
     y = torch.empty_like(x)
-    R.conv(x, W, None, y, hist, _segs([29], [-1], [0]), 29, residual=True)
+    R.conv(x, W, None, y, hist, _segs([29], [-1], [0]), 29, R.CONV_RESIDUAL)
     assert (y.float().cpu() - (xs[0] + P.causal_conv(xs[0], w))).abs().max() < 3 * _tol(dt)
 
 
@@ -124,7 +124,7 @@ def test_gated_recurrence_chunks_and_single_rows(dt, parts, bs, taps):
         x, y = c(torch.cat(parts_x), dt), c(torch.cat(parts_y), dt)
         n = len(x)
         u, o, gates = torch.empty_like(x), torch.empty_like(x), torch.empty(parts, n, 2 * bs, device="cuda")
-        R.conv(x, W, B, u, hist, seg, n, residual=False)
+        R.conv(x, W, B, u, hist, seg, n)
         for _ in range(2):          # a repeated launch gives the same result
             with R.exact_matmul():
                 R.block_gates(u, wg, gates)
