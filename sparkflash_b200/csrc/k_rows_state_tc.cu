@@ -1,0 +1,467 @@
+// The matrix-state recurrence of k_rows_state.cu for long runs of rows, on tcgen05: S_t = a_t S_(t-1) + w_t k_t v_t^T, y_t = S_t^T q_t + D v_t.
+//
+// A run is cut into chunks of 128 rows.  With c_t the running sum of log a inside a chunk and S_0 the state at its start,
+//
+//   y_i = sum_{j <= i} exp(c_i - c_j) w_j (q_i . k_j) v_j + exp(c_i) S_0^T q_i + D v_i,
+//   S_0 of the next chunk = exp(c_last) S_0 + sum_j exp(c_last - c_j) w_j k_j v_j^T
+//
+//   state_turn     rotated (and scaled) q and k as two bf16 terms each, where the recurrence turns them
+//   chunk_sums     the sum in the second line of every (chunk, head):  K^T (weight V)
+//   chunk_starts   S_0 of every chunk, element by element along the run, as two bf16 terms; the run's final state, 32-bit
+//   chunk_out      the first line: scores Q K^T, weighted in registers, back through tensor memory for the product with V; Q S_0 beside it
+//
+// Inputs are bf16.  Everything else that enters a product is a 32-bit value taken as two bf16 terms (16 mantissa bits): weighted scores,
+// weighted values, states, turned q and k.  Accumulators, decays, weights and states are 32-bit.  Every wait is bounded and reports
+// through the status word; no cluster, no multicast.
+#include "k_rows_tc.cuh"
+
+namespace sfb {
+namespace rst {
+using namespace tc;
+
+constexpr int L = 128, SLAB = L * 128, HSLAB = 64 * 128, THREADS = 256;      // rows of a chunk; bytes of 128 / 64 rows of 64 elements
+
+struct Args {
+  const int *c_row0, *c_rows;      // chunks
+  const int *seg, *first;          // runs: segment, first chunk (one entry more than runs)
+  const int *seg_src, *seg_dst;
+  const __nv_bfloat16* dt;         // [n, dt_stride] raw step sizes or null
+  int64_t dt_stride;
+  const float *dt_bias, *a;        // [H]: A with dt, else the logarithm of the decay
+  const float* D;                  // [H] or null
+  float* S;                        // [slots, H, P, Np]
+  float* sums;                     // [chunks, H, P, Np]
+  float* dec;                      // [chunks, H] decay over the whole chunk
+  __nv_bfloat16* starts;           // [2, chunks, H, P, Np]: upper terms, then lower terms
+  __nv_bfloat16* y;                // [n, H P]
+  int H, G, N, P, Np, ns, terms;   // ns: 64-element slabs of a q / k row
+  int q_col, k_col, v_col;         // first columns in the maps
+  int q_lo, k_lo;                  // distance to the columns of the lower terms
+  int chunks;
+  Status* status;
+};
+
+struct Ctl {
+  float c[L], w[L];                // running sum of log2 a, weight
+  float part[4];
+  uint64_t full[3], done;
+  uint32_t tmem;
+  int dead;
+};
+
+// running sums and weights of the chunk's rows (the first 128 threads); past the end: decay 1, weight 0
+__device__ __forceinline__ void chunk_decays(const Args& a, Ctl& C, int h, int row0, int rows) {
+  const int t = threadIdx.x, lane = t & 31, warp = t >> 5;
+  float la = 0.f, w = 0.f;
+  if (t < L) {
+    if (t < rows) {
+      if (a.dt) {
+        const float z = __bfloat162float(a.dt[(size_t)(row0 + t) * a.dt_stride + h]) + a.dt_bias[h];
+        w = log1pf(expf(-fabsf(z))) + fmaxf(z, 0.f);
+        la = a.a[h] * w * LOG2E;
+      } else {
+        w = 1.f;
+        la = a.a[h] * LOG2E;
+      }
+    }
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) { const float v = __shfl_up_sync(0xffffffffu, la, o); if (lane >= o) la += v; }
+    if (lane == 31) C.part[warp] = la;
+  }
+  __syncthreads();
+  if (t < L) {
+    for (int i = 0; i < warp; ++i) la += C.part[i];
+    C.c[t] = la;
+    C.w[t] = w;
+  }
+  __syncthreads();
+}
+
+__device__ __forceinline__ void setup(Ctl& C, uint32_t cols) {
+  if (threadIdx.x == 0) {
+    C.dead = 0;
+    for (int i = 0; i < 3; ++i) mbar_init(&C.full[i], 1);
+    mbar_init(&C.done, 1);
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (threadIdx.x < 32) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&C.tmem)), "r"(cols) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
+  fence_before();
+  __syncthreads();
+  fence_after();
+}
+__device__ __forceinline__ void teardown(Ctl& C, uint32_t cols, Status* status, int where) {
+  fence_before();
+  __syncthreads();
+  if (threadIdx.x == 0 && C.dead) status_set(status, ST_TIMEOUT, where, blockIdx.x, blockIdx.y);
+  if (threadIdx.x < 32) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(C.tmem), "r"(cols) : "memory");
+}
+
+// copies that were issued must land before the CTA ends
+__device__ __forceinline__ void drain(Ctl& C, int bar, uint32_t parity) {
+  if (threadIdx.x == 0)
+    for (int i = 0; i < 100000 && !mbar_try(&C.full[bar], parity); ++i) __nanosleep(64);
+}
+
+__global__ void __launch_bounds__(THREADS)
+chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv, Args a) {
+  extern __shared__ uint8_t raw[];
+  uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
+  __shared__ Ctl C;
+  const int nb = (a.ns + 1) / 2;                          // blocks of 128 state rows
+  uint8_t* ks = sm;                                       // [terms][2 nb] slabs
+  uint8_t* vh = ks + (size_t)a.terms * 2 * nb * SLAB;     // weighted values, upper terms (the copy lands here), lower terms
+  uint8_t* vl = vh + SLAB;
+  setup(C, 128);
+  pdl_launch_dependents();
+  pdl_wait();
+  const int chunk = blockIdx.y, h = blockIdx.x, g = h / (a.H / a.G), row0 = a.c_row0[chunk], rows = a.c_rows[chunk];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, pts = (a.P + 63) / 64;
+  volatile int* dead = &C.dead;
+  if (warp == 0 && elect_one()) {
+    mbar_expect(&C.full[0], a.terms * a.ns * SLAB);
+    for (int t = 0; t < a.terms; ++t)
+      for (int s = 0; s < a.ns; ++s) tma2d(ks + (size_t)(t * 2 * nb + s) * SLAB, &mk, a.k_col + t * a.k_lo + g * a.N + 64 * s, row0, &C.full[0]);
+    mbar_expect(&C.full[1], SLAB);
+    tma2d(vh, &mv, a.v_col + h * a.P, row0, &C.full[1]);
+  }
+  chunk_decays(a, C, h, row0, rows);
+  const float last = C.c[L - 1];
+  if (tid == 0) a.dec[(size_t)chunk * a.H + h] = ex2(last);
+  const uint32_t id = idesc(64, 1, 1);
+  bool ok = true, k_seen = false;
+  for (int pt = 0; pt < pts && ok; ++pt) {
+    ok = __syncthreads_and(mbar_wait(&C.full[1], pt & 1, dead));
+    if (!ok) break;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int u = tid + i * THREADS, r = u >> 3;                   // a 16-byte unit and its row
+      const float wt = ex2(last - C.c[r]) * C.w[r];
+      float f[8];
+      uint4 hi, lo;
+      rows::load_v<__nv_bfloat16, 8>(reinterpret_cast<const __nv_bfloat16*>(vh) + u * 8, f);
+#pragma unroll
+      for (int k = 0; k < 8; ++k) f[k] *= wt;
+      split2(f[0], f[1], hi.x, lo.x); split2(f[2], f[3], hi.y, lo.y); split2(f[4], f[5], hi.z, lo.z); split2(f[6], f[7], hi.w, lo.w);
+      reinterpret_cast<uint4*>(vh)[u] = hi;
+      reinterpret_cast<uint4*>(vl)[u] = lo;
+    }
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    fence_before();
+    if (!k_seen) ok = mbar_wait(&C.full[0], 0, dead);
+    k_seen = true;
+    ok = __syncthreads_and(ok);
+    if (!ok) break;
+    fence_after();
+    if (warp == 0 && elect_one()) {
+      const uint64_t dh = desc(smem_u32(vh), SLAB), dl = desc(smem_u32(vl), SLAB);
+      for (int b = 0; b < nb; ++b) {
+        const uint64_t k0 = desc(smem_u32(ks) + (2 * b) * SLAB, SLAB), k1 = desc(smem_u32(ks) + (2 * nb + 2 * b) * SLAB, SLAB);
+        for (int t = 0; t < 8; ++t) {
+          const uint64_t o = (uint64_t)t * (2048 >> 4);
+          mma_ss(C.tmem + b * 64, k0 + o, dh + o, id, t ? 1u : 0u);
+          mma_ss(C.tmem + b * 64, k0 + o, dl + o, id, 1u);
+          if (a.terms > 1) mma_ss(C.tmem + b * 64, k1 + o, dh + o, id, 1u);
+        }
+      }
+      commit(&C.done);
+    }
+    ok = __syncthreads_and(mbar_wait(&C.done, pt & 1, dead));
+    if (!ok) break;
+    fence_after();
+    if (pt + 1 < pts && warp == 0 && elect_one()) {
+      mbar_expect(&C.full[1], SLAB);
+      tma2d(vh, &mv, a.v_col + h * a.P + 64 * (pt + 1), row0, &C.full[1]);
+    }
+    // lane = state row: columns of the tile go out as runs of consecutive state rows
+    const int w4 = warp & 3, half = warp >> 2;
+    for (int b = 0; b < nb; ++b) {
+      float f[32];
+      ld32(C.tmem + b * 64 + half * 32 + ((uint32_t)(w4 * 32) << 16), f);
+      wait_ld();
+      const int n = b * 128 + w4 * 32 + lane;
+      if (n < a.Np) {
+        float* o = a.sums + (((size_t)chunk * a.H + h) * a.P + pt * 64 + half * 32) * a.Np + n;
+        const int cols = min(32, a.P - pt * 64 - half * 32);
+#pragma unroll
+        for (int c = 0; c < 32; ++c)
+          if (c < cols) o[(size_t)c * a.Np] = n < a.N ? f[c] : 0.f;
+      }
+    }
+    fence_before();
+  }
+  if (C.dead) { drain(C, 0, 0); drain(C, 1, 0); drain(C, 1, 1); }
+  teardown(C, 128, a.status, 69);
+}
+
+// grid (elements / 1024, runs): a thread follows four elements through the run's chunks
+constexpr int AHEAD = 4;
+__global__ void __launch_bounds__(256) chunk_starts_kernel(Args a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const size_t per = (size_t)a.H * a.P * a.Np, e = ((size_t)blockIdx.x * 256 + threadIdx.x) * 4;
+  if (e >= per) return;
+  const int h = (int)(e / ((size_t)a.P * a.Np)), run = blockIdx.y, seg = a.seg[run], c0 = a.first[run], c1 = a.first[run + 1];
+  const int src = a.seg_src[seg];
+  float4 S = src >= 0 ? *reinterpret_cast<const float4*>(a.S + (size_t)src * per + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+  __nv_bfloat16 *hi = a.starts + e, *lo = a.starts + (size_t)a.chunks * per + e;
+  float4 E[AHEAD];
+  float d[AHEAD];
+#pragma unroll
+  for (int i = 0; i < AHEAD; ++i)
+    if (c0 + i < c1) { E[i] = *reinterpret_cast<const float4*>(a.sums + (size_t)(c0 + i) * per + e); d[i] = a.dec[(size_t)(c0 + i) * a.H + h]; }
+  for (int c = c0; c < c1; c += AHEAD) {
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+      if (c + i >= c1) break;
+      const float4 x = E[i];
+      const float dd = d[i];
+      if (c + i + AHEAD < c1) {
+        E[i] = *reinterpret_cast<const float4*>(a.sums + (size_t)(c + i + AHEAD) * per + e);
+        d[i] = a.dec[(size_t)(c + i + AHEAD) * a.H + h];
+      }
+      uint2 u, v;
+      split2(S.x, S.y, u.x, v.x);
+      split2(S.z, S.w, u.y, v.y);
+      *reinterpret_cast<uint2*>(hi + (size_t)(c + i) * per) = u;
+      *reinterpret_cast<uint2*>(lo + (size_t)(c + i) * per) = v;
+      S.x = fmaf(dd, S.x, x.x); S.y = fmaf(dd, S.y, x.y); S.z = fmaf(dd, S.z, x.z); S.w = fmaf(dd, S.w, x.w);
+    }
+  }
+  *reinterpret_cast<float4*>(a.S + (size_t)a.seg_dst[seg] * per + e) = S;
+}
+
+__global__ void __launch_bounds__(THREADS)
+chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv,
+                 const __grid_constant__ CUtensorMap ms, Args a) {
+  extern __shared__ uint8_t raw[];
+  uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
+  __shared__ Ctl C;
+  uint8_t* qs = sm;                                      // [terms][ns] slabs
+  uint8_t* ks = qs + (size_t)a.terms * a.ns * SLAB;
+  uint8_t* vs = ks + (size_t)a.terms * a.ns * SLAB;      // one slab
+  uint8_t* ss = vs + SLAB;                               // start state, [2][ns] slabs of 64 rows
+  setup(C, 256);
+  pdl_launch_dependents();
+  pdl_wait();
+  const int chunk = blockIdx.y, h = blockIdx.x, g = h / (a.H / a.G), row0 = a.c_row0[chunk], rows = a.c_rows[chunk];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, pts = (a.P + 63) / 64, w4 = warp & 3, half = warp >> 2;
+  volatile int* dead = &C.dead;
+  const uint32_t tp = C.tmem, ta = tp + 128, tb = tp + 192, lanes = (uint32_t)(w4 * 32) << 16;
+  auto tile = [&](int pt) {                              // values and start state of a tile of 64 value dims
+    mbar_expect(&C.full[1], SLAB + 2 * a.ns * HSLAB);
+    tma2d(vs, &mv, a.v_col + h * a.P + 64 * pt, row0, &C.full[1]);
+    const int y = (chunk * a.H + h) * a.P + 64 * pt;
+    for (int t = 0; t < 2; ++t)
+      for (int s = 0; s < a.ns; ++s) tma2d(ss + (size_t)(t * a.ns + s) * HSLAB, &ms, 64 * s, t * a.chunks * a.H * a.P + y, &C.full[1]);
+  };
+  const int kst = a.N / 16;
+  if (warp == 0 && elect_one()) {
+    mbar_expect(&C.full[0], 2 * a.terms * a.ns * SLAB);
+    for (int t = 0; t < a.terms; ++t)
+      for (int s = 0; s < a.ns; ++s) {
+        tma2d(qs + (size_t)(t * a.ns + s) * SLAB, &mq, a.q_col + t * a.q_lo + g * a.N + 64 * s, row0, &C.full[0]);
+        tma2d(ks + (size_t)(t * a.ns + s) * SLAB, &mk, a.k_col + t * a.k_lo + g * a.N + 64 * s, row0, &C.full[0]);
+      }
+    tile(0);
+  }
+  chunk_decays(a, C, h, row0, rows);
+  bool ok = __syncthreads_and(mbar_wait(&C.full[0], 0, dead));
+  const uint64_t lo = (uint64_t)a.ns * (SLAB >> 4), dq = desc(smem_u32(qs), 16), dk = desc(smem_u32(ks), 16);
+  const int i = w4 * 32 + lane;
+  if (ok) {
+    fence_after();
+    if (warp == 0 && elect_one()) {
+      const uint32_t id = idesc(128, 0, 0);
+      for (int t = 0; t < kst; ++t) {
+        const uint64_t o = (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2;
+        mma_ss(tp, dq + o, dk + o, id, t ? 1u : 0u);
+        if (a.terms > 1) {
+          mma_ss(tp, dq + o, dk + lo + o, id, 1u);
+          mma_ss(tp, dq + lo + o, dk + o, id, 1u);
+        }
+      }
+      commit(&C.done);
+    }
+    ok = __syncthreads_and(mbar_wait(&C.done, 0, dead));
+  }
+  if (ok) {
+    fence_after();
+    float s[64];
+    const bool any = w4 * 32 + 31 >= half * 64;          // the warp's rows reach these columns
+    if (any) {
+      ld32(tp + half * 64 + lanes, s);
+      ld32(tp + half * 64 + 32 + lanes, s + 32);
+      wait_ld();
+    }
+    fence_before();
+    __syncthreads();                                     // every score has been read: the weights may take their place
+    fence_after();
+    uint32_t hi[32], lw[32];
+    const float ci = C.c[i];
+#pragma unroll
+    for (int q = 0; q < 32; ++q) {
+      const int j = half * 64 + 2 * q;
+      float x = 0.f, y = 0.f;
+      if (any) {
+        const float2 cj = *reinterpret_cast<const float2*>(C.c + j), wj = *reinterpret_cast<const float2*>(C.w + j);
+        x = j <= i ? s[2 * q] * (ex2(ci - cj.x) * wj.x) : 0.f;
+        y = j + 1 <= i ? s[2 * q + 1] * (ex2(ci - cj.y) * wj.y) : 0.f;
+      }
+      split2(x, y, hi[q], lw[q]);
+    }
+    st16(tp + half * 32 + lanes, hi); st16(tp + half * 32 + 16 + lanes, hi + 16);
+    st16(tp + 64 + half * 32 + lanes, lw); st16(tp + 64 + half * 32 + 16 + lanes, lw + 16);
+    wait_st();
+    fence_before();
+  }
+  const float ei = ex2(C.c[i]), D = a.D ? a.D[h] : 0.f;
+  for (int pt = 0; pt < pts && ok; ++pt) {
+    ok = __syncthreads_and(mbar_wait(&C.full[1], pt & 1, dead));
+    if (!ok) break;
+    fence_after();
+    if (warp == 0 && elect_one()) {
+      const uint32_t ia = idesc(64, 0, 1), ib = idesc(64, 0, 0);
+      const uint64_t dv = desc(smem_u32(vs), SLAB), ds = desc(smem_u32(ss), 16), sl = (uint64_t)a.ns * (HSLAB >> 4);
+      for (int t = 0; t < 16; ++t) mma_ts(ta, tp + (t & 7) * 8 + (t >> 3) * 64, dv + (uint64_t)(t & 7) * (2048 >> 4), ia, t ? 1u : 0u);
+      for (int t = 0; t < kst; ++t) {
+        const uint64_t o = (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, os = (uint64_t)(t >> 2) * (HSLAB >> 4) + (t & 3) * 2;
+        mma_ss(tb, dq + o, ds + os, ib, t ? 1u : 0u);
+        mma_ss(tb, dq + o, ds + sl + os, ib, 1u);
+        if (a.terms > 1) mma_ss(tb, dq + lo + o, ds + os, ib, 1u);
+      }
+      commit(&C.done);
+    }
+    ok = __syncthreads_and(mbar_wait(&C.done, (pt + 1) & 1, dead));
+    if (!ok) break;
+    fence_after();
+    float x[32], z[32], v[32];
+    ld32(ta + half * 32 + lanes, x);
+    ld32(tb + half * 32 + lanes, z);
+    if (a.D) {
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+        rows::load_v<__nv_bfloat16, 8>(reinterpret_cast<const __nv_bfloat16*>(vs + i * 128 + (((half * 4 + u) ^ (i & 7)) * 16)), v + 8 * u);
+    }
+    wait_ld();
+    fence_before();
+    __syncthreads();                                     // tile and accumulators have been read
+    if (pt + 1 < pts && warp == 0 && elect_one()) tile(pt + 1);
+    if (i < rows) {
+      __nv_bfloat16* o = a.y + ((size_t)(row0 + i) * a.H + h) * a.P + pt * 64 + half * 32;
+      const int cols = min(32, a.P - pt * 64 - half * 32);
+#pragma unroll
+      for (int u = 0; u < 4; ++u)
+        if (8 * u < cols) {                              // P is a multiple of eight
+          float f[8];
+#pragma unroll
+          for (int k = 0; k < 8; ++k) {
+            f[k] = fmaf(ei, z[8 * u + k], x[8 * u + k]);
+            if (a.D) f[k] = fmaf(D, v[8 * u + k], f[k]);
+          }
+          rows::store_v<__nv_bfloat16, 8>(o + 8 * u, f);
+        }
+    }
+  }
+  if (C.dead) { drain(C, 0, 0); drain(C, 1, 0); drain(C, 1, 1); }
+  teardown(C, 256, a.status, 70);
+}
+
+// q and k of a row, turned by its position, k scaled: out [n][q hi | q lo | k hi | k lo], each [H, N]
+struct TurnArgs {
+  const __nv_bfloat16 *q, *k;
+  int64_t q_stride, k_stride;
+  const float2* rot;
+  const int* row_pos;
+  __nv_bfloat16* out;
+  int n, H, N, dims;
+  float k_scale;
+};
+__global__ void __launch_bounds__(256) state_turn_kernel(TurnArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x, half = a.dims >> 1, HN = a.H * a.N, N2 = a.N >> 1;
+  const float2* cs = a.rot + (size_t)a.row_pos[row] * half;
+  const __nv_bfloat16 *q = a.q + (size_t)row * a.q_stride, *k = a.k + (size_t)row * a.k_stride;
+  __nv_bfloat16* o = a.out + (size_t)row * 4 * HN;
+  // a thread takes two neighbouring dims of a head (half is even or the pair is handled element by element below)
+  for (int x = blockIdx.y * 256 + threadIdx.x; x < a.H * N2; x += gridDim.y * 256) {
+    const int h = x / N2, d = (x - h * N2) * 2;
+    float qf[2], kf[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const int n = d + e, at = h * a.N + n;
+      qf[e] = __bfloat162float(q[at]);
+      kf[e] = __bfloat162float(k[at]);
+      if (n < a.dims) {
+        const int i = n < half ? n : n - half, p = n < half ? at + half : at - half;
+        const float2 t = cs[i];
+        const float s = n < half ? -t.y : t.y;
+        qf[e] = qf[e] * t.x + __bfloat162float(q[p]) * s;
+        kf[e] = kf[e] * t.x + __bfloat162float(k[p]) * s;
+      }
+      kf[e] *= a.k_scale;
+    }
+    uint32_t qh, ql, kh, kl;
+    split2(qf[0], qf[1], qh, ql);
+    split2(kf[0], kf[1], kh, kl);
+    uint32_t* w = reinterpret_cast<uint32_t*>(o + h * a.N + d);
+    w[0] = qh; w[HN / 2] = ql; w[HN] = kh; w[HN + HN / 2] = kl;
+  }
+}
+
+static size_t sums_smem(const Args& a) { return (size_t)(a.terms * 2 * ((a.ns + 1) / 2) + 2) * SLAB + 1024; }
+static size_t out_smem(const Args& a) { return (size_t)(2 * a.terms * a.ns + 1) * SLAB + (size_t)2 * a.ns * HSLAB + 1024; }
+
+}  // namespace rst
+}  // namespace sfb
+
+using namespace sfb;
+using namespace sfb::rst;
+
+extern "C" {
+
+int sfb_rows_state_turn(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* rot, const int* row_pos, void* out, int n, int H, int N,
+                        int dims, float k_scale, cudaStream_t stream) {
+  if (n < 1 || N < 2 || N % 2 || dims % 2 || dims > N) return (int)cudaErrorInvalidValue;
+  TurnArgs a{(const __nv_bfloat16*)q, (const __nv_bfloat16*)k, q_stride, k_stride, (const float2*)rot, row_pos, (__nv_bfloat16*)out, n, H, N, dims, k_scale};
+  return (int)sfb_launch(state_turn_kernel, dim3(n, (H * N / 2 + 1023) / 1024), dim3(256), 0, stream, a);
+}
+
+// mq, mk: rows of q / k terms, box 128 rows; mv: values, box 128 rows; ms: starts seen as [2 chunks H P, Np], box 64 rows.  N: a multiple of
+// 16 up to 256 (128 with two terms); P: a multiple of 8; first columns multiples of 8.
+int sfb_rows_state_tc(const void* mq, const void* mk, const void* mv, const void* ms, const int* c_row0, const int* c_rows, const int* seg, const int* first,
+                      const int* seg_src, const int* seg_dst, const void* dt, int64_t dt_stride, const void* dt_bias, const void* la, const void* D, void* S,
+                      void* sums, void* dec, void* starts, void* y, int runs, int chunks, int H, int G, int N, int P, int Np, int terms, int q_col, int k_col,
+                      int v_col, int q_lo, int k_lo, void* status, cudaStream_t stream) {
+  const int ns = (N + 63) / 64;
+  if (runs < 1 || runs > 65535 || chunks < 1 || chunks > 65535 || G < 1 || H % G || N % 16 || P % 8 || ns > (terms > 1 ? 2 : 4) || Np < N || Np % 32 ||
+      terms < 1 || terms > 2 || (q_col | k_col | v_col | q_lo | k_lo | N) % 8)
+    return (int)cudaErrorInvalidValue;
+  Args a{c_row0, c_rows, seg, first, seg_src, seg_dst, (const __nv_bfloat16*)dt, dt_stride, (const float*)dt_bias, (const float*)la, (const float*)D, (float*)S,
+         (float*)sums, (float*)dec, (__nv_bfloat16*)starts, (__nv_bfloat16*)y, H, G, N, P, Np, ns, terms, q_col, k_col, v_col, q_lo, k_lo, chunks,
+         (Status*)status};
+  const size_t s1 = sums_smem(a), s2 = out_smem(a);
+  static size_t g1 = 0, g2 = 0;
+  if (s1 > g1) {
+    const cudaError_t e = cudaFuncSetAttribute(chunk_sums_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
+    if (e != cudaSuccess) return (int)e;
+    g1 = s1;
+  }
+  if (s2 > g2) {
+    const cudaError_t e = cudaFuncSetAttribute(chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2);
+    if (e != cudaSuccess) return (int)e;
+    g2 = s2;
+  }
+  const CUtensorMap *q = (const CUtensorMap*)mq, *k = (const CUtensorMap*)mk, *v = (const CUtensorMap*)mv, *s = (const CUtensorMap*)ms;
+  cudaError_t rc = sfb_launch(chunk_sums_kernel, dim3(H, chunks), dim3(THREADS), s1, stream, *k, *v, a);
+  if (rc != cudaSuccess) return (int)rc;
+  const size_t per = (size_t)H * P * Np;
+  rc = sfb_launch(chunk_starts_kernel, dim3((unsigned)((per / 4 + 255) / 256), runs), dim3(256), 0, stream, a);
+  if (rc != cudaSuccess) return (int)rc;
+  return (int)sfb_launch(chunk_out_kernel, dim3(H, chunks), dim3(THREADS), s2, stream, *q, *k, *v, *s, a);
+}
+
+}  // extern "C"

@@ -414,6 +414,10 @@ class LayeredEngine:
         """Most rows of a step that do not go to the tensor-core arm."""
         return self.max_lanes * TC_MIN_ROWS if tc else self.max_rows
 
+    def state_chunks(self) -> int:
+        """Most chunks of the tensor-core recurrence in a step: a run's last one may be short."""
+        return self.max_rows // STATE_CHUNK + min(self.max_lanes, max(1, self.max_rows // TC_MIN_ROWS))
+
     def expanded_rows(self, window: int) -> int:
         """Most positions whose keys the long runs of a step need: their own and a window before each run, in whole pages."""
         runs = min(self.max_lanes, max(1, self.max_rows // TC_MIN_ROWS))

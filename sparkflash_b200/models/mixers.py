@@ -195,23 +195,43 @@ def rotation_table(base: float, dims: int, length: int, device) -> torch.Tensor:
 
 class MatrixState:
     """S_t = a_t S_(t-1) + w_t k_t v_t^T, y_t = S_t^T q_t + D v_t: one 32-bit state [P, N] and one decay per head, q and k shared by
-    groups of heads.  Decay and input weight come from a step size per token (a = exp(A dt), w = dt), or the decay is a constant."""
+    groups of heads.  Decay and input weight come from a step size per token (a = exp(A dt), w = dt; ``decay`` is A), or the decay is a
+    constant.  q and k may be turned by their position (``rot``) and k scaled.  Long runs of bf16 rows take the tensor-core arm."""
 
-    def __init__(self, heads: int, groups: int, n: int, p: int, decay: torch.Tensor, dt_bias=None, skip=None, rot=None, rot_dims: int = 0,
-                 k_scale: float = 1.0):
+    def __init__(self, heads: int, groups: int, n: int, p: int, decay: torch.Tensor, dtype: torch.dtype, dt_bias=None, skip=None, rot=None,
+                 rot_dims: int = 0, k_scale: float = 1.0):
         self.H, self.G, self.N, self.P = heads, groups, n, p
+        self.log_decay = decay if dt_bias is not None else torch.log(decay.double()).float().contiguous()
         self.decay, self.dt_bias, self.skip, self.rot, self.rot_dims, self.k_scale = decay, dt_bias, skip, rot, rot_dims, k_scale
-        self.tc = False
+        self.terms = 2 if rot is not None else 1
+        self.tc = R.state_tc_supports(dtype, n, p, self.terms)
 
     def state(self, e, tag: str) -> torch.Tensor:
         return e.state.add(tag, (self.H, self.P, R.state_pad(self.N)), torch.float32)
 
-    def reserve(self, e, dtype) -> None:
-        pass
+    def reserve(self, e) -> None:
+        if self.tc:
+            chunks = e.state_chunks()
+            per = self.H * self.P * R.state_pad(self.N)
+            e.scratch.reserve("state_sums", chunks * per, torch.float32)
+            e.scratch.reserve("state_starts", 2 * chunks * per, torch.bfloat16)
+            e.scratch.reserve("state_dec", chunks * self.H, torch.float32)
+            if self.terms > 1:
+                e.scratch.reserve("state_turned", e.max_rows * 4 * self.H * self.N, torch.bfloat16)
 
-    def run(self, s, q, k, v, dt, S, y, conv=None) -> None:
-        R.state_rows(q, k, v, dt, self.dt_bias, self.decay, self.skip, self.rot, self.rot_dims, self.k_scale, s.row_pos, y, S, self.N, self.G, s.short_segs,
-                     s.nshort, s, conv)
+    def run(self, s, src, cols, dt, S, y, conv=None) -> None:
+        """``src`` [n, stride] holds q, k, v from the columns ``cols`` on; ``conv``: they are the inputs of a convolution, see R.state_rows."""
+        q, k, v = (src[:, c:] for c in cols)
+        if s.nshort:
+            R.state_rows(q, k, v, dt, self.dt_bias, self.decay, self.skip, self.rot, self.rot_dims, self.k_scale, s.row_pos, y, S, self.N, self.G,
+                         s.short_segs, s.nshort, s, conv)
+        if s.nlong:
+            hn, qk, at = self.H * self.N, src, (cols[0], cols[1], 0, 0)
+            if self.terms > 1:
+                qk, at = s.scratch.get("state_turned", s.n, 4 * hn), (0, 2 * hn, hn, hn)
+                R.state_turn(q, k, self.rot, self.rot_dims, self.k_scale, s.row_pos, qk, s.n, self.H, self.N)
+            R.state_tc(qk, at, src, cols[2], dt, self.dt_bias, self.log_decay, self.skip, S, s.scratch.buf["state_sums"], s.scratch.buf["state_dec"],
+                       s.scratch.buf["state_starts"], y, self.N, self.G, s, self.terms, s.status)
 
 
 class StateSpaceMixer:
@@ -226,7 +246,7 @@ class StateSpaceMixer:
         self.w_in, self.w_out = w.act("in", pad=8), w.act("o")
         self.cw, self.cb, self.norm = w.taps("conv"), w.f32("conv.b"), w.f32("norm")
         A = -torch.exp(w.t[w.p + "A_log"].to(w.device, torch.float64)).to(torch.float32)
-        self.core = MatrixState(H, G, N, P, A.contiguous(), w.f32("dt_bias"), w.f32("D"))
+        self.core = MatrixState(H, G, N, P, A.contiguous(), w.dtype, w.f32("dt_bias"), w.f32("D"))
         self.merge, self.kv_run = (None, None), None
 
     def reserve(self, e) -> None:
@@ -235,7 +255,7 @@ class StateSpaceMixer:
         e.scratch.reserve("mix_u", n * self.channels, dt)
         e.scratch.reserve("mix_y", n * self.inner, dt)
         e.scratch.reserve("mix_o", n * self.inner, dt)
-        self.core.reserve(e, dt)
+        self.core.reserve(e)
 
     def bind_run(self, e, tag: str, kv_index):
         return {"conv": e.state.add(tag + ".conv", (self.taps - 1, self.channels), self.w_in.dtype), "S": self.core.state(e, tag + ".S")}
@@ -249,7 +269,7 @@ class StateSpaceMixer:
         if conv is None:
             raw, u = u, s.scratch.get("mix_u", n, self.channels)
             R.conv(raw, self.cw, self.cb, u, run["conv"], s, n, R.CONV_SILU)
-        self.core.run(s, u[:, i + bc:], u[:, i:i + bc], u[:, :i], dt, run["S"], y, conv)
+        self.core.run(s, u, (i + bc, i, 0), dt, run["S"], y, conv)
         o = s.scratch.get("mix_o", n, i)
         R.gated_norm(y, z, self.norm, o, self.part, True, self.eps)
         return R.linear(o, self.w_out, None, s.scratch.get("y", n, h.shape[1])), None
@@ -266,7 +286,7 @@ class RetentionMixer:
         self.inner, self.qk, self.P, self.eps = H * P, H * N, P, eps
         self.w_in, self.w_out = w.act(*self.PROJ, pad=8), w.act("o")
         decay = torch.tensor(spec["decay"], dtype=torch.float64).to(w.device, torch.float32)
-        self.core = MatrixState(H, H, N, P, decay, rot=rotation_table(rot["base"], rot["dims"], max_context, w.device), rot_dims=rot["dims"],
+        self.core = MatrixState(H, H, N, P, decay, w.dtype, rot=rotation_table(rot["base"], rot["dims"], max_context, w.device), rot_dims=rot["dims"],
                                 k_scale=N ** -0.5)
         self.merge, self.kv_run = (None, None), None
 
@@ -275,7 +295,7 @@ class RetentionMixer:
         e.scratch.reserve("proj", n * self.w_in.shape[0], dt)
         e.scratch.reserve("mix_y", n * self.inner, dt)
         e.scratch.reserve("mix_o", n * self.inner, dt)
-        self.core.reserve(e, dt)
+        self.core.reserve(e)
 
     def bind_run(self, e, tag: str, kv_index):
         return {"S": self.core.state(e, tag + ".S")}
@@ -284,7 +304,7 @@ class RetentionMixer:
         n, i, qk = s.n, self.inner, self.qk
         proj = R.linear(h, self.w_in, None, s.scratch.get("proj", n, self.w_in.shape[0]))
         y, o = s.scratch.get("mix_y", n, i), s.scratch.get("mix_o", n, i)
-        self.core.run(s, proj[:, :qk], proj[:, qk:2 * qk], proj[:, 2 * qk:2 * qk + i], None, run["S"], y)
+        self.core.run(s, proj, (0, qk, 2 * qk), None, run["S"], y)
         R.gated_norm(y, proj[:, 2 * qk + i:2 * qk + 2 * i], None, o, self.P, False, self.eps)
         return R.linear(o, self.w_out, None, s.scratch.get("y", n, h.shape[1])), None
 

@@ -103,6 +103,30 @@ def state_rows(q, k, v, dt, dt_bias, a, D, rot, rot_dims, k_scale, row_pos, y, S
                                       c_int(Np), c_float(k_scale), _fp32(y), _stream()), "rows_state")
 
 
+def state_tc_supports(dtype: torch.dtype, n: int, p: int, terms: int) -> bool:
+    """Shapes the tensor-core arm of the matrix-state recurrence takes (csrc/k_rows_state_tc.cu)."""
+    return dtype == torch.bfloat16 and n % 16 == 0 and n <= (128 if terms > 1 else 256) and p % 8 == 0
+
+
+def state_turn(q, k, rot, rot_dims, k_scale, row_pos, out, n, heads, N):
+    """Turned q and k of every row as two bf16 terms each: out [n, 4 heads N] = q hi | q lo | k hi | k lo."""
+    _check(_lib.rows().sfb_rows_state_turn(*_strides(q), *_strides(k), _p(rot), _p(row_pos), _p(out), c_int(n), c_int(heads), c_int(N), c_int(rot_dims),
+                                           c_float(k_scale), _stream()), "rows_state_turn")
+
+
+def state_tc(qk, qk_cols, v, v_col, dt, dt_bias, log_a, D, S, sums, dec, starts, y, N, groups, seg, terms, status):
+    """Long segments in chunks of 128 rows.  ``qk``: [n, stride] tensor with the columns (q, k, distance to q's and to k's lower terms) of
+    ``qk_cols``; ``v``: [n, stride] tensor with values from column ``v_col`` on; sums, dec, starts: scratch of all chunks."""
+    _, H, P, Np = S.shape
+    mqk, mv = tensor_map(qk, qk.shape[1], 128), tensor_map(v, v.shape[1], 128)
+    ms = tensor_map(starts, Np, 64)
+    qc, kc, ql, kl = qk_cols
+    _check(_lib.rows().sfb_rows_state_tc(mqk.ptr, mqk.ptr, mv.ptr, ms.ptr, _p(seg.long_row0), _p(seg.long_rows), _p(seg.long_seg), _p(seg.long_first),
+                                         _p(seg.seg_src), _p(seg.seg_dst), *_strides(dt), _p(dt_bias), _p(log_a), _p(D), _p(S), _p(sums), _p(dec),
+                                         _p(starts), _p(y), c_int(seg.nlong), c_int(seg.nchunks), c_int(H), c_int(groups), c_int(N), c_int(P), c_int(Np),
+                                         c_int(terms), c_int(qc), c_int(kc), c_int(v_col), c_int(ql), c_int(kl), _p(status), _stream()), "rows_state_tc")
+
+
 STATE_PADS = tuple(range(32, 257, 32)) + (384, 512)
 
 
