@@ -57,7 +57,7 @@ def design_arm(args) -> None:
     sampler.start()
     time.sleep(1.0)
     sampler.mark()
-    sizes = LB.run(args.design_sizes.split(","), args.steps)
+    sizes = LB.run(args.design, args.design_sizes.split(","), args.steps)
     first = sizes[args.design_sizes.split(",")[-1]]["throughput"]
     print(json.dumps({"metric": f"{args.design}: decode tok/s, 16 streams, {args.design_sizes.split(',')[-1]}", "value": first["decode_16"]["tok_s"],
                       "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": 3, "higher_is_better": True, "dtype": "bf16, 32-bit residual / norms / "
@@ -510,7 +510,7 @@ def main() -> None:
     ap.add_argument("--prefill-chunk", type=int, default=4096, help="rows per prompt chunk (the reference prefills 4,096-row chunks)")
     ap.add_argument("--no-mtp", action="store_true", help="skip the DSpark draft-path section")
     ap.add_argument("--no-ep", action="store_true", help="skip the expert-parallel section (2+ GPUs)")
-    ap.add_argument("--design", default="", choices=["", "fanodra"], help="benchmark a layered design instead of the headline model: prefill and "
+    ap.add_argument("--design", default="", choices=["", "fanodra", "gudutar"], help="benchmark a layered design instead of the headline model: prefill and "
                     "decode throughput and per-kernel roofline fractions, beside the closest model (one JSON line)")
     ap.add_argument("--design-sizes", default="w1024,w2048,w4096", help="sizes of --design (sparkflash_b200/utils/layered_bench.py)")
     args = ap.parse_args()

@@ -68,28 +68,76 @@ struct HeadProjArgs {
   void* out;                // (T)
   int64_t out_row, out_head;
   const int* rows;          // row of x (x_list) or of out (out_list) for every launch row, or null: identity
-  int x_list, out_list, n, K, M, tail;      // tail: elements after x's K that are copied after out's M
+  const float *part, *ml;   // or x is to be merged: [launch rows, H, blocks, K] and (log2 maximum, sum) of every block
+  const int* row_pos;
+  int window, blocks;
+  int x_list, out_list, n, H, K, M, tail;   // tail: elements after x's K that are copied after out's M
 };
-constexpr int HP_M = 128, HP_R = 4, HP_T = 128;      // outputs and rows per block; 16 threads x 8 outputs, 8 shares of K
+constexpr int HP_R = 4, HP_T = 256;                    // rows and threads per block
 
-template <typename T, int V>
+// MG threads x 8 outputs side by side, the others share K
+template <typename T, int V, int MG>
 __global__ void __launch_bounds__(HP_T) head_proj_kernel(HeadProjArgs a) {
-  extern __shared__ __align__(16) float sm[];          // x [HP_R][K], then partials [8][HP_R][HP_M]
+  extern __shared__ __align__(16) float sm[];          // x [HP_R][K], then partials [KG][HP_R][HP_M] (before that: merge weights)
+  constexpr int HP_M = MG * 8, KG = HP_T / MG, PRE = 4;
   float* xs = sm;
-  float* red = sm + HP_R * a.K;
-  const int tid = threadIdx.x, mg = tid & 15, kg = tid >> 4;
+  float* red = sm + ((HP_R * a.K + 3) & ~3);
+  const int tid = threadIdx.x, mg = tid % MG, kg = tid / MG;
   const int mt = (a.M + HP_M - 1) / HP_M, h = blockIdx.x / mt, m0 = (blockIdx.x % mt) * HP_M + mg * 8;
   const int r0 = blockIdx.y * HP_R, nr = min(HP_R, a.n - r0);
+  const T* w = (const T*)a.w + (size_t)h * a.K * a.M + m0;
+  auto weights = [&](int k, float (&f)[8]) {
+    if constexpr (V == 8) load_v<T, 8>(w + (size_t)k * a.M, f);
+    else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[j] = m0 + j < a.M ? to_f<T>(w[(size_t)k * a.M + j]) : 0.f;
+    }
+  };
+  // the first weights are requested before the previous kernel has finished: they do not depend on it
+  float pre[PRE][8];
+#pragma unroll
+  for (int p = 0; p < PRE; ++p)
+    if (m0 < a.M && kg + p * KG < a.K) weights(kg + p * KG, pre[p]);
   pdl_launch_dependents();
   pdl_wait();
-  for (int i = tid; i < HP_R * a.K; i += HP_T) {
-    const int r = i / a.K, k = i - r * a.K;
-    float f = 0.f;
-    if (r < nr) {
-      const int row = a.rows && a.x_list ? a.rows[r0 + r] : r0 + r;
-      f = to_f<T>(((const T*)a.x)[(size_t)row * a.x_row + (size_t)h * a.x_head + k]);
+  if (a.part) {
+    float* wt = red;                                   // [HP_R][blocks]
+    const int warp = tid >> 5, lane = tid & 31;
+    if (warp < nr) {
+      const int row = a.rows ? a.rows[r0 + warp] : r0 + warp, pos = a.row_pos[row], first = max(0, pos - a.window + 1);
+      const int nb = min(a.blocks, (pos / 64 - first / 64) / 2 + 1);
+      const float* ml = a.ml + ((size_t)(r0 + warp) * a.H + h) * a.blocks * 2;
+      float m = -INFINITY, l = 0.f;
+      for (int b = lane; b < nb; b += 32) m = fmaxf(m, ml[2 * b]);
+      m = warp_max(m);
+      for (int b = lane; b < nb; b += 32) l += ml[2 * b + 1] * exp2f(ml[2 * b] - m);
+      const float inv = 1.f / warp_sum(l);
+      for (int b = lane; b < a.blocks; b += 32) wt[warp * a.blocks + b] = b < nb ? exp2f(ml[2 * b] - m) * inv : 0.f;
     }
-    xs[i] = f;
+    __syncthreads();
+    for (int i = tid; i < HP_R * a.K; i += HP_T) {
+      const int r = i / a.K, k = i - r * a.K;
+      float f = 0.f;
+      if (r < nr) {
+        const float* p = a.part + ((size_t)(r0 + r) * a.H + h) * a.blocks * a.K + k;
+#pragma unroll 4
+        for (int b = 0; b < a.blocks; ++b) {
+          const float wb = wt[r * a.blocks + b];
+          if (wb != 0.f) f = fmaf(wb, p[(size_t)b * a.K], f);
+        }
+      }
+      xs[i] = f;
+    }
+  } else {
+    for (int i = tid; i < HP_R * a.K; i += HP_T) {
+      const int r = i / a.K, k = i - r * a.K;
+      float f = 0.f;
+      if (r < nr) {
+        const int row = a.rows && a.x_list ? a.rows[r0 + r] : r0 + r;
+        f = to_f<T>(((const T*)a.x)[(size_t)row * a.x_row + (size_t)h * a.x_head + k]);
+      }
+      xs[i] = f;
+    }
   }
   if (a.tail && blockIdx.x % mt == 0) {
     for (int i = tid; i < nr * a.tail; i += HP_T) {
@@ -104,22 +152,23 @@ __global__ void __launch_bounds__(HP_T) head_proj_kernel(HeadProjArgs a) {
   for (int r = 0; r < HP_R; ++r)
 #pragma unroll
     for (int j = 0; j < 8; ++j) acc[r][j] = 0.f;
-  const T* w = (const T*)a.w + (size_t)h * a.K * a.M + m0;
+  auto add = [&](int k, const float (&f)[8]) {
+#pragma unroll
+    for (int r = 0; r < HP_R; ++r) {
+      const float xv = xs[r * a.K + k];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) acc[r][j] = fmaf(xv, f[j], acc[r][j]);
+    }
+  };
   if (m0 < a.M) {
-#pragma unroll 8
-    for (int k = kg; k < a.K; k += 8) {
+#pragma unroll
+    for (int p = 0; p < PRE; ++p)
+      if (kg + p * KG < a.K) add(kg + p * KG, pre[p]);
+#pragma unroll 4
+    for (int k = kg + PRE * KG; k < a.K; k += KG) {
       float f[8];
-      if constexpr (V == 8) load_v<T, 8>(w + (size_t)k * a.M, f);
-      else {
-#pragma unroll
-        for (int j = 0; j < 8; ++j) f[j] = m0 + j < a.M ? to_f<T>(w[(size_t)k * a.M + j]) : 0.f;
-      }
-#pragma unroll
-      for (int r = 0; r < HP_R; ++r) {
-        const float xv = xs[r * a.K + k];
-#pragma unroll
-        for (int j = 0; j < 8; ++j) acc[r][j] = fmaf(xv, f[j], acc[r][j]);
-      }
+      weights(k, f);
+      add(k, f);
     }
   }
 #pragma unroll
@@ -128,15 +177,15 @@ __global__ void __launch_bounds__(HP_T) head_proj_kernel(HeadProjArgs a) {
     *reinterpret_cast<float4*>(red + ((size_t)kg * HP_R + r) * HP_M + mg * 8 + 4) = make_float4(acc[r][4], acc[r][5], acc[r][6], acc[r][7]);
   }
   __syncthreads();
-  const int m = (blockIdx.x % mt) * HP_M + tid;
-  if (m < a.M)
-    for (int r = 0; r < nr; ++r) {
-      float t = 0.f;
+  for (int i = tid; i < nr * HP_M; i += HP_T) {
+    const int r = i / HP_M, c = i - r * HP_M, m = (blockIdx.x % mt) * HP_M + c;
+    if (m >= a.M) continue;
+    float t = 0.f;
 #pragma unroll
-      for (int q = 0; q < 8; ++q) t += red[((size_t)q * HP_R + r) * HP_M + tid];
-      const int row = a.rows && a.out_list ? a.rows[r0 + r] : r0 + r;
-      ((T*)a.out)[(size_t)row * a.out_row + (size_t)h * a.out_head + m] = from_f<T>(t);
-    }
+    for (int q = 0; q < KG; ++q) t += red[((size_t)q * HP_R + r) * HP_M + c];
+    const int row = a.rows && a.out_list ? a.rows[r0 + r] : r0 + r;
+    ((T*)a.out)[(size_t)row * a.out_row + (size_t)h * a.out_head + m] = from_f<T>(t);
+  }
 }
 
 __global__ void __launch_bounds__(256) gather_pages_kernel(const uint4* pool, const int* pages, uint4* out, int words, int n_pages, Status* status) {
@@ -150,16 +199,24 @@ __global__ void __launch_bounds__(256) gather_pages_kernel(const uint4* pool, co
   for (int i = blockIdx.y * 256 + threadIdx.x; i < words; i += gridDim.y * 256) d[i] = s[i];
 }
 
-template <typename T, int V>
-static int launch_head_proj(const HeadProjArgs& a, int H, cudaStream_t st) {
-  const size_t smem = ((size_t)HP_R * a.K + (size_t)8 * HP_R * HP_M) * sizeof(float);
+template <typename T, int V, int MG>
+static int launch_head_proj(const HeadProjArgs& a, cudaStream_t st) {
+  const size_t red = (size_t)HP_T * HP_R * 8, wts = (size_t)HP_R * a.blocks;
+  const size_t smem = (((size_t)HP_R * a.K + 3) / 4 * 4 + (red > wts ? red : wts)) * sizeof(float);
+  if (smem > 220 * 1024) return (int)cudaErrorInvalidValue;
   static size_t granted = 48 * 1024;
   if (smem > granted) {
-    const cudaError_t e = cudaFuncSetAttribute(head_proj_kernel<T, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const cudaError_t e = cudaFuncSetAttribute(head_proj_kernel<T, V, MG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     granted = smem;
   }
-  return (int)sfb_launch(head_proj_kernel<T, V>, dim3(H * ((a.M + HP_M - 1) / HP_M), (a.n + HP_R - 1) / HP_R), dim3(HP_T), smem, st, a);
+  return (int)sfb_launch(head_proj_kernel<T, V, MG>, dim3(a.H * ((a.M + MG * 8 - 1) / (MG * 8)), (a.n + HP_R - 1) / HP_R), dim3(HP_T), smem, st, a);
+}
+template <typename T>
+static int launch_head_proj_t(const HeadProjArgs& a, cudaStream_t st) {
+  if (a.M % 8) return launch_head_proj<T, 1, 16>(a, st);
+  // long sums: fewer outputs per block and more threads on each
+  return a.K > 256 ? launch_head_proj<T, 8, 4>(a, st) : launch_head_proj<T, 8, 16>(a, st);
 }
 
 }  // namespace rows
@@ -178,14 +235,14 @@ int sfb_rows_latent_append(void* proj, int64_t stride, const void* w, const void
                     : sfb_launch(latent_append_kernel<__nv_bfloat16>, dim3(n), dim3(128), 0, stream, a));
 }
 
-// list: 0 = rows ignored, 1 = it names x's rows, 2 = it names out's rows
+// list: 0 = rows ignored, 1 = it names x's rows, 2 = it names out's rows.  part (then x is null): see HeadProjArgs; list is 2 or 0.
 int sfb_rows_head_proj(const void* x, int64_t x_row, int64_t x_head, const void* w, void* out, int64_t out_row, int64_t out_head, const int* rows, int list,
-                       int n, int H, int K, int M, int tail, int fp32, cudaStream_t stream) {
-  if (n < 1 || n > 65535 * HP_R || H < 1 || K < 1 || M < 1 || K > 8192) return (int)cudaErrorInvalidValue;
-  HeadProjArgs a{x, x_row, x_head, w, out, out_row, out_head, list ? rows : nullptr, list == 1, list == 2, n, K, M, tail};
-  const bool v8 = M % 8 == 0;
-  if (fp32) return v8 ? launch_head_proj<float, 8>(a, H, stream) : launch_head_proj<float, 1>(a, H, stream);
-  return v8 ? launch_head_proj<__nv_bfloat16, 8>(a, H, stream) : launch_head_proj<__nv_bfloat16, 1>(a, H, stream);
+                       const void* part, const void* ml, const int* row_pos, int window, int blocks, int n, int H, int K, int M, int tail, int fp32,
+                       cudaStream_t stream) {
+  if (n < 1 || n > 65535 * HP_R || H < 1 || K < 1 || M < 1 || K > 8192 || (part && (blocks < 1 || tail || list == 1))) return (int)cudaErrorInvalidValue;
+  HeadProjArgs a{x, x_row, x_head, w, out, out_row, out_head, list ? rows : nullptr, (const float*)part, (const float*)ml, row_pos, window, part ? blocks : 0,
+                 list == 1, list == 2, n, H, K, M, tail};
+  return fp32 ? launch_head_proj_t<float>(a, stream) : launch_head_proj_t<__nv_bfloat16>(a, stream);
 }
 
 // bytes of a page: a multiple of 16

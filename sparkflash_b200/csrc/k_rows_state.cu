@@ -40,16 +40,26 @@ constexpr int STB = 8;              // rows whose q, k, v are staged together
 __device__ __forceinline__ float softplus_f(float z) { return log1pf(expf(-fabsf(z))) + fmaxf(z, 0.f); }
 
 // the convolution's output at one channel of a single row, rounded to activation precision; `keep`: this block carries the inputs on
+constexpr int ST_TAPS = 4;           // taps requested together
 template <typename T>
 __device__ __forceinline__ float conv_silu(const StateArgs& a, T x, int ch, int src, int dst, bool keep) {
   const int W = a.taps - 1;
-  float acc = a.cb[ch] + a.cw[(size_t)W * a.C + ch] * to_f<T>(x);
   const T* hs = (const T*)a.hist + (size_t)(src >= 0 ? src : 0) * W * a.C + ch;
   T* hd = (T*)a.hist + (size_t)dst * W * a.C + ch;
-  for (int j = 0; j < W; ++j) {
-    const T g = src >= 0 ? hs[(size_t)j * a.C] : from_f<T>(0.f);
-    acc += a.cw[(size_t)j * a.C + ch] * to_f<T>(g);
-    if (keep && j > 0) hd[(size_t)(j - 1) * a.C] = g;
+  float acc = a.cb[ch] + a.cw[(size_t)W * a.C + ch] * to_f<T>(x);
+  for (int j0 = 0; j0 < W; j0 += ST_TAPS) {
+    T gv[ST_TAPS];
+    float w[ST_TAPS];
+#pragma unroll
+    for (int j = 0; j < ST_TAPS; ++j) {
+      gv[j] = src >= 0 && j0 + j < W ? hs[(size_t)(j0 + j) * a.C] : from_f<T>(0.f);
+      w[j] = j0 + j < W ? a.cw[(size_t)(j0 + j) * a.C + ch] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < ST_TAPS; ++j) {
+      acc += w[j] * to_f<T>(gv[j]);
+      if (keep && j0 + j > 0 && j0 + j < W) hd[(size_t)(j0 + j - 1) * a.C] = gv[j];
+    }
   }
   if (keep && W > 0) hd[(size_t)(W - 1) * a.C] = x;
   return to_f<T>(from_f<T>(acc * sigmoid_f(acc)));
@@ -82,16 +92,28 @@ __global__ void __launch_bounds__(256) state_rows_kernel(StateArgs a) {
   for (int t0 = 0; t0 < len; t0 += STB) {
     const int nb = min(STB, len - t0);
     if (t0) __syncthreads();
-    for (int x = tid; x < nb * a.Np; x += blockDim.x) {
-      const int t = x / a.Np, n = x - t * a.Np, row = row0 + t0 + t;
-      float qf = 0.f, kf = 0.f;
-      if (n < a.N) {
-        const T* qp = (const T*)a.q + (size_t)row * a.q_stride + (size_t)g * a.N;
-        const T* kp = (const T*)a.k + (size_t)row * a.k_stride + (size_t)g * a.N;
-        if (a.cw) {
-          qf = conv_silu<T>(a, qp[n], a.q_ch + g * a.N + n, src, dst, keep_g);
-          kf = conv_silu<T>(a, kp[n], a.k_ch + g * a.N + n, src, dst, keep_g);
-        } else {
+    if (a.cw) {                       // one row: channels of q, then k, then the tile's v, one per thread
+      const int span = 2 * a.Np + PT;
+      for (int x = tid; x < span; x += blockDim.x) {
+        const bool isv = x >= 2 * a.Np, isk = !isv && x >= a.Np;
+        const int n = isv ? tile * PT + x - 2 * a.Np : isk ? x - a.Np : x, base = isv ? h * a.P : g * a.N;
+        float f = 0.f;
+        if (n < (isv ? a.P : a.N)) {
+          const T r = isv ? ((const T*)a.v)[(size_t)row0 * a.v_stride + base + n]
+                          : isk ? ((const T*)a.k)[(size_t)row0 * a.k_stride + base + n] : ((const T*)a.q)[(size_t)row0 * a.q_stride + base + n];
+          f = conv_silu<T>(a, r, (isv ? a.v_ch : isk ? a.k_ch : a.q_ch) + base + n, src, dst, isv || keep_g);
+        }
+        if (isv) vs[x - 2 * a.Np] = f;
+        else if (isk) ks[n] = f * a.k_scale;
+        else qs[n] = f;
+      }
+    } else {
+      for (int x = tid; x < nb * a.Np; x += blockDim.x) {
+        const int t = x / a.Np, n = x - t * a.Np, row = row0 + t0 + t;
+        float qf = 0.f, kf = 0.f;
+        if (n < a.N) {
+          const T* qp = (const T*)a.q + (size_t)row * a.q_stride + (size_t)g * a.N;
+          const T* kp = (const T*)a.k + (size_t)row * a.k_stride + (size_t)g * a.N;
           qf = to_f<T>(qp[n]); kf = to_f<T>(kp[n]);
           if (n < a.rot_dims) {
             const int i = n < half ? n : n - half, o = n < half ? n + half : n - half;
@@ -101,17 +123,12 @@ __global__ void __launch_bounds__(256) state_rows_kernel(StateArgs a) {
             kf = kf * cs.x + to_f<T>(kp[o]) * sn;
           }
         }
+        qs[x] = qf; ks[x] = kf * a.k_scale;
       }
-      qs[x] = qf; ks[x] = kf * a.k_scale;
-    }
-    for (int x = tid; x < nb * PT; x += blockDim.x) {
-      const int t = x / PT, c = tile * PT + x - t * PT, row = row0 + t0 + t;
-      float f = 0.f;
-      if (c < a.P) {
-        const T r = ((const T*)a.v)[(size_t)row * a.v_stride + (size_t)h * a.P + c];
-        f = a.cw ? conv_silu<T>(a, r, a.v_ch + h * a.P + c, src, dst, true) : to_f<T>(r);
+      for (int x = tid; x < nb * PT; x += blockDim.x) {
+        const int t = x / PT, c = tile * PT + x - t * PT;
+        vs[x] = c < a.P ? to_f<T>(((const T*)a.v)[(size_t)(row0 + t0 + t) * a.v_stride + (size_t)h * a.P + c]) : 0.f;
       }
-      vs[x] = f;
     }
     if (tid < nb) {
       if (a.dt) {

@@ -37,44 +37,39 @@ struct Args {
   int H, G, N, P, Np, ns, terms;   // ns: 64-element slabs of a q / k row
   int q_col, k_col, v_col;         // first columns in the maps
   int q_lo, k_lo;                  // distance to the columns of the lower terms
-  int chunks;
+  int chunks, hpc;                 // hpc: heads per block
   Status* status;
 };
 
 struct Ctl {
-  float c[L], w[L];                // running sum of log2 a, weight
+  float c[L];                      // running sum of log2 a, less log2 of the weight (chunk_out); weight of a row's values (chunk_sums)
   float part[4];
   uint64_t full[3], done;
   uint32_t tmem;
   int dead;
 };
 
-// running sums and weights of the chunk's rows (the first 128 threads); past the end: decay 1, weight 0
-__device__ __forceinline__ void chunk_decays(const Args& a, Ctl& C, int h, int row0, int rows) {
-  const int t = threadIdx.x, lane = t & 31, warp = t >> 5;
-  float la = 0.f, w = 0.f;
-  if (t < L) {
-    if (t < rows) {
-      if (a.dt) {
-        const float z = __bfloat162float(a.dt[(size_t)(row0 + t) * a.dt_stride + h]) + a.dt_bias[h];
-        w = log1pf(expf(-fabsf(z))) + fmaxf(z, 0.f);
-        la = a.a[h] * w * LOG2E;
-      } else {
-        w = 1.f;
-        la = a.a[h] * LOG2E;
-      }
+// Running sum of log2 a up to the thread's row (thread t: row t & 127) and the row's weight; past the end: decay 1, weight 0.  One barrier.
+__device__ __forceinline__ float chunk_decays(const Args& a, Ctl& C, int h, int row0, int rows, float& w) {
+  const int t = threadIdx.x & (L - 1), lane = t & 31, warp = t >> 5;
+  float la = 0.f;
+  w = 0.f;
+  if (t < rows) {
+    if (a.dt) {
+      const float z = __bfloat162float(a.dt[(size_t)(row0 + t) * a.dt_stride + h]) + a.dt_bias[h];
+      w = log1pf(expf(-fabsf(z))) + fmaxf(z, 0.f);
+      la = a.a[h] * w * LOG2E;
+    } else {
+      w = 1.f;
+      la = a.a[h] * LOG2E;
     }
+  }
 #pragma unroll
-    for (int o = 1; o < 32; o <<= 1) { const float v = __shfl_up_sync(0xffffffffu, la, o); if (lane >= o) la += v; }
-    if (lane == 31) C.part[warp] = la;
-  }
+  for (int o = 1; o < 32; o <<= 1) { const float v = __shfl_up_sync(0xffffffffu, la, o); if (lane >= o) la += v; }
+  if (lane == 31 && threadIdx.x < L) C.part[warp] = la;
   __syncthreads();
-  if (t < L) {
-    for (int i = 0; i < warp; ++i) la += C.part[i];
-    C.c[t] = la;
-    C.w[t] = w;
-  }
-  __syncthreads();
+  for (int i = 0; i < warp; ++i) la += C.part[i];
+  return la;
 }
 
 __device__ __forceinline__ void setup(Ctl& C, uint32_t cols) {
@@ -99,64 +94,73 @@ __device__ __forceinline__ void teardown(Ctl& C, uint32_t cols, Status* status, 
   if (threadIdx.x < 32) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(C.tmem), "r"(cols) : "memory");
 }
 
-// copies that were issued must land before the CTA ends
-__device__ __forceinline__ void drain(Ctl& C, int bar, uint32_t parity) {
+// after a wait that gave up: copies and products under way must end before the CTA does (bounded: a phase that never comes is not waited for)
+__device__ __forceinline__ void drain(Ctl& C) {
+  if (!C.dead) return;
   if (threadIdx.x == 0)
-    for (int i = 0; i < 100000 && !mbar_try(&C.full[bar], parity); ++i) __nanosleep(64);
+    for (int i = 0; i < 100000; ++i) __nanosleep(64);
 }
 
+// grid (groups x parts of a group's heads, chunks): k stays in shared memory while the heads (and their tiles of 64 value dims) go by
 __global__ void __launch_bounds__(THREADS)
 chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv, Args a) {
-  extern __shared__ uint8_t raw[];
-  uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
-  __shared__ Ctl C;
+  extern __shared__ __align__(1024) uint8_t sm[];
   const int nb = (a.ns + 1) / 2;                          // blocks of 128 state rows
   uint8_t* ks = sm;                                       // [terms][2 nb] slabs
-  uint8_t* vh = ks + (size_t)a.terms * 2 * nb * SLAB;     // weighted values, upper terms (the copy lands here), lower terms
-  uint8_t* vl = vh + SLAB;
+  uint8_t* vh = ks + (size_t)a.terms * 2 * nb * SLAB;     // weighted values, upper terms (the copy lands here): two stages
+  uint8_t* vl = vh + 2 * SLAB;                            // lower terms
+  Ctl& C = *reinterpret_cast<Ctl*>(vl + SLAB);
   setup(C, 128);
   pdl_launch_dependents();
   pdl_wait();
-  const int chunk = blockIdx.y, h = blockIdx.x, g = h / (a.H / a.G), row0 = a.c_row0[chunk], rows = a.c_rows[chunk];
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, pts = (a.P + 63) / 64;
+  const int chunk = blockIdx.y, rep = a.H / a.G, parts = (rep + a.hpc - 1) / a.hpc, g = blockIdx.x / parts;
+  const int h0 = g * rep + (blockIdx.x % parts) * a.hpc, nh = min(a.hpc, (g + 1) * rep - h0), row0 = a.c_row0[chunk], rows = a.c_rows[chunk];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, pts = (a.P + 63) / 64, items = nh * pts;
   volatile int* dead = &C.dead;
+  auto fetch = [&](int it) {
+    mbar_expect(&C.full[it & 1], SLAB);
+    tma2d(vh + (it & 1) * SLAB, &mv, a.v_col + (h0 + it / pts) * a.P + 64 * (it % pts), row0, &C.full[it & 1]);
+  };
   if (warp == 0 && elect_one()) {
-    mbar_expect(&C.full[0], a.terms * a.ns * SLAB);
+    mbar_expect(&C.full[2], a.terms * a.ns * SLAB);
     for (int t = 0; t < a.terms; ++t)
-      for (int s = 0; s < a.ns; ++s) tma2d(ks + (size_t)(t * 2 * nb + s) * SLAB, &mk, a.k_col + t * a.k_lo + g * a.N + 64 * s, row0, &C.full[0]);
-    mbar_expect(&C.full[1], SLAB);
-    tma2d(vh, &mv, a.v_col + h * a.P, row0, &C.full[1]);
+      for (int s = 0; s < a.ns; ++s) tma2d(ks + (size_t)(t * 2 * nb + s) * SLAB, &mk, a.k_col + t * a.k_lo + g * a.N + 64 * s, row0, &C.full[2]);
+    fetch(0);
   }
-  chunk_decays(a, C, h, row0, rows);
-  const float last = C.c[L - 1];
-  if (tid == 0) a.dec[(size_t)chunk * a.H + h] = ex2(last);
   const uint32_t id = idesc(64, 1, 1);
-  bool ok = true, k_seen = false;
-  for (int pt = 0; pt < pts && ok; ++pt) {
-    ok = __syncthreads_and(mbar_wait(&C.full[1], pt & 1, dead));
+  bool ok = mbar_wait(&C.full[2], 0, dead);
+  for (int it = 0; it < items; ++it) {
+    const int h = h0 + it / pts, pt = it % pts;
+    uint8_t* vs = vh + (it & 1) * SLAB;
+    if (pt == 0) {
+      float w;
+      const float c = chunk_decays(a, C, h, row0, rows, w), last = C.part[0] + C.part[1] + C.part[2] + C.part[3];
+      if (tid < L) C.c[tid] = ex2(last - c) * w;
+      if (tid == 0) a.dec[(size_t)chunk * a.H + h] = ex2(last);
+    }
+    if (ok) ok = mbar_wait(&C.full[it & 1], (it >> 1) & 1, dead);
+    ok = __syncthreads_and(ok);
     if (!ok) break;
+    if (it + 1 < items && warp == 0 && elect_one()) fetch(it + 1);
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      const int u = tid + i * THREADS, r = u >> 3;                   // a 16-byte unit and its row
-      const float wt = ex2(last - C.c[r]) * C.w[r];
+      const int u = tid + i * THREADS;                               // a 16-byte unit; its row is u / 8
+      const float wt = C.c[u >> 3];
       float f[8];
       uint4 hi, lo;
-      rows::load_v<__nv_bfloat16, 8>(reinterpret_cast<const __nv_bfloat16*>(vh) + u * 8, f);
+      rows::load_v<__nv_bfloat16, 8>(reinterpret_cast<const __nv_bfloat16*>(vs) + u * 8, f);
 #pragma unroll
       for (int k = 0; k < 8; ++k) f[k] *= wt;
       split2(f[0], f[1], hi.x, lo.x); split2(f[2], f[3], hi.y, lo.y); split2(f[4], f[5], hi.z, lo.z); split2(f[6], f[7], hi.w, lo.w);
-      reinterpret_cast<uint4*>(vh)[u] = hi;
+      reinterpret_cast<uint4*>(vs)[u] = hi;
       reinterpret_cast<uint4*>(vl)[u] = lo;
     }
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     fence_before();
-    if (!k_seen) ok = mbar_wait(&C.full[0], 0, dead);
-    k_seen = true;
-    ok = __syncthreads_and(ok);
-    if (!ok) break;
+    __syncthreads();
     fence_after();
     if (warp == 0 && elect_one()) {
-      const uint64_t dh = desc(smem_u32(vh), SLAB), dl = desc(smem_u32(vl), SLAB);
+      const uint64_t dh = desc(smem_u32(vs), SLAB), dl = desc(smem_u32(vl), SLAB);
       for (int b = 0; b < nb; ++b) {
         const uint64_t k0 = desc(smem_u32(ks) + (2 * b) * SLAB, SLAB), k1 = desc(smem_u32(ks) + (2 * nb + 2 * b) * SLAB, SLAB);
         for (int t = 0; t < 8; ++t) {
@@ -168,13 +172,9 @@ chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant_
       }
       commit(&C.done);
     }
-    ok = __syncthreads_and(mbar_wait(&C.done, pt & 1, dead));
+    ok = __syncthreads_and(mbar_wait(&C.done, it & 1, dead));
     if (!ok) break;
     fence_after();
-    if (pt + 1 < pts && warp == 0 && elect_one()) {
-      mbar_expect(&C.full[1], SLAB);
-      tma2d(vh, &mv, a.v_col + h * a.P + 64 * (pt + 1), row0, &C.full[1]);
-    }
     // lane = state row: columns of the tile go out as runs of consecutive state rows
     const int w4 = warp & 3, half = warp >> 2;
     for (int b = 0; b < nb; ++b) {
@@ -192,7 +192,7 @@ chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant_
     }
     fence_before();
   }
-  if (C.dead) { drain(C, 0, 0); drain(C, 1, 0); drain(C, 1, 1); }
+  drain(C);
   teardown(C, 128, a.status, 69);
 }
 
@@ -233,93 +233,106 @@ __global__ void __launch_bounds__(256) chunk_starts_kernel(Args a) {
   *reinterpret_cast<float4*>(a.S + (size_t)a.seg_dst[seg] * per + e) = S;
 }
 
-__global__ void __launch_bounds__(THREADS)
+// grid as chunk_sums: q and k stay in shared memory while the heads go by; the scores are computed again for every head (their tensor
+// memory is where the weighted scores go)
+__global__ void __launch_bounds__(THREADS, 2)
 chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv,
                  const __grid_constant__ CUtensorMap ms, Args a) {
-  extern __shared__ uint8_t raw[];
-  uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
-  __shared__ Ctl C;
+  extern __shared__ __align__(1024) uint8_t sm[];
   uint8_t* qs = sm;                                      // [terms][ns] slabs
   uint8_t* ks = qs + (size_t)a.terms * a.ns * SLAB;
   uint8_t* vs = ks + (size_t)a.terms * a.ns * SLAB;      // one slab
   uint8_t* ss = vs + SLAB;                               // start state, [2][ns] slabs of 64 rows
+  Ctl& C = *reinterpret_cast<Ctl*>(ss + (size_t)2 * a.ns * HSLAB);
   setup(C, 256);
   pdl_launch_dependents();
   pdl_wait();
-  const int chunk = blockIdx.y, h = blockIdx.x, g = h / (a.H / a.G), row0 = a.c_row0[chunk], rows = a.c_rows[chunk];
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, pts = (a.P + 63) / 64, w4 = warp & 3, half = warp >> 2;
+  const int chunk = blockIdx.y, rep = a.H / a.G, parts = (rep + a.hpc - 1) / a.hpc, g = blockIdx.x / parts;
+  const int h0 = g * rep + (blockIdx.x % parts) * a.hpc, nh = min(a.hpc, (g + 1) * rep - h0), row0 = a.c_row0[chunk], rows = a.c_rows[chunk];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, pts = (a.P + 63) / 64, items = nh * pts, w4 = warp & 3, half = warp >> 2;
   volatile int* dead = &C.dead;
   const uint32_t tp = C.tmem, ta = tp + 128, tb = tp + 192, lanes = (uint32_t)(w4 * 32) << 16;
-  auto tile = [&](int pt) {                              // values and start state of a tile of 64 value dims
-    mbar_expect(&C.full[1], SLAB + 2 * a.ns * HSLAB);
-    tma2d(vs, &mv, a.v_col + h * a.P + 64 * pt, row0, &C.full[1]);
-    const int y = (chunk * a.H + h) * a.P + 64 * pt;
+  auto tile = [&](int it) {                              // values and start state of a tile of 64 value dims
+    const int h = h0 + it / pts, pt = it % pts, y = (chunk * a.H + h) * a.P + 64 * pt;
+    mbar_expect(&C.full[0], SLAB + 2 * a.ns * HSLAB);
+    tma2d(vs, &mv, a.v_col + h * a.P + 64 * pt, row0, &C.full[0]);
     for (int t = 0; t < 2; ++t)
-      for (int s = 0; s < a.ns; ++s) tma2d(ss + (size_t)(t * a.ns + s) * HSLAB, &ms, 64 * s, t * a.chunks * a.H * a.P + y, &C.full[1]);
+      for (int s = 0; s < a.ns; ++s) tma2d(ss + (size_t)(t * a.ns + s) * HSLAB, &ms, 64 * s, t * a.chunks * a.H * a.P + y, &C.full[0]);
   };
   const int kst = a.N / 16;
+  const uint64_t lo = (uint64_t)a.ns * (SLAB >> 4), dq = desc(smem_u32(qs), 16), dk = desc(smem_u32(ks), 16);
+  auto scores = [&]() {
+    const uint32_t id = idesc(128, 0, 0);
+    for (int t = 0; t < kst; ++t) {
+      const uint64_t o = (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2;
+      mma_ss(tp, dq + o, dk + o, id, t ? 1u : 0u);
+      if (a.terms > 1) {
+        mma_ss(tp, dq + o, dk + lo + o, id, 1u);
+        mma_ss(tp, dq + lo + o, dk + o, id, 1u);
+      }
+    }
+    commit(&C.done);
+  };
   if (warp == 0 && elect_one()) {
-    mbar_expect(&C.full[0], 2 * a.terms * a.ns * SLAB);
+    mbar_expect(&C.full[2], 2 * a.terms * a.ns * SLAB);
     for (int t = 0; t < a.terms; ++t)
       for (int s = 0; s < a.ns; ++s) {
-        tma2d(qs + (size_t)(t * a.ns + s) * SLAB, &mq, a.q_col + t * a.q_lo + g * a.N + 64 * s, row0, &C.full[0]);
-        tma2d(ks + (size_t)(t * a.ns + s) * SLAB, &mk, a.k_col + t * a.k_lo + g * a.N + 64 * s, row0, &C.full[0]);
+        tma2d(qs + (size_t)(t * a.ns + s) * SLAB, &mq, a.q_col + t * a.q_lo + g * a.N + 64 * s, row0, &C.full[2]);
+        tma2d(ks + (size_t)(t * a.ns + s) * SLAB, &mk, a.k_col + t * a.k_lo + g * a.N + 64 * s, row0, &C.full[2]);
       }
     tile(0);
   }
-  chunk_decays(a, C, h, row0, rows);
-  bool ok = __syncthreads_and(mbar_wait(&C.full[0], 0, dead));
-  const uint64_t lo = (uint64_t)a.ns * (SLAB >> 4), dq = desc(smem_u32(qs), 16), dk = desc(smem_u32(ks), 16);
+  bool ok = __syncthreads_and(mbar_wait(&C.full[2], 0, dead));
+  if (ok && warp == 0 && elect_one()) {
+    fence_after();
+    scores();
+  }
   const int i = w4 * 32 + lane;
-  if (ok) {
-    fence_after();
-    if (warp == 0 && elect_one()) {
-      const uint32_t id = idesc(128, 0, 0);
-      for (int t = 0; t < kst; ++t) {
-        const uint64_t o = (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2;
-        mma_ss(tp, dq + o, dk + o, id, t ? 1u : 0u);
-        if (a.terms > 1) {
-          mma_ss(tp, dq + o, dk + lo + o, id, 1u);
-          mma_ss(tp, dq + lo + o, dk + o, id, 1u);
-        }
-      }
-      commit(&C.done);
-    }
-    ok = __syncthreads_and(mbar_wait(&C.done, 0, dead));
-  }
-  if (ok) {
-    fence_after();
-    float s[64];
-    const bool any = w4 * 32 + 31 >= half * 64;          // the warp's rows reach these columns
-    if (any) {
-      ld32(tp + half * 64 + lanes, s);
-      ld32(tp + half * 64 + 32 + lanes, s + 32);
-      wait_ld();
-    }
-    fence_before();
-    __syncthreads();                                     // every score has been read: the weights may take their place
-    fence_after();
-    uint32_t hi[32], lw[32];
-    const float ci = C.c[i];
-#pragma unroll
-    for (int q = 0; q < 32; ++q) {
-      const int j = half * 64 + 2 * q;
-      float x = 0.f, y = 0.f;
+  float ci = 0.f, ei = 0.f, D = 0.f;
+  uint32_t used = 0;                                     // completions of `done` that were waited for
+  for (int it = 0; it < items && ok; ++it) {
+    const int h = h0 + it / pts, pt = it % pts;
+    if (pt == 0) {
+      float w;
+      ci = chunk_decays(a, C, h, row0, rows, w);
+      if (tid < L) C.c[tid] = ci - __log2f(w);           // weight 0: infinity, and its exponential below 0
+      ei = ex2(ci);
+      D = a.D ? a.D[h] : 0.f;
+      ok = __syncthreads_and(mbar_wait(&C.done, used & 1, dead));
+      if (!ok) break;
+      ++used;
+      fence_after();
+      float s[64];
+      const bool any = w4 * 32 + 31 >= half * 64;        // the warp's rows reach these columns
       if (any) {
-        const float2 cj = *reinterpret_cast<const float2*>(C.c + j), wj = *reinterpret_cast<const float2*>(C.w + j);
-        x = j <= i ? s[2 * q] * (ex2(ci - cj.x) * wj.x) : 0.f;
-        y = j + 1 <= i ? s[2 * q + 1] * (ex2(ci - cj.y) * wj.y) : 0.f;
+        ld32(tp + half * 64 + lanes, s);
+        ld32(tp + half * 64 + 32 + lanes, s + 32);
+        wait_ld();
       }
-      split2(x, y, hi[q], lw[q]);
+      fence_before();
+      __syncthreads();                                   // every score has been read: the weighted ones may take their place
+      fence_after();
+#pragma unroll
+      for (int b = 0; b < 2; ++b) {
+        uint32_t hi[16], lw[16];
+#pragma unroll
+        for (int q = 0; q < 16; ++q) {
+          const int j = half * 64 + 32 * b + 2 * q;
+          float x = 0.f, y = 0.f;
+          if (any) {
+            const float2 cj = *reinterpret_cast<const float2*>(C.c + j);
+            x = j <= i ? s[32 * b + 2 * q] * ex2(ci - cj.x) : 0.f;
+            y = j + 1 <= i ? s[32 * b + 2 * q + 1] * ex2(ci - cj.y) : 0.f;
+          }
+          split2(x, y, hi[q], lw[q]);
+        }
+        st16(tp + half * 32 + 16 * b + lanes, hi);
+        st16(tp + 64 + half * 32 + 16 * b + lanes, lw);
+      }
+      wait_st();
+      fence_before();
     }
-    st16(tp + half * 32 + lanes, hi); st16(tp + half * 32 + 16 + lanes, hi + 16);
-    st16(tp + 64 + half * 32 + lanes, lw); st16(tp + 64 + half * 32 + 16 + lanes, lw + 16);
-    wait_st();
-    fence_before();
-  }
-  const float ei = ex2(C.c[i]), D = a.D ? a.D[h] : 0.f;
-  for (int pt = 0; pt < pts && ok; ++pt) {
-    ok = __syncthreads_and(mbar_wait(&C.full[1], pt & 1, dead));
+    ok = __syncthreads_and(mbar_wait(&C.full[0], it & 1, dead));
     if (!ok) break;
     fence_after();
     if (warp == 0 && elect_one()) {
@@ -334,38 +347,37 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
       }
       commit(&C.done);
     }
-    ok = __syncthreads_and(mbar_wait(&C.done, (pt + 1) & 1, dead));
+    ok = __syncthreads_and(mbar_wait(&C.done, used & 1, dead));
     if (!ok) break;
+    ++used;
     fence_after();
-    float x[32], z[32], v[32];
-    ld32(ta + half * 32 + lanes, x);
-    ld32(tb + half * 32 + lanes, z);
-    if (a.D) {
+    if (pt + 1 == pts && it + 1 < items && warp == 0 && elect_one()) scores();       // of the next head
+    __nv_bfloat16* o = a.y + ((size_t)(row0 + i) * a.H + h) * a.P + pt * 64 + half * 32;
+    const int cols = min(32, a.P - pt * 64 - half * 32);
 #pragma unroll
-      for (int u = 0; u < 4; ++u)
-        rows::load_v<__nv_bfloat16, 8>(reinterpret_cast<const __nv_bfloat16*>(vs + i * 128 + (((half * 4 + u) ^ (i & 7)) * 16)), v + 8 * u);
-    }
-    wait_ld();
-    fence_before();
-    __syncthreads();                                     // tile and accumulators have been read
-    if (pt + 1 < pts && warp == 0 && elect_one()) tile(pt + 1);
-    if (i < rows) {
-      __nv_bfloat16* o = a.y + ((size_t)(row0 + i) * a.H + h) * a.P + pt * 64 + half * 32;
-      const int cols = min(32, a.P - pt * 64 - half * 32);
+    for (int b = 0; b < 2; ++b) {
+      float x[16], z[16];
+      ld16(ta + half * 32 + 16 * b + lanes, x);
+      ld16(tb + half * 32 + 16 * b + lanes, z);
+      wait_ld();
 #pragma unroll
-      for (int u = 0; u < 4; ++u)
-        if (8 * u < cols) {                              // P is a multiple of eight
-          float f[8];
+      for (int u = 0; u < 2; ++u)
+        if (i < rows && 16 * b + 8 * u < cols) {         // P is a multiple of eight
+          float f[8], v[8];
+          if (a.D) rows::load_v<__nv_bfloat16, 8>(reinterpret_cast<const __nv_bfloat16*>(vs + i * 128 + (((half * 4 + 2 * b + u) ^ (i & 7)) * 16)), v);
 #pragma unroll
           for (int k = 0; k < 8; ++k) {
             f[k] = fmaf(ei, z[8 * u + k], x[8 * u + k]);
-            if (a.D) f[k] = fmaf(D, v[8 * u + k], f[k]);
+            if (a.D) f[k] = fmaf(D, v[k], f[k]);
           }
-          rows::store_v<__nv_bfloat16, 8>(o + 8 * u, f);
+          rows::store_v<__nv_bfloat16, 8>(o + 16 * b + 8 * u, f);
         }
     }
+    fence_before();
+    __syncthreads();                                     // tile and accumulators have been read
+    if (it + 1 < items && warp == 0 && elect_one()) tile(it + 1);
   }
-  if (C.dead) { drain(C, 0, 0); drain(C, 1, 0); drain(C, 1, 1); }
+  drain(C);
   teardown(C, 256, a.status, 70);
 }
 
@@ -412,8 +424,8 @@ __global__ void __launch_bounds__(256) state_turn_kernel(TurnArgs a) {
   }
 }
 
-static size_t sums_smem(const Args& a) { return (size_t)(a.terms * 2 * ((a.ns + 1) / 2) + 2) * SLAB + 1024; }
-static size_t out_smem(const Args& a) { return (size_t)(2 * a.terms * a.ns + 1) * SLAB + (size_t)2 * a.ns * HSLAB + 1024; }
+static size_t sums_smem(const Args& a) { return (size_t)(a.terms * 2 * ((a.ns + 1) / 2) + 3) * SLAB + sizeof(Ctl); }
+static size_t out_smem(const Args& a) { return (size_t)(2 * a.terms * a.ns + 1) * SLAB + (size_t)2 * a.ns * HSLAB + sizeof(Ctl); }
 
 }  // namespace rst
 }  // namespace sfb
@@ -441,8 +453,12 @@ int sfb_rows_state_tc(const void* mq, const void* mk, const void* mv, const void
       terms < 1 || terms > 2 || (q_col | k_col | v_col | q_lo | k_lo | N) % 8)
     return (int)cudaErrorInvalidValue;
   Args a{c_row0, c_rows, seg, first, seg_src, seg_dst, (const __nv_bfloat16*)dt, dt_stride, (const float*)dt_bias, (const float*)la, (const float*)D, (float*)S,
-         (float*)sums, (float*)dec, (__nv_bfloat16*)starts, (__nv_bfloat16*)y, H, G, N, P, Np, ns, terms, q_col, k_col, v_col, q_lo, k_lo, chunks,
+         (float*)sums, (float*)dec, (__nv_bfloat16*)starts, (__nv_bfloat16*)y, H, G, N, P, Np, ns, terms, q_col, k_col, v_col, q_lo, k_lo, chunks, 1,
          (Status*)status};
+  const int rep = H / G;
+  a.hpc = rep < 8 ? rep : 8;         // fewer heads per block where that leaves SMs empty
+  while (a.hpc > 1 && (long long)G * ((rep + a.hpc - 1) / a.hpc) * chunks < 148) a.hpc = (a.hpc + 1) / 2;
+  const int blocks = G * ((rep + a.hpc - 1) / a.hpc);
   const size_t s1 = sums_smem(a), s2 = out_smem(a);
   static size_t g1 = 0, g2 = 0;
   if (s1 > g1) {
@@ -456,12 +472,12 @@ int sfb_rows_state_tc(const void* mq, const void* mk, const void* mv, const void
     g2 = s2;
   }
   const CUtensorMap *q = (const CUtensorMap*)mq, *k = (const CUtensorMap*)mk, *v = (const CUtensorMap*)mv, *s = (const CUtensorMap*)ms;
-  cudaError_t rc = sfb_launch(chunk_sums_kernel, dim3(H, chunks), dim3(THREADS), s1, stream, *k, *v, a);
+  cudaError_t rc = sfb_launch(chunk_sums_kernel, dim3(blocks, chunks), dim3(THREADS), s1, stream, *k, *v, a);
   if (rc != cudaSuccess) return (int)rc;
   const size_t per = (size_t)H * P * Np;
   rc = sfb_launch(chunk_starts_kernel, dim3((unsigned)((per / 4 + 255) / 256), runs), dim3(256), 0, stream, a);
   if (rc != cudaSuccess) return (int)rc;
-  return (int)sfb_launch(chunk_out_kernel, dim3(H, chunks), dim3(THREADS), s2, stream, *q, *k, *v, *s, a);
+  return (int)sfb_launch(chunk_out_kernel, dim3(blocks, chunks), dim3(THREADS), s2, stream, *q, *k, *v, *s, a);
 }
 
 }  // extern "C"

@@ -13,6 +13,7 @@ import torch.nn.functional as F
 
 from ..ops import rows as R
 
+DECODE_ROWS = 64           # single rows of latent attention whose partial results are held at a time
 GATED_STEP_ROWS = 16       # up to this many single rows run convolution, gates and recurrence as one kernel
 
 
@@ -325,6 +326,7 @@ class LatentAttention:
         self.uv = w.act("uv").view(self.H, self.vdim, self.rank).transpose(1, 2).contiguous()       # [H, rank, vdim]
         self.cs = rotation_table(spec["rot"]["base"], self.rot, max_context, w.device)
         self.tc = R.latent_tc_supports(w.dtype, self.dim, self.rot, self.vdim, self.rank)
+        self.dec = R.latent_decode_supports(w.dtype, self.rot, self.rank)
         self.merge, self.kv_run = (None, None), (1, self.rank + self.rot, 0)
 
     def reserve(self, e) -> None:
@@ -334,7 +336,11 @@ class LatentAttention:
         short = min(n, e.short_rows(self.tc))
         e.scratch.reserve("lat_q", short * self.H * key, dt)
         e.scratch.reserve("lat_o", short * self.H * self.rank, dt)
-        parts = max(1, self.H // R.attn_blocks(self.H, 1)) * 1024 + self.H * 64
+        if self.dec:
+            self.slice = min(short, DECODE_ROWS)
+            parts = self.slice * self.H * R.latent_blocks(self.window, e.max_context - 1)
+        else:
+            parts = max(1, self.H // R.attn_blocks(self.H, 1)) * 1024 + self.H * 64
         e.scratch.reserve("attn_part", parts * self.rank, torch.float32)
         e.scratch.reserve("attn_ml", parts * 2, torch.float32)
         if self.tc:
@@ -365,6 +371,16 @@ class LatentAttention:
             m = s.short
             q, c = s.scratch.get("lat_q", m, H * key), s.scratch.get("lat_o", m, H * self.rank)
             R.head_proj(proj, dim + rot, self.uk, q, key, m, s.short_rows, 1, rot)
+        if s.short and self.dec:
+            part, ml = s.scratch.buf["attn_part"], s.scratch.buf["attn_ml"]
+            blocks = R.latent_blocks(self.window, min(s.pages * 64, s.engine.max_context) - 1)
+            idx = s.short_rows if s.short_rows is not None else s.engine._iota[:m]
+            for a in range(0, m, self.slice):
+                b = min(m, a + self.slice)
+                R.latent_decode(q[a:b], pool, self.rank, rot, s.table, s.row_lane, s.row_pos, idx[a:b], b - a, H, part, ml, self.window, blocks,
+                                self.scale, s.status)
+                R.head_proj(None, 0, self.uv, o, self.vdim, b - a, idx[a:b], 2, merge=(part, ml, s.row_pos, self.window, blocks))
+        elif s.short:
             blocks = R.attn_blocks(H, 1)
             sp = s.engine.splits(s, m, blocks, self.window)
             part, ml = (s.scratch.buf["attn_part"], s.scratch.buf["attn_ml"]) if sp > 1 else (None, None)

@@ -151,12 +151,14 @@ def latent_append(proj, w, cs, pool, table, row_lane, row_pos, n, heads, dim, ro
                                               _p(status), _stream()), "rows_latent_append")
 
 
-def head_proj(x, x_head, w, out, out_head, n, rows=None, lists=0, tail=0):
+def head_proj(x, x_head, w, out, out_head, n, rows=None, lists=0, tail=0, merge=None):
     """out[row][h] = x[row][h] w[h], w [heads, K, M]; heads ``x_head`` / ``out_head`` elements apart.  ``rows`` names rows of x (lists=1) or
-    of out (lists=2); ``tail`` elements behind x's K are copied behind out's M."""
+    of out (lists=2); ``tail`` elements behind x's K are copied behind out's M.  ``merge``: (part, ml, row_pos, window, blocks) of
+    latent_decode; x is then the merged attention output."""
+    part, ml, pos, window, blocks = merge or (None, None, None, 1, 0)
     H, K, M = w.shape
     _check(_lib.rows().sfb_rows_head_proj(*_strides(x), c_int64(x_head), _p(w), *_strides(out), c_int64(out_head), _p(rows), c_int(lists if rows is not None else 0),
-                                          c_int(n), c_int(H), c_int(K), c_int(M), c_int(tail), _fp32(w), _stream()), "rows_head_proj")
+                                          _p(part), _p(ml), _p(pos), c_int(window), c_int(blocks), c_int(n), c_int(H), c_int(K), c_int(M), c_int(tail), _fp32(w), _stream()), "rows_head_proj")
 
 
 def gather_pages(pool, pages, out, count, status):
@@ -307,7 +309,8 @@ _maps: dict[tuple, TensorMap] = {}
 
 
 def tensor_map(t: torch.Tensor, cols: int, box: int, stride: int | None = None, first: int = 0) -> TensorMap:
-    """The map over all of ``t``'s storage, kept, so that one map serves every step over a scratch buffer."""
+    """The map over all of ``t``'s storage, kept, so that one map serves every step over a scratch buffer (it is an address and a shape:
+    memory that is allocated again at the same place may use it again)."""
     stride = stride or cols
     total = t.untyped_storage().nbytes() // 2
     key = (t.untyped_storage().data_ptr(), total, cols, box, stride, first)
@@ -331,6 +334,26 @@ def attn_tc(q, kv, table, row_lane, row_pos, tiles, n_tiles, bias, out, heads, s
 
 def latent_tc_supports(dtype: torch.dtype, dim: int, rot: int, vdim: int, rank: int) -> bool:
     return attn_tc_supports(dtype, dim, vdim) and rot % 8 == 0 and 0 < rot <= 64 and rank % 8 == 0
+
+
+def latent_decode_supports(dtype: torch.dtype, rot: int, rank: int) -> bool:
+    """Shapes the tensor-core arm for single rows takes (csrc/k_rows_latent_dec.cu)."""
+    return dtype == torch.bfloat16 and rot % 8 == 0 and 0 < rot <= 64 and rank % 8 == 0 and rank <= 512
+
+
+def latent_blocks(window: int, max_pos: int) -> int:
+    """Pairs of pages that the window of a position up to ``max_pos`` can touch."""
+    return -(-min((window + 62) // 64 + 1, max_pos // 64 + 1) // 2)
+
+
+def latent_decode(q, pool, rank, rot, table, row_lane, row_pos, rows, n, heads, part, ml, window, blocks, scale, status):
+    """Attention of single rows over the cached latents, per block of two pages: (log2 maximum, sum, output) to ml and part.  q: [n, heads
+    (rank + rot)] of the launch's rows."""
+    key, box = rank + rot, _lib.rows().sfb_rows_latent_heads(heads)
+    maps = (tensor_map(q, rank, box, key), tensor_map(q, rot, box, key, rank), tensor_map(pool, rank, 64, key), tensor_map(pool, rot, 64, key, rank))
+    _check(_lib.rows().sfb_rows_latent_decode(*(m.ptr for m in maps), _p(table), _p(row_lane), _p(row_pos), _p(rows), _p(part), _p(ml),
+                                              c_int(table.shape[1]), c_int(pool.shape[0]), c_int(n), c_int(heads), c_int(rank), c_int(rot), c_int(window),
+                                              c_int(blocks), c_int(q.storage_offset() // key), c_float(scale), _p(status), _stream()), "rows_latent_decode")
 
 
 def expand(c: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:

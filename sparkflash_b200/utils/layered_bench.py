@@ -1,6 +1,7 @@
-"""Throughput of a layered decoder (models/fanodra.py) at sizes that resemble a real model's layers, per-kernel roofline fractions,
-and the same for the closest model of the package, the hybrid decoder of models/qwen.py (linear attention three layers in four,
-softmax attention in the fourth).  ``python bench.py --design fanodra`` prints it as one JSON line.
+"""Throughput of a layered decoder (models/fanodra.py, models/gudutar.py) at sizes that resemble a real model's layers, per-kernel
+roofline fractions, and the same for the closest model of the package: for Fanodra the hybrid decoder of models/qwen.py (linear
+attention three layers in four, softmax attention in the fourth), for Gudutar the Fanodra of the same width, head size, feed-forward
+width and number of layer runs.  ``python bench.py --design NAME`` prints it as one JSON line.
 
 Everything is timed on the device with CUDA events after warm-up; inputs are larger than L2, or L2 is flushed in between.
 """
@@ -10,7 +11,9 @@ import statistics
 
 import torch
 
-from ..models.fanodra import Fanodra, FanodraConfig, random_tensors
+from ..models import fanodra, gudutar
+from ..models.fanodra import FanodraConfig
+from ..models.gudutar import GudutarConfig
 from ..models.layered import LayeredEngine
 from . import roofline
 
@@ -22,7 +25,7 @@ SIZES = {
 }
 
 
-def config(name: str) -> FanodraConfig:
+def fanodra_config(name: str) -> FanodraConfig:
     w, n, H, G, dim, rp, ra, parts, ff, vocab, loop = SIZES[name]
     mlp = {"kind": "dense", "ff": ff}
     par = {"type": "parallel", "mlp": mlp, "mixer": {"left": {"heads": H, "kv_heads": G, "dim": dim, "vdim": dim, "scale": dim ** -0.5},
@@ -33,9 +36,31 @@ def config(name: str) -> FanodraConfig:
                                     "loop": dict(zip(("start", "stop", "times"), loop)) if loop else None})
 
 
-def engine(name: str, lanes: int, context: int, rows: int) -> LayeredEngine:
-    cfg = config(name)
-    return LayeredEngine(Fanodra(cfg, random_tensors(cfg, 0, "cuda"), max_context=context), max_lanes=lanes, max_context=context, max_rows=rows)
+WINDOW, RANK, ROT = 1024, 512, 64        # latent attention
+ORDER = ("mamba2", "retention", "latent_attention", "mamba2")
+
+
+def gudutar_config(name: str) -> GudutarConfig:
+    """As many layers as the Fanodra of that size has layer runs; recurrences of twice / once the width, heads of 64 x 128 and 128 x 128."""
+    w, n, H, _, dim, _, _, _, ff, vocab, loop = SIZES[name]
+    runs = n + (loop[1] - loop[0]) * (loop[2] - 1) if loop else n
+    rot = lambda dims: {"base": 10000.0, "dims": dims}
+    mixers = {"mamba2": {"heads": 2 * w // 64, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1},
+              "retention": {"heads": w // dim, "dim": dim, "vdim": dim, "rot": rot(dim), "decay": [1 - 2.0 ** (-5 - 7 * i / (w // dim)) for i in range(w // dim)]},
+              "latent_attention": {"heads": H, "dim": dim, "rot_dim": ROT, "vdim": dim, "kv_rank": RANK, "scale": (dim + ROT) ** -0.5,
+                                   "mask": {"size": WINDOW}, "rot": rot(ROT)}}
+    return GudutarConfig.from_dict({"architecture": "Gudutar", "name": f"gudutar-{name}", "vocab": vocab, "width": w, "norm": {"eps": 1e-6},
+                                    "embedding": {"scale": 1.0}, "layers": [{"type": t, "mixer": mixers[t], "mlp": {"kind": "dense", "ff": ff}}
+                                                                            for t in (ORDER[i % 4] for i in range(runs))]})
+
+
+CONFIGS = {"fanodra": (fanodra_config, fanodra.Fanodra, fanodra.random_tensors), "gudutar": (gudutar_config, gudutar.Gudutar, gudutar.random_tensors)}
+
+
+def engine(design: str, name: str, lanes: int, context: int, rows: int) -> LayeredEngine:
+    make, cls, weights = CONFIGS[design]
+    cfg = make(name)
+    return LayeredEngine(cls(cfg, weights(cfg, 0, "cuda"), max_context=context), max_lanes=lanes, max_context=context, max_rows=rows)
 
 
 def timed(fn, reps: int, warm: int = 3, flush=None) -> float:
@@ -54,13 +79,13 @@ def timed(fn, reps: int, warm: int = 3, flush=None) -> float:
     return statistics.median(ts)
 
 
-def throughput(name: str, prompt: int = 8192, chunk: int = 4096, streams=(1, 16, 64), steps: int = 32) -> dict:
+def throughput(design: str, name: str, prompt: int = 8192, chunk: int = 4096, streams=(1, 16, 64), steps: int = 32) -> dict:
     """Prefill tok/s of one prompt in portions, decode tok/s at several stream counts against ``prompt`` cached tokens (and end to
     end through ``step``, which copies inputs from pinned memory and reads the tokens back)."""
     import time
     lanes, out = max(streams), {}
     g = torch.Generator().manual_seed(0)
-    eng = engine(name, lanes, prompt + 256, chunk)
+    eng = engine(design, name, lanes, prompt + 256, chunk)
     ids = torch.randint(0, eng.model.vocab, (prompt,), generator=g).tolist()
     cuts = [(p, min(p + chunk, prompt)) for p in range(0, prompt, chunk)]
 
@@ -98,7 +123,69 @@ def throughput(name: str, prompt: int = 8192, chunk: int = 4096, streams=(1, 16,
     return out
 
 
-def work(cfg: FanodraConfig, n: int, ctx: int, head_rows: int, decode: bool) -> dict[str, roofline.ClassWork]:
+def gudutar_work(cfg: GudutarConfig, n: int, ctx: int, head_rows: int, decode: bool) -> dict[str, roofline.ClassWork]:
+    """The same accounting for Gudutar.  Recurrences: inputs and outputs once, the state of every segment in and out, and the products
+    of chunks of 128 rows with every operand taken once (prompts); attention: the window's keys (prompts: multiplied out, in ``linear``)."""
+    d, W = cfg.width, roofline.ClassWork
+    out = {k: W() for k in ("rows_seam", "rows_conv", "rows_state", "rows_state_tc", "rows_state_turn", "rows_gated_norm", "rows_latent_append", "rows_head_proj",
+                            "rows_latent_decode", "rows_attn_tc", "rows_gather_pages", "rows_act_mul", "linear", "head")}
+    out["rows_attn"] = out["rows_latent_decode"]
+
+    def linear(k, m, rows=n):
+        out["linear"].flops += 2.0 * rows * k * m
+        out["linear"].bytes += 2.0 * (k * m + rows * (k + m))
+
+    def state(H, G, N, P, cols, turned):
+        segs = n if decode else 1
+        if decode:
+            out["rows_state"].bytes += segs * H * N * P * 8.0 + 2.0 * n * (cols + H * P)
+        else:
+            out["rows_state_tc"].bytes += segs * H * N * P * 8.0 + 2.0 * n * (cols + H * P)
+            out["rows_state_tc"].flops += n * H * (2.0 * 128 * (N + P) / 2 + 4.0 * N * P)
+            out["rows_state_turn"].bytes += 2.0 * n * 6 * H * N if turned else 0.0
+    out["rows_seam"].bytes += n * d * 8.0
+    for L in cfg.layers:
+        m, H = L.mixer, L.mixer["heads"]
+        inner = H * m["vdim"]
+        linear(inner, d)
+        if L.type == "mamba2":
+            bc = 2 * m["groups"] * m["state"]
+            linear(d, 2 * inner + bc + H)
+            state(H, m["groups"], m["state"], m["vdim"], inner + bc + H, False)
+            out["rows_conv"].bytes += 0.0 if decode else 4.0 * n * (inner + bc)
+            out["rows_gated_norm"].bytes += 6.0 * n * inner
+        elif L.type == "retention":
+            linear(d, 2 * H * m["dim"] + 2 * inner)
+            state(H, H, m["dim"], m["vdim"], 2 * H * m["dim"] + inner, True)
+            out["rows_gated_norm"].bytes += 6.0 * n * inner
+        else:
+            r, key, win = m["kv_rank"], m["kv_rank"] + m["rot_dim"], min(m["mask"]["size"], ctx)
+            qd = m["dim"] + m["rot_dim"]
+            linear(d, H * qd + key)
+            out["rows_latent_append"].bytes += 2.0 * n * (2 * H * m["rot_dim"] + 2 * key)
+            if decode:
+                out["rows_head_proj"].bytes += 2.0 * H * r * (m["dim"] + m["vdim"]) + 2.0 * n * H * (m["dim"] + m["vdim"] + r + key)
+                out["rows_latent_decode"].bytes += 2.0 * n * (win * key + H * (key + r))
+                out["rows_latent_decode"].flops += 2.0 * n * H * win * (key + r)
+            else:
+                keys = n + min(ctx - n, win - 1)
+                out["rows_gather_pages"].bytes += 4.0 * keys * key
+                linear(r, H * (m["dim"] + m["vdim"]), keys)
+                seen = n * win if ctx - n >= win else n * (ctx - n) + n * (n + 1) / 2
+                out["rows_attn_tc"].flops += 2.0 * H * seen * (qd + m["vdim"])
+                out["rows_attn_tc"].bytes += 2.0 * (n * H * (qd + m["vdim"]) + keys * H * (m["dim"] + m["vdim"]))
+        out["rows_seam"].bytes += n * d * 12.0
+        if L.ff is not None:
+            linear(d, 2 * L.ff)
+            linear(L.ff, d)
+            out["rows_act_mul"].bytes += n * L.ff * 6.0
+            out["rows_seam"].bytes += n * d * 12.0
+    out["head"].flops += 2.0 * head_rows * cfg.vocab * d
+    out["head"].bytes += 2.0 * cfg.vocab * d
+    return out
+
+
+def fanodra_work(cfg: FanodraConfig, n: int, ctx: int, head_rows: int, decode: bool) -> dict[str, roofline.ClassWork]:
     """Bytes that must move and FLOPs that must be done by a step of n rows that ends at ``ctx`` cached positions (prefill: one
     segment; decode: one row in each of n lanes), per launch name."""
     d, W = cfg.width, roofline.ClassWork
@@ -165,9 +252,12 @@ def _fractions(timings: list[list[tuple[str, float]]], wk: dict[str, roofline.Cl
     return out
 
 
-def kernel_table(name: str, rows: int = 4096, ctx: int = 8192, reps: int = 5) -> list[dict]:
+WORK = {"fanodra": fanodra_work, "gudutar": gudutar_work}
+
+
+def kernel_table(design: str, name: str, rows: int = 4096, ctx: int = 8192, reps: int = 5) -> list[dict]:
     """Roofline fractions per kernel of one prompt portion (the last ``rows`` of ``ctx`` positions)."""
-    eng = engine(name, 1, ctx + 64, rows)
+    eng = engine(design, name, 1, ctx + 64, rows)
     ids = torch.randint(0, eng.model.vocab, (ctx,), generator=torch.Generator().manual_seed(0)).tolist()
     for a in range(0, ctx - rows, rows):
         eng.step(ids[a:a + rows], [0] * rows, list(range(a, a + rows)), head=False)
@@ -178,12 +268,12 @@ def kernel_table(name: str, rows: int = 4096, ctx: int = 8192, reps: int = 5) ->
     eng.check_status()
     cfg = eng.cfg
     eng.close()
-    return _fractions(ts[1:], work(cfg, rows, ctx, 1, False))
+    return _fractions(ts[1:], WORK[design](cfg, rows, ctx, 1, False))
 
 
-def decode_table(name: str, n: int = 16, ctx: int = 8192, reps: int = 5) -> list[dict]:
+def decode_table(design: str, name: str, n: int = 16, ctx: int = 8192, reps: int = 5) -> list[dict]:
     """The same of a decode step of n rows against ``ctx`` cached tokens each."""
-    eng = engine(name, n, ctx + 64, 4096)
+    eng = engine(design, name, n, ctx + 64, 4096)
     eng.use_graphs = False
     ids = torch.randint(0, eng.model.vocab, (ctx,), generator=torch.Generator().manual_seed(0)).tolist()
     for lane in range(n):
@@ -194,10 +284,11 @@ def decode_table(name: str, n: int = 16, ctx: int = 8192, reps: int = 5) -> list
     eng.check_status()
     cfg = eng.cfg
     eng.close()
-    wk = work(cfg, n, ctx, n, True)
+    wk = WORK[design](cfg, n, ctx, n, True)
     if n <= 4:           # the streaming products take the projections and the head, gate and up fused with their activation
         wk["rows_gemv"] = roofline.ClassWork(wk["linear"].bytes + wk["head"].bytes, wk["linear"].flops + wk["head"].flops)
-    wk["rows_attn_stream"] = wk["rows_attn"]
+    if design == "fanodra":
+        wk["rows_attn_stream"] = wk["rows_attn"]
     return _fractions(ts[1:], wk)
 
 
@@ -254,12 +345,18 @@ def _meta_weights(c):
         torch.randn = real
 
 
-def run(sizes: list[str], steps: int, compare: bool = True) -> dict:
+def measure(design: str, name: str, steps: int) -> dict:
+    out = {"throughput": throughput(design, name, steps=steps), "prefill_kernels": kernel_table(design, name),
+           "decode16_kernels": decode_table(design, name, 16), "decode1_kernels": decode_table(design, name, 1)}
+    torch.cuda.empty_cache()
+    return out
+
+
+def run(design: str, sizes: list[str], steps: int, compare: bool = True) -> dict:
     out = {}
     for name in sizes:
-        out[name] = {"throughput": throughput(name, steps=steps), "prefill_kernels": kernel_table(name), "decode16_kernels": decode_table(name, 16),
-                     "decode1_kernels": decode_table(name, 1)}
+        out[name] = measure(design, name, steps)
         if compare:
-            out[name]["closest_model"] = closest(name)
+            out[name]["closest_model"] = closest(name) if design == "fanodra" else measure("fanodra", name, steps)
         torch.cuda.empty_cache()
     return out
