@@ -79,7 +79,7 @@ constexpr int HP_R = 4, HP_T = 256;                    // rows and threads per b
 template <typename T, int V, int MG>
 __global__ void __launch_bounds__(HP_T) head_proj_kernel(HeadProjArgs a) {
   extern __shared__ __align__(16) float sm[];          // x [HP_R][K], then partials [KG][HP_R][HP_M] (before that: merge weights)
-  constexpr int HP_M = MG * 8, KG = HP_T / MG, PRE = 4;
+  constexpr int HP_M = MG * 8, KG = HP_T / MG, PRE = 8;
   float* xs = sm;
   float* red = sm + ((HP_R * a.K + 3) & ~3);
   const int tid = threadIdx.x, mg = tid % MG, kg = tid / MG;
@@ -101,6 +101,7 @@ __global__ void __launch_bounds__(HP_T) head_proj_kernel(HeadProjArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   if (a.part) {
+    __shared__ int wn[HP_R];
     float* wt = red;                                   // [HP_R][blocks]
     const int warp = tid >> 5, lane = tid & 31;
     if (warp < nr) {
@@ -112,21 +113,25 @@ __global__ void __launch_bounds__(HP_T) head_proj_kernel(HeadProjArgs a) {
       m = warp_max(m);
       for (int b = lane; b < nb; b += 32) l += ml[2 * b + 1] * exp2f(ml[2 * b] - m);
       const float inv = 1.f / warp_sum(l);
-      for (int b = lane; b < a.blocks; b += 32) wt[warp * a.blocks + b] = b < nb ? exp2f(ml[2 * b] - m) * inv : 0.f;
+      for (int b = lane; b < nb; b += 32) wt[warp * a.blocks + b] = exp2f(ml[2 * b] - m) * inv;
+      if (lane == 0) wn[warp] = nb;
     }
     __syncthreads();
-    for (int i = tid; i < HP_R * a.K; i += HP_T) {
-      const int r = i / a.K, k = i - r * a.K;
-      float f = 0.f;
+    const int K4 = a.K >> 2;                           // K (the latent's size) is a multiple of eight
+    for (int i = tid; i < HP_R * K4; i += HP_T) {
+      const int r = i / K4, k = (i - r * K4) * 4;
+      float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
       if (r < nr) {
+        const int nb = wn[r];
         const float* p = a.part + ((size_t)(r0 + r) * a.H + h) * a.blocks * a.K + k;
-#pragma unroll 4
-        for (int b = 0; b < a.blocks; ++b) {
+#pragma unroll 8
+        for (int b = 0; b < nb; ++b) {
           const float wb = wt[r * a.blocks + b];
-          if (wb != 0.f) f = fmaf(wb, p[(size_t)b * a.K], f);
+          const float4 v = *reinterpret_cast<const float4*>(p + (size_t)b * a.K);
+          f.x = fmaf(wb, v.x, f.x); f.y = fmaf(wb, v.y, f.y); f.z = fmaf(wb, v.z, f.z); f.w = fmaf(wb, v.w, f.w);
         }
       }
-      xs[i] = f;
+      *reinterpret_cast<float4*>(xs + r * a.K + k) = f;
     }
   } else {
     for (int i = tid; i < HP_R * a.K; i += HP_T) {
@@ -239,7 +244,7 @@ int sfb_rows_latent_append(void* proj, int64_t stride, const void* w, const void
 int sfb_rows_head_proj(const void* x, int64_t x_row, int64_t x_head, const void* w, void* out, int64_t out_row, int64_t out_head, const int* rows, int list,
                        const void* part, const void* ml, const int* row_pos, int window, int blocks, int n, int H, int K, int M, int tail, int fp32,
                        cudaStream_t stream) {
-  if (n < 1 || n > 65535 * HP_R || H < 1 || K < 1 || M < 1 || K > 8192 || (part && (blocks < 1 || tail || list == 1))) return (int)cudaErrorInvalidValue;
+  if (n < 1 || n > 65535 * HP_R || H < 1 || K < 1 || M < 1 || K > 8192 || (part && (K % 8 || blocks < 1 || tail || list == 1))) return (int)cudaErrorInvalidValue;
   HeadProjArgs a{x, x_row, x_head, w, out, out_row, out_head, list ? rows : nullptr, (const float*)part, (const float*)ml, row_pos, window, part ? blocks : 0,
                  list == 1, list == 2, n, H, K, M, tail};
   return fp32 ? launch_head_proj_t<float>(a, stream) : launch_head_proj_t<__nv_bfloat16>(a, stream);

@@ -66,7 +66,7 @@ __device__ __forceinline__ float conv_silu(const StateArgs& a, T x, int ch, int 
 }
 
 template <typename T, int NI>
-__global__ void __launch_bounds__(256) state_rows_kernel(StateArgs a) {
+__global__ void __launch_bounds__(256, NI <= 4 ? 5 : NI <= 8 ? 3 : 1) state_rows_kernel(StateArgs a) {
   extern __shared__ __align__(16) float sm[];
   const int PT = blockDim.x >> 3, tiles = (a.P + PT - 1) / PT;
   const int h = blockIdx.x / tiles, tile = blockIdx.x % tiles, g = h / (a.H / a.G);

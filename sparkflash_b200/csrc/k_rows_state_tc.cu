@@ -44,7 +44,8 @@ struct Args {
 struct Ctl {
   float c[L];                      // running sum of log2 a, less log2 of the weight (chunk_out); weight of a row's values (chunk_sums)
   float part[4];
-  uint64_t full[3], done;
+  uint64_t full[3], done[2];       // copies; products (chunk_out: weighted ones, scores - a barrier each, since the next head's scores are issued
+                                   // before every thread has seen the products end)
   uint32_t tmem;
   int dead;
 };
@@ -76,7 +77,7 @@ __device__ __forceinline__ void setup(Ctl& C, uint32_t cols) {
   if (threadIdx.x == 0) {
     C.dead = 0;
     for (int i = 0; i < 3; ++i) mbar_init(&C.full[i], 1);
-    mbar_init(&C.done, 1);
+    for (int i = 0; i < 2; ++i) mbar_init(&C.done[i], 1);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
   if (threadIdx.x < 32) {
@@ -90,10 +91,16 @@ __device__ __forceinline__ void setup(Ctl& C, uint32_t cols) {
 __device__ __forceinline__ void teardown(Ctl& C, uint32_t cols, Status* status, int where) {
   fence_before();
   __syncthreads();
-  if (threadIdx.x == 0 && C.dead) status_set(status, ST_TIMEOUT, where, blockIdx.x, blockIdx.y);
+  if (threadIdx.x == 0 && C.dead) status_set(status, ST_TIMEOUT, where, C.dead, blockIdx.y << 16 | blockIdx.x);
   if (threadIdx.x < 32) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(C.tmem), "r"(cols) : "memory");
 }
 
+// a wait of whole warps: what follows it is executed by all lanes together
+// `id`: what the status word says if the wait gives up.
+__device__ __forceinline__ void wait_warp(uint64_t* b, uint32_t parity, volatile int* dead, int id) {
+  if (!mbar_wait(b, parity, dead) && *dead == 1) *dead = id;
+  __syncwarp();
+}
 // after a wait that gave up: copies and products under way must end before the CTA does (bounded: a phase that never comes is not waited for)
 __device__ __forceinline__ void drain(Ctl& C) {
   if (!C.dead) return;
@@ -102,15 +109,16 @@ __device__ __forceinline__ void drain(Ctl& C) {
 }
 
 // grid (groups x parts of a group's heads, chunks): k stays in shared memory while the heads (and their tiles of 64 value dims) go by
+template <int TERMS>
 __global__ void __launch_bounds__(THREADS)
 chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv, Args a) {
   extern __shared__ __align__(1024) uint8_t sm[];
   const int nb = (a.ns + 1) / 2;                          // blocks of 128 state rows
   uint8_t* ks = sm;                                       // [terms][2 nb] slabs
-  uint8_t* vh = ks + (size_t)a.terms * 2 * nb * SLAB;     // weighted values, upper terms (the copy lands here): two stages
+  uint8_t* vh = ks + (size_t)TERMS * 2 * nb * SLAB;     // weighted values, upper terms (the copy lands here): two stages
   uint8_t* vl = vh + 2 * SLAB;                            // lower terms
   Ctl& C = *reinterpret_cast<Ctl*>(vl + SLAB);
-  setup(C, 128);
+  setup(C, nb > 1 ? 256 : 128);
   pdl_launch_dependents();
   pdl_wait();
   const int chunk = blockIdx.y, rep = a.H / a.G, parts = (rep + a.hpc - 1) / a.hpc, g = blockIdx.x / parts;
@@ -122,78 +130,85 @@ chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant_
     tma2d(vh + (it & 1) * SLAB, &mv, a.v_col + (h0 + it / pts) * a.P + 64 * (it % pts), row0, &C.full[it & 1]);
   };
   if (warp == 0 && elect_one()) {
-    mbar_expect(&C.full[2], a.terms * a.ns * SLAB);
-    for (int t = 0; t < a.terms; ++t)
+    mbar_expect(&C.full[2], TERMS * a.ns * SLAB);
+    for (int t = 0; t < TERMS; ++t)
       for (int s = 0; s < a.ns; ++s) tma2d(ks + (size_t)(t * 2 * nb + s) * SLAB, &mk, a.k_col + t * a.k_lo + g * a.N + 64 * s, row0, &C.full[2]);
     fetch(0);
   }
-  const uint32_t id = idesc(64, 1, 1);
-  bool ok = mbar_wait(&C.full[2], 0, dead);
-  for (int it = 0; it < items; ++it) {
+  const uint32_t id = idesc(64, 1, 1), cols = 64 * nb;
+  const int w4 = warp & 3, half = warp >> 2;
+  auto decays = [&](int hi) {      // of the block's head hi
+    float w;
+    const float c = chunk_decays(a, C, h0 + hi, row0, rows, w), last = C.part[0] + C.part[1] + C.part[2] + C.part[3];
+    if (tid < L) C.c[tid] = ex2(last - c) * w;
+    if (tid == 0) a.dec[(size_t)chunk * a.H + h0 + hi] = ex2(last);
+  };
+  auto store = [&](int it) {       // lane = state row: columns of the tile go out as runs of consecutive state rows
     const int h = h0 + it / pts, pt = it % pts;
-    uint8_t* vs = vh + (it & 1) * SLAB;
-    if (pt == 0) {
-      float w;
-      const float c = chunk_decays(a, C, h, row0, rows, w), last = C.part[0] + C.part[1] + C.part[2] + C.part[3];
-      if (tid < L) C.c[tid] = ex2(last - c) * w;
-      if (tid == 0) a.dec[(size_t)chunk * a.H + h] = ex2(last);
+    for (int b = 0; b < nb; ++b) {
+      float f[32];
+      ld32(C.tmem + (it & 1) * cols + b * 64 + half * 32 + ((uint32_t)(w4 * 32) << 16), f);
+      wait_ld();
+      const int n = b * 128 + w4 * 32 + lane;
+      if (n < a.Np) {
+        float* o = a.sums + (((size_t)chunk * a.H + h) * a.P + pt * 64 + half * 32) * a.Np + n;
+        const int m = min(32, a.P - pt * 64 - half * 32);
+#pragma unroll
+        for (int c = 0; c < 32; ++c)
+          if (c < m) o[(size_t)c * a.Np] = n < a.N ? f[c] : 0.f;
+      }
     }
-    if (ok) ok = mbar_wait(&C.full[it & 1], (it >> 1) & 1, dead);
-    ok = __syncthreads_and(ok);
-    if (!ok) break;
+    fence_before();
+  };
+  decays(0);
+  wait_warp(&C.full[2], 0, dead, 2);
+  for (int it = 0; it < items; ++it) {
+    const int hi = it / pts;
+    uint8_t* vs = vh + (it & 1) * SLAB;
+    wait_warp(&C.full[it & 1], (it >> 1) & 1, dead, 3);
+    if (it > 0) wait_warp(&C.done[0], (it - 1) & 1, dead, 4);               // the other stage and the lower terms are free
+    __syncthreads();
+    fence_after();
     if (it + 1 < items && warp == 0 && elect_one()) fetch(it + 1);
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int u = tid + i * THREADS;                               // a 16-byte unit; its row is u / 8
       const float wt = C.c[u >> 3];
       float f[8];
-      uint4 hi, lo;
+      uint4 hv, lv;
       rows::load_v<__nv_bfloat16, 8>(reinterpret_cast<const __nv_bfloat16*>(vs) + u * 8, f);
 #pragma unroll
       for (int k = 0; k < 8; ++k) f[k] *= wt;
-      split2(f[0], f[1], hi.x, lo.x); split2(f[2], f[3], hi.y, lo.y); split2(f[4], f[5], hi.z, lo.z); split2(f[6], f[7], hi.w, lo.w);
-      reinterpret_cast<uint4*>(vs)[u] = hi;
-      reinterpret_cast<uint4*>(vl)[u] = lo;
+      split2(f[0], f[1], hv.x, lv.x); split2(f[2], f[3], hv.y, lv.y); split2(f[4], f[5], hv.z, lv.z); split2(f[6], f[7], hv.w, lv.w);
+      reinterpret_cast<uint4*>(vs)[u] = hv;
+      reinterpret_cast<uint4*>(vl)[u] = lv;
     }
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-    fence_before();
     __syncthreads();
-    fence_after();
-    if (warp == 0 && elect_one()) {
+    if (warp == 0 && elect_one() && !*dead) {
+      fence_after();
       const uint64_t dh = desc(smem_u32(vs), SLAB), dl = desc(smem_u32(vl), SLAB);
       for (int b = 0; b < nb; ++b) {
+        const uint32_t d = C.tmem + (it & 1) * cols + b * 64;
         const uint64_t k0 = desc(smem_u32(ks) + (2 * b) * SLAB, SLAB), k1 = desc(smem_u32(ks) + (2 * nb + 2 * b) * SLAB, SLAB);
+#pragma unroll
         for (int t = 0; t < 8; ++t) {
           const uint64_t o = (uint64_t)t * (2048 >> 4);
-          mma_ss(C.tmem + b * 64, k0 + o, dh + o, id, t ? 1u : 0u);
-          mma_ss(C.tmem + b * 64, k0 + o, dl + o, id, 1u);
-          if (a.terms > 1) mma_ss(C.tmem + b * 64, k1 + o, dh + o, id, 1u);
+          mma_ss(d, k0 + o, dh + o, id, t ? 1u : 0u);
+          mma_ss(d, k0 + o, dl + o, id, 1u);
+          if (TERMS > 1) mma_ss(d, k1 + o, dh + o, id, 1u);
         }
       }
-      commit(&C.done);
+      commit(&C.done[0]);
     }
-    ok = __syncthreads_and(mbar_wait(&C.done, it & 1, dead));
-    if (!ok) break;
-    fence_after();
-    // lane = state row: columns of the tile go out as runs of consecutive state rows
-    const int w4 = warp & 3, half = warp >> 2;
-    for (int b = 0; b < nb; ++b) {
-      float f[32];
-      ld32(C.tmem + b * 64 + half * 32 + ((uint32_t)(w4 * 32) << 16), f);
-      wait_ld();
-      const int n = b * 128 + w4 * 32 + lane;
-      if (n < a.Np) {
-        float* o = a.sums + (((size_t)chunk * a.H + h) * a.P + pt * 64 + half * 32) * a.Np + n;
-        const int cols = min(32, a.P - pt * 64 - half * 32);
-#pragma unroll
-        for (int c = 0; c < 32; ++c)
-          if (c < cols) o[(size_t)c * a.Np] = n < a.N ? f[c] : 0.f;
-      }
-    }
-    fence_before();
+    if (it > 0) store(it - 1);                                       // while the products run
+    if ((it + 1) % pts == 0 && it + 1 < items) decays(hi + 1);
   }
+  wait_warp(&C.done[0], (items - 1) & 1, dead, 5);
+  fence_after();
+  store(items - 1);
   drain(C);
-  teardown(C, 128, a.status, 69);
+  teardown(C, nb > 1 ? 256 : 128, a.status, 69);
 }
 
 // grid (elements / 1024, runs): a thread follows four elements through the run's chunks
@@ -235,15 +250,16 @@ __global__ void __launch_bounds__(256) chunk_starts_kernel(Args a) {
 
 // grid as chunk_sums: q and k stay in shared memory while the heads go by; the scores are computed again for every head (their tensor
 // memory is where the weighted scores go)
+template <int NS, int TERMS>
 __global__ void __launch_bounds__(THREADS, 2)
 chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv,
                  const __grid_constant__ CUtensorMap ms, Args a) {
   extern __shared__ __align__(1024) uint8_t sm[];
   uint8_t* qs = sm;                                      // [terms][ns] slabs
-  uint8_t* ks = qs + (size_t)a.terms * a.ns * SLAB;
-  uint8_t* vs = ks + (size_t)a.terms * a.ns * SLAB;      // one slab
+  uint8_t* ks = qs + (size_t)TERMS * NS * SLAB;
+  uint8_t* vs = ks + (size_t)TERMS * NS * SLAB;      // one slab
   uint8_t* ss = vs + SLAB;                               // start state, [2][ns] slabs of 64 rows
-  Ctl& C = *reinterpret_cast<Ctl*>(ss + (size_t)2 * a.ns * HSLAB);
+  Ctl& C = *reinterpret_cast<Ctl*>(ss + (size_t)2 * NS * HSLAB);
   setup(C, 256);
   pdl_launch_dependents();
   pdl_wait();
@@ -254,53 +270,52 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
   const uint32_t tp = C.tmem, ta = tp + 128, tb = tp + 192, lanes = (uint32_t)(w4 * 32) << 16;
   auto tile = [&](int it) {                              // values and start state of a tile of 64 value dims
     const int h = h0 + it / pts, pt = it % pts, y = (chunk * a.H + h) * a.P + 64 * pt;
-    mbar_expect(&C.full[0], SLAB + 2 * a.ns * HSLAB);
+    mbar_expect(&C.full[0], SLAB + 2 * NS * HSLAB);
     tma2d(vs, &mv, a.v_col + h * a.P + 64 * pt, row0, &C.full[0]);
     for (int t = 0; t < 2; ++t)
-      for (int s = 0; s < a.ns; ++s) tma2d(ss + (size_t)(t * a.ns + s) * HSLAB, &ms, 64 * s, t * a.chunks * a.H * a.P + y, &C.full[0]);
+      for (int s = 0; s < NS; ++s) tma2d(ss + (size_t)(t * NS + s) * HSLAB, &ms, 64 * s, t * a.chunks * a.H * a.P + y, &C.full[0]);
   };
   const int kst = a.N / 16;
-  const uint64_t lo = (uint64_t)a.ns * (SLAB >> 4), dq = desc(smem_u32(qs), 16), dk = desc(smem_u32(ks), 16);
+  const uint64_t lo = (uint64_t)NS * (SLAB >> 4), dq = desc(smem_u32(qs), 16), dk = desc(smem_u32(ks), 16);
   auto scores = [&]() {
     const uint32_t id = idesc(128, 0, 0);
-    for (int t = 0; t < kst; ++t) {
+#pragma unroll
+    for (int t = 0; t < 4 * NS; ++t) {
+      if (t >= kst) break;
       const uint64_t o = (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2;
       mma_ss(tp, dq + o, dk + o, id, t ? 1u : 0u);
-      if (a.terms > 1) {
+      if (TERMS > 1) {
         mma_ss(tp, dq + o, dk + lo + o, id, 1u);
         mma_ss(tp, dq + lo + o, dk + o, id, 1u);
       }
     }
-    commit(&C.done);
+    commit(&C.done[1]);
   };
   if (warp == 0 && elect_one()) {
-    mbar_expect(&C.full[2], 2 * a.terms * a.ns * SLAB);
-    for (int t = 0; t < a.terms; ++t)
-      for (int s = 0; s < a.ns; ++s) {
-        tma2d(qs + (size_t)(t * a.ns + s) * SLAB, &mq, a.q_col + t * a.q_lo + g * a.N + 64 * s, row0, &C.full[2]);
-        tma2d(ks + (size_t)(t * a.ns + s) * SLAB, &mk, a.k_col + t * a.k_lo + g * a.N + 64 * s, row0, &C.full[2]);
+    mbar_expect(&C.full[2], 2 * TERMS * NS * SLAB);
+    for (int t = 0; t < TERMS; ++t)
+      for (int s = 0; s < NS; ++s) {
+        tma2d(qs + (size_t)(t * NS + s) * SLAB, &mq, a.q_col + t * a.q_lo + g * a.N + 64 * s, row0, &C.full[2]);
+        tma2d(ks + (size_t)(t * NS + s) * SLAB, &mk, a.k_col + t * a.k_lo + g * a.N + 64 * s, row0, &C.full[2]);
       }
     tile(0);
   }
-  bool ok = __syncthreads_and(mbar_wait(&C.full[2], 0, dead));
-  if (ok && warp == 0 && elect_one()) {
-    fence_after();
-    scores();
-  }
   const int i = w4 * 32 + lane;
-  float ci = 0.f, ei = 0.f, D = 0.f;
-  uint32_t used = 0;                                     // completions of `done` that were waited for
-  for (int it = 0; it < items && ok; ++it) {
-    const int h = h0 + it / pts, pt = it % pts;
+  float ci, wi;
+  auto decays = [&](int hi) {                            // of the block's head hi
+    ci = chunk_decays(a, C, h0 + hi, row0, rows, wi);
+    if (tid < L) C.c[tid] = ci - __log2f(wi);    // weight 0: infinity, and its exponential below 0
+  };
+  decays(0);
+  wait_warp(&C.full[2], 0, dead, 6);
+  if (warp == 0 && elect_one()) scores();
+  float ei = 0.f;
+  for (int it = 0; it < items; ++it) {
+    const int hi = it / pts, h = h0 + hi, pt = it % pts;
     if (pt == 0) {
-      float w;
-      ci = chunk_decays(a, C, h, row0, rows, w);
-      if (tid < L) C.c[tid] = ci - __log2f(w);           // weight 0: infinity, and its exponential below 0
       ei = ex2(ci);
-      D = a.D ? a.D[h] : 0.f;
-      ok = __syncthreads_and(mbar_wait(&C.done, used & 1, dead));
-      if (!ok) break;
-      ++used;
+      const float D = a.D ? a.D[h] : 0.f;
+      wait_warp(&C.done[1], hi & 1, dead, 7);
       fence_after();
       float s[64];
       const bool any = w4 * 32 + 31 >= half * 64;        // the warp's rows reach these columns
@@ -312,46 +327,57 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
       fence_before();
       __syncthreads();                                   // every score has been read: the weighted ones may take their place
       fence_after();
+      const float* cs = C.c + half * 64;
+      const int vis = i - half * 64;                     // columns up to the row's own
 #pragma unroll
       for (int b = 0; b < 2; ++b) {
-        uint32_t hi[16], lw[16];
+        uint32_t hv[16], lv[16];
+        if (any) {
 #pragma unroll
-        for (int q = 0; q < 16; ++q) {
-          const int j = half * 64 + 32 * b + 2 * q;
-          float x = 0.f, y = 0.f;
-          if (any) {
-            const float2 cj = *reinterpret_cast<const float2*>(C.c + j);
-            x = j <= i ? s[32 * b + 2 * q] * ex2(ci - cj.x) : 0.f;
-            y = j + 1 <= i ? s[32 * b + 2 * q + 1] * ex2(ci - cj.y) : 0.f;
+          for (int q = 0; q < 16; ++q) {
+            const int j = 32 * b + 2 * q;
+            const float2 cj = *reinterpret_cast<const float2*>(cs + j);
+            float x = j <= vis ? s[j] * ex2(ci - cj.x) : 0.f, y = j + 1 <= vis ? s[j + 1] * ex2(ci - cj.y) : 0.f;
+            if (j == vis) x += D;                        // D v_i
+            if (j + 1 == vis) y += D;
+            split2(x, y, hv[q], lv[q]);
           }
-          split2(x, y, hi[q], lw[q]);
+        } else {
+#pragma unroll
+          for (int q = 0; q < 16; ++q) hv[q] = lv[q] = 0u;
         }
-        st16(tp + half * 32 + 16 * b + lanes, hi);
-        st16(tp + 64 + half * 32 + 16 * b + lanes, lw);
+        st16(tp + half * 32 + 16 * b + lanes, hv);
+        st16(tp + 64 + half * 32 + 16 * b + lanes, lv);
       }
       wait_st();
       fence_before();
     }
-    ok = __syncthreads_and(mbar_wait(&C.full[0], it & 1, dead));
-    if (!ok) break;
-    fence_after();
-    if (warp == 0 && elect_one()) {
+    wait_warp(&C.full[0], it & 1, dead, 8);
+    __syncthreads();                                     // weights are in place, accumulators have been read
+    if (warp == 0 && elect_one() && !*dead) {
+      fence_after();
       const uint32_t ia = idesc(64, 0, 1), ib = idesc(64, 0, 0);
-      const uint64_t dv = desc(smem_u32(vs), SLAB), ds = desc(smem_u32(ss), 16), sl = (uint64_t)a.ns * (HSLAB >> 4);
-      for (int t = 0; t < 16; ++t) mma_ts(ta, tp + (t & 7) * 8 + (t >> 3) * 64, dv + (uint64_t)(t & 7) * (2048 >> 4), ia, t ? 1u : 0u);
-      for (int t = 0; t < kst; ++t) {
+      const uint64_t dv = desc(smem_u32(vs), SLAB), ds = desc(smem_u32(ss), 16), sl = (uint64_t)NS * (HSLAB >> 4);
+#pragma unroll
+      for (int t = 0; t < 4 * NS; ++t) {
+        if (t >= kst) break;
         const uint64_t o = (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, os = (uint64_t)(t >> 2) * (HSLAB >> 4) + (t & 3) * 2;
         mma_ss(tb, dq + o, ds + os, ib, t ? 1u : 0u);
         mma_ss(tb, dq + o, ds + sl + os, ib, 1u);
-        if (a.terms > 1) mma_ss(tb, dq + lo + o, ds + os, ib, 1u);
+        if (TERMS > 1) mma_ss(tb, dq + lo + o, ds + os, ib, 1u);
       }
-      commit(&C.done);
+#pragma unroll
+      for (int t = 0; t < 16; ++t) mma_ts(ta, tp + (t & 7) * 8 + (t >> 3) * 64, dv + (uint64_t)(t & 7) * (2048 >> 4), ia, t ? 1u : 0u);
+      commit(&C.done[0]);
     }
-    ok = __syncthreads_and(mbar_wait(&C.done, used & 1, dead));
-    if (!ok) break;
-    ++used;
+    const bool head_ends = pt + 1 == pts && it + 1 < items;
+    if (head_ends) decays(hi + 1);                       // while the products run
+    wait_warp(&C.done[0], it & 1, dead, 9);
     fence_after();
-    if (pt + 1 == pts && it + 1 < items && warp == 0 && elect_one()) scores();       // of the next head
+    if (it + 1 < items && warp == 0 && elect_one() && !*dead) {
+      if (head_ends) scores();                           // of the next head
+      tile(it + 1);
+    }
     __nv_bfloat16* o = a.y + ((size_t)(row0 + i) * a.H + h) * a.P + pt * 64 + half * 32;
     const int cols = min(32, a.P - pt * 64 - half * 32);
 #pragma unroll
@@ -363,19 +389,13 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
 #pragma unroll
       for (int u = 0; u < 2; ++u)
         if (i < rows && 16 * b + 8 * u < cols) {         // P is a multiple of eight
-          float f[8], v[8];
-          if (a.D) rows::load_v<__nv_bfloat16, 8>(reinterpret_cast<const __nv_bfloat16*>(vs + i * 128 + (((half * 4 + 2 * b + u) ^ (i & 7)) * 16)), v);
+          float f[8];
 #pragma unroll
-          for (int k = 0; k < 8; ++k) {
-            f[k] = fmaf(ei, z[8 * u + k], x[8 * u + k]);
-            if (a.D) f[k] = fmaf(D, v[k], f[k]);
-          }
+          for (int k = 0; k < 8; ++k) f[k] = fmaf(ei, z[8 * u + k], x[8 * u + k]);
           rows::store_v<__nv_bfloat16, 8>(o + 16 * b + 8 * u, f);
         }
     }
     fence_before();
-    __syncthreads();                                     // tile and accumulators have been read
-    if (it + 1 < items && warp == 0 && elect_one()) tile(it + 1);
   }
   drain(C);
   teardown(C, 256, a.status, 70);
@@ -427,6 +447,28 @@ __global__ void __launch_bounds__(256) state_turn_kernel(TurnArgs a) {
 static size_t sums_smem(const Args& a) { return (size_t)(a.terms * 2 * ((a.ns + 1) / 2) + 3) * SLAB + sizeof(Ctl); }
 static size_t out_smem(const Args& a) { return (size_t)(2 * a.terms * a.ns + 1) * SLAB + (size_t)2 * a.ns * HSLAB + sizeof(Ctl); }
 
+template <typename K>
+static cudaError_t grant(K kernel, size_t smem, size_t& granted) {
+  if (smem <= granted) return cudaSuccess;
+  const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  if (e == cudaSuccess) granted = smem;
+  return e;
+}
+template <int TERMS>
+static cudaError_t launch_sums(const CUtensorMap* k, const CUtensorMap* v, const Args& a, dim3 grid, cudaStream_t st) {
+  static size_t granted = 0;
+  const size_t smem = sums_smem(a);
+  const cudaError_t e = grant(chunk_sums_kernel<TERMS>, smem, granted);
+  return e != cudaSuccess ? e : sfb_launch(chunk_sums_kernel<TERMS>, grid, dim3(THREADS), smem, st, *k, *v, a);
+}
+template <int NS, int TERMS>
+static cudaError_t launch_out(const CUtensorMap* q, const CUtensorMap* k, const CUtensorMap* v, const CUtensorMap* s, const Args& a, dim3 grid, cudaStream_t st) {
+  static size_t granted = 0;
+  const size_t smem = out_smem(a);
+  const cudaError_t e = grant(chunk_out_kernel<NS, TERMS>, smem, granted);
+  return e != cudaSuccess ? e : sfb_launch(chunk_out_kernel<NS, TERMS>, grid, dim3(THREADS), smem, st, *q, *k, *v, *s, a);
+}
+
 }  // namespace rst
 }  // namespace sfb
 
@@ -459,25 +501,20 @@ int sfb_rows_state_tc(const void* mq, const void* mk, const void* mv, const void
   a.hpc = rep < 8 ? rep : 8;         // fewer heads per block where that leaves SMs empty
   while (a.hpc > 1 && (long long)G * ((rep + a.hpc - 1) / a.hpc) * chunks < 148) a.hpc = (a.hpc + 1) / 2;
   const int blocks = G * ((rep + a.hpc - 1) / a.hpc);
-  const size_t s1 = sums_smem(a), s2 = out_smem(a);
-  static size_t g1 = 0, g2 = 0;
-  if (s1 > g1) {
-    const cudaError_t e = cudaFuncSetAttribute(chunk_sums_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
-    if (e != cudaSuccess) return (int)e;
-    g1 = s1;
-  }
-  if (s2 > g2) {
-    const cudaError_t e = cudaFuncSetAttribute(chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2);
-    if (e != cudaSuccess) return (int)e;
-    g2 = s2;
-  }
   const CUtensorMap *q = (const CUtensorMap*)mq, *k = (const CUtensorMap*)mk, *v = (const CUtensorMap*)mv, *s = (const CUtensorMap*)ms;
-  cudaError_t rc = sfb_launch(chunk_sums_kernel, dim3(blocks, chunks), dim3(THREADS), s1, stream, *k, *v, a);
+  const dim3 grid(blocks, chunks);
+  cudaError_t rc = terms > 1 ? launch_sums<2>(k, v, a, grid, stream) : launch_sums<1>(k, v, a, grid, stream);
   if (rc != cudaSuccess) return (int)rc;
   const size_t per = (size_t)H * P * Np;
   rc = sfb_launch(chunk_starts_kernel, dim3((unsigned)((per / 4 + 255) / 256), runs), dim3(256), 0, stream, a);
   if (rc != cudaSuccess) return (int)rc;
-  return (int)sfb_launch(chunk_out_kernel, dim3(blocks, chunks), dim3(THREADS), s2, stream, *q, *k, *v, *s, a);
+  if (terms > 1) return (int)(ns == 1 ? launch_out<1, 2>(q, k, v, s, a, grid, stream) : launch_out<2, 2>(q, k, v, s, a, grid, stream));
+  switch (ns) {
+    case 1: return (int)launch_out<1, 1>(q, k, v, s, a, grid, stream);
+    case 2: return (int)launch_out<2, 1>(q, k, v, s, a, grid, stream);
+    case 3: return (int)launch_out<3, 1>(q, k, v, s, a, grid, stream);
+    default: return (int)launch_out<4, 1>(q, k, v, s, a, grid, stream);
+  }
 }
 
 }  // extern "C"

@@ -14,6 +14,7 @@ import torch.nn.functional as F
 from ..ops import rows as R
 
 DECODE_ROWS = 64           # single rows of latent attention whose partial results are held at a time
+CONV_STEP_ROWS = 4         # up to this many single rows the matrix-state kernel applies the convolution itself (every head does B and C again)
 GATED_STEP_ROWS = 16       # up to this many single rows run convolution, gates and recurrence as one kernel
 
 
@@ -266,7 +267,7 @@ class StateSpaceMixer:
         proj = R.linear(h, self.w_in, None, s.scratch.get("proj", n, self.w_in.shape[0]))
         z, u, dt = proj[:, :i], proj[:, i:i + self.channels], proj[:, i + self.channels:]
         y = s.scratch.get("mix_y", n, i)
-        conv = (self.cw, self.cb, run["conv"], (i + bc, i, 0)) if s.single else None
+        conv = (self.cw, self.cb, run["conv"], (i + bc, i, 0)) if s.single and n <= CONV_STEP_ROWS else None
         if conv is None:
             raw, u = u, s.scratch.get("mix_u", n, self.channels)
             R.conv(raw, self.cw, self.cb, u, run["conv"], s, n, R.CONV_SILU)
