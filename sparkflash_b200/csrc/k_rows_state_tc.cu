@@ -51,19 +51,23 @@ struct Ctl {
 };
 
 // Running sum of log2 a up to the thread's row (thread t: row t & 127) and the row's weight; past the end: decay 1, weight 0.  One barrier.
-__device__ __forceinline__ float chunk_decays(const Args& a, Ctl& C, int h, int row0, int rows, float& w) {
+// What it reads from memory (chunk_rate) is requested a head ahead.
+struct Rate {
+  float z, a;                      // raw step size with its bias; A or the logarithm of the decay
+};
+__device__ __forceinline__ Rate chunk_rate(const Args& a, int h, int row0, int rows) {
+  const int t = threadIdx.x & (L - 1);
+  Rate r{0.f, a.a[h]};
+  if (a.dt && t < rows) r.z = __bfloat162float(a.dt[(size_t)(row0 + t) * a.dt_stride + h]) + a.dt_bias[h];
+  return r;
+}
+__device__ __forceinline__ float chunk_decays(const Args& a, Ctl& C, const Rate& r, int rows, float& w) {
   const int t = threadIdx.x & (L - 1), lane = t & 31, warp = t >> 5;
   float la = 0.f;
   w = 0.f;
   if (t < rows) {
-    if (a.dt) {
-      const float z = __bfloat162float(a.dt[(size_t)(row0 + t) * a.dt_stride + h]) + a.dt_bias[h];
-      w = log1pf(expf(-fabsf(z))) + fmaxf(z, 0.f);
-      la = a.a[h] * w * LOG2E;
-    } else {
-      w = 1.f;
-      la = a.a[h] * LOG2E;
-    }
+    w = a.dt ? log1pf(expf(-fabsf(r.z))) + fmaxf(r.z, 0.f) : 1.f;
+    la = r.a * w * LOG2E;
   }
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) { const float v = __shfl_up_sync(0xffffffffu, la, o); if (lane >= o) la += v; }
@@ -124,12 +128,13 @@ chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant_
   const int chunk = blockIdx.y, rep = a.H / a.G, parts = (rep + a.hpc - 1) / a.hpc, g = blockIdx.x / parts;
   const int h0 = g * rep + (blockIdx.x % parts) * a.hpc, nh = min(a.hpc, (g + 1) * rep - h0), row0 = a.c_row0[chunk], rows = a.c_rows[chunk];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, pts = (a.P + 63) / 64, items = nh * pts;
+  const bool leader = __shfl_sync(0xffffffffu, warp, 0) == 0;          // uniform: the elected thread's operands stay in uniform registers
   volatile int* dead = &C.dead;
   auto fetch = [&](int it) {
     mbar_expect(&C.full[it & 1], SLAB);
     tma2d(vh + (it & 1) * SLAB, &mv, a.v_col + (h0 + it / pts) * a.P + 64 * (it % pts), row0, &C.full[it & 1]);
   };
-  if (warp == 0 && elect_one()) {
+  if (leader) if (elect_one()) {
     mbar_expect(&C.full[2], TERMS * a.ns * SLAB);
     for (int t = 0; t < TERMS; ++t)
       for (int s = 0; s < a.ns; ++s) tma2d(ks + (size_t)(t * 2 * nb + s) * SLAB, &mk, a.k_col + t * a.k_lo + g * a.N + 64 * s, row0, &C.full[2]);
@@ -137,11 +142,13 @@ chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant_
   }
   const uint32_t id = idesc(64, 1, 1), cols = 64 * nb;
   const int w4 = warp & 3, half = warp >> 2;
+  Rate rate = chunk_rate(a, h0, row0, rows);
   auto decays = [&](int hi) {      // of the block's head hi
     float w;
-    const float c = chunk_decays(a, C, h0 + hi, row0, rows, w), last = C.part[0] + C.part[1] + C.part[2] + C.part[3];
+    const float c = chunk_decays(a, C, rate, rows, w), last = C.part[0] + C.part[1] + C.part[2] + C.part[3];
     if (tid < L) C.c[tid] = ex2(last - c) * w;
     if (tid == 0) a.dec[(size_t)chunk * a.H + h0 + hi] = ex2(last);
+    if (hi + 1 < nh) rate = chunk_rate(a, h0 + hi + 1, row0, rows);
   };
   auto store = [&](int it) {       // lane = state row: columns of the tile go out as runs of consecutive state rows
     const int h = h0 + it / pts, pt = it % pts;
@@ -169,7 +176,7 @@ chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant_
     if (it > 0) wait_warp(&C.done[0], (it - 1) & 1, dead, 4);               // the other stage and the lower terms are free
     __syncthreads();
     fence_after();
-    if (it + 1 < items && warp == 0 && elect_one()) fetch(it + 1);
+    if (it + 1 < items && leader) if (elect_one()) fetch(it + 1);
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int u = tid + i * THREADS;                               // a 16-byte unit; its row is u / 8
@@ -185,7 +192,7 @@ chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant_
     }
     asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     __syncthreads();
-    if (warp == 0 && elect_one() && !*dead) {
+    if (leader) if (elect_one()) {
       fence_after();
       const uint64_t dh = desc(smem_u32(vs), SLAB), dl = desc(smem_u32(vl), SLAB);
       for (int b = 0; b < nb; ++b) {
@@ -266,6 +273,7 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
   const int chunk = blockIdx.y, rep = a.H / a.G, parts = (rep + a.hpc - 1) / a.hpc, g = blockIdx.x / parts;
   const int h0 = g * rep + (blockIdx.x % parts) * a.hpc, nh = min(a.hpc, (g + 1) * rep - h0), row0 = a.c_row0[chunk], rows = a.c_rows[chunk];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, pts = (a.P + 63) / 64, items = nh * pts, w4 = warp & 3, half = warp >> 2;
+  const bool leader = __shfl_sync(0xffffffffu, warp, 0) == 0;          // uniform: the elected thread's operands stay in uniform registers
   volatile int* dead = &C.dead;
   const uint32_t tp = C.tmem, ta = tp + 128, tb = tp + 192, lanes = (uint32_t)(w4 * 32) << 16;
   auto tile = [&](int it) {                              // values and start state of a tile of 64 value dims
@@ -291,7 +299,7 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
     }
     commit(&C.done[1]);
   };
-  if (warp == 0 && elect_one()) {
+  if (leader) if (elect_one()) {
     mbar_expect(&C.full[2], 2 * TERMS * NS * SLAB);
     for (int t = 0; t < TERMS; ++t)
       for (int s = 0; s < NS; ++s) {
@@ -302,13 +310,15 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
   }
   const int i = w4 * 32 + lane;
   float ci, wi;
+  Rate rate = chunk_rate(a, h0, row0, rows);
   auto decays = [&](int hi) {                            // of the block's head hi
-    ci = chunk_decays(a, C, h0 + hi, row0, rows, wi);
-    if (tid < L) C.c[tid] = ci - __log2f(wi);    // weight 0: infinity, and its exponential below 0
+    ci = chunk_decays(a, C, rate, rows, wi);
+    if (tid < L) C.c[tid] = ci - __log2f(wi);            // weight 0: infinity, and its exponential below 0
+    if (hi + 1 < nh) rate = chunk_rate(a, h0 + hi + 1, row0, rows);
   };
   decays(0);
   wait_warp(&C.full[2], 0, dead, 6);
-  if (warp == 0 && elect_one()) scores();
+  if (leader) if (elect_one()) scores();
   float ei = 0.f;
   for (int it = 0; it < items; ++it) {
     const int hi = it / pts, h = h0 + hi, pt = it % pts;
@@ -318,28 +328,33 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
       wait_warp(&C.done[1], hi & 1, dead, 7);
       fence_after();
       float s[64];
-      const bool any = w4 * 32 + 31 >= half * 64;        // the warp's rows reach these columns
-      if (any) {
-        ld32(tp + half * 64 + lanes, s);
-        ld32(tp + half * 64 + 32 + lanes, s + 32);
-        wait_ld();
-      }
+      // blocks of 32 columns: before the warp's diagonal block all are visible, after it none
+      if (2 * half <= w4) ld32(tp + half * 64 + lanes, s);
+      if (2 * half + 1 <= w4) ld32(tp + half * 64 + 32 + lanes, s + 32);
+      wait_ld();
       fence_before();
       __syncthreads();                                   // every score has been read: the weighted ones may take their place
       fence_after();
       const float* cs = C.c + half * 64;
-      const int vis = i - half * 64;                     // columns up to the row's own
 #pragma unroll
       for (int b = 0; b < 2; ++b) {
+        const int blk = 2 * half + b;
         uint32_t hv[16], lv[16];
-        if (any) {
+        if (blk < w4) {
 #pragma unroll
           for (int q = 0; q < 16; ++q) {
             const int j = 32 * b + 2 * q;
             const float2 cj = *reinterpret_cast<const float2*>(cs + j);
-            float x = j <= vis ? s[j] * ex2(ci - cj.x) : 0.f, y = j + 1 <= vis ? s[j + 1] * ex2(ci - cj.y) : 0.f;
-            if (j == vis) x += D;                        // D v_i
-            if (j + 1 == vis) y += D;
+            split2(s[j] * ex2(ci - cj.x), s[j + 1] * ex2(ci - cj.y), hv[q], lv[q]);
+          }
+        } else if (blk == w4) {
+#pragma unroll
+          for (int q = 0; q < 16; ++q) {
+            const int j = 32 * b + 2 * q;
+            const float2 cj = *reinterpret_cast<const float2*>(cs + j);
+            float x = 2 * q <= lane ? s[j] * ex2(ci - cj.x) : 0.f, y = 2 * q + 1 <= lane ? s[j + 1] * ex2(ci - cj.y) : 0.f;
+            if (2 * q == lane) x += D;                   // D v_i
+            if (2 * q + 1 == lane) y += D;
             split2(x, y, hv[q], lv[q]);
           }
         } else {
@@ -354,7 +369,7 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
     }
     wait_warp(&C.full[0], it & 1, dead, 8);
     __syncthreads();                                     // weights are in place, accumulators have been read
-    if (warp == 0 && elect_one() && !*dead) {
+    if (leader) if (elect_one()) {
       fence_after();
       const uint32_t ia = idesc(64, 0, 1), ib = idesc(64, 0, 0);
       const uint64_t dv = desc(smem_u32(vs), SLAB), ds = desc(smem_u32(ss), 16), sl = (uint64_t)NS * (HSLAB >> 4);
@@ -374,7 +389,7 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
     if (head_ends) decays(hi + 1);                       // while the products run
     wait_warp(&C.done[0], it & 1, dead, 9);
     fence_after();
-    if (it + 1 < items && warp == 0 && elect_one() && !*dead) {
+    if (it + 1 < items && leader) if (elect_one()) {
       if (head_ends) scores();                           // of the next head
       tile(it + 1);
     }
