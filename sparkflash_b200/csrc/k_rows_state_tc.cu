@@ -19,7 +19,8 @@ namespace sfb {
 namespace rst {
 using namespace tc;
 
-constexpr int L = 128, SLAB = L * 128, HSLAB = 64 * 128, THREADS = 256;      // rows of a chunk; bytes of 128 / 64 rows of 64 elements
+constexpr int L = 128, SLAB = L * 128, HSLAB = 64 * 128;         // rows of a chunk; bytes of 128 / 64 rows of 64 elements
+constexpr int WORK = 256, THREADS = WORK + 32, HEADS = 8;        // threads that compute, and one warp that issues copies and products; heads per block
 
 struct Args {
   const int *c_row0, *c_rows;      // chunks
@@ -32,49 +33,53 @@ struct Args {
   float* S;                        // [slots, H, P, Np]
   float* sums;                     // [chunks, H, P, Np]
   float* dec;                      // [chunks, H] decay over the whole chunk
+  float* rates;                    // [chunks, H, 2, 128] running sum of log2 a; the same less log2 of the weight
   __nv_bfloat16* starts;           // [2, chunks, H, P, Np]: upper terms, then lower terms
   __nv_bfloat16* y;                // [n, H P]
   int H, G, N, P, Np, ns, terms;   // ns: 64-element slabs of a q / k row
   int q_col, k_col, v_col;         // first columns in the maps
   int q_lo, k_lo;                  // distance to the columns of the lower terms
   int chunks, hpc;                 // hpc: heads per block
+  int wide;                        // outputs lie on 32-byte boundaries
   Status* status;
 };
 
 struct Ctl {
-  float c[L];                      // running sum of log2 a, less log2 of the weight (chunk_out); weight of a row's values (chunk_sums)
-  float part[4];
   uint64_t full[3], done[2];       // copies; products (chunk_out: weighted ones, scores - a barrier each, since the next head's scores are issued
                                    // before every thread has seen the products end)
   uint32_t tmem;
   int dead;
 };
 
-// Running sum of log2 a up to the thread's row (thread t: row t & 127) and the row's weight; past the end: decay 1, weight 0.  One barrier.
-// What it reads from memory (chunk_rate) is requested a head ahead.
-struct Rate {
-  float z, a;                      // raw step size with its bias; A or the logarithm of the decay
-};
-__device__ __forceinline__ Rate chunk_rate(const Args& a, int h, int row0, int rows) {
-  const int t = threadIdx.x & (L - 1);
-  Rate r{0.f, a.a[h]};
-  if (a.dt && t < rows) r.z = __bfloat162float(a.dt[(size_t)(row0 + t) * a.dt_stride + h]) + a.dt_bias[h];
-  return r;
-}
-__device__ __forceinline__ float chunk_decays(const Args& a, Ctl& C, const Rate& r, int rows, float& w) {
-  const int t = threadIdx.x & (L - 1), lane = t & 31, warp = t >> 5;
-  float la = 0.f;
-  w = 0.f;
-  if (t < rows) {
-    w = a.dt ? log1pf(expf(-fabsf(r.z))) + fmaxf(r.z, 0.f) : 1.f;
-    la = r.a * w * LOG2E;
-  }
+// One warp, one head: running sums of log2 a over the chunk's rows (a lane takes four), weights; past the end: decay 1, weight 0.  The
+// numbers go to memory for chunk_out, the factors of the values (decay to the chunk's end times weight) to `wt`.
+__device__ __forceinline__ void head_rates(const Args& a, int chunk, int h, int row0, int rows, float* wt) {
+  const int lane = threadIdx.x & 31;
+  const float ah = a.a[h] * LOG2E, bias = a.dt ? a.dt_bias[h] : 0.f;
+  float z[4], w[4], c[4], t = 0.f;
 #pragma unroll
-  for (int o = 1; o < 32; o <<= 1) { const float v = __shfl_up_sync(0xffffffffu, la, o); if (lane >= o) la += v; }
-  if (lane == 31 && threadIdx.x < L) C.part[warp] = la;
-  __syncthreads();
-  for (int i = 0; i < warp; ++i) la += C.part[i];
-  return la;
+  for (int k = 0; k < 4; ++k) z[k] = a.dt && lane * 4 + k < rows ? __bfloat162float(a.dt[(size_t)(row0 + lane * 4 + k) * a.dt_stride + h]) + bias : 0.f;
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    w[k] = lane * 4 + k >= rows ? 0.f : a.dt ? log1pf(expf(-fabsf(z[k]))) + fmaxf(z[k], 0.f) : 1.f;
+    t += ah * w[k];
+    c[k] = t;
+  }
+  float s = t;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) { const float v = __shfl_up_sync(0xffffffffu, s, o); if (lane >= o) s += v; }
+  const float last = __shfl_sync(0xffffffffu, s, 31), before = s - t;
+  float* out = a.rates + ((size_t)chunk * a.H + h) * 2 * L + lane * 4;
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    c[k] += before;
+    wt[lane * 4 + k] = ex2(last - c[k]) * w[k];
+  }
+  rows::store_v<float, 4>(out, c);
+#pragma unroll
+  for (int k = 0; k < 4; ++k) c[k] -= __log2f(w[k]);       // weight 0: infinity, and its exponential below 0
+  rows::store_v<float, 4>(out + L, c);
+  if (lane == 0) a.dec[(size_t)chunk * a.H + h] = ex2(last);
 }
 
 __device__ __forceinline__ void setup(Ctl& C, uint32_t cols) {
@@ -105,6 +110,14 @@ __device__ __forceinline__ void wait_warp(uint64_t* b, uint32_t parity, volatile
   if (!mbar_wait(b, parity, dead) && *dead == 1) *dead = id;
   __syncwarp();
 }
+// sixteen values as one 32-byte store (a whole sector)
+__device__ __forceinline__ void store32(__nv_bfloat16* p, const float* f) {
+  uint32_t w[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) { const __nv_bfloat162 t = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]); w[i] = *reinterpret_cast<const uint32_t*>(&t); }
+  asm volatile("st.global.v8.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(p), "r"(w[0]), "r"(w[1]), "r"(w[2]), "r"(w[3]), "r"(w[4]), "r"(w[5]), "r"(w[6]),
+               "r"(w[7]) : "memory");
+}
 // after a wait that gave up: copies and products under way must end before the CTA does (bounded: a phase that never comes is not waited for)
 __device__ __forceinline__ void drain(Ctl& C) {
   if (!C.dead) return;
@@ -121,20 +134,21 @@ chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant_
   uint8_t* ks = sm;                                       // [terms][2 nb] slabs
   uint8_t* vh = ks + (size_t)TERMS * 2 * nb * SLAB;     // weighted values, upper terms (the copy lands here): two stages
   uint8_t* vl = vh + 2 * SLAB;                            // lower terms
-  Ctl& C = *reinterpret_cast<Ctl*>(vl + SLAB);
+  float* wts = reinterpret_cast<float*>(vl + SLAB);       // [HEADS][L] factors of the values
+  Ctl& C = *reinterpret_cast<Ctl*>(wts + HEADS * L);
   setup(C, nb > 1 ? 256 : 128);
   pdl_launch_dependents();
   pdl_wait();
   const int chunk = blockIdx.y, rep = a.H / a.G, parts = (rep + a.hpc - 1) / a.hpc, g = blockIdx.x / parts;
   const int h0 = g * rep + (blockIdx.x % parts) * a.hpc, nh = min(a.hpc, (g + 1) * rep - h0), row0 = a.c_row0[chunk], rows = a.c_rows[chunk];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, pts = (a.P + 63) / 64, items = nh * pts;
-  const bool leader = __shfl_sync(0xffffffffu, warp, 0) == 0;          // uniform: the elected thread's operands stay in uniform registers
+  const bool issuer = __shfl_sync(0xffffffffu, warp, 0) == WORK / 32;  // uniform: the elected thread's operands stay in uniform registers
   volatile int* dead = &C.dead;
   auto fetch = [&](int it) {
     mbar_expect(&C.full[it & 1], SLAB);
     tma2d(vh + (it & 1) * SLAB, &mv, a.v_col + (h0 + it / pts) * a.P + 64 * (it % pts), row0, &C.full[it & 1]);
   };
-  if (leader) if (elect_one()) {
+  if (issuer && elect_one()) {
     mbar_expect(&C.full[2], TERMS * a.ns * SLAB);
     for (int t = 0; t < TERMS; ++t)
       for (int s = 0; s < a.ns; ++s) tma2d(ks + (size_t)(t * 2 * nb + s) * SLAB, &mk, a.k_col + t * a.k_lo + g * a.N + 64 * s, row0, &C.full[2]);
@@ -142,14 +156,6 @@ chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant_
   }
   const uint32_t id = idesc(64, 1, 1), cols = 64 * nb;
   const int w4 = warp & 3, half = warp >> 2;
-  Rate rate = chunk_rate(a, h0, row0, rows);
-  auto decays = [&](int hi) {      // of the block's head hi
-    float w;
-    const float c = chunk_decays(a, C, rate, rows, w), last = C.part[0] + C.part[1] + C.part[2] + C.part[3];
-    if (tid < L) C.c[tid] = ex2(last - c) * w;
-    if (tid == 0) a.dec[(size_t)chunk * a.H + h0 + hi] = ex2(last);
-    if (hi + 1 < nh) rate = chunk_rate(a, h0 + hi + 1, row0, rows);
-  };
   auto store = [&](int it) {       // lane = state row: columns of the tile go out as runs of consecutive state rows
     const int h = h0 + it / pts, pt = it % pts;
     for (int b = 0; b < nb; ++b) {
@@ -167,53 +173,61 @@ chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant_
     }
     fence_before();
   };
-  decays(0);
+  if (!issuer) {
+    for (int x = warp; x < nh; x += WORK / 32) head_rates(a, chunk, h0 + x, row0, rows, wts + x * L);
+  }
   wait_warp(&C.full[2], 0, dead, 2);
   for (int it = 0; it < items; ++it) {
-    const int hi = it / pts;
     uint8_t* vs = vh + (it & 1) * SLAB;
     wait_warp(&C.full[it & 1], (it >> 1) & 1, dead, 3);
     if (it > 0) wait_warp(&C.done[0], (it - 1) & 1, dead, 4);               // the other stage and the lower terms are free
     __syncthreads();
-    fence_after();
-    if (it + 1 < items && leader) if (elect_one()) fetch(it + 1);
+    if (issuer) {
+      if (it + 1 < items && elect_one()) fetch(it + 1);
+    } else {
+      const float* wt = wts + it / pts * L;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int u = tid + i * THREADS;                               // a 16-byte unit; its row is u / 8
-      const float wt = C.c[u >> 3];
-      float f[8];
-      uint4 hv, lv;
-      rows::load_v<__nv_bfloat16, 8>(reinterpret_cast<const __nv_bfloat16*>(vs) + u * 8, f);
+      for (int i = 0; i < 4; ++i) {
+        const int u = tid + i * WORK;                                // a 16-byte unit; its row is u / 8
+        const float wr = wt[u >> 3];
+        float f[8];
+        uint4 hv, lv;
+        rows::load_v<__nv_bfloat16, 8>(reinterpret_cast<const __nv_bfloat16*>(vs) + u * 8, f);
 #pragma unroll
-      for (int k = 0; k < 8; ++k) f[k] *= wt;
-      split2(f[0], f[1], hv.x, lv.x); split2(f[2], f[3], hv.y, lv.y); split2(f[4], f[5], hv.z, lv.z); split2(f[6], f[7], hv.w, lv.w);
-      reinterpret_cast<uint4*>(vs)[u] = hv;
-      reinterpret_cast<uint4*>(vl)[u] = lv;
-    }
-    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-    __syncthreads();
-    if (leader) if (elect_one()) {
-      fence_after();
-      const uint64_t dh = desc(smem_u32(vs), SLAB), dl = desc(smem_u32(vl), SLAB);
-      for (int b = 0; b < nb; ++b) {
-        const uint32_t d = C.tmem + (it & 1) * cols + b * 64;
-        const uint64_t k0 = desc(smem_u32(ks) + (2 * b) * SLAB, SLAB), k1 = desc(smem_u32(ks) + (2 * nb + 2 * b) * SLAB, SLAB);
-#pragma unroll
-        for (int t = 0; t < 8; ++t) {
-          const uint64_t o = (uint64_t)t * (2048 >> 4);
-          mma_ss(d, k0 + o, dh + o, id, t ? 1u : 0u);
-          mma_ss(d, k0 + o, dl + o, id, 1u);
-          if (TERMS > 1) mma_ss(d, k1 + o, dh + o, id, 1u);
-        }
+        for (int k = 0; k < 8; ++k) f[k] *= wr;
+        split2(f[0], f[1], hv.x, lv.x); split2(f[2], f[3], hv.y, lv.y); split2(f[4], f[5], hv.z, lv.z); split2(f[6], f[7], hv.w, lv.w);
+        reinterpret_cast<uint4*>(vs)[u] = hv;
+        reinterpret_cast<uint4*>(vl)[u] = lv;
       }
-      commit(&C.done[0]);
+      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     }
-    if (it > 0) store(it - 1);                                       // while the products run
-    if ((it + 1) % pts == 0 && it + 1 < items) decays(hi + 1);
+    __syncthreads();
+    if (issuer) {
+      if (elect_one()) {
+        fence_after();
+        const uint64_t dh = desc(smem_u32(vs), SLAB), dl = desc(smem_u32(vl), SLAB);
+        for (int b = 0; b < nb; ++b) {
+          const uint32_t d = C.tmem + (it & 1) * cols + b * 64;
+          const uint64_t k0 = desc(smem_u32(ks) + (2 * b) * SLAB, SLAB), k1 = desc(smem_u32(ks) + (2 * nb + 2 * b) * SLAB, SLAB);
+#pragma unroll
+          for (int t = 0; t < 8; ++t) {
+            const uint64_t o = (uint64_t)t * (2048 >> 4);
+            mma_ss(d, k0 + o, dh + o, id, t ? 1u : 0u);
+            mma_ss(d, k0 + o, dl + o, id, 1u);
+            if (TERMS > 1) mma_ss(d, k1 + o, dh + o, id, 1u);
+          }
+        }
+        commit(&C.done[0]);
+      }
+      __syncwarp();
+    } else if (it > 0) {
+      fence_after();
+      store(it - 1);                                                 // while the products run
+    }
   }
   wait_warp(&C.done[0], (items - 1) & 1, dead, 5);
   fence_after();
-  store(items - 1);
+  if (!issuer) store(items - 1);
   drain(C);
   teardown(C, nb > 1 ? 256 : 128, a.status, 69);
 }
@@ -273,7 +287,7 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
   const int chunk = blockIdx.y, rep = a.H / a.G, parts = (rep + a.hpc - 1) / a.hpc, g = blockIdx.x / parts;
   const int h0 = g * rep + (blockIdx.x % parts) * a.hpc, nh = min(a.hpc, (g + 1) * rep - h0), row0 = a.c_row0[chunk], rows = a.c_rows[chunk];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, pts = (a.P + 63) / 64, items = nh * pts, w4 = warp & 3, half = warp >> 2;
-  const bool leader = __shfl_sync(0xffffffffu, warp, 0) == 0;          // uniform: the elected thread's operands stay in uniform registers
+  const bool issuer = __shfl_sync(0xffffffffu, warp, 0) == WORK / 32;  // uniform: the elected thread's operands stay in uniform registers
   volatile int* dead = &C.dead;
   const uint32_t tp = C.tmem, ta = tp + 128, tb = tp + 192, lanes = (uint32_t)(w4 * 32) << 16;
   auto tile = [&](int it) {                              // values and start state of a tile of 64 value dims
@@ -299,7 +313,7 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
     }
     commit(&C.done[1]);
   };
-  if (leader) if (elect_one()) {
+  if (issuer && elect_one()) {
     mbar_expect(&C.full[2], 2 * TERMS * NS * SLAB);
     for (int t = 0; t < TERMS; ++t)
       for (int s = 0; s < NS; ++s) {
@@ -309,108 +323,115 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
     tile(0);
   }
   const int i = w4 * 32 + lane;
-  float ci, wi;
-  Rate rate = chunk_rate(a, h0, row0, rows);
-  auto decays = [&](int hi) {                            // of the block's head hi
-    ci = chunk_decays(a, C, rate, rows, wi);
-    if (tid < L) C.c[tid] = ci - __log2f(wi);            // weight 0: infinity, and its exponential below 0
-    if (hi + 1 < nh) rate = chunk_rate(a, h0 + hi + 1, row0, rows);
-  };
-  decays(0);
+  const float* rates = a.rates + ((size_t)chunk * a.H + h0) * 2 * L;
   wait_warp(&C.full[2], 0, dead, 6);
-  if (leader) if (elect_one()) scores();
-  float ei = 0.f;
-  for (int it = 0; it < items; ++it) {
-    const int hi = it / pts, h = h0 + hi, pt = it % pts;
-    if (pt == 0) {
-      ei = ex2(ci);
-      const float D = a.D ? a.D[h] : 0.f;
-      wait_warp(&C.done[1], hi & 1, dead, 7);
+  if (issuer) {
+    // after every barrier of the workers below comes what it makes possible
+    if (elect_one()) scores();
+    __syncwarp();
+    for (int it = 0; it < items; ++it) {
+      const bool next = it + 1 < items, head_ends = (it + 1) % pts == 0;
+      wait_warp(&C.full[0], it & 1, dead, 7);
+      __syncthreads();
+      if (elect_one()) {
+        fence_after();
+        const uint32_t ia = idesc(64, 0, 1), ib = idesc(64, 0, 0);
+        const uint64_t dv = desc(smem_u32(vs), SLAB), ds = desc(smem_u32(ss), 16), sl = (uint64_t)NS * (HSLAB >> 4);
+#pragma unroll
+        for (int t = 0; t < 4 * NS; ++t) {
+          if (t >= kst) break;
+          const uint64_t o = (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, os = (uint64_t)(t >> 2) * (HSLAB >> 4) + (t & 3) * 2;
+          mma_ss(tb, dq + o, ds + os, ib, t ? 1u : 0u);
+          mma_ss(tb, dq + o, ds + sl + os, ib, 1u);
+          if (TERMS > 1) mma_ss(tb, dq + lo + o, ds + os, ib, 1u);
+        }
+#pragma unroll
+        for (int t = 0; t < 16; ++t)                     // eight steps of 16 rows with the upper terms, then with the lower ones
+          mma_ts(ta, tp + ((t & 7) >> 1) * 32 + (t & 1) * 8 + (t >> 3) * 16, dv + (uint64_t)(t & 7) * (2048 >> 4), ia, t ? 1u : 0u);
+        commit(&C.done[0]);
+      }
+      __syncwarp();
+      wait_warp(&C.done[0], it & 1, dead, 8);
+      if (next && elect_one()) {
+        fence_after();
+        if (head_ends) scores();                         // of the next head
+        tile(it + 1);
+      }
+      __syncwarp();
+    }
+  } else {
+    float next_ci = rates[i], ei = 0.f;
+    for (int it = 0; it < items; ++it) {
+      const int hi = it / pts, h = h0 + hi, pt = it % pts;
+      if (pt == 0) {
+        const float ci = next_ci, D = a.D ? a.D[h] : 0.f;
+        const float* cs = rates + (size_t)hi * 2 * L + L;
+        ei = ex2(ci);
+        if (hi + 1 < nh) next_ci = rates[(size_t)(hi + 1) * 2 * L + i];
+        wait_warp(&C.done[1], hi & 1, dead, 9);
+        fence_after();
+        // Blocks of 32 columns: before the warp's diagonal block all are visible, after it none.  A thread's weights take the place of the
+        // scores it has read: upper terms in the block's first 16 columns, lower terms in the others.
+#pragma unroll
+        for (int b = 0; b < 2; ++b) {
+          const int blk = 2 * half + b;
+          uint32_t hv[16], lv[16];
+          if (blk <= w4) {
+            float s[32];
+            ld32(tp + blk * 32 + lanes, s);
+            float4 cj[8];
+#pragma unroll
+            for (int q = 0; q < 8; ++q) cj[q] = *reinterpret_cast<const float4*>(cs + blk * 32 + 4 * q);
+            wait_ld();
+#pragma unroll
+            for (int q = 0; q < 8; ++q) {
+              const float c4[4] = {cj[q].x, cj[q].y, cj[q].z, cj[q].w};
+#pragma unroll
+              for (int k = 0; k < 4; ++k) s[4 * q + k] *= ex2(ci - c4[k]);
+            }
+            if (blk == w4) {
+#pragma unroll
+              for (int k = 0; k < 32; ++k) {
+                if (k > lane) s[k] = 0.f;
+                if (k == lane) s[k] += D;                // D v_i
+              }
+            }
+#pragma unroll
+            for (int q = 0; q < 16; ++q) split2(s[2 * q], s[2 * q + 1], hv[q], lv[q]);
+          } else {
+#pragma unroll
+            for (int q = 0; q < 16; ++q) hv[q] = lv[q] = 0u;
+          }
+          st16(tp + blk * 32 + lanes, hv);
+          st16(tp + blk * 32 + 16 + lanes, lv);
+        }
+        wait_st();
+        fence_before();
+      }
+      __syncthreads();                                   // weights are in place, accumulators have been read
+      wait_warp(&C.done[0], it & 1, dead, 10);
       fence_after();
-      float s[64];
-      // blocks of 32 columns: before the warp's diagonal block all are visible, after it none
-      if (2 * half <= w4) ld32(tp + half * 64 + lanes, s);
-      if (2 * half + 1 <= w4) ld32(tp + half * 64 + 32 + lanes, s + 32);
-      wait_ld();
-      fence_before();
-      __syncthreads();                                   // every score has been read: the weighted ones may take their place
-      fence_after();
-      const float* cs = C.c + half * 64;
+      __nv_bfloat16* o = a.y + ((size_t)(row0 + i) * a.H + h) * a.P + pt * 64 + half * 32;
+      const int cols = min(32, a.P - pt * 64 - half * 32);
 #pragma unroll
       for (int b = 0; b < 2; ++b) {
-        const int blk = 2 * half + b;
-        uint32_t hv[16], lv[16];
-        if (blk < w4) {
+        float x[16], z[16];
+        ld16(ta + half * 32 + 16 * b + lanes, x);
+        ld16(tb + half * 32 + 16 * b + lanes, z);
+        wait_ld();
+        if (i < rows) {
 #pragma unroll
-          for (int q = 0; q < 16; ++q) {
-            const int j = 32 * b + 2 * q;
-            const float2 cj = *reinterpret_cast<const float2*>(cs + j);
-            split2(s[j] * ex2(ci - cj.x), s[j + 1] * ex2(ci - cj.y), hv[q], lv[q]);
+          for (int k = 0; k < 16; ++k) x[k] = fmaf(ei, z[k], x[k]);
+          if (a.wide && 16 * b + 16 <= cols) store32(o + 16 * b, x);
+          else {
+#pragma unroll
+            for (int u = 0; u < 2; ++u)
+              if (16 * b + 8 * u < cols) rows::store_v<__nv_bfloat16, 8>(o + 16 * b + 8 * u, x + 8 * u);      // P is a multiple of eight
           }
-        } else if (blk == w4) {
-#pragma unroll
-          for (int q = 0; q < 16; ++q) {
-            const int j = 32 * b + 2 * q;
-            const float2 cj = *reinterpret_cast<const float2*>(cs + j);
-            float x = 2 * q <= lane ? s[j] * ex2(ci - cj.x) : 0.f, y = 2 * q + 1 <= lane ? s[j + 1] * ex2(ci - cj.y) : 0.f;
-            if (2 * q == lane) x += D;                   // D v_i
-            if (2 * q + 1 == lane) y += D;
-            split2(x, y, hv[q], lv[q]);
-          }
-        } else {
-#pragma unroll
-          for (int q = 0; q < 16; ++q) hv[q] = lv[q] = 0u;
         }
-        st16(tp + half * 32 + 16 * b + lanes, hv);
-        st16(tp + 64 + half * 32 + 16 * b + lanes, lv);
       }
-      wait_st();
       fence_before();
     }
-    wait_warp(&C.full[0], it & 1, dead, 8);
-    __syncthreads();                                     // weights are in place, accumulators have been read
-    if (leader) if (elect_one()) {
-      fence_after();
-      const uint32_t ia = idesc(64, 0, 1), ib = idesc(64, 0, 0);
-      const uint64_t dv = desc(smem_u32(vs), SLAB), ds = desc(smem_u32(ss), 16), sl = (uint64_t)NS * (HSLAB >> 4);
-#pragma unroll
-      for (int t = 0; t < 4 * NS; ++t) {
-        if (t >= kst) break;
-        const uint64_t o = (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, os = (uint64_t)(t >> 2) * (HSLAB >> 4) + (t & 3) * 2;
-        mma_ss(tb, dq + o, ds + os, ib, t ? 1u : 0u);
-        mma_ss(tb, dq + o, ds + sl + os, ib, 1u);
-        if (TERMS > 1) mma_ss(tb, dq + lo + o, ds + os, ib, 1u);
-      }
-#pragma unroll
-      for (int t = 0; t < 16; ++t) mma_ts(ta, tp + (t & 7) * 8 + (t >> 3) * 64, dv + (uint64_t)(t & 7) * (2048 >> 4), ia, t ? 1u : 0u);
-      commit(&C.done[0]);
-    }
-    const bool head_ends = pt + 1 == pts && it + 1 < items;
-    if (head_ends) decays(hi + 1);                       // while the products run
-    wait_warp(&C.done[0], it & 1, dead, 9);
-    fence_after();
-    if (it + 1 < items && leader) if (elect_one()) {
-      if (head_ends) scores();                           // of the next head
-      tile(it + 1);
-    }
-    __nv_bfloat16* o = a.y + ((size_t)(row0 + i) * a.H + h) * a.P + pt * 64 + half * 32;
-    const int cols = min(32, a.P - pt * 64 - half * 32);
-#pragma unroll
-    for (int b = 0; b < 2; ++b) {
-      float x[16], z[16];
-      ld16(ta + half * 32 + 16 * b + lanes, x);
-      ld16(tb + half * 32 + 16 * b + lanes, z);
-      wait_ld();
-#pragma unroll
-      for (int u = 0; u < 2; ++u)
-        if (i < rows && 16 * b + 8 * u < cols) {         // P is a multiple of eight
-          float f[8];
-#pragma unroll
-          for (int k = 0; k < 8; ++k) f[k] = fmaf(ei, z[8 * u + k], x[8 * u + k]);
-          rows::store_v<__nv_bfloat16, 8>(o + 16 * b + 8 * u, f);
-        }
-    }
-    fence_before();
   }
   drain(C);
   teardown(C, 256, a.status, 70);
@@ -459,7 +480,7 @@ __global__ void __launch_bounds__(256) state_turn_kernel(TurnArgs a) {
   }
 }
 
-static size_t sums_smem(const Args& a) { return (size_t)(a.terms * 2 * ((a.ns + 1) / 2) + 3) * SLAB + sizeof(Ctl); }
+static size_t sums_smem(const Args& a) { return (size_t)(a.terms * 2 * ((a.ns + 1) / 2) + 3) * SLAB + HEADS * L * sizeof(float) + sizeof(Ctl); }
 static size_t out_smem(const Args& a) { return (size_t)(2 * a.terms * a.ns + 1) * SLAB + (size_t)2 * a.ns * HSLAB + sizeof(Ctl); }
 
 template <typename K>
@@ -503,17 +524,17 @@ int sfb_rows_state_turn(const void* q, int64_t q_stride, const void* k, int64_t 
 // 16 up to 256 (128 with two terms); P: a multiple of 8; first columns multiples of 8.
 int sfb_rows_state_tc(const void* mq, const void* mk, const void* mv, const void* ms, const int* c_row0, const int* c_rows, const int* seg, const int* first,
                       const int* seg_src, const int* seg_dst, const void* dt, int64_t dt_stride, const void* dt_bias, const void* la, const void* D, void* S,
-                      void* sums, void* dec, void* starts, void* y, int runs, int chunks, int H, int G, int N, int P, int Np, int terms, int q_col, int k_col,
+                      void* sums, void* dec, void* rates, void* starts, void* y, int runs, int chunks, int H, int G, int N, int P, int Np, int terms, int q_col, int k_col,
                       int v_col, int q_lo, int k_lo, void* status, cudaStream_t stream) {
   const int ns = (N + 63) / 64;
   if (runs < 1 || runs > 65535 || chunks < 1 || chunks > 65535 || G < 1 || H % G || N % 16 || P % 8 || ns > (terms > 1 ? 2 : 4) || Np < N || Np % 32 ||
       terms < 1 || terms > 2 || (q_col | k_col | v_col | q_lo | k_lo | N) % 8)
     return (int)cudaErrorInvalidValue;
   Args a{c_row0, c_rows, seg, first, seg_src, seg_dst, (const __nv_bfloat16*)dt, dt_stride, (const float*)dt_bias, (const float*)la, (const float*)D, (float*)S,
-         (float*)sums, (float*)dec, (__nv_bfloat16*)starts, (__nv_bfloat16*)y, H, G, N, P, Np, ns, terms, q_col, k_col, v_col, q_lo, k_lo, chunks, 1,
+         (float*)sums, (float*)dec, (float*)rates, (__nv_bfloat16*)starts, (__nv_bfloat16*)y, H, G, N, P, Np, ns, terms, q_col, k_col, v_col, q_lo, k_lo, chunks, 1, (H * P) % 16 == 0 && P % 16 == 0 && (uintptr_t)y % 32 == 0,
          (Status*)status};
   const int rep = H / G;
-  a.hpc = rep < 8 ? rep : 8;         // fewer heads per block where that leaves SMs empty
+  a.hpc = rep < HEADS ? rep : HEADS;         // fewer heads per block where that leaves SMs empty
   while (a.hpc > 1 && (long long)G * ((rep + a.hpc - 1) / a.hpc) * chunks < 148) a.hpc = (a.hpc + 1) / 2;
   const int blocks = G * ((rep + a.hpc - 1) / a.hpc);
   const CUtensorMap *q = (const CUtensorMap*)mq, *k = (const CUtensorMap*)mk, *v = (const CUtensorMap*)mv, *s = (const CUtensorMap*)ms;

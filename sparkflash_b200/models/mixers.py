@@ -218,6 +218,7 @@ class MatrixState:
             e.scratch.reserve("state_sums", chunks * per, torch.float32)
             e.scratch.reserve("state_starts", 2 * chunks * per, torch.bfloat16)
             e.scratch.reserve("state_dec", chunks * self.H, torch.float32)
+            e.scratch.reserve("state_rates", chunks * self.H * 256, torch.float32)
             if self.terms > 1:
                 e.scratch.reserve("state_turned", e.max_rows * 4 * self.H * self.N, torch.bfloat16)
 
@@ -233,7 +234,7 @@ class MatrixState:
                 qk, at = s.scratch.get("state_turned", s.n, 4 * hn), (0, 2 * hn, hn, hn)
                 R.state_turn(q, k, self.rot, self.rot_dims, self.k_scale, s.row_pos, qk, s.n, self.H, self.N)
             R.state_tc(qk, at, src, cols[2], dt, self.dt_bias, self.log_decay, self.skip, S, s.scratch.buf["state_sums"], s.scratch.buf["state_dec"],
-                       s.scratch.buf["state_starts"], y, self.N, self.G, s, self.terms, s.status)
+                       s.scratch.buf["state_rates"], s.scratch.buf["state_starts"], y, self.N, self.G, s, self.terms, s.status)
 
 
 class StateSpaceMixer:

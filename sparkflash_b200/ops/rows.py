@@ -114,15 +114,15 @@ def state_turn(q, k, rot, rot_dims, k_scale, row_pos, out, n, heads, N):
                                            c_float(k_scale), _stream()), "rows_state_turn")
 
 
-def state_tc(qk, qk_cols, v, v_col, dt, dt_bias, log_a, D, S, sums, dec, starts, y, N, groups, seg, terms, status):
+def state_tc(qk, qk_cols, v, v_col, dt, dt_bias, log_a, D, S, sums, dec, rates, starts, y, N, groups, seg, terms, status):
     """Long segments in chunks of 128 rows.  ``qk``: [n, stride] tensor with the columns (q, k, distance to q's and to k's lower terms) of
-    ``qk_cols``; ``v``: [n, stride] tensor with values from column ``v_col`` on; sums, dec, starts: scratch of all chunks."""
+    ``qk_cols``; ``v``: [n, stride] tensor with values from column ``v_col`` on; sums, dec, rates, starts: scratch of all chunks."""
     _, H, P, Np = S.shape
     mqk, mv = tensor_map(qk, qk.shape[1], 128), tensor_map(v, v.shape[1], 128)
     ms = tensor_map(starts, Np, 64)
     qc, kc, ql, kl = qk_cols
     _check(_lib.rows().sfb_rows_state_tc(mqk.ptr, mqk.ptr, mv.ptr, ms.ptr, _p(seg.long_row0), _p(seg.long_rows), _p(seg.long_seg), _p(seg.long_first),
-                                         _p(seg.seg_src), _p(seg.seg_dst), *_strides(dt), _p(dt_bias), _p(log_a), _p(D), _p(S), _p(sums), _p(dec),
+                                         _p(seg.seg_src), _p(seg.seg_dst), *_strides(dt), _p(dt_bias), _p(log_a), _p(D), _p(S), _p(sums), _p(dec), _p(rates),
                                          _p(starts), _p(y), c_int(seg.nlong), c_int(seg.nchunks), c_int(H), c_int(groups), c_int(N), c_int(P), c_int(Np),
                                          c_int(terms), c_int(qc), c_int(kc), c_int(v_col), c_int(ql), c_int(kl), _p(status), _stream()), "rows_state_tc")
 
