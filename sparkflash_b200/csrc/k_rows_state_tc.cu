@@ -20,7 +20,7 @@ namespace rst {
 using namespace tc;
 
 constexpr int L = 128, SLAB = L * 128, HSLAB = 64 * 128;         // rows of a chunk; bytes of 128 / 64 rows of 64 elements
-constexpr int WORK = 256, THREADS = WORK + 32, HEADS = 8;        // threads that compute, and one warp that issues copies and products; heads per block
+constexpr int WORK = 256, THREADS = WORK + 32, HEADS = 8;        // threads that compute, and one warp that issues copies and products; most heads per block
 
 struct Args {
   const int *c_row0, *c_rows;      // chunks
@@ -132,10 +132,10 @@ chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant_
   extern __shared__ __align__(1024) uint8_t sm[];
   const int nb = (a.ns + 1) / 2;                          // blocks of 128 state rows
   uint8_t* ks = sm;                                       // [terms][2 nb] slabs
-  uint8_t* vh = ks + (size_t)TERMS * 2 * nb * SLAB;     // weighted values, upper terms (the copy lands here): two stages
+  uint8_t* vh = ks + (size_t)TERMS * 2 * nb * SLAB;       // weighted values, upper terms (the copy lands here): two stages
   uint8_t* vl = vh + 2 * SLAB;                            // lower terms
-  float* wts = reinterpret_cast<float*>(vl + SLAB);       // [HEADS][L] factors of the values
-  Ctl& C = *reinterpret_cast<Ctl*>(wts + HEADS * L);
+  float* wts = reinterpret_cast<float*>(vl + SLAB);       // [hpc][L] factors of the values
+  Ctl& C = *reinterpret_cast<Ctl*>(wts + a.hpc * L);
   setup(C, nb > 1 ? 256 : 128);
   pdl_launch_dependents();
   pdl_wait();
@@ -337,25 +337,32 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
         fence_after();
         const uint32_t ia = idesc(64, 0, 1), ib = idesc(64, 0, 0);
         const uint64_t dv = desc(smem_u32(vs), SLAB), ds = desc(smem_u32(ss), 16), sl = (uint64_t)NS * (HSLAB >> 4);
+        // the two sums by turns: products on one accumulator follow each other slowly at this size
+        auto weighted = [&](int t) {                     // eight steps of 16 rows with the upper terms, then with the lower ones
+          mma_ts(ta, tp + ((t & 7) >> 1) * 32 + (t & 1) * 8 + (t >> 3) * 16, dv + (uint64_t)(t & 7) * (2048 >> 4), ia, t ? 1u : 0u);
+        };
+        constexpr int PER = 16 / (4 * NS);               // weighted products for every step of the other sum
 #pragma unroll
         for (int t = 0; t < 4 * NS; ++t) {
-          if (t >= kst) break;
           const uint64_t o = (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, os = (uint64_t)(t >> 2) * (HSLAB >> 4) + (t & 3) * 2;
-          mma_ss(tb, dq + o, ds + os, ib, t ? 1u : 0u);
-          mma_ss(tb, dq + o, ds + sl + os, ib, 1u);
-          if (TERMS > 1) mma_ss(tb, dq + lo + o, ds + os, ib, 1u);
+          if (t < kst) mma_ss(tb, dq + o, ds + os, ib, t ? 1u : 0u);
+          weighted(PER * t);
+          if (t < kst) mma_ss(tb, dq + o, ds + sl + os, ib, 1u);
+          if (PER > 1) weighted(PER * t + 1);
+          if (TERMS > 1 && t < kst) mma_ss(tb, dq + lo + o, ds + os, ib, 1u);
+#pragma unroll
+          for (int u = 2; u < PER; ++u) weighted(PER * t + u);
         }
 #pragma unroll
-        for (int t = 0; t < 16; ++t)                     // eight steps of 16 rows with the upper terms, then with the lower ones
-          mma_ts(ta, tp + ((t & 7) >> 1) * 32 + (t & 1) * 8 + (t >> 3) * 16, dv + (uint64_t)(t & 7) * (2048 >> 4), ia, t ? 1u : 0u);
+        for (int t = PER * 4 * NS; t < 16; ++t) weighted(t);
         commit(&C.done[0]);
       }
       __syncwarp();
       wait_warp(&C.done[0], it & 1, dead, 8);
       if (next && elect_one()) {
         fence_after();
-        if (head_ends) scores();                         // of the next head
         tile(it + 1);
+        if (head_ends) scores();                         // of the next head
       }
       __syncwarp();
     }
@@ -480,7 +487,7 @@ __global__ void __launch_bounds__(256) state_turn_kernel(TurnArgs a) {
   }
 }
 
-static size_t sums_smem(const Args& a) { return (size_t)(a.terms * 2 * ((a.ns + 1) / 2) + 3) * SLAB + HEADS * L * sizeof(float) + sizeof(Ctl); }
+static size_t sums_smem(const Args& a) { return (size_t)(a.terms * 2 * ((a.ns + 1) / 2) + 3) * SLAB + a.hpc * L * sizeof(float) + sizeof(Ctl); }
 static size_t out_smem(const Args& a) { return (size_t)(2 * a.terms * a.ns + 1) * SLAB + (size_t)2 * a.ns * HSLAB + sizeof(Ctl); }
 
 template <typename K>

@@ -124,8 +124,9 @@ def throughput(design: str, name: str, prompt: int = 8192, chunk: int = 4096, st
 
 
 def gudutar_work(cfg: GudutarConfig, n: int, ctx: int, head_rows: int, decode: bool) -> dict[str, roofline.ClassWork]:
-    """The same accounting for Gudutar.  Recurrences: inputs and outputs once, the state of every segment in and out, and the products
-    of chunks of 128 rows with every operand taken once (prompts); attention: the window's keys (prompts: multiplied out, in ``linear``)."""
+    """The same accounting for Gudutar.  Recurrences: inputs and outputs once, the state of every segment in and out, and for prompts the
+    products of chunks of 128 rows, those with a 32-bit operand counted once per pair of bf16 terms (the products the chunked form needs
+    at that precision); attention: the window's keys (prompts: multiplied out, in ``linear``)."""
     d, W = cfg.width, roofline.ClassWork
     out = {k: W() for k in ("rows_seam", "rows_conv", "rows_state", "rows_state_tc", "rows_state_turn", "rows_gated_norm", "rows_latent_append", "rows_head_proj",
                             "rows_latent_decode", "rows_attn_tc", "rows_gather_pages", "rows_act_mul", "linear", "head")}
@@ -141,7 +142,9 @@ def gudutar_work(cfg: GudutarConfig, n: int, ctx: int, head_rows: int, decode: b
             out["rows_state"].bytes += segs * H * N * P * 8.0 + 2.0 * n * (cols + H * P)
         else:
             out["rows_state_tc"].bytes += segs * H * N * P * 8.0 + 2.0 * n * (cols + H * P)
-            out["rows_state_tc"].flops += n * H * (2.0 * 128 * (N + P) / 2 + 4.0 * N * P)
+            # q k^T of a group (visible half), weights times v, q S, k^T v; turned q and k have two terms: three products, less lo x lo
+            s, i = (3, 3) if turned else (1, 2)
+            out["rows_state_tc"].flops += n * (G * s * 128.0 * N + H * (2 * 128.0 * P + 2.0 * i * N * P + 2.0 * i * N * P))
             out["rows_state_turn"].bytes += 2.0 * n * 6 * H * N if turned else 0.0
     out["rows_seam"].bytes += n * d * 8.0
     for L in cfg.layers:
