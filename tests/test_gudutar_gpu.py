@@ -32,7 +32,7 @@ CONFIGS = {
     "lat": P.make_config(90, 64, 1.0, [P.latent(6, 16, 8, 24, 40, 100, 1000.0, 0.5)]),
 }
 NAMES = list(CONFIGS)
-TOL = {torch.float32: 2e-4, torch.bfloat16: 0.12}      # rms of the logits' difference over the logits' spread
+TOL = {torch.float32: 2e-4, torch.bfloat16: 0.18}      # rms of the logits' difference over the logits' spread
 
 
 @functools.lru_cache(None)
@@ -78,13 +78,14 @@ def feed(eng, lane, toks, at, cuts):
 def test_whole_prompt_and_layers(name, dt):
     toks = tokens(name, 333)
     eng = engine(name, dt)
-    assert (eng.model.tc_attention, eng.model.tc_state) == ((name in ("tc", "lat"), name in ("tc", "ssm")) if dt == torch.bfloat16 else (False, False))
+    assert (eng.model.tc_attention, eng.model.tc_state) == ((name in ("mix", "tc", "lat"), name in ("tc", "ssm")) if dt == torch.bfloat16 else (False, False))
     taps, eng.tap_layers = [], []
     P.forward(weights(name), CONFIGS[name], list(toks[:40]), torch.float64, taps)
     eng.step(toks[:40], [1] * 40, list(range(40)))
     assert len(taps) == len(eng.tap_layers) == len(CONFIGS[name]["layers"])
     for i, (a, b) in enumerate(zip(eng.tap_layers, taps)):
-        assert (a.cpu() - b.float()).abs().max() < (1e-4 if dt == torch.float32 else 0.5), (i, (a.cpu() - b.float()).abs().max())
+        off = (a.cpu() - b.float()).pow(2).mean().sqrt() / b.float().pow(2).mean().sqrt()
+        assert off < (1e-5 if dt == torch.float32 else 0.05), (i, off)
     eng.tap_layers = None
     assert error(feed(eng, 0, toks, 0, [333]), expected(name, toks)) < TOL[dt]
 
@@ -99,7 +100,7 @@ def test_portions_and_token_by_token_match_the_whole(name, dt):
     ref = want if dt == torch.float32 else whole
     for lane, cuts in enumerate(([2] * 100, [1] * 200, [64, 64, 64, 8], [3, 61, 1, 65, 33, 2, 2, 32, 1])):
         got = feed(eng, lane, toks, 0, cuts)
-        assert error(got, ref) < (2e-4 if dt == torch.float32 else 0.1), (cuts[:4], error(got, ref))
+        assert error(got, ref) < TOL[dt], (cuts[:4], error(got, ref))
         assert error(got, want) < TOL[dt]
 
 
