@@ -279,20 +279,20 @@ struct ConvRowsArgs {
   const int *row_seg, *seg_row0, *seg_len, *seg_src, *seg_dst;
   int n, C, mode;           // 1: y = x + conv(x), 2: y = silu(conv(x))
 };
-constexpr int CONV_RT = 8;  // rows per block: their loads are all in flight before the first product
+constexpr int CONV_RT = 8;  // most rows per block: their loads are all in flight before the first product
 
-template <typename T, int V, int TAPS>
+template <typename T, int V, int TAPS, int RT>
 __global__ void __launch_bounds__(128) conv_rows_kernel(ConvRowsArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * V;
   if (c >= a.C) return;
   constexpr int W = TAPS - 1;
-  const int r0 = blockIdx.y * CONV_RT, r1 = min(r0 + CONV_RT, a.n);
+  const int r0 = blockIdx.y * RT, r1 = min(r0 + RT, a.n);
   const T* X = (const T*)a.x;
-  float in[CONV_RT][V], w[TAPS][V], win[W > 0 ? W : 1][V], bias[V];
+  float in[RT][V], w[TAPS][V], win[W > 0 ? W : 1][V], bias[V];
 #pragma unroll
-  for (int i = 0; i < CONV_RT; ++i)
+  for (int i = 0; i < RT; ++i)
     if (r0 + i < r1) load_v<T, V>(X + (size_t)(r0 + i) * a.x_stride + c, in[i]);
 #pragma unroll
   for (int j = 0; j < TAPS; ++j) load_v<float, V>(a.w + (size_t)j * a.C + c, w[j]);
@@ -314,7 +314,7 @@ __global__ void __launch_bounds__(128) conv_rows_kernel(ConvRowsArgs a) {
     }
   }
 #pragma unroll
-  for (int i = 0; i < CONV_RT; ++i) {
+  for (int i = 0; i < RT; ++i) {
     const int r = r0 + i;
     if (r >= r1) break;
     if (r == s1) {                        // next segment: its window comes from its own state
@@ -719,20 +719,25 @@ static int launch_seam(const SeamArgs& a, int n, cudaStream_t st) {
     default: return (int)sfb_launch(seam_kernel<T, V, 8, false>, g, b, 0, st, a);
   }
 }
-template <typename T, int V>
-static int launch_conv(const ConvRowsArgs& a, int taps, cudaStream_t st) {
-  const dim3 g((a.C + 128 * V - 1) / (128 * V), (a.n + CONV_RT - 1) / CONV_RT), b(128);
+template <typename T, int V, int RT>
+static int launch_conv_rt(const ConvRowsArgs& a, int taps, cudaStream_t st) {
+  const dim3 g((a.C + 128 * V - 1) / (128 * V), (a.n + RT - 1) / RT), b(128);
   switch (taps) {
-    case 1: return (int)sfb_launch(conv_rows_kernel<T, V, 1>, g, b, 0, st, a);
-    case 2: return (int)sfb_launch(conv_rows_kernel<T, V, 2>, g, b, 0, st, a);
-    case 3: return (int)sfb_launch(conv_rows_kernel<T, V, 3>, g, b, 0, st, a);
-    case 4: return (int)sfb_launch(conv_rows_kernel<T, V, 4>, g, b, 0, st, a);
-    case 5: return (int)sfb_launch(conv_rows_kernel<T, V, 5>, g, b, 0, st, a);
-    case 6: return (int)sfb_launch(conv_rows_kernel<T, V, 6>, g, b, 0, st, a);
-    case 7: return (int)sfb_launch(conv_rows_kernel<T, V, 7>, g, b, 0, st, a);
-    case 8: return (int)sfb_launch(conv_rows_kernel<T, V, 8>, g, b, 0, st, a);
+    case 1: return (int)sfb_launch(conv_rows_kernel<T, V, 1, RT>, g, b, 0, st, a);
+    case 2: return (int)sfb_launch(conv_rows_kernel<T, V, 2, RT>, g, b, 0, st, a);
+    case 3: return (int)sfb_launch(conv_rows_kernel<T, V, 3, RT>, g, b, 0, st, a);
+    case 4: return (int)sfb_launch(conv_rows_kernel<T, V, 4, RT>, g, b, 0, st, a);
+    case 5: return (int)sfb_launch(conv_rows_kernel<T, V, 5, RT>, g, b, 0, st, a);
+    case 6: return (int)sfb_launch(conv_rows_kernel<T, V, 6, RT>, g, b, 0, st, a);
+    case 7: return (int)sfb_launch(conv_rows_kernel<T, V, 7, RT>, g, b, 0, st, a);
+    case 8: return (int)sfb_launch(conv_rows_kernel<T, V, 8, RT>, g, b, 0, st, a);
     default: return (int)cudaErrorInvalidValue;
   }
+}
+template <typename T, int V>
+static int launch_conv(const ConvRowsArgs& a, int taps, cudaStream_t st) {
+  // few rows are mostly decoded ones, each with its own carried inputs: side by side instead of one after another
+  return a.n <= 128 ? launch_conv_rt<T, V, 1>(a, taps, st) : launch_conv_rt<T, V, CONV_RT>(a, taps, st);
 }
 
 }  // namespace rows

@@ -24,7 +24,8 @@ struct LatentArgs {
   Status* status;
 };
 
-template <typename T>
+// V: elements a thread takes together (4: every width and offset is a multiple of four; 2 otherwise: pairs, element by element)
+template <typename T, int V>
 __global__ void __launch_bounds__(128) latent_append_kernel(LatentArgs a) {
   __shared__ float sh[2 * 2 * 32];
   int phase = 0;
@@ -34,15 +35,42 @@ __global__ void __launch_bounds__(128) latent_append_kernel(LatentArgs a) {
   T* p = (T*)a.proj + (size_t)row * a.stride;
   T* c = p + (size_t)a.H * qd;
   const float2* cs = a.cs + (size_t)pos * half;
+  auto load = [](const T* x, float (&f)[V]) {
+    if constexpr (V == 4) load_v<T, 4>(x, f);
+    else { f[0] = to_f<T>(x[0]); f[1] = to_f<T>(x[1]); }
+  };
+  auto store = [](T* x, const float (&f)[V]) {
+    if constexpr (V == 4) store_v<T, 4>(x, f);
+    else { x[0] = from_f<T>(f[0]); x[1] = from_f<T>(f[1]); }
+  };
+  auto turn = [&](const T* x, T* o, int k) {             // pairs k / 2 ..
+    float f[V], g[V];
+    load(x, f);
+#pragma unroll
+    for (int i = 0; i < V; i += 2) {
+      const float2 t = cs[(k + i) >> 1];
+      g[i] = f[i] * t.x - f[i + 1] * t.y;
+      g[i + 1] = f[i + 1] * t.x + f[i] * t.y;
+    }
+    store(o, g);
+  };
   float s[1] = {0.f};
-  for (int i = threadIdx.x; i < a.rank; i += 128) { const float f = to_f<T>(c[i]); s[0] += f * f; }
-  for (int i = threadIdx.x; i < a.H * half; i += 128) {
-    const int h = i / half, k = i - h * half;
-    T* x = p + (size_t)h * qd + a.dim + 2 * k;
-    const float u = to_f<T>(x[0]), v = to_f<T>(x[1]);
-    const float2 t = cs[k];
-    x[0] = from_f<T>(u * t.x - v * t.y);
-    x[1] = from_f<T>(v * t.x + u * t.y);
+  if constexpr (V == 4) {
+    for (int i = threadIdx.x * 4; i < a.rank; i += 512) {
+      float f[V];
+      load(c + i, f);
+#pragma unroll
+      for (int k = 0; k < V; ++k) s[0] += f[k] * f[k];
+    }
+  } else {
+    for (int i = threadIdx.x; i < a.rank; i += 128) { const float f = to_f<T>(c[i]); s[0] += f * f; }
+  }
+  const int per = a.rot / V;
+#pragma unroll 4
+  for (int i = threadIdx.x; i < a.H * per; i += 128) {
+    const int h = i / per, k = (i - h * per) * V;
+    T* x = p + (size_t)h * qd + a.dim + k;
+    turn(x, x, k);
   }
   block_sums<1>(s, sh, phase);
   const float r = 1.f / sqrtf(s[0] / (float)a.rank + a.eps);
@@ -52,13 +80,19 @@ __global__ void __launch_bounds__(128) latent_append_kernel(LatentArgs a) {
     return;
   }
   T* o = (T*)a.pool + ((size_t)page * 64 + pos % 64) * (a.rank + a.rot);
-  for (int i = threadIdx.x; i < a.rank; i += 128) o[i] = from_f<T>(to_f<T>(c[i]) * r * a.w[i]);
-  for (int k = threadIdx.x; k < half; k += 128) {
-    const float u = to_f<T>(c[a.rank + 2 * k]), v = to_f<T>(c[a.rank + 2 * k + 1]);
-    const float2 t = cs[k];
-    o[a.rank + 2 * k] = from_f<T>(u * t.x - v * t.y);
-    o[a.rank + 2 * k + 1] = from_f<T>(v * t.x + u * t.y);
+  if constexpr (V == 4) {
+    for (int i = threadIdx.x * 4; i < a.rank; i += 512) {
+      float f[V], w[V];
+      load(c + i, f);
+      load_v<float, 4>(a.w + i, w);
+#pragma unroll
+      for (int k = 0; k < V; ++k) f[k] *= r * w[k];
+      store(o + i, f);
+    }
+  } else {
+    for (int i = threadIdx.x; i < a.rank; i += 128) o[i] = from_f<T>(to_f<T>(c[i]) * r * a.w[i]);
   }
+  for (int k = (127 - threadIdx.x) * V; k < a.rot; k += 128 * V) turn(c + a.rank + k, o + a.rank + k, k);
 }
 
 struct HeadProjArgs {
@@ -236,8 +270,11 @@ int sfb_rows_latent_append(void* proj, int64_t stride, const void* w, const void
                            int max_pages, int n_pages, int n, int H, int dim, int rot, int rank, float eps, int fp32, void* status, cudaStream_t stream) {
   if (n < 1 || H < 1 || dim < 1 || rot < 0 || rot % 2 || rank < 1) return (int)cudaErrorInvalidValue;
   LatentArgs a{proj, stride, (const float*)w, (const float2*)cs, pool, table, row_lane, row_pos, max_pages, n_pages, H, dim, rot, rank, eps, (Status*)status};
-  return (int)(fp32 ? sfb_launch(latent_append_kernel<float>, dim3(n), dim3(128), 0, stream, a)
-                    : sfb_launch(latent_append_kernel<__nv_bfloat16>, dim3(n), dim3(128), 0, stream, a));
+  const bool v4 = (dim | rot | rank) % 4 == 0 && stride % 4 == 0;
+  if (fp32) return (int)(v4 ? sfb_launch(latent_append_kernel<float, 4>, dim3(n), dim3(128), 0, stream, a)
+                            : sfb_launch(latent_append_kernel<float, 2>, dim3(n), dim3(128), 0, stream, a));
+  return (int)(v4 ? sfb_launch(latent_append_kernel<__nv_bfloat16, 4>, dim3(n), dim3(128), 0, stream, a)
+                  : sfb_launch(latent_append_kernel<__nv_bfloat16, 2>, dim3(n), dim3(128), 0, stream, a));
 }
 
 // list: 0 = rows ignored, 1 = it names x's rows, 2 = it names out's rows.  part (then x is null): see HeadProjArgs; list is 2 or 0.

@@ -173,64 +173,48 @@ struct GatedNormArgs {
   float eps;
 };
 
-// TPG threads per part: a warp (parts side by side in a block) or the whole block
-template <typename T, int V, bool WARP>
+// A part belongs to a warp (parts side by side in a block) or to the whole block; a thread holds NV vectors of it.
+template <typename T, int V, int NV, bool WARP>
 __global__ void __launch_bounds__(256) gated_norm_kernel(GatedNormArgs a) {
   __shared__ float sh[2 * 2 * 32];
   pdl_launch_dependents();
   pdl_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int g = WARP ? blockIdx.y * (blockDim.x >> 5) + warp : blockIdx.y, x0 = WARP ? lane : threadIdx.x, step = WARP ? 32 : blockDim.x;
+  const int g = WARP ? blockIdx.y * (blockDim.x >> 5) + warp : blockIdx.y, x0 = (WARP ? lane : threadIdx.x) * V, step = (WARP ? 32 : blockDim.x) * V;
   if (WARP && g * a.part >= a.width) return;
   const T* y = (const T*)a.y + (size_t)blockIdx.x * a.width + (size_t)g * a.part;
   const T* z = (const T*)a.gate + (size_t)blockIdx.x * a.gate_stride + (size_t)g * a.part;
   T* o = (T*)a.out + (size_t)blockIdx.x * a.width + (size_t)g * a.part;
-  constexpr int HOLD = 2;            // vectors kept from the first pass to the second
-  float held[HOLD][V], gate[HOLD][V], s[1] = {0.f};
-  auto value = [&](int c, float (&f)[V], float (&gt)[V]) {
-    float t[V];
-    load_v<T, V>(y + c, f);
-    load_v<T, V>(z + c, t);
+  float f[NV][V], gt[NV][V], s[1] = {0.f};
 #pragma unroll
-    for (int k = 0; k < V; ++k) {
-      gt[k] = t[k] * (sizeof(T) == 4 ? sigmoid_f(t[k]) : __fdividef(1.f, 1.f + __expf(-t[k])));
-      if (a.before) f[k] *= gt[k];
-    }
-  };
-  int i = 0;
-  for (int c = x0 * V; c < a.part; c += step * V, ++i) {
-    float f[V], gt[V];
-    value(c, f, gt);
+  for (int i = 0; i < NV; ++i)
+    if (x0 + i * step < a.part) { load_v<T, V>(y + x0 + i * step, f[i]); load_v<T, V>(z + x0 + i * step, gt[i]); }
 #pragma unroll
-    for (int k = 0; k < V; ++k) s[0] += f[k] * f[k];
+  for (int i = 0; i < NV; ++i)
+    if (x0 + i * step < a.part) {
 #pragma unroll
-    for (int q = 0; q < HOLD; ++q)
-      if (i == q) {
-#pragma unroll
-        for (int k = 0; k < V; ++k) { held[q][k] = f[k]; gate[q][k] = gt[k]; }
+      for (int k = 0; k < V; ++k) {
+        gt[i][k] *= gate_sigmoid<T>(gt[i][k]);
+        if (a.before) f[i][k] *= gt[i][k];
+        s[0] += f[i][k] * f[i][k];
       }
-  }
+    }
   if constexpr (WARP) s[0] = warp_sum(s[0]);
   else { int phase = 0; block_sums<1>(s, sh, phase); }
   const float r = 1.f / sqrtf(s[0] / (float)a.part + a.eps);
-  i = 0;
-  for (int c = x0 * V; c < a.part; c += step * V, ++i) {
-    float f[V], gt[V], w[V];
-    if (i >= HOLD) value(c, f, gt);
 #pragma unroll
-    for (int q = 0; q < HOLD; ++q)
-      if (i == q) {
-#pragma unroll
-        for (int k = 0; k < V; ++k) { f[k] = held[q][k]; gt[k] = gate[q][k]; }
-      }
+  for (int i = 0; i < NV; ++i) {
+    const int c = x0 + i * step;
+    if (c >= a.part) continue;
+    float w[V];
     if (a.w) load_v<float, V>(a.w + (size_t)g * a.part + c, w);
 #pragma unroll
     for (int k = 0; k < V; ++k) {
-      f[k] *= r;
-      if (a.w) f[k] *= w[k];
-      if (!a.before) f[k] *= gt[k];
+      f[i][k] *= r;
+      if (a.w) f[i][k] *= w[k];
+      if (!a.before) f[i][k] *= gt[i][k];
     }
-    store_v<T, V>(o + c, f);
+    store_v<T, V>(o + c, f[i]);
   }
 }
 
@@ -249,10 +233,22 @@ static int launch_state(const StateArgs& a, int segs, cudaStream_t st) {
 }
 template <typename T, int V>
 static int launch_gated_norm(const GatedNormArgs& a, int n, cudaStream_t st) {
-  const int parts = a.width / a.part;
-  if (a.part <= 64 * V) return (int)sfb_launch(gated_norm_kernel<T, V, true>, dim3(n, (parts + 7) / 8), dim3(parts < 8 ? 32 * parts : 256), 0, st, a);
-  const int threads = min(256, (a.part / V + 31) / 32 * 32);
-  return (int)sfb_launch(gated_norm_kernel<T, V, false>, dim3(n, parts), dim3(threads), 0, st, a);
+  const int parts = a.width / a.part, vecs = (a.part + V - 1) / V;
+  if (vecs <= 64) {
+    const dim3 g(n, (parts + 7) / 8), b(parts < 8 ? 32 * parts : 256);
+    return (int)(vecs <= 32 ? sfb_launch(gated_norm_kernel<T, V, 1, true>, g, b, 0, st, a) : sfb_launch(gated_norm_kernel<T, V, 2, true>, g, b, 0, st, a));
+  }
+  int nv = 1;
+  while (nv < 16 && (vecs + nv - 1) / nv > 256) nv *= 2;
+  const dim3 g(n, parts), b(((vecs + nv - 1) / nv + 31) / 32 * 32);
+  if (b.x > 256) return (int)cudaErrorInvalidValue;
+  switch (nv) {
+    case 1: return (int)sfb_launch(gated_norm_kernel<T, V, 1, false>, g, b, 0, st, a);
+    case 2: return (int)sfb_launch(gated_norm_kernel<T, V, 2, false>, g, b, 0, st, a);
+    case 4: return (int)sfb_launch(gated_norm_kernel<T, V, 4, false>, g, b, 0, st, a);
+    case 8: return (int)sfb_launch(gated_norm_kernel<T, V, 8, false>, g, b, 0, st, a);
+    default: return (int)sfb_launch(gated_norm_kernel<T, V, 16, false>, g, b, 0, st, a);
+  }
 }
 
 }  // namespace rows
@@ -281,7 +277,7 @@ int sfb_rows_gated_norm(const void* y, const void* gate, int64_t gate_stride, co
                         int fp32, cudaStream_t stream) {
   if (n < 1 || part < 1 || width % part || width / part > 65535) return (int)cudaErrorInvalidValue;
   GatedNormArgs a{y, gate, gate_stride, (const float*)w, out, width, part, before, eps};
-  const int v = part % 8 == 0 && gate_stride % 8 == 0 && (uintptr_t)gate % 16 == 0 ? 8 : part % 4 == 0 && gate_stride % 4 == 0 && (uintptr_t)gate % (fp32 ? 16 : 8) == 0 ? 4 : 1;
+  const int v = part % 8 == 0 && part > 128 && gate_stride % 8 == 0 && (uintptr_t)gate % 16 == 0 ? 8 : part % 4 == 0 && gate_stride % 4 == 0 && (uintptr_t)gate % (fp32 ? 16 : 8) == 0 ? 4 : 1;
   if (fp32) return v >= 4 ? launch_gated_norm<float, 4>(a, n, stream) : launch_gated_norm<float, 1>(a, n, stream);
   return v == 8 ? launch_gated_norm<__nv_bfloat16, 8>(a, n, stream) : v == 4 ? launch_gated_norm<__nv_bfloat16, 4>(a, n, stream)
                                                                             : launch_gated_norm<__nv_bfloat16, 1>(a, n, stream);

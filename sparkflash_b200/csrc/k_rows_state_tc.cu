@@ -166,9 +166,14 @@ chunk_sums_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant_
       if (n < a.Np) {
         float* o = a.sums + (((size_t)chunk * a.H + h) * a.P + pt * 64 + half * 32) * a.Np + n;
         const int m = min(32, a.P - pt * 64 - half * 32);
+        if (m == 32 && n < a.N) {
 #pragma unroll
-        for (int c = 0; c < 32; ++c)
-          if (c < m) o[(size_t)c * a.Np] = n < a.N ? f[c] : 0.f;
+          for (int c = 0; c < 32; ++c) o[(size_t)c * a.Np] = f[c];
+        } else {
+#pragma unroll
+          for (int c = 0; c < 32; ++c)
+            if (c < m) o[(size_t)c * a.Np] = n < a.N ? f[c] : 0.f;
+        }
       }
     }
     fence_before();
