@@ -2,16 +2,19 @@
 // attention.  A step holds n rows of any mix of lanes; the rows of one lane are a *segment* (consecutive, in position order).
 //
 //   seam       residual += norm(sublayer output), then the next sublayer's norm, in one pass over a row; options: the output is
-//              half the sum of two branches with an RMS norm each; the row starts from the embedding table; a loop pass adds
+//              half the sum of two branches with an RMS norm each, or a weighted sum of several parts; it is scaled element by element
+//              instead of normed; norms are layer norms or RMS norms; the row starts from the embedding table; a loop pass adds
 //              the embedding output and a vector; a step of single-row segments also applies the input convolution; the embedding is
 //              scaled; without a next norm h is the residual at activation precision.
 //   conv       causal depthwise convolution with carried inputs, optionally added to its input or followed by silu, optionally with a
 //              bias.
 //   qk_append  RMS norm over a whole query / key projection, keys and values into the paged cache.
+//   rot_append rotated queries and keys, values mixed with another layer's, into the paged cache.
+//   token_gate gelu(projection) * the token's row of a table.
 //   gated scan real-gated linear recurrence S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t with a = exp(-c r softplus(lam)):
 //              two passes over chunks of rows for prompts (the chunks' start states in between), one fused kernel (convolution, gates, recurrence,
 //              output gate) for single rows.
-//   act_mul    act(gate) * up, act = silu or the tanh form of gelu.
+//   act_mul    act(gate) * up, act = silu, the tanh form of gelu, or the clamped gate.
 //
 // Recurrent state (scan state, convolution inputs) has two versions per lane.  A segment reads version `src` (-1: zeros) and
 // writes version `dst`, so every block of a launch sees the state before the step, a replayed graph repeats the same result,
@@ -27,7 +30,8 @@ struct SeamArgs {
   const void* y;            // [rows, d] sublayer output (T) or null: no residual update
   const void* y2;           // second branch (T) or null
   const float *mw, *mw2;    // RMS weights of the two branches
-  const float *pw, *pb;     // post-norm
+  const float* parts_w;     // [rows, parts]: y is [rows, parts, d] and the output their weighted sum; or null
+  const float *pw, *pb;     // post-norm (pb null: no bias), or the scale
   const void* embed;        // [vocab, d] (T)
   const int* tokens;        // [rows]
   const float* step_vec;    // [d] or null: added after the update
@@ -39,9 +43,12 @@ struct SeamArgs {
   void* hist;               // [slots, taps - 1, d] (T)
   const int *src, *dst;     // [rows] state versions of single-row segments
   int from_embed, add_embed, taps, d, vocab;
+  int parts, post, rms;     // post: POST_*; rms: the next norm is an RMS norm
   float eps, embed_scale;
   Status* status;
 };
+
+constexpr int POST_LAYER = 0, POST_RMS = 1, POST_SCALE = 2;
 
 // Mean and sum of squared deviations of a row held as x[NV][V] per thread (`wcnt` = how many of the elements are this warp's):
 // each warp takes both about its own mean, then the warps' pairs are combined - one barrier.
@@ -90,8 +97,10 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512, !AHEAD && NV == 4 ? 4 : 1)
     for (int i = 0; i < NV; ++i) {
       const int c = c0 + i * step;
       if (c >= d) continue;
-      if (a.y) { load_v<float, V>(a.pw + c, pw[i]); load_v<float, V>(a.pb + c, pb[i]); }
-      if (a.nw) { load_v<float, V>(a.nw + c, nw[i]); load_v<float, V>(a.nb + c, nb[i]); }
+#pragma unroll
+      for (int k = 0; k < V; ++k) pb[i][k] = nb[i][k] = 0.f;
+      if (a.y) { load_v<float, V>(a.pw + c, pw[i]); if (a.pb) load_v<float, V>(a.pb + c, pb[i]); }
+      if (a.nw) { load_v<float, V>(a.nw + c, nw[i]); if (a.nb) load_v<float, V>(a.nb + c, nb[i]); }
       if (ahead_conv) {
 #pragma unroll
         for (int j = 0; j < TW; ++j)
@@ -164,21 +173,46 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512, !AHEAD && NV == 4 ? 4 : 1)
 #pragma unroll
           for (int k = 0; k < V; ++k) y[i][k] = y[i][k] * r0 * w0[k] + z[k] * r1 * w1[k];
         }
+    } else if (a.parts_w) {
+      const float* wr = a.parts_w + (size_t)row * a.parts;
+      yr = (const T*)a.y + (size_t)row * a.parts * d;
+#pragma unroll
+      for (int i = 0; i < NV; ++i)
+#pragma unroll
+        for (int k = 0; k < V; ++k) y[i][k] = 0.f;
+#pragma unroll 2
+      for (int j = 0; j < a.parts; ++j) {
+        const float wj = wr[j];
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+          if (c0 + i * step < d) {
+            float z[V];
+            load_v<T, V>(yr + (size_t)j * d + c0 + i * step, z);
+#pragma unroll
+            for (int k = 0; k < V; ++k) y[i][k] = fmaf(wj, z[k], y[i][k]);
+          }
+      }
     } else {
 #pragma unroll
       for (int i = 0; i < NV; ++i)
         if (c0 + i * step < d) load_v<T, V>(yr + c0 + i * step, y[i]);
     }
-    float mu, m2;
-    row_moments<V, NV>(y, c0, step, d, wcnt, winv, inv_d, sh, phase, mu, m2);
-    const float rs = 1.f / sqrtf(m2 * inv_d + a.eps);
+    float mu = 0.f, rs = 1.f;
+    if (a.post != POST_SCALE) {
+      float m2;
+      row_moments<V, NV>(y, c0, step, d, wcnt, winv, inv_d, sh, phase, mu, m2);
+      rs = 1.f / sqrtf((a.post == POST_RMS ? fmaf(mu, mu, m2 * inv_d) : m2 * inv_d) + a.eps);
+      if (a.post == POST_RMS) mu = 0.f;
+    }
 #pragma unroll
     for (int i = 0; i < NV; ++i)
       if (c0 + i * step < d) {
         if constexpr (!AHEAD) {
           float w[V], b[V];
           load_v<float, V>(a.pw + c0 + i * step, w);
-          load_v<float, V>(a.pb + c0 + i * step, b);
+#pragma unroll
+          for (int k = 0; k < V; ++k) b[k] = 0.f;
+          if (a.pb) load_v<float, V>(a.pb + c0 + i * step, b);
 #pragma unroll
           for (int k = 0; k < V; ++k) x[i][k] += (y[i][k] - mu) * rs * w[k] + b[k];
         } else {
@@ -209,14 +243,20 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512, !AHEAD && NV == 4 ? 4 : 1)
   if (!a.nw) return;
   float mu, m2;
   row_moments<V, NV>(x, c0, step, d, wcnt, winv, inv_d, sh, phase, mu, m2);
-  const float rs = 1.f / sqrtf(m2 * inv_d + a.eps);
+  const float rs = 1.f / sqrtf((a.rms ? fmaf(mu, mu, m2 * inv_d) : m2 * inv_d) + a.eps);
+  if (a.rms) mu = 0.f;
   T* hr = (T*)a.h + (size_t)out_row * d;
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int c = c0 + i * step;
     if (c >= d) continue;
     float o[V];
-    if constexpr (!AHEAD) { load_v<float, V>(a.nw + c, nw[i]); load_v<float, V>(a.nb + c, nb[i]); }
+    if constexpr (!AHEAD) {
+      load_v<float, V>(a.nw + c, nw[i]);
+#pragma unroll
+      for (int k = 0; k < V; ++k) nb[i][k] = 0.f;
+      if (a.nb) load_v<float, V>(a.nb + c, nb[i]);
+    }
 #pragma unroll
     for (int k = 0; k < V; ++k) o[k] = (x[i][k] - mu) * rs * nw[i][k] + nb[i][k];
     if (a.cw) {
@@ -408,6 +448,96 @@ __global__ void __launch_bounds__(256) qk_append_kernel(QkAppendArgs a) {
       const int cc = c - HD - GD, g = cc / a.vdim, x = cc - g * a.vdim;
       if (ok) store_v<T, V>((T*)a.vpool + (((size_t)page * a.G + g) * PAGE + slot) * a.vdim + x, f);
     }
+  }
+}
+
+// ---- rotated queries and keys, mixed values, cache append -------------------------------------------------------------------
+struct RotAppendArgs {
+  const void* proj;         // [n, stride] (T): q, k, v side by side
+  int64_t stride;
+  const float2* cs;         // [positions, half] (cos, sin)
+  void* q;                  // [n, H dim] (T)
+  void *kpool, *vpool;      // [pages, G, 64, dim] / [pages, G, 64, vdim] (T)
+  void* v_first;            // [n, G vdim] (T) or null: values of the layer that the others mix with
+  const float* lam;         // its share, or null: this layer is that one and leaves its values there
+  const int* table;
+  const int *row_lane, *row_pos;
+  int max_pages, n_pages, H, G, dim, vdim, half;
+  Status* status;
+};
+
+template <typename T, int V>
+__global__ void __launch_bounds__(256) rot_append_kernel(RotAppendArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x, HG = a.H + a.G, GV = a.G * a.vdim;
+  const T* p = (const T*)a.proj + (size_t)row * a.stride;
+  const int pos = a.row_pos[row];
+  const int page = a.table[(size_t)a.row_lane[row] * a.max_pages + pos / PAGE], slot = pos % PAGE;
+  const bool ok = page >= 0 && page < a.n_pages;
+  if (!ok && threadIdx.x == 0) status_set(a.status, ST_BOUNDS, 71, page, a.n_pages);
+  const float2* cs = a.cs + (size_t)pos * a.half;
+  // a head's units: V pairs of dims that turn together, then V dims that pass
+  const int turn = a.half / V, units = turn + (a.dim - 2 * a.half) / V;
+  for (int u = threadIdx.x; u < HG * units + GV / V; u += blockDim.x) {
+    if (u < HG * units) {
+      const int h = u / units, i = u - h * units;
+      const T* src = p + (size_t)h * a.dim;
+      T* dst = h < a.H ? (T*)a.q + ((size_t)row * a.H + h) * a.dim : (T*)a.kpool + (((size_t)page * a.G + h - a.H) * PAGE + slot) * a.dim;
+      if (h >= a.H && !ok) continue;
+      if (i < turn) {
+        float x[V], y[V], c[2 * V];
+        const int d = i * V;
+        load_v<T, V>(src + d, x);
+        load_v<T, V>(src + a.half + d, y);
+        if constexpr (V == 1) { const float2 t = cs[d]; c[0] = t.x; c[1] = t.y; }
+        else {
+#pragma unroll
+          for (int k = 0; k < V / 2; ++k) load_v<float, 4>(reinterpret_cast<const float*>(cs + d + 2 * k), c + 4 * k);
+        }
+#pragma unroll
+        for (int k = 0; k < V; ++k) {
+          const float t = x[k];
+          x[k] = t * c[2 * k] - y[k] * c[2 * k + 1];
+          y[k] = y[k] * c[2 * k] + t * c[2 * k + 1];
+        }
+        store_v<T, V>(dst + d, x);
+        store_v<T, V>(dst + a.half + d, y);
+      } else {
+        const int d = 2 * a.half + (i - turn) * V;
+        float x[V];
+        load_v<T, V>(src + d, x);
+        store_v<T, V>(dst + d, x);
+      }
+    } else {
+      const int c = (u - HG * units) * V, g = c / a.vdim, d = c - g * a.vdim;
+      float x[V];
+      load_v<T, V>(p + (size_t)HG * a.dim + c, x);
+      if (a.lam) {
+        const float lam = *a.lam;
+        float f[V];
+        load_v<T, V>((const T*)a.v_first + (size_t)row * GV + c, f);
+#pragma unroll
+        for (int k = 0; k < V; ++k) x[k] = (1.f - lam) * x[k] + lam * f[k];
+      } else if (a.v_first) {
+        store_v<T, V>((T*)a.v_first + (size_t)row * GV + c, x);
+      }
+      if (ok) store_v<T, V>((T*)a.vpool + (((size_t)page * a.G + g) * PAGE + slot) * a.vdim + d, x);
+    }
+  }
+}
+
+// ---- gelu(projection) * a part of the token's row of a table ----------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256) token_gate_kernel(const T* z, const T* table, const int* tokens, T* out, int n, int dim, int64_t table_stride, int col0, int vocab,
+                                                         Status* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < (int64_t)n * dim; i += (int64_t)gridDim.x * blockDim.x) {
+    const int row = (int)(i / dim), c = (int)(i - (int64_t)row * dim);
+    int tok = tokens[row];
+    if (tok < 0 || tok >= vocab) { status_set(status, ST_BOUNDS, 72, tok, vocab); tok = 0; }
+    out[i] = from_f<T>(gate_gelu<T>(to_f<T>(z[i])) * to_f<T>(table[(size_t)tok * table_stride + col0 + c]));
   }
 }
 
@@ -688,7 +818,7 @@ __global__ void __launch_bounds__(256, 2) gated_row_kernel(GatedRowArgs a) {
 
 // ---- act(gate) * up --------------------------------------------------------------------------------------------------------
 template <typename T, int V>
-__global__ void __launch_bounds__(256) act_mul_kernel(const T* gu, T* out, int ff, int act) {
+__global__ void __launch_bounds__(256) act_mul_kernel(const T* gu, T* out, int ff, int64_t out_stride, int act, float alpha, float limit) {
   pdl_launch_dependents();
   pdl_wait();
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
@@ -698,8 +828,9 @@ __global__ void __launch_bounds__(256) act_mul_kernel(const T* gu, T* out, int f
   load_v<T, V>(gu + row * 2 * ff + c, g);
   load_v<T, V>(gu + row * 2 * ff + ff + c, u);
 #pragma unroll
-  for (int k = 0; k < V; ++k) g[k] = (act == ACT_GELU ? gate_gelu<T>(g[k]) : g[k] * gate_sigmoid<T>(g[k])) * u[k];
-  store_v<T, V>(out + row * ff + c, g);
+  for (int k = 0; k < V; ++k)
+    g[k] = act == ACT_CLAMP ? gate_clamp<T>(g[k], u[k], alpha, limit) : (act == ACT_GELU ? gate_gelu<T>(g[k]) : g[k] * gate_sigmoid<T>(g[k])) * u[k];
+  store_v<T, V>(out + row * out_stride + c, g);
 }
 
 // ---- dispatch ---------------------------------------------------------------------------------------------------------------
@@ -749,14 +880,14 @@ using namespace sfb::rows;
 extern "C" {
 
 // fp32: 1 = float activations, 0 = bf16.  See SeamArgs for the rest; null pointers switch the parts off.
-int sfb_rows_seam(void* x, const void* y, const void* y2, const void* mw, const void* mw2, const void* pw, const void* pb, const void* embed,
+int sfb_rows_seam(void* x, const void* y, const void* y2, const void* mw, const void* mw2, const void* parts_w, const void* pw, const void* pb, const void* embed,
                   const int* tokens, const void* step_vec, void* tap, const void* nw, const void* nb, void* h, const int* row_map,
-                  const void* cw, void* hist, const int* src, const int* dst, int from_embed, int add_embed, int taps, int n, int d,
+                  const void* cw, void* hist, const int* src, const int* dst, int from_embed, int add_embed, int taps, int parts, int post, int rms, int n, int d,
                   int vocab, float eps, float embed_scale, int fp32, void* status, cudaStream_t stream) {
-  if (n < 1 || d < 1) return (int)cudaErrorInvalidValue;
-  SeamArgs a{(float*)x, y, y2, (const float*)mw, (const float*)mw2, (const float*)pw, (const float*)pb, embed, tokens, (const float*)step_vec,
+  if (n < 1 || d < 1 || (parts_w && (parts < 1 || y2))) return (int)cudaErrorInvalidValue;
+  SeamArgs a{(float*)x, y, y2, (const float*)mw, (const float*)mw2, (const float*)parts_w, (const float*)pw, (const float*)pb, embed, tokens, (const float*)step_vec,
              (float*)tap, (const float*)nw, (const float*)nb, h, row_map, (const float*)cw, hist, src, dst, from_embed, add_embed, taps, d,
-             vocab, eps, embed_scale, (Status*)status};
+             vocab, parts, post, rms, eps, embed_scale, (Status*)status};
   if (fp32) return d % 4 ? launch_seam<float, 1>(a, n, stream) : launch_seam<float, 4>(a, n, stream);
   return d % 4 ? launch_seam<__nv_bfloat16, 1>(a, n, stream) : launch_seam<__nv_bfloat16, 4>(a, n, stream);
 }
@@ -824,15 +955,41 @@ int sfb_rows_gated_step(const void* x, int64_t x_stride, const void* y, int64_t 
                   : sfb_launch(gated_row_kernel<__nv_bfloat16, 1>, g, b, smem, stream, a));
 }
 
-int sfb_rows_act_mul(const void* gu, void* out, int n, int ff, int act, int fp32, cudaStream_t stream) {
+int sfb_rows_rot_append(const void* proj, int64_t stride, const void* cs, void* q, void* kpool, void* vpool, void* v_first, const void* lam,
+                        const int* table, const int* row_lane, const int* row_pos, int max_pages, int n_pages, int n, int H, int G, int dim, int vdim,
+                        int dims, int fp32, void* status, cudaStream_t stream) {
+  if (n < 1 || G < 1 || dims % 2 || dims < 0 || dims > dim || (lam && !v_first)) return (int)cudaErrorInvalidValue;
+  RotAppendArgs a{proj, stride, (const float2*)cs, q, kpool, vpool, v_first, (const float*)lam, table, row_lane, row_pos, max_pages, n_pages, H, G, dim, vdim,
+                  dims / 2, (Status*)status};
+  const int all = (dims / 2) | dim | vdim | (int)(stride & 1023);
+  const dim3 g(n), b(256);
+  if (!fp32 && all % 8 == 0) return (int)sfb_launch(rot_append_kernel<__nv_bfloat16, 8>, g, b, 0, stream, a);
+  const bool v4 = all % 4 == 0;
+  if (fp32) return (int)(v4 ? sfb_launch(rot_append_kernel<float, 4>, g, b, 0, stream, a) : sfb_launch(rot_append_kernel<float, 1>, g, b, 0, stream, a));
+  return (int)(v4 ? sfb_launch(rot_append_kernel<__nv_bfloat16, 4>, g, b, 0, stream, a) : sfb_launch(rot_append_kernel<__nv_bfloat16, 1>, g, b, 0, stream, a));
+}
+
+int sfb_rows_token_gate(const void* z, const void* table, const int* tokens, void* out, int n, int dim, int64_t table_stride, int col0, int vocab, int fp32,
+                        void* status, cudaStream_t stream) {
+  if (n < 1 || dim < 1) return (int)cudaErrorInvalidValue;
+  const int64_t blocks = ((int64_t)n * dim + 255) / 256;
+  const dim3 g((unsigned)(blocks < 1184 ? blocks : 1184)), b(256);
+  if (fp32) return (int)sfb_launch(token_gate_kernel<float>, g, b, 0, stream, (const float*)z, (const float*)table, tokens, (float*)out, n, dim, table_stride, col0, vocab, (Status*)status);
+  return (int)sfb_launch(token_gate_kernel<__nv_bfloat16>, g, b, 0, stream, (const __nv_bfloat16*)z, (const __nv_bfloat16*)table, tokens, (__nv_bfloat16*)out, n, dim,
+                         table_stride, col0, vocab, (Status*)status);
+}
+
+int sfb_rows_act_mul(const void* gu, void* out, int64_t out_stride, int n, int ff, int act, float alpha, float limit, int fp32, cudaStream_t stream) {
   if (n < 1 || ff < 1) return (int)cudaErrorInvalidValue;
-  const int V = ff % 4 ? 1 : (fp32 || ff % 8) ? 4 : 8;
+  const int all = ff | (int)(out_stride & 1023), V = all % 4 ? 1 : (fp32 || all % 8) ? 4 : 8;
   const dim3 g(n, (ff + 256 * V - 1) / (256 * V)), b(256);
-  if (fp32) return (int)(V == 4 ? sfb_launch(act_mul_kernel<float, 4>, g, b, 0, stream, (const float*)gu, (float*)out, ff, act)
-                                : sfb_launch(act_mul_kernel<float, 1>, g, b, 0, stream, (const float*)gu, (float*)out, ff, act));
-  if (V == 8) return (int)sfb_launch(act_mul_kernel<__nv_bfloat16, 8>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff, act);
-  return (int)(V == 4 ? sfb_launch(act_mul_kernel<__nv_bfloat16, 4>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff, act)
-                      : sfb_launch(act_mul_kernel<__nv_bfloat16, 1>, g, b, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, ff, act));
+  if (fp32) return (int)(V == 4 ? sfb_launch(act_mul_kernel<float, 4>, g, b, 0, stream, (const float*)gu, (float*)out, ff, out_stride, act, alpha, limit)
+                                : sfb_launch(act_mul_kernel<float, 1>, g, b, 0, stream, (const float*)gu, (float*)out, ff, out_stride, act, alpha, limit));
+  const __nv_bfloat16* i = (const __nv_bfloat16*)gu;
+  __nv_bfloat16* o = (__nv_bfloat16*)out;
+  if (V == 8) return (int)sfb_launch(act_mul_kernel<__nv_bfloat16, 8>, g, b, 0, stream, i, o, ff, out_stride, act, alpha, limit);
+  return (int)(V == 4 ? sfb_launch(act_mul_kernel<__nv_bfloat16, 4>, g, b, 0, stream, i, o, ff, out_stride, act, alpha, limit)
+                      : sfb_launch(act_mul_kernel<__nv_bfloat16, 1>, g, b, 0, stream, i, o, ff, out_stride, act, alpha, limit));
 }
 
 }  // extern "C"

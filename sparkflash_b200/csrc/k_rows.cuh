@@ -77,7 +77,7 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
 }
 
 
-constexpr int ACT_SILU = 1, ACT_GELU = 2;      // activations of the gated products
+constexpr int ACT_SILU = 1, ACT_GELU = 2, ACT_CLAMP = 3;      // activations of the gated products
 
 // exp, reciprocal and square root of the gates, all 32-bit: library-accurate with float activations; with bf16 activations the
 // hardware approximations (relative error below 2^-21), whose error is far below the rounding of u
@@ -91,6 +91,13 @@ template <typename T> __device__ __forceinline__ float gate_gelu(float z) {
     const float k = 1.5957691216057308f * (z + 0.044715f * z * z * z);
     return z * gate_sigmoid<T>(k);
   }
+}
+
+// clamped gate: g = min(gate, limit), u = clamp(up, -limit, limit): g sigmoid(alpha g) (u + 1)
+template <typename T> __device__ __forceinline__ float gate_clamp(float g, float u, float alpha, float limit) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g * gate_sigmoid<T>(alpha * g) * (u + 1.f);
 }
 
 }  // namespace rows

@@ -1,5 +1,6 @@
 // Softmax attention over the paged cache for single rows and short runs of rows (k_rows_attn_tc.cu takes long runs), in bf16
-// or true 32-bit, any head sizes: score = (q . k) * scale - bias[head][distance], causal, the last `window` positions.
+// or true 32-bit, any head sizes: score = (q . k) * scale - bias[head][distance], causal, the last `window` positions; optionally
+// cap * tanh(score / cap), and a sink: a number per head whose exponential is in the softmax's denominator only.
 //
 // Values may be the first columns of the keys (vpool null): then only key pages are read.  The bias is a table over the distance i - j ([heads, table length], 32-bit), so any distance-only bias is one row of
 // numbers per head; null: none.
@@ -21,6 +22,8 @@ struct AttnRowsArgs {
   const int* rows;          // [rows in this launch] row indices, or null: identity
   const float* bias;        // [H, bias_len] or null
   int64_t bias_len;
+  const float* sink;        // [H] or null
+  float cap;                // 0: none
   void* out;                // [n, H vdim] (T)
   float* part;              // [launch rows, H, splits, vdim]
   float* ml;                // [launch rows, H, splits, 2]
@@ -136,7 +139,10 @@ __global__ void __launch_bounds__(ATHREADS) attn_rows_kernel(AttnRowsArgs a) {
         dot[r] += __shfl_xor_sync(0xffffffffu, dot[r], 1);
         if (half == (r & 1) && r < nh) {
           float v = -INFINITY;
-          if (dist >= 0 && dist < a.window) v = a.bias ? dot[r] - a.bias[(size_t)(h0 + r) * a.bias_len + dist] : dot[r];
+          if (dist >= 0 && dist < a.window) {
+            v = a.bias ? dot[r] - a.bias[(size_t)(h0 + r) * a.bias_len + dist] : dot[r];
+            if (a.cap > 0.f) v = a.cap * tanhf(v / a.cap);
+          }
           ps[r * AP + key] = v;
         }
       }
@@ -202,7 +208,15 @@ __global__ void __launch_bounds__(ATHREADS) attn_rows_kernel(AttnRowsArgs a) {
     const int r = i / a.vdim, v = i - r * a.vdim;
     float t = 0.f;
     for (int k = 0; k < groups; ++k) t += red[((size_t)k * R + r) * cols * 4 + v];
-    if (a.splits == 1) ((T*)a.out)[(io * a.H + h0 + r) * a.vdim + v] = from_f<T>(t / msum[2 * r + 1]);
+    if (a.splits == 1) {
+      float l = msum[2 * r + 1];
+      if (a.sink) {                       // relative to the larger of the sink and the scores' maximum
+        const float sk = a.sink[h0 + r], m = fmaxf(msum[2 * r], sk), f = expf(msum[2 * r] - m);
+        t *= f;
+        l = l * f + expf(sk - m);
+      }
+      ((T*)a.out)[(io * a.H + h0 + r) * a.vdim + v] = from_f<T>(t / l);
+    }
     else a.part[(((size_t)blockIdx.y * a.H + h0 + r) * a.splits + blockIdx.z) * a.vdim + v] = t;
   }
   if (a.splits > 1 && tid < 2 * nh) a.ml[(((size_t)blockIdx.y * a.H + h0 + (tid >> 1)) * a.splits + blockIdx.z) * 2 + (tid & 1)] = msum[tid];
@@ -218,6 +232,7 @@ __global__ void __launch_bounds__(128) attn_rows_merge_kernel(AttnRowsArgs a) {
   const float* part = a.part + ((size_t)blockIdx.y * a.H + h) * a.splits * a.vdim;
   float m = -INFINITY, l = 0.f;
   for (int s = 0; s < a.splits; ++s) m = fmaxf(m, ml[2 * s]);
+  if (a.sink) { m = fmaxf(m, a.sink[h]); l = expf(a.sink[h] - m); }
   for (int s = 0; s < a.splits; ++s) l += ml[2 * s + 1] * expf(ml[2 * s] - m);
   for (int v = threadIdx.x; v < a.vdim; v += blockDim.x) {
     float t = 0.f;
@@ -270,12 +285,12 @@ using namespace sfb::rows;
 extern "C" {
 
 int sfb_rows_attn(const void* q, const void* kpool, const void* vpool, const int* table, const int* row_lane, const int* row_pos,
-                  const int* rows, const void* bias, int64_t bias_len, void* out, void* part, void* ml, int max_pages, int n_pages,
+                  const int* rows, const void* bias, int64_t bias_len, const void* sink, float cap, void* out, void* part, void* ml, int max_pages, int n_pages,
                   int n_rows, int H, int G, int dim, int vdim, int splits, int window, int compact, float scale, int fp32, void* status, cudaStream_t stream) {
   if (n_rows < 1 || n_rows > 65535 || G < 1 || H % G || vdim > 4 * ATHREADS || dim < 1 || vdim < 1 || splits < 1 || window < 1 || (!vpool && vdim > dim)) return (int)cudaErrorInvalidValue;
   AttnRowsArgs a{};
   a.q = q; a.kpool = kpool; a.vpool = vpool; a.table = table; a.row_lane = row_lane; a.row_pos = row_pos; a.rows = rows;
-  a.bias = (const float*)bias; a.bias_len = bias_len; a.out = out; a.part = (float*)part; a.ml = (float*)ml; a.max_pages = max_pages;
+  a.bias = (const float*)bias; a.bias_len = bias_len; a.sink = (const float*)sink; a.cap = cap; a.out = out; a.part = (float*)part; a.ml = (float*)ml; a.max_pages = max_pages;
   a.n_pages = n_pages; a.H = H; a.G = G; a.dim = dim; a.vdim = vdim; a.splits = splits; a.scale = scale; a.status = (Status*)status;
   a.window = window; a.compact = compact;
   return fp32 ? launch_attn_r<float>(a, n_rows, stream) : launch_attn_r<__nv_bfloat16>(a, n_rows, stream);

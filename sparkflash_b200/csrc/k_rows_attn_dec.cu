@@ -1,4 +1,5 @@
-// Softmax attention of single rows over the paged cache, bf16, paced by memory: score = (q . k) * scale - bias[head][distance].
+// Softmax attention of single rows over the paged cache, bf16, paced by memory: score = (q . k) * scale - bias[head][distance], the last
+// `window` positions; optionally cap * tanh(score / cap), and a sink per head whose exponential is in the denominator only.
 //
 // The pages of all (row, head group) units of the launch form one sequence that is cut evenly over a fixed number of CTAs, so
 // rows of any lengths keep every SM busy to the end.  A CTA's producer warp streams its pages (a page of one head's keys and of
@@ -23,6 +24,9 @@ struct Args {
   const int* rows;              // row indices or null
   const float* bias;            // [H, bias_len] or null
   int64_t bias_len;
+  const float* sink;            // [H] or null
+  float cap;                    // 0: none
+  int window;                   // keys a row sees: itself and the window - 1 before it
   __nv_bfloat16* out;           // [n, H vdim]
   float* part;                  // [2 CTAs, R, vdim]
   float* ml;                    // [2 CTAs, R, 2]
@@ -57,7 +61,22 @@ __device__ __forceinline__ float ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-__device__ __forceinline__ int row_pages(const Args& a, int r) { return a.row_pos[a.rows ? a.rows[r] : r] / PAGE + 1; }
+__device__ __forceinline__ int first_page(const Args& a, int pos) { return max(0, pos - a.window + 1) / PAGE; }
+__device__ __forceinline__ int row_pages(const Args& a, int r) {
+  const int pos = a.row_pos[a.rows ? a.rows[r] : r];
+  return pos / PAGE + 1 - first_page(a, pos);
+}
+// cap * tanh(x / cap) without cancellation that would show next to the cap's rounding
+__device__ __forceinline__ float capped(float x, float cap) {
+  const float e = __expf(-2.f * fabsf(x) / cap);
+  return copysignf(cap * __fdividef(1.f - e, 1.f + e), x);
+}
+// a finished unit: output relative to the larger of the scores' maximum and the sink (both in units of log2)
+__device__ __forceinline__ float finish(const Args& a, int head, float o, float m, float l) {
+  if (!a.sink) return o / l;
+  const float sk = a.sink[head] * LOG2E, top = fmaxf(m, sk), f = ex2(m - top);
+  return o * f / (l * f + ex2(sk - top));
+}
 // pages per CTA: even shares, but no CTA for less than a couple of pages
 __device__ __forceinline__ int share(int total, int ctas) { return max((total + ctas - 1) / ctas, MIN_PAGES); }
 
@@ -124,7 +143,7 @@ __global__ void __launch_bounds__(THREADS, KC * R <= 8 && NVV == 1 ? 2 : 1) attn
       for (int at = begin; at < end; ++at, ++i, next(c)) {
         const int st = i % a.stages, ph = (i / a.stages) & 1;
         const int row = a.rows ? a.rows[c.r] : c.r;
-        int page = a.table[(size_t)a.row_lane[row] * a.max_pages + c.p];
+        int page = a.table[(size_t)a.row_lane[row] * a.max_pages + first_page(a, a.row_pos[row]) + c.p];
         if (page < 0 || page >= a.n_pages) { status_set(a.status, ST_BOUNDS, 65, page, a.n_pages); page = 0; }
         const size_t blk = (size_t)page * a.G + c.u / a.hgroups;
         mbar_wait(&empty[st], ph ^ 1, dead);
@@ -174,7 +193,7 @@ __global__ void __launch_bounds__(THREADS, KC * R <= 8 && NVV == 1 ? 2 : 1) attn
           }
         }
       }
-      const int dist = pos - (c.p * PAGE + key);
+      const int dist = pos - ((first_page(a, pos) + c.p) * PAGE + key);
       float b[R];
 #pragma unroll
       for (int r = 0; r < R; ++r) b[r] = (a.bias && dist >= 0 && r < nh) ? a.bias[(size_t)(h0 + r) * a.bias_len + dist] : 0.f;
@@ -204,7 +223,9 @@ __global__ void __launch_bounds__(THREADS, KC * R <= 8 && NVV == 1 ? 2 : 1) attn
         float s = dot[r];
         s += __shfl_xor_sync(0xffffffffu, s, 1);
         s += __shfl_xor_sync(0xffffffffu, s, 2);
-        s = dist >= 0 ? (s * a.scale - b[r]) * LOG2E : -INFINITY;
+        s = s * a.scale - b[r];
+        if (a.cap > 0.f) s = capped(s, a.cap);
+        s = dist >= 0 && dist < a.window ? s * LOG2E : -INFINITY;
         float mx = s;
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 4));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 8));
@@ -287,7 +308,7 @@ __global__ void __launch_bounds__(THREADS, KC * R <= 8 && NVV == 1 ? 2 : 1) attn
             o += red[((size_t)w * R + r) * a.vdim + v] * f;
             ll += wl[w][r] * f;
           }
-          if (whole) a.out[((size_t)row * a.H + h0 + r) * a.vdim + v] = __float2bfloat16_rn(o / ll);
+          if (whole) a.out[((size_t)row * a.H + h0 + r) * a.vdim + v] = __float2bfloat16_rn(finish(a, h0 + r, o, mm, ll));
           else {
             a.part[((size_t)slot * R + r) * a.vdim + v] = o;
             if (v == 0) { a.ml[((size_t)slot * R + r) * 2] = mm; a.ml[((size_t)slot * R + r) * 2 + 1] = ll; }
@@ -334,6 +355,10 @@ __global__ void __launch_bounds__(128) attn_stream_merge_kernel(Args a) {
     float m = -INFINITY, l = 0.f;
     for (int c = lane; c < parts; c += 32) m = fmaxf(m, a.ml[((size_t)(2 * (c0 + c) + (start > (c0 + c) * per)) * R + k) * 2]);
     m = warp_max(m);
+    if (a.sink) {
+      m = fmaxf(m, a.sink[h0 + k] * LOG2E);
+      if (lane == 0) l = ex2(a.sink[h0 + k] * LOG2E - m);
+    }
     for (int c = lane; c < parts; c += 32) {
       const size_t s = (size_t)(2 * (c0 + c) + (start > (c0 + c) * per)) * R + k;
       const float f = ex2(a.ml[2 * s] - m);
@@ -414,13 +439,13 @@ extern "C" {
 // bf16 only; dim and vdim multiples of 32 up to 256 (dim: 32, 64, 96, 128, 256), at most 1,024 rows.  heads_per_unit: 1, 2 or 4.
 // page_bound: upper bound of the sum of the rows' pages.  part / ml: 2 x 592 x heads_per_unit x vdim (x 2) floats.
 int sfb_rows_attn_stream(const void* q, const void* kpool, const void* vpool, const int* table, const int* row_lane, const int* row_pos,
-                         const int* rows, const void* bias, int64_t bias_len, void* out, void* part, void* ml, int max_pages, int n_pages,
+                         const int* rows, const void* bias, int64_t bias_len, const void* sink, float cap, int window, void* out, void* part, void* ml, int max_pages, int n_pages,
                          int n_rows, int H, int G, int dim, int vdim, int heads_per_unit, int page_bound, float scale, void* status,
                          cudaStream_t stream) {
-  if (n_rows < 1 || n_rows > MAX_ROWS || G < 1 || H % G || vdim % 32 || vdim < 32 || vdim > 256) return (int)cudaErrorInvalidValue;
+  if (n_rows < 1 || n_rows > MAX_ROWS || G < 1 || H % G || window < 1 || vdim % 32 || vdim < 32 || vdim > 256) return (int)cudaErrorInvalidValue;
   Args a{};
   a.q = (const __nv_bfloat16*)q; a.kpool = (const __nv_bfloat16*)kpool; a.vpool = (const __nv_bfloat16*)vpool; a.table = table;
-  a.row_lane = row_lane; a.row_pos = row_pos; a.rows = rows; a.bias = (const float*)bias; a.bias_len = bias_len; a.out = (__nv_bfloat16*)out;
+  a.row_lane = row_lane; a.row_pos = row_pos; a.rows = rows; a.bias = (const float*)bias; a.bias_len = bias_len; a.sink = (const float*)sink; a.cap = cap; a.window = window; a.out = (__nv_bfloat16*)out;
   a.part = (float*)part; a.ml = (float*)ml; a.max_pages = max_pages; a.n_pages = n_pages; a.n_rows = n_rows; a.H = H; a.G = G; a.dim = dim;
   a.vdim = vdim; a.scale = scale; a.status = (Status*)status;
   switch (dim) {

@@ -1,5 +1,6 @@
 // Softmax attention over the paged cache for long runs of rows, on tcgen05: score = (q . k) * scale - bias[head][distance],
-// causal, the last `window` positions, bf16 queries / keys / values, 32-bit scores, softmax and accumulators.
+// causal, the last `window` positions, bf16 queries / keys / values, 32-bit scores, softmax and accumulators.  Optionally
+// cap * tanh(score / cap) (no bias then), and a sink per head whose exponential is in the softmax's denominator only.
 //
 // One CTA: 256 consecutive query rows of one segment (two halves of 128) x one head.  Key tiles of one cache page (64 positions)
 // stream through shared memory by TMA: a (page, head) block is contiguous, so 64 dims of a tile are one box copy.
@@ -18,7 +19,8 @@
 //
 // Keys come from the page pool through the page table, or (`offs`) from rows that were multiplied out for this step: page p of a
 // tile's lane is then page p + offs[tile], heads k_head rows apart.  A key may have a second part that all heads share (template RS:
-// its own map, one 64-element slab), matched by the last columns of the head's query; there is no bias then.
+// its own map, one 64-element slab), matched by the last columns of the head's query; there is no bias then.  Template MODE: what
+// happens to a scaled score (nothing, the bias, the cap).
 //
 // No cluster, no multicast; every wait is bounded and reports through the status word.
 #include "k_rows_tc.cuh"
@@ -28,6 +30,7 @@ namespace rtc {
 using namespace tc;
 
 constexpr int THREADS = 384, ROWS = 256, HALF = 128, KT = 64, QSLAB = HALF * 128, SLAB = KT * 128, BST = 4;
+constexpr int PLAIN = 0, BIAS = 1, CAP = 2;
 constexpr int BW = 328;                       // bias copy stride: 319 values, = 8 mod 32 banks
 
 struct Args {
@@ -37,6 +40,8 @@ struct Args {
   const int* offs;           // page offset of every tile, or null: through the table
   const float* bias;         // [H, bias_len] or null
   int64_t bias_len;
+  const float* sink;         // [H] or null
+  float cap;
   __nv_bfloat16* out;        // [n, H vdim]
   int max_pages, n_pages, H, G, dim, vdim, rot;    // n_pages: of the pool, or of the rows multiplied out
   int k_page, k_head;        // rows between the pages and between the heads of the keys and values
@@ -45,24 +50,40 @@ struct Args {
   Status* status;
 };
 
-template <int DS, int VS, int RS>    // 64-element slabs of a query / key row, of a value row, and of the shared key part
+// tanh for |x| <= 1/2: the Taylor polynomial to x^13 (the next term is below 2^-24)
+__device__ __forceinline__ float2 tanh_small2(float2 x) {
+  const float2 t = fma2(x, x, make_float2(0.f, 0.f));
+  auto c = [](float v) { return make_float2(v, v); };
+  float2 p = fma2(t, c(21844.f / 6081075.f), c(-1382.f / 155925.f));
+  p = fma2(p, t, c(62.f / 2835.f));
+  p = fma2(p, t, c(-17.f / 315.f));
+  p = fma2(p, t, c(2.f / 15.f));
+  p = fma2(p, t, c(-1.f / 3.f));
+  return fma2(fma2(p, t, c(0.f)), x, x);
+}
+__device__ __forceinline__ float tanh_any(float x) {
+  const float e = ex2(-2.f * LOG2E * fabsf(x));
+  return copysignf(__fdividef(1.f - e, 1.f + e), x);
+}
+
+template <int DS, int VS, int RS, int MODE>    // 64-element slabs of a query / key row, of a value row, and of the shared key part
 struct Smem {
   static constexpr int ST = RS ? 3 : 4, QS = DS + RS;
   alignas(1024) uint8_t q[2 * QS * QSLAB];
   alignas(1024) uint8_t k[ST * QS * SLAB];
   alignas(1024) uint8_t v[ST * VS * SLAB];
-  alignas(16) float bias[RS ? 4 : BST * 4 * BW];
+  alignas(16) float bias[MODE == BIAS ? BST * 4 * BW : 4];
   alignas(8) uint64_t q_full, k_full[ST], k_empty[ST], v_full[ST], v_empty[ST], s_full[2], s_free[2], p_full[2], pv_done[2], b_full[BST], b_empty[BST];
   uint32_t tmem;
   int dead;
 };
 
-template <int DS, int VS, int RS>
+template <int DS, int VS, int RS, int MODE>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv,
                 const __grid_constant__ CUtensorMap mr, Args a) {
   extern __shared__ uint8_t raw[];
-  using SM = Smem<DS, VS, RS>;
+  using SM = Smem<DS, VS, RS, MODE>;
   constexpr int ST = SM::ST, QS = SM::QS;
   SM& S = *reinterpret_cast<SM*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -181,7 +202,7 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
         ok = mbar_wait(&S.k_empty[j % ST], (j / ST) & 1, dead) && mbar_wait(&S.v_empty[j % ST], (j / ST) & 1, dead);
     }
   } else if (warp == 11) {
-    if constexpr (RS == 0) {
+    if constexpr (MODE == BIAS) {
     const float* brow = a.bias ? a.bias + (size_t)h * a.bias_len : nullptr;
     for (int j = 0; j < nt; ++j) {
       const int st = j % BST, ph = (j / BST) & 1;
@@ -207,17 +228,17 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
     const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
     const uint32_t ts = tmem + w * 64 + lanes, tp = tmem + 128 + w * 64 + lanes, to = tmem + 256 + w * 128 + lanes;
     const int pos = pos0 + w * HALF + r, rr = w * HALF + r, shift = (ROWS - 1 - rr) & 3;
-    const float sl2 = a.scale * LOG2E;
+    const float sl2 = MODE == CAP ? a.scale / a.cap : a.scale * LOG2E;
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int j = 0; j < nt; ++j) {
       const int st = j % BST, ph = (j / BST) & 1;
-      if constexpr (RS == 0) {
+      if constexpr (MODE == BIAS) {
         ok = mbar_wait(&S.b_full[st], ph, dead);
         if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
       }
       if (j >= nw) {
-        if constexpr (RS == 0) mbar_arrive(&S.b_empty[st]);
+        if constexpr (MODE == BIAS) mbar_arrive(&S.b_empty[st]);
         continue;
       }
       ok = mbar_wait(&S.s_full[w], j & 1, dead);
@@ -228,15 +249,31 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
       wait_ld();
       fence_before();
       mbar_arrive(&S.s_free[w]);
-      const float* bp = S.bias + (RS ? 0 : st * 4 * BW + shift * BW + (ROWS - 1 - rr - shift));
+      const float* bp = S.bias + (MODE == BIAS ? st * 4 * BW + shift * BW + (ROWS - 1 - rr - shift) : 0);
+      if constexpr (MODE == CAP) {       // sl2: scale over cap
+        float big = 0.f;
+#pragma unroll
+        for (int c = 0; c < KT; ++c) big = fmaxf(big, fabsf(s[c]));
+        const float2 to2 = make_float2(sl2, sl2), back = make_float2(a.cap * LOG2E, a.cap * LOG2E), zero = make_float2(0.f, 0.f);
+        if (__all_sync(0xffffffffu, big * fabsf(sl2) <= 0.5f)) {
+#pragma unroll
+          for (int c = 0; c < KT; c += 2) {
+            const float2 t = fma2(tanh_small2(fma2(make_float2(s[c], s[c + 1]), to2, zero)), back, zero);
+            s[c] = t.x; s[c + 1] = t.y;
+          }
+        } else {
+#pragma unroll
+          for (int c = 0; c < KT; ++c) s[c] = tanh_any(s[c] * sl2) * back.x;
+        }
+      } else
 #pragma unroll
       for (int q = 0; q < KT / 4; ++q) {
-        const float4 b = RS ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(bp + 4 * q);
+        const float4 b = MODE != BIAS ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(bp + 4 * q);
         const float2 x = fma2(make_float2(s[4 * q], s[4 * q + 1]), make_float2(sl2, sl2), make_float2(b.x, b.y));
         const float2 y = fma2(make_float2(s[4 * q + 2], s[4 * q + 3]), make_float2(sl2, sl2), make_float2(b.z, b.w));
         s[4 * q] = x.x; s[4 * q + 1] = x.y; s[4 * q + 2] = y.x; s[4 * q + 3] = y.y;
       }
-      if constexpr (RS == 0) mbar_arrive(&S.b_empty[st]);
+      if constexpr (MODE == BIAS) mbar_arrive(&S.b_empty[st]);
       const int k0 = (j0 + j) * KT, vis = pos - k0, out = vis - a.window;      // keys out + 1 .. vis of the tile are visible
       if (k0 + KT - 1 > pos0 + w * HALF || k0 <= pos0 + w * HALF + HALF - 1 - a.window) {
 #pragma unroll
@@ -289,7 +326,7 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
       ok = mbar_wait(&S.pv_done[w], (nw - 1) & 1, dead);
       if (__all_sync(0xffffffffu, ok)) {
         fence_after();
-        const float inv = 1.f / l;
+        const float inv = 1.f / (a.sink ? l + ex2(a.sink[h] * LOG2E - m) : l);
         const bool valid = rr < rows;
         __nv_bfloat16* o = a.out + ((size_t)(row0 + rr) * a.H + h) * a.vdim;
         for (int c = 0; c < a.vdim; c += 16) {
@@ -319,16 +356,24 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
 typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
                              const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
-template <int DS, int VS, int RS>
-static int launch(const CUtensorMap* mq, const CUtensorMap* mk, const CUtensorMap* mv, const CUtensorMap* mr, const Args& a, int n_tiles, cudaStream_t st) {
-  const size_t smem = sizeof(Smem<DS, VS, RS>) + 1024;
+template <int DS, int VS, int RS, int MODE>
+static int launch_mode(const CUtensorMap* mq, const CUtensorMap* mk, const CUtensorMap* mv, const CUtensorMap* mr, const Args& a, int n_tiles, cudaStream_t st) {
+  const size_t smem = sizeof(Smem<DS, VS, RS, MODE>) + 1024;
   static bool done = false;
   if (!done) {
-    const cudaError_t e = cudaFuncSetAttribute(attn_run_kernel<DS, VS, RS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const cudaError_t e = cudaFuncSetAttribute(attn_run_kernel<DS, VS, RS, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     done = true;
   }
-  return (int)sfb_launch(attn_run_kernel<DS, VS, RS>, dim3(a.H, n_tiles), dim3(THREADS), smem, st, *mq, *mk, *mv, *mr, a);
+  return (int)sfb_launch(attn_run_kernel<DS, VS, RS, MODE>, dim3(a.H, n_tiles), dim3(THREADS), smem, st, *mq, *mk, *mv, *mr, a);
+}
+template <int DS, int VS, int RS>
+static int launch(const CUtensorMap* mq, const CUtensorMap* mk, const CUtensorMap* mv, const CUtensorMap* mr, const Args& a, int n_tiles, cudaStream_t st) {
+  if constexpr (RS == 0) {
+    if (a.cap > 0.f) return launch_mode<DS, VS, RS, CAP>(mq, mk, mv, mr, a, n_tiles, st);
+    if (a.bias) return launch_mode<DS, VS, RS, BIAS>(mq, mk, mv, mr, a, n_tiles, st);
+  }
+  return launch_mode<DS, VS, RS, PLAIN>(mq, mk, mv, mr, a, n_tiles, st);
 }
 
 }  // namespace rtc
@@ -359,12 +404,12 @@ int sfb_rows_tmap(void* out_map, const void* base, int64_t rows, int64_t cols, i
 // p k_page + g k_head (through the page table, or p + offs[tile]); mr: the shared key part [rows, rot] or null.  dim and vdim: multiples
 // of 8 up to 128; rot: a multiple of 8 up to 64.
 int sfb_rows_attn_tc(const void* mq, const void* mk, const void* mv, const void* mr, const int* table, const int* row_lane, const int* row_pos,
-                     const int* tiles, const int* offs, int n_tiles, const void* bias, int64_t bias_len, void* out, int max_pages, int n_pages, int H, int G,
+                     const int* tiles, const int* offs, int n_tiles, const void* bias, int64_t bias_len, const void* sink, float cap, void* out, int max_pages, int n_pages, int H, int G,
                      int dim, int vdim, int rot, int k_page, int k_head, int window, float scale, void* status, cudaStream_t stream) {
   if (n_tiles < 1 || n_tiles > 65535 || G < 1 || H % G || dim % 8 || vdim % 8 || dim < 8 || dim > 128 || vdim < 8 || vdim > 128 || rot % 8 || rot > 64 ||
-      (rot > 0) != (mr != nullptr) || (rot && bias) || window < 1)
+      (rot > 0) != (mr != nullptr) || (rot && bias) || (cap > 0.f && (bias || rot)) || window < 1)
     return (int)cudaErrorInvalidValue;
-  Args a{tiles, table, row_lane, row_pos, offs, (const float*)bias, bias_len, (__nv_bfloat16*)out, max_pages, n_pages, H, G, dim, vdim, rot, k_page, k_head,
+  Args a{tiles, table, row_lane, row_pos, offs, (const float*)bias, bias_len, (const float*)sink, cap, (__nv_bfloat16*)out, max_pages, n_pages, H, G, dim, vdim, rot, k_page, k_head,
          window, scale, (Status*)status};
   const CUtensorMap *q = (const CUtensorMap*)mq, *k = (const CUtensorMap*)mk, *v = (const CUtensorMap*)mv, *r = mr ? (const CUtensorMap*)mr : k;
   if (rot) {

@@ -14,6 +14,8 @@ struct Args {
   const __nv_bfloat16* bias;  // [M] or null
   void* out;                  // [n, M] bf16 (or float)
   int M, K, n, wk, f32, act;
+  int64_t out_stride;         // elements between the rows of out
+  float alpha, limit;         // of the clamped gate
 };
 
 template <int N>
@@ -105,9 +107,11 @@ __global__ void __launch_bounds__(256, 2) gemv_kernel(Args a) {
       for (int r = 1; r < N; ++r)
         if (lane == r) { s0 = acc[0][r]; s1 = acc[1][r]; }
       const int o = first + t * stride + g;
-      const size_t at = (size_t)lane * a.M;
+      const size_t at = (size_t)lane * a.out_stride;
       if (a.act) {
-        if (o < a.M) ((__nv_bfloat16*)a.out)[at + o] = __float2bfloat16_rn((a.act == rows::ACT_GELU ? rows::gelu_tanh_f(s0) : s0 * rows::sigmoid_f(s0)) * s1);
+        if (o < a.M)
+          ((__nv_bfloat16*)a.out)[at + o] = __float2bfloat16_rn(a.act == rows::ACT_CLAMP ? rows::gate_clamp<float>(s0, s1, a.alpha, a.limit)
+                                                                : (a.act == rows::ACT_GELU ? rows::gelu_tanh_f(s0) : s0 * rows::sigmoid_f(s0)) * s1);
       } else {
         const int r0 = 2 * o, r1 = r0 + 1;
         if (a.bias) { if (r0 < a.M) s0 += __bfloat162float(a.bias[r0]); if (r1 < a.M) s1 += __bfloat162float(a.bias[r1]); }
@@ -145,15 +149,16 @@ using namespace sfb::rgemv;
 
 extern "C" {
 
-// n <= 4 rows, K a multiple of 8, n K bounded by shared memory (4 K rows of 200 KB).  act (1 silu, 2 gelu): w holds 2 M rows, out [n, M].
-int sfb_rows_gemv(const void* w, const void* x, const void* bias, void* out, int n, int M, int K, int f32, int act, cudaStream_t stream) {
+// n <= 4 rows, K a multiple of 8, n K bounded by shared memory (4 K rows of 200 KB).  act (1 silu, 2 gelu, 3 clamped): w holds 2 M rows.
+int sfb_rows_gemv(const void* w, const void* x, const void* bias, void* out, int64_t out_stride, int n, int M, int K, int f32, int act, float alpha, float limit,
+                  cudaStream_t stream) {
   const int N = n <= 1 ? 1 : n <= 2 ? 2 : 4;
   if (n < 1 || n > 4 || M < 1 || K < 8 || K % 8 || (size_t)N * K * 2 > 200 * 1024) return (int)cudaErrorInvalidValue;
   const int pairs = act ? M : (M + 1) / 2, steps = (K + 255) / 256;
   int wk = 1;              // enough pairs of rows for every SM, at least a batch of K per warp
   while (wk < 8 && (long long)pairs * wk / 8 < 296 && steps / (wk * 2) >= 2) wk *= 2;
   const int needed = (pairs + 8 / wk - 1) / (8 / wk), blocks = needed < 296 ? needed : 296;
-  Args a{(const __nv_bfloat16*)w, (const __nv_bfloat16*)x, (const __nv_bfloat16*)bias, out, M, K, n, wk, f32, act};
+  Args a{(const __nv_bfloat16*)w, (const __nv_bfloat16*)x, (const __nv_bfloat16*)bias, out, M, K, n, wk, f32, act, out_stride, alpha, limit};
   return N == 1 ? launch<1>(a, blocks, stream) : N == 2 ? launch<2>(a, blocks, stream) : launch<4>(a, blocks, stream);
 }
 

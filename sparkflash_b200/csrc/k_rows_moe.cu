@@ -1,0 +1,308 @@
+// Mixture of experts on a step's rows: every row goes through `top` of E gated feed-forwards, and through a shared one.
+//
+//   moe_route   the chosen experts of a row and their weights (softmax over the chosen logits), and the shared expert's weight
+//               (sigmoid of one more logit); one warp per row
+//   moe_plan    (row, choice) pairs in order of their expert, cut into tiles of `tile` pairs of one expert
+//   moe_tile    one tile x 64 output columns on CUDA cores: any sizes, bf16 or 32-bit (k_rows_moe_tc.cu takes bf16 on tcgen05)
+//   moe_gemv    one to four rows, bf16: a block per (pair, share of the output), weights streamed; the shared expert's rows beside the pairs
+//
+// Both products of an expert go through the same kernels: `gated` (gate and up rows stacked, act(gate) * up, rows picked by the plan) and
+// down (rows of the first product in plan order, results at [row][choice], where the seam sums them with their weights).
+#include "k_rows.cuh"
+
+namespace sfb {
+namespace rmoe {
+using namespace rows;
+
+constexpr int MAX_E = 1024, MAX_TOP = 32;
+
+// ---- choice ---------------------------------------------------------------------------------------------------------------
+struct RouteArgs {
+  const float* z;           // [n, ld] router logits, then (shared) the shared expert's
+  int64_t ld;
+  int* ids;                 // [n, top]
+  float* wts;               // [n, top + shared]
+  int n, E, top, shared;
+};
+__global__ void __launch_bounds__(256) moe_route_kernel(RouteArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (row >= a.n) return;
+  const float* z = a.z + (size_t)row * a.ld;
+  uint32_t taken = 0;       // of this lane's experts lane, lane + 32, ...
+  float mine = 0.f;         // lane j: logit of choice j
+  int id = 0;
+  for (int j = 0; j < a.top; ++j) {
+    float best = -INFINITY;
+    int at = a.E;
+    for (int e = lane, k = 0; e < a.E; e += 32, ++k) {
+      const float v = z[e];
+      if (!(taken >> k & 1) && (v > best || at == a.E)) { best = v; at = e; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float v = __shfl_xor_sync(0xffffffffu, best, o);
+      const int e = __shfl_xor_sync(0xffffffffu, at, o);
+      if (e < a.E && (at == a.E || v > best || (v == best && e < at))) { best = v; at = e; }
+    }
+    at = __shfl_sync(0xffffffffu, at, 0);
+    best = __shfl_sync(0xffffffffu, best, 0);
+    at = min(at, a.E - 1);
+    if ((at & 31) == lane) taken |= 1u << (at >> 5);
+    if (lane == j) { mine = best; id = at; }
+  }
+  const float top = __shfl_sync(0xffffffffu, mine, 0), e = lane < a.top ? expf(mine - top) : 0.f, sum = warp_sum(e);
+  float* w = a.wts + (size_t)row * (a.top + a.shared);
+  if (lane < a.top) {
+    a.ids[(size_t)row * a.top + lane] = id;
+    w[lane] = e / sum;
+  }
+  if (a.shared && lane == 0) w[a.top] = sigmoid_f(z[a.E]);
+}
+
+// ---- plan -----------------------------------------------------------------------------------------------------------------
+struct PlanArgs {
+  const int* ids;           // [pairs]
+  int* order;               // [pairs] pair at every place
+  int* tiles;               // [max tiles][4]: expert, first place, pairs, -
+  int* count;               // number of tiles
+  int pairs, E, tile;
+};
+__global__ void __launch_bounds__(1024) moe_plan_kernel(PlanArgs a) {
+  __shared__ int cnt[MAX_E], wsum[2][32];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  cnt[tid] = 0;
+  pdl_launch_dependents();
+  pdl_wait();
+  __syncthreads();
+  for (int p0 = 0; p0 < a.pairs; p0 += 4096) {
+    int e[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) e[k] = p0 + k * 1024 + tid < a.pairs ? a.ids[p0 + k * 1024 + tid] : -1;
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if (e[k] >= 0) atomicAdd(&cnt[e[k]], 1);
+  }
+  __syncthreads();
+  const int c = cnt[tid], t = (c + a.tile - 1) / a.tile;
+  int sc = c, st = t;       // inclusive sums of pairs and of tiles over the experts
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int x = __shfl_up_sync(0xffffffffu, sc, o), y = __shfl_up_sync(0xffffffffu, st, o);
+    if (lane >= o) { sc += x; st += y; }
+  }
+  if (lane == 31) { wsum[0][warp] = sc; wsum[1][warp] = st; }
+  __syncthreads();
+  for (int w = 0; w < warp; ++w) { sc += wsum[0][w]; st += wsum[1][w]; }
+  const int first = sc - c;
+  for (int k = 0; k < t; ++k) reinterpret_cast<int4*>(a.tiles)[st - t + k] = make_int4(tid, first + k * a.tile, min(a.tile, c - k * a.tile), 0);
+  if (tid == 1023) *a.count = st;
+  cnt[tid] = first;         // from here on: the expert's next free place
+  __syncthreads();
+  for (int p0 = 0; p0 < a.pairs; p0 += 4096) {
+    int e[4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) e[k] = p0 + k * 1024 + tid < a.pairs ? a.ids[p0 + k * 1024 + tid] : -1;
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if (e[k] >= 0) a.order[atomicAdd(&cnt[e[k]], 1)] = p0 + k * 1024 + tid;
+  }
+}
+
+// ---- tiles on CUDA cores ----------------------------------------------------------------------------------------------------
+struct TileArgs {
+  const void* x;            // gated: [n, K] rows; down: [pairs, K] in plan order
+  const void* w;            // [E, (2) M, K]
+  void* out;                // gated: [pairs, M] in plan order; down: [n, slots, M]
+  const int *order, *tiles, *count;
+  int M, K, top, slots, gated;
+  float alpha, limit;
+};
+constexpr int TR = 32, TC = 64, TK = 16;
+
+template <typename T>
+__global__ void __launch_bounds__(256) moe_tile_kernel(TileArgs a) {
+  __shared__ float xs[TK][TR + 1], ws[2][TK][TC + 1];
+  pdl_launch_dependents();
+  pdl_wait();
+  if ((int)blockIdx.y >= *a.count) return;
+  const int4 t = reinterpret_cast<const int4*>(a.tiles)[blockIdx.y];
+  const int e = t.x, p0 = t.y, rows = t.z, c0 = blockIdx.x * TC, tid = threadIdx.x;
+  const int tr = tid >> 4, tc = tid & 15;            // rows tr, tr + 16; columns tc + 16 i
+  const int xr = tid >> 3, xk = (tid & 7) * 2;       // staged: row xr, two of its elements
+  const int place = p0 + min(xr, rows - 1);
+  const T* xp = (const T*)a.x + (size_t)(a.gated ? a.order[place] / a.top : place) * a.K;
+  const T* wp = (const T*)a.w + (size_t)e * (a.gated ? 2 : 1) * a.M * a.K;
+  float acc[2][2][4] = {};
+  for (int k0 = 0; k0 < a.K; k0 += TK) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) xs[xk + i][xr] = k0 + xk + i < a.K ? to_f<T>(xp[k0 + xk + i]) : 0.f;
+    for (int i = tid; i < (a.gated ? 2 : 1) * TC * TK; i += 256) {
+      const int g = i / (TC * TK), c = (i / TK) % TC, k = i % TK;
+      ws[g][k][c] = c0 + c < a.M && k0 + k < a.K ? to_f<T>(wp[((size_t)g * a.M + c0 + c) * a.K + k0 + k]) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < TK; ++k) {
+      const float x0 = xs[k][tr], x1 = xs[k][tr + 16];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float w0 = ws[0][k][tc + 16 * i];
+        acc[0][0][i] = fmaf(x0, w0, acc[0][0][i]);
+        acc[0][1][i] = fmaf(x1, w0, acc[0][1][i]);
+        if (a.gated) {
+          const float w1 = ws[1][k][tc + 16 * i];
+          acc[1][0][i] = fmaf(x0, w1, acc[1][0][i]);
+          acc[1][1][i] = fmaf(x1, w1, acc[1][1][i]);
+        }
+      }
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int row = tr + 16 * r;
+    if (row >= rows) continue;
+    size_t o;
+    if (a.gated) o = (size_t)(p0 + row);
+    else { const int pair = a.order[p0 + row]; o = (size_t)(pair / a.top) * a.slots + pair % a.top; }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int c = c0 + tc + 16 * i;
+      if (c < a.M) ((T*)a.out)[o * a.M + c] = from_f<T>(a.gated ? gate_clamp<T>(acc[0][r][i], acc[1][r][i], a.alpha, a.limit) : acc[0][r][i]);
+    }
+  }
+}
+
+// ---- few rows -----------------------------------------------------------------------------------------------------------------
+struct GemvArgs {
+  const int* ids;             // [pairs] experts
+  const __nv_bfloat16* x;     // gated: [n, K]; down: [pairs, K]
+  const __nv_bfloat16* w;     // [E, (2) M, K]
+  __nv_bfloat16* out;         // gated: [pairs, M]; down: [n, slots, M]
+  const __nv_bfloat16 *sx, *sw;     // the shared expert: gated [n, SK], down [n, SK]; null: none
+  __nv_bfloat16* sout;        // gated: [n, SM]
+  int pairs, n, M, K, SM, SK, top, slots, gated;
+  float alpha, limit, slimit;
+};
+constexpr int GU = 4;         // 256-element steps in flight per weight row
+
+__global__ void __launch_bounds__(256) moe_gemv_kernel(GemvArgs a) {
+  extern __shared__ __align__(16) uint8_t raw[];
+  __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(raw);
+  pdl_launch_dependents();
+  pdl_wait();
+  const int job = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool sh = job >= a.pairs;
+  const int row = sh ? job - a.pairs : job / a.top, M = sh ? a.SM : a.M, K = sh ? a.SK : a.K, words = K / 8;
+  const __nv_bfloat16* w = sh ? a.sw : a.w + (size_t)a.ids[job] * (a.gated ? 2 : 1) * M * K;
+  const __nv_bfloat16* x = a.gated ? (sh ? a.sx : a.x) + (size_t)row * K : (sh ? a.sx + (size_t)row * K : a.x + (size_t)job * K);
+  __nv_bfloat16* out = a.gated ? (sh ? a.sout + (size_t)row * M : a.out + (size_t)job * M)
+                               : a.out + ((size_t)row * a.slots + (sh ? a.top : job % a.top)) * M;
+  const int outs = a.gated ? M : (M + 1) / 2, stride = gridDim.x * 8;
+  uint4 c0[GU], c1[GU];
+  auto fetch = [&](int o, int b) {
+    const int r0 = a.gated ? o : 2 * o, r1 = a.gated ? o + M : 2 * o + 1;
+    const uint4 *w0 = reinterpret_cast<const uint4*>(w + (size_t)r0 * K), *w1 = reinterpret_cast<const uint4*>(w + (size_t)r1 * K);
+    const bool v = o < outs, v1 = v && (a.gated || r1 < M);
+#pragma unroll
+    for (int i = 0; i < GU; ++i) {
+      const int k = (b * GU + i) * 32 + lane;
+      c0[i] = v && k < words ? ldg_nc(w0 + k) : make_uint4(0u, 0u, 0u, 0u);
+      c1[i] = v1 && k < words ? ldg_nc(w1 + k) : make_uint4(0u, 0u, 0u, 0u);
+    }
+  };
+  int o = blockIdx.x * 8 + warp;
+  fetch(o, 0);
+  for (int i = threadIdx.x; i < words; i += 256) reinterpret_cast<uint4*>(xs)[i] = reinterpret_cast<const uint4*>(x)[i];
+  __syncthreads();
+  const int batches = (words + 32 * GU - 1) / (32 * GU);
+  for (; o < outs; o += stride) {
+    float s0 = 0.f, s1 = 0.f;
+    for (int b = 0; b < batches; ++b) {
+      uint4 d0[GU], d1[GU];
+#pragma unroll
+      for (int i = 0; i < GU; ++i) { d0[i] = c0[i]; d1[i] = c1[i]; }
+      if (b + 1 < batches) fetch(o, b + 1);
+      else fetch(o + stride, 0);
+#pragma unroll
+      for (int i = 0; i < GU; ++i) {
+        const int k = (b * GU + i) * 32 + lane;
+        if (k >= words) continue;
+        const uint4 xv = reinterpret_cast<const uint4*>(xs)[k];
+        const uint32_t xw[4] = {xv.x, xv.y, xv.z, xv.w}, p[4] = {d0[i].x, d0[i].y, d0[i].z, d0[i].w}, q[4] = {d1[i].x, d1[i].y, d1[i].z, d1[i].w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float x0 = __uint_as_float(xw[j] << 16), x1 = __uint_as_float(xw[j] & 0xffff0000u);
+          s0 = fmaf(__uint_as_float(p[j] << 16), x0, s0);
+          s0 = fmaf(__uint_as_float(p[j] & 0xffff0000u), x1, s0);
+          s1 = fmaf(__uint_as_float(q[j] << 16), x0, s1);
+          s1 = fmaf(__uint_as_float(q[j] & 0xffff0000u), x1, s1);
+        }
+      }
+    }
+    s0 = warp_sum(s0);
+    s1 = warp_sum(s1);
+    if (lane == 0) {
+      if (a.gated) out[o] = __float2bfloat16_rn(gate_clamp<float>(s0, s1, a.alpha, sh ? a.slimit : a.limit));
+      else {
+        out[2 * o] = __float2bfloat16_rn(s0);
+        if (2 * o + 1 < M) out[2 * o + 1] = __float2bfloat16_rn(s1);
+      }
+    }
+  }
+}
+
+}  // namespace rmoe
+}  // namespace sfb
+
+using namespace sfb;
+using namespace sfb::rmoe;
+
+extern "C" {
+
+int sfb_rows_moe_route(const void* z, int64_t ld, void* ids, void* wts, int n, int E, int top, int shared, cudaStream_t stream) {
+  if (n < 1 || E < 1 || E > MAX_E || top < 1 || top > MAX_TOP || top > E) return (int)cudaErrorInvalidValue;
+  RouteArgs a{(const float*)z, ld, (int*)ids, (float*)wts, n, E, top, shared};
+  return (int)sfb_launch(moe_route_kernel, dim3((n + 7) / 8), dim3(256), 0, stream, a);
+}
+
+// tiles: 4 ints each, at most pairs / tile + min(E, pairs) of them
+int sfb_rows_moe_plan(const void* ids, void* order, void* tiles, void* count, int pairs, int E, int tile, cudaStream_t stream) {
+  if (pairs < 1 || E < 1 || E > MAX_E || tile < 1) return (int)cudaErrorInvalidValue;
+  PlanArgs a{(const int*)ids, (int*)order, (int*)tiles, (int*)count, pairs, E, tile};
+  return (int)sfb_launch(moe_plan_kernel, dim3(1), dim3(1024), 0, stream, a);
+}
+
+// tiles of at most 32 pairs
+int sfb_rows_moe_tile(const void* x, const void* w, void* out, const void* order, const void* tiles, const void* count, int max_tiles, int M, int K, int top,
+                      int slots, int gated, float alpha, float limit, int fp32, cudaStream_t stream) {
+  if (max_tiles < 1 || max_tiles > 65535 || M < 1 || K < 1) return (int)cudaErrorInvalidValue;
+  TileArgs a{x, w, out, (const int*)order, (const int*)tiles, (const int*)count, M, K, top, slots, gated, alpha, limit};
+  const dim3 g((M + TC - 1) / TC, max_tiles), b(256);
+  return (int)(fp32 ? sfb_launch(moe_tile_kernel<float>, g, b, 0, stream, a) : sfb_launch(moe_tile_kernel<__nv_bfloat16>, g, b, 0, stream, a));
+}
+
+// bf16, K and SK multiples of 8
+int sfb_rows_moe_gemv(const void* ids, const void* x, const void* w, void* out, const void* sx, const void* sw, void* sout, int pairs, int n, int M, int K, int SM,
+                      int SK, int top, int slots, int gated, float alpha, float limit, float slimit, cudaStream_t stream) {
+  const int kmax = sw && SK > K ? SK : K;
+  if (n < 1 || pairs != n * top || pairs + n > 65535 || M < 1 || K < 8 || K % 8 || (sw && (SM < 1 || SK < 8 || SK % 8)) || kmax * 2 > 200 * 1024)
+    return (int)cudaErrorInvalidValue;
+  GemvArgs a{(const int*)ids, (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, (const __nv_bfloat16*)sx, (const __nv_bfloat16*)sw,
+             (__nv_bfloat16*)sout, pairs, n, M, K, SM, SK, top, slots, gated, alpha, limit, slimit};
+  const int jobs = pairs + (sw ? n : 0), big = sw && SM > M ? SM : M, outs = gated ? big : (big + 1) / 2;
+  int bx = (outs + 7) / 8, cap = (148 * 4 + jobs - 1) / jobs;
+  if (bx > cap) bx = cap;
+  static size_t granted = 40 * 1024;
+  const size_t smem = (size_t)kmax * 2;
+  if (smem > granted) {
+    const cudaError_t e = cudaFuncSetAttribute(moe_gemv_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    granted = smem;
+  }
+  return (int)sfb_launch(moe_gemv_kernel, dim3(bx, jobs), dim3(256), smem, stream, a);
+}
+
+}  // extern "C"

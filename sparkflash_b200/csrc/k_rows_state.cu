@@ -1,9 +1,13 @@
-// Linear recurrence with a matrix state and one decay per head (models/mixers.py: state-space duality, retention):
+// Linear recurrence with a matrix state and one decay per head (models/mixers.py: state-space duality, retention, delta rule):
 //
 //   S_t = a_t S_(t-1) + w_t k_t v_t^T,   y_t = S_t^T q_t + D v_t        S: N x P per head, 32-bit
 //
 // a_t = exp(A dt_t), w_t = dt_t with dt_t = softplus(raw_t + bias) per token and head, or a_t a constant of the head and w_t = 1.
 // q and k belong to groups of heads; they may be turned by their position (rotate-half layout) and k scaled.
+//
+// Delta rule: q and k are unit vectors (q scaled), and what is written is what the state does not yet say about k:
+//
+//   S = a_t S_(t-1),   u_t = b_t (v_t - S^T k_t),   S_t = S + k_t u_t^T,   y_t = S_t^T q_t        b_t = sigmoid(raw_t)
 //
 //   state_rows    one block per (segment, head, tile of P): the state stays in registers while the segment's rows go by.  Any
 //                 sizes, bf16 or 32-bit; decode steps and short runs.  Steps of single rows also apply the causal convolution
@@ -24,6 +28,8 @@ struct StateArgs {
   const float* dt_bias;             // [H]
   const float* a;                   // [H]: A with dt, else the decay itself
   const float* D;                   // [H] or null
+  const void* beta;                 // (T) [n, beta_stride] raw write strengths: delta rule; or null
+  int64_t beta_stride;
   const float2* rot;                // [positions, rot_dims / 2] (cos, sin) or null
   const int* row_pos;
   void* y;                          // [n, H P] (T)
@@ -33,7 +39,7 @@ struct StateArgs {
   const int *segs, *seg_row0, *seg_len, *seg_src, *seg_dst;      // segs: segment of every blockIdx.y, or null: identity
   int rot_dims, taps, C, q_ch, k_ch, v_ch;                       // *_ch: first convolution channel of q, k, v
   int H, G, N, P, Np;
-  float k_scale;
+  float k_scale, q_scale, unit_eps; // q_scale, unit_eps: of the delta rule's unit vectors
 };
 constexpr int STB = 8;              // rows whose q, k, v are staged together
 
@@ -46,7 +52,7 @@ __device__ __forceinline__ float conv_silu(const StateArgs& a, T x, int ch, int 
   const int W = a.taps - 1;
   const T* hs = (const T*)a.hist + (size_t)(src >= 0 ? src : 0) * W * a.C + ch;
   T* hd = (T*)a.hist + (size_t)dst * W * a.C + ch;
-  float acc = a.cb[ch] + a.cw[(size_t)W * a.C + ch] * to_f<T>(x);
+  float acc = (a.cb ? a.cb[ch] : 0.f) + a.cw[(size_t)W * a.C + ch] * to_f<T>(x);
   for (int j0 = 0; j0 < W; j0 += ST_TAPS) {
     T gv[ST_TAPS];
     float w[ST_TAPS];
@@ -65,8 +71,8 @@ __device__ __forceinline__ float conv_silu(const StateArgs& a, T x, int ch, int 
   return to_f<T>(from_f<T>(acc * sigmoid_f(acc)));
 }
 
-template <typename T, int NI>
-__global__ void __launch_bounds__(256, NI <= 4 ? 5 : NI <= 8 ? 3 : 1) state_rows_kernel(StateArgs a) {
+template <typename T, int NI, bool DELTA>
+__global__ void __launch_bounds__(256, NI <= 4 ? (DELTA ? 4 : 5) : NI <= 8 ? 3 : 1) state_rows_kernel(StateArgs a) {
   extern __shared__ __align__(16) float sm[];
   const int PT = blockDim.x >> 3, tiles = (a.P + PT - 1) / PT;
   const int h = blockIdx.x / tiles, tile = blockIdx.x % tiles, g = h / (a.H / a.G);
@@ -75,7 +81,9 @@ __global__ void __launch_bounds__(256, NI <= 4 ? 5 : NI <= 8 ? 3 : 1) state_rows
   float* ks = qs + STB * a.Np;
   float* vs = ks + STB * a.Np;        // [STB][PT]
   float* av = vs + STB * PT;          // [STB] decay
-  float* wv = av + STB;               // [STB] input scale
+  float* wv = av + STB;               // [STB] input scale (delta rule: write strength)
+  float* qr = wv + STB;               // [STB], [STB] delta rule: factors that make q and k unit vectors
+  float* kr = qr + STB;
   pdl_launch_dependents();
   pdl_wait();
   const int seg = a.segs ? a.segs[blockIdx.y] : blockIdx.y;
@@ -133,14 +141,38 @@ __global__ void __launch_bounds__(256, NI <= 4 ? 5 : NI <= 8 ? 3 : 1) state_rows
     if (tid < nb) {
       if (a.dt) {
         const float dt = softplus_f(to_f<T>(((const T*)a.dt)[(size_t)(row0 + t0 + tid) * a.dt_stride + h]) + a.dt_bias[h]);
-        av[tid] = expf(a.a[h] * dt); wv[tid] = dt;
+        av[tid] = expf(a.a[h] * dt);
+        wv[tid] = DELTA ? sigmoid_f(to_f<T>(((const T*)a.beta)[(size_t)(row0 + t0 + tid) * a.beta_stride + h])) : dt;
       } else {
         av[tid] = a.a[h]; wv[tid] = 1.f;
       }
     }
     __syncthreads();
+    if constexpr (DELTA) {
+      for (int x = tid >> 5; x < 2 * nb; x += blockDim.x >> 5) {
+        const float* p0 = (x & 1 ? ks : qs) + (x >> 1) * a.Np;
+        float s = 0.f;
+        for (int n = tid & 31; n < a.Np; n += 32) s = fmaf(p0[n], p0[n], s);
+        s = warp_sum(s);
+        if ((tid & 31) == 0) (x & 1 ? kr : qr)[x >> 1] = (x & 1 ? 1.f : a.q_scale) / sqrtf(s + a.unit_eps);
+      }
+      __syncthreads();
+    }
     for (int t = 0; t < nb; ++t) {
-      const float dec = av[t], v = vs[t * PT + pl], in = v * wv[t];
+      const float dec = av[t], v = vs[t * PT + pl];
+      float in = v * wv[t];
+      if constexpr (DELTA) {              // what the decayed state says about k
+        float m = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+          const float4 kk = *reinterpret_cast<const float4*>(ks + t * a.Np + i * 32 + ng * 4);
+          m = fmaf(S[i].x, kk.x, m); m = fmaf(S[i].y, kk.y, m); m = fmaf(S[i].z, kk.z, m); m = fmaf(S[i].w, kk.w, m);
+        }
+        m += __shfl_xor_sync(0xffffffffu, m, 1);
+        m += __shfl_xor_sync(0xffffffffu, m, 2);
+        m += __shfl_xor_sync(0xffffffffu, m, 4);
+        in = wv[t] * (v - dec * kr[t] * m) * kr[t];
+      }
       float y = 0.f;
 #pragma unroll
       for (int i = 0; i < NI; ++i) {
@@ -153,6 +185,7 @@ __global__ void __launch_bounds__(256, NI <= 4 ? 5 : NI <= 8 ? 3 : 1) state_rows
       y += __shfl_xor_sync(0xffffffffu, y, 1);
       y += __shfl_xor_sync(0xffffffffu, y, 2);
       y += __shfl_xor_sync(0xffffffffu, y, 4);
+      if constexpr (DELTA) y *= qr[t];
       if (ng == 0 && on) ((T*)a.y)[((size_t)(row0 + t0 + t) * a.H + h) * a.P + p] = from_f<T>(fmaf(D, v, y));
     }
   }
@@ -218,12 +251,12 @@ __global__ void __launch_bounds__(256) gated_norm_kernel(GatedNormArgs a) {
   }
 }
 
-template <typename T>
+template <typename T, bool DELTA>
 static int launch_state(const StateArgs& a, int segs, cudaStream_t st) {
   const int threads = a.P > 16 ? 256 : 128, PT = threads / 8, tiles = (a.P + PT - 1) / PT;
   const dim3 g(a.H * tiles, segs), b(threads);
-  const size_t smem = ((size_t)2 * STB * a.Np + STB * PT + 2 * STB) * sizeof(float);
-#define SFB_STATE(NI) case NI: return (int)sfb_launch(state_rows_kernel<T, NI>, g, b, smem, st, a)
+  const size_t smem = ((size_t)2 * STB * a.Np + STB * PT + 4 * STB) * sizeof(float);
+#define SFB_STATE(NI) case NI: return (int)sfb_launch(state_rows_kernel<T, NI, DELTA>, g, b, smem, st, a)
   switch (a.Np / 32) {
     SFB_STATE(1); SFB_STATE(2); SFB_STATE(3); SFB_STATE(4); SFB_STATE(5); SFB_STATE(6); SFB_STATE(7); SFB_STATE(8);
     SFB_STATE(12); SFB_STATE(16);
@@ -261,16 +294,17 @@ extern "C" {
 
 // Np: N rounded up to 32 (up to 256), then 384 or 512.  cw: every segment of the launch is one row and q, k, v are the convolution's inputs.
 int sfb_rows_state(const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v, int64_t v_stride, const void* dt, int64_t dt_stride,
-                   const void* dt_bias, const void* a, const void* D, const void* rot, const int* row_pos, void* y, void* S, const void* cw,
+                   const void* dt_bias, const void* a, const void* D, const void* beta, int64_t beta_stride, const void* rot, const int* row_pos, void* y, void* S, const void* cw,
                    const void* cb, void* hist, const int* segs, const int* seg_row0, const int* seg_len, const int* seg_src, const int* seg_dst,
                    int n_segs, int rot_dims, int taps, int C, int q_ch, int k_ch, int v_ch, int H, int G, int N, int P, int Np, float k_scale,
-                   int fp32, cudaStream_t stream) {
-  if (n_segs < 1 || n_segs > 65535 || G < 1 || H % G || N < 1 || P < 1 || Np % 32 || Np < N || (rot_dims && (!rot || rot_dims > N || rot_dims % 2)))
+                   float q_scale, float unit_eps, int fp32, cudaStream_t stream) {
+  if (n_segs < 1 || n_segs > 65535 || G < 1 || H % G || (beta && (!dt || rot || D || k_scale != 1.f)) || N < 1 || P < 1 || Np % 32 || Np < N || (rot_dims && (!rot || rot_dims > N || rot_dims % 2)))
     return (int)cudaErrorInvalidValue;
-  StateArgs s{q, k, v, q_stride, k_stride, v_stride, dt, dt_stride, (const float*)dt_bias, (const float*)a, (const float*)D, (const float2*)rot, row_pos, y,
+  StateArgs s{q, k, v, q_stride, k_stride, v_stride, dt, dt_stride, (const float*)dt_bias, (const float*)a, (const float*)D, beta, beta_stride, (const float2*)rot, row_pos, y,
               (float*)S, (const float*)cw, (const float*)cb, hist, segs, seg_row0, seg_len, seg_src, seg_dst, rot_dims, taps, C, q_ch, k_ch, v_ch,
-              H, G, N, P, Np, k_scale};
-  return fp32 ? launch_state<float>(s, n_segs, stream) : launch_state<__nv_bfloat16>(s, n_segs, stream);
+              H, G, N, P, Np, k_scale, q_scale, unit_eps};
+  if (beta) return fp32 ? launch_state<float, true>(s, n_segs, stream) : launch_state<__nv_bfloat16, true>(s, n_segs, stream);
+  return fp32 ? launch_state<float, false>(s, n_segs, stream) : launch_state<__nv_bfloat16, false>(s, n_segs, stream);
 }
 
 int sfb_rows_gated_norm(const void* y, const void* gate, int64_t gate_stride, const void* w, void* out, int n, int width, int part, int before, float eps,

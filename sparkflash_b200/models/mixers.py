@@ -1,12 +1,15 @@
-"""Sublayers of the layered decoders (models/layered.py): attention with a distance bias, the real-gated linear recurrence, two
-mixers side by side, matrix-state recurrences (state-space duality, retention), latent attention in a window, and the dense gated
-feed-forward.  Each takes its sizes and constants as arguments, reads its weights by
+"""Sublayers of the layered decoders (models/layered.py): attention with a distance bias, attention with rotated keys in a window (sinks,
+capped scores, values mixed across layers), the real-gated linear recurrence, two mixers side by side, matrix-state recurrences
+(state-space duality, retention, the gated delta rule), latent attention in a window, the dense gated feed-forward, the mixture of
+experts, and the per-layer token input.  Each takes its sizes and constants as arguments, reads its weights by
 name, keeps its caches in the engine's page pool or state slots, and runs on a step's rows through the kernels of ops/rows.py.
 
 A sublayer is built once per layer (``weights``) and bound once per run of the layer (``bind_run``): a looped layer shares its
 weights between passes, every pass has its own keys, values and states.
 """
 from __future__ import annotations
+
+import math
 
 import torch
 import torch.nn.functional as F
@@ -37,9 +40,9 @@ class W:
     def f32(self, name: str) -> torch.Tensor:
         return self.t[self.p + name].to(self.device, torch.float32).contiguous()
 
-    def taps(self, name: str) -> torch.Tensor:
-        """Convolution weights [channels, taps] as the kernels read them: [taps, channels], 32-bit."""
-        return self.t[self.p + name].to(self.device, torch.float32).t().contiguous()
+    def taps(self, *names: str) -> torch.Tensor:
+        """Convolution weights [channels, taps], stacked, as the kernels read them: [taps, channels], 32-bit."""
+        return torch.cat([self.t[self.p + n] for n in names], 0).to(self.device, torch.float32).t().contiguous()
 
 
 def log_distance_bias(r1: torch.Tensor, r2: torch.Tensor, length: int, device) -> torch.Tensor:
@@ -48,24 +51,25 @@ def log_distance_bias(r1: torch.Tensor, r2: torch.Tensor, length: int, device) -
     return (r1.to(device, torch.float64)[:, None] * torch.log1p(r2.to(device, torch.float64)[:, None] * d)).to(torch.float32).contiguous()
 
 
-class BiasedAttention:
-    """Grouped-query attention over the paged cache: RMS norm over the whole query and key projections, no rotation, a distance
-    bias taken off the scaled score.  Reads its q | k | v columns out of the layer's stacked projection."""
-
-    def __init__(self, w: W, spec: dict, eps: float, max_context: int):
-        self.H, self.G, self.dim, self.vdim = spec["heads"], spec["kv_heads"], spec["dim"], spec["vdim"]
-        self.scale, self.eps = float(spec["scale"]), eps
-        self.cols = self.H * self.dim + self.G * (self.dim + self.vdim)
-        self.q_norm, self.k_norm = w.f32("q.norm"), w.f32("k.norm")
-        self.bias = log_distance_bias(w.f32("r1"), w.f32("r2"), max_context, w.device)
-        self.wo, self.bo = w.act("o"), w.act("o.b")
-        self.tc = R.attn_tc_supports(self.wo.dtype, self.dim, self.vdim)
-        self.stream = R.attn_stream_supports(self.wo.dtype, self.dim, self.vdim)
+class PagedAttention:
+    """Grouped-query softmax attention over the paged cache: the rows of a step go to the arm that suits them.  ``bias`` [heads, distance]
+    is taken off the scaled score, ``cap`` bounds it, a position sees the last ``window`` ones, ``sink`` [heads] joins the denominator."""
 
     PROJ, PROJ_BIAS = ("q", "k", "v"), ("q.b", "k.b", "v.b")
+    bias: torch.Tensor | None = None
+    sink: torch.Tensor | None = None
+    window, cap = R.NO_WINDOW, 0.0
+
+    def __init__(self, w: W, spec: dict):
+        self.H, self.G, self.dim, self.vdim = spec["heads"], spec["kv_heads"], spec["dim"], spec["vdim"]
+        self.scale = float(spec["scale"])
+        self.cols = self.H * self.dim + self.G * (self.dim + self.vdim)
+        self.tc = R.attn_tc_supports(w.dtype, self.dim, self.vdim)
+        self.stream = R.attn_stream_supports(w.dtype, self.dim, self.vdim)
+        self.dtype = w.dtype
 
     def reserve(self, e) -> None:
-        n, dt = e.max_rows, self.wo.dtype
+        n, dt = e.max_rows, self.dtype
         e.scratch.reserve("attn_q", n * self.H * self.dim, dt)
         e.scratch.reserve("attn_o", n * self.H * self.vdim, dt)
         # partial outputs of split rows: rows x heads x ranges, bounded by the blocks of one launch (see LayeredEngine.splits)
@@ -76,23 +80,41 @@ class BiasedAttention:
         e.scratch.reserve("attn_part", parts * self.vdim, torch.float32)
         e.scratch.reserve("attn_ml", parts * 2, torch.float32)
 
-    def run(self, s, proj, kv, out):
-        """proj [n, >= cols] view whose first columns are q | k | v; kv = (k pool, v pool) of this run."""
-        n, k, v = s.n, kv[0], kv[1]
-        q = s.scratch.get("attn_q", n, self.H * self.dim)
-        o = s.scratch.get("attn_o", n, self.H * self.vdim)
-        R.qk_append(proj, self.q_norm, self.k_norm, q, k, v, s.table, s.row_lane, s.row_pos, n, self.H, self.eps, s.status)
+    def attend(self, s, q, kv, o) -> None:
+        """q [n, H dim] against this run's pools, whose rows of the step have been appended; kv from R.attn_pools."""
+        k, v, opts = kv[0], kv[1], dict(window=self.window, sink=self.sink, cap=self.cap)
         if s.ntiles:
-            R.attn_tc(q, kv, s.table, s.row_lane, s.row_pos, s.tiles, s.ntiles, self.bias, o, self.H, self.scale, s.status)
+            R.attn_tc(q, kv, s.table, s.row_lane, s.row_pos, s.tiles, s.ntiles, self.bias, o, self.H, self.scale, s.status, **opts)
         if s.short and self.stream and s.short <= R.STREAM_ROWS:
+            pages = min(s.pages, (self.window + R.PAGE - 2) // R.PAGE + 1)
             R.attn_stream(q, k, v, s.table, s.row_lane, s.row_pos, s.short_rows, s.short, self.bias, o, s.scratch.buf["attn_part"],
-                          s.scratch.buf["attn_ml"], self.H, self.scale, s.short * s.pages, s.status)
+                          s.scratch.buf["attn_ml"], self.H, self.scale, s.short * pages, s.status, **opts)
         elif s.short:
             blocks = R.attn_blocks(self.H, self.G)
-            sp = s.engine.splits(s, s.short, blocks)
+            sp = s.engine.splits(s, s.short, blocks, self.window)
             part = s.scratch.buf["attn_part"] if sp > 1 else None
             ml = s.scratch.buf["attn_ml"] if sp > 1 else None
-            R.attn(q, k, v, s.table, s.row_lane, s.row_pos, s.short_rows, s.short, self.bias, o, part, ml, self.H, self.scale, sp, s.status)
+            R.attn(q, k, v, s.table, s.row_lane, s.row_pos, s.short_rows, s.short, self.bias, o, part, ml, self.H, self.scale, sp, s.status, **opts)
+
+
+class BiasedAttention(PagedAttention):
+    """RMS norm over the whole query and key projections, no rotation, a distance bias taken off the scaled score.  Reads its q | k | v
+    columns out of the layer's stacked projection."""
+
+    def __init__(self, w: W, spec: dict, eps: float, max_context: int):
+        super().__init__(w, spec)
+        self.eps = eps
+        self.q_norm, self.k_norm = w.f32("q.norm"), w.f32("k.norm")
+        self.bias = log_distance_bias(w.f32("r1"), w.f32("r2"), max_context, w.device)
+        self.wo, self.bo = w.act("o"), w.act("o.b")
+
+    def run(self, s, proj, kv, out):
+        """proj [n, >= cols] view whose first columns are q | k | v; kv = (k pool, v pool) of this run."""
+        n = s.n
+        q = s.scratch.get("attn_q", n, self.H * self.dim)
+        o = s.scratch.get("attn_o", n, self.H * self.vdim)
+        R.qk_append(proj, self.q_norm, self.k_norm, q, kv[0], kv[1], s.table, s.row_lane, s.row_pos, n, self.H, self.eps, s.status)
+        self.attend(s, q, kv, o)
         return R.linear(o, self.wo, self.bo, out)
 
 
@@ -188,11 +210,79 @@ class ParallelMixer:
         return y, y2
 
 
-def rotation_table(base: float, dims: int, length: int, device) -> torch.Tensor:
-    """[length, dims / 2, 2]: cosine and sine of p base^(-2 i / dims), evaluated in 64-bit and rounded once."""
-    f = torch.tensor([base ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64)
-    a = torch.arange(length, dtype=torch.float64)[:, None] * f
-    return torch.stack([a.cos(), a.sin()], -1).to(torch.float32).to(device).contiguous()
+def rotation_frequencies(base: float, dims: int, scaling: dict | None = None) -> tuple[list[float], float]:
+    """Radians per position of every pair, and a factor on cosine and sine.  ``scaling``: None; {factor, low, high, original}: a pair keeps its
+    frequency where the original context holds more than ``high`` of its wavelengths, has it divided by ``factor`` where it holds less than
+    ``low``, and a blend in between; {factor, original, fast, slow}: YaRN (Peng et al., "YaRN: Efficient Context Window Extension of Large Language
+    Models"), the division comes in along a ramp over the pairs between those that turn ``fast`` and ``slow`` times in the original context."""
+    f = [base ** (-2.0 * i / dims) for i in range(dims // 2)]
+    if scaling is None:
+        return f, 1.0
+    factor, original = float(scaling["factor"]), float(scaling["original"])
+    if "fast" in scaling:
+        pair = lambda turns: dims * math.log(original / (2 * math.pi * turns)) / (2 * math.log(base))
+        first, last = max(math.floor(pair(scaling["fast"])), 0), min(math.ceil(pair(scaling["slow"])), dims - 1)
+        share = [min(max((i - first) / max(last - first, 0.001), 0.0), 1.0) for i in range(len(f))]
+        return [x * (1 - r) + x / factor * r for x, r in zip(f, share)], 0.1 * math.log(factor) + 1.0
+    out = []
+    for x in f:
+        turns = original * x / (2 * math.pi)          # wavelengths in the original context
+        kept = 1.0 if turns > scaling["high"] else 0.0 if turns < scaling["low"] else (turns - scaling["low"]) / (scaling["high"] - scaling["low"])
+        out.append(kept * x + (1 - kept) * x / factor)
+    return out, 1.0
+
+
+def rotation_table(base: float, dims: int, length: int, device, scaling: dict | None = None) -> torch.Tensor:
+    """[length, dims / 2, 2]: cosine and sine of position times frequency, evaluated in 64-bit and rounded once."""
+    f, gain = rotation_frequencies(base, dims, scaling)
+    a = torch.arange(length, dtype=torch.float64)[:, None] * torch.tensor(f, dtype=torch.float64)
+    return (torch.stack([a.cos(), a.sin()], -1) * gain).to(torch.float32).to(device).contiguous()
+
+
+class ValueMix:
+    """Values that the layers of a model share within a step: the first layer that takes part leaves its own, the others mix theirs with them."""
+
+    def __init__(self, cols: int):
+        self.cols, self.layers = cols, 0
+
+    def reserve(self, e, dtype) -> None:
+        e.scratch.reserve("v_first", e.max_rows * self.cols, dtype)
+
+
+class RotaryAttention(PagedAttention):
+    """Rotated queries and keys (the first ``rot`` dims of a head, rotate-half layout, scaled frequencies), a sliding window, a learned sink per
+    head, optionally capped scores, and values mixed with another layer's (``mix``) ahead of the cache.  A layer's only mixer."""
+
+    def __init__(self, w: W, spec: dict, max_context: int, mix: ValueMix | None = None):
+        super().__init__(w, spec)
+        rot = spec["rot"]
+        self.window, self.cap = min(int(spec["mask"]["size"]), max_context), float(spec.get("softcap") or 0.0)
+        self.dims, self.cs = rot["dims"], rotation_table(rot["base"], rot["dims"], max_context, w.device, rot.get("scaling"))
+        self.sink = w.f32("sink")
+        self.w_in, self.b_in, self.wo = w.act(*self.PROJ), w.act(*self.PROJ_BIAS), w.act("o")
+        self.mix, self.lam = mix, None
+        if mix is not None:
+            self.lam = w.f32("vmix") if mix.layers else None        # the first such layer has nothing to mix with
+            mix.layers += 1
+        self.merge, self.kv_run = (None, None), (self.G, self.dim, self.vdim)
+
+    def reserve(self, e) -> None:
+        super().reserve(e)
+        e.scratch.reserve("proj", e.max_rows * self.w_in.shape[0], self.dtype)
+        if self.mix is not None:
+            self.mix.reserve(e, self.dtype)
+
+    def bind_run(self, e, tag: str, kv_index):
+        return {"kv": R.attn_pools(e.kv, kv_index, self.tc)}
+
+    def run(self, s, h, run):
+        n, kv = s.n, run["kv"]
+        proj = R.linear(h, self.w_in, self.b_in, s.scratch.get("proj", n, self.w_in.shape[0]))
+        q, o = s.scratch.get("attn_q", n, self.H * self.dim), s.scratch.get("attn_o", n, self.H * self.vdim)
+        first = s.scratch.get("v_first", n, self.mix.cols) if self.mix is not None else None
+        R.rot_append(proj, self.cs, self.dims, q, kv[0], kv[1], first, self.lam, s.table, s.row_lane, s.row_pos, n, self.H, s.status)
+        self.attend(s, q, kv, o)
+        return R.linear(o, self.wo, None, s.scratch.get("y", n, h.shape[1])), None
 
 
 class MatrixState:
@@ -312,6 +402,63 @@ class RetentionMixer:
         return R.linear(o, self.w_out, None, s.scratch.get("y", n, h.shape[1])), None
 
 
+class DeltaState(MatrixState):
+    """The gated delta rule (Yang et al., "Gated Delta Networks: Improving Mamba2 with Delta Rule"): S = a_t S_(t-1), u_t = b_t (v_t - S^T k_t),
+    S_t = S + k_t u_t^T, y_t = S_t^T q_t, with unit vectors q and k (q over the root of its length), a_t = exp(A softplus(.)), b_t = sigmoid(.)."""
+
+    UNIT_EPS = 1e-6
+
+    def __init__(self, heads: int, groups: int, n: int, p: int, decay: torch.Tensor, dtype: torch.dtype, dt_bias):
+        super().__init__(heads, groups, n, p, decay, dtype, dt_bias)
+        self.tc = False
+
+    def run(self, s, src, cols, dt, beta, S, y, conv=None) -> None:
+        q, k, v = (src[:, c:] for c in cols)
+        R.state_rows(q, k, v, dt, self.dt_bias, self.decay, None, None, 0, 1.0, s.row_pos, y, S, self.N, self.G, s.short_segs, s.nshort, s, conv,
+                     beta, self.N ** -0.5, self.UNIT_EPS)
+
+
+class DeltaMixer:
+    """q | k | v through a causal convolution and silu, the gated delta rule, every head's output over its RMS times a weight that the heads
+    share, silu(W_g h) gate, W_o."""
+
+    PROJ = ("q", "k", "v", "g", "b", "a")
+
+    def __init__(self, w: W, spec: dict, eps: float):
+        H, G, N, P = spec["heads"], spec["kv_heads"], spec["dim"], spec["vdim"]
+        self.H, self.P, self.qk, self.inner, self.taps, self.eps = H, P, G * N, H * P, spec["conv"], eps
+        self.channels = 2 * self.qk + self.inner
+        self.w_in, self.w_out = w.act(*self.PROJ, pad=8), w.act("o")
+        self.cw, self.norm = w.taps("q.conv", "k.conv", "v.conv"), w.f32("norm").repeat(H).contiguous()
+        A = -torch.exp(w.t[w.p + "A_log"].to(w.device, torch.float64)).to(torch.float32)
+        self.core = DeltaState(H, G, N, P, A.contiguous(), w.dtype, w.f32("dt_bias"))
+        self.merge, self.kv_run = (None, None), None
+
+    def reserve(self, e) -> None:
+        n, dt = e.max_rows, self.w_in.dtype
+        e.scratch.reserve("proj", n * self.w_in.shape[0], dt)
+        e.scratch.reserve("mix_u", n * self.channels, dt)
+        e.scratch.reserve("mix_y", n * self.inner, dt)
+        e.scratch.reserve("mix_o", n * self.inner, dt)
+        self.core.reserve(e)
+
+    def bind_run(self, e, tag: str, kv_index):
+        return {"conv": e.state.add(tag + ".conv", (self.taps - 1, self.channels), self.w_in.dtype), "S": self.core.state(e, tag + ".S")}
+
+    def run(self, s, h, run):
+        n, c, i = s.n, self.channels, self.inner
+        proj = R.linear(h, self.w_in, None, s.scratch.get("proj", n, self.w_in.shape[0]))
+        u, gate, beta, dt = proj[:, :c], proj[:, c:c + i], proj[:, c + i:], proj[:, c + i + self.H:]
+        y, o, cols = s.scratch.get("mix_y", n, i), s.scratch.get("mix_o", n, i), (0, self.qk, 2 * self.qk)
+        conv = (self.cw, None, run["conv"], cols) if s.single and n <= CONV_STEP_ROWS else None
+        if conv is None:
+            raw, u = u, s.scratch.get("mix_u", n, c)
+            R.conv(raw, self.cw, None, u, run["conv"], s, n, R.CONV_SILU)
+        self.core.run(s, u, cols, dt, beta, run["S"], y, conv)
+        R.gated_norm(y, gate, self.norm, o, self.P, False, self.eps)
+        return R.linear(o, self.w_out, None, s.scratch.get("y", n, h.shape[1])), None
+
+
 class LatentAttention:
     """Attention whose keys and values are products of one cached vector per token (DeepSeek-AI, "DeepSeek-V2: A Strong, Economical, and
     Efficient Mixture-of-Experts Language Model"): the RMS-normed latent c, beside one rotated key part that the heads share.  A
@@ -406,3 +553,76 @@ class DenseFF:
     def run(self, s, h):
         act = R.gated_linear(h, self.w_in, s.scratch.get("proj", s.n, 2 * self.ff), s.scratch.get("ff_act", s.n, self.ff), self.act)
         return R.linear(act, self.w_out, None, s.scratch.get("y", s.n, h.shape[1]))
+
+
+class MixtureFF:
+    """Every row through ``top`` of ``experts`` small feed-forwards, weighted by the softmax over their router logits, and through a shared one,
+    weighted by the sigmoid of a logit of its own.  An expert: W_down (g sigmoid(alpha g) (u + 1)), g = min(W_gate h, limit), u = W_up h within
+    +-limit.  ``run`` returns the parts [n, top + shared, width] and their weights; the seam adds them up."""
+
+    def __init__(self, w: W, spec: dict, alpha: float):
+        self.E, self.top = spec["router"]["experts"], spec["router"]["top"]
+        self.ff, self.limit, self.alpha = spec["expert"]["ff"], float(spec["expert"]["limit"]), alpha
+        sh = spec.get("shared")
+        self.shared, self.shared_ff, self.shared_limit = int(sh is not None), sh["ff"] if sh else 0, float(sh["limit"]) if sh else 0.0
+        self.slots = self.top + self.shared
+        self.w_in = torch.stack([w.act(f"e{i}.gate", f"e{i}.up") for i in range(self.E)]).contiguous()        # [E, 2 ff, width]
+        self.w_out = torch.stack([w.act(f"e{i}.down") for i in range(self.E)]).contiguous()                   # [E, width, ff]
+        self.router = w.act("router", *(["shared.sg"] if sh else []), pad=8)
+        self.s_in, self.s_out = (w.act("shared.gate", "shared.up"), w.act("shared.down")) if sh else (None, None)
+
+    def reserve(self, e) -> None:
+        n, dt, d = e.max_rows, self.router.dtype, self.router.shape[1]
+        self.tile = R.MOE_TILE
+        e.scratch.reserve("moe_z", n * self.router.shape[0], torch.float32)
+        e.scratch.reserve("moe_w", n * self.slots, torch.float32)
+        for name, size in (("moe_ids", n * self.top), ("moe_order", n * self.top), ("moe_tiles", 4 * R.moe_tiles(n, self.E, self.top, self.tile)), ("moe_count", 4)):
+            e.scratch.reserve(name, size, torch.int32)
+        e.scratch.reserve("moe_act", n * self.top * self.ff, dt)
+        e.scratch.reserve("moe_parts", n * self.slots * d, dt)
+        if self.shared:
+            e.scratch.reserve("proj", n * 2 * self.shared_ff, dt)
+            e.scratch.reserve("ff_act", n * self.shared_ff, dt)
+
+    def run(self, s, h):
+        n, d, top, slots = s.n, h.shape[1], self.top, self.slots
+        z = R.head(h, self.router, s.scratch.get("moe_z", n, self.router.shape[0]), "router")
+        ids, wts = s.scratch.get("moe_ids", n, top), s.scratch.get("moe_w", n, slots)
+        R.moe_route(z, ids, wts, self.E, top, self.shared)
+        act, parts = s.scratch.get("moe_act", n * top, self.ff), s.scratch.get("moe_parts", n, slots, d)
+        s_act = s.scratch.get("ff_act", n, self.shared_ff) if self.shared else None
+        if R.moe_gemv_takes(h, self.ff, self.shared_ff):
+            side = (h, self.s_in, s_act, self.shared_ff, self.shared_limit) if self.shared else None
+            R.moe_gemv(ids, h, self.w_in, act, side, n, self.ff, top, slots, True, self.alpha, self.limit)
+            R.moe_gemv(ids, act, self.w_out, parts, (s_act, self.s_out, None, d, 0.0) if self.shared else None, n, d, top, slots, False)
+            return parts, wts
+        plan = (s.scratch.get("moe_order", n * top), s.scratch.get("moe_tiles", R.moe_tiles(n, self.E, top, self.tile), 4), s.scratch.get("moe_count", 4),
+                R.moe_tiles(n, self.E, top, self.tile))
+        R.moe_plan(ids, *plan[:3], self.E, self.tile)
+        R.moe_tile(h, self.w_in, act, plan, self.ff, top, slots, True, self.alpha, self.limit)
+        R.moe_tile(act, self.w_out, parts, plan, d, top, slots, False)
+        if self.shared:
+            R.gated_linear(h, self.s_in, s.scratch.get("proj", n, 2 * self.shared_ff), s_act, "clamp", self.alpha, self.shared_limit)
+            R.linear(s_act, self.s_out, None, parts[:, top])
+        return parts, wts
+
+
+class TokenInput:
+    """What a layer adds from a table of its own rows per token: W_proj (gelu(W_gate x) * table[token]), to be RMS-normed by the seam.  ``x``
+    is the residual itself; all layers' rows lie side by side in one table."""
+
+    def __init__(self, w: W, table: torch.Tensor, col0: int):
+        self.table, self.col0 = table, col0
+        self.gate, self.proj = w.act("gate"), w.act("proj")
+        self.dim = self.gate.shape[0]
+
+    def reserve(self, e) -> None:
+        e.scratch.reserve("side_z", e.max_rows * self.dim, self.gate.dtype)
+        e.scratch.reserve("side_g", e.max_rows * self.dim, self.gate.dtype)
+
+    def run(self, s, h):
+        n = s.n
+        z = R.linear(h, self.gate, None, s.scratch.get("side_z", n, self.dim))
+        g = s.scratch.get("side_g", n, self.dim)
+        R.token_gate(z, self.table, self.col0, s.tokens, g, n, s.status)
+        return R.linear(g, self.proj, None, s.scratch.get("y", n, h.shape[1]))

@@ -15,21 +15,30 @@ from ..runtime.segments import note
 from .native import _check, _p, _stream
 
 MAX_TAPS = 8
+PAGE = 64                 # positions of a cache page (kv/paged.py)
 
 
 def _fp32(t: torch.Tensor) -> c_int:
     return c_int(1 if t.dtype == torch.float32 else 0)
 
 
+POST = {"layer": 0, "rms": 1, "scale": 2}
+
+
 def seam(x, n, *, h=None, y=None, y2=None, merge_w=(None, None), post=(None, None), embed=None, tokens=None, from_embed=False, add_embed=False,
-         step_vec=None, tap=None, norm=(None, None), row_map=None, conv=None, eps=1e-6, status=None, embed_scale=1.0):
+         step_vec=None, tap=None, norm=(None, None), row_map=None, conv=None, eps=1e-6, status=None, embed_scale=1.0, parts_w=None, post_kind="layer",
+         norm_kind="layer"):
     """x += LN(y; post) (y and y2: half the sum of their RMS norms), + embedding * embed_scale, + step_vec; h = LN(x; norm), or x itself.
+    ``post_kind``: layer norm, "rms" norm or "scale" (y * post[0]); ``norm_kind``: "layer" or "rms".  ``parts_w`` [n, parts]: y is [n, parts, d]
+    and its weighted sum over the parts is the output.
     ``conv``: (weight [taps, d], history, src, dst) applies h + conv(h) on a step of single-row segments."""
+    rms = norm_kind == "rms"
     act = h if h is not None else (y if y is not None else embed)
     cw, hist, src, dst = conv if conv is not None else (None, None, None, None)
-    _check(_lib.rows().sfb_rows_seam(_p(x), _p(y), _p(y2), _p(merge_w[0]), _p(merge_w[1]), _p(post[0]), _p(post[1]), _p(embed), _p(tokens),
+    _check(_lib.rows().sfb_rows_seam(_p(x), _p(y), _p(y2), _p(merge_w[0]), _p(merge_w[1]), _p(parts_w), _p(post[0]), _p(post[1]), _p(embed), _p(tokens),
                                      _p(step_vec), _p(tap), _p(norm[0]), _p(norm[1]), _p(h), _p(row_map), _p(cw), _p(hist), _p(src), _p(dst),
-                                     c_int(from_embed), c_int(add_embed), c_int(cw.shape[0] if cw is not None else 0), c_int(n), c_int(x.shape[1]),
+                                     c_int(from_embed), c_int(add_embed), c_int(cw.shape[0] if cw is not None else 0),
+                                     c_int(parts_w.shape[1] if parts_w is not None else 0), c_int(POST[post_kind]), c_int(rms), c_int(n), c_int(x.shape[1]),
                                      c_int(embed.shape[0] if embed is not None else 0), c_float(eps), c_float(embed_scale), _fp32(act), _p(status), _stream()), "rows_seam")
 
 
@@ -50,15 +59,31 @@ def qk_append(proj, qw, kw, q, kpool, vpool, table, row_lane, row_pos, n, heads,
                                           c_int(vdim), c_float(eps), _fp32(q), _p(status), _stream()), "rows_qk_append")
 
 
+def rot_append(proj, cs, dims, q, kpool, vpool, v_first, lam, table, row_lane, row_pos, n, heads, status):
+    """q | k | v of ``proj``: queries and keys turned (cs [positions, dims / 2, 2]), values mixed with ``v_first`` by ``lam`` (None: left there,
+    if given), queries to ``q``, the rest to the pools."""
+    G, dim, vdim = kpool.shape[1], kpool.shape[3], vpool.shape[3]
+    _check(_lib.rows().sfb_rows_rot_append(*_strides(proj), _p(cs), _p(q), _p(kpool), _p(vpool), _p(v_first), _p(lam), _p(table), _p(row_lane), _p(row_pos),
+                                           c_int(table.shape[1]), c_int(kpool.shape[0]), c_int(n), c_int(heads), c_int(G), c_int(dim), c_int(vdim),
+                                           c_int(dims), _fp32(q), _p(status), _stream()), "rows_rot_append")
+
+
+def token_gate(z, table, col0, tokens, out, n, status):
+    """out = gelu(z) * table[token, col0 : col0 + dim]."""
+    _check(_lib.rows().sfb_rows_token_gate(_p(z), _p(table), _p(tokens), _p(out), c_int(n), c_int(z.shape[1]), c_int64(table.stride(0)), c_int(col0),
+                                           c_int(table.shape[0]), _fp32(z), _p(status), _stream()), "rows_token_gate")
+
+
 NO_WINDOW = 2 ** 31 - 1
 
 
 def attn(q, kpool, vpool, table, row_lane, row_pos, rows, n_rows, bias, out, part, ml, heads, scale, splits, status, window=NO_WINDOW, vdim=None,
-         compact=False):
+         compact=False, sink=None, cap=0.0):
     """Exact arm: one block per (row, group of heads, range of pages).  ``rows``: indices of the rows to run, or None for all.
-    ``vpool`` None: values are the first ``vdim`` columns of the keys.  ``compact``: q and out hold only the rows of the launch."""
+    ``vpool`` None: values are the first ``vdim`` columns of the keys.  ``compact``: q and out hold only the rows of the launch.
+    ``cap``: scores become cap tanh(score / cap), 0: not.  ``sink`` [heads]: logits that only the denominator sees."""
     _check(_lib.rows().sfb_rows_attn(_p(q), _p(kpool), _p(vpool), _p(table), _p(row_lane), _p(row_pos), _p(rows), _p(bias),
-                                     c_int64(bias.shape[1] if bias is not None else 0), _p(out), _p(part), _p(ml), c_int(table.shape[1]),
+                                     c_int64(bias.shape[1] if bias is not None else 0), _p(sink), c_float(cap), _p(out), _p(part), _p(ml), c_int(table.shape[1]),
                                      c_int(kpool.shape[0]), c_int(n_rows), c_int(heads), c_int(kpool.shape[1]), c_int(kpool.shape[3]),
                                      c_int(vdim or vpool.shape[3]), c_int(splits), c_int(window), c_int(compact), c_float(scale), _fp32(q), _p(status), _stream()),
            "rows_attn")
@@ -79,28 +104,32 @@ def gated_step(x, y, cw, cb, hist, wg, rb, ib, decay, S, out, src, dst, n):
                                            c_int(cw.shape[0]), _fp32(out), _stream()), "rows_gated_step")
 
 
-ACT = {"silu": 1, "gelu_tanh": 2}
+ACT = {"silu": 1, "gelu_tanh": 2, "clamp": 3}
 
 
-def act_mul(gate_up, out, n, act="silu"):
-    _check(_lib.rows().sfb_rows_act_mul(_p(gate_up), _p(out), c_int(n), c_int(out.shape[1]), c_int(ACT[act]), _fp32(out), _stream()), "rows_act_mul")
+def act_mul(gate_up, out, n, act="silu", alpha=0.0, limit=0.0):
+    """out = act(gate) * up; "clamp": g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = up within +-limit."""
+    _check(_lib.rows().sfb_rows_act_mul(_p(gate_up), *_strides(out), c_int(n), c_int(out.shape[1]), c_int(ACT[act]), c_float(alpha), c_float(limit), _fp32(out),
+                                        _stream()), "rows_act_mul")
 
 
 def _strides(t) -> tuple:
     return (_p(t), c_int64(t.stride(0))) if t is not None else (None, c_int64(0))
 
 
-def state_rows(q, k, v, dt, dt_bias, a, D, rot, rot_dims, k_scale, row_pos, y, S, N, groups, segs, n_segs, seg, conv=None):
+def state_rows(q, k, v, dt, dt_bias, a, D, rot, rot_dims, k_scale, row_pos, y, S, N, groups, segs, n_segs, seg, conv=None,
+               beta=None, q_scale=1.0, unit_eps=0.0):
     """S = a S + w k v^T, y = S^T q + D v, one block per (segment, head, tile of value dims); q, k, v, dt: [n, .] views.
     ``rot``: [positions, rot_dims / 2, 2] or None.  ``conv``: (weight [taps, C], bias, history, first channels of q, k, v) where every
-    segment is one row and q, k, v are the inputs of a convolution with silu.  ``segs``: segments to run, or None for all."""
+    segment is one row and q, k, v are the inputs of a convolution with silu.  ``segs``: segments to run, or None for all.
+    ``beta``: raw write strengths: the delta rule on unit vectors q (times ``q_scale``) and k."""
     _, H, P, Np = S.shape
     cw, cb, hist, ch = conv if conv is not None else (None, None, None, (0, 0, 0))
-    _check(_lib.rows().sfb_rows_state(*_strides(q), *_strides(k), *_strides(v), *_strides(dt), _p(dt_bias), _p(a), _p(D), _p(rot), _p(row_pos), _p(y), _p(S),
+    _check(_lib.rows().sfb_rows_state(*_strides(q), *_strides(k), *_strides(v), *_strides(dt), _p(dt_bias), _p(a), _p(D), *_strides(beta), _p(rot), _p(row_pos), _p(y), _p(S),
                                       _p(cw), _p(cb), _p(hist), _p(segs), _p(seg.seg_row0), _p(seg.seg_len), _p(seg.seg_src), _p(seg.seg_dst),
                                       c_int(n_segs), c_int(rot_dims), c_int(cw.shape[0] if cw is not None else 0),
                                       c_int(cw.shape[1] if cw is not None else 0), *map(c_int, ch), c_int(H), c_int(groups), c_int(N), c_int(P),
-                                      c_int(Np), c_float(k_scale), _fp32(y), _stream()), "rows_state")
+                                      c_int(Np), c_float(k_scale), c_float(q_scale), c_float(unit_eps), _fp32(y), _stream()), "rows_state")
 
 
 def state_tc_supports(dtype: torch.dtype, n: int, p: int, terms: int) -> bool:
@@ -181,9 +210,9 @@ def _gemv_takes(x: torch.Tensor) -> bool:
     return x.dtype == torch.bfloat16 and n <= GEMV_ROWS and K % 8 == 0 and (n if n < 3 else 4) * K * 2 <= 200 * 1024
 
 
-def _gemv(x, w, b, out, act: int = 0) -> None:
-    _check(_lib.rows().sfb_rows_gemv(_p(w), _p(x), _p(b), _p(out), c_int(x.shape[0]), c_int(out.shape[1]), c_int(x.shape[1]),
-                                     c_int(out.dtype == torch.float32), c_int(act), _stream()), "rows_gemv")
+def _gemv(x, w, b, out, act: int = 0, alpha: float = 0.0, limit: float = 0.0) -> None:
+    _check(_lib.rows().sfb_rows_gemv(_p(w), _p(x), _p(b), *_strides(out), c_int(x.shape[0]), c_int(out.shape[1]), c_int(x.shape[1]),
+                                     c_int(out.dtype == torch.float32), c_int(act), c_float(alpha), c_float(limit), _stream()), "rows_gemv")
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor | None, out: torch.Tensor) -> torch.Tensor:
@@ -199,13 +228,14 @@ def linear(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor | None, out: torch.
     return out
 
 
-def gated_linear(x: torch.Tensor, w: torch.Tensor, scratch: torch.Tensor | None, out: torch.Tensor, act: str = "silu") -> torch.Tensor:
+def gated_linear(x: torch.Tensor, w: torch.Tensor, scratch: torch.Tensor | None, out: torch.Tensor, act: str = "silu", alpha: float = 0.0,
+                 limit: float = 0.0) -> torch.Tensor:
     """out = act(x wg^T) * (x wu^T), w = wg stacked on wu; ``scratch`` [n, 2 ff] holds both products where they are not fused."""
     if _gemv_takes(x):
-        _gemv(x, w, None, out, ACT[act])
+        _gemv(x, w, None, out, ACT[act], alpha, limit)
         return out
     linear(x, w, None, scratch)
-    act_mul(scratch, out, x.shape[0], act)
+    act_mul(scratch, out, x.shape[0], act, alpha, limit)
     return out
 
 
@@ -234,8 +264,8 @@ def block_gates(u: torch.Tensor, wg: torch.Tensor, out: torch.Tensor) -> torch.T
     return out
 
 
-def head(x: torch.Tensor, embed: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """32-bit logits of x [rows, width] against the output table."""
+def head(x: torch.Tensor, embed: torch.Tensor, out: torch.Tensor, name: str = "head") -> torch.Tensor:
+    """32-bit logits of x [rows, width] against the output table (or a router's)."""
     if _gemv_takes(x):
         _gemv(x, embed, None, out)
         return out
@@ -243,7 +273,7 @@ def head(x: torch.Tensor, embed: torch.Tensor, out: torch.Tensor) -> torch.Tenso
         torch.mm(x, embed.t(), out=out)
     else:
         torch.mm(x, embed.t(), out_dtype=torch.float32, out=out)
-    note("head")
+    note(name)
     return out
 
 
@@ -269,12 +299,13 @@ def attn_stream_supports(dtype: torch.dtype, dim: int, vdim: int) -> bool:
     return dtype == torch.bfloat16 and dim in (32, 64, 96, 128, 256) and vdim % 32 == 0 and vdim <= 256
 
 
-def attn_stream(q, kpool, vpool, table, row_lane, row_pos, rows, n_rows, bias, out, part, ml, heads, scale, page_bound, status):
-    """Single rows, bf16: the pages of all rows cut evenly over the machine.  ``page_bound``: at least the sum of the rows' pages."""
+def attn_stream(q, kpool, vpool, table, row_lane, row_pos, rows, n_rows, bias, out, part, ml, heads, scale, page_bound, status,
+                window=NO_WINDOW, sink=None, cap=0.0):
+    """Single rows, bf16: the pages of all rows cut evenly over the machine.  ``page_bound``: at least the sum of the pages that rows see."""
     G, dim, vdim = kpool.shape[1], kpool.shape[3], vpool.shape[3]
     _check(_lib.rows().sfb_rows_attn_stream(_p(q), _p(kpool), _p(vpool), _p(table), _p(row_lane), _p(row_pos), _p(rows), _p(bias),
-                                            c_int64(bias.shape[1] if bias is not None else 0), _p(out), _p(part), _p(ml), c_int(table.shape[1]),
-                                            c_int(kpool.shape[0]), c_int(n_rows), c_int(heads), c_int(G), c_int(dim), c_int(vdim),
+                                            c_int64(bias.shape[1] if bias is not None else 0), _p(sink), c_float(cap), c_int(window), _p(out), _p(part), _p(ml),
+                                            c_int(table.shape[1]), c_int(kpool.shape[0]), c_int(n_rows), c_int(heads), c_int(G), c_int(dim), c_int(vdim),
                                             c_int(attn_stream_heads(heads, G, dim)), c_int(page_bound), c_float(scale), _p(status), _stream()),
            "rows_attn_stream")
 
@@ -321,15 +352,15 @@ def tensor_map(t: torch.Tensor, cols: int, box: int, stride: int | None = None, 
     return m
 
 
-def attn_tc(q, kv, table, row_lane, row_pos, tiles, n_tiles, bias, out, heads, scale, status):
+def attn_tc(q, kv, table, row_lane, row_pos, tiles, n_tiles, bias, out, heads, scale, status, window=NO_WINDOW, sink=None, cap=0.0):
     """Tensor-core arm over runs of rows: ``tiles`` are (row0, rows <= 256) pairs, each inside one segment; kv from attn_pools."""
     k, v, (mk, mv) = kv
     mq = tensor_map(q, q.shape[1], 128)
     G = k.shape[1]
     _check(_lib.rows().sfb_rows_attn_tc(mq.ptr, mk.ptr, mv.ptr, None, _p(table), _p(row_lane), _p(row_pos), _p(tiles), None, c_int(n_tiles), _p(bias),
-                                        c_int64(bias.shape[1] if bias is not None else 0), _p(out), c_int(table.shape[1]), c_int(k.shape[0]),
-                                        c_int(heads), c_int(G), c_int(k.shape[3]), c_int(v.shape[3]), c_int(0), c_int(G * 64), c_int(64),
-                                        c_int(NO_WINDOW), c_float(scale), _p(status), _stream()), "rows_attn_tc")
+                                        c_int64(bias.shape[1] if bias is not None else 0), _p(sink), c_float(cap), _p(out), c_int(table.shape[1]),
+                                        c_int(k.shape[0]), c_int(heads), c_int(G), c_int(k.shape[3]), c_int(v.shape[3]), c_int(0), c_int(G * 64), c_int(64),
+                                        c_int(window), c_float(scale), _p(status), _stream()), "rows_attn_tc")
 
 
 def latent_tc_supports(dtype: torch.dtype, dim: int, rot: int, vdim: int, rank: int) -> bool:
@@ -369,6 +400,47 @@ def latent_attn_tc(q, q_stride, kx, vx, rows, rank, row_pos, tiles, offs, n_tile
     m = kx.shape[1]
     mq, mk, mv = tensor_map(q, heads * (dim + rot), 128, q_stride), tensor_map(kx, dim, 64), tensor_map(vx, vdim, 64)
     mr = tensor_map(rows, rot, 64, rank + rot, rank)
-    _check(_lib.rows().sfb_rows_attn_tc(mq.ptr, mk.ptr, mv.ptr, mr.ptr, None, None, _p(row_pos), _p(tiles), _p(offs), c_int(n_tiles), None, c_int64(0),
+    _check(_lib.rows().sfb_rows_attn_tc(mq.ptr, mk.ptr, mv.ptr, mr.ptr, None, None, _p(row_pos), _p(tiles), _p(offs), c_int(n_tiles), None, c_int64(0), None, c_float(0.0),
                                         _p(out), c_int(0), c_int(m // 64), c_int(heads), c_int(heads), c_int(dim), c_int(vdim), c_int(rot), c_int(64),
                                         c_int(m), c_int(window), c_float(scale), _p(status), _stream()), "rows_attn_tc")
+
+
+# ---- mixture of experts (csrc/k_rows_moe.cu, csrc/k_rows_moe_tc.cu) --------------------------------------------------------
+MOE_TILE, MOE_TC_TILE = 32, 128          # pairs of a tile on CUDA cores, on the tensor cores
+MOE_MAX_EXPERTS, MOE_MAX_TOP = 1024, 32
+
+
+def moe_tiles(n: int, experts: int, top: int, tile: int) -> int:
+    """Most tiles of a step of n rows."""
+    return n * top // tile + min(experts, n * top)
+
+
+def moe_route(z, ids, wts, experts, top, shared):
+    """Choices [n, top] and weights [n, top + shared] of logits z [n, >= experts + shared]."""
+    _check(_lib.rows().sfb_rows_moe_route(*_strides(z), _p(ids), _p(wts), c_int(z.shape[0]), c_int(experts), c_int(top), c_int(shared), _stream()),
+           "rows_moe_route")
+
+
+def moe_plan(ids, order, tiles, count, experts, tile):
+    _check(_lib.rows().sfb_rows_moe_plan(_p(ids), _p(order), _p(tiles), _p(count), c_int(ids.numel()), c_int(experts), c_int(tile), _stream()), "rows_moe_plan")
+
+
+def moe_tile(x, w, out, plan, M, top, slots, gated, alpha=0.0, limit=0.0):
+    """One product of every expert on its pairs; ``plan``: (order, tiles, count, most tiles).  gated: x [n, K], w [E, 2 M, K], out [pairs, M] in
+    plan order; else x [pairs, K], w [E, M, K], out [n, slots, M]."""
+    order, tiles, count, most = plan
+    _check(_lib.rows().sfb_rows_moe_tile(_p(x), _p(w), _p(out), _p(order), _p(tiles), _p(count), c_int(most), c_int(M), c_int(w.shape[2]), c_int(top),
+                                         c_int(slots), c_int(gated), c_float(alpha), c_float(limit), _fp32(out), _stream()), "rows_moe_tile")
+
+
+def moe_gemv_takes(x: torch.Tensor, ff: int, shared_ff: int) -> bool:
+    n, K = x.shape
+    return x.dtype == torch.bfloat16 and n <= GEMV_ROWS and K % 8 == 0 and ff % 8 == 0 and shared_ff % 8 == 0 and max(K, ff, shared_ff) * 2 <= 200 * 1024
+
+
+def moe_gemv(ids, x, w, out, shared, n, M, top, slots, gated, alpha=0.0, limit=0.0):
+    """Few rows; ``shared``: (x, w, out, M, limit) of the shared expert or None."""
+    sx, sw, sout, sm, sl = shared if shared is not None else (None, None, None, 0, 0.0)
+    _check(_lib.rows().sfb_rows_moe_gemv(_p(ids), _p(x), _p(w), _p(out), _p(sx), _p(sw), _p(sout), c_int(ids.numel()), c_int(n), c_int(M), c_int(w.shape[2]),
+                                         c_int(sm), c_int(sw.shape[1] if sw is not None else 0), c_int(top), c_int(slots), c_int(gated), c_float(alpha),
+                                         c_float(limit), c_float(sl), _stream()), "rows_moe_gemv")
