@@ -1,0 +1,523 @@
+// The gated delta rule of k_rows_state.cu for long runs of rows, on tcgen05.  With unit vectors q and k of a head,
+//
+//   S = a_t S_(t-1),   u_t = b_t (v_t - S^T k_t),   S_t = S + k_t u_t^T,   y_t = S_t^T q_t
+//
+// A run is cut into chunks of 128 rows.  With c_t the running sum of log a inside a chunk, S_0 the state at its start and
+// A_ij = b_i exp(c_i - c_j) (k_i . k_j) for j < i, the writes of a chunk solve (I + A) U = X, so that
+//
+//   U = (I + A)^-1 X,   X_i = b_i (v_i - exp(c_i) S_0^T k_i),
+//   S_0 of the next chunk = exp(c_last) S_0 + sum_j exp(c_last - c_j) k_j u_j^T,
+//   y_i = sum_{j <= i} exp(c_i - c_j) (q_i . k_j) u_j + exp(c_i) S_0^T q_i
+//
+//   delta_prep    per (chunk, group of heads): K K^T, the numbers of the rows (RATES), and (I + A)^-1 of every head in 32-bit: diagonal blocks
+//                 of 32 by substitution, the others from pairs of blocks
+//   delta_chain   per (head, 32 value dims), chunk after chunk: three products (K S_0, inverse X, K^T U), the state in registers
+//   chunk_out     the third line, all chunks at once (k_rows_state_tc.cu)
+//
+// q and k stay the bf16 vectors they come as; what makes them unit vectors is a factor per row on a product's result or on its other
+// operand.  Everything else that enters a product is a 32-bit value taken as two bf16 terms (16 mantissa bits): state, X, U, the inverse
+// (whose product with X leaves out lower times lower).  Accumulators, decays, the inverse and the state are 32-bit.  Every wait is bounded
+// and reports through the status word; no cluster, no multicast.
+#include "k_rows_state_tc.cuh"
+
+namespace sfb {
+namespace rdelta {
+using namespace rst;
+
+struct Args {
+  const int *c_row0, *c_rows;      // chunks
+  const int *seg, *first;          // runs: segment, first chunk (one entry more than runs)
+  const int *seg_src, *seg_dst;
+  const __nv_bfloat16* qkv;        // [n, stride]: q, k, v from the columns below
+  int64_t stride;
+  const __nv_bfloat16 *dt, *beta;  // [n, .] raw step sizes, raw write strengths
+  int64_t dt_stride, beta_stride;
+  const float *dt_bias, *a;        // [H]
+  float* S;                        // [slots, H, P, Np]
+  float* rates;                    // [chunks, H, RATES, 128]
+  float* dec;                      // [chunks, H] decay over the whole chunk
+  __nv_bfloat16* inv;              // [chunks, H, 2, 128, 128]: upper terms, lower terms (columns 64.. of rows below 64 are not written)
+  __nv_bfloat16* u;                // [2, u_lo, H P]
+  __nv_bfloat16* starts;           // [2, chunks, H, N, P]
+  int H, G, N, P, Np, ns, hpc, chunks, u_lo;
+  int q_col, k_col, v_col;
+  float q_scale, unit_eps;
+  Status* status;
+};
+
+constexpr int LD = 132;            // row stride of the matrix that is inverted
+
+// One warp, one head: running sums of log2 of the decays (a lane takes four rows; past the end: decay 1), and the numbers of the rows from
+// k's and q's factors to unit length.  c and the write strengths (0 past the end) also to `cs` and `bs`.
+__device__ __forceinline__ void head_rates(const Args& a, int chunk, int h, int row0, int rows, const float* rk, const float* rq, float* cs, float* bs) {
+  const int lane = threadIdx.x & 31;
+  const float ah = a.a[h] * LOG2E, bias = a.dt_bias[h];
+  float c[4], b[4], t = 0.f;
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const int i = lane * 4 + k;
+    float w = 0.f;
+    b[k] = 0.f;
+    if (i < rows) {
+      const float z = __bfloat162float(a.dt[(size_t)(row0 + i) * a.dt_stride + h]) + bias;
+      w = log1pf(expf(-fabsf(z))) + fmaxf(z, 0.f);
+      b[k] = 1.f / (1.f + expf(-__bfloat162float(a.beta[(size_t)(row0 + i) * a.beta_stride + h])));
+    }
+    t += ah * w;
+    c[k] = t;
+  }
+  float s = t;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) { const float v = __shfl_up_sync(0xffffffffu, s, o); if (lane >= o) s += v; }
+  const float last = __shfl_sync(0xffffffffu, s, 31), before = s - t;
+  float* out = a.rates + ((size_t)chunk * a.H + h) * RATES * L + lane * 4;
+  float x[RATES][4];
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const int i = lane * 4 + k;
+    c[k] += before;
+    cs[i] = c[k];
+    bs[i] = b[k];
+    const bool in = i < rows;
+    const float f = rk[i];
+    x[0][k] = c[k];
+    x[1][k] = in ? c[k] - __log2f(f) : INFINITY;         // its exponential: 0
+    x[2][k] = rq[i];
+    x[3][k] = in ? ex2(c[k]) * f : 0.f;
+    x[4][k] = b[k];
+    x[5][k] = in ? ex2(last - c[k]) * f : 0.f;
+  }
+#pragma unroll
+  for (int r = 0; r < RATES; ++r) rows::store_v<float, 4>(out + r * L, x[r]);
+  if (lane == 0) a.dec[(size_t)chunk * a.H + h] = ex2(last);
+}
+
+// acc[r][c] += sum over k in [k0, k1) of x[r][k] y[k][c], four by four; x, y: rows of LD / ldy floats, k0 and k1 multiples of four
+__device__ __forceinline__ void micro(float (&acc)[4][4], const float* x, const float* y, int ldy, int k0, int k1) {
+  for (int k = k0; k < k1; k += 4) {
+    float4 l[4], r[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      l[i] = *reinterpret_cast<const float4*>(x + i * LD + k);
+      r[i] = *reinterpret_cast<const float4*>(y + (k + i) * ldy);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float lv[4] = {l[i].x, l[i].y, l[i].z, l[i].w};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        acc[i][0] = fmaf(lv[j], r[j].x, acc[i][0]); acc[i][1] = fmaf(lv[j], r[j].y, acc[i][1]);
+        acc[i][2] = fmaf(lv[j], r[j].z, acc[i][2]); acc[i][3] = fmaf(lv[j], r[j].w, acc[i][3]);
+      }
+    }
+  }
+}
+
+// The block below a pair of inverted diagonal blocks of B rows at `b0`: -T22 (A21 T11), by B x B / 16 threads (`t` counts them).
+// `w`: B x (B + 4) floats.  Two calls, a barrier in between: the inner product, then the outer one.
+template <int B>
+__device__ __forceinline__ void pair_inner(const float* A, float* w, int b0, int t) {
+  const int r = t / (B / 4) * 4, c = t % (B / 4) * 4;
+  float acc[4][4] = {};
+  micro(acc, A + (b0 + B + r) * LD + b0, A + b0 * LD + b0 + c, LD, c, B);      // T11 is lower triangular
+#pragma unroll
+  for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(w + (r + i) * (B + 4) + c) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+}
+template <int B>
+__device__ __forceinline__ void pair_outer(float* A, const float* w, int b0, int t) {
+  const int r = t / (B / 4) * 4, c = t % (B / 4) * 4;
+  float acc[4][4] = {};
+  micro(acc, A + (b0 + B + r) * LD + b0 + B, w + c, B + 4, 0, r + 4);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(A + (b0 + B + r + i) * LD + b0 + c) = make_float4(-acc[i][0], -acc[i][1], -acc[i][2], -acc[i][3]);
+}
+
+// grid (groups x parts of a group's heads, chunks); 256 threads
+__global__ void __launch_bounds__(WORK, 2) delta_prep_kernel(const __grid_constant__ CUtensorMap mk, Args a) {
+  extern __shared__ __align__(1024) uint8_t sm[];
+  uint8_t* ks = sm;                                       // k, two slabs; later the pairs' inner products
+  float* w = reinterpret_cast<float*>(sm);
+  float* A = reinterpret_cast<float*>(sm + 2 * SLAB);     // [128][LD]
+  float* rk = A + L * LD;                                 // [128] each
+  float *rq = rk + L, *cs = rq + L, *bs = cs + L;
+  Ctl& C = *reinterpret_cast<Ctl*>(bs + L);
+  setup(C, 128);
+  pdl_launch_dependents();
+  pdl_wait();
+  const int chunk = blockIdx.y, rep = a.H / a.G, parts = (rep + a.hpc - 1) / a.hpc, g = blockIdx.x / parts;
+  const int h0 = g * rep + (blockIdx.x % parts) * a.hpc, nh = min(a.hpc, (g + 1) * rep - h0), row0 = a.c_row0[chunk], rows = a.c_rows[chunk];
+  const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0), lane = tid & 31;
+  volatile int* dead = &C.dead;
+  if (warp == 0) {
+    if (elect_one()) {
+      mbar_expect(&C.full[0], a.ns * SLAB);
+      for (int s = 0; s < a.ns; ++s) tma2d(ks + s * SLAB, &mk, a.k_col + g * a.N + 64 * s, row0, &C.full[0]);
+    }
+    wait_warp(&C.full[0], 0, dead, 2);
+    if (elect_one()) {
+      const uint32_t id = idesc(128, 0, 0);
+      const uint64_t dk = desc(smem_u32(ks), 16);
+      for (int t = 0; t < a.N / 16; ++t) {
+        const uint64_t o = (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2;
+        mma_ss(C.tmem, dk + o, dk + o, id, t ? 1u : 0u);
+      }
+      commit(&C.done[0]);
+    }
+    __syncwarp();
+  }
+  {   // a thread per row and vector: its factor to unit length
+    const int i = tid & (L - 1), isk = tid >> 7;
+    float s = 0.f;
+    if (i < rows) {
+      const __nv_bfloat16* p = a.qkv + (size_t)(row0 + i) * a.stride + (isk ? a.k_col : a.q_col) + g * a.N;
+      for (int n = 0; n < a.N; n += 8) {
+        float f[8];
+        rows::load_v<__nv_bfloat16, 8>(p + n, f);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) s = fmaf(f[k], f[k], s);
+      }
+    }
+    (isk ? rk : rq)[i] = (isk ? 1.f : a.q_scale) / sqrtf(s + a.unit_eps);
+  }
+  const int w4 = warp & 3, half = warp >> 2, i = w4 * 32 + lane;
+  wait_warp(&C.done[0], 0, dead, 3);
+  fence_after();
+  for (int x = 0; x < nh; ++x) {
+    const int h = h0 + x;
+    __syncthreads();                                      // factors are there; the matrix of the head before has been written out
+    if (warp == 0) head_rates(a, chunk, h, row0, rows, rk, rq, cs, bs);
+    __syncthreads();
+    {
+      const float ci = cs[i], bi = i < rows ? bs[i] * rk[i] : 0.f;
+#pragma unroll
+      for (int b = 0; b < 2; ++b) {
+        const int j0 = half * 64 + b * 32;
+        if (j0 > w4 * 32 + 31) continue;                  // above the diagonal: not read below
+        float s[32];
+        ld32(C.tmem + j0 + ((uint32_t)(w4 * 32) << 16), s);
+        wait_ld();
+#pragma unroll
+        for (int q = 0; q < 8; ++q) {
+          float o[4];
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const int j = j0 + 4 * q + k;
+            o[k] = j < i && i < rows ? s[4 * q + k] * bi * rk[j] * ex2(ci - cs[j]) : 0.f;
+          }
+          *reinterpret_cast<float4*>(A + i * LD + j0 + 4 * q) = make_float4(o[0], o[1], o[2], o[3]);
+        }
+      }
+    }
+    __syncthreads();
+    if (warp < 4) {   // a diagonal block: lane = column, row after row
+      float t[32];
+      float* B = A + (warp * 32) * LD + warp * 32;
+#pragma unroll
+      for (int r = 0; r < 32; ++r) {
+        float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
+#pragma unroll
+        for (int k = 0; k < r; k += 4) {                  // elements at and past the diagonal are 0
+          const float4 v = *reinterpret_cast<const float4*>(B + r * LD + k);
+          s0 = fmaf(v.x, t[k], s0);
+          if (k + 1 < r) s1 = fmaf(v.y, t[k + 1], s1);
+          if (k + 2 < r) s2 = fmaf(v.z, t[k + 2], s2);
+          if (k + 3 < r) s3 = fmaf(v.w, t[k + 3], s3);
+        }
+        t[r] = r == lane ? 1.f : -((s0 + s1) + (s2 + s3));
+      }
+      __syncwarp();
+#pragma unroll
+      for (int r = 0; r < 32; ++r) B[r * LD + lane] = t[r];
+    }
+    __syncthreads();
+    if (tid < 128) pair_inner<32>(A, w + (tid >> 6) * 32 * 36, (tid >> 6) * 64, tid & 63);
+    __syncthreads();
+    if (tid < 128) pair_outer<32>(A, w + (tid >> 6) * 32 * 36, (tid >> 6) * 64, tid & 63);
+    else {            // the two blocks of 32 above the diagonal inside the blocks of 64
+      const int z = tid - 128, p = z >> 6, r = z & 63;
+      if (r < 32)
+        for (int c = 0; c < 32; c += 4) *reinterpret_cast<float4*>(A + (p * 64 + r) * LD + p * 64 + 32 + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    __syncthreads();
+    pair_inner<64>(A, w, 0, tid);
+    __syncthreads();
+    pair_outer<64>(A, w, 0, tid);
+    __syncthreads();
+    __nv_bfloat16* hi = a.inv + ((size_t)chunk * a.H + h) * 2 * L * L;
+    for (int r = warp; r < L; r += WORK / 32) {
+      if (r < 64 && lane >= 16) continue;
+      const float4 v = *reinterpret_cast<const float4*>(A + r * LD + lane * 4);
+      uint2 u, l;
+      split2(v.x, v.y, u.x, l.x);
+      split2(v.z, v.w, u.y, l.y);
+      *reinterpret_cast<uint2*>(hi + r * L + lane * 4) = u;
+      *reinterpret_cast<uint2*>(hi + (L + r) * L + lane * 4) = l;
+    }
+  }
+  fence_before();
+  if (*dead) drain(C);
+  teardown(C, 128, a.status, 73);
+}
+
+// sixteen 32-bit values as two bf16 terms: 16-byte words of the upper and of the lower ones
+__device__ __forceinline__ void split16(const float* f, uint4 (&hi)[2], uint4 (&lo)[2]) {
+#pragma unroll
+  for (int q = 0; q < 2; ++q) {
+    split2(f[8 * q], f[8 * q + 1], hi[q].x, lo[q].x); split2(f[8 * q + 2], f[8 * q + 3], hi[q].y, lo[q].y);
+    split2(f[8 * q + 4], f[8 * q + 5], hi[q].z, lo[q].z); split2(f[8 * q + 6], f[8 * q + 7], hi[q].w, lo[q].w);
+  }
+}
+
+constexpr int PT = 32;             // value dims of a block
+
+// grid (heads x tiles of 32 value dims, runs).  Operands with the value dims along a row (state, X, U) are 128 rows of 128 bytes, of which the
+// tile takes the first 64 bytes.
+__global__ void __launch_bounds__(THREADS, 1)
+delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mt, const __grid_constant__ CUtensorMap mt64, Args a) {
+  extern __shared__ __align__(1024) uint8_t sm[];
+  uint8_t* ks = sm;                                       // two stages of two slabs
+  uint8_t* ts = ks + 4 * SLAB;                            // inverse: upper terms (two slabs), lower terms
+  uint8_t* ss = ts + 4 * SLAB;                            // state, two terms
+  uint8_t* xs = ss + 2 * SLAB;                            // X, then U, two terms
+  Ctl& C = *reinterpret_cast<Ctl*>(xs + 2 * SLAB);
+  setup(C, 128);
+  const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0), lane = tid & 31;
+  // columns 64.. of the inverse's rows below 64 are zero and never loaded
+  for (int x = tid; x < 2 * HSLAB / 16; x += THREADS)
+    reinterpret_cast<uint4*>(ts + (x / (HSLAB / 16)) * 2 * SLAB + SLAB)[x % (HSLAB / 16)] = make_uint4(0u, 0u, 0u, 0u);
+  asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+  __syncthreads();
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tiles = (a.P + PT - 1) / PT, h = blockIdx.x / tiles, pt = blockIdx.x % tiles, g = h / (a.H / a.G);
+  const int run = blockIdx.y, seg = a.seg[run], c0 = a.first[run], nc = a.first[run + 1] - c0;
+  const bool issuer = warp == WORK / 32;
+  volatile int* dead = &C.dead;
+  const uint32_t t_ks = C.tmem, t_u = t_ks + PT, t_d = t_ks + 2 * PT;
+  if (issuer) {
+    auto load_k = [&](int c) {
+      mbar_expect(&C.full[c & 1], a.ns * SLAB);
+      for (int s = 0; s < a.ns; ++s) tma2d(ks + ((c & 1) * 2 + s) * SLAB, &mk, a.k_col + g * a.N + 64 * s, a.c_row0[c0 + c], &C.full[c & 1]);
+    };
+    auto load_t = [&](int c) {
+      const int y = ((c0 + c) * a.H + h) * 2 * L;
+      mbar_expect(&C.full[2], 2 * (SLAB + HSLAB));
+      for (int t = 0; t < 2; ++t) {
+        tma2d(ts + t * 2 * SLAB, &mt, 0, y + t * L, &C.full[2]);
+        tma2d(ts + t * 2 * SLAB + SLAB + HSLAB, &mt64, 64, y + t * L + 64, &C.full[2]);
+      }
+    };
+    if (elect_one()) {
+      load_k(0);
+      load_t(0);
+      if (nc > 1) load_k(1);
+    }
+    __syncwarp();
+    const uint32_t id = idesc(PT, 0, 1), idt = idesc(PT, 1, 1);
+    const uint64_t dt = desc(smem_u32(ts), 16), ds = desc(smem_u32(ss), SLAB), dx = desc(smem_u32(xs), SLAB), term = SLAB >> 4;
+    const int kst = a.N / 16;
+    for (int c = 0; c < nc; ++c) {
+      const uint64_t dk = desc(smem_u32(ks) + (c & 1) * 2 * SLAB, 16), dkt = desc(smem_u32(ks) + (c & 1) * 2 * SLAB, SLAB);
+      wait_warp(&C.full[c & 1], (c >> 1) & 1, dead, 4);
+      __syncthreads();                                    // the state is in place
+      if (elect_one()) {
+        fence_after();
+        for (int t = 0; t < kst; ++t) {
+          const uint64_t ka = dk + (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, sb = ds + (uint64_t)t * (2048 >> 4);
+          mma_ss(t_ks, ka, sb, id, t ? 1u : 0u);
+          mma_ss(t_ks, ka, sb + term, id, 1u);
+        }
+        commit(&C.done[0]);
+      }
+      __syncwarp();
+      wait_warp(&C.full[2], c & 1, dead, 5);
+      __syncthreads();                                    // X is in place
+      if (elect_one()) {
+        fence_after();
+#pragma unroll
+        for (int t = 0; t < 8; ++t) {
+          const uint64_t ta = dt + (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, xb = dx + (uint64_t)t * (2048 >> 4);
+          mma_ss(t_u, ta, xb, id, t ? 1u : 0u);
+          mma_ss(t_u, ta, xb + term, id, 1u);
+          mma_ss(t_u, ta + 2 * term, xb, id, 1u);
+        }
+        commit(&C.done[1]);
+      }
+      __syncwarp();
+      wait_warp(&C.done[1], c & 1, dead, 6);
+      if (c + 1 < nc && elect_one()) load_t(c + 1);
+      __syncwarp();
+      __syncthreads();                                    // U is in place
+      if (elect_one()) {
+        fence_after();
+#pragma unroll
+        for (int t = 0; t < 8; ++t) {
+          const uint64_t o = (uint64_t)t * (2048 >> 4);
+          mma_ss(t_d, dkt + o, dx + o, idt, t ? 1u : 0u);
+          mma_ss(t_d, dkt + o, dx + term + o, idt, 1u);
+        }
+        commit(&C.done[2]);
+      }
+      __syncwarp();
+      wait_warp(&C.done[2], c & 1, dead, 7);
+      if (c + 2 < nc && elect_one()) load_k(c + 2);
+      __syncwarp();
+    }
+  } else {
+    // a thread has one row (of the chunk, or of the state) and sixteen value dims
+    const int w4 = warp & 3, half = warp >> 2, i = w4 * 32 + lane, p0 = pt * PT + half * 16, width = min(16, a.P - p0);      // width: a multiple of 8, or none
+    const uint32_t at = ((uint32_t)(w4 * 32) << 16) + half * 16;
+    const size_t slot = (size_t)a.H * a.P * a.Np, HP = (size_t)a.H * a.P;
+    const bool in_n = i < a.N;
+    float S[16];
+    {
+      const int src = a.seg_src[seg];
+      const float* s0 = a.S + (size_t)(src >= 0 ? src : 0) * slot + ((size_t)h * a.P + p0) * a.Np + i;
+#pragma unroll
+      for (int k = 0; k < 16; ++k) S[k] = src >= 0 && in_n && k < width ? s0[(size_t)k * a.Np] : 0.f;
+    }
+    auto put = [&](uint8_t* op, const uint4 (&hi)[2], const uint4 (&lo)[2]) {      // row i, both terms, 128-byte swizzle
+#pragma unroll
+      for (int q = 0; q < 2; ++q) {
+        const int o = i * 128 + (((half * 2 + q) ^ (i & 7)) << 4);
+        *reinterpret_cast<uint4*>(op + o) = hi[q];
+        *reinterpret_cast<uint4*>(op + SLAB + o) = lo[q];
+      }
+    };
+    auto put_state = [&](int c) {
+      uint4 hi[2], lo[2];
+      split16(S, hi, lo);
+      put(ss, hi, lo);
+      if (in_n) {
+        __nv_bfloat16* o = a.starts + (((size_t)(c0 + c) * a.H + h) * a.N + i) * a.P + p0;
+        const size_t lower = (size_t)a.chunks * a.H * a.N * a.P;
+#pragma unroll
+        for (int q = 0; q < 2; ++q)
+          if (q * 8 < width) {
+            *reinterpret_cast<uint4*>(o + 8 * q) = hi[q];
+            *reinterpret_cast<uint4*>(o + lower + 8 * q) = lo[q];
+          }
+      }
+      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    };
+    uint4 v[2];
+    float ek, b, ue, dec;
+    int row, rows;
+    auto fetch = [&](int c) {
+      row = a.c_row0[c0 + c] + i;
+      rows = a.c_rows[c0 + c];
+      const float* r = a.rates + ((size_t)(c0 + c) * a.H + h) * RATES * L + i;
+      ek = r[3 * L]; b = r[4 * L]; ue = r[5 * L];
+      dec = a.dec[(size_t)(c0 + c) * a.H + h];
+      const __nv_bfloat16* p = a.qkv + (size_t)row * a.stride + a.v_col + (size_t)h * a.P + p0;
+#pragma unroll
+      for (int q = 0; q < 2; ++q) v[q] = i < rows && q * 8 < width ? *reinterpret_cast<const uint4*>(p + 8 * q) : make_uint4(0u, 0u, 0u, 0u);
+    };
+    fetch(0);
+    put_state(0);
+    __syncthreads();
+    for (int c = 0; c < nc; ++c) {
+      float f[16];
+      uint4 hi[2], lo[2];
+      wait_warp(&C.done[0], c & 1, dead, 8);
+      fence_after();
+      ld16(t_ks + at, f);
+      wait_ld();
+#pragma unroll
+      for (int q = 0; q < 2; ++q) {
+        const uint32_t vw[4] = {v[q].x, v[q].y, v[q].z, v[q].w};
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          float* x = f + 8 * q + 2 * k;
+          x[0] = i < rows ? b * (__uint_as_float(vw[k] << 16) - ek * x[0]) : 0.f;
+          x[1] = i < rows ? b * (__uint_as_float(vw[k] & 0xffff0000u) - ek * x[1]) : 0.f;
+        }
+      }
+      split16(f, hi, lo);
+      put(xs, hi, lo);
+      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+      fence_before();
+      __syncthreads();
+      wait_warp(&C.done[1], c & 1, dead, 9);
+      fence_after();
+      ld16(t_u + at, f);
+      wait_ld();
+      uint4 uh[2], ul[2];
+      split16(f, uh, ul);
+#pragma unroll
+      for (int k = 0; k < 16; ++k) f[k] = i < rows ? f[k] * ue : 0.f;
+      split16(f, hi, lo);
+      put(xs, hi, lo);
+      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+      fence_before();
+      __syncthreads();
+      if (i < rows) {                                     // under the product
+        __nv_bfloat16* o = a.u + (size_t)row * HP + (size_t)h * a.P + p0;
+#pragma unroll
+        for (int q = 0; q < 2; ++q)
+          if (q * 8 < width) {
+            *reinterpret_cast<uint4*>(o + 8 * q) = uh[q];
+            *reinterpret_cast<uint4*>(o + (size_t)a.u_lo * HP + 8 * q) = ul[q];
+          }
+      }
+      const float d = dec;
+      if (c + 1 < nc) fetch(c + 1);
+      wait_warp(&C.done[2], c & 1, dead, 10);
+      fence_after();
+      ld16(t_d + at, f);
+      wait_ld();
+#pragma unroll
+      for (int k = 0; k < 16; ++k) S[k] = in_n ? fmaf(d, S[k], f[k]) : 0.f;
+      fence_before();
+      if (c + 1 < nc) {
+        put_state(c + 1);
+        __syncthreads();
+      }
+    }
+    if (in_n) {
+      float* s1 = a.S + (size_t)a.seg_dst[seg] * slot + ((size_t)h * a.P + p0) * a.Np + i;
+#pragma unroll
+      for (int k = 0; k < 16; ++k)
+        if (k < width) s1[(size_t)k * a.Np] = S[k];
+    }
+  }
+  drain(C);
+  teardown(C, 128, a.status, 74);
+}
+
+}  // namespace rdelta
+}  // namespace sfb
+
+using namespace sfb;
+using namespace sfb::rdelta;
+
+extern "C" {
+
+// mk: rows of q | k | v, box 128 rows; mt, mt64: inv seen as [256 chunks H, 128], boxes of 128 and 64 rows.  N: a multiple of 16 up to 128; P: a
+// multiple of 8; first columns and stride multiples of 8.  The rows between N and Np of the stored states are not written.
+int sfb_rows_delta_tc(const void* mk, const void* mt, const void* mt64, const int* c_row0, const int* c_rows, const int* seg, const int* first, const int* seg_src,
+                      const int* seg_dst, const void* qkv, int64_t stride, const void* dt, int64_t dt_stride, const void* beta, int64_t beta_stride,
+                      const void* dt_bias, const void* la, void* S, void* rates, void* dec, void* inv, void* u, int u_lo, void* starts, int runs, int chunks, int H,
+                      int G, int N, int P, int Np, int q_col, int k_col, int v_col, float q_scale, float unit_eps, void* status, cudaStream_t stream) {
+  if (runs < 1 || runs > 65535 || chunks < 1 || chunks > 65535 || G < 1 || H % G || N < 16 || N % 16 || N > 128 || P < 8 || P % 8 || Np < N ||
+      (q_col | k_col | v_col) % 8 || stride % 8 || (uintptr_t)qkv % 16)
+    return (int)cudaErrorInvalidValue;
+  Args a{c_row0, c_rows, seg, first, seg_src, seg_dst, (const __nv_bfloat16*)qkv, stride, (const __nv_bfloat16*)dt, (const __nv_bfloat16*)beta, dt_stride,
+         beta_stride, (const float*)dt_bias, (const float*)la, (float*)S, (float*)rates, (float*)dec, (__nv_bfloat16*)inv, (__nv_bfloat16*)u,
+         (__nv_bfloat16*)starts, H, G, N, P, Np, (N + 63) / 64, 1, chunks, u_lo, q_col, k_col, v_col, q_scale, unit_eps, (Status*)status};
+  const int rep = H / G;
+  a.hpc = rep < 8 ? rep : 8;                 // heads that share a block's K K^T: fewer where that leaves SMs empty
+  while (a.hpc > 1 && (long long)G * ((rep + a.hpc - 1) / a.hpc) * chunks < 296) a.hpc = (a.hpc + 1) / 2;
+  static size_t granted[2] = {0, 0};
+  const size_t prep = (size_t)2 * SLAB + ((size_t)L * LD + 4 * L) * sizeof(float) + sizeof(Ctl), chain = (size_t)12 * SLAB + sizeof(Ctl);
+  cudaError_t rc = grant(delta_prep_kernel, prep, granted[0]);
+  if (rc == cudaSuccess) rc = grant(delta_chain_kernel, chain, granted[1]);
+  if (rc == cudaSuccess)
+    rc = sfb_launch(delta_prep_kernel, dim3(G * ((rep + a.hpc - 1) / a.hpc), chunks), dim3(WORK), prep, stream, *(const CUtensorMap*)mk, a);
+  if (rc == cudaSuccess)
+    rc = sfb_launch(delta_chain_kernel, dim3(H * ((P + PT - 1) / PT), runs), dim3(THREADS), chain, stream, *(const CUtensorMap*)mk, *(const CUtensorMap*)mt,
+                    *(const CUtensorMap*)mt64, a);
+  return (int)rc;
+}
+
+}  // extern "C"

@@ -13,14 +13,12 @@
 // Inputs are bf16.  Everything else that enters a product is a 32-bit value taken as two bf16 terms (16 mantissa bits): weighted scores,
 // weighted values, states, turned q and k.  Accumulators, decays, weights and states are 32-bit.  Every wait is bounded and reports
 // through the status word; no cluster, no multicast.
-#include "k_rows_tc.cuh"
+#include "k_rows_state_tc.cuh"
 
 namespace sfb {
 namespace rst {
-using namespace tc;
 
-constexpr int L = 128, SLAB = L * 128, HSLAB = 64 * 128;         // rows of a chunk; bytes of 128 / 64 rows of 64 elements
-constexpr int WORK = 256, THREADS = WORK + 32, HEADS = 8;        // threads that compute, and one warp that issues copies and products; most heads per block
+constexpr int HEADS = 8;         // most heads per block
 
 struct Args {
   const int *c_row0, *c_rows;      // chunks
@@ -33,22 +31,15 @@ struct Args {
   float* S;                        // [slots, H, P, Np]
   float* sums;                     // [chunks, H, P, Np]
   float* dec;                      // [chunks, H] decay over the whole chunk
-  float* rates;                    // [chunks, H, 2, 128] running sum of log2 a; the same less log2 of the weight
-  __nv_bfloat16* starts;           // [2, chunks, H, P, Np]: upper terms, then lower terms
+  float* rates;                    // [chunks, H, 2, 128] running sum of log2 a; the same less log2 of the weight; delta rule: see RATES
+  __nv_bfloat16* starts;           // [2, chunks, H, P, Np]: upper terms, then lower terms; delta rule: [2, chunks, H, N, P]
   __nv_bfloat16* y;                // [n, H P]
   int H, G, N, P, Np, ns, terms;   // ns: 64-element slabs of a q / k row
   int q_col, k_col, v_col;         // first columns in the maps
-  int q_lo, k_lo;                  // distance to the columns of the lower terms
+  int q_lo, k_lo;                  // distance to the columns of the lower terms; delta rule: to the rows of the values' lower terms (q_lo)
   int chunks, hpc;                 // hpc: heads per block
   int wide;                        // outputs lie on 32-byte boundaries
   Status* status;
-};
-
-struct Ctl {
-  uint64_t full[3], done[2];       // copies; products (chunk_out: weighted ones, scores - a barrier each, since the next head's scores are issued
-                                   // before every thread has seen the products end)
-  uint32_t tmem;
-  int dead;
 };
 
 // One warp, one head: running sums of log2 a over the chunk's rows (a lane takes four), weights; past the end: decay 1, weight 0.  The
@@ -80,49 +71,6 @@ __device__ __forceinline__ void head_rates(const Args& a, int chunk, int h, int 
   for (int k = 0; k < 4; ++k) c[k] -= __log2f(w[k]);       // weight 0: infinity, and its exponential below 0
   rows::store_v<float, 4>(out + L, c);
   if (lane == 0) a.dec[(size_t)chunk * a.H + h] = ex2(last);
-}
-
-__device__ __forceinline__ void setup(Ctl& C, uint32_t cols) {
-  if (threadIdx.x == 0) {
-    C.dead = 0;
-    for (int i = 0; i < 3; ++i) mbar_init(&C.full[i], 1);
-    for (int i = 0; i < 2; ++i) mbar_init(&C.done[i], 1);
-    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
-  }
-  if (threadIdx.x < 32) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&C.tmem)), "r"(cols) : "memory");
-    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
-  }
-  fence_before();
-  __syncthreads();
-  fence_after();
-}
-__device__ __forceinline__ void teardown(Ctl& C, uint32_t cols, Status* status, int where) {
-  fence_before();
-  __syncthreads();
-  if (threadIdx.x == 0 && C.dead) status_set(status, ST_TIMEOUT, where, C.dead, blockIdx.y << 16 | blockIdx.x);
-  if (threadIdx.x < 32) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(C.tmem), "r"(cols) : "memory");
-}
-
-// a wait of whole warps: what follows it is executed by all lanes together
-// `id`: what the status word says if the wait gives up.
-__device__ __forceinline__ void wait_warp(uint64_t* b, uint32_t parity, volatile int* dead, int id) {
-  if (!mbar_wait(b, parity, dead) && *dead == 1) *dead = id;
-  __syncwarp();
-}
-// sixteen values as one 32-byte store (a whole sector)
-__device__ __forceinline__ void store32(__nv_bfloat16* p, const float* f) {
-  uint32_t w[8];
-#pragma unroll
-  for (int i = 0; i < 8; ++i) { const __nv_bfloat162 t = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]); w[i] = *reinterpret_cast<const uint32_t*>(&t); }
-  asm volatile("st.global.v8.b32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(p), "r"(w[0]), "r"(w[1]), "r"(w[2]), "r"(w[3]), "r"(w[4]), "r"(w[5]), "r"(w[6]),
-               "r"(w[7]) : "memory");
-}
-// after a wait that gave up: copies and products under way must end before the CTA does (bounded: a phase that never comes is not waited for)
-__device__ __forceinline__ void drain(Ctl& C) {
-  if (!C.dead) return;
-  if (threadIdx.x == 0)
-    for (int i = 0; i < 100000; ++i) __nanosleep(64);
 }
 
 // grid (groups x parts of a group's heads, chunks): k stays in shared memory while the heads (and their tiles of 64 value dims) go by
@@ -275,17 +223,19 @@ __global__ void __launch_bounds__(256) chunk_starts_kernel(Args a) {
 }
 
 // grid as chunk_sums: q and k stay in shared memory while the heads go by; the scores are computed again for every head (their tensor
-// memory is where the weighted scores go)
-template <int NS, int TERMS>
+// memory is where the weighted scores go).  DELTA: one head per block; the values are u (two terms), the state lies with its N rows one after
+// another and takes k's place in shared memory once the scores are done; rows are scaled at the end.
+template <int NS, int TERMS, bool DELTA>
 __global__ void __launch_bounds__(THREADS, 2)
 chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mv,
                  const __grid_constant__ CUtensorMap ms, Args a) {
   extern __shared__ __align__(1024) uint8_t sm[];
   uint8_t* qs = sm;                                      // [terms][ns] slabs
   uint8_t* ks = qs + (size_t)TERMS * NS * SLAB;
-  uint8_t* vs = ks + (size_t)TERMS * NS * SLAB;      // one slab
-  uint8_t* ss = vs + SLAB;                               // start state, [2][ns] slabs of 64 rows
-  Ctl& C = *reinterpret_cast<Ctl*>(ss + (size_t)2 * NS * HSLAB);
+  uint8_t* vs = ks + (size_t)TERMS * NS * SLAB;      // one slab (DELTA: two)
+  uint8_t* ss = DELTA ? ks : vs + SLAB;                  // start state, [2][ns] slabs of 64 rows
+  Ctl& C = *reinterpret_cast<Ctl*>(DELTA ? vs + 2 * SLAB : ss + (size_t)2 * NS * HSLAB);
+  constexpr int RW = DELTA ? RATES : 2;
   setup(C, 256);
   pdl_launch_dependents();
   pdl_wait();
@@ -296,11 +246,16 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
   volatile int* dead = &C.dead;
   const uint32_t tp = C.tmem, ta = tp + 128, tb = tp + 192, lanes = (uint32_t)(w4 * 32) << 16;
   auto tile = [&](int it) {                              // values and start state of a tile of 64 value dims
-    const int h = h0 + it / pts, pt = it % pts, y = (chunk * a.H + h) * a.P + 64 * pt;
-    mbar_expect(&C.full[0], SLAB + 2 * NS * HSLAB);
+    const int h = h0 + it / pts, pt = it % pts;
+    mbar_expect(&C.full[0], (DELTA ? 2 : 1) * SLAB + 2 * NS * HSLAB);
     tma2d(vs, &mv, a.v_col + h * a.P + 64 * pt, row0, &C.full[0]);
+    if (DELTA) tma2d(vs + SLAB, &mv, a.v_col + h * a.P + 64 * pt, a.q_lo + row0, &C.full[0]);
+  };
+  auto state = [&](int it) {
+    const int h = h0 + it / pts, pt = it % pts, rows1 = DELTA ? a.N : a.P, y = (chunk * a.H + h) * rows1 + (DELTA ? 0 : 64 * pt);
     for (int t = 0; t < 2; ++t)
-      for (int s = 0; s < NS; ++s) tma2d(ss + (size_t)(t * NS + s) * HSLAB, &ms, 64 * s, t * a.chunks * a.H * a.P + y, &C.full[0]);
+      for (int s = 0; s < NS; ++s)
+        tma2d(ss + (size_t)(t * NS + s) * HSLAB, &ms, DELTA ? 64 * pt : 64 * s, t * a.chunks * a.H * rows1 + y + (DELTA ? 64 * s : 0), &C.full[0]);
   };
   const int kst = a.N / 16;
   const uint64_t lo = (uint64_t)NS * (SLAB >> 4), dq = desc(smem_u32(qs), 16), dk = desc(smem_u32(ks), 16);
@@ -326,30 +281,37 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
         tma2d(ks + (size_t)(t * NS + s) * SLAB, &mk, a.k_col + t * a.k_lo + g * a.N + 64 * s, row0, &C.full[2]);
       }
     tile(0);
+    if (!DELTA) state(0);
   }
   const int i = w4 * 32 + lane;
-  const float* rates = a.rates + ((size_t)chunk * a.H + h0) * 2 * L;
+  const float* rates = a.rates + ((size_t)chunk * a.H + h0) * RW * L;
   wait_warp(&C.full[2], 0, dead, 6);
   if (issuer) {
     // after every barrier of the workers below comes what it makes possible
     if (elect_one()) scores();
     __syncwarp();
+    if constexpr (DELTA) {
+      wait_warp(&C.done[1], 0, dead, 11);
+      if (elect_one()) state(0);
+      __syncwarp();
+    }
     for (int it = 0; it < items; ++it) {
       const bool next = it + 1 < items, head_ends = (it + 1) % pts == 0;
       wait_warp(&C.full[0], it & 1, dead, 7);
       __syncthreads();
       if (elect_one()) {
         fence_after();
-        const uint32_t ia = idesc(64, 0, 1), ib = idesc(64, 0, 0);
-        const uint64_t dv = desc(smem_u32(vs), SLAB), ds = desc(smem_u32(ss), 16), sl = (uint64_t)NS * (HSLAB >> 4);
+        const uint32_t ia = idesc(64, 0, 1), ib = idesc(64, 0, DELTA);
+        const uint64_t dv = desc(smem_u32(vs), SLAB), ds = desc(smem_u32(ss), DELTA ? SLAB : 16), sl = (uint64_t)NS * (HSLAB >> 4);
         // the two sums by turns: products on one accumulator follow each other slowly at this size
         auto weighted = [&](int t) {                     // eight steps of 16 rows with the upper terms, then with the lower ones
-          mma_ts(ta, tp + ((t & 7) >> 1) * 32 + (t & 1) * 8 + (t >> 3) * 16, dv + (uint64_t)(t & 7) * (2048 >> 4), ia, t ? 1u : 0u);
+          const int lower = t >> 3 & 1, vl = t >> 4;     // of the weights, of the values
+          mma_ts(ta, tp + ((t & 7) >> 1) * 32 + (t & 1) * 8 + lower * 16, dv + (uint64_t)vl * (SLAB >> 4) + (uint64_t)(t & 7) * (2048 >> 4), ia, t ? 1u : 0u);
         };
         constexpr int PER = 16 / (4 * NS);               // weighted products for every step of the other sum
 #pragma unroll
         for (int t = 0; t < 4 * NS; ++t) {
-          const uint64_t o = (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, os = (uint64_t)(t >> 2) * (HSLAB >> 4) + (t & 3) * 2;
+          const uint64_t o = (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, os = DELTA ? (uint64_t)t * (2048 >> 4) : (uint64_t)(t >> 2) * (HSLAB >> 4) + (t & 3) * 2;
           if (t < kst) mma_ss(tb, dq + o, ds + os, ib, t ? 1u : 0u);
           weighted(PER * t);
           if (t < kst) mma_ss(tb, dq + o, ds + sl + os, ib, 1u);
@@ -359,7 +321,7 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
           for (int u = 2; u < PER; ++u) weighted(PER * t + u);
         }
 #pragma unroll
-        for (int t = PER * 4 * NS; t < 16; ++t) weighted(t);
+        for (int t = PER * 4 * NS; t < (DELTA ? 24 : 16); ++t) weighted(t);
         commit(&C.done[0]);
       }
       __syncwarp();
@@ -367,19 +329,21 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
       if (next && elect_one()) {
         fence_after();
         tile(it + 1);
-        if (head_ends) scores();                         // of the next head
+        state(it + 1);
+        if (!DELTA && head_ends) scores();                         // of the next head
       }
       __syncwarp();
     }
   } else {
     float next_ci = rates[i], ei = 0.f;
+    const float scale = DELTA ? rates[2 * L + i] : 1.f;
     for (int it = 0; it < items; ++it) {
       const int hi = it / pts, h = h0 + hi, pt = it % pts;
       if (pt == 0) {
         const float ci = next_ci, D = a.D ? a.D[h] : 0.f;
-        const float* cs = rates + (size_t)hi * 2 * L + L;
+        const float* cs = rates + (size_t)hi * RW * L + L;
         ei = ex2(ci);
-        if (hi + 1 < nh) next_ci = rates[(size_t)(hi + 1) * 2 * L + i];
+        if (hi + 1 < nh) next_ci = rates[(size_t)(hi + 1) * RW * L + i];
         wait_warp(&C.done[1], hi & 1, dead, 9);
         fence_after();
         // Blocks of 32 columns: before the warp's diagonal block all are visible, after it none.  A thread's weights take the place of the
@@ -433,7 +397,7 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
         wait_ld();
         if (i < rows) {
 #pragma unroll
-          for (int k = 0; k < 16; ++k) x[k] = fmaf(ei, z[k], x[k]);
+          for (int k = 0; k < 16; ++k) x[k] = fmaf(ei, z[k], x[k]) * scale;
           if (a.wide && 16 * b + 16 <= cols) store32(o + 16 * b, x);
           else {
 #pragma unroll
@@ -493,15 +457,8 @@ __global__ void __launch_bounds__(256) state_turn_kernel(TurnArgs a) {
 }
 
 static size_t sums_smem(const Args& a) { return (size_t)(a.terms * 2 * ((a.ns + 1) / 2) + 3) * SLAB + a.hpc * L * sizeof(float) + sizeof(Ctl); }
-static size_t out_smem(const Args& a) { return (size_t)(2 * a.terms * a.ns + 1) * SLAB + (size_t)2 * a.ns * HSLAB + sizeof(Ctl); }
+static size_t out_smem(const Args& a, bool delta) { return (size_t)(2 * a.terms * a.ns + (delta ? 2 : 1)) * SLAB + (size_t)(delta ? 0 : 2 * a.ns * HSLAB) + sizeof(Ctl); }
 
-template <typename K>
-static cudaError_t grant(K kernel, size_t smem, size_t& granted) {
-  if (smem <= granted) return cudaSuccess;
-  const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  if (e == cudaSuccess) granted = smem;
-  return e;
-}
 template <int TERMS>
 static cudaError_t launch_sums(const CUtensorMap* k, const CUtensorMap* v, const Args& a, dim3 grid, cudaStream_t st) {
   static size_t granted = 0;
@@ -509,12 +466,12 @@ static cudaError_t launch_sums(const CUtensorMap* k, const CUtensorMap* v, const
   const cudaError_t e = grant(chunk_sums_kernel<TERMS>, smem, granted);
   return e != cudaSuccess ? e : sfb_launch(chunk_sums_kernel<TERMS>, grid, dim3(THREADS), smem, st, *k, *v, a);
 }
-template <int NS, int TERMS>
+template <int NS, int TERMS, bool DELTA = false>
 static cudaError_t launch_out(const CUtensorMap* q, const CUtensorMap* k, const CUtensorMap* v, const CUtensorMap* s, const Args& a, dim3 grid, cudaStream_t st) {
   static size_t granted = 0;
-  const size_t smem = out_smem(a);
-  const cudaError_t e = grant(chunk_out_kernel<NS, TERMS>, smem, granted);
-  return e != cudaSuccess ? e : sfb_launch(chunk_out_kernel<NS, TERMS>, grid, dim3(THREADS), smem, st, *q, *k, *v, *s, a);
+  const size_t smem = out_smem(a, DELTA);
+  const cudaError_t e = grant(chunk_out_kernel<NS, TERMS, DELTA>, smem, granted);
+  return e != cudaSuccess ? e : sfb_launch(chunk_out_kernel<NS, TERMS, DELTA>, grid, dim3(THREADS), smem, st, *q, *k, *v, *s, a);
 }
 
 }  // namespace rst
@@ -563,6 +520,20 @@ int sfb_rows_state_tc(const void* mq, const void* mk, const void* mv, const void
     case 3: return (int)launch_out<3, 1>(q, k, v, s, a, grid, stream);
     default: return (int)launch_out<4, 1>(q, k, v, s, a, grid, stream);
   }
+}
+
+// The outputs of the delta rule, after sfb_rows_delta_tc: mq, mk: rows of q / k, box 128 rows; mu: u seen as [2 x u_lo rows, H P], box 128
+// rows; ms: starts seen as [2 chunks H N, P], box 64 rows.  N: a multiple of 16 up to 128; P: a multiple of 8.
+int sfb_rows_delta_out(const void* mq, const void* mk, const void* mu, const void* ms, const int* c_row0, const int* c_rows, void* rates, void* starts, void* y,
+                       int chunks, int H, int G, int N, int P, int q_col, int k_col, int u_lo, void* status, cudaStream_t stream) {
+  if (chunks < 1 || chunks > 65535 || G < 1 || H % G || N % 16 || N < 16 || N > 128 || P % 8 || P < 8 || (q_col | k_col) % 8) return (int)cudaErrorInvalidValue;
+  Args a{};
+  a.c_row0 = c_row0; a.c_rows = c_rows; a.rates = (float*)rates; a.starts = (__nv_bfloat16*)starts; a.y = (__nv_bfloat16*)y; a.H = H; a.G = G; a.N = N; a.P = P;
+  a.ns = (N + 63) / 64; a.terms = 1; a.q_col = q_col; a.k_col = k_col; a.q_lo = u_lo; a.chunks = chunks; a.hpc = 1;
+  a.wide = (H * P) % 16 == 0 && P % 16 == 0 && (uintptr_t)y % 32 == 0; a.status = (Status*)status;
+  const dim3 grid(H, chunks);
+  const CUtensorMap *q = (const CUtensorMap*)mq, *k = (const CUtensorMap*)mk, *u = (const CUtensorMap*)mu, *s = (const CUtensorMap*)ms;
+  return (int)(a.ns == 1 ? launch_out<1, 1, true>(q, k, u, s, a, grid, stream) : launch_out<2, 1, true>(q, k, u, s, a, grid, stream));
 }
 
 }  // extern "C"

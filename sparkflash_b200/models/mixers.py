@@ -410,12 +410,29 @@ class DeltaState(MatrixState):
 
     def __init__(self, heads: int, groups: int, n: int, p: int, decay: torch.Tensor, dtype: torch.dtype, dt_bias):
         super().__init__(heads, groups, n, p, decay, dtype, dt_bias)
-        self.tc = False
+        self.tc = R.delta_tc_supports(dtype, n, p)
+
+    def reserve(self, e) -> None:
+        if self.tc:
+            chunks = e.state_chunks()
+            e.scratch.reserve("state_rates", chunks * self.H * R.DELTA_RATES * 128, torch.float32)
+            e.scratch.reserve("state_dec", chunks * self.H, torch.float32)
+            e.scratch.reserve("state_starts", 2 * chunks * self.H * self.P * self.N, torch.bfloat16)
+            e.scratch.reserve("delta_inv", chunks * self.H * 2 * 128 * 128, torch.bfloat16)
+            e.scratch.reserve("delta_u", 2 * e.max_rows * self.H * self.P, torch.bfloat16)
 
     def run(self, s, src, cols, dt, beta, S, y, conv=None) -> None:
-        q, k, v = (src[:, c:] for c in cols)
-        R.state_rows(q, k, v, dt, self.dt_bias, self.decay, None, None, 0, 1.0, s.row_pos, y, S, self.N, self.G, s.short_segs, s.nshort, s, conv,
-                     beta, self.N ** -0.5, self.UNIT_EPS)
+        """``src`` [n, stride] holds q, k, v from the columns ``cols`` on; ``conv``: they are the inputs of a convolution, see R.state_rows."""
+        scale = self.N ** -0.5
+        if s.nshort:
+            q, k, v = (src[:, c:] for c in cols)
+            R.state_rows(q, k, v, dt, self.dt_bias, self.decay, None, None, 0, 1.0, s.row_pos, y, S, self.N, self.G, s.short_segs, s.nshort, s, conv,
+                         beta, scale, self.UNIT_EPS)
+        if s.nlong:
+            buf = s.scratch.buf
+            u = s.scratch.get("delta_u", 2 * s.engine.max_rows, self.H * self.P)
+            R.delta_tc(src, cols, dt, beta, self.dt_bias, self.decay, S, buf["state_rates"], buf["state_dec"], buf["delta_inv"], u, buf["state_starts"], y,
+                       self.N, self.G, s, scale, self.UNIT_EPS, s.status)
 
 
 class DeltaMixer:

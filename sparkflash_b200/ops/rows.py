@@ -156,6 +156,30 @@ def state_tc(qk, qk_cols, v, v_col, dt, dt_bias, log_a, D, S, sums, dec, rates, 
                                          c_int(terms), c_int(qc), c_int(kc), c_int(v_col), c_int(ql), c_int(kl), _p(status), _stream()), "rows_state_tc")
 
 
+DELTA_RATES = 6           # numbers per (chunk, head) and row (csrc/k_rows_state_tc.cuh)
+
+
+def delta_tc_supports(dtype: torch.dtype, n: int, p: int) -> bool:
+    """Shapes the tensor-core arm of the delta rule takes (csrc/k_rows_delta_tc.cu)."""
+    return dtype == torch.bfloat16 and n % 16 == 0 and n <= 128 and p % 8 == 0
+
+
+def delta_tc(qkv, cols, dt, beta, dt_bias, log_a, S, rates, dec, inv, u, starts, y, N, groups, seg, q_scale, unit_eps, status):
+    """Long segments in chunks of 128 rows.  ``qkv``: [n, stride] tensor with q, k, v from the columns ``cols`` on.  Scratch of all chunks: rates,
+    dec (32-bit), inv [chunks, H, 2, 128, 128], starts [2, chunks, H, N, P] and u [2 x most rows, H P] in bf16."""
+    _, H, P, Np = S.shape
+    mqk, mu = tensor_map(qkv, qkv.shape[1], 128), tensor_map(u, H * P, 128)
+    mt, mt64, ms = tensor_map(inv, 128, 128), tensor_map(inv, 128, 64), tensor_map(starts, P, 64)
+    u_lo, at = u.shape[0] // 2, [c_int(c) for c in cols]
+    _check(_lib.rows().sfb_rows_delta_tc(mqk.ptr, mt.ptr, mt64.ptr, _p(seg.long_row0), _p(seg.long_rows), _p(seg.long_seg), _p(seg.long_first), _p(seg.seg_src),
+                                         _p(seg.seg_dst), *_strides(qkv), *_strides(dt), *_strides(beta), _p(dt_bias), _p(log_a), _p(S), _p(rates), _p(dec),
+                                         _p(inv), _p(u), c_int(u_lo), _p(starts), c_int(seg.nlong), c_int(seg.nchunks), c_int(H), c_int(groups), c_int(N),
+                                         c_int(P), c_int(Np), *at, c_float(q_scale), c_float(unit_eps), _p(status), _stream()), "rows_delta_tc")
+    _check(_lib.rows().sfb_rows_delta_out(mqk.ptr, mqk.ptr, mu.ptr, ms.ptr, _p(seg.long_row0), _p(seg.long_rows), _p(rates), _p(starts), _p(y),
+                                          c_int(seg.nchunks), c_int(H), c_int(groups), c_int(N), c_int(P), at[0], at[1], c_int(u_lo), _p(status),
+                                          _stream()), "rows_delta_out")
+
+
 STATE_PADS = tuple(range(32, 257, 32)) + (384, 512)
 
 
