@@ -1,0 +1,210 @@
+// Products of a mixture of experts on tcgen05, bf16: the tiles of k_rows_moe.cu's plan (up to 128 pairs of one expert) against that expert's
+// weights, 32-bit accumulators.
+//
+//   gated   act(x Wg^T, x Wu^T): 128 pairs x 128 gate columns beside their 128 up columns; the pairs' rows are gathered by TMA straight from the
+//           layer's input (four rows a copy); results in plan order
+//   down    128 pairs x 256 columns; rows in plan order; every result row goes to its [row][choice]
+//
+// Persistent: one CTA per SM takes every gridDim-th of the tiles x column blocks (the column blocks of a tile side by side, so that its rows
+// and its expert's weights stay in L2).  Warp 0 copies (K in steps of 64 through a ring of four stages), warp 1 issues the products, warps
+// 2-5 take the results out of tensor memory, where two accumulators of 256 columns take turns, so that a tile's results leave under the
+// next tile's products.  Every wait is bounded and reports through the status word; no cluster, no multicast.
+#include "k_rows_tc.cuh"
+
+namespace sfb {
+namespace rmoetc {
+using namespace tc;
+
+constexpr int THREADS = 192, ROWS = 128, COLS = 256, KS = 64, ST = 4, XSLAB = ROWS * 128, WSLAB = COLS * 128;
+
+struct Args {
+  const int *order, *tiles, *count;
+  __nv_bfloat16* out;        // gated: [pairs, M]; down: [n, slots, M]
+  int M, K, top, slots, cblocks;     // cblocks: blocks of 128 (gated) or 256 columns
+  int wide;                  // result rows lie on 16-byte boundaries
+  float alpha, limit;
+  Status* status;
+};
+
+struct Smem {
+  alignas(1024) uint8_t x[ST * XSLAB];
+  alignas(1024) uint8_t w[ST * WSLAB];
+  alignas(8) uint64_t full[ST], empty[ST], acc_full[2], acc_empty[2];
+  uint32_t tmem;
+  int dead;
+};
+
+// rows y[0..3] of the map, 64 columns from x on, one after another
+__device__ __forceinline__ void gather4(void* dst, const CUtensorMap* map, int x, int4 y, uint64_t* bar) {
+  asm volatile("cp.async.bulk.tensor.2d.shared::cta.global.tile::gather4.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4, %5, %6}], [%7];"
+               ::"r"(smem_u32(dst)), "l"(map), "r"(x), "r"(y.x), "r"(y.y), "r"(y.z), "r"(y.w), "r"(smem_u32(bar)) : "memory");
+}
+
+template <bool GATED>
+__global__ void __launch_bounds__(THREADS, 1)
+moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ CUtensorMap mw, Args a) {
+  extern __shared__ uint8_t raw[];
+  Smem& S = *reinterpret_cast<Smem*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
+  const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0), lane = tid & 31;
+  volatile int* dead = &S.dead;
+  if (tid == 0) {
+    S.dead = 0;
+    for (int i = 0; i < ST; ++i) { mbar_init(&S.full[i], 1); mbar_init(&S.empty[i], 1); }
+    for (int i = 0; i < 2; ++i) { mbar_init(&S.acc_full[i], 1); mbar_init(&S.acc_empty[i], 128); }
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
+  if (warp == 1) {
+    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], 512;" ::"r"(smem_u32(&S.tmem)) : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+  }
+  pdl_launch_dependents();
+  fence_before();
+  __syncthreads();
+  fence_after();
+  pdl_wait();
+  const uint32_t tmem = S.tmem;
+  const int total = *a.count * a.cblocks, steps = (a.K + KS - 1) / KS;
+  const int4* plan = reinterpret_cast<const int4*>(a.tiles);
+
+  if (warp == 0) {
+    int it = 0;              // stages filled so far
+    for (int b = blockIdx.x; b < total && !*dead; b += gridDim.x) {
+      const int4 t = plan[b / a.cblocks];
+      const int c0 = (b % a.cblocks) * (GATED ? 128 : 256);
+      int4 rows = make_int4(0, 0, 0, 0);      // a lane gathers four rows; past the tile's end its last one again
+      if (GATED) {
+        int* r = reinterpret_cast<int*>(&rows);
+#pragma unroll
+        for (int k = 0; k < 4; ++k) r[k] = a.order[t.y + min(lane * 4 + k, t.z - 1)] / a.top;
+      }
+      const int wrow = t.x * (GATED ? 2 : 1) * a.M + c0;
+      for (int k = 0; k < steps; ++k, ++it) {
+        const int st = it % ST, ph = (it / ST) & 1;
+        const bool ok = mbar_wait(&S.empty[st], ph ^ 1, dead);
+        if (!__all_sync(0xffffffffu, ok)) break;
+        if (lane == 0) mbar_expect(&S.full[st], XSLAB + WSLAB);
+        __syncwarp();
+        if (GATED) gather4(S.x + st * XSLAB + lane * 512, &mx, k * KS, rows, &S.full[st]);
+        if (lane == 0) {
+          if (!GATED) tma2d(S.x + st * XSLAB, &mx, k * KS, t.y, &S.full[st]);
+          tma2d(S.w + st * WSLAB, &mw, k * KS, wrow, &S.full[st]);
+          tma2d(S.w + st * WSLAB + XSLAB, &mw, k * KS, wrow + (GATED ? a.M : 128), &S.full[st]);
+        }
+      }
+    }
+    if (*dead && lane == 0) {       // copies still in flight must land before the CTA ends
+      for (int k = max(0, it - ST); k < it; ++k)
+        for (int i = 0; i < 100000 && !mbar_try(&S.full[k % ST], (k / ST) & 1); ++i) __nanosleep(64);
+    }
+  } else if (warp == 1) {
+    if (elect_one()) {
+      const uint32_t id = idesc(COLS, 0, 0);
+      const uint64_t dx = desc(smem_u32(S.x), 16), dw = desc(smem_u32(S.w), 16);
+      int it = 0, n = 0;
+      bool ok = true;
+      for (int b = blockIdx.x; ok && b < total; b += gridDim.x, ++n) {
+        const int acc = n & 1;
+        if (!(ok = mbar_wait(&S.acc_empty[acc], ((n >> 1) & 1) ^ 1, dead))) break;
+        fence_after();
+        for (int k = 0; k < steps; ++k, ++it) {
+          const int st = it % ST;
+          if (!(ok = mbar_wait(&S.full[st], (it / ST) & 1, dead))) break;
+          fence_after();
+          const uint64_t x = dx + (uint64_t)st * (XSLAB >> 4), w = dw + (uint64_t)st * (WSLAB >> 4);
+#pragma unroll
+          for (int q = 0; q < KS / 16; ++q) mma_ss(tmem + acc * COLS, x + q * 2, w + q * 2, id, (k | q) ? 1u : 0u);
+          commit(&S.empty[st]);
+        }
+        if (ok) commit(&S.acc_full[acc]);
+      }
+      // no arrival may be under way when the CTA ends
+      for (int k = max(0, it - ST); ok && k < it; ++k) ok = mbar_wait(&S.empty[k % ST], (k / ST) & 1, dead);
+    }
+  } else {
+    const int w4 = warp & 3, r = w4 * 32 + lane;      // tensor memory lanes of this warp
+    const uint32_t lanes = (uint32_t)(w4 * 32) << 16;
+    int n = 0;
+    for (int b = blockIdx.x; b < total; b += gridDim.x, ++n) {
+      const int4 t = plan[b / a.cblocks];
+      const int c0 = (b % a.cblocks) * (GATED ? 128 : 256), acc = n & 1;
+      const bool in = r < t.z;
+      size_t row = 0;
+      if (GATED) row = (size_t)(t.y + r);
+      else if (in) { const int pair = a.order[t.y + r]; row = (size_t)(pair / a.top) * a.slots + pair % a.top; }
+      __nv_bfloat16* o = a.out + row * a.M + c0;
+      const bool ok = mbar_wait(&S.acc_full[acc], (n >> 1) & 1, dead);
+      if (!__all_sync(0xffffffffu, ok)) break;
+      fence_after();
+      const uint32_t ta = tmem + acc * COLS + lanes;
+      const int width = min(GATED ? 128 : 256, a.M - c0);
+      for (int c = 0; c < width; c += 32) {
+        float f[32];
+        ld32(ta + c, f);
+        if constexpr (GATED) {
+          float u[32];
+          ld32(ta + 128 + c, u);
+          wait_ld();
+#pragma unroll
+          for (int k = 0; k < 32; ++k) f[k] = rows::gate_clamp<__nv_bfloat16>(f[k], u[k], a.alpha, a.limit);
+        } else {
+          wait_ld();
+        }
+        if (in) {
+          if (a.wide) {
+#pragma unroll
+            for (int k = 0; k < 32; k += 8)
+              if (c + k < width) rows::store_v<__nv_bfloat16, 8>(o + c + k, f + k);      // M is a multiple of eight
+          } else {
+#pragma unroll
+            for (int k = 0; k < 32; ++k)
+              if (c + k < width) o[c + k] = __float2bfloat16_rn(f[k]);
+          }
+        }
+      }
+      fence_before();
+      mbar_arrive(&S.acc_empty[acc]);
+    }
+  }
+  fence_before();
+  __syncthreads();
+  if (tid == 0 && *dead) status_set(a.status, ST_TIMEOUT, 75, blockIdx.x, GATED);
+  if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, 512;" ::"r"(tmem) : "memory");
+}
+
+template <bool GATED>
+static int launch(const CUtensorMap* mx, const CUtensorMap* mw, const Args& a, int most, cudaStream_t st) {
+  const size_t smem = sizeof(Smem) + 1024;
+  static bool done = false;
+  if (!done) {
+    const cudaError_t e = cudaFuncSetAttribute(moe_gemm_kernel<GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    done = true;
+  }
+  int dev = 0, sms = 148;
+  cudaGetDevice(&dev);
+  cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+  const long long blocks = (long long)most * a.cblocks;
+  return (int)sfb_launch(moe_gemm_kernel<GATED>, dim3((unsigned)(blocks < sms ? blocks : sms)), dim3(THREADS), smem, st, *mx, *mw, a);
+}
+
+}  // namespace rmoetc
+}  // namespace sfb
+
+using namespace sfb;
+using namespace sfb::rmoetc;
+
+extern "C" {
+
+// mx: gated: rows [n, K], box of one row (gathered); down: rows [pairs, K] in plan order, box 128 rows; mw: weights [E (2) M, K], box 128 rows.  K: a
+// multiple of 8; most: the most tiles (of up to 128 pairs) that the plan can hold.
+int sfb_rows_moe_gemm(const void* mx, const void* mw, const void* order, const void* tiles, const void* count, void* out, int most, int M, int K, int top, int slots,
+                      int gated, float alpha, float limit, void* status, cudaStream_t stream) {
+  if (most < 1 || M < 1 || K < 8 || K % 8 || top < 1) return (int)cudaErrorInvalidValue;
+  const int per = gated ? 128 : 256;
+  Args a{(const int*)order, (const int*)tiles, (const int*)count, (__nv_bfloat16*)out, M, K, top, slots, (M + per - 1) / per, M % 8 == 0 && (uintptr_t)out % 16 == 0,
+         alpha, limit, (Status*)status};
+  const CUtensorMap *x = (const CUtensorMap*)mx, *w = (const CUtensorMap*)mw;
+  return gated ? launch<true>(x, w, a, most, stream) : launch<false>(x, w, a, most, stream);
+}
+
+}  // extern "C"

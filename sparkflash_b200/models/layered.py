@@ -16,6 +16,7 @@ and writes no loop, cache or batching of its own (models/fanodra.py and models/g
 """
 from __future__ import annotations
 
+import gc
 import json
 import os
 import warnings
@@ -375,9 +376,14 @@ class LayeredEngine:
                 self._run(s, sample)
             self.launches[key] = sum(x not in ("linear", "block_gates", "head") for x in log.items)
             torch.cuda.current_stream().synchronize()
-            g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g):
-                self._run(s, sample)
+            g, collecting = torch.cuda.CUDAGraph(), gc.isenabled()
+            gc.disable()                  # the collector may not release another engine's graphs while this one is captured
+            try:
+                with torch.cuda.graph(g):
+                    self._run(s, sample)
+            finally:
+                if collecting:
+                    gc.enable()
             self.graphs[key] = g
         self.logits = self.scratch.get("logits", s.n, self.model.vocab)
         g.replay()

@@ -590,7 +590,8 @@ class MixtureFF:
 
     def reserve(self, e) -> None:
         n, dt, d = e.max_rows, self.router.dtype, self.router.shape[1]
-        self.tile = R.MOE_TILE
+        self.tc = R.moe_tc_supports(dt, d, self.ff)
+        self.tile = R.MOE_TC_TILE if self.tc else R.MOE_TILE
         e.scratch.reserve("moe_z", n * self.router.shape[0], torch.float32)
         e.scratch.reserve("moe_w", n * self.slots, torch.float32)
         for name, size in (("moe_ids", n * self.top), ("moe_order", n * self.top), ("moe_tiles", 4 * R.moe_tiles(n, self.E, self.top, self.tile)), ("moe_count", 4)):
@@ -616,8 +617,12 @@ class MixtureFF:
         plan = (s.scratch.get("moe_order", n * top), s.scratch.get("moe_tiles", R.moe_tiles(n, self.E, top, self.tile), 4), s.scratch.get("moe_count", 4),
                 R.moe_tiles(n, self.E, top, self.tile))
         R.moe_plan(ids, *plan[:3], self.E, self.tile)
-        R.moe_tile(h, self.w_in, act, plan, self.ff, top, slots, True, self.alpha, self.limit)
-        R.moe_tile(act, self.w_out, parts, plan, d, top, slots, False)
+        if self.tc:
+            R.moe_gemm(h, self.w_in, act, plan, self.ff, top, slots, True, s.status, self.alpha, self.limit)
+            R.moe_gemm(act, self.w_out, parts, plan, d, top, slots, False, s.status)
+        else:
+            R.moe_tile(h, self.w_in, act, plan, self.ff, top, slots, True, self.alpha, self.limit)
+            R.moe_tile(act, self.w_out, parts, plan, d, top, slots, False)
         if self.shared:
             R.gated_linear(h, self.s_in, s.scratch.get("proj", n, 2 * self.shared_ff), s_act, "clamp", self.alpha, self.shared_limit)
             R.linear(s_act, self.s_out, None, parts[:, top])

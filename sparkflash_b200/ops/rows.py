@@ -177,7 +177,7 @@ def delta_tc(qkv, cols, dt, beta, dt_bias, log_a, S, rates, dec, inv, u, starts,
                                          c_int(P), c_int(Np), *at, c_float(q_scale), c_float(unit_eps), _p(status), _stream()), "rows_delta_tc")
     _check(_lib.rows().sfb_rows_delta_out(mqk.ptr, mqk.ptr, mu.ptr, ms.ptr, _p(seg.long_row0), _p(seg.long_rows), _p(rates), _p(starts), _p(y),
                                           c_int(seg.nchunks), c_int(H), c_int(groups), c_int(N), c_int(P), at[0], at[1], c_int(u_lo), _p(status),
-                                          _stream()), "rows_delta_out")
+                                          _stream()), "rows_delta_tc")
 
 
 STATE_PADS = tuple(range(32, 257, 32)) + (384, 512)
@@ -455,6 +455,19 @@ def moe_tile(x, w, out, plan, M, top, slots, gated, alpha=0.0, limit=0.0):
     order, tiles, count, most = plan
     _check(_lib.rows().sfb_rows_moe_tile(_p(x), _p(w), _p(out), _p(order), _p(tiles), _p(count), c_int(most), c_int(M), c_int(w.shape[2]), c_int(top),
                                          c_int(slots), c_int(gated), c_float(alpha), c_float(limit), _fp32(out), _stream()), "rows_moe_tile")
+
+
+def moe_tc_supports(dtype: torch.dtype, width: int, ff: int) -> bool:
+    """Shapes the tensor-core products take (csrc/k_rows_moe_tc.cu)."""
+    return dtype == torch.bfloat16 and width % 8 == 0 and ff % 8 == 0
+
+
+def moe_gemm(x, w, out, plan, M, top, slots, gated, status, alpha=0.0, limit=0.0):
+    """``moe_tile`` on the tensor cores (tiles of up to 128 pairs); x, w and out in bf16."""
+    order, tiles, count, most = plan
+    mx, mw = tensor_map(x, x.shape[1], 1 if gated else 128), tensor_map(w, w.shape[2], 128)
+    _check(_lib.rows().sfb_rows_moe_gemm(mx.ptr, mw.ptr, _p(order), _p(tiles), _p(count), _p(out), c_int(most), c_int(M), c_int(w.shape[2]), c_int(top),
+                                         c_int(slots), c_int(gated), c_float(alpha), c_float(limit), _p(status), _stream()), "rows_moe_gemm")
 
 
 def moe_gemv_takes(x: torch.Tensor, ff: int, shared_ff: int) -> bool:

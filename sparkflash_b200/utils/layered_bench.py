@@ -1,7 +1,7 @@
-"""Throughput of a layered decoder (models/fanodra.py, models/gudutar.py) at sizes that resemble a real model's layers, per-kernel
-roofline fractions, and the same for the closest model of the package: for Fanodra the hybrid decoder of models/qwen.py (linear
+"""Throughput of a layered decoder (models/fanodra.py, models/gudutar.py, models/lifulorn.py) at sizes that resemble a real model's layers,
+per-kernel roofline fractions, and the same for the closest model of the package: for Fanodra the hybrid decoder of models/qwen.py (linear
 attention three layers in four, softmax attention in the fourth), for Gudutar the Fanodra of the same width, head size, feed-forward
-width and number of layer runs.  ``python bench.py --design NAME`` prints it as one JSON line.
+width and number of layer runs, for Lifulorn the Gudutar of the same width, number of layers, head size and active feed-forward width.  ``python bench.py --design NAME`` prints it as one JSON line.
 
 Everything is timed on the device with CUDA events after warm-up; inputs are larger than L2, or L2 is flushed in between.
 """
@@ -11,9 +11,10 @@ import statistics
 
 import torch
 
-from ..models import fanodra, gudutar
+from ..models import fanodra, gudutar, lifulorn
 from ..models.fanodra import FanodraConfig
 from ..models.gudutar import GudutarConfig
+from ..models.lifulorn import LifulornConfig
 from ..models.layered import LayeredEngine
 from . import roofline
 
@@ -54,7 +55,29 @@ def gudutar_config(name: str) -> GudutarConfig:
                                                                             for t in (ORDER[i % 4] for i in range(runs))]})
 
 
-CONFIGS = {"fanodra": (fanodra_config, fanodra.Fanodra, fanodra.random_tensors), "gudutar": (gudutar_config, gudutar.Gudutar, gudutar.random_tensors)}
+EXPERTS, TOP, SIDE = 32, 4, 128
+RULES = ("delta", "attention", "delta", "attention_2")
+
+
+def lifulorn_config(name: str) -> LifulornConfig:
+    """As many layers as the Gudutar of that size; the delta rule with a head of 128 x 128 per 128 of the width, attention with the Gudutar's heads
+    and window.  Every row uses TOP of EXPERTS experts and the shared one, together as wide as the other design's feed-forward."""
+    w, _, H, G, dim, _, _, _, ff, vocab, _ = SIZES[name]
+    each = ff // (TOP + 2)
+    mlp = {"kind": "moe", "router": {"experts": EXPERTS, "top": TOP}, "expert": {"ff": each, "limit": 7.0}, "shared": {"ff": ff - TOP * each, "limit": 7.0}}
+    att = {"heads": H, "kv_heads": G, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": WINDOW}, "v_mix": True}
+    wave = {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 4096}
+    yarn = {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    mixers = {"delta": {"heads": w // dim, "kv_heads": w // dim, "dim": dim, "vdim": dim, "conv": 4},
+              "attention": {**att, "rot": {"base": 500000.0, "dims": dim, "scaling": wave}},
+              "attention_2": {**att, "softcap": 50.0, "rot": {"base": 500000.0, "dims": dim, "scaling": yarn}}}
+    return LifulornConfig.from_dict({"architecture": "Lifulorn", "name": f"lifulorn-{name}", "vocab": vocab, "width": w, "norm": {"eps": 1e-6},
+                                     "residual_mult": 0.5, "token_side": {"dim": SIDE},
+                                     "layers": [{"type": t, "mixer": mixers[t], "mlp": mlp} for t in (RULES[i % 4] for i in range(len(gudutar_config(name).layers)))]})
+
+
+CONFIGS = {"fanodra": (fanodra_config, fanodra.Fanodra, fanodra.random_tensors), "gudutar": (gudutar_config, gudutar.Gudutar, gudutar.random_tensors),
+           "lifulorn": (lifulorn_config, lifulorn.Lifulorn, lifulorn.random_tensors)}
 
 
 def engine(design: str, name: str, lanes: int, context: int, rows: int) -> LayeredEngine:
@@ -188,6 +211,73 @@ def gudutar_work(cfg: GudutarConfig, n: int, ctx: int, head_rows: int, decode: b
     return out
 
 
+def lifulorn_work(cfg: LifulornConfig, n: int, ctx: int, head_rows: int, decode: bool) -> dict[str, roofline.ClassWork]:
+    """The same accounting for Lifulorn.  Delta rule: as the other recurrences, the chunked products (with the inverse of every chunk's triangle) once
+    per pair of bf16 terms; experts: the weights of those that the rows can touch, and their products."""
+    d, W, side = cfg.width, roofline.ClassWork, cfg.side_dim
+    out = {k: W() for k in ("rows_seam", "rows_conv", "rows_state", "rows_delta_tc", "rows_gated_norm", "rows_rot_append", "rows_attn_stream", "rows_attn_tc",
+                            "rows_act_mul", "rows_token_gate", "rows_moe_gemm", "rows_moe_gemv", "rows_moe_route", "rows_moe_plan", "linear", "router", "head")}
+    few = n <= 4
+
+    def linear(k, m, name="linear"):
+        out[name].flops += 2.0 * n * k * m
+        out[name].bytes += 2.0 * (k * m + n * (k + m))
+    out["rows_seam"].bytes += n * d * 8.0
+    for L in cfg.layers:
+        m, H, G = L.mixer, L.mixer["heads"], L.mixer["kv_heads"]
+        dim, vdim = m["dim"], m["vdim"]
+        inner = H * vdim
+        linear(inner, d)
+        if L.type == "delta":
+            cols = 2 * G * dim + inner
+            linear(d, cols + inner + 2 * H)
+            segs, nbytes = n if decode else 1, 2.0 * n * (cols + 2 * H + inner)
+            if decode:
+                out["rows_state"].bytes += segs * H * dim * vdim * 8.0 + nbytes
+            else:
+                # visible halves of k k^T and q k^T, the inverse (a third of a full product, 32-bit: as three), then per value dim: K S and Q S, inverse X
+                # and weights U (visible halves, three products), K^T U; two products where one operand has two terms
+                out["rows_delta_tc"].bytes += segs * H * dim * vdim * 8.0 + nbytes
+                out["rows_delta_tc"].flops += n * (G * 2 * 128.0 * dim + H * (3 * 2 * 128.0 * 128 / 6 + vdim * (3 * 4.0 * dim + 2 * 3 * 128.0)))
+                out["rows_conv"].bytes += 4.0 * n * cols
+            if decode and n > 4:
+                out["rows_conv"].bytes += 4.0 * n * cols
+            out["rows_gated_norm"].bytes += 6.0 * n * inner
+        else:
+            cols, win = H * dim + G * (dim + vdim), min(m["mask"]["size"], ctx)
+            linear(d, cols)
+            out["rows_rot_append"].bytes += 4.0 * n * cols
+            if decode:
+                out["rows_attn_stream"].bytes += 2.0 * n * (win * G * (dim + vdim) + H * (dim + vdim))
+            else:
+                seen, keys = n * win if ctx - n >= win else n * (ctx - n) + n * (n + 1) / 2, n + min(ctx - n, win - 1)
+                out["rows_attn_tc"].flops += 2.0 * H * seen * (dim + vdim)
+                out["rows_attn_tc"].bytes += 2.0 * (n * H * (dim + vdim) + keys * G * (dim + vdim))
+        out["rows_seam"].bytes += n * d * 12.0
+        if L.mlp is not None:
+            E, top, ff, sff = L.mlp["router"]["experts"], L.mlp["router"]["top"], L.mlp["expert"]["ff"], L.mlp["shared"]["ff"]
+            used = E * (1 - (1 - top / E) ** n)              # experts that n rows touch, on average
+            linear(d, E + 1, "router")
+            out["rows_moe_route"].bytes += n * (4.0 * E + 8.0 * top)
+            out["rows_moe_plan"].bytes += n * top * 16.0
+            if few:
+                out["rows_moe_gemv"].bytes += 2.0 * 3 * d * (n * top * ff + sff)
+            else:
+                out["rows_moe_gemm"].bytes += 2.0 * (used * 3 * d * ff + n * (d + top * (2 * ff + d)))
+                out["rows_moe_gemm"].flops += 2.0 * n * top * 3 * d * ff
+                linear(d, 2 * sff)
+                linear(sff, d)
+                out["rows_act_mul"].bytes += n * sff * 6.0
+            out["rows_seam"].bytes += n * d * (10.0 + 2.0 * (top + 1))
+        linear(d, side)
+        linear(side, d)
+        out["rows_token_gate"].bytes += n * side * 6.0
+        out["rows_seam"].bytes += n * d * 12.0
+    out["head"].flops += 2.0 * head_rows * cfg.vocab * d
+    out["head"].bytes += 2.0 * cfg.vocab * d
+    return out
+
+
 def fanodra_work(cfg: FanodraConfig, n: int, ctx: int, head_rows: int, decode: bool) -> dict[str, roofline.ClassWork]:
     """Bytes that must move and FLOPs that must be done by a step of n rows that ends at ``ctx`` cached positions (prefill: one
     segment; decode: one row in each of n lanes), per launch name."""
@@ -255,7 +345,8 @@ def _fractions(timings: list[list[tuple[str, float]]], wk: dict[str, roofline.Cl
     return out
 
 
-WORK = {"fanodra": fanodra_work, "gudutar": gudutar_work}
+WORK = {"fanodra": fanodra_work, "gudutar": gudutar_work, "lifulorn": lifulorn_work}
+CLOSEST = {"gudutar": "fanodra", "lifulorn": "gudutar"}
 
 
 def kernel_table(design: str, name: str, rows: int = 4096, ctx: int = 8192, reps: int = 5) -> list[dict]:
@@ -289,7 +380,7 @@ def decode_table(design: str, name: str, n: int = 16, ctx: int = 8192, reps: int
     eng.close()
     wk = WORK[design](cfg, n, ctx, n, True)
     if n <= 4:           # the streaming products take the projections and the head, gate and up fused with their activation
-        wk["rows_gemv"] = roofline.ClassWork(wk["linear"].bytes + wk["head"].bytes, wk["linear"].flops + wk["head"].flops)
+        wk["rows_gemv"] = roofline.ClassWork(*(sum(getattr(wk[k], f) for k in ("linear", "head", "router") if k in wk) for f in ("bytes", "flops")))
     if design == "fanodra":
         wk["rows_attn_stream"] = wk["rows_attn"]
     return _fractions(ts[1:], wk)
@@ -360,6 +451,6 @@ def run(design: str, sizes: list[str], steps: int, compare: bool = True) -> dict
     for name in sizes:
         out[name] = measure(design, name, steps)
         if compare:
-            out[name]["closest_model"] = closest(name) if design == "fanodra" else measure("fanodra", name, steps)
+            out[name]["closest_model"] = closest(name) if design == "fanodra" else measure(CLOSEST[design], name, steps)
         torch.cuda.empty_cache()
     return out

@@ -118,7 +118,7 @@ def write_safetensors(path: str, tensors: dict[str, torch.Tensor], metadata: dic
         table["__metadata__"] = {k: str(v) for k, v in metadata.items()}
     for name, t in tensors.items():
         t = t.contiguous()
-        raw = t.view(torch.uint8).reshape(-1).numpy().tobytes() if t.numel() else b""
+        raw = t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b""
         table[name] = {"dtype": _NAME[t.dtype], "shape": list(t.shape), "data_offsets": [off, off + len(raw)]}
         off += len(raw)
         blobs.append(raw)

@@ -163,8 +163,12 @@ def route(z, top):
     return ids, e / e.sum()
 
 
-def mixture(w, p, m, h):
+def mixture(w, p, m, h, margins=None):
+    """``margins``: optional list that collects how far every row's last choice is ahead of the next expert."""
     z = h @ w[p + "router"].T
+    if margins is not None and m["router"]["top"] < z.shape[1]:
+        best = z.sort(descending=True).values
+        margins.append(best[:, m["router"]["top"] - 1] - best[:, m["router"]["top"]])
     y = torch.zeros_like(h)
     for t in range(h.shape[0]):
         ids, wt = route(z[t], m["router"]["top"])
@@ -181,22 +185,105 @@ def token_input(w, p, i, dim, x, tokens, eps):
     return unit_rms((gelu_tanh(x @ w[p + "side.gate"].T) * e) @ w[p + "side.proj"].T, eps) * w[p + "side.norm"]
 
 
-def layer(w, cfg, i, x, tokens, first):
+def layer(w, cfg, i, x, tokens, first, margins=None):
     L, eps, m, p = cfg["layers"][i], cfg["norm"]["eps"], cfg["residual_mult"], f"l{i}."
     h = unit_rms(x, eps) * w[p + "norm1"]
     y = delta(w, p + "mix.", L["mixer"], h, eps) if L["type"] == "delta" else attention(w, p + "mix.", L["mixer"], h, first)
     x = x + m * y * w[p + "ls1"]
     if L.get("mlp"):
-        x = x + m * mixture(w, p + "mlp.", L["mlp"], unit_rms(x, eps) * w[p + "norm2"]) * w[p + "ls2"]
+        x = x + m * mixture(w, p + "mlp.", L["mlp"], unit_rms(x, eps) * w[p + "norm2"], margins) * w[p + "ls2"]
     return x + m * token_input(w, p, i, cfg["token_side"]["dim"], x, tokens, eps)
 
 
-def forward(w, cfg, tokens, dtype=torch.float64, taps=None):
-    """Logits [T, vocab]; ``taps``: optional list that collects the residual after every layer."""
+def forward(w, cfg, tokens, dtype=torch.float64, taps=None, margins=None):
+    """Logits [T, vocab]; ``taps``: optional list that collects the residual after every layer; ``margins``: see mixture."""
     w, tokens, first = {k: v.to(dtype) for k, v in w.items()}, torch.tensor(tokens), []
     x = w["embed"][tokens]
     for i in range(len(cfg["layers"])):
-        x = layer(w, cfg, i, x, tokens, first)
+        x = layer(w, cfg, i, x, tokens, first, margins)
         if taps is not None:
             taps.append(x.clone())
     return (unit_rms(x, cfg["norm"]["eps"]) * w["final.norm"]) @ w["head"].T
+
+
+# ---- small random models ---------------------------------------------------------------------------------------------
+def wave(factor, low, high, original):
+    return {"factor": factor, "low": low, "high": high, "original": original}
+
+
+def yarn(factor, original, fast, slow):
+    return {"factor": factor, "original": original, "fast": fast, "slow": slow}
+
+
+def attend(heads, kv_heads, dim, vdim, window, base, dims, scaling, scale, v_mix=True, softcap=None, mlp=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "mask": {"size": window},
+         "rot": {"base": base, "dims": dims, "scaling": scaling}}
+    if v_mix is not None:
+        m["v_mix"] = v_mix
+    if softcap is not None:
+        m["softcap"] = softcap
+    return {"type": "attention" if softcap is None else "attention_2", "mixer": m, "mlp": mlp}
+
+
+def rule(heads, kv_heads, dim, vdim, conv, mlp=None):
+    return {"type": "delta", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}, "mlp": mlp}
+
+
+def moe(experts, top, ff, limit, shared_ff, shared_limit):
+    out = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff, "limit": limit}}
+    if shared_ff:
+        out["shared"] = {"ff": shared_ff, "limit": shared_limit}
+    return out
+
+
+def make_config(vocab, width, side, mult, layers, eps=1e-5):
+    return {"architecture": "Lifulorn", "vocab": vocab, "width": width, "norm": {"eps": eps}, "residual_mult": mult, "token_side": {"dim": side},
+            "layers": layers}
+
+
+def make_weights(cfg, seed=0):
+    """Random bf16 tensors; every norm weight, scale, bias, sink and share differs from 1 and 0, so that leaving one out shows."""
+    g = torch.Generator().manual_seed(seed)
+    w, d, side = {}, cfg["width"], cfg["token_side"]["dim"]
+
+    def put(name, *shape, s=None, mean=0.0):
+        w[name] = (mean + torch.randn(*shape, generator=g) * (shape[-1] ** -0.5 if s is None else s)).to(torch.bfloat16)
+
+    def expert(p, ff):
+        put(p + "gate", ff, d, s=1.5 * d ** -0.5); put(p + "up", ff, d, s=1.5 * d ** -0.5); put(p + "down", d, ff)
+    put("embed", cfg["vocab"], d, s=1.0)
+    put("head", cfg["vocab"], d)
+    put("final.norm", d, s=0.3, mean=1.0)
+    put("side.embed", cfg["vocab"], side * len(cfg["layers"]), s=1.0)
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        q, H, G, dim, vdim = p + "mix.", m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        for n in ("norm1", "ls1", "side.norm"):
+            put(p + n, d, s=0.3, mean=1.0)
+        put(p + "side.gate", side, d); put(p + "side.proj", d, side)
+        put(q + "o", d, H * vdim)
+        if L["type"] == "delta":
+            for n, rows in (("q", G * dim), ("k", G * dim), ("v", H * vdim)):
+                put(q + n, rows, d)
+                put(q + n + ".conv", rows, m["conv"], s=0.6)
+            put(q + "g", H * vdim, d); put(q + "a", H, d); put(q + "b", H, d)
+            put(q + "norm", vdim, s=0.3, mean=1.0)
+            put(q + "dt_bias", H, s=1.0, mean=-2.0)
+            put(q + "A_log", H, s=1.0, mean=-1.0)      # decays from a few tokens to hundreds
+        else:
+            for n, rows in (("q", H * dim), ("k", G * dim), ("v", G * vdim)):
+                put(q + n, rows, d, s=(1.5 if n == "q" else 1.0) * d ** -0.5)
+                put(q + n + ".b", rows, s=0.3)
+            put(q + "sink", H, s=1.0, mean=1.0)
+            if m.get("v_mix"):
+                w[q + "vmix"] = torch.tensor(0.2 + 0.6 * float(torch.rand(1, generator=g))).to(torch.bfloat16)
+        if L.get("mlp"):
+            r = L["mlp"]
+            put(p + "norm2", d, s=0.3, mean=1.0); put(p + "ls2", d, s=0.3, mean=1.0)
+            put(p + "mlp.router", r["router"]["experts"], d, s=2 * d ** -0.5)
+            for e in range(r["router"]["experts"]):
+                expert(f"{p}mlp.e{e}.", r["expert"]["ff"])
+            if r.get("shared"):
+                expert(p + "mlp.shared.", r["shared"]["ff"])
+                put(p + "mlp.shared.sg", 1, d)
+    return w
