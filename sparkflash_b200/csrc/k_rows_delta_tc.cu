@@ -47,48 +47,32 @@ struct Args {
 
 constexpr int LD = 132;            // row stride of the matrix that is inverted
 
-// One warp, one head: running sums of log2 of the decays (a lane takes four rows; past the end: decay 1), and the numbers of the rows from
-// k's and q's factors to unit length.  c and the write strengths (0 past the end) also to `cs` and `bs`.
-__device__ __forceinline__ void head_rates(const Args& a, int chunk, int h, int row0, int rows, const float* rk, const float* rq, float* cs, float* bs) {
+// One warp, one head: running sums of log2 of the decays (a lane takes four rows; past the end: decay 1) and write strengths (past the end: 0).
+__device__ __forceinline__ void head_rates(const Args& a, int chunk, int h, int row0, int rows, float* cs, float* bs) {
   const int lane = threadIdx.x & 31;
   const float ah = a.a[h] * LOG2E, bias = a.dt_bias[h];
-  float c[4], b[4], t = 0.f;
+  float z[4], b[4], c[4], t = 0.f;
 #pragma unroll
   for (int k = 0; k < 4; ++k) {
-    const int i = lane * 4 + k;
-    float w = 0.f;
-    b[k] = 0.f;
-    if (i < rows) {
-      const float z = __bfloat162float(a.dt[(size_t)(row0 + i) * a.dt_stride + h]) + bias;
-      w = log1pf(expf(-fabsf(z))) + fmaxf(z, 0.f);
-      b[k] = 1.f / (1.f + expf(-__bfloat162float(a.beta[(size_t)(row0 + i) * a.beta_stride + h])));
-    }
-    t += ah * w;
+    const int i = min(lane * 4 + k, rows - 1);
+    z[k] = __bfloat162float(a.dt[(size_t)(row0 + i) * a.dt_stride + h]) + bias;
+    b[k] = __bfloat162float(a.beta[(size_t)(row0 + i) * a.beta_stride + h]);
+  }
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const bool in = lane * 4 + k < rows;
+    b[k] = in ? 1.f / (1.f + expf(-b[k])) : 0.f;
+    t += in ? ah * (log1pf(expf(-fabsf(z[k]))) + fmaxf(z[k], 0.f)) : 0.f;
     c[k] = t;
   }
   float s = t;
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) { const float v = __shfl_up_sync(0xffffffffu, s, o); if (lane >= o) s += v; }
   const float last = __shfl_sync(0xffffffffu, s, 31), before = s - t;
-  float* out = a.rates + ((size_t)chunk * a.H + h) * RATES * L + lane * 4;
-  float x[RATES][4];
 #pragma unroll
-  for (int k = 0; k < 4; ++k) {
-    const int i = lane * 4 + k;
-    c[k] += before;
-    cs[i] = c[k];
-    bs[i] = b[k];
-    const bool in = i < rows;
-    const float f = rk[i];
-    x[0][k] = c[k];
-    x[1][k] = in ? c[k] - __log2f(f) : INFINITY;         // its exponential: 0
-    x[2][k] = rq[i];
-    x[3][k] = in ? ex2(c[k]) * f : 0.f;
-    x[4][k] = b[k];
-    x[5][k] = in ? ex2(last - c[k]) * f : 0.f;
-  }
-#pragma unroll
-  for (int r = 0; r < RATES; ++r) rows::store_v<float, 4>(out + r * L, x[r]);
+  for (int k = 0; k < 4; ++k) c[k] += before;
+  rows::store_v<float, 4>(cs + lane * 4, c);
+  rows::store_v<float, 4>(bs + lane * 4, b);
   if (lane == 0) a.dec[(size_t)chunk * a.H + h] = ex2(last);
 }
 
@@ -113,21 +97,21 @@ __device__ __forceinline__ void micro(float (&acc)[4][4], const float* x, const 
   }
 }
 
-// The block below a pair of inverted diagonal blocks of B rows at `b0`: -T22 (A21 T11), by B x B / 16 threads (`t` counts them).
-// `w`: B x (B + 4) floats.  Two calls, a barrier in between: the inner product, then the outer one.
+// The block below a pair of inverted diagonal blocks of B rows at `b0`: -T22 (A21 T11).  A warp takes 16 rows (from `r0`) x 32 columns (from
+// `c0`), four by four a thread.  `w`: B x (B + 4) floats.  Two calls, a barrier in between: the inner product, then the outer one.
 template <int B>
-__device__ __forceinline__ void pair_inner(const float* A, float* w, int b0, int t) {
-  const int r = t / (B / 4) * 4, c = t % (B / 4) * 4;
+__device__ __forceinline__ void pair_inner(const float* A, float* w, int b0, int r0, int c0) {
+  const int r = r0 + (threadIdx.x >> 3 & 3) * 4, c = c0 + (threadIdx.x & 7) * 4;
   float acc[4][4] = {};
-  micro(acc, A + (b0 + B + r) * LD + b0, A + b0 * LD + b0 + c, LD, c, B);      // T11 is lower triangular
+  micro(acc, A + (b0 + B + r) * LD + b0, A + b0 * LD + b0 + c, LD, c0, B);      // T11 is lower triangular
 #pragma unroll
   for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(w + (r + i) * (B + 4) + c) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
 }
 template <int B>
-__device__ __forceinline__ void pair_outer(float* A, const float* w, int b0, int t) {
-  const int r = t / (B / 4) * 4, c = t % (B / 4) * 4;
+__device__ __forceinline__ void pair_outer(float* A, const float* w, int b0, int r0, int c0) {
+  const int r = r0 + (threadIdx.x >> 3 & 3) * 4, c = c0 + (threadIdx.x & 7) * 4;
   float acc[4][4] = {};
-  micro(acc, A + (b0 + B + r) * LD + b0 + B, w + c, B + 4, 0, r + 4);
+  micro(acc, A + (b0 + B + r) * LD + b0 + B, w + c, B + 4, 0, r0 + 16);
 #pragma unroll
   for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(A + (b0 + B + r + i) * LD + b0 + c) = make_float4(-acc[i][0], -acc[i][1], -acc[i][2], -acc[i][3]);
 }
@@ -138,9 +122,9 @@ __global__ void __launch_bounds__(WORK, 2) delta_prep_kernel(const __grid_consta
   uint8_t* ks = sm;                                       // k, two slabs; later the pairs' inner products
   float* w = reinterpret_cast<float*>(sm);
   float* A = reinterpret_cast<float*>(sm + 2 * SLAB);     // [128][LD]
-  float* rk = A + L * LD;                                 // [128] each
-  float *rq = rk + L, *cs = rq + L, *bs = cs + L;
-  Ctl& C = *reinterpret_cast<Ctl*>(bs + L);
+  float* rk = A + L * LD;                                 // [128] each: factors to unit length
+  float *rq = rk + L, *css = rq + L, *bss = css + a.hpc * L;      // [hpc][128]: running sums, write strengths
+  Ctl& C = *reinterpret_cast<Ctl*>(bss + a.hpc * L);
   setup(C, 128);
   pdl_launch_dependents();
   pdl_wait();
@@ -165,28 +149,55 @@ __global__ void __launch_bounds__(WORK, 2) delta_prep_kernel(const __grid_consta
     }
     __syncwarp();
   }
-  {   // a thread per row and vector: its factor to unit length
-    const int i = tid & (L - 1), isk = tid >> 7;
-    float s = 0.f;
-    if (i < rows) {
-      const __nv_bfloat16* p = a.qkv + (size_t)(row0 + i) * a.stride + (isk ? a.k_col : a.q_col) + g * a.N;
-      for (int n = 0; n < a.N; n += 8) {
-        float f[8];
-        rows::load_v<__nv_bfloat16, 8>(p + n, f);
+  for (int x = WORK / 32 - 1 - warp; x < nh; x += WORK / 32) head_rates(a, chunk, h0 + x, row0, rows, css + x * L, bss + x * L);
+  {   // eight lanes per row and vector: its factor to unit length
+    const int sub = lane & 7, words = a.N / 8;
+    uint4 v[8][2];
 #pragma unroll
-        for (int k = 0; k < 8; ++k) s = fmaf(f[k], f[k], s);
-      }
+    for (int t = 0; t < 8; ++t) {
+      const int rv = warp * 32 + t * 4 + (lane >> 3), i = rv & (L - 1);      // the first 128: q, then k
+      const uint4* p = reinterpret_cast<const uint4*>(a.qkv + (size_t)(row0 + min(i, rows - 1)) * a.stride + (rv >> 7 ? a.k_col : a.q_col) + g * a.N);
+#pragma unroll
+      for (int q = 0; q < 2; ++q) v[t][q] = sub + 8 * q < words ? p[sub + 8 * q] : make_uint4(0u, 0u, 0u, 0u);
     }
-    (isk ? rk : rq)[i] = (isk ? 1.f : a.q_scale) / sqrtf(s + a.unit_eps);
+#pragma unroll
+    for (int t = 0; t < 8; ++t) {
+      float s = 0.f;
+#pragma unroll
+      for (int q = 0; q < 2; ++q) {
+        const uint32_t x[4] = {v[t][q].x, v[t][q].y, v[t][q].z, v[t][q].w};
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const float f0 = __uint_as_float(x[k] << 16), f1 = __uint_as_float(x[k] & 0xffff0000u);
+          s = fmaf(f0, f0, s);
+          s = fmaf(f1, f1, s);
+        }
+      }
+      s += __shfl_xor_sync(0xffffffffu, s, 1);
+      s += __shfl_xor_sync(0xffffffffu, s, 2);
+      s += __shfl_xor_sync(0xffffffffu, s, 4);
+      const int rv = warp * 32 + t * 4 + (lane >> 3);
+      if (sub == 0) (rv >> 7 ? rk : rq)[rv & (L - 1)] = (rv >> 7 ? 1.f : a.q_scale) / sqrtf(s + a.unit_eps);
+    }
   }
   const int w4 = warp & 3, half = warp >> 2, i = w4 * 32 + lane;
   wait_warp(&C.done[0], 0, dead, 3);
   fence_after();
   for (int x = 0; x < nh; ++x) {
     const int h = h0 + x;
-    __syncthreads();                                      // factors are there; the matrix of the head before has been written out
-    if (warp == 0) head_rates(a, chunk, h, row0, rows, rk, rq, cs, bs);
-    __syncthreads();
+    const float *cs = css + x * L, *bs = bss + x * L;
+    __syncthreads();                                      // the numbers are there; the matrix of the head before has been written out
+    if (tid < L) {
+      float* o = a.rates + ((size_t)chunk * a.H + h) * RATES * L + tid;
+      const bool in = tid < rows;
+      const float c = cs[tid], f = rk[tid];
+      o[0] = c;
+      o[L] = in ? c - __log2f(f) : INFINITY;              // its exponential: 0
+      o[2 * L] = rq[tid];
+      o[3 * L] = in ? ex2(c) * f : 0.f;
+      o[4 * L] = bs[tid];
+      o[5 * L] = in ? ex2(cs[L - 1] - c) * f : 0.f;
+    }
     {
       const float ci = cs[i], bi = i < rows ? bs[i] * rk[i] : 0.f;
 #pragma unroll
@@ -198,12 +209,11 @@ __global__ void __launch_bounds__(WORK, 2) delta_prep_kernel(const __grid_consta
         wait_ld();
 #pragma unroll
         for (int q = 0; q < 8; ++q) {
-          float o[4];
+          float o[4], cj[4], rj[4];
+          rows::load_v<float, 4>(cs + j0 + 4 * q, cj);
+          rows::load_v<float, 4>(rk + j0 + 4 * q, rj);
 #pragma unroll
-          for (int k = 0; k < 4; ++k) {
-            const int j = j0 + 4 * q + k;
-            o[k] = j < i && i < rows ? s[4 * q + k] * bi * rk[j] * ex2(ci - cs[j]) : 0.f;
-          }
+          for (int k = 0; k < 4; ++k) o[k] = j0 + 4 * q + k < i && i < rows ? s[4 * q + k] * bi * rj[k] * ex2(ci - cj[k]) : 0.f;
           *reinterpret_cast<float4*>(A + i * LD + j0 + 4 * q) = make_float4(o[0], o[1], o[2], o[3]);
         }
       }
@@ -230,28 +240,29 @@ __global__ void __launch_bounds__(WORK, 2) delta_prep_kernel(const __grid_consta
       for (int r = 0; r < 32; ++r) B[r * LD + lane] = t[r];
     }
     __syncthreads();
-    if (tid < 128) pair_inner<32>(A, w + (tid >> 6) * 32 * 36, (tid >> 6) * 64, tid & 63);
+    if (warp < 4) pair_inner<32>(A, w + (warp >> 1) * 32 * 36, (warp >> 1) * 64, (warp & 1) * 16, 0);
     __syncthreads();
-    if (tid < 128) pair_outer<32>(A, w + (tid >> 6) * 32 * 36, (tid >> 6) * 64, tid & 63);
+    if (warp < 4) pair_outer<32>(A, w + (warp >> 1) * 32 * 36, (warp >> 1) * 64, (warp & 1) * 16, 0);
     else {            // the two blocks of 32 above the diagonal inside the blocks of 64
-      const int z = tid - 128, p = z >> 6, r = z & 63;
-      if (r < 32)
-        for (int c = 0; c < 32; c += 4) *reinterpret_cast<float4*>(A + (p * 64 + r) * LD + p * 64 + 32 + c) = make_float4(0.f, 0.f, 0.f, 0.f);
+      const int z = tid - 128, p = z >> 6, r = (z & 63) >> 1, c = (z & 1) * 16;
+#pragma unroll
+      for (int k = 0; k < 16; k += 4) *reinterpret_cast<float4*>(A + (p * 64 + r) * LD + p * 64 + 32 + c + k) = make_float4(0.f, 0.f, 0.f, 0.f);
     }
     __syncthreads();
-    pair_inner<64>(A, w, 0, tid);
+    pair_inner<64>(A, w, 0, (warp >> 1) * 16, (warp & 1) * 32);
     __syncthreads();
-    pair_outer<64>(A, w, 0, tid);
+    pair_outer<64>(A, w, 0, (warp >> 1) * 16, (warp & 1) * 32);
     __syncthreads();
     __nv_bfloat16* hi = a.inv + ((size_t)chunk * a.H + h) * 2 * L * L;
-    for (int r = warp; r < L; r += WORK / 32) {
-      if (r < 64 && lane >= 16) continue;
-      const float4 v = *reinterpret_cast<const float4*>(A + r * LD + lane * 4);
+#pragma unroll 4
+    for (int k = 0; k < 12; ++k) {       // a warp: two of the first 64 rows (their first half) at a time, then one of the others
+      const int r = k < 4 ? (warp * 4 + k) * 2 + (lane >> 4) : 64 + warp * 8 + k - 4, c = (k < 4 ? lane & 15 : lane) * 4;
+      const float4 v = *reinterpret_cast<const float4*>(A + r * LD + c);
       uint2 u, l;
       split2(v.x, v.y, u.x, l.x);
       split2(v.z, v.w, u.y, l.y);
-      *reinterpret_cast<uint2*>(hi + r * L + lane * 4) = u;
-      *reinterpret_cast<uint2*>(hi + (L + r) * L + lane * 4) = l;
+      *reinterpret_cast<uint2*>(hi + r * L + c) = u;
+      *reinterpret_cast<uint2*>(hi + (L + r) * L + c) = l;
     }
   }
   fence_before();
@@ -270,17 +281,17 @@ __device__ __forceinline__ void split16(const float* f, uint4 (&hi)[2], uint4 (&
 
 constexpr int PT = 32;             // value dims of a block
 
-// grid (heads x tiles of 32 value dims, runs).  Operands with the value dims along a row (state, X, U) are 128 rows of 128 bytes, of which the
-// tile takes the first 64 bytes.
+// grid (heads x tiles of 32 value dims, runs).  Operands with the value dims along a row (state, X, U) are 128 rows of 128 bytes: the upper terms
+// of the tile, then the lower ones, so that one product takes both (64 columns, whose halves are added up as they are read).
 __global__ void __launch_bounds__(THREADS, 1)
 delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mt, const __grid_constant__ CUtensorMap mt64, Args a) {
   extern __shared__ __align__(1024) uint8_t sm[];
   uint8_t* ks = sm;                                       // two stages of two slabs
   uint8_t* ts = ks + 4 * SLAB;                            // inverse: upper terms (two slabs), lower terms
-  uint8_t* ss = ts + 4 * SLAB;                            // state, two terms
-  uint8_t* xs = ss + 2 * SLAB;                            // X, then U, two terms
-  Ctl& C = *reinterpret_cast<Ctl*>(xs + 2 * SLAB);
-  setup(C, 128);
+  uint8_t* ss = ts + 4 * SLAB;                            // state
+  uint8_t* xs = ss + SLAB;                                // X, then U
+  Ctl& C = *reinterpret_cast<Ctl*>(xs + SLAB);
+  setup(C, 256);
   const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0), lane = tid & 31;
   // columns 64.. of the inverse's rows below 64 are zero and never loaded
   for (int x = tid; x < 2 * HSLAB / 16; x += THREADS)
@@ -293,7 +304,7 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
   const int run = blockIdx.y, seg = a.seg[run], c0 = a.first[run], nc = a.first[run + 1] - c0;
   const bool issuer = warp == WORK / 32;
   volatile int* dead = &C.dead;
-  const uint32_t t_ks = C.tmem, t_u = t_ks + PT, t_d = t_ks + 2 * PT;
+  const uint32_t t_ks = C.tmem, t_u = t_ks + 2 * PT, t_d = t_u + 2 * PT, t_l = t_d + 2 * PT;      // t_l: lower terms of the inverse
   if (issuer) {
     auto load_k = [&](int c) {
       mbar_expect(&C.full[c & 1], a.ns * SLAB);
@@ -313,8 +324,8 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
       if (nc > 1) load_k(1);
     }
     __syncwarp();
-    const uint32_t id = idesc(PT, 0, 1), idt = idesc(PT, 1, 1);
-    const uint64_t dt = desc(smem_u32(ts), 16), ds = desc(smem_u32(ss), SLAB), dx = desc(smem_u32(xs), SLAB), term = SLAB >> 4;
+    const uint32_t id = idesc(2 * PT, 0, 1), id1 = idesc(PT, 0, 1), idt = idesc(2 * PT, 1, 1);
+    const uint64_t dt = desc(smem_u32(ts), 16), ds = desc(smem_u32(ss), SLAB), dx = desc(smem_u32(xs), SLAB);
     const int kst = a.N / 16;
     for (int c = 0; c < nc; ++c) {
       const uint64_t dk = desc(smem_u32(ks) + (c & 1) * 2 * SLAB, 16), dkt = desc(smem_u32(ks) + (c & 1) * 2 * SLAB, SLAB);
@@ -325,7 +336,6 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
         for (int t = 0; t < kst; ++t) {
           const uint64_t ka = dk + (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, sb = ds + (uint64_t)t * (2048 >> 4);
           mma_ss(t_ks, ka, sb, id, t ? 1u : 0u);
-          mma_ss(t_ks, ka, sb + term, id, 1u);
         }
         commit(&C.done[0]);
       }
@@ -338,8 +348,7 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
         for (int t = 0; t < 8; ++t) {
           const uint64_t ta = dt + (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, xb = dx + (uint64_t)t * (2048 >> 4);
           mma_ss(t_u, ta, xb, id, t ? 1u : 0u);
-          mma_ss(t_u, ta, xb + term, id, 1u);
-          mma_ss(t_u, ta + 2 * term, xb, id, 1u);
+          mma_ss(t_l, ta + 2 * (SLAB >> 4), xb, id1, t ? 1u : 0u);
         }
         commit(&C.done[1]);
       }
@@ -354,7 +363,6 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
         for (int t = 0; t < 8; ++t) {
           const uint64_t o = (uint64_t)t * (2048 >> 4);
           mma_ss(t_d, dkt + o, dx + o, idt, t ? 1u : 0u);
-          mma_ss(t_d, dkt + o, dx + term + o, idt, 1u);
         }
         commit(&C.done[2]);
       }
@@ -376,21 +384,31 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
 #pragma unroll
       for (int k = 0; k < 16; ++k) S[k] = src >= 0 && in_n && k < width ? s0[(size_t)k * a.Np] : 0.f;
     }
-    auto put = [&](uint8_t* op, const uint4 (&hi)[2], const uint4 (&lo)[2]) {      // row i, both terms, 128-byte swizzle
+    auto put = [&](uint8_t* op, const uint4 (&hi)[2], const uint4 (&lo)[2]) {      // row i, 128-byte swizzle
 #pragma unroll
       for (int q = 0; q < 2; ++q) {
-        const int o = i * 128 + (((half * 2 + q) ^ (i & 7)) << 4);
-        *reinterpret_cast<uint4*>(op + o) = hi[q];
-        *reinterpret_cast<uint4*>(op + SLAB + o) = lo[q];
+        *reinterpret_cast<uint4*>(op + i * 128 + (((half * 2 + q) ^ (i & 7)) << 4)) = hi[q];
+        *reinterpret_cast<uint4*>(op + i * 128 + (((half * 2 + q + 4) ^ (i & 7)) << 4)) = lo[q];
       }
+      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+      fence_before();
+      __syncthreads();
     };
-    auto put_state = [&](int c) {
-      uint4 hi[2], lo[2];
+    auto read = [&](uint32_t t, float (&f)[16]) {                                   // the sum of both terms' products
+      float l[16];
+      ld16(t + at, f);
+      ld16(t + PT + at, l);
+      wait_ld();
+#pragma unroll
+      for (int k = 0; k < 16; ++k) f[k] += l[k];
+    };
+    uint4 hi[2], lo[2];
+    const size_t lower = (size_t)a.chunks * a.H * a.N * a.P;
+    auto put_state = [&](int c) {         // the copy for chunk_out leaves under the first product
       split16(S, hi, lo);
       put(ss, hi, lo);
       if (in_n) {
         __nv_bfloat16* o = a.starts + (((size_t)(c0 + c) * a.H + h) * a.N + i) * a.P + p0;
-        const size_t lower = (size_t)a.chunks * a.H * a.N * a.P;
 #pragma unroll
         for (int q = 0; q < 2; ++q)
           if (q * 8 < width) {
@@ -398,31 +416,27 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
             *reinterpret_cast<uint4*>(o + lower + 8 * q) = lo[q];
           }
       }
-      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
     };
     uint4 v[2];
     float ek, b, ue, dec;
-    int row, rows;
-    auto fetch = [&](int c) {
-      row = a.c_row0[c0 + c] + i;
-      rows = a.c_rows[c0 + c];
-      const float* r = a.rates + ((size_t)(c0 + c) * a.H + h) * RATES * L + i;
-      ek = r[3 * L]; b = r[4 * L]; ue = r[5 * L];
-      dec = a.dec[(size_t)(c0 + c) * a.H + h];
-      const __nv_bfloat16* p = a.qkv + (size_t)row * a.stride + a.v_col + (size_t)h * a.P + p0;
+    int row = a.c_row0[c0] + i, rows = a.c_rows[c0], row1 = 0, rows1 = 0;           // this chunk's, the next one's
+    auto fetch = [&](int c, int r, int m, float& e) {                               // numbers and values of chunk c
+      const float* n = a.rates + ((size_t)(c0 + c) * a.H + h) * RATES * L + i;
+      ek = n[3 * L]; b = n[4 * L]; e = n[5 * L];
+      const __nv_bfloat16* p = a.qkv + (size_t)r * a.stride + a.v_col + (size_t)h * a.P + p0;
 #pragma unroll
-      for (int q = 0; q < 2; ++q) v[q] = i < rows && q * 8 < width ? *reinterpret_cast<const uint4*>(p + 8 * q) : make_uint4(0u, 0u, 0u, 0u);
+      for (int q = 0; q < 2; ++q) v[q] = i < m && q * 8 < width ? *reinterpret_cast<const uint4*>(p + 8 * q) : make_uint4(0u, 0u, 0u, 0u);
     };
-    fetch(0);
+    fetch(0, row, rows, ue);
+    dec = a.dec[(size_t)c0 * a.H + h];
+    if (nc > 1) { row1 = a.c_row0[c0 + 1] + i; rows1 = a.c_rows[c0 + 1]; }
     put_state(0);
-    __syncthreads();
     for (int c = 0; c < nc; ++c) {
-      float f[16];
-      uint4 hi[2], lo[2];
+      float f[16], ue1 = 0.f, dec1 = 0.f;
+      int row2 = 0, rows2 = 0;
       wait_warp(&C.done[0], c & 1, dead, 8);
       fence_after();
-      ld16(t_ks + at, f);
-      wait_ld();
+      read(t_ks, f);
 #pragma unroll
       for (int q = 0; q < 2; ++q) {
         const uint32_t vw[4] = {v[q].x, v[q].y, v[q].z, v[q].w};
@@ -435,23 +449,27 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
       }
       split16(f, hi, lo);
       put(xs, hi, lo);
-      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-      fence_before();
-      __syncthreads();
+      if (c + 1 < nc) {                                   // requested under the product
+        fetch(c + 1, row1, rows1, ue1);
+        dec1 = a.dec[(size_t)(c0 + c + 1) * a.H + h];
+        if (c + 2 < nc) { row2 = a.c_row0[c0 + c + 2] + i; rows2 = a.c_rows[c0 + c + 2]; }
+      }
       wait_warp(&C.done[1], c & 1, dead, 9);
       fence_after();
-      ld16(t_u + at, f);
-      wait_ld();
+      {
+        float l[16];
+        ld16(t_l + at, l);
+        read(t_u, f);
+#pragma unroll
+        for (int k = 0; k < 16; ++k) f[k] += l[k];
+      }
       uint4 uh[2], ul[2];
       split16(f, uh, ul);
 #pragma unroll
       for (int k = 0; k < 16; ++k) f[k] = i < rows ? f[k] * ue : 0.f;
       split16(f, hi, lo);
       put(xs, hi, lo);
-      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-      fence_before();
-      __syncthreads();
-      if (i < rows) {                                     // under the product
+      if (i < rows) {                                     // u for chunk_out, under the product
         __nv_bfloat16* o = a.u + (size_t)row * HP + (size_t)h * a.P + p0;
 #pragma unroll
         for (int q = 0; q < 2; ++q)
@@ -460,19 +478,14 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
             *reinterpret_cast<uint4*>(o + (size_t)a.u_lo * HP + 8 * q) = ul[q];
           }
       }
-      const float d = dec;
-      if (c + 1 < nc) fetch(c + 1);
       wait_warp(&C.done[2], c & 1, dead, 10);
       fence_after();
-      ld16(t_d + at, f);
-      wait_ld();
+      read(t_d, f);
 #pragma unroll
-      for (int k = 0; k < 16; ++k) S[k] = in_n ? fmaf(d, S[k], f[k]) : 0.f;
-      fence_before();
-      if (c + 1 < nc) {
-        put_state(c + 1);
-        __syncthreads();
-      }
+      for (int k = 0; k < 16; ++k) S[k] = in_n ? fmaf(dec, S[k], f[k]) : 0.f;
+      if (c + 1 < nc) put_state(c + 1);
+      else fence_before();
+      ue = ue1; dec = dec1; row = row1; rows = rows1; row1 = row2; rows1 = rows2;
     }
     if (in_n) {
       float* s1 = a.S + (size_t)a.seg_dst[seg] * slot + ((size_t)h * a.P + p0) * a.Np + i;
@@ -482,7 +495,7 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
     }
   }
   drain(C);
-  teardown(C, 128, a.status, 74);
+  teardown(C, 256, a.status, 74);
 }
 
 }  // namespace rdelta
@@ -509,7 +522,7 @@ int sfb_rows_delta_tc(const void* mk, const void* mt, const void* mt64, const in
   a.hpc = rep < 8 ? rep : 8;                 // heads that share a block's K K^T: fewer where that leaves SMs empty
   while (a.hpc > 1 && (long long)G * ((rep + a.hpc - 1) / a.hpc) * chunks < 296) a.hpc = (a.hpc + 1) / 2;
   static size_t granted[2] = {0, 0};
-  const size_t prep = (size_t)2 * SLAB + ((size_t)L * LD + 4 * L) * sizeof(float) + sizeof(Ctl), chain = (size_t)12 * SLAB + sizeof(Ctl);
+  const size_t prep = (size_t)2 * SLAB + ((size_t)L * LD + (2 + 2 * a.hpc) * L) * sizeof(float) + sizeof(Ctl), chain = (size_t)10 * SLAB + sizeof(Ctl);
   cudaError_t rc = grant(delta_prep_kernel, prep, granted[0]);
   if (rc == cudaSuccess) rc = grant(delta_chain_kernel, chain, granted[1]);
   if (rc == cudaSuccess)

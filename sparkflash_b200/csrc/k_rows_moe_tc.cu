@@ -1,8 +1,8 @@
 // Products of a mixture of experts on tcgen05, bf16: the tiles of k_rows_moe.cu's plan (up to 128 pairs of one expert) against that expert's
 // weights, 32-bit accumulators.
 //
-//   gated   act(x Wg^T, x Wu^T): 128 pairs x 128 gate columns beside their 128 up columns; the pairs' rows are gathered by TMA straight from the
-//           layer's input (four rows a copy); results in plan order
+//   gated   act(x Wg^T, x Wu^T): 128 pairs x 128 gate columns beside their 128 up columns; results in plan order.  With few rows the pairs' rows
+//           are gathered by TMA straight from the layer's input (four rows a copy); many are brought into plan order first (`pick`)
 //   down    128 pairs x 256 columns; rows in plan order; every result row goes to its [row][choice]
 //
 // Persistent: one CTA per SM takes every gridDim-th of the tiles x column blocks (the column blocks of a tile side by side, so that its rows
@@ -40,7 +40,26 @@ __device__ __forceinline__ void gather4(void* dst, const CUtensorMap* map, int x
                ::"r"(smem_u32(dst)), "l"(map), "r"(x), "r"(y.x), "r"(y.y), "r"(y.z), "r"(y.w), "r"(smem_u32(bar)) : "memory");
 }
 
-template <bool GATED>
+// the layer's input rows in plan order, 16-byte words; a warp per pair
+__global__ void __launch_bounds__(256) moe_pick_kernel(const uint4* x, const int* order, uint4* out, int pairs, int top, int words) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int place = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (place >= pairs) return;
+  const uint4* src = x + (size_t)(order[place] / top) * words;
+  uint4* dst = out + (size_t)place * words;
+  for (int w = lane; w < words; w += 256) {
+    uint4 v[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k)
+      if (w + 32 * k < words) v[k] = src[w + 32 * k];
+#pragma unroll
+    for (int k = 0; k < 8; ++k)
+      if (w + 32 * k < words) dst[w + 32 * k] = v[k];
+  }
+}
+
+template <bool GATED, bool GATHER>
 __global__ void __launch_bounds__(THREADS, 1)
 moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ CUtensorMap mw, Args a) {
   extern __shared__ uint8_t raw[];
@@ -71,8 +90,8 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
     for (int b = blockIdx.x; b < total && !*dead; b += gridDim.x) {
       const int4 t = plan[b / a.cblocks];
       const int c0 = (b % a.cblocks) * (GATED ? 128 : 256);
-      int4 rows = make_int4(0, 0, 0, 0);      // a lane gathers four rows; past the tile's end its last one again
-      if (GATED) {
+      int4 rows = make_int4(0, 0, 0, 0);      // a lane gathers four rows, the tile's last one again past its end; lanes past it none
+      if (GATHER) {
         int* r = reinterpret_cast<int*>(&rows);
 #pragma unroll
         for (int k = 0; k < 4; ++k) r[k] = a.order[t.y + min(lane * 4 + k, t.z - 1)] / a.top;
@@ -82,11 +101,11 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
         const int st = it % ST, ph = (it / ST) & 1;
         const bool ok = mbar_wait(&S.empty[st], ph ^ 1, dead);
         if (!__all_sync(0xffffffffu, ok)) break;
-        if (lane == 0) mbar_expect(&S.full[st], XSLAB + WSLAB);
+        if (lane == 0) mbar_expect(&S.full[st], (GATHER ? (t.z + 3) / 4 * 512 : XSLAB) + WSLAB);
         __syncwarp();
-        if (GATED) gather4(S.x + st * XSLAB + lane * 512, &mx, k * KS, rows, &S.full[st]);
+        if (GATHER && lane * 4 < t.z) gather4(S.x + st * XSLAB + lane * 512, &mx, k * KS, rows, &S.full[st]);
         if (lane == 0) {
-          if (!GATED) tma2d(S.x + st * XSLAB, &mx, k * KS, t.y, &S.full[st]);
+          if (!GATHER) tma2d(S.x + st * XSLAB, &mx, k * KS, t.y, &S.full[st]);
           tma2d(S.w + st * WSLAB, &mw, k * KS, wrow, &S.full[st]);
           tma2d(S.w + st * WSLAB + XSLAB, &mw, k * KS, wrow + (GATED ? a.M : 128), &S.full[st]);
         }
@@ -171,12 +190,12 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
   if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, 512;" ::"r"(tmem) : "memory");
 }
 
-template <bool GATED>
+template <bool GATED, bool GATHER>
 static int launch(const CUtensorMap* mx, const CUtensorMap* mw, const Args& a, int most, cudaStream_t st) {
   const size_t smem = sizeof(Smem) + 1024;
   static bool done = false;
   if (!done) {
-    const cudaError_t e = cudaFuncSetAttribute(moe_gemm_kernel<GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const cudaError_t e = cudaFuncSetAttribute(moe_gemm_kernel<GATED, GATHER>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     done = true;
   }
@@ -184,7 +203,7 @@ static int launch(const CUtensorMap* mx, const CUtensorMap* mw, const Args& a, i
   cudaGetDevice(&dev);
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
   const long long blocks = (long long)most * a.cblocks;
-  return (int)sfb_launch(moe_gemm_kernel<GATED>, dim3((unsigned)(blocks < sms ? blocks : sms)), dim3(THREADS), smem, st, *mx, *mw, a);
+  return (int)sfb_launch(moe_gemm_kernel<GATED, GATHER>, dim3((unsigned)(blocks < sms ? blocks : sms)), dim3(THREADS), smem, st, *mx, *mw, a);
 }
 
 }  // namespace rmoetc
@@ -195,16 +214,23 @@ using namespace sfb::rmoetc;
 
 extern "C" {
 
-// mx: gated: rows [n, K], box of one row (gathered); down: rows [pairs, K] in plan order, box 128 rows; mw: weights [E (2) M, K], box 128 rows.  K: a
+// x [n, K] to out [pairs, K] in plan order; K a multiple of 8
+int sfb_rows_moe_pick(const void* x, const void* order, void* out, int pairs, int top, int K, cudaStream_t stream) {
+  if (pairs < 1 || top < 1 || K < 8 || K % 8) return (int)cudaErrorInvalidValue;
+  return (int)sfb_launch(moe_pick_kernel, dim3((pairs + 7) / 8), dim3(256), 0, stream, (const uint4*)x, (const int*)order, (uint4*)out, pairs, top, K / 8);
+}
+
+// mx: rows [pairs, K] in plan order, box 128 rows, or (gather) rows [n, K], box of one row; mw: weights [E (2) M, K], box 128 rows.  K: a
 // multiple of 8; most: the most tiles (of up to 128 pairs) that the plan can hold.
 int sfb_rows_moe_gemm(const void* mx, const void* mw, const void* order, const void* tiles, const void* count, void* out, int most, int M, int K, int top, int slots,
-                      int gated, float alpha, float limit, void* status, cudaStream_t stream) {
-  if (most < 1 || M < 1 || K < 8 || K % 8 || top < 1) return (int)cudaErrorInvalidValue;
+                      int gated, int gather, float alpha, float limit, void* status, cudaStream_t stream) {
+  if (most < 1 || M < 1 || K < 8 || K % 8 || top < 1 || (gather && !gated)) return (int)cudaErrorInvalidValue;
   const int per = gated ? 128 : 256;
   Args a{(const int*)order, (const int*)tiles, (const int*)count, (__nv_bfloat16*)out, M, K, top, slots, (M + per - 1) / per, M % 8 == 0 && (uintptr_t)out % 16 == 0,
          alpha, limit, (Status*)status};
   const CUtensorMap *x = (const CUtensorMap*)mx, *w = (const CUtensorMap*)mw;
-  return gated ? launch<true>(x, w, a, most, stream) : launch<false>(x, w, a, most, stream);
+  if (gather) return launch<true, true>(x, w, a, most, stream);
+  return gated ? launch<true, false>(x, w, a, most, stream) : launch<false, false>(x, w, a, most, stream);
 }
 
 }  // extern "C"

@@ -598,6 +598,8 @@ class MixtureFF:
             e.scratch.reserve(name, size, torch.int32)
         e.scratch.reserve("moe_act", n * self.top * self.ff, dt)
         e.scratch.reserve("moe_parts", n * self.slots * d, dt)
+        if self.tc and n > R.MOE_GATHER_ROWS:
+            e.scratch.reserve("moe_x", n * self.top * d, dt)
         if self.shared:
             e.scratch.reserve("proj", n * 2 * self.shared_ff, dt)
             e.scratch.reserve("ff_act", n * self.shared_ff, dt)
@@ -618,7 +620,11 @@ class MixtureFF:
                 R.moe_tiles(n, self.E, top, self.tile))
         R.moe_plan(ids, *plan[:3], self.E, self.tile)
         if self.tc:
-            R.moe_gemm(h, self.w_in, act, plan, self.ff, top, slots, True, s.status, self.alpha, self.limit)
+            few, x = n <= R.MOE_GATHER_ROWS, h
+            if not few:
+                x = s.scratch.get("moe_x", n * top, d)
+                R.moe_pick(h, plan[0], x, top)
+            R.moe_gemm(x, self.w_in, act, plan, self.ff, top, slots, True, s.status, self.alpha, self.limit, few)
             R.moe_gemm(act, self.w_out, parts, plan, d, top, slots, False, s.status)
         else:
             R.moe_tile(h, self.w_in, act, plan, self.ff, top, slots, True, self.alpha, self.limit)

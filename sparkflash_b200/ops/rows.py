@@ -462,12 +462,20 @@ def moe_tc_supports(dtype: torch.dtype, width: int, ff: int) -> bool:
     return dtype == torch.bfloat16 and width % 8 == 0 and ff % 8 == 0
 
 
-def moe_gemm(x, w, out, plan, M, top, slots, gated, status, alpha=0.0, limit=0.0):
-    """``moe_tile`` on the tensor cores (tiles of up to 128 pairs); x, w and out in bf16."""
+MOE_GATHER_ROWS = 256      # up to this many rows the product gathers its rows itself (csrc/k_rows_moe_tc.cu)
+
+
+def moe_pick(x, order, out, top):
+    """Rows x [n, K] in plan order: out [pairs, K]."""
+    _check(_lib.rows().sfb_rows_moe_pick(_p(x), _p(order), _p(out), c_int(out.shape[0]), c_int(top), c_int(x.shape[1]), _stream()), "rows_moe_pick")
+
+
+def moe_gemm(x, w, out, plan, M, top, slots, gated, status, alpha=0.0, limit=0.0, gather=False):
+    """``moe_tile`` on the tensor cores (tiles of up to 128 pairs); w and out in bf16; x in plan order, or ``gather``: the layer's rows."""
     order, tiles, count, most = plan
-    mx, mw = tensor_map(x, x.shape[1], 1 if gated else 128), tensor_map(w, w.shape[2], 128)
+    mx, mw = tensor_map(x, x.shape[1], 1 if gather else 128), tensor_map(w, w.shape[2], 128)
     _check(_lib.rows().sfb_rows_moe_gemm(mx.ptr, mw.ptr, _p(order), _p(tiles), _p(count), _p(out), c_int(most), c_int(M), c_int(w.shape[2]), c_int(top),
-                                         c_int(slots), c_int(gated), c_float(alpha), c_float(limit), _p(status), _stream()), "rows_moe_gemm")
+                                         c_int(slots), c_int(gated), c_int(gather), c_float(alpha), c_float(limit), _p(status), _stream()), "rows_moe_gemm")
 
 
 def moe_gemv_takes(x: torch.Tensor, ff: int, shared_ff: int) -> bool:
