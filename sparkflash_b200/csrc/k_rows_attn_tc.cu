@@ -384,9 +384,10 @@ using namespace sfb::rtc;
 
 extern "C" {
 
-// 2-D bf16 map over [rows, cols] (row stride in bytes, a multiple of 16) with a 128-byte swizzled box of 64 columns x box_rows; columns
-// past the row's end read as zero.  0, a CUresult, or -1 without the driver entry point.
-int sfb_rows_tmap(void* out_map, const void* base, int64_t rows, int64_t cols, int64_t row_bytes, int box_rows) {
+// 2-D bf16 map over [rows, cols] (row stride in bytes, a multiple of 16) with a box of 64 columns x box_rows, 128-byte swizzled, or of 32
+// columns, 64-byte swizzled; columns past the row's end read as zero and are not stored.  0, a CUresult, or -1 without the driver entry point.
+int sfb_rows_tmap(void* out_map, const void* base, int64_t rows, int64_t cols, int64_t row_bytes, int box_rows, int box_cols) {
+  if (box_cols != 64 && box_cols != 32) return (int)CUDA_ERROR_INVALID_VALUE;
   static EncodeFn fn = nullptr;
   if (!fn) {
     void* p = nullptr;
@@ -395,9 +396,9 @@ int sfb_rows_tmap(void* out_map, const void* base, int64_t rows, int64_t cols, i
   }
   if (!fn) return -1;
   cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)row_bytes};
-  cuuint32_t box[2] = {64u, (cuuint32_t)box_rows}, estr[2] = {1u, 1u};
+  cuuint32_t box[2] = {(cuuint32_t)box_cols, (cuuint32_t)box_rows}, estr[2] = {1u, 1u};
   return (int)fn((CUtensorMap*)out_map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr,
-                 CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+                 CU_TENSOR_MAP_INTERLEAVE_NONE, box_cols == 64 ? CU_TENSOR_MAP_SWIZZLE_128B : CU_TENSOR_MAP_SWIZZLE_64B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
 }
 
 // mq: queries [rows, H (dim + rot)], box 128 rows; mk, mv: keys and values [rows, dim / vdim], box 64 rows, page p of head g at row

@@ -11,7 +11,8 @@
 //
 //   delta_prep    per (chunk, group of heads): K K^T, the numbers of the rows (RATES), and (I + A)^-1 of every head in 32-bit: diagonal blocks
 //                 of 32 by substitution, the others from pairs of blocks
-//   delta_chain   per (head, 32 value dims), chunk after chunk: three products (K S_0, inverse X, K^T U), the state in registers
+//   delta_chain   per (head, 32 value dims), chunk after chunk: three products (K S_0, inverse X, K^T U), the state in registers; U and S_0
+//                 leave for chunk_out as tiles of two terms, [2, chunks, H, 128, P] and [2, chunks, H, N, P]
 //   chunk_out     the third line, all chunks at once (k_rows_state_tc.cu)
 //
 // q and k stay the bf16 vectors they come as; what makes them unit vectors is a factor per row on a product's result or on its other
@@ -37,9 +38,7 @@ struct Args {
   float* rates;                    // [chunks, H, RATES, 128]
   float* dec;                      // [chunks, H] decay over the whole chunk
   __nv_bfloat16* inv;              // [chunks, H, 2, 128, 128]: upper terms, lower terms (columns 64.. of rows below 64 are not written)
-  __nv_bfloat16* u;                // [2, u_lo, H P]
-  __nv_bfloat16* starts;           // [2, chunks, H, N, P]
-  int H, G, N, P, Np, ns, hpc, chunks, u_lo;
+  int H, G, N, P, Np, ns, hpc, chunks;
   int q_col, k_col, v_col;
   float q_scale, unit_eps;
   Status* status;
@@ -279,18 +278,22 @@ __device__ __forceinline__ void split16(const float* f, uint4 (&hi)[2], uint4 (&
   }
 }
 
-constexpr int PT = 32;             // value dims of a block
+constexpr int PT = 32, TILE = L * PT * 2;             // value dims of a block; bytes of 128 rows of them
 
 // grid (heads x tiles of 32 value dims, runs).  Operands with the value dims along a row (state, X, U) are 128 rows of 128 bytes: the upper terms
 // of the tile, then the lower ones, so that one product takes both (64 columns, whose halves are added up as they are read).
 __global__ void __launch_bounds__(THREADS, 1)
-delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mt, const __grid_constant__ CUtensorMap mt64, Args a) {
+delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant__ CUtensorMap mt, const __grid_constant__ CUtensorMap mt64,
+                   const __grid_constant__ CUtensorMap mv, const __grid_constant__ CUtensorMap mu, const __grid_constant__ CUtensorMap ms, Args a) {
   extern __shared__ __align__(1024) uint8_t sm[];
   uint8_t* ks = sm;                                       // two stages of two slabs
   uint8_t* ts = ks + 4 * SLAB;                            // inverse: upper terms (two slabs), lower terms
   uint8_t* ss = ts + 4 * SLAB;                            // state
   uint8_t* xs = ss + SLAB;                                // X, then U
-  Ctl& C = *reinterpret_cast<Ctl*>(xs + SLAB);
+  uint8_t* vs = xs + SLAB;                                // values, two stages of a tile (128 rows of 64 bytes)
+  uint8_t* us = vs + 2 * TILE;                            // U and the state on their way out: tiles of the upper and of the lower terms
+  uint8_t* so = us + 2 * TILE;
+  Ctl& C = *reinterpret_cast<Ctl*>(so + 2 * TILE);
   setup(C, 256);
   const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0), lane = tid & 31;
   // columns 64.. of the inverse's rows below 64 are zero and never loaded
@@ -307,8 +310,10 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
   const uint32_t t_ks = C.tmem, t_u = t_ks + 2 * PT, t_d = t_u + 2 * PT, t_l = t_d + 2 * PT;      // t_l: lower terms of the inverse
   if (issuer) {
     auto load_k = [&](int c) {
-      mbar_expect(&C.full[c & 1], a.ns * SLAB);
-      for (int s = 0; s < a.ns; ++s) tma2d(ks + ((c & 1) * 2 + s) * SLAB, &mk, a.k_col + g * a.N + 64 * s, a.c_row0[c0 + c], &C.full[c & 1]);
+      const int y = a.c_row0[c0 + c];
+      mbar_expect(&C.full[c & 1], a.ns * SLAB + TILE);
+      for (int s = 0; s < a.ns; ++s) tma2d(ks + ((c & 1) * 2 + s) * SLAB, &mk, a.k_col + g * a.N + 64 * s, y, &C.full[c & 1]);
+      tma2d(vs + (c & 1) * TILE, &mv, a.v_col + h * a.P + pt * PT, y, &C.full[c & 1]);
     };
     auto load_t = [&](int c) {
       const int y = ((c0 + c) * a.H + h) * 2 * L;
@@ -318,7 +323,8 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
         tma2d(ts + t * 2 * SLAB + SLAB + HSLAB, &mt64, 64, y + t * L + 64, &C.full[2]);
       }
     };
-    if (elect_one()) {
+    const bool leader = elect_one();
+    if (leader) {
       load_k(0);
       load_t(0);
       if (nc > 1) load_k(1);
@@ -331,18 +337,19 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
       const uint64_t dk = desc(smem_u32(ks) + (c & 1) * 2 * SLAB, 16), dkt = desc(smem_u32(ks) + (c & 1) * 2 * SLAB, SLAB);
       wait_warp(&C.full[c & 1], (c >> 1) & 1, dead, 4);
       __syncthreads();                                    // the state is in place
-      if (elect_one()) {
+      if (leader) {
         fence_after();
-        for (int t = 0; t < kst; ++t) {
-          const uint64_t ka = dk + (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, sb = ds + (uint64_t)t * (2048 >> 4);
-          mma_ss(t_ks, ka, sb, id, t ? 1u : 0u);
-        }
+        for (int t = 0; t < kst; ++t)
+          mma_ss(t_ks, dk + (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, ds + (uint64_t)t * (2048 >> 4), id, t ? 1u : 0u);
         commit(&C.done[0]);
+        for (int t = 0; t < 2; ++t) tma_store2d(&ms, pt * PT, ((t * a.chunks + c0 + c) * a.H + h) * a.N, so + t * TILE);
+        bulk_commit();
       }
       __syncwarp();
       wait_warp(&C.full[2], c & 1, dead, 5);
       __syncthreads();                                    // X is in place
-      if (elect_one()) {
+      if (leader) {
+        bulk_wait_read();                                 // what the workers write next has left
         fence_after();
 #pragma unroll
         for (int t = 0; t < 8; ++t) {
@@ -354,10 +361,10 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
       }
       __syncwarp();
       wait_warp(&C.done[1], c & 1, dead, 6);
-      if (c + 1 < nc && elect_one()) load_t(c + 1);
+      if (c + 1 < nc && leader) load_t(c + 1);
       __syncwarp();
       __syncthreads();                                    // U is in place
-      if (elect_one()) {
+      if (leader) {
         fence_after();
 #pragma unroll
         for (int t = 0; t < 8; ++t) {
@@ -365,17 +372,21 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
           mma_ss(t_d, dkt + o, dx + o, idt, t ? 1u : 0u);
         }
         commit(&C.done[2]);
+        for (int t = 0; t < 2; ++t) tma_store2d(&mu, pt * PT, ((t * a.chunks + c0 + c) * a.H + h) * L, us + t * TILE);
+        bulk_commit();
       }
       __syncwarp();
       wait_warp(&C.done[2], c & 1, dead, 7);
-      if (c + 2 < nc && elect_one()) load_k(c + 2);
+      if (c + 2 < nc && leader) load_k(c + 2);
       __syncwarp();
     }
+    if (leader) bulk_wait();
+    __syncwarp();
   } else {
     // a thread has one row (of the chunk, or of the state) and sixteen value dims
     const int w4 = warp & 3, half = warp >> 2, i = w4 * 32 + lane, p0 = pt * PT + half * 16, width = min(16, a.P - p0);      // width: a multiple of 8, or none
     const uint32_t at = ((uint32_t)(w4 * 32) << 16) + half * 16;
-    const size_t slot = (size_t)a.H * a.P * a.Np, HP = (size_t)a.H * a.P;
+    const size_t slot = (size_t)a.H * a.P * a.Np;
     const bool in_n = i < a.N;
     float S[16];
     {
@@ -402,38 +413,40 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
 #pragma unroll
       for (int k = 0; k < 16; ++k) f[k] += l[k];
     };
-    uint4 hi[2], lo[2];
-    const size_t lower = (size_t)a.chunks * a.H * a.N * a.P;
-    auto put_state = [&](int c) {         // the copy for chunk_out leaves under the first product
-      split16(S, hi, lo);
-      put(ss, hi, lo);
-      if (in_n) {
-        __nv_bfloat16* o = a.starts + (((size_t)(c0 + c) * a.H + h) * a.N + i) * a.P + p0;
+    auto put_out = [&](uint8_t* tile, const uint4 (&h2)[2], const uint4 (&l2)[2]) {      // row i of the tiles on their way out, 64-byte swizzle
 #pragma unroll
-        for (int q = 0; q < 2; ++q)
-          if (q * 8 < width) {
-            *reinterpret_cast<uint4*>(o + 8 * q) = hi[q];
-            *reinterpret_cast<uint4*>(o + lower + 8 * q) = lo[q];
-          }
+      for (int q = 0; q < 2; ++q) {
+        const int o = i * 64 + (((half * 2 + q) ^ (i >> 1 & 3)) << 4);
+        *reinterpret_cast<uint4*>(tile + o) = h2[q];
+        *reinterpret_cast<uint4*>(tile + TILE + o) = l2[q];
       }
     };
-    uint4 v[2];
-    float ek, b, ue, dec;
-    int row = a.c_row0[c0] + i, rows = a.c_rows[c0], row1 = 0, rows1 = 0;           // this chunk's, the next one's
-    auto fetch = [&](int c, int r, int m, float& e) {                               // numbers and values of chunk c
-      const float* n = a.rates + ((size_t)(c0 + c) * a.H + h) * RATES * L + i;
-      ek = n[3 * L]; b = n[4 * L]; e = n[5 * L];
-      const __nv_bfloat16* p = a.qkv + (size_t)r * a.stride + a.v_col + (size_t)h * a.P + p0;
-#pragma unroll
-      for (int q = 0; q < 2; ++q) v[q] = i < m && q * 8 < width ? *reinterpret_cast<const uint4*>(p + 8 * q) : make_uint4(0u, 0u, 0u, 0u);
+    uint4 hi[2], lo[2];
+    auto put_state = [&]() {
+      split16(S, hi, lo);
+      put_out(so, hi, lo);
+      put(ss, hi, lo);
     };
-    fetch(0, row, rows, ue);
-    dec = a.dec[(size_t)c0 * a.H + h];
-    if (nc > 1) { row1 = a.c_row0[c0 + 1] + i; rows1 = a.c_rows[c0 + 1]; }
-    put_state(0);
+    float ek, b, ue, dec;
+    int rows = a.c_rows[c0], rows1 = nc > 1 ? a.c_rows[c0 + 1] : 0;                 // this chunk's, the next one's
+    auto fetch = [&](int c, float& x, float& y, float& z, float& d) {               // numbers of chunk c
+      const float* n = a.rates + ((size_t)(c0 + c) * a.H + h) * RATES * L + i;
+      x = n[3 * L]; y = n[4 * L]; z = n[5 * L];
+      d = a.dec[(size_t)(c0 + c) * a.H + h];
+    };
+    fetch(0, ek, b, ue, dec);
+    put_state();
     for (int c = 0; c < nc; ++c) {
-      float f[16], ue1 = 0.f, dec1 = 0.f;
-      int row2 = 0, rows2 = 0;
+      float f[16], ek1 = 0.f, b1 = 0.f, ue1 = 0.f, dec1 = 0.f;
+      int rows2 = 0;
+      uint4 v[2];
+      wait_warp(&C.full[c & 1], (c >> 1) & 1, dead, 11);
+#pragma unroll
+      for (int q = 0; q < 2; ++q) v[q] = *reinterpret_cast<const uint4*>(vs + (c & 1) * TILE + i * 64 + (((half * 2 + q) ^ (i >> 1 & 3)) << 4));
+      if (c + 1 < nc) {                                   // requested a chunk ahead
+        fetch(c + 1, ek1, b1, ue1, dec1);
+        if (c + 2 < nc) rows2 = a.c_rows[c0 + c + 2];
+      }
       wait_warp(&C.done[0], c & 1, dead, 8);
       fence_after();
       read(t_ks, f);
@@ -449,11 +462,6 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
       }
       split16(f, hi, lo);
       put(xs, hi, lo);
-      if (c + 1 < nc) {                                   // requested under the product
-        fetch(c + 1, row1, rows1, ue1);
-        dec1 = a.dec[(size_t)(c0 + c + 1) * a.H + h];
-        if (c + 2 < nc) { row2 = a.c_row0[c0 + c + 2] + i; rows2 = a.c_rows[c0 + c + 2]; }
-      }
       wait_warp(&C.done[1], c & 1, dead, 9);
       fence_after();
       {
@@ -463,29 +471,20 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
 #pragma unroll
         for (int k = 0; k < 16; ++k) f[k] += l[k];
       }
-      uint4 uh[2], ul[2];
-      split16(f, uh, ul);
+      split16(f, hi, lo);
+      put_out(us, hi, lo);
 #pragma unroll
       for (int k = 0; k < 16; ++k) f[k] = i < rows ? f[k] * ue : 0.f;
       split16(f, hi, lo);
       put(xs, hi, lo);
-      if (i < rows) {                                     // u for chunk_out, under the product
-        __nv_bfloat16* o = a.u + (size_t)row * HP + (size_t)h * a.P + p0;
-#pragma unroll
-        for (int q = 0; q < 2; ++q)
-          if (q * 8 < width) {
-            *reinterpret_cast<uint4*>(o + 8 * q) = uh[q];
-            *reinterpret_cast<uint4*>(o + (size_t)a.u_lo * HP + 8 * q) = ul[q];
-          }
-      }
       wait_warp(&C.done[2], c & 1, dead, 10);
       fence_after();
       read(t_d, f);
 #pragma unroll
       for (int k = 0; k < 16; ++k) S[k] = in_n ? fmaf(dec, S[k], f[k]) : 0.f;
-      if (c + 1 < nc) put_state(c + 1);
+      if (c + 1 < nc) put_state();
       else fence_before();
-      ue = ue1; dec = dec1; row = row1; rows = rows1; row1 = row2; rows1 = rows2;
+      ek = ek1; b = b1; ue = ue1; dec = dec1; rows = rows1; rows1 = rows2;
     }
     if (in_n) {
       float* s1 = a.S + (size_t)a.seg_dst[seg] * slot + ((size_t)h * a.P + p0) * a.Np + i;
@@ -506,30 +505,31 @@ using namespace sfb::rdelta;
 
 extern "C" {
 
-// mk: rows of q | k | v, box 128 rows; mt, mt64: inv seen as [256 chunks H, 128], boxes of 128 and 64 rows.  N: a multiple of 16 up to 128; P: a
+// mk: rows of q | k | v, box 128 rows; mt, mt64: inv seen as [256 chunks H, 128], boxes of 128 and 64 rows; with 32 columns: mv: as mk; mu: u seen as
+// [2 chunks H 128, P], box 128 rows; ms: starts seen as [2 chunks H N, P], box N rows.  N: a multiple of 16 up to 128; P: a
 // multiple of 8; first columns and stride multiples of 8.  The rows between N and Np of the stored states are not written.
-int sfb_rows_delta_tc(const void* mk, const void* mt, const void* mt64, const int* c_row0, const int* c_rows, const int* seg, const int* first, const int* seg_src,
+int sfb_rows_delta_tc(const void* mk, const void* mt, const void* mt64, const void* mv, const void* mu, const void* ms, const int* c_row0, const int* c_rows, const int* seg, const int* first, const int* seg_src,
                       const int* seg_dst, const void* qkv, int64_t stride, const void* dt, int64_t dt_stride, const void* beta, int64_t beta_stride,
-                      const void* dt_bias, const void* la, void* S, void* rates, void* dec, void* inv, void* u, int u_lo, void* starts, int runs, int chunks, int H,
+                      const void* dt_bias, const void* la, void* S, void* rates, void* dec, void* inv, int runs, int chunks, int H,
                       int G, int N, int P, int Np, int q_col, int k_col, int v_col, float q_scale, float unit_eps, void* status, cudaStream_t stream) {
   if (runs < 1 || runs > 65535 || chunks < 1 || chunks > 65535 || G < 1 || H % G || N < 16 || N % 16 || N > 128 || P < 8 || P % 8 || Np < N ||
       (q_col | k_col | v_col) % 8 || stride % 8 || (uintptr_t)qkv % 16)
     return (int)cudaErrorInvalidValue;
   Args a{c_row0, c_rows, seg, first, seg_src, seg_dst, (const __nv_bfloat16*)qkv, stride, (const __nv_bfloat16*)dt, (const __nv_bfloat16*)beta, dt_stride,
-         beta_stride, (const float*)dt_bias, (const float*)la, (float*)S, (float*)rates, (float*)dec, (__nv_bfloat16*)inv, (__nv_bfloat16*)u,
-         (__nv_bfloat16*)starts, H, G, N, P, Np, (N + 63) / 64, 1, chunks, u_lo, q_col, k_col, v_col, q_scale, unit_eps, (Status*)status};
+         beta_stride, (const float*)dt_bias, (const float*)la, (float*)S, (float*)rates, (float*)dec, (__nv_bfloat16*)inv,
+         H, G, N, P, Np, (N + 63) / 64, 1, chunks, q_col, k_col, v_col, q_scale, unit_eps, (Status*)status};
   const int rep = H / G;
   a.hpc = rep < 8 ? rep : 8;                 // heads that share a block's K K^T: fewer where that leaves SMs empty
   while (a.hpc > 1 && (long long)G * ((rep + a.hpc - 1) / a.hpc) * chunks < 296) a.hpc = (a.hpc + 1) / 2;
   static size_t granted[2] = {0, 0};
-  const size_t prep = (size_t)2 * SLAB + ((size_t)L * LD + (2 + 2 * a.hpc) * L) * sizeof(float) + sizeof(Ctl), chain = (size_t)10 * SLAB + sizeof(Ctl);
+  const size_t prep = (size_t)2 * SLAB + ((size_t)L * LD + (2 + 2 * a.hpc) * L) * sizeof(float) + sizeof(Ctl), chain = (size_t)10 * SLAB + 6 * TILE + sizeof(Ctl);
   cudaError_t rc = grant(delta_prep_kernel, prep, granted[0]);
   if (rc == cudaSuccess) rc = grant(delta_chain_kernel, chain, granted[1]);
   if (rc == cudaSuccess)
     rc = sfb_launch(delta_prep_kernel, dim3(G * ((rep + a.hpc - 1) / a.hpc), chunks), dim3(WORK), prep, stream, *(const CUtensorMap*)mk, a);
   if (rc == cudaSuccess)
     rc = sfb_launch(delta_chain_kernel, dim3(H * ((P + PT - 1) / PT), runs), dim3(THREADS), chain, stream, *(const CUtensorMap*)mk, *(const CUtensorMap*)mt,
-                    *(const CUtensorMap*)mt64, a);
+                    *(const CUtensorMap*)mt64, *(const CUtensorMap*)mv, *(const CUtensorMap*)mu, *(const CUtensorMap*)ms, a);
   return (int)rc;
 }
 

@@ -36,7 +36,7 @@ struct Args {
   __nv_bfloat16* y;                // [n, H P]
   int H, G, N, P, Np, ns, terms;   // ns: 64-element slabs of a q / k row
   int q_col, k_col, v_col;         // first columns in the maps
-  int q_lo, k_lo;                  // distance to the columns of the lower terms; delta rule: to the rows of the values' lower terms (q_lo)
+  int q_lo, k_lo;                  // distance to the columns of the lower terms
   int chunks, hpc;                 // hpc: heads per block
   int wide;                        // outputs lie on 32-byte boundaries
   Status* status;
@@ -248,8 +248,11 @@ chunk_out_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
   auto tile = [&](int it) {                              // values and start state of a tile of 64 value dims
     const int h = h0 + it / pts, pt = it % pts;
     mbar_expect(&C.full[0], (DELTA ? 2 : 1) * SLAB + 2 * NS * HSLAB);
-    tma2d(vs, &mv, a.v_col + h * a.P + 64 * pt, row0, &C.full[0]);
-    if (DELTA) tma2d(vs + SLAB, &mv, a.v_col + h * a.P + 64 * pt, a.q_lo + row0, &C.full[0]);
+    if constexpr (DELTA) {
+      for (int t = 0; t < 2; ++t) tma2d(vs + t * SLAB, &mv, 64 * pt, ((t * a.chunks + chunk) * a.H + h) * L, &C.full[0]);
+    } else {
+      tma2d(vs, &mv, a.v_col + h * a.P + 64 * pt, row0, &C.full[0]);
+    }
   };
   auto state = [&](int it) {
     const int h = h0 + it / pts, pt = it % pts, rows1 = DELTA ? a.N : a.P, y = (chunk * a.H + h) * rows1 + (DELTA ? 0 : 64 * pt);
@@ -522,14 +525,14 @@ int sfb_rows_state_tc(const void* mq, const void* mk, const void* mv, const void
   }
 }
 
-// The outputs of the delta rule, after sfb_rows_delta_tc: mq, mk: rows of q / k, box 128 rows; mu: u seen as [2 x u_lo rows, H P], box 128
+// The outputs of the delta rule, after sfb_rows_delta_tc: mq, mk: rows of q / k, box 128 rows; mu: u seen as [2 chunks H 128, P], box 128
 // rows; ms: starts seen as [2 chunks H N, P], box 64 rows.  N: a multiple of 16 up to 128; P: a multiple of 8.
 int sfb_rows_delta_out(const void* mq, const void* mk, const void* mu, const void* ms, const int* c_row0, const int* c_rows, void* rates, void* starts, void* y,
-                       int chunks, int H, int G, int N, int P, int q_col, int k_col, int u_lo, void* status, cudaStream_t stream) {
+                       int chunks, int H, int G, int N, int P, int q_col, int k_col, void* status, cudaStream_t stream) {
   if (chunks < 1 || chunks > 65535 || G < 1 || H % G || N % 16 || N < 16 || N > 128 || P % 8 || P < 8 || (q_col | k_col) % 8) return (int)cudaErrorInvalidValue;
   Args a{};
   a.c_row0 = c_row0; a.c_rows = c_rows; a.rates = (float*)rates; a.starts = (__nv_bfloat16*)starts; a.y = (__nv_bfloat16*)y; a.H = H; a.G = G; a.N = N; a.P = P;
-  a.ns = (N + 63) / 64; a.terms = 1; a.q_col = q_col; a.k_col = k_col; a.q_lo = u_lo; a.chunks = chunks; a.hpc = 1;
+  a.ns = (N + 63) / 64; a.terms = 1; a.q_col = q_col; a.k_col = k_col; a.chunks = chunks; a.hpc = 1;
   a.wide = (H * P) % 16 == 0 && P % 16 == 0 && (uintptr_t)y % 32 == 0; a.status = (Status*)status;
   const dim3 grid(H, chunks);
   const CUtensorMap *q = (const CUtensorMap*)mq, *k = (const CUtensorMap*)mk, *u = (const CUtensorMap*)mu, *s = (const CUtensorMap*)ms;

@@ -419,7 +419,7 @@ class DeltaState(MatrixState):
             e.scratch.reserve("state_dec", chunks * self.H, torch.float32)
             e.scratch.reserve("state_starts", 2 * chunks * self.H * self.P * self.N, torch.bfloat16)
             e.scratch.reserve("delta_inv", chunks * self.H * 2 * 128 * 128, torch.bfloat16)
-            e.scratch.reserve("delta_u", 2 * e.max_rows * self.H * self.P, torch.bfloat16)
+            e.scratch.reserve("delta_u", 2 * chunks * self.H * 128 * self.P, torch.bfloat16)
 
     def run(self, s, src, cols, dt, beta, S, y, conv=None) -> None:
         """``src`` [n, stride] holds q, k, v from the columns ``cols`` on; ``conv``: they are the inputs of a convolution, see R.state_rows."""
@@ -430,8 +430,7 @@ class DeltaState(MatrixState):
                          beta, scale, self.UNIT_EPS)
         if s.nlong:
             buf = s.scratch.buf
-            u = s.scratch.get("delta_u", 2 * s.engine.max_rows, self.H * self.P)
-            R.delta_tc(src, cols, dt, beta, self.dt_bias, self.decay, S, buf["state_rates"], buf["state_dec"], buf["delta_inv"], u, buf["state_starts"], y,
+            R.delta_tc(src, cols, dt, beta, self.dt_bias, self.decay, S, buf["state_rates"], buf["state_dec"], buf["delta_inv"], buf["delta_u"], buf["state_starts"], y,
                        self.N, self.G, s, scale, self.UNIT_EPS, s.status)
 
 

@@ -166,17 +166,17 @@ def delta_tc_supports(dtype: torch.dtype, n: int, p: int) -> bool:
 
 def delta_tc(qkv, cols, dt, beta, dt_bias, log_a, S, rates, dec, inv, u, starts, y, N, groups, seg, q_scale, unit_eps, status):
     """Long segments in chunks of 128 rows.  ``qkv``: [n, stride] tensor with q, k, v from the columns ``cols`` on.  Scratch of all chunks: rates,
-    dec (32-bit), inv [chunks, H, 2, 128, 128], starts [2, chunks, H, N, P] and u [2 x most rows, H P] in bf16."""
+    dec (32-bit), inv [chunks, H, 2, 128, 128], starts [2, chunks, H, N, P] and u [2, chunks, H, 128, P] in bf16."""
     _, H, P, Np = S.shape
-    mqk, mu = tensor_map(qkv, qkv.shape[1], 128), tensor_map(u, H * P, 128)
-    mt, mt64, ms = tensor_map(inv, 128, 128), tensor_map(inv, 128, 64), tensor_map(starts, P, 64)
-    u_lo, at = u.shape[0] // 2, [c_int(c) for c in cols]
-    _check(_lib.rows().sfb_rows_delta_tc(mqk.ptr, mt.ptr, mt64.ptr, _p(seg.long_row0), _p(seg.long_rows), _p(seg.long_seg), _p(seg.long_first), _p(seg.seg_src),
+    mqk, mt, mt64 = tensor_map(qkv, qkv.shape[1], 128), tensor_map(inv, 128, 128), tensor_map(inv, 128, 64)
+    mv, us, ss = tensor_map(qkv, qkv.shape[1], 128, box_cols=32), tensor_map(u, P, 128, box_cols=32), tensor_map(starts, P, N, box_cols=32)
+    mu, ms, at = tensor_map(u, P, 128), tensor_map(starts, P, 64), [c_int(c) for c in cols]
+    _check(_lib.rows().sfb_rows_delta_tc(mqk.ptr, mt.ptr, mt64.ptr, mv.ptr, us.ptr, ss.ptr, _p(seg.long_row0), _p(seg.long_rows), _p(seg.long_seg), _p(seg.long_first), _p(seg.seg_src),
                                          _p(seg.seg_dst), *_strides(qkv), *_strides(dt), *_strides(beta), _p(dt_bias), _p(log_a), _p(S), _p(rates), _p(dec),
-                                         _p(inv), _p(u), c_int(u_lo), _p(starts), c_int(seg.nlong), c_int(seg.nchunks), c_int(H), c_int(groups), c_int(N),
+                                         _p(inv), c_int(seg.nlong), c_int(seg.nchunks), c_int(H), c_int(groups), c_int(N),
                                          c_int(P), c_int(Np), *at, c_float(q_scale), c_float(unit_eps), _p(status), _stream()), "rows_delta_tc")
     _check(_lib.rows().sfb_rows_delta_out(mqk.ptr, mqk.ptr, mu.ptr, ms.ptr, _p(seg.long_row0), _p(seg.long_rows), _p(rates), _p(starts), _p(y),
-                                          c_int(seg.nchunks), c_int(H), c_int(groups), c_int(N), c_int(P), at[0], at[1], c_int(u_lo), _p(status),
+                                          c_int(seg.nchunks), c_int(H), c_int(groups), c_int(N), c_int(P), at[0], at[1], _p(status),
                                           _stream()), "rows_delta_tc")
 
 
@@ -341,12 +341,13 @@ def attn_tc_supports(dtype: torch.dtype, dim: int, vdim: int) -> bool:
 
 class TensorMap:
     """A 2-D TMA map over a bf16 tensor seen as [rows, cols] with rows ``stride`` elements apart (cols by default), from element
-    ``first`` on; boxes of 64 columns x ``box`` rows."""
+    ``first`` on; boxes of ``box_cols`` (64 or 32) columns x ``box`` rows."""
 
-    def __init__(self, t: torch.Tensor, rows: int, cols: int, box: int, stride: int | None = None, first: int = 0):
+    def __init__(self, t: torch.Tensor, rows: int, cols: int, box: int, stride: int | None = None, first: int = 0, box_cols: int = 64):
         self._raw = (ctypes.c_uint8 * 192)()
         self.ptr = c_void_p((ctypes.addressof(self._raw) + 63) & ~63)
-        rc = _lib.rows().sfb_rows_tmap(self.ptr, c_void_p(t.data_ptr() + 2 * first), c_int64(rows), c_int64(cols), c_int64((stride or cols) * 2), c_int(box))
+        rc = _lib.rows().sfb_rows_tmap(self.ptr, c_void_p(t.data_ptr() + 2 * first), c_int64(rows), c_int64(cols), c_int64((stride or cols) * 2), c_int(box),
+                                       c_int(box_cols))
         if rc:
             raise RuntimeError(f"tensor map over [{rows}, {cols}]: error {rc}")
 
@@ -363,16 +364,16 @@ def attn_pools(kv, index: int, tc: bool):
 _maps: dict[tuple, TensorMap] = {}
 
 
-def tensor_map(t: torch.Tensor, cols: int, box: int, stride: int | None = None, first: int = 0) -> TensorMap:
+def tensor_map(t: torch.Tensor, cols: int, box: int, stride: int | None = None, first: int = 0, box_cols: int = 64) -> TensorMap:
     """The map over all of ``t``'s storage, kept, so that one map serves every step over a scratch buffer (it is an address and a shape:
     memory that is allocated again at the same place may use it again)."""
     stride = stride or cols
     total = t.untyped_storage().nbytes() // 2
-    key = (t.untyped_storage().data_ptr(), total, cols, box, stride, first)
+    key = (t.untyped_storage().data_ptr(), total, cols, box, stride, first, box_cols)
     m = _maps.get(key)
     if m is None:
         base = t if t.storage_offset() == 0 else torch.empty(0, dtype=t.dtype, device=t.device).set_(t.untyped_storage())
-        m = _maps[key] = TensorMap(base, (total - first - cols) // stride + 1, cols, box, stride, first)
+        m = _maps[key] = TensorMap(base, (total - first - cols) // stride + 1, cols, box, stride, first, box_cols)
     return m
 
 
