@@ -528,17 +528,30 @@ __global__ void __launch_bounds__(256) rot_append_kernel(RotAppendArgs a) {
 }
 
 // ---- gelu(projection) * a part of the token's row of a table ----------------------------------------------------------------
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(256) token_gate_kernel(const T* z, const T* table, const int* tokens, T* out, int n, int dim, int64_t table_stride, int col0, int vocab,
                                                          Status* status) {
   pdl_launch_dependents();
   pdl_wait();
-  for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < (int64_t)n * dim; i += (int64_t)gridDim.x * blockDim.x) {
-    const int row = (int)(i / dim), c = (int)(i - (int64_t)row * dim);
-    int tok = tokens[row];
-    if (tok < 0 || tok >= vocab) { status_set(status, ST_BOUNDS, 72, tok, vocab); tok = 0; }
-    out[i] = from_f<T>(gate_gelu<T>(to_f<T>(z[i])) * to_f<T>(table[(size_t)tok * table_stride + col0 + c]));
-  }
+  const int per = dim / V;
+  const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  const int row = (int)(i / per), c = (int)(i - (int64_t)row * per) * V;
+  if (row >= n) return;
+  int tok = tokens[row];
+  if (tok < 0 || tok >= vocab) { status_set(status, ST_BOUNDS, 72, tok, vocab); tok = 0; }
+  float f[V], e[V];
+  load_v<T, V>(z + (size_t)row * dim + c, f);
+  load_v<T, V>(table + (size_t)tok * table_stride + col0 + c, e);
+#pragma unroll
+  for (int k = 0; k < V; ++k) f[k] = gate_gelu<T>(f[k]) * e[k];
+  store_v<T, V>(out + (size_t)row * dim + c, f);
+}
+template <typename T, int V>
+static int launch_token_gate(const void* z, const void* table, const int* tokens, void* out, int n, int dim, int64_t table_stride, int col0, int vocab, Status* status,
+                             cudaStream_t st) {
+  const int64_t blocks = ((int64_t)n * (dim / V) + 255) / 256;
+  return (int)sfb_launch(token_gate_kernel<T, V>, dim3((unsigned)blocks), dim3(256), 0, st, (const T*)z, (const T*)table, tokens, (T*)out, n, dim, table_stride, col0,
+                         vocab, status);
 }
 
 // ---- real-gated linear recurrence -------------------------------------------------------------------------------------------
@@ -972,11 +985,13 @@ int sfb_rows_rot_append(const void* proj, int64_t stride, const void* cs, void* 
 int sfb_rows_token_gate(const void* z, const void* table, const int* tokens, void* out, int n, int dim, int64_t table_stride, int col0, int vocab, int fp32,
                         void* status, cudaStream_t stream) {
   if (n < 1 || dim < 1) return (int)cudaErrorInvalidValue;
-  const int64_t blocks = ((int64_t)n * dim + 255) / 256;
-  const dim3 g((unsigned)(blocks < 1184 ? blocks : 1184)), b(256);
-  if (fp32) return (int)sfb_launch(token_gate_kernel<float>, g, b, 0, stream, (const float*)z, (const float*)table, tokens, (float*)out, n, dim, table_stride, col0, vocab, (Status*)status);
-  return (int)sfb_launch(token_gate_kernel<__nv_bfloat16>, g, b, 0, stream, (const __nv_bfloat16*)z, (const __nv_bfloat16*)table, tokens, (__nv_bfloat16*)out, n, dim,
-                         table_stride, col0, vocab, (Status*)status);
+  const int all = dim | col0 | (int)(table_stride & 1023);
+  Status* s = (Status*)status;
+  if (fp32) return all % 4 ? launch_token_gate<float, 1>(z, table, tokens, out, n, dim, table_stride, col0, vocab, s, stream)
+                           : launch_token_gate<float, 4>(z, table, tokens, out, n, dim, table_stride, col0, vocab, s, stream);
+  if (all % 8 == 0) return launch_token_gate<__nv_bfloat16, 8>(z, table, tokens, out, n, dim, table_stride, col0, vocab, s, stream);
+  return all % 4 ? launch_token_gate<__nv_bfloat16, 1>(z, table, tokens, out, n, dim, table_stride, col0, vocab, s, stream)
+                 : launch_token_gate<__nv_bfloat16, 4>(z, table, tokens, out, n, dim, table_stride, col0, vocab, s, stream);
 }
 
 int sfb_rows_act_mul(const void* gu, void* out, int64_t out_stride, int n, int ff, int act, float alpha, float limit, int fp32, cudaStream_t stream) {

@@ -75,14 +75,14 @@ __device__ __forceinline__ void head_rates(const Args& a, int chunk, int h, int 
   if (lane == 0) a.dec[(size_t)chunk * a.H + h] = ex2(last);
 }
 
-// acc[r][c] += sum over k in [k0, k1) of x[r][k] y[k][c], four by four; x, y: rows of LD / ldy floats, k0 and k1 multiples of four
-__device__ __forceinline__ void micro(float (&acc)[4][4], const float* x, const float* y, int ldy, int k0, int k1) {
+// acc[r][c] += sum over k in [k0, k1) of x[r][k] y[k][c], four by four; x, y: rows of LD floats, k0 and k1 multiples of four
+__device__ __forceinline__ void micro(float (&acc)[4][4], const float* x, const float* y, int k0, int k1) {
   for (int k = k0; k < k1; k += 4) {
     float4 l[4], r[4];
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       l[i] = *reinterpret_cast<const float4*>(x + i * LD + k);
-      r[i] = *reinterpret_cast<const float4*>(y + (k + i) * ldy);
+      r[i] = *reinterpret_cast<const float4*>(y + (k + i) * LD);
     }
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
@@ -97,30 +97,29 @@ __device__ __forceinline__ void micro(float (&acc)[4][4], const float* x, const 
 }
 
 // The block below a pair of inverted diagonal blocks of B rows at `b0`: -T22 (A21 T11).  A warp takes 16 rows (from `r0`) x 32 columns (from
-// `c0`), four by four a thread.  `w`: B x (B + 4) floats.  Two calls, a barrier in between: the inner product, then the outer one.
+// `c0`), four by four a thread.  The block above the diagonal holds the inner product.  Two calls, a barrier in between.
 template <int B>
-__device__ __forceinline__ void pair_inner(const float* A, float* w, int b0, int r0, int c0) {
+__device__ __forceinline__ void pair_inner(float* A, int b0, int r0, int c0) {
   const int r = r0 + (threadIdx.x >> 3 & 3) * 4, c = c0 + (threadIdx.x & 7) * 4;
   float acc[4][4] = {};
-  micro(acc, A + (b0 + B + r) * LD + b0, A + b0 * LD + b0 + c, LD, c0, B);      // T11 is lower triangular
+  micro(acc, A + (b0 + B + r) * LD + b0, A + b0 * LD + b0 + c, c0, B);      // T11 is lower triangular
 #pragma unroll
-  for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(w + (r + i) * (B + 4) + c) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+  for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(A + (b0 + r + i) * LD + b0 + B + c) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
 }
 template <int B>
-__device__ __forceinline__ void pair_outer(float* A, const float* w, int b0, int r0, int c0) {
+__device__ __forceinline__ void pair_outer(float* A, int b0, int r0, int c0) {
   const int r = r0 + (threadIdx.x >> 3 & 3) * 4, c = c0 + (threadIdx.x & 7) * 4;
   float acc[4][4] = {};
-  micro(acc, A + (b0 + B + r) * LD + b0 + B, w + c, B + 4, 0, r0 + 16);
+  micro(acc, A + (b0 + B + r) * LD + b0 + B, A + b0 * LD + b0 + B + c, 0, r0 + 16);
 #pragma unroll
   for (int i = 0; i < 4; ++i) *reinterpret_cast<float4*>(A + (b0 + B + r + i) * LD + b0 + c) = make_float4(-acc[i][0], -acc[i][1], -acc[i][2], -acc[i][3]);
 }
 
 // grid (groups x parts of a group's heads, chunks); 256 threads
-__global__ void __launch_bounds__(WORK, 2) delta_prep_kernel(const __grid_constant__ CUtensorMap mk, Args a) {
+__global__ void __launch_bounds__(WORK, 3) delta_prep_kernel(const __grid_constant__ CUtensorMap mk, Args a) {
   extern __shared__ __align__(1024) uint8_t sm[];
-  uint8_t* ks = sm;                                       // k, two slabs; later the pairs' inner products
-  float* w = reinterpret_cast<float*>(sm);
-  float* A = reinterpret_cast<float*>(sm + 2 * SLAB);     // [128][LD]
+  uint8_t* ks = sm;                                       // k, two slabs; after k k^T:
+  float* A = reinterpret_cast<float*>(sm);                // [128][LD]
   float* rk = A + L * LD;                                 // [128] each: factors to unit length
   float *rq = rk + L, *css = rq + L, *bss = css + a.hpc * L;      // [hpc][128]: running sums, write strengths
   Ctl& C = *reinterpret_cast<Ctl*>(bss + a.hpc * L);
@@ -151,32 +150,35 @@ __global__ void __launch_bounds__(WORK, 2) delta_prep_kernel(const __grid_consta
   for (int x = WORK / 32 - 1 - warp; x < nh; x += WORK / 32) head_rates(a, chunk, h0 + x, row0, rows, css + x * L, bss + x * L);
   {   // eight lanes per row and vector: its factor to unit length
     const int sub = lane & 7, words = a.N / 8;
-    uint4 v[8][2];
 #pragma unroll
-    for (int t = 0; t < 8; ++t) {
-      const int rv = warp * 32 + t * 4 + (lane >> 3), i = rv & (L - 1);      // the first 128: q, then k
-      const uint4* p = reinterpret_cast<const uint4*>(a.qkv + (size_t)(row0 + min(i, rows - 1)) * a.stride + (rv >> 7 ? a.k_col : a.q_col) + g * a.N);
+    for (int t0 = 0; t0 < 8; t0 += 4) {
+      uint4 v[4][2];
 #pragma unroll
-      for (int q = 0; q < 2; ++q) v[t][q] = sub + 8 * q < words ? p[sub + 8 * q] : make_uint4(0u, 0u, 0u, 0u);
-    }
+      for (int t = 0; t < 4; ++t) {
+        const int rv = warp * 32 + (t0 + t) * 4 + (lane >> 3), i = rv & (L - 1);      // the first 128: q, then k
+        const uint4* p = reinterpret_cast<const uint4*>(a.qkv + (size_t)(row0 + min(i, rows - 1)) * a.stride + (rv >> 7 ? a.k_col : a.q_col) + g * a.N);
 #pragma unroll
-    for (int t = 0; t < 8; ++t) {
-      float s = 0.f;
-#pragma unroll
-      for (int q = 0; q < 2; ++q) {
-        const uint32_t x[4] = {v[t][q].x, v[t][q].y, v[t][q].z, v[t][q].w};
-#pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          const float f0 = __uint_as_float(x[k] << 16), f1 = __uint_as_float(x[k] & 0xffff0000u);
-          s = fmaf(f0, f0, s);
-          s = fmaf(f1, f1, s);
-        }
+        for (int q = 0; q < 2; ++q) v[t][q] = sub + 8 * q < words ? p[sub + 8 * q] : make_uint4(0u, 0u, 0u, 0u);
       }
-      s += __shfl_xor_sync(0xffffffffu, s, 1);
-      s += __shfl_xor_sync(0xffffffffu, s, 2);
-      s += __shfl_xor_sync(0xffffffffu, s, 4);
-      const int rv = warp * 32 + t * 4 + (lane >> 3);
-      if (sub == 0) (rv >> 7 ? rk : rq)[rv & (L - 1)] = (rv >> 7 ? 1.f : a.q_scale) / sqrtf(s + a.unit_eps);
+#pragma unroll
+      for (int t = 0; t < 4; ++t) {
+        float s = 0.f;
+#pragma unroll
+        for (int q = 0; q < 2; ++q) {
+          const uint32_t x[4] = {v[t][q].x, v[t][q].y, v[t][q].z, v[t][q].w};
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const float f0 = __uint_as_float(x[k] << 16), f1 = __uint_as_float(x[k] & 0xffff0000u);
+            s = fmaf(f0, f0, s);
+            s = fmaf(f1, f1, s);
+          }
+        }
+        s += __shfl_xor_sync(0xffffffffu, s, 1);
+        s += __shfl_xor_sync(0xffffffffu, s, 2);
+        s += __shfl_xor_sync(0xffffffffu, s, 4);
+        const int rv = warp * 32 + (t0 + t) * 4 + (lane >> 3);
+        if (sub == 0) (rv >> 7 ? rk : rq)[rv & (L - 1)] = (rv >> 7 ? 1.f : a.q_scale) / sqrtf(s + a.unit_eps);
+      }
     }
   }
   const int w4 = warp & 3, half = warp >> 2, i = w4 * 32 + lane;
@@ -239,18 +241,18 @@ __global__ void __launch_bounds__(WORK, 2) delta_prep_kernel(const __grid_consta
       for (int r = 0; r < 32; ++r) B[r * LD + lane] = t[r];
     }
     __syncthreads();
-    if (warp < 4) pair_inner<32>(A, w + (warp >> 1) * 32 * 36, (warp >> 1) * 64, (warp & 1) * 16, 0);
+    if (warp < 4) pair_inner<32>(A, (warp >> 1) * 64, (warp & 1) * 16, 0);
     __syncthreads();
-    if (warp < 4) pair_outer<32>(A, w + (warp >> 1) * 32 * 36, (warp >> 1) * 64, (warp & 1) * 16, 0);
-    else {            // the two blocks of 32 above the diagonal inside the blocks of 64
-      const int z = tid - 128, p = z >> 6, r = (z & 63) >> 1, c = (z & 1) * 16;
+    if (warp < 4) pair_outer<32>(A, (warp >> 1) * 64, (warp & 1) * 16, 0);
+    __syncthreads();
+    {                 // the two blocks of 32 above the diagonal inside the blocks of 64
+      const int p = tid >> 7, r = tid >> 2 & 31, c = (tid & 3) * 8;
 #pragma unroll
-      for (int k = 0; k < 16; k += 4) *reinterpret_cast<float4*>(A + (p * 64 + r) * LD + p * 64 + 32 + c + k) = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int k = 0; k < 8; k += 4) *reinterpret_cast<float4*>(A + (p * 64 + r) * LD + p * 64 + 32 + c + k) = make_float4(0.f, 0.f, 0.f, 0.f);
     }
+    pair_inner<64>(A, 0, (warp >> 1) * 16, (warp & 1) * 32);
     __syncthreads();
-    pair_inner<64>(A, w, 0, (warp >> 1) * 16, (warp & 1) * 32);
-    __syncthreads();
-    pair_outer<64>(A, w, 0, (warp >> 1) * 16, (warp & 1) * 32);
+    pair_outer<64>(A, 0, (warp >> 1) * 16, (warp & 1) * 32);
     __syncthreads();
     __nv_bfloat16* hi = a.inv + ((size_t)chunk * a.H + h) * 2 * L * L;
 #pragma unroll 4
@@ -522,7 +524,7 @@ int sfb_rows_delta_tc(const void* mk, const void* mt, const void* mt64, const vo
   a.hpc = rep < 8 ? rep : 8;                 // heads that share a block's K K^T: fewer where that leaves SMs empty
   while (a.hpc > 1 && (long long)G * ((rep + a.hpc - 1) / a.hpc) * chunks < 296) a.hpc = (a.hpc + 1) / 2;
   static size_t granted[2] = {0, 0};
-  const size_t prep = (size_t)2 * SLAB + ((size_t)L * LD + (2 + 2 * a.hpc) * L) * sizeof(float) + sizeof(Ctl), chain = (size_t)10 * SLAB + 6 * TILE + sizeof(Ctl);
+  const size_t prep = ((size_t)L * LD + (2 + 2 * a.hpc) * L) * sizeof(float) + sizeof(Ctl), chain = (size_t)10 * SLAB + 6 * TILE + sizeof(Ctl);
   cudaError_t rc = grant(delta_prep_kernel, prep, granted[0]);
   if (rc == cudaSuccess) rc = grant(delta_chain_kernel, chain, granted[1]);
   if (rc == cudaSuccess)

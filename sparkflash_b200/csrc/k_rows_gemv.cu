@@ -1,5 +1,5 @@
 // Matrix products of one to four rows, bf16 weights streamed once: out = x W^T (+ bias), to bf16 or 32-bit, or act(x Wg^T) * (x Wu^T)
-// with gate and up stacked.  Paced by memory: a warp (or two, four, eight of them, each on a share of K) owns two weight rows, whose first
+// with gate and up stacked, or gelu(x W^T) times the token's row of a table.  Paced by memory: a warp (or two, four, eight of them, each on a share of K) owns two weight rows, whose first
 // 16-byte words are requested before the previous kernel has finished - weights do not depend on it; x sits in shared memory.
 #include "k_rows.cuh"
 
@@ -16,6 +16,11 @@ struct Args {
   int M, K, n, wk, f32, act;
   int64_t out_stride;         // elements between the rows of out
   float alpha, limit;         // of the clamped gate
+  const __nv_bfloat16* table; // [vocab, table_stride] or null: out = gelu(x W^T) * table[token][col0 + .]
+  int64_t table_stride;
+  const int* tokens;
+  int col0, vocab;
+  Status* status;
 };
 
 template <int N>
@@ -115,6 +120,13 @@ __global__ void __launch_bounds__(256, 2) gemv_kernel(Args a) {
       } else {
         const int r0 = 2 * o, r1 = r0 + 1;
         if (a.bias) { if (r0 < a.M) s0 += __bfloat162float(a.bias[r0]); if (r1 < a.M) s1 += __bfloat162float(a.bias[r1]); }
+        if (a.table) {
+          int tok = a.tokens[lane];
+          if (tok < 0 || tok >= a.vocab) { status_set(a.status, ST_BOUNDS, 76, tok, a.vocab); tok = 0; }
+          const __nv_bfloat16* e = a.table + (size_t)tok * a.table_stride + a.col0;
+          s0 = r0 < a.M ? rows::gelu_tanh_f(s0) * __bfloat162float(e[r0]) : 0.f;
+          s1 = r1 < a.M ? rows::gelu_tanh_f(s1) * __bfloat162float(e[r1]) : 0.f;
+        }
         if (a.f32) {
           if (r0 < a.M) ((float*)a.out)[at + r0] = s0;
           if (r1 < a.M) ((float*)a.out)[at + r1] = s1;
@@ -147,19 +159,34 @@ static int launch(const Args& a, int blocks, cudaStream_t st) {
 using namespace sfb;
 using namespace sfb::rgemv;
 
+static int run(Args a, cudaStream_t stream) {
+  const int N = a.n <= 1 ? 1 : a.n <= 2 ? 2 : 4;
+  if (a.n < 1 || a.n > 4 || a.M < 1 || a.K < 8 || a.K % 8 || (size_t)N * a.K * 2 > 200 * 1024) return (int)cudaErrorInvalidValue;
+  const int pairs = a.act ? a.M : (a.M + 1) / 2, steps = (a.K + 255) / 256;
+  a.wk = 1;                // enough pairs of rows for every SM, at least a batch of K per warp
+  while (a.wk < 8 && (long long)pairs * a.wk / 8 < 296 && steps / (a.wk * 2) >= 2) a.wk *= 2;
+  const int needed = (pairs + 8 / a.wk - 1) / (8 / a.wk), blocks = needed < 296 ? needed : 296;
+  return N == 1 ? launch<1>(a, blocks, stream) : N == 2 ? launch<2>(a, blocks, stream) : launch<4>(a, blocks, stream);
+}
+
 extern "C" {
 
 // n <= 4 rows, K a multiple of 8, n K bounded by shared memory (4 K rows of 200 KB).  act (1 silu, 2 gelu, 3 clamped): w holds 2 M rows.
 int sfb_rows_gemv(const void* w, const void* x, const void* bias, void* out, int64_t out_stride, int n, int M, int K, int f32, int act, float alpha, float limit,
                   cudaStream_t stream) {
-  const int N = n <= 1 ? 1 : n <= 2 ? 2 : 4;
-  if (n < 1 || n > 4 || M < 1 || K < 8 || K % 8 || (size_t)N * K * 2 > 200 * 1024) return (int)cudaErrorInvalidValue;
-  const int pairs = act ? M : (M + 1) / 2, steps = (K + 255) / 256;
-  int wk = 1;              // enough pairs of rows for every SM, at least a batch of K per warp
-  while (wk < 8 && (long long)pairs * wk / 8 < 296 && steps / (wk * 2) >= 2) wk *= 2;
-  const int needed = (pairs + 8 / wk - 1) / (8 / wk), blocks = needed < 296 ? needed : 296;
-  Args a{(const __nv_bfloat16*)w, (const __nv_bfloat16*)x, (const __nv_bfloat16*)bias, out, M, K, n, wk, f32, act, out_stride, alpha, limit};
-  return N == 1 ? launch<1>(a, blocks, stream) : N == 2 ? launch<2>(a, blocks, stream) : launch<4>(a, blocks, stream);
+  Args a{};
+  a.w = (const __nv_bfloat16*)w; a.x = (const __nv_bfloat16*)x; a.bias = (const __nv_bfloat16*)bias; a.out = out; a.M = M; a.K = K; a.n = n; a.f32 = f32;
+  a.act = act; a.out_stride = out_stride; a.alpha = alpha; a.limit = limit;
+  return run(a, stream);
+}
+
+// out [n, M] = gelu(x w^T) * table[token][col0 + .]
+int sfb_rows_gemv_token(const void* w, const void* x, void* out, const void* table, int64_t table_stride, const int* tokens, int col0, int vocab, int n, int M, int K,
+                        void* status, cudaStream_t stream) {
+  Args a{};
+  a.w = (const __nv_bfloat16*)w; a.x = (const __nv_bfloat16*)x; a.out = out; a.M = M; a.K = K; a.n = n; a.out_stride = M; a.table = (const __nv_bfloat16*)table;
+  a.table_stride = table_stride; a.tokens = tokens; a.col0 = col0; a.vocab = vocab; a.status = (Status*)status;
+  return run(a, stream);
 }
 
 }  // extern "C"

@@ -2,9 +2,10 @@
 //
 //   moe_route   the chosen experts of a row and their weights (softmax over the chosen logits), and the shared expert's weight
 //               (sigmoid of one more logit); one warp per row
-//   moe_plan    (row, choice) pairs in order of their expert, cut into tiles of `tile` pairs of one expert
+//   moe_plan    (row, choice) pairs in order of their expert, cut into tiles of `tile` pairs of one expert; chooses as well when rows are few
 //   moe_tile    one tile x 64 output columns on CUDA cores: any sizes, bf16 or 32-bit (k_rows_moe_tc.cu takes bf16 on tcgen05)
-//   moe_gemv    one to four rows, bf16: a block per (pair, share of the output), weights streamed; the shared expert's rows beside the pairs
+//   moe_gemv    one to four rows, bf16: a block per (pair, share of the output), weights streamed; the shared expert's rows beside the
+//               pairs; every block of the first product chooses for its row
 //
 // Both products of an expert go through the same kernels: `gated` (gate and up rows stacked, act(gate) * up, rows picked by the plan) and
 // down (rows of the first product in plan order, results at [row][choice], where the seam sums them with their weights).
@@ -24,66 +25,91 @@ struct RouteArgs {
   float* wts;               // [n, top + shared]
   int n, E, top, shared;
 };
+// One warp, one row: lane j ends up with choice j and its weight (the lower number wins among equal logits); `shared_w`: the shared expert's.
+constexpr int HELD = 8;     // logits a lane holds, the rest is read again
+// bits that compare as the numbers do; above 0 for every number
+__device__ __forceinline__ uint32_t rank_bits(float v) {
+  const uint32_t b = __float_as_uint(v);
+  return b & 0x80000000u ? ~b : b | 0x80000000u;
+}
+__device__ __forceinline__ void choose(const RouteArgs& a, const float* z, int& id, float& weight, float& shared_w) {
+  const int lane = threadIdx.x & 31;
+  uint32_t v[HELD];         // 0: taken, or past the end
+#pragma unroll
+  for (int k = 0; k < HELD; ++k) v[k] = k * 32 + lane < a.E ? rank_bits(z[k * 32 + lane]) : 0u;
+  const float zs = a.shared ? z[a.E] : 0.f;
+  uint32_t taken = 0, mine = 0;      // taken: of this lane's experts beyond those it holds; mine: lane j: logit of choice j
+  id = 0;
+  for (int j = 0; j < a.top; ++j) {
+    uint32_t best = 0;
+    int at = a.E;
+#pragma unroll
+    for (int k = 0; k < HELD; ++k)
+      if (v[k] > best) { best = v[k]; at = k * 32 + lane; }
+    for (int e = HELD * 32 + lane, k = HELD; e < a.E; e += 32, ++k) {
+      const uint32_t x = taken >> k & 1 ? 0u : rank_bits(z[e]);
+      if (x > best) { best = x; at = e; }
+    }
+    const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+    at = (int)min(__reduce_min_sync(0xffffffffu, (unsigned)(best == top ? at : a.E)), (unsigned)(a.E - 1));
+    if ((at & 31) == lane) {
+      taken |= 1u << (at >> 5);
+#pragma unroll
+      for (int k = 0; k < HELD; ++k)
+        if (at >> 5 == k) v[k] = 0u;
+    }
+    if (lane == j) { mine = top; id = at; }
+  }
+  const float mz = __uint_as_float(mine & 0x80000000u ? mine ^ 0x80000000u : ~mine);
+  const float top = __shfl_sync(0xffffffffu, mz, 0), e = lane < a.top ? expf(mz - top) : 0.f;
+  weight = e / warp_sum(e);
+  shared_w = sigmoid_f(zs);
+}
+__device__ __forceinline__ void route_row(const RouteArgs& a, int row) {
+  const int lane = threadIdx.x & 31;
+  int id;
+  float w, sw;
+  choose(a, a.z + (size_t)row * a.ld, id, w, sw);
+  float* o = a.wts + (size_t)row * (a.top + a.shared);
+  if (lane < a.top) { a.ids[(size_t)row * a.top + lane] = id; o[lane] = w; }
+  if (a.shared && lane == 0) o[a.top] = sw;
+}
 __global__ void __launch_bounds__(256) moe_route_kernel(RouteArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  const int row = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (row >= a.n) return;
-  const float* z = a.z + (size_t)row * a.ld;
-  uint32_t taken = 0;       // of this lane's experts lane, lane + 32, ...
-  float mine = 0.f;         // lane j: logit of choice j
-  int id = 0;
-  for (int j = 0; j < a.top; ++j) {
-    float best = -INFINITY;
-    int at = a.E;
-    for (int e = lane, k = 0; e < a.E; e += 32, ++k) {
-      const float v = z[e];
-      if (!(taken >> k & 1) && (v > best || at == a.E)) { best = v; at = e; }
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float v = __shfl_xor_sync(0xffffffffu, best, o);
-      const int e = __shfl_xor_sync(0xffffffffu, at, o);
-      if (e < a.E && (at == a.E || v > best || (v == best && e < at))) { best = v; at = e; }
-    }
-    at = __shfl_sync(0xffffffffu, at, 0);
-    best = __shfl_sync(0xffffffffu, best, 0);
-    at = min(at, a.E - 1);
-    if ((at & 31) == lane) taken |= 1u << (at >> 5);
-    if (lane == j) { mine = best; id = at; }
-  }
-  const float top = __shfl_sync(0xffffffffu, mine, 0), e = lane < a.top ? expf(mine - top) : 0.f, sum = warp_sum(e);
-  float* w = a.wts + (size_t)row * (a.top + a.shared);
-  if (lane < a.top) {
-    a.ids[(size_t)row * a.top + lane] = id;
-    w[lane] = e / sum;
-  }
-  if (a.shared && lane == 0) w[a.top] = sigmoid_f(z[a.E]);
+  const int row = blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (row < a.n) route_row(a, row);
 }
 
 // ---- plan -----------------------------------------------------------------------------------------------------------------
 struct PlanArgs {
-  const int* ids;           // [pairs]
+  RouteArgs r;              // r.z null: ids are there
   int* order;               // [pairs] pair at every place
   int* tiles;               // [max tiles][4]: expert, first place, pairs, -
   int* count;               // number of tiles
   int pairs, E, tile;
 };
+constexpr int BATCH = 32;   // pairs a thread holds: their expert, and how many of it came before (20 bits)
+
 __global__ void __launch_bounds__(1024) moe_plan_kernel(PlanArgs a) {
   __shared__ int cnt[MAX_E], wsum[2][32];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   cnt[tid] = 0;
   pdl_launch_dependents();
   pdl_wait();
-  __syncthreads();
-  for (int p0 = 0; p0 < a.pairs; p0 += 4096) {
-    int e[4];
+  if (a.r.z)
+    for (int row = warp; row < a.r.n; row += 32) route_row(a.r, row);
+  __syncthreads();          // (orders the block's own ids too)
+  uint32_t held[BATCH];
+  // a place inside its expert for every pair
+  auto places = [&](int p0) {
 #pragma unroll
-    for (int k = 0; k < 4; ++k) e[k] = p0 + k * 1024 + tid < a.pairs ? a.ids[p0 + k * 1024 + tid] : -1;
+    for (int k = 0; k < BATCH; ++k) held[k] = p0 + k * 1024 + tid < a.pairs ? (uint32_t)a.r.ids[p0 + k * 1024 + tid] : 0u;
 #pragma unroll
-    for (int k = 0; k < 4; ++k)
-      if (e[k] >= 0) atomicAdd(&cnt[e[k]], 1);
-  }
+    for (int k = 0; k < BATCH; ++k)
+      if (p0 + k * 1024 + tid < a.pairs) held[k] = held[k] << 20 | (uint32_t)atomicAdd(&cnt[held[k]], 1);
+  };
+  for (int p0 = 0; p0 < a.pairs; p0 += BATCH * 1024) places(p0);
   __syncthreads();
   const int c = cnt[tid], t = (c + a.tile - 1) / a.tile;
   int sc = c, st = t;       // inclusive sums of pairs and of tiles over the experts
@@ -98,15 +124,16 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(PlanArgs a) {
   const int first = sc - c;
   for (int k = 0; k < t; ++k) reinterpret_cast<int4*>(a.tiles)[st - t + k] = make_int4(tid, first + k * a.tile, min(a.tile, c - k * a.tile), 0);
   if (tid == 1023) *a.count = st;
-  cnt[tid] = first;         // from here on: the expert's next free place
+  const bool once = a.pairs <= BATCH * 1024;
+  __shared__ int base[MAX_E];
+  base[tid] = first;
+  cnt[tid] = 0;             // more pairs than the threads hold: they take their places again
   __syncthreads();
-  for (int p0 = 0; p0 < a.pairs; p0 += 4096) {
-    int e[4];
+  for (int p0 = 0; p0 < a.pairs; p0 += BATCH * 1024) {
+    if (!once) places(p0);
 #pragma unroll
-    for (int k = 0; k < 4; ++k) e[k] = p0 + k * 1024 + tid < a.pairs ? a.ids[p0 + k * 1024 + tid] : -1;
-#pragma unroll
-    for (int k = 0; k < 4; ++k)
-      if (e[k] >= 0) a.order[atomicAdd(&cnt[e[k]], 1)] = p0 + k * 1024 + tid;
+    for (int k = 0; k < BATCH; ++k)
+      if (p0 + k * 1024 + tid < a.pairs) a.order[base[held[k] >> 20] + (int)(held[k] & 0xfffffu)] = p0 + k * 1024 + tid;
   }
 }
 
@@ -177,7 +204,7 @@ __global__ void __launch_bounds__(256) moe_tile_kernel(TileArgs a) {
 
 // ---- few rows -----------------------------------------------------------------------------------------------------------------
 struct GemvArgs {
-  const int* ids;             // [pairs] experts
+  RouteArgs r;                // r.z: the first product chooses the experts (and leaves them in r.ids and r.wts)
   const __nv_bfloat16* x;     // gated: [n, K]; down: [pairs, K]
   const __nv_bfloat16* w;     // [E, (2) M, K]
   __nv_bfloat16* out;         // gated: [pairs, M]; down: [n, slots, M]
@@ -190,13 +217,29 @@ constexpr int GU = 4;         // 256-element steps in flight per weight row
 
 __global__ void __launch_bounds__(256) moe_gemv_kernel(GemvArgs a) {
   extern __shared__ __align__(16) uint8_t raw[];
+  __shared__ int chosen;
   __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(raw);
   pdl_launch_dependents();
   pdl_wait();
   const int job = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const bool sh = job >= a.pairs;
+  if (a.r.z && !sh) {
+    if (warp == 0) {
+      int id;
+      float w, sw;
+      choose(a.r, a.r.z + (size_t)(job / a.top) * a.r.ld, id, w, sw);
+      if (lane == job % a.top) chosen = id;
+      if (blockIdx.x == 0 && job % a.top == 0) {
+        float* o = a.r.wts + (size_t)(job / a.top) * a.slots;
+        if (lane < a.top) { a.r.ids[job + lane] = id; o[lane] = w; }
+        if (a.r.shared && lane == 0) o[a.top] = sw;
+      }
+    }
+    __syncthreads();
+  }
+  const int expert = sh ? 0 : a.r.z ? chosen : a.r.ids[job];
   const int row = sh ? job - a.pairs : job / a.top, M = sh ? a.SM : a.M, K = sh ? a.SK : a.K, words = K / 8;
-  const __nv_bfloat16* w = sh ? a.sw : a.w + (size_t)a.ids[job] * (a.gated ? 2 : 1) * M * K;
+  const __nv_bfloat16* w = sh ? a.sw : a.w + (size_t)expert * (a.gated ? 2 : 1) * M * K;
   const __nv_bfloat16* x = a.gated ? (sh ? a.sx : a.x) + (size_t)row * K : (sh ? a.sx + (size_t)row * K : a.x + (size_t)job * K);
   __nv_bfloat16* out = a.gated ? (sh ? a.sout + (size_t)row * M : a.out + (size_t)job * M)
                                : a.out + ((size_t)row * a.slots + (sh ? a.top : job % a.top)) * M;
@@ -268,10 +311,11 @@ int sfb_rows_moe_route(const void* z, int64_t ld, void* ids, void* wts, int n, i
   return (int)sfb_launch(moe_route_kernel, dim3((n + 7) / 8), dim3(256), 0, stream, a);
 }
 
-// tiles: 4 ints each, at most pairs / tile + min(E, pairs) of them
-int sfb_rows_moe_plan(const void* ids, void* order, void* tiles, void* count, int pairs, int E, int tile, cudaStream_t stream) {
-  if (pairs < 1 || E < 1 || E > MAX_E || tile < 1) return (int)cudaErrorInvalidValue;
-  PlanArgs a{(const int*)ids, (int*)order, (int*)tiles, (int*)count, pairs, E, tile};
+// tiles: 4 ints each, at most pairs / tile + min(E, pairs) of them.  z: the choice is made here (few rows), null: ids are there.
+int sfb_rows_moe_plan(const void* z, int64_t ld, void* ids, void* wts, void* order, void* tiles, void* count, int n, int E, int top, int shared, int tile,
+                      cudaStream_t stream) {
+  if (n < 1 || E < 1 || E > MAX_E || top < 1 || top > MAX_TOP || top > E || tile < 1 || (long long)n * top >= 1 << 20) return (int)cudaErrorInvalidValue;
+  PlanArgs a{{(const float*)z, ld, (int*)ids, (float*)wts, n, E, top, shared}, (int*)order, (int*)tiles, (int*)count, n * top, E, tile};
   return (int)sfb_launch(moe_plan_kernel, dim3(1), dim3(1024), 0, stream, a);
 }
 
@@ -284,13 +328,14 @@ int sfb_rows_moe_tile(const void* x, const void* w, void* out, const void* order
   return (int)(fp32 ? sfb_launch(moe_tile_kernel<float>, g, b, 0, stream, a) : sfb_launch(moe_tile_kernel<__nv_bfloat16>, g, b, 0, stream, a));
 }
 
-// bf16, K and SK multiples of 8
-int sfb_rows_moe_gemv(const void* ids, const void* x, const void* w, void* out, const void* sx, const void* sw, void* sout, int pairs, int n, int M, int K, int SM,
+// bf16, K and SK multiples of 8; z: the choice of E experts is made here, null: ids are there
+int sfb_rows_moe_gemv(const void* z, int64_t ld, int E, void* ids, void* wts, const void* x, const void* w, void* out, const void* sx, const void* sw, void* sout, int pairs, int n, int M, int K, int SM,
                       int SK, int top, int slots, int gated, float alpha, float limit, float slimit, cudaStream_t stream) {
   const int kmax = sw && SK > K ? SK : K;
   if (n < 1 || pairs != n * top || pairs + n > 65535 || M < 1 || K < 8 || K % 8 || (sw && (SM < 1 || SK < 8 || SK % 8)) || kmax * 2 > 200 * 1024)
     return (int)cudaErrorInvalidValue;
-  GemvArgs a{(const int*)ids, (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, (const __nv_bfloat16*)sx, (const __nv_bfloat16*)sw,
+  if (z && (!gated || E < top || E > MAX_E || top > MAX_TOP || slots < top)) return (int)cudaErrorInvalidValue;
+  GemvArgs a{{(const float*)z, ld, (int*)ids, (float*)wts, n, E, top, slots - top}, (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, (const __nv_bfloat16*)sx, (const __nv_bfloat16*)sw,
              (__nv_bfloat16*)sout, pairs, n, M, K, SM, SK, top, slots, gated, alpha, limit, slimit};
   const int jobs = pairs + (sw ? n : 0), big = sw && SM > M ? SM : M, outs = gated ? big : (big + 1) / 2;
   int bx = (outs + 7) / 8, cap = (148 * 4 + jobs - 1) / jobs;

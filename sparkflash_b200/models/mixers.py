@@ -607,17 +607,18 @@ class MixtureFF:
         n, d, top, slots = s.n, h.shape[1], self.top, self.slots
         z = R.head(h, self.router, s.scratch.get("moe_z", n, self.router.shape[0]), "router")
         ids, wts = s.scratch.get("moe_ids", n, top), s.scratch.get("moe_w", n, slots)
-        R.moe_route(z, ids, wts, self.E, top, self.shared)
         act, parts = s.scratch.get("moe_act", n * top, self.ff), s.scratch.get("moe_parts", n, slots, d)
         s_act = s.scratch.get("ff_act", n, self.shared_ff) if self.shared else None
         if R.moe_gemv_takes(h, self.ff, self.shared_ff):
             side = (h, self.s_in, s_act, self.shared_ff, self.shared_limit) if self.shared else None
-            R.moe_gemv(ids, h, self.w_in, act, side, n, self.ff, top, slots, True, self.alpha, self.limit)
-            R.moe_gemv(ids, act, self.w_out, parts, (s_act, self.s_out, None, d, 0.0) if self.shared else None, n, d, top, slots, False)
+            R.moe_gemv(z, ids, wts, h, self.w_in, act, side, n, self.ff, top, slots, True, self.alpha, self.limit)
+            R.moe_gemv(None, ids, wts, act, self.w_out, parts, (s_act, self.s_out, None, d, 0.0) if self.shared else None, n, d, top, slots, False)
             return parts, wts
         plan = (s.scratch.get("moe_order", n * top), s.scratch.get("moe_tiles", R.moe_tiles(n, self.E, top, self.tile), 4), s.scratch.get("moe_count", 4),
                 R.moe_tiles(n, self.E, top, self.tile))
-        R.moe_plan(ids, *plan[:3], self.E, self.tile)
+        if n > R.MOE_PLAN_ROWS:
+            R.moe_route(z, ids, wts, self.E, top, self.shared)
+        R.moe_plan(z if n <= R.MOE_PLAN_ROWS else None, ids, wts, *plan[:3], self.E, top, self.shared, self.tile)
         if self.tc:
             few, x = n <= R.MOE_GATHER_ROWS, h
             if not few:
@@ -649,7 +650,6 @@ class TokenInput:
 
     def run(self, s, h):
         n = s.n
-        z = R.linear(h, self.gate, None, s.scratch.get("side_z", n, self.dim))
-        g = s.scratch.get("side_g", n, self.dim)
-        R.token_gate(z, self.table, self.col0, s.tokens, g, n, s.status)
+        z, g = s.scratch.get("side_z", n, self.dim), s.scratch.get("side_g", n, self.dim)
+        R.token_linear(h, self.gate, self.table, self.col0, s.tokens, z, g, s.status)
         return R.linear(g, self.proj, None, s.scratch.get("y", n, h.shape[1]))

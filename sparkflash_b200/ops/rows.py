@@ -68,6 +68,17 @@ def rot_append(proj, cs, dims, q, kpool, vpool, v_first, lam, table, row_lane, r
                                            c_int(dims), _fp32(q), _p(status), _stream()), "rows_rot_append")
 
 
+def token_linear(x, w, table, col0, tokens, z, out, status):
+    """out = gelu(x w^T) * table[token, col0 : col0 + dim]: one kernel for few rows, else a product to ``z`` and token_gate."""
+    if _gemv_takes(x):
+        _check(_lib.rows().sfb_rows_gemv_token(_p(w), _p(x), _p(out), *_strides(table), _p(tokens), c_int(col0), c_int(table.shape[0]), c_int(x.shape[0]),
+                                               c_int(w.shape[0]), c_int(x.shape[1]), _p(status), _stream()), "rows_gemv")
+        return out
+    linear(x, w, None, z)
+    token_gate(z, table, col0, tokens, out, x.shape[0], status)
+    return out
+
+
 def token_gate(z, table, col0, tokens, out, n, status):
     """out = gelu(z) * table[token, col0 : col0 + dim]."""
     _check(_lib.rows().sfb_rows_token_gate(_p(z), _p(table), _p(tokens), _p(out), c_int(n), c_int(z.shape[1]), c_int64(table.stride(0)), c_int(col0),
@@ -446,8 +457,14 @@ def moe_route(z, ids, wts, experts, top, shared):
            "rows_moe_route")
 
 
-def moe_plan(ids, order, tiles, count, experts, tile):
-    _check(_lib.rows().sfb_rows_moe_plan(_p(ids), _p(order), _p(tiles), _p(count), c_int(ids.numel()), c_int(experts), c_int(tile), _stream()), "rows_moe_plan")
+MOE_PLAN_ROWS = 128        # up to this many rows the plan makes the choice itself
+
+
+def moe_plan(z, ids, wts, order, tiles, count, experts, top, shared, tile):
+    """``z``: logits (few rows: the choice is made here), or None: ``ids`` are there."""
+    zp, ld = _strides(z)
+    _check(_lib.rows().sfb_rows_moe_plan(zp, ld, _p(ids), _p(wts), _p(order), _p(tiles), _p(count), c_int(ids.shape[0]), c_int(experts), c_int(top),
+                                         c_int(shared), c_int(tile), _stream()), "rows_moe_plan")
 
 
 def moe_tile(x, w, out, plan, M, top, slots, gated, alpha=0.0, limit=0.0):
@@ -484,9 +501,10 @@ def moe_gemv_takes(x: torch.Tensor, ff: int, shared_ff: int) -> bool:
     return x.dtype == torch.bfloat16 and n <= GEMV_ROWS and K % 8 == 0 and ff % 8 == 0 and shared_ff % 8 == 0 and max(K, ff, shared_ff) * 2 <= 200 * 1024
 
 
-def moe_gemv(ids, x, w, out, shared, n, M, top, slots, gated, alpha=0.0, limit=0.0):
-    """Few rows; ``shared``: (x, w, out, M, limit) of the shared expert or None."""
+def moe_gemv(z, ids, wts, x, w, out, shared, n, M, top, slots, gated, alpha=0.0, limit=0.0):
+    """Few rows; ``z``: logits, the experts are chosen here and left in ``ids`` and ``wts``; None: ``ids`` are there.  ``shared``: (x, w, out, M,
+    limit) of the shared expert or None."""
     sx, sw, sout, sm, sl = shared if shared is not None else (None, None, None, 0, 0.0)
-    _check(_lib.rows().sfb_rows_moe_gemv(_p(ids), _p(x), _p(w), _p(out), _p(sx), _p(sw), _p(sout), c_int(ids.numel()), c_int(n), c_int(M), c_int(w.shape[2]),
+    _check(_lib.rows().sfb_rows_moe_gemv(*_strides(z), c_int(w.shape[0]), _p(ids), _p(wts), _p(x), _p(w), _p(out), _p(sx), _p(sw), _p(sout), c_int(ids.numel()), c_int(n), c_int(M), c_int(w.shape[2]),
                                          c_int(sm), c_int(sw.shape[1] if sw is not None else 0), c_int(top), c_int(slots), c_int(gated), c_float(alpha),
                                          c_float(limit), c_float(sl), _stream()), "rows_moe_gemv")

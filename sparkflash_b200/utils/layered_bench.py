@@ -102,6 +102,12 @@ def timed(fn, reps: int, warm: int = 3, flush=None) -> float:
     return statistics.median(ts)
 
 
+def _own(ids: list[int], lane: int) -> list[int]:
+    """A lane's prompt: the same tokens from another place on, so that lanes do not choose the same experts."""
+    k = 97 * lane % len(ids)
+    return ids[k:] + ids[:k]
+
+
 def throughput(design: str, name: str, prompt: int = 8192, chunk: int = 4096, streams=(1, 16, 64), steps: int = 32) -> dict:
     """Prefill tok/s of one prompt in portions, decode tok/s at several stream counts against ``prompt`` cached tokens (and end to
     end through ``step``, which copies inputs from pinned memory and reads the tokens back)."""
@@ -113,15 +119,16 @@ def throughput(design: str, name: str, prompt: int = 8192, chunk: int = 4096, st
     cuts = [(p, min(p + chunk, prompt)) for p in range(0, prompt, chunk)]
 
     def prefill(lane):
+        own = _own(ids, lane)
         for a, b in cuts:
-            eng.step(ids[a:b], [lane] * (b - a), list(range(a, b)), head="last" if b == prompt else False, sync=False)
+            eng.step(own[a:b], [lane] * (b - a), list(range(a, b)), head="last" if b == prompt else False, sync=False)
     ms = timed(lambda: prefill(0), 5)
     out["prefill"] = {"tok_s": prompt / ms * 1e3, "ms": ms, "prompt": prompt, "chunk": chunk}
     for lane in range(1, lanes):
         prefill(lane)
     torch.cuda.synchronize()
     for n in streams:
-        tok, lane, pos = [5] * n, list(range(n)), prompt
+        tok, lane, pos = [(5 + 37 * k) % eng.model.vocab for k in range(n)], list(range(n)), prompt
 
         def one(sync):
             nonlocal pos
@@ -374,8 +381,8 @@ def decode_table(design: str, name: str, n: int = 16, ctx: int = 8192, reps: int
     for lane in range(n):
         for a in range(0, ctx, 4096):
             b = min(ctx, a + 4096)
-            eng.step(ids[a:b], [lane] * (b - a), list(range(a, b)), head=False)
-    ts = [roofline.timed_step(eng, [5] * n, list(range(n)), [ctx + i] * n, lead_cycles=30_000_000) for i in range(reps + 1)]
+            eng.step(_own(ids, lane)[a:b], [lane] * (b - a), list(range(a, b)), head=False)
+    ts = [roofline.timed_step(eng, [(5 + 37 * k) % eng.model.vocab for k in range(n)], list(range(n)), [ctx + i] * n, lead_cycles=30_000_000) for i in range(reps + 1)]
     eng.check_status()
     cfg = eng.cfg
     eng.close()
