@@ -89,27 +89,33 @@ struct PlanArgs {
   int* count;               // number of tiles
   int pairs, E, tile;
 };
-constexpr int BATCH = 32;   // pairs a thread holds: their expert, and how many of it came before (20 bits)
+constexpr int BATCH = 16;   // pairs a thread holds: their expert, and how many of it came before (20 bits)
 
+// one block of at least E threads
 __global__ void __launch_bounds__(1024) moe_plan_kernel(PlanArgs a) {
-  __shared__ int cnt[MAX_E], wsum[2][32];
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  __shared__ int cnt[MAX_E], base[MAX_E], wsum[2][32];
+  const int tid = threadIdx.x, nt = blockDim.x, lane = tid & 31, warp = tid >> 5;
   cnt[tid] = 0;
   pdl_launch_dependents();
   pdl_wait();
   if (a.r.z)
-    for (int row = warp; row < a.r.n; row += 32) route_row(a.r, row);
+    for (int row = warp; row < a.r.n; row += nt >> 5) route_row(a.r, row);
   __syncthreads();          // (orders the block's own ids too)
   uint32_t held[BATCH];
   // a place inside its expert for every pair
   auto places = [&](int p0) {
 #pragma unroll
-    for (int k = 0; k < BATCH; ++k) held[k] = p0 + k * 1024 + tid < a.pairs ? (uint32_t)a.r.ids[p0 + k * 1024 + tid] : 0u;
+    for (int k = 0; k < BATCH; ++k) {
+      if (p0 + k * nt >= a.pairs) break;
+      held[k] = p0 + k * nt + tid < a.pairs ? (uint32_t)a.r.ids[p0 + k * nt + tid] : 0u;
+    }
 #pragma unroll
-    for (int k = 0; k < BATCH; ++k)
-      if (p0 + k * 1024 + tid < a.pairs) held[k] = held[k] << 20 | (uint32_t)atomicAdd(&cnt[held[k]], 1);
+    for (int k = 0; k < BATCH; ++k) {
+      if (p0 + k * nt >= a.pairs) break;
+      if (p0 + k * nt + tid < a.pairs) held[k] = held[k] << 20 | (uint32_t)atomicAdd(&cnt[held[k]], 1);
+    }
   };
-  for (int p0 = 0; p0 < a.pairs; p0 += BATCH * 1024) places(p0);
+  for (int p0 = 0; p0 < a.pairs; p0 += BATCH * nt) places(p0);
   __syncthreads();
   const int c = cnt[tid], t = (c + a.tile - 1) / a.tile;
   int sc = c, st = t;       // inclusive sums of pairs and of tiles over the experts
@@ -121,19 +127,18 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(PlanArgs a) {
   if (lane == 31) { wsum[0][warp] = sc; wsum[1][warp] = st; }
   __syncthreads();
   for (int w = 0; w < warp; ++w) { sc += wsum[0][w]; st += wsum[1][w]; }
-  const int first = sc - c;
-  for (int k = 0; k < t; ++k) reinterpret_cast<int4*>(a.tiles)[st - t + k] = make_int4(tid, first + k * a.tile, min(a.tile, c - k * a.tile), 0);
-  if (tid == 1023) *a.count = st;
-  const bool once = a.pairs <= BATCH * 1024;
-  __shared__ int base[MAX_E];
-  base[tid] = first;
+  for (int k = 0; k < t; ++k) reinterpret_cast<int4*>(a.tiles)[st - t + k] = make_int4(tid, sc - c + k * a.tile, min(a.tile, c - k * a.tile), 0);
+  if (tid == nt - 1) *a.count = st;
+  base[tid] = sc - c;
   cnt[tid] = 0;             // more pairs than the threads hold: they take their places again
   __syncthreads();
-  for (int p0 = 0; p0 < a.pairs; p0 += BATCH * 1024) {
-    if (!once) places(p0);
+  for (int p0 = 0; p0 < a.pairs; p0 += BATCH * nt) {
+    if (a.pairs > BATCH * nt) places(p0);
 #pragma unroll
-    for (int k = 0; k < BATCH; ++k)
-      if (p0 + k * 1024 + tid < a.pairs) a.order[base[held[k] >> 20] + (int)(held[k] & 0xfffffu)] = p0 + k * 1024 + tid;
+    for (int k = 0; k < BATCH; ++k) {
+      if (p0 + k * nt >= a.pairs) break;
+      if (p0 + k * nt + tid < a.pairs) a.order[base[held[k] >> 20] + (int)(held[k] & 0xfffffu)] = p0 + k * nt + tid;
+    }
   }
 }
 
@@ -316,7 +321,7 @@ int sfb_rows_moe_plan(const void* z, int64_t ld, void* ids, void* wts, void* ord
                       cudaStream_t stream) {
   if (n < 1 || E < 1 || E > MAX_E || top < 1 || top > MAX_TOP || top > E || tile < 1 || (long long)n * top >= 1 << 20) return (int)cudaErrorInvalidValue;
   PlanArgs a{{(const float*)z, ld, (int*)ids, (float*)wts, n, E, top, shared}, (int*)order, (int*)tiles, (int*)count, n * top, E, tile};
-  return (int)sfb_launch(moe_plan_kernel, dim3(1), dim3(1024), 0, stream, a);
+  return (int)sfb_launch(moe_plan_kernel, dim3(1), dim3(E > 256 || n * top > 2048 ? 1024 : 256), 0, stream, a);
 }
 
 // tiles of at most 32 pairs

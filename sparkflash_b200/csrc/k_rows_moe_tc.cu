@@ -5,6 +5,8 @@
 //           are gathered by TMA straight from the layer's input (four rows a copy); many are brought into plan order first (`pick`)
 //   down    128 pairs x 256 columns; rows in plan order; every result row goes to its [row][choice]
 //
+// The shared expert's rows (all of the step, in order, with sizes of their own) are tiles of the same launches, ahead of the others.
+//
 // Persistent: one CTA per SM takes every gridDim-th of the tiles x column blocks (the column blocks of a tile side by side, so that its rows
 // and its expert's weights stay in L2).  Warp 0 copies (K in steps of 64 through a ring of four stages), warp 1 issues the products, warps
 // 2-5 take the results out of tensor memory, where two accumulators of 256 columns take turns, so that a tile's results leave under the
@@ -19,12 +21,29 @@ constexpr int THREADS = 192, ROWS = 128, COLS = 256, KS = 64, ST = 4, XSLAB = RO
 
 struct Args {
   const int *order, *tiles, *count;
-  __nv_bfloat16* out;        // gated: [pairs, M]; down: [n, slots, M]
-  int M, K, top, slots, cblocks;     // cblocks: blocks of 128 (gated) or 256 columns
-  int wide;                  // result rows lie on 16-byte boundaries
-  float alpha, limit;
+  __nv_bfloat16 *out, *sout; // gated: [pairs, M], the shared expert's [n, SM]; down: [n, slots, M]
+  int M, K, SM, SK, top, slots, cblocks, sblocks;     // cblocks, sblocks: blocks of 128 (gated) or 256 columns
+  int stotal, n;             // tiles x column blocks of the shared expert (0: none), its rows
+  float alpha, limit, slimit;
   Status* status;
 };
+
+// what one turn of a CTA works on
+struct Job {
+  int4 t;                    // expert, first place (shared: row), pairs, -
+  int c0, M, K, shared;
+};
+template <bool GATED>
+__device__ __forceinline__ Job job(const Args& a, int b) {
+  Job j;
+  j.shared = b < a.stotal;
+  const int x = j.shared ? b : b - a.stotal, blocks = j.shared ? a.sblocks : a.cblocks, ti = x / blocks;
+  j.t = j.shared ? make_int4(0, ti * 128, min(128, a.n - ti * 128), 0) : reinterpret_cast<const int4*>(a.tiles)[ti];
+  j.c0 = (x % blocks) * (GATED ? 128 : 256);
+  j.M = j.shared ? a.SM : a.M;
+  j.K = j.shared ? a.SK : a.K;
+  return j;
+}
 
 struct Smem {
   alignas(1024) uint8_t x[ST * XSLAB];
@@ -61,7 +80,8 @@ __global__ void __launch_bounds__(256) moe_pick_kernel(const uint4* x, const int
 
 template <bool GATED, bool GATHER>
 __global__ void __launch_bounds__(THREADS, 1)
-moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ CUtensorMap mw, Args a) {
+moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ CUtensorMap mw, const __grid_constant__ CUtensorMap msx,
+                const __grid_constant__ CUtensorMap msw, Args a) {
   extern __shared__ uint8_t raw[];
   Smem& S = *reinterpret_cast<Smem*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
   const int tid = threadIdx.x, warp = __shfl_sync(0xffffffffu, tid >> 5, 0), lane = tid & 31;
@@ -82,32 +102,33 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
   fence_after();
   pdl_wait();
   const uint32_t tmem = S.tmem;
-  const int total = *a.count * a.cblocks, steps = (a.K + KS - 1) / KS;
-  const int4* plan = reinterpret_cast<const int4*>(a.tiles);
+  const int total = a.stotal + *a.count * a.cblocks;
 
   if (warp == 0) {
     int it = 0;              // stages filled so far
     for (int b = blockIdx.x; b < total && !*dead; b += gridDim.x) {
-      const int4 t = plan[b / a.cblocks];
-      const int c0 = (b % a.cblocks) * (GATED ? 128 : 256);
+      const Job j = job<GATED>(a, b);
+      const int4 t = j.t;
+      const bool gather = GATHER && !j.shared;
       int4 rows = make_int4(0, 0, 0, 0);      // a lane gathers four rows, the tile's last one again past its end; lanes past it none
-      if (GATHER) {
+      if (gather) {
         int* r = reinterpret_cast<int*>(&rows);
 #pragma unroll
         for (int k = 0; k < 4; ++k) r[k] = a.order[t.y + min(lane * 4 + k, t.z - 1)] / a.top;
       }
-      const int wrow = t.x * (GATED ? 2 : 1) * a.M + c0;
+      const int wrow = t.x * (GATED ? 2 : 1) * j.M + j.c0, steps = (j.K + KS - 1) / KS;
+      const CUtensorMap *x = j.shared ? &msx : &mx, *w = j.shared ? &msw : &mw;
       for (int k = 0; k < steps; ++k, ++it) {
         const int st = it % ST, ph = (it / ST) & 1;
         const bool ok = mbar_wait(&S.empty[st], ph ^ 1, dead);
         if (!__all_sync(0xffffffffu, ok)) break;
-        if (lane == 0) mbar_expect(&S.full[st], (GATHER ? (t.z + 3) / 4 * 512 : XSLAB) + WSLAB);
+        if (lane == 0) mbar_expect(&S.full[st], (gather ? (t.z + 3) / 4 * 512 : XSLAB) + WSLAB);
         __syncwarp();
-        if (GATHER && lane * 4 < t.z) gather4(S.x + st * XSLAB + lane * 512, &mx, k * KS, rows, &S.full[st]);
+        if (gather && lane * 4 < t.z) gather4(S.x + st * XSLAB + lane * 512, &mx, k * KS, rows, &S.full[st]);
         if (lane == 0) {
-          if (!GATHER) tma2d(S.x + st * XSLAB, &mx, k * KS, t.y, &S.full[st]);
-          tma2d(S.w + st * WSLAB, &mw, k * KS, wrow, &S.full[st]);
-          tma2d(S.w + st * WSLAB + XSLAB, &mw, k * KS, wrow + (GATED ? a.M : 128), &S.full[st]);
+          if (!gather) tma2d(S.x + st * XSLAB, x, k * KS, t.y, &S.full[st]);
+          tma2d(S.w + st * WSLAB, w, k * KS, wrow, &S.full[st]);
+          tma2d(S.w + st * WSLAB + XSLAB, w, k * KS, wrow + (GATED ? j.M : 128), &S.full[st]);
         }
       }
     }
@@ -122,7 +143,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
       int it = 0, n = 0;
       bool ok = true;
       for (int b = blockIdx.x; ok && b < total; b += gridDim.x, ++n) {
-        const int acc = n & 1;
+        const int acc = n & 1, steps = ((b < a.stotal ? a.SK : a.K) + KS - 1) / KS;
         if (!(ok = mbar_wait(&S.acc_empty[acc], ((n >> 1) & 1) ^ 1, dead))) break;
         fence_after();
         for (int k = 0; k < steps; ++k, ++it) {
@@ -144,18 +165,20 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
     const uint32_t lanes = (uint32_t)(w4 * 32) << 16;
     int n = 0;
     for (int b = blockIdx.x; b < total; b += gridDim.x, ++n) {
-      const int4 t = plan[b / a.cblocks];
-      const int c0 = (b % a.cblocks) * (GATED ? 128 : 256), acc = n & 1;
-      const bool in = r < t.z;
+      const Job j = job<GATED>(a, b);
+      const int acc = n & 1;
+      const bool in = r < j.t.z;
       size_t row = 0;
-      if (GATED) row = (size_t)(t.y + r);
-      else if (in) { const int pair = a.order[t.y + r]; row = (size_t)(pair / a.top) * a.slots + pair % a.top; }
-      __nv_bfloat16* o = a.out + row * a.M + c0;
+      if (GATED) row = (size_t)(j.t.y + r);
+      else if (j.shared) row = (size_t)(j.t.y + r) * a.slots + a.top;
+      else if (in) { const int pair = a.order[j.t.y + r]; row = (size_t)(pair / a.top) * a.slots + pair % a.top; }
+      __nv_bfloat16* o = (GATED && j.shared ? a.sout : a.out) + row * j.M + j.c0;
+      const float limit = j.shared ? a.slimit : a.limit;
       const bool ok = mbar_wait(&S.acc_full[acc], (n >> 1) & 1, dead);
       if (!__all_sync(0xffffffffu, ok)) break;
       fence_after();
       const uint32_t ta = tmem + acc * COLS + lanes;
-      const int width = min(GATED ? 128 : 256, a.M - c0);
+      const int width = min(GATED ? 128 : 256, j.M - j.c0);
       for (int c = 0; c < width; c += 32) {
         float f[32];
         ld32(ta + c, f);
@@ -164,20 +187,14 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
           ld32(ta + 128 + c, u);
           wait_ld();
 #pragma unroll
-          for (int k = 0; k < 32; ++k) f[k] = rows::gate_clamp<__nv_bfloat16>(f[k], u[k], a.alpha, a.limit);
+          for (int k = 0; k < 32; ++k) f[k] = rows::gate_clamp<__nv_bfloat16>(f[k], u[k], a.alpha, limit);
         } else {
           wait_ld();
         }
         if (in) {
-          if (a.wide) {
 #pragma unroll
-            for (int k = 0; k < 32; k += 8)
-              if (c + k < width) rows::store_v<__nv_bfloat16, 8>(o + c + k, f + k);      // M is a multiple of eight
-          } else {
-#pragma unroll
-            for (int k = 0; k < 32; ++k)
-              if (c + k < width) o[c + k] = __float2bfloat16_rn(f[k]);
-          }
+          for (int k = 0; k < 32; k += 8)
+            if (c + k < width) rows::store_v<__nv_bfloat16, 8>(o + c + k, f + k);      // M is a multiple of eight
         }
       }
       fence_before();
@@ -191,7 +208,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
 }
 
 template <bool GATED, bool GATHER>
-static int launch(const CUtensorMap* mx, const CUtensorMap* mw, const Args& a, int most, cudaStream_t st) {
+static int launch(const CUtensorMap* mx, const CUtensorMap* mw, const CUtensorMap* msx, const CUtensorMap* msw, const Args& a, int most, cudaStream_t st) {
   const size_t smem = sizeof(Smem) + 1024;
   static bool done = false;
   if (!done) {
@@ -202,8 +219,8 @@ static int launch(const CUtensorMap* mx, const CUtensorMap* mw, const Args& a, i
   int dev = 0, sms = 148;
   cudaGetDevice(&dev);
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-  const long long blocks = (long long)most * a.cblocks;
-  return (int)sfb_launch(moe_gemm_kernel<GATED, GATHER>, dim3((unsigned)(blocks < sms ? blocks : sms)), dim3(THREADS), smem, st, *mx, *mw, a);
+  const long long blocks = (long long)most * a.cblocks + a.stotal;
+  return (int)sfb_launch(moe_gemm_kernel<GATED, GATHER>, dim3((unsigned)(blocks < sms ? blocks : sms)), dim3(THREADS), smem, st, *mx, *mw, *msx, *msw, a);
 }
 
 }  // namespace rmoetc
@@ -220,17 +237,22 @@ int sfb_rows_moe_pick(const void* x, const void* order, void* out, int pairs, in
   return (int)sfb_launch(moe_pick_kernel, dim3((pairs + 7) / 8), dim3(256), 0, stream, (const uint4*)x, (const int*)order, (uint4*)out, pairs, top, K / 8);
 }
 
-// mx: rows [pairs, K] in plan order, box 128 rows, or (gather) rows [n, K], box of one row; mw: weights [E (2) M, K], box 128 rows.  K: a
-// multiple of 8; most: the most tiles (of up to 128 pairs) that the plan can hold.
-int sfb_rows_moe_gemm(const void* mx, const void* mw, const void* order, const void* tiles, const void* count, void* out, int most, int M, int K, int top, int slots,
-                      int gated, int gather, float alpha, float limit, void* status, cudaStream_t stream) {
-  if (most < 1 || M < 1 || K < 8 || K % 8 || top < 1 || (gather && !gated)) return (int)cudaErrorInvalidValue;
+// mx: rows [pairs, K] in plan order, box 128 rows, or (gather) rows [n, K], box of one row; mw: weights [E (2) M, K], box 128 rows.  msx, msw: the
+// same of the shared expert (rows in order), or null.  M, K, SM and SK: multiples of 8; most: the most tiles (of up to 128 pairs) that the plan
+// can hold.
+int sfb_rows_moe_gemm(const void* mx, const void* mw, const void* msx, const void* msw, const void* order, const void* tiles, const void* count, void* out, void* sout,
+                      int most, int n, int M, int K, int SM, int SK, int top, int slots, int gated, int gather, float alpha, float limit, float slimit, void* status,
+                      cudaStream_t stream) {
+  if (most < 1 || n < 1 || M < 8 || M % 8 || K < 8 || K % 8 || top < 1 || (gather && !gated) || (msx && (SM < 8 || SM % 8 || SK < 8 || SK % 8 || slots <= top)) ||
+      (uintptr_t)out % 16 || (uintptr_t)sout % 16)
+    return (int)cudaErrorInvalidValue;
   const int per = gated ? 128 : 256;
-  Args a{(const int*)order, (const int*)tiles, (const int*)count, (__nv_bfloat16*)out, M, K, top, slots, (M + per - 1) / per, M % 8 == 0 && (uintptr_t)out % 16 == 0,
-         alpha, limit, (Status*)status};
-  const CUtensorMap *x = (const CUtensorMap*)mx, *w = (const CUtensorMap*)mw;
-  if (gather) return launch<true, true>(x, w, a, most, stream);
-  return gated ? launch<true, false>(x, w, a, most, stream) : launch<false, false>(x, w, a, most, stream);
+  Args a{(const int*)order, (const int*)tiles, (const int*)count, (__nv_bfloat16*)out, (__nv_bfloat16*)sout, M, K, SM, SK, top, slots, (M + per - 1) / per,
+         (SM + per - 1) / per, 0, n, alpha, limit, slimit, (Status*)status};
+  if (msx) a.stotal = (n + 127) / 128 * a.sblocks;
+  const CUtensorMap *x = (const CUtensorMap*)mx, *w = (const CUtensorMap*)mw, *sx = msx ? (const CUtensorMap*)msx : x, *sw = msw ? (const CUtensorMap*)msw : w;
+  if (gather) return launch<true, true>(x, w, sx, sw, a, most, stream);
+  return gated ? launch<true, false>(x, w, sx, sw, a, most, stream) : launch<false, false>(x, w, sx, sw, a, most, stream);
 }
 
 }  // extern "C"

@@ -12,7 +12,7 @@ row selection and the sampler - and speaks the contract of serve/driver.py.  A m
     bind(engine)                       reserve scratch, register state tensors
     forward(step) -> [head rows, vocab] float32 logits (None without a head)
 
-and writes no loop, cache or batching of its own (models/fanodra.py and models/gudutar.py are two; ``LayeredModel`` has what they share).
+and writes no loop, cache or batching of its own (models/fanodra.py, models/gudutar.py and models/lifulorn.py; ``LayeredModel`` has what they share).
 """
 from __future__ import annotations
 

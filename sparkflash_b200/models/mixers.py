@@ -589,7 +589,7 @@ class MixtureFF:
 
     def reserve(self, e) -> None:
         n, dt, d = e.max_rows, self.router.dtype, self.router.shape[1]
-        self.tc = R.moe_tc_supports(dt, d, self.ff)
+        self.tc = R.moe_tc_supports(dt, d, self.ff, self.shared_ff)
         self.tile = R.MOE_TC_TILE if self.tc else R.MOE_TILE
         e.scratch.reserve("moe_z", n * self.router.shape[0], torch.float32)
         e.scratch.reserve("moe_w", n * self.slots, torch.float32)
@@ -600,8 +600,9 @@ class MixtureFF:
         if self.tc and n > R.MOE_GATHER_ROWS:
             e.scratch.reserve("moe_x", n * self.top * d, dt)
         if self.shared:
-            e.scratch.reserve("proj", n * 2 * self.shared_ff, dt)
             e.scratch.reserve("ff_act", n * self.shared_ff, dt)
+            if not self.tc:
+                e.scratch.reserve("proj", n * 2 * self.shared_ff, dt)
 
     def run(self, s, h):
         n, d, top, slots = s.n, h.shape[1], self.top, self.slots
@@ -609,10 +610,11 @@ class MixtureFF:
         ids, wts = s.scratch.get("moe_ids", n, top), s.scratch.get("moe_w", n, slots)
         act, parts = s.scratch.get("moe_act", n * top, self.ff), s.scratch.get("moe_parts", n, slots, d)
         s_act = s.scratch.get("ff_act", n, self.shared_ff) if self.shared else None
+        first = (h, self.s_in, s_act, self.shared_ff, self.shared_limit) if self.shared else None        # the shared expert's part in both products
+        second = (s_act, self.s_out, None, d, 0.0) if self.shared else None
         if R.moe_gemv_takes(h, self.ff, self.shared_ff):
-            side = (h, self.s_in, s_act, self.shared_ff, self.shared_limit) if self.shared else None
-            R.moe_gemv(z, ids, wts, h, self.w_in, act, side, n, self.ff, top, slots, True, self.alpha, self.limit)
-            R.moe_gemv(None, ids, wts, act, self.w_out, parts, (s_act, self.s_out, None, d, 0.0) if self.shared else None, n, d, top, slots, False)
+            R.moe_gemv(z, ids, wts, h, self.w_in, act, first, n, self.ff, top, slots, True, self.alpha, self.limit)
+            R.moe_gemv(None, ids, wts, act, self.w_out, parts, second, n, d, top, slots, False)
             return parts, wts
         plan = (s.scratch.get("moe_order", n * top), s.scratch.get("moe_tiles", R.moe_tiles(n, self.E, top, self.tile), 4), s.scratch.get("moe_count", 4),
                 R.moe_tiles(n, self.E, top, self.tile))
@@ -624,11 +626,11 @@ class MixtureFF:
             if not few:
                 x = s.scratch.get("moe_x", n * top, d)
                 R.moe_pick(h, plan[0], x, top)
-            R.moe_gemm(x, self.w_in, act, plan, self.ff, top, slots, True, s.status, self.alpha, self.limit, few)
-            R.moe_gemm(act, self.w_out, parts, plan, d, top, slots, False, s.status)
-        else:
-            R.moe_tile(h, self.w_in, act, plan, self.ff, top, slots, True, self.alpha, self.limit)
-            R.moe_tile(act, self.w_out, parts, plan, d, top, slots, False)
+            R.moe_gemm(x, self.w_in, act, plan, first, n, self.ff, top, slots, True, s.status, self.alpha, self.limit, few)
+            R.moe_gemm(act, self.w_out, parts, plan, second, n, d, top, slots, False, s.status)
+            return parts, wts
+        R.moe_tile(h, self.w_in, act, plan, self.ff, top, slots, True, self.alpha, self.limit)
+        R.moe_tile(act, self.w_out, parts, plan, d, top, slots, False)
         if self.shared:
             R.gated_linear(h, self.s_in, s.scratch.get("proj", n, 2 * self.shared_ff), s_act, "clamp", self.alpha, self.shared_limit)
             R.linear(s_act, self.s_out, None, parts[:, top])

@@ -475,9 +475,9 @@ def moe_tile(x, w, out, plan, M, top, slots, gated, alpha=0.0, limit=0.0):
                                          c_int(slots), c_int(gated), c_float(alpha), c_float(limit), _fp32(out), _stream()), "rows_moe_tile")
 
 
-def moe_tc_supports(dtype: torch.dtype, width: int, ff: int) -> bool:
+def moe_tc_supports(dtype: torch.dtype, width: int, ff: int, shared_ff: int) -> bool:
     """Shapes the tensor-core products take (csrc/k_rows_moe_tc.cu)."""
-    return dtype == torch.bfloat16 and width % 8 == 0 and ff % 8 == 0
+    return dtype == torch.bfloat16 and width % 8 == 0 and ff % 8 == 0 and shared_ff % 8 == 0
 
 
 MOE_GATHER_ROWS = 256      # up to this many rows the product gathers its rows itself (csrc/k_rows_moe_tc.cu)
@@ -488,12 +488,16 @@ def moe_pick(x, order, out, top):
     _check(_lib.rows().sfb_rows_moe_pick(_p(x), _p(order), _p(out), c_int(out.shape[0]), c_int(top), c_int(x.shape[1]), _stream()), "rows_moe_pick")
 
 
-def moe_gemm(x, w, out, plan, M, top, slots, gated, status, alpha=0.0, limit=0.0, gather=False):
-    """``moe_tile`` on the tensor cores (tiles of up to 128 pairs); w and out in bf16; x in plan order, or ``gather``: the layer's rows."""
+def moe_gemm(x, w, out, plan, shared, n, M, top, slots, gated, status, alpha=0.0, limit=0.0, gather=False):
+    """``moe_tile`` on the tensor cores (tiles of up to 128 pairs); w and out in bf16; x in plan order, or ``gather``: the layer's rows.
+    ``shared``: (x, w, out, M, limit) of the shared expert, whose rows are done beside the pairs, or None."""
     order, tiles, count, most = plan
+    sx, sw, sout, sm, sl = shared if shared is not None else (None, None, None, 0, 0.0)
+    msx, msw = (tensor_map(sx, sx.shape[1], 128).ptr, tensor_map(sw, sw.shape[1], 128).ptr) if shared is not None else (None, None)
     mx, mw = tensor_map(x, x.shape[1], 1 if gather else 128), tensor_map(w, w.shape[2], 128)
-    _check(_lib.rows().sfb_rows_moe_gemm(mx.ptr, mw.ptr, _p(order), _p(tiles), _p(count), _p(out), c_int(most), c_int(M), c_int(w.shape[2]), c_int(top),
-                                         c_int(slots), c_int(gated), c_int(gather), c_float(alpha), c_float(limit), _p(status), _stream()), "rows_moe_gemm")
+    _check(_lib.rows().sfb_rows_moe_gemm(mx.ptr, mw.ptr, msx, msw, _p(order), _p(tiles), _p(count), _p(out), _p(sout), c_int(most), c_int(n), c_int(M),
+                                         c_int(w.shape[2]), c_int(sm), c_int(sw.shape[1] if sw is not None else 0), c_int(top), c_int(slots), c_int(gated),
+                                         c_int(gather), c_float(alpha), c_float(limit), c_float(sl), _p(status), _stream()), "rows_moe_gemm")
 
 
 def moe_gemv_takes(x: torch.Tensor, ff: int, shared_ff: int) -> bool:

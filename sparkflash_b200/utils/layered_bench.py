@@ -223,7 +223,7 @@ def lifulorn_work(cfg: LifulornConfig, n: int, ctx: int, head_rows: int, decode:
     per pair of bf16 terms; experts: the weights of those that the rows can touch, and their products."""
     d, W, side = cfg.width, roofline.ClassWork, cfg.side_dim
     out = {k: W() for k in ("rows_seam", "rows_conv", "rows_state", "rows_delta_tc", "rows_gated_norm", "rows_rot_append", "rows_attn_stream", "rows_attn_tc",
-                            "rows_act_mul", "rows_token_gate", "rows_moe_gemm", "rows_moe_gemv", "rows_moe_route", "rows_moe_plan", "rows_moe_pick", "linear", "router", "head")}
+                            "rows_token_gate", "rows_moe_gemm", "rows_moe_gemv", "rows_moe_route", "rows_moe_plan", "rows_moe_pick", "linear", "router", "head")}
     few = n <= 4
 
     def linear(k, m, name="linear"):
@@ -270,12 +270,9 @@ def lifulorn_work(cfg: LifulornConfig, n: int, ctx: int, head_rows: int, decode:
             if few:
                 out["rows_moe_gemv"].bytes += 2.0 * 3 * d * (n * top * ff + sff)
             else:
-                out["rows_moe_gemm"].bytes += 2.0 * (used * 3 * d * ff + n * (d + top * (2 * ff + d)))
+                out["rows_moe_gemm"].bytes += 2.0 * (3 * d * (used * ff + sff) + n * (d + top * (2 * ff + d) + 2 * sff + d))
                 out["rows_moe_pick"].bytes += 0.0 if decode else 2.0 * n * d * (1 + top)
-                out["rows_moe_gemm"].flops += 2.0 * n * top * 3 * d * ff
-                linear(d, 2 * sff)
-                linear(sff, d)
-                out["rows_act_mul"].bytes += n * sff * 6.0
+                out["rows_moe_gemm"].flops += 2.0 * n * 3 * d * (top * ff + sff)
             out["rows_seam"].bytes += n * d * (10.0 + 2.0 * (top + 1))
         linear(d, side)
         linear(side, d)

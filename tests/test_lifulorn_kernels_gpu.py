@@ -297,7 +297,7 @@ def test_mixture_of_experts(d, E, top, ff, sff, limits, n, dt):
     moe, s = MixtureFF(W({"p." + k: v for k, v in w.items()}, "p.", dt, "cuda"), spec, 1.702), _Step(n)
     assert moe.slots == top + (sff > 0)
     moe.reserve(s)
-    assert moe.tc == (dt == torch.bfloat16 and d % 8 == 0 and ff % 8 == 0)
+    assert moe.tc == (dt == torch.bfloat16 and d % 8 == ff % 8 == sff % 8 == 0)
     with R.exact_matmul():
         parts, wts = moe.run(s, h.cuda())
     assert s.status.tolist()[0] == 0
