@@ -335,23 +335,29 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
     const uint32_t id = idesc(2 * PT, 0, 1), id1 = idesc(PT, 0, 1), idt = idesc(2 * PT, 1, 1);
     const uint64_t dt = desc(smem_u32(ts), 16), ds = desc(smem_u32(ss), SLAB), dx = desc(smem_u32(xs), SLAB);
     const int kst = a.N / 16;
+    auto store_u = [&](int c) {
+      for (int t = 0; t < 2; ++t) tma_store2d(&mu, pt * PT, ((t * a.chunks + c0 + c) * a.H + h) * L, us + t * TILE);
+      bulk_commit();
+    };
     for (int c = 0; c < nc; ++c) {
       const uint64_t dk = desc(smem_u32(ks) + (c & 1) * 2 * SLAB, 16), dkt = desc(smem_u32(ks) + (c & 1) * 2 * SLAB, SLAB);
       wait_warp(&C.full[c & 1], (c >> 1) & 1, dead, 4);
-      __syncthreads();                                    // the state is in place
+      if (leader) bulk_wait_read();                       // the tile of the state before has left
+      __syncwarp();
+      __syncthreads();                                    // the state is in place (and the tile of U before)
       if (leader) {
         fence_after();
-        for (int t = 0; t < kst; ++t)
-          mma_ss(t_ks, dk + (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, ds + (uint64_t)t * (2048 >> 4), id, t ? 1u : 0u);
+#pragma unroll
+        for (int t = 0; t < 8; ++t)
+          if (t < kst) mma_ss(t_ks, dk + (uint64_t)(t >> 2) * (SLAB >> 4) + (t & 3) * 2, ds + (uint64_t)t * (2048 >> 4), id, t ? 1u : 0u);
         commit(&C.done[0]);
-        for (int t = 0; t < 2; ++t) tma_store2d(&ms, pt * PT, ((t * a.chunks + c0 + c) * a.H + h) * a.N, so + t * TILE);
-        bulk_commit();
+        if (c > 0) store_u(c - 1);
       }
       __syncwarp();
       wait_warp(&C.full[2], c & 1, dead, 5);
-      __syncthreads();                                    // X is in place
+      __syncthreads();                                    // X is in place (and the tile of the state)
       if (leader) {
-        bulk_wait_read();                                 // what the workers write next has left
+        bulk_wait_read();                                 // the tile of U before has left
         fence_after();
 #pragma unroll
         for (int t = 0; t < 8; ++t) {
@@ -360,6 +366,8 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
           mma_ss(t_l, ta + 2 * (SLAB >> 4), xb, id1, t ? 1u : 0u);
         }
         commit(&C.done[1]);
+        for (int t = 0; t < 2; ++t) tma_store2d(&ms, pt * PT, ((t * a.chunks + c0 + c) * a.H + h) * a.N, so + t * TILE);
+        bulk_commit();
       }
       __syncwarp();
       wait_warp(&C.done[1], c & 1, dead, 6);
@@ -374,15 +382,17 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
           mma_ss(t_d, dkt + o, dx + o, idt, t ? 1u : 0u);
         }
         commit(&C.done[2]);
-        for (int t = 0; t < 2; ++t) tma_store2d(&mu, pt * PT, ((t * a.chunks + c0 + c) * a.H + h) * L, us + t * TILE);
-        bulk_commit();
       }
       __syncwarp();
       wait_warp(&C.done[2], c & 1, dead, 7);
       if (c + 2 < nc && leader) load_k(c + 2);
       __syncwarp();
     }
-    if (leader) bulk_wait();
+    __syncthreads();                                      // the last tile of U is in place
+    if (leader) {
+      store_u(nc - 1);
+      bulk_wait();
+    }
     __syncwarp();
   } else {
     // a thread has one row (of the chunk, or of the state) and sixteen value dims
@@ -421,13 +431,13 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
         const int o = i * 64 + (((half * 2 + q) ^ (i >> 1 & 3)) << 4);
         *reinterpret_cast<uint4*>(tile + o) = h2[q];
         *reinterpret_cast<uint4*>(tile + TILE + o) = l2[q];
-      }
+      }                                                   // (the next `put` orders them ahead of the copy)
     };
     uint4 hi[2], lo[2];
     auto put_state = [&]() {
       split16(S, hi, lo);
-      put_out(so, hi, lo);
       put(ss, hi, lo);
+      put_out(so, hi, lo);                                // under the product
     };
     float ek, b, ue, dec;
     int rows = a.c_rows[c0], rows1 = nc > 1 ? a.c_rows[c0 + 1] : 0;                 // this chunk's, the next one's
@@ -473,21 +483,26 @@ delta_chain_kernel(const __grid_constant__ CUtensorMap mk, const __grid_constant
 #pragma unroll
         for (int k = 0; k < 16; ++k) f[k] += l[k];
       }
-      split16(f, hi, lo);
-      put_out(us, hi, lo);
+      {
+        float x[16];
 #pragma unroll
-      for (int k = 0; k < 16; ++k) f[k] = i < rows ? f[k] * ue : 0.f;
-      split16(f, hi, lo);
+        for (int k = 0; k < 16; ++k) x[k] = i < rows ? f[k] * ue : 0.f;
+        split16(x, hi, lo);
+      }
       put(xs, hi, lo);
+      split16(f, hi, lo);
+      put_out(us, hi, lo);                                // under the product
       wait_warp(&C.done[2], c & 1, dead, 10);
       fence_after();
       read(t_d, f);
 #pragma unroll
       for (int k = 0; k < 16; ++k) S[k] = in_n ? fmaf(dec, S[k], f[k]) : 0.f;
       if (c + 1 < nc) put_state();
-      else fence_before();
       ek = ek1; b = b1; ue = ue1; dec = dec1; rows = rows1; rows1 = rows2;
     }
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    fence_before();
+    __syncthreads();
     if (in_n) {
       float* s1 = a.S + (size_t)a.seg_dst[seg] * slot + ((size_t)h * a.P + p0) * a.Np + i;
 #pragma unroll
