@@ -1,10 +1,12 @@
-// Matrix products of one to four rows (of up to sixteen where the matrix is small), bf16 weights streamed once: out = x W^T (+ bias), to bf16 or 32-bit, or act(x Wg^T) * (x Wu^T)
+// Matrix products of one to four rows, bf16 weights streamed once: out = x W^T (+ bias), to bf16 or 32-bit, or act(x Wg^T) * (x Wu^T)
 // with gate and up stacked, or gelu(x W^T) times the token's row of a table.  Paced by memory: a warp (or two, four, eight of them, each on a share of K) owns two weight rows, whose first
 // 16-byte words are requested before the previous kernel has finished - weights do not depend on it; x sits in shared memory.
 #include "k_rows.cuh"
 
 namespace sfb {
 namespace rgemv {
+
+constexpr int U = 4;          // 256-element steps of K in flight per weight row
 
 struct Args {
   const __nv_bfloat16* w;     // [M, K] ([2 M, K] with act: gate rows, then up rows)
@@ -22,8 +24,7 @@ struct Args {
 };
 
 template <int N>
-__global__ void __launch_bounds__(256, N > 4 ? 1 : 2) gemv_kernel(Args a) {
-  constexpr int U = N > 8 ? 2 : 4;          // 256-element steps of K in flight per weight row
+__global__ void __launch_bounds__(256, 2) gemv_kernel(Args a) {
   extern __shared__ __align__(16) uint8_t raw[];
   __shared__ float part[2][8][2][N];
   __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(raw);      // [N][K]
@@ -159,24 +160,18 @@ using namespace sfb;
 using namespace sfb::rgemv;
 
 static int run(Args a, cudaStream_t stream) {
-  const int N = a.n <= 1 ? 1 : a.n <= 2 ? 2 : a.n <= 4 ? 4 : a.n <= 8 ? 8 : 16;
-  if (a.n < 1 || a.n > 16 || a.M < 1 || a.K < 8 || a.K % 8 || (size_t)N * a.K * 2 > 200 * 1024) return (int)cudaErrorInvalidValue;
+  const int N = a.n <= 1 ? 1 : a.n <= 2 ? 2 : 4;
+  if (a.n < 1 || a.n > 4 || a.M < 1 || a.K < 8 || a.K % 8 || (size_t)N * a.K * 2 > 200 * 1024) return (int)cudaErrorInvalidValue;
   const int pairs = a.act ? a.M : (a.M + 1) / 2, steps = (a.K + 255) / 256;
   a.wk = 1;                // enough pairs of rows for every SM, at least a batch of K per warp
   while (a.wk < 8 && (long long)pairs * a.wk / 8 < 296 && steps / (a.wk * 2) >= 2) a.wk *= 2;
   const int needed = (pairs + 8 / a.wk - 1) / (8 / a.wk), blocks = needed < 296 ? needed : 296;
-  switch (N) {
-    case 1: return launch<1>(a, blocks, stream);
-    case 2: return launch<2>(a, blocks, stream);
-    case 4: return launch<4>(a, blocks, stream);
-    case 8: return launch<8>(a, blocks, stream);
-    default: return launch<16>(a, blocks, stream);
-  }
+  return N == 1 ? launch<1>(a, blocks, stream) : N == 2 ? launch<2>(a, blocks, stream) : launch<4>(a, blocks, stream);
 }
 
 extern "C" {
 
-// n <= 16 rows, K a multiple of 8, n K bounded by shared memory (n rounded up to a power of two: 200 KB).  act (1 silu, 2 gelu, 3 clamped): w holds 2 M rows.
+// n <= 4 rows, K a multiple of 8, n K bounded by shared memory (4 K rows of 200 KB).  act (1 silu, 2 gelu, 3 clamped): w holds 2 M rows.
 int sfb_rows_gemv(const void* w, const void* x, const void* bias, void* out, int64_t out_stride, int n, int M, int K, int f32, int act, float alpha, float limit,
                   cudaStream_t stream) {
   Args a{};

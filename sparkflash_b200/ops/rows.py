@@ -70,7 +70,7 @@ def rot_append(proj, cs, dims, q, kpool, vpool, v_first, lam, table, row_lane, r
 
 def token_linear(x, w, table, col0, tokens, z, out, status):
     """out = gelu(x w^T) * table[token, col0 : col0 + dim]: one kernel for few rows, else a product to ``z`` and token_gate."""
-    if _gemv_takes(x, w):
+    if _gemv_takes(x):
         _check(_lib.rows().sfb_rows_gemv_token(_p(w), _p(x), _p(out), *_strides(table), _p(tokens), c_int(col0), c_int(table.shape[0]), c_int(x.shape[0]),
                                                c_int(w.shape[0]), c_int(x.shape[1]), _p(status), _stream()), "rows_gemv")
         return out
@@ -238,13 +238,11 @@ def sample(logits, row_pos, temperature, seed, mask, best_val, best_id, n):
 
 
 GEMV_ROWS = 4
-GEMV_SMALL_ROWS, GEMV_SMALL = 16, 1 << 20        # up to this many rows against matrices of up to this many elements
 
 
-def _gemv_takes(x: torch.Tensor, w: torch.Tensor) -> bool:
+def _gemv_takes(x: torch.Tensor) -> bool:
     n, K = x.shape
-    most = GEMV_SMALL_ROWS if w.numel() <= GEMV_SMALL else GEMV_ROWS
-    return x.dtype == torch.bfloat16 and n <= most and K % 8 == 0 and (1 << (n - 1).bit_length()) * K * 2 <= 200 * 1024
+    return x.dtype == torch.bfloat16 and n <= GEMV_ROWS and K % 8 == 0 and (n if n < 3 else 4) * K * 2 <= 200 * 1024
 
 
 def _gemv(x, w, b, out, act: int = 0, alpha: float = 0.0, limit: float = 0.0) -> None:
@@ -253,8 +251,8 @@ def _gemv(x, w, b, out, act: int = 0, alpha: float = 0.0, limit: float = 0.0) ->
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor | None, out: torch.Tensor) -> torch.Tensor:
-    """out = x w^T (+ b) with 32-bit accumulation: few bf16 rows by the streaming kernel, a library product otherwise."""
-    if _gemv_takes(x, w):
+    """out = x w^T (+ b) with 32-bit accumulation: up to four bf16 rows by the streaming kernel, a library product otherwise."""
+    if _gemv_takes(x):
         _gemv(x, w, b, out)
         return out
     if b is not None:
@@ -268,7 +266,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, b: torch.Tensor | None, out: torch.
 def gated_linear(x: torch.Tensor, w: torch.Tensor, scratch: torch.Tensor | None, out: torch.Tensor, act: str = "silu", alpha: float = 0.0,
                  limit: float = 0.0) -> torch.Tensor:
     """out = act(x wg^T) * (x wu^T), w = wg stacked on wu; ``scratch`` [n, 2 ff] holds both products where they are not fused."""
-    if _gemv_takes(x, w):
+    if _gemv_takes(x):
         _gemv(x, w, None, out, ACT[act], alpha, limit)
         return out
     linear(x, w, None, scratch)
@@ -303,7 +301,7 @@ def block_gates(u: torch.Tensor, wg: torch.Tensor, out: torch.Tensor) -> torch.T
 
 def head(x: torch.Tensor, embed: torch.Tensor, out: torch.Tensor, name: str = "head") -> torch.Tensor:
     """32-bit logits of x [rows, width] against the output table (or a router's)."""
-    if _gemv_takes(x, embed):
+    if _gemv_takes(x):
         _gemv(x, embed, None, out)
         return out
     if x.dtype == torch.float32:

@@ -16,7 +16,6 @@ from ..models.fanodra import FanodraConfig
 from ..models.gudutar import GudutarConfig
 from ..models.lifulorn import LifulornConfig
 from ..models.layered import LayeredEngine
-from ..ops import rows as R
 from . import roofline
 
 # width, layers, heads, kv heads, dim, recurrence width beside attention, recurrence width alone, parts, ff, vocabulary, loop
@@ -224,11 +223,10 @@ def lifulorn_work(cfg: LifulornConfig, n: int, ctx: int, head_rows: int, decode:
     per pair of bf16 terms; experts: the weights of those that the rows can touch, and their products."""
     d, W, side = cfg.width, roofline.ClassWork, cfg.side_dim
     out = {k: W() for k in ("rows_seam", "rows_conv", "rows_state", "rows_delta_tc", "rows_gated_norm", "rows_rot_append", "rows_attn_stream", "rows_attn_tc",
-                            "rows_token_gate", "router", "rows_moe_gemm", "rows_moe_gemv", "rows_moe_route", "rows_moe_plan", "rows_moe_pick", "linear", "small", "head")}
+                            "rows_token_gate", "rows_moe_gemm", "rows_moe_gemv", "rows_moe_route", "rows_moe_plan", "rows_moe_pick", "linear", "router", "head")}
     few = n <= 4
 
-    def linear(k, m):
-        name = "small" if 4 < n <= R.GEMV_SMALL_ROWS and k * m <= R.GEMV_SMALL else "linear"
+    def linear(k, m, name="linear"):
         out[name].flops += 2.0 * n * k * m
         out[name].bytes += 2.0 * (k * m + n * (k + m))
     out["rows_seam"].bytes += n * d * 8.0
@@ -266,10 +264,7 @@ def lifulorn_work(cfg: LifulornConfig, n: int, ctx: int, head_rows: int, decode:
         if L.mlp is not None:
             E, top, ff, sff = L.mlp["router"]["experts"], L.mlp["router"]["top"], L.mlp["expert"]["ff"], L.mlp["shared"]["ff"]
             used = E * (1 - (1 - top / E) ** n)              # experts that n rows touch, on average
-            if n <= R.GEMV_SMALL_ROWS:
-                linear(d, E + 1)
-            else:
-                out["router"] = W(out["router"].bytes + 2.0 * (d * (E + 1) + n * d) + 4.0 * n * (E + 1), out["router"].flops + 2.0 * n * d * (E + 1))
+            linear(d, E + 1, "router")
             out["rows_moe_route"].bytes += n * (4.0 * E + 8.0 * top)
             out["rows_moe_plan"].bytes += n * top * 16.0
             if few:
@@ -389,8 +384,8 @@ def decode_table(design: str, name: str, n: int = 16, ctx: int = 8192, reps: int
     cfg = eng.cfg
     eng.close()
     wk = WORK[design](cfg, n, ctx, n, True)
-    parts = ("linear", "head", "router") if n <= 4 else ("small",)      # what the streaming products take: all of it, or the small matrices
-    wk["rows_gemv"] = roofline.ClassWork(*(sum(getattr(wk[k], f) for k in parts if k in wk) for f in ("bytes", "flops")))
+    if n <= 4:           # the streaming products take the projections and the head, gate and up fused with their activation
+        wk["rows_gemv"] = roofline.ClassWork(*(sum(getattr(wk[k], f) for k in ("linear", "head", "router") if k in wk) for f in ("bytes", "flops")))
     if design == "fanodra":
         wk["rows_attn_stream"] = wk["rows_attn"]
     return _fractions(ts[1:], wk)

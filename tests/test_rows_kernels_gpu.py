@@ -365,11 +365,11 @@ def test_query_key_norm_covers_the_whole_projection(dt, H, G, dim, vdim):
 @pytest.mark.parametrize("M,K", [(40, 64), (33, 24), (2048, 2048), (96, 5128), (4100, 512)])
 def test_few_row_products(M, K):
     g = torch.Generator().manual_seed(M)
-    for n in (1, 2, 3, 4) + ((5, 8, 9, 16) if M * K <= R.GEMV_SMALL else ()):
+    for n in (1, 2, 3, 4):
         x, w, b = torch.randn(n, K, generator=g).bfloat16(), (torch.randn(M, K, generator=g) * K ** -0.5).bfloat16(), torch.randn(M, generator=g).bfloat16()
         want = x.double() @ w.double().T
         out = torch.zeros(n, M, dtype=torch.bfloat16, device="cuda")
-        assert R._gemv_takes(x, w)
+        assert R._gemv_takes(x)
         R.linear(x.cuda(), w.cuda(), b.cuda(), out)
         assert (out.cpu().double() - want - b.double()).abs().max() < 0.04
         logits = torch.zeros(n, M, device="cuda")
