@@ -33,12 +33,20 @@ CONFIGS = {
         P.attend(1, 1, 3, 7, 14, 20.0, 2, P.yarn(2.0, 30, 3.0, 0.4), 0.4, softcap=8.0)], eps=1e-3),
     # recurrences only
     "rule": P.make_config(97, 48, 8, 0.8, [P.rule(2, 1, 64, 16, 3, P.moe(4, 2, 24, 1.0, 16, 1.0)), P.rule(4, 4, 16, 40, 4), P.rule(2, 2, 32, 24, 2, P.moe(3, 1, 16, 1.0, 0, 0))]),
+    # every row uses every expert, so that bf16 turns no choice over; tensor-core arms
+    "full": P.make_config(112, 96, 16, 0.75, [
+        P.rule(2, 1, 64, 48, 5, P.moe(3, 3, 56, 1.5, 48, 2.0)), P.attend(6, 2, 48, 32, 90, 3e3, 24, P.wave(4.0, 1.0, 2.0, 96), 0.2, mlp=P.moe(2, 2, 40, 0.8, 0, 0)),
+        P.attend(4, 2, 96, 32, 45, 1e4, 96, P.yarn(8.0, 96, 16.0, 2.0), 0.12, softcap=6.0, mlp=P.moe(4, 4, 24, 7.0, 136, 1.0)), P.rule(6, 3, 16, 8, 2)]),
     # attention only
     "att": P.make_config(90, 64, 16, 1.0, [P.attend(6, 2, 32, 32, 100, 1000.0, 16, P.wave(2.0, 1.0, 4.0, 512), 0.5)]),
 }
 NAMES = list(CONFIGS)
 CLOSE = 0.15              # router logits closer than this may swap in bf16
-TOL = {torch.float32: 2e-4, torch.bfloat16: 0.18}      # rms of the logits' difference over the logits' spread
+TOL = {torch.float32: 5e-5, torch.bfloat16: 0.18}      # rms of the logits' difference over the logits' spread
+
+
+def tol(name, dt):
+    return TOL[dt] if dt == torch.float32 or name not in ("full", "att") else 0.06
 
 
 @functools.lru_cache(None)
@@ -100,7 +108,7 @@ def feed(eng, lane, toks, at, cuts):
 def test_whole_prompt_and_layers(name, dt):
     toks = tokens(name, 333)
     eng = engine(name, dt)
-    assert (eng.model.tc_attention, eng.model.tc_state) == ((name in ("mix", "tc", "att"), name in ("tc", "rule")) if dt == torch.bfloat16 else (False, False))
+    assert (eng.model.tc_attention, eng.model.tc_state) == ((name in ("mix", "tc", "full", "att"), name in ("tc", "full", "rule")) if dt == torch.bfloat16 else (False, False))
     taps, eng.tap_layers = [], []
     P.forward(weights(name), CONFIGS[name], list(toks[:40]), torch.float64, taps)
     rows = clear(name, toks[:40], dt)
@@ -110,7 +118,7 @@ def test_whole_prompt_and_layers(name, dt):
         off = (a.cpu() - b.float())[rows].pow(2).mean().sqrt() / b.float().pow(2).mean().sqrt()
         assert off < (1e-5 if dt == torch.float32 else 0.05), (i, off)
     eng.tap_layers = None
-    assert error(feed(eng, 0, toks, 0, [333]), expected(name, toks), clear(name, toks, dt)) < TOL[dt]
+    assert error(feed(eng, 0, toks, 0, [333]), expected(name, toks), clear(name, toks, dt)) < tol(name, dt)
 
 
 @pytest.mark.parametrize("dt", list(TOL))
@@ -123,8 +131,8 @@ def test_portions_and_token_by_token_match_the_whole(name, dt):
     ref, rows = want if dt == torch.float32 else whole, clear(name, toks, dt)
     for lane, cuts in enumerate(([2] * 100, [1] * 200, [64, 64, 64, 8], [3, 61, 1, 65, 33, 2, 2, 32, 1])):
         got = feed(eng, lane, toks, 0, cuts)
-        assert error(got, ref, rows) < TOL[dt], (cuts[:4], error(got, ref, rows))
-        assert error(got, want, rows) < TOL[dt]
+        assert error(got, ref, rows) < tol(name, dt), (cuts[:4], error(got, ref, rows))
+        assert error(got, want, rows) < tol(name, dt)
 
 
 @pytest.mark.parametrize("dt", list(TOL))
@@ -163,7 +171,7 @@ def test_a_far_token_reaches_prompt_and_decoded_rows(n, key, dt):
 
 
 @pytest.mark.parametrize("dt", list(TOL))
-@pytest.mark.parametrize("name", ["mix", "tc", "odd"])
+@pytest.mark.parametrize("name", ["mix", "tc", "odd", "full"])
 def test_mixed_batches_with_reused_pages_and_slots(name, dt):
     """Random schedules over a pool too small for the sum of the requests: portions beside single tokens, requests that pause,
     finish and make room for others; every position's logits match the request alone."""
@@ -195,15 +203,15 @@ def test_mixed_batches_with_reused_pages_and_slots(name, dt):
                 eng.release_lane(lane)
                 del live[lane]
     eng.check_status()
-    assert worst < TOL[dt] and reused > 4 and eng.kv.free_pages == eng.n_pages
+    assert worst < tol(name, dt) and reused > 4 and eng.kv.free_pages == eng.n_pages
 
 
 @pytest.mark.parametrize("dt", list(TOL))
-@pytest.mark.parametrize("name", ["mix", "tc"])
+@pytest.mark.parametrize("name", ["mix", "tc", "full"])
 def test_long_decoding_crosses_pages_windows_and_graph_buckets(name, dt):
     toks = tokens(name, 420)
     eng = engine(name, dt)
-    assert error(feed(eng, 2, toks, 0, [50] + [1] * 370), expected(name, toks), clear(name, toks, dt)) < TOL[dt]
+    assert error(feed(eng, 2, toks, 0, [50] + [1] * 370), expected(name, toks), clear(name, toks, dt)) < tol(name, dt)
     assert len(eng.graphs) >= 1
 
 
