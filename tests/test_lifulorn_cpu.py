@@ -9,6 +9,7 @@ from oracles import plain_lifulorn as P
 from sparkflash_b200.models import registry
 from sparkflash_b200.models.layered import LayeredEngine
 from sparkflash_b200.models.lifulorn import Lifulorn, LifulornConfig, random_tensors
+from sparkflash_b200.models.mixers import rotation_frequencies, rotation_table
 from sparkflash_b200.weights.files import write_safetensors
 
 MOE = P.moe(5, 2, 12, 1.0, 7, 2.0)
@@ -96,3 +97,21 @@ def test_plain_choice_and_clamps():
     w = {"gate": torch.eye(2), "up": torch.eye(2), "down": torch.eye(2)}
     y = P.expert(w, "", torch.tensor([[5.0, -5.0]]), 1.5)
     assert torch.allclose(y, torch.tensor([[1.5 / (1 + torch.exp(torch.tensor(-1.702 * 1.5))) * 2.5, -5 / (1 + torch.exp(torch.tensor(1.702 * 5))) * -0.5]]))
+
+
+SCALINGS = {"plain": None, "wave": {"factor": 4.0, "low": 1.0, "high": 3.0, "original": 300}, "yarn": {"factor": 5.0, "original": 200, "fast": 9.0, "slow": 0.5},
+            "step": {"factor": 3.0, "original": 4000, "fast": 600.0, "slow": 590.0}}
+
+
+@pytest.mark.parametrize("kind", list(SCALINGS))
+@pytest.mark.parametrize("dims", [2, 20, 64])
+def test_rotation_tables(kind, dims):
+    sc = SCALINGS[kind]
+    freqs, gain = ([500.0 ** (-2.0 * i / dims) for i in range(dims // 2)], 1.0) if sc is None else (P.yarn_frequencies if "fast" in sc else P.wavelength_frequencies)(500.0, dims, sc)
+    got, g = rotation_frequencies(500.0, dims, sc)
+    assert got == pytest.approx(freqs, rel=1e-12) and g == pytest.approx(gain, rel=1e-12)
+    x = torch.randn(40, 1, dims + 3, dtype=torch.float64)
+    t = rotation_table(500.0, dims, 40, "cpu", sc).double()
+    u, v = x[:, 0, :dims // 2], x[:, 0, dims // 2:dims]
+    want = P.rotate(x, freqs, gain)[:, 0]
+    assert (torch.cat([u * t[..., 0] - v * t[..., 1], v * t[..., 0] + u * t[..., 1], x[:, 0, dims:]], 1) - want).abs().max() < 1e-5

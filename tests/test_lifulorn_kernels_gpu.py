@@ -5,7 +5,7 @@ import torch
 
 from oracles import plain_lifulorn as P
 from sparkflash_b200.kv.paged import PAGE, PagedKV
-from sparkflash_b200.models.mixers import MixtureFF, W, rotation_frequencies, rotation_table
+from sparkflash_b200.models.mixers import MixtureFF, W, rotation_table
 from sparkflash_b200.ops import rows as R
 
 pytestmark = pytest.mark.gpu
@@ -48,22 +48,7 @@ def test_seam_scales_sums_parts_and_takes_rms_norms(dt, n, d, parts):
 
 
 # ---- rotation, values, cache ----------------------------------------------------------------------------------------------
-SCALINGS = {"plain": None, "wave": {"factor": 4.0, "low": 1.0, "high": 3.0, "original": 300}, "yarn": {"factor": 5.0, "original": 200, "fast": 9.0, "slow": 0.5},
-            "step": {"factor": 3.0, "original": 4000, "fast": 600.0, "slow": 590.0}}
-
-
-@pytest.mark.parametrize("kind", list(SCALINGS))
-@pytest.mark.parametrize("dims", [2, 20, 64])
-def test_rotation_tables(kind, dims):
-    sc = SCALINGS[kind]
-    freqs, gain = ([500.0 ** (-2.0 * i / dims) for i in range(dims // 2)], 1.0) if sc is None else (P.yarn_frequencies if "fast" in sc else P.wavelength_frequencies)(500.0, dims, sc)
-    got, g = rotation_frequencies(500.0, dims, sc)
-    assert got == pytest.approx(freqs, rel=1e-12) and g == pytest.approx(gain, rel=1e-12)
-    x = torch.randn(40, 1, dims + 3, dtype=torch.float64)
-    t = rotation_table(500.0, dims, 40, "cpu", sc).double()
-    u, v = x[:, 0, :dims // 2], x[:, 0, dims // 2:dims]
-    want = P.rotate(x, freqs, gain)[:, 0]
-    assert (torch.cat([u * t[..., 0] - v * t[..., 1], v * t[..., 0] + u * t[..., 1], x[:, 0, dims:]], 1) - want).abs().max() < 1e-5
+SCALING = {"factor": 5.0, "original": 200, "fast": 9.0, "slow": 0.5}
 
 
 @pytest.mark.parametrize("dt", DTYPES)
@@ -79,8 +64,7 @@ def test_append_turns_queries_and_keys_and_mixes_values(dt, H, G, dim, vdim, dim
     where = [(a, p) for a, n in enumerate(lens) for p in range(n)]
     first, lam = torch.zeros(len(where), G * vdim, dtype=dt, device="cuda"), torch.tensor(0.3, device="cuda")
     proj = torch.nn.functional.pad(torch.cat(xs), (0, 5)).to("cuda", dt)      # a wider row
-    sc = SCALINGS["yarn"]
-    cs, (freqs, gain) = rotation_table(90.0, dims, 256, "cuda", sc), P.yarn_frequencies(90.0, dims, sc)
+    cs, (freqs, gain) = rotation_table(90.0, dims, 256, "cuda", SCALING), P.yarn_frequencies(90.0, dims, SCALING)
     q = torch.empty(len(where), H * dim, dtype=dt, device="cuda")
     for mixed in (False, True):
         st = _status()
@@ -286,7 +270,7 @@ class _Step:
 
 # width, experts, choices, ff, shared ff, limits
 MOES = [(64, 16, 2, 24, 40, (1.0, 2.0)), (96, 5, 5, 200, 0, (0.5, 1.0)), (40, 40, 3, 136, 16, (3.0, 0.7)), (37, 6, 2, 11, 7, (1.0, 1.0)), (320, 3, 1, 64, 128, (9.0, 9.0)),
-        (520, 130, 8, 264, 72, (0.4, 4.0))]
+        (520, 130, 8, 264, 72, (0.4, 4.0)), (24, 300, 4, 8, 0, (1.0, 1.0))]
 
 
 @pytest.mark.parametrize("dt", DTYPES)
@@ -323,9 +307,11 @@ def test_mixture_of_experts(d, E, top, ff, sff, limits, n, dt):
             assert (wts[:, top].double().cpu() - P.sigmoid(h.double() @ w64["shared.sg"].T)[:, 0]).abs().max() < (1e-5 if dt == torch.float32 else 1e-5)
 
 
-def test_all_rows_on_one_expert_and_close_calls():
-    """A router that sends everything to the same experts (one long list), and equal logits (the lower number wins)."""
-    n, d, E, top = 700, 64, 9, 2
+@pytest.mark.parametrize("n", [700, 9000])
+def test_all_rows_on_one_expert_and_close_calls(n):
+    """A router that sends everything to the same experts (one long list, more pairs than the plan holds at once), and equal logits (the
+    lower number wins)."""
+    d, E, top = 64, 9, 2
     w, spec, h = _mixture(torch.bfloat16, d, E, top, 40, 0, (2.0, 1.0), 3, n)
     w["router"].zero_()
     moe, s = MixtureFF(W({"p." + k: v for k, v in w.items()}, "p.", torch.bfloat16, "cuda"), spec, 1.702), _Step(n)
