@@ -9,17 +9,19 @@
 //   conv       causal depthwise convolution with carried inputs, optionally added to its input or followed by silu, optionally with a
 //              bias.
 //   qk_append  RMS norm over a whole query / key projection, keys and values into the paged cache.
+//   head_append  RMS norm of every query and key head with a weight that the heads share, keys and values into the paged cache.
 //   rot_append rotated queries and keys, values mixed with another layer's, into the paged cache.
 //   token_gate gelu(projection) * the token's row of a table.
 //   gated scan real-gated linear recurrence S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t with a = exp(-c r softplus(lam)):
 //              two passes over chunks of rows for prompts (the chunks' start states in between), one fused kernel (convolution, gates, recurrence,
 //              output gate) for single rows.
 //   act_mul    act(gate) * up, act = silu, the tanh form of gelu, or the clamped gate.
+//   act        the ungated activations: xIELU, the square of relu.
 //
 // Recurrent state (scan state, convolution inputs) has two versions per lane.  A segment reads version `src` (-1: zeros) and
 // writes version `dst`, so every block of a launch sees the state before the step, a replayed graph repeats the same result,
 // and a step can be undone by going back to `src`.
-#include "k_rows.cuh"
+#include "k_rows_seam.cuh"
 
 namespace sfb {
 namespace rows {
@@ -259,51 +261,7 @@ __global__ void __launch_bounds__(NV < 8 ? 256 : 512, !AHEAD && NV == 4 ? 4 : 1)
     }
 #pragma unroll
     for (int k = 0; k < V; ++k) o[k] = (x[i][k] - mu) * rs * nw[i][k] + nb[i][k];
-    if (a.cw) {
-      // the convolution sees the norm's output at activation precision, as the many-row kernel does
-      float acc[V], t[V];
-#pragma unroll
-      for (int k = 0; k < V; ++k) o[k] = to_f<T>(from_f<T>(o[k]));
-      if (ahead_conv) {
-#pragma unroll
-        for (int k = 0; k < V; ++k) acc[k] = 0.f;
-#pragma unroll
-        for (int j = 0; j < TW; ++j) {
-          if (j < W) {
-#pragma unroll
-            for (int k = 0; k < V; ++k) acc[k] += cw[j][i][k] * cg[j][i][k];
-            if (j > 0) store_v<T, V>(hd + (size_t)(j - 1) * d + c, cg[j][i]);
-          } else if (j == W) {
-#pragma unroll
-            for (int k = 0; k < V; ++k) acc[k] += cw[j][i][k] * o[k];
-          }
-        }
-        if (W > 0) store_v<T, V>(hd + (size_t)(W - 1) * d + c, o);
-#pragma unroll
-        for (int k = 0; k < V; ++k) o[k] += acc[k];
-        store_v<T, V>(hr + c, o);
-        continue;
-      }
-      load_v<float, V>(a.cw + (size_t)W * d + c, t);
-#pragma unroll
-      for (int k = 0; k < V; ++k) acc[k] = t[k] * o[k];
-#pragma unroll 4
-      for (int j = 0; j < W; ++j) {
-        float g[V];
-        if (hs) load_v<T, V>(hs + (size_t)j * d + c, g);
-        else {
-#pragma unroll
-          for (int k = 0; k < V; ++k) g[k] = 0.f;
-        }
-        load_v<float, V>(a.cw + (size_t)j * d + c, t);
-#pragma unroll
-        for (int k = 0; k < V; ++k) acc[k] += t[k] * g[k];
-        if (j > 0) store_v<T, V>(hd + (size_t)(j - 1) * d + c, g);
-      }
-      if (W > 0) store_v<T, V>(hd + (size_t)(W - 1) * d + c, o);
-#pragma unroll
-      for (int k = 0; k < V; ++k) o[k] += acc[k];
-    }
+    if (a.cw) step_conv<T, V, TW, NV>(o, i, c, d, W, a.cw, hs, hd, ahead_conv, cw, cg);
     store_v<T, V>(hr + c, o);
   }
 }
@@ -448,6 +406,56 @@ __global__ void __launch_bounds__(256) qk_append_kernel(QkAppendArgs a) {
       const int cc = c - HD - GD, g = cc / a.vdim, x = cc - g * a.vdim;
       if (ok) store_v<T, V>((T*)a.vpool + (((size_t)page * a.G + g) * PAGE + slot) * a.vdim + x, f);
     }
+  }
+}
+
+// ---- query / key norm head by head, cache append ---------------------------------------------------------------------------
+// Lanes in groups of `per` (a power of two) own a head each; a lane holds NV times V of its elements.  The other lanes copy the values.
+template <typename T, int V, int NV>
+__global__ void __launch_bounds__(256) head_append_kernel(QkAppendArgs a, int per) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int row = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, HG = a.H + a.G, GV = a.G * a.vdim;
+  const T* p = (const T*)a.proj + (size_t)row * a.stride;
+  const int pos = a.row_pos[row];
+  const int page = a.table[(size_t)a.row_lane[row] * a.max_pages + pos / PAGE], slot = pos % PAGE;
+  const bool ok = page >= 0 && page < a.n_pages;
+  if (!ok && threadIdx.x == 0) status_set(a.status, ST_BOUNDS, 78, page, a.n_pages);
+  const int groups = 32 / per, at = lane & (per - 1);
+  const float inv_d = 1.f / (float)a.dim;
+  for (int h0 = warp * groups; h0 < HG; h0 += 8 * groups) {        // the same for every lane of the warp
+    const int h = h0 + lane / per;
+    const T* src = p + (size_t)h * a.dim;
+    float f[NV][V], w[NV][V], t = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * per + at) * V;
+      if (h < HG && c < a.dim) {
+        load_v<T, V>(src + c, f[i]);
+        load_v<float, V>((h < a.H ? a.qw : a.kw) + c, w[i]);
+#pragma unroll
+        for (int k = 0; k < V; ++k) t = fmaf(f[i][k], f[i][k], t);
+      }
+    }
+    for (int o = 1; o < per; o <<= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
+    const float r = 1.f / sqrtf(t * inv_d + a.eps);
+    if (h >= HG || (h >= a.H && !ok)) continue;
+    T* dst = h < a.H ? (T*)a.q + ((size_t)row * a.H + h) * a.dim : (T*)a.kpool + (((size_t)page * a.G + h - a.H) * PAGE + slot) * a.dim;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * per + at) * V;
+      if (c >= a.dim) continue;
+#pragma unroll
+      for (int k = 0; k < V; ++k) f[i][k] *= r * w[i][k];
+      store_v<T, V>(dst + c, f[i]);
+    }
+  }
+  if (!ok) return;
+  for (int c = (255 - threadIdx.x) * V; c < GV; c += 256 * V) {
+    const int g = c / a.vdim, x = c - g * a.vdim;
+    float f[V];
+    load_v<T, V>(p + (size_t)HG * a.dim + c, f);
+    store_v<T, V>((T*)a.vpool + (((size_t)page * a.G + g) * PAGE + slot) * a.vdim + x, f);
   }
 }
 
@@ -846,6 +854,20 @@ __global__ void __launch_bounds__(256) act_mul_kernel(const T* gu, T* out, int f
   store_v<T, V>(out + row * out_stride + c, g);
 }
 
+// ---- ungated activations ---------------------------------------------------------------------------------------------------
+template <typename T, int V>
+__global__ void __launch_bounds__(256) act_kernel(const T* z, T* out, int64_t count, int act, float p0, float p1) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t c = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (c >= count) return;
+  float f[V];
+  load_v<T, V>(z + c, f);
+#pragma unroll
+  for (int k = 0; k < V; ++k) f[k] = act_single<T>(f[k], act, p0, p1);
+  store_v<T, V>(out + c, f);
+}
+
 // ---- dispatch ---------------------------------------------------------------------------------------------------------------
 template <typename T, int V>
 static int launch_seam(const SeamArgs& a, int n, cudaStream_t st) {
@@ -930,6 +952,25 @@ int sfb_rows_qk_append(const void* proj, int64_t stride, const void* qw, const v
                   : sfb_launch(qk_append_kernel<__nv_bfloat16, 1>, dim3(n), dim3(256), 0, stream, a));
 }
 
+// qw, kw: [dim]; heads up to 512 wide
+int sfb_rows_head_append(const void* proj, int64_t stride, const void* qw, const void* kw, void* q, void* kpool, void* vpool, const int* table,
+                         const int* row_lane, const int* row_pos, int max_pages, int n_pages, int n, int H, int G, int dim, int vdim, float eps,
+                         int fp32, void* status, cudaStream_t stream) {
+  if (n < 1 || G < 1 || dim < 1 || dim > 512) return (int)cudaErrorInvalidValue;
+  QkAppendArgs a{proj, stride, (const float*)qw, (const float*)kw, q, kpool, vpool, table, row_lane, row_pos, max_pages, n_pages, H, G, dim, vdim,
+                 eps, (Status*)status};
+  const int all = dim | vdim | (int)(stride & 1023), V = all % 4 ? 1 : fp32 || all % 8 ? 4 : 8;
+  int per = 1;             // lanes of a head
+  while (per < 32 && per * V < dim) per *= 2;
+  const dim3 g(n), b(256);
+  if (fp32) return (int)(V == 4 ? sfb_launch(head_append_kernel<float, 4, 4>, g, b, 0, stream, a, per)
+                                : sfb_launch(head_append_kernel<float, 1, 16>, g, b, 0, stream, a, per));
+  if (V == 8) return (int)(dim <= 256 ? sfb_launch(head_append_kernel<__nv_bfloat16, 8, 1>, g, b, 0, stream, a, per)
+                                      : sfb_launch(head_append_kernel<__nv_bfloat16, 8, 2>, g, b, 0, stream, a, per));
+  return (int)(V == 4 ? sfb_launch(head_append_kernel<__nv_bfloat16, 4, 4>, g, b, 0, stream, a, per)
+                      : sfb_launch(head_append_kernel<__nv_bfloat16, 1, 16>, g, b, 0, stream, a, per));
+}
+
 // summaries: a segment has more than one chunk (two passes; the gates are overwritten); otherwise one pass
 int sfb_rows_scan(const void* gates, const void* rb, const void* ib, const void* decay, const void* u, const void* y, int64_t y_stride, void* out,
                   void* S, void* sums, const int* chunk_seg, const int* chunk_row0, const int* chunk_rows, const int* chunk_first,
@@ -1005,6 +1046,22 @@ int sfb_rows_act_mul(const void* gu, void* out, int64_t out_stride, int n, int f
   if (V == 8) return (int)sfb_launch(act_mul_kernel<__nv_bfloat16, 8>, g, b, 0, stream, i, o, ff, out_stride, act, alpha, limit);
   return (int)(V == 4 ? sfb_launch(act_mul_kernel<__nv_bfloat16, 4>, g, b, 0, stream, i, o, ff, out_stride, act, alpha, limit)
                       : sfb_launch(act_mul_kernel<__nv_bfloat16, 1>, g, b, 0, stream, i, o, ff, out_stride, act, alpha, limit));
+}
+
+// out = act(z), `count` elements (z and out may be the same)
+int sfb_rows_act(const void* z, void* out, int64_t count, int act, float p0, float p1, int fp32, cudaStream_t stream) {
+  if (count < 1 || (act != ACT_RELU2 && act != ACT_XIELU)) return (int)cudaErrorInvalidValue;
+  const int V = count % 4 ? 1 : fp32 || count % 8 ? 4 : 8;
+  const int64_t blocks = (count + 256 * V - 1) / (256 * V);
+  if (blocks > 0x7fffffff) return (int)cudaErrorInvalidValue;
+  const dim3 g((unsigned)blocks), b(256);
+  if (fp32) return (int)(V == 4 ? sfb_launch(act_kernel<float, 4>, g, b, 0, stream, (const float*)z, (float*)out, count, act, p0, p1)
+                                : sfb_launch(act_kernel<float, 1>, g, b, 0, stream, (const float*)z, (float*)out, count, act, p0, p1));
+  const __nv_bfloat16* i = (const __nv_bfloat16*)z;
+  __nv_bfloat16* o = (__nv_bfloat16*)out;
+  if (V == 8) return (int)sfb_launch(act_kernel<__nv_bfloat16, 8>, g, b, 0, stream, i, o, count, act, p0, p1);
+  return (int)(V == 4 ? sfb_launch(act_kernel<__nv_bfloat16, 4>, g, b, 0, stream, i, o, count, act, p0, p1)
+                      : sfb_launch(act_kernel<__nv_bfloat16, 1>, g, b, 0, stream, i, o, count, act, p0, p1));
 }
 
 }  // extern "C"

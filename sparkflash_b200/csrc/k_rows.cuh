@@ -78,6 +78,7 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
 
 
 constexpr int ACT_SILU = 1, ACT_GELU = 2, ACT_CLAMP = 3;      // activations of the gated products
+constexpr int ACT_RELU2 = 4, ACT_XIELU = 5;                   // of the ungated ones
 
 // exp, reciprocal and square root of the gates, all 32-bit: library-accurate with float activations; with bf16 activations the
 // hardware approximations (relative error below 2^-21), whose error is far below the rounding of u
@@ -98,6 +99,24 @@ template <typename T> __device__ __forceinline__ float gate_clamp(float g, float
   g = fminf(g, limit);
   u = fminf(fmaxf(u, -limit), limit);
   return g * gate_sigmoid<T>(alpha * g) * (u + 1.f);
+}
+
+// exp(z) - 1 - z for z <= 0: the series near 0, where the difference would cancel (the first term left out is below 2^-28 of the sum)
+template <typename T> __device__ __forceinline__ float expm1_minus(float z) {
+  float p = 1.f / 3628800.f;
+  p = fmaf(p, z, 1.f / 362880.f); p = fmaf(p, z, 1.f / 40320.f); p = fmaf(p, z, 1.f / 5040.f); p = fmaf(p, z, 1.f / 720.f); p = fmaf(p, z, 1.f / 120.f);
+  p = fmaf(p, z, 1.f / 24.f); p = fmaf(p, z, 1.f / 6.f); p = fmaf(p, z, 0.5f);
+  float e;
+  if constexpr (sizeof(T) == 4) e = expf(z);
+  else e = __expf(z);
+  return z > -0.75f ? z * z * p : e - 1.f - z;
+}
+
+// One input.  RELU2: max(z, 0)^2.  XIELU (Huang and Schlag, "Deriving Activation Functions Using Integration"): a z^2 + z / 2 above 0,
+// b (exp(z) - 1 - z) + z / 2 below it.
+template <typename T> __device__ __forceinline__ float act_single(float z, int act, float a, float b) {
+  if (act == ACT_RELU2) { const float r = fmaxf(z, 0.f); return r * r; }
+  return (z > 0.f ? a * z * z : b * expm1_minus<T>(fminf(z, 0.f))) + 0.5f * z;
 }
 
 }  // namespace rows

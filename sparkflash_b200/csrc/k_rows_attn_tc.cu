@@ -1,6 +1,7 @@
 // Softmax attention over the paged cache for long runs of rows, on tcgen05: score = (q . k) * scale - bias[head][distance],
 // causal, the last `window` positions, bf16 queries / keys / values, 32-bit scores, softmax and accumulators.  Optionally
-// cap * tanh(score / cap) (no bias then), and a sink per head whose exponential is in the softmax's denominator only.
+// cap * tanh(score / cap) (no bias then), a sink per head whose exponential is in the softmax's denominator only, and a
+// sigmoid gate on the output.
 //
 // One CTA: 256 consecutive query rows of one segment (two halves of 128) x one head.  Key tiles of one cache page (64 positions)
 // stream through shared memory by TMA: a (page, head) block is contiguous, so 64 dims of a tile are one box copy.
@@ -43,6 +44,8 @@ struct Args {
   const float* sink;         // [H] or null
   float cap;
   __nv_bfloat16* out;        // [n, H vdim]
+  const __nv_bfloat16* gate; // [n, gate_row]: outputs are multiplied by its sigmoid; or null
+  int64_t gate_row;
   int max_pages, n_pages, H, G, dim, vdim, rot;    // n_pages: of the pool, or of the rows multiplied out
   int k_page, k_head;        // rows between the pages and between the heads of the keys and values
   int window;
@@ -334,6 +337,17 @@ attn_run_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ 
           ld16(to + c, f);
           wait_ld();
           uint32_t u[8];
+          if (a.gate && valid) {
+            const __nv_bfloat16* gp = a.gate + (size_t)(row0 + rr) * a.gate_row + (size_t)h * a.vdim + c;
+#pragma unroll
+            for (int i = 0; i < 16; i += 8) {
+              if (c + i >= a.vdim) break;
+              float z[8];
+              rows::load_v<__nv_bfloat16, 8>(gp + i, z);
+#pragma unroll
+              for (int k = 0; k < 8; ++k) f[i + k] *= rows::gate_sigmoid<__nv_bfloat16>(z[k]);
+            }
+          }
 #pragma unroll
           for (int i = 0; i < 8; ++i) {
             const __nv_bfloat162 t = __floats2bfloat162_rn(f[2 * i] * inv, f[2 * i + 1] * inv);
@@ -403,14 +417,15 @@ int sfb_rows_tmap(void* out_map, const void* base, int64_t rows, int64_t cols, i
 
 // mq: queries [rows, H (dim + rot)], box 128 rows; mk, mv: keys and values [rows, dim / vdim], box 64 rows, page p of head g at row
 // p k_page + g k_head (through the page table, or p + offs[tile]); mr: the shared key part [rows, rot] or null.  dim and vdim: multiples
-// of 8 up to 128; rot: a multiple of 8 up to 64.
+// of 8 up to 128; rot: a multiple of 8 up to 64.  gate: as in Args, rows on 16-byte boundaries.
 int sfb_rows_attn_tc(const void* mq, const void* mk, const void* mv, const void* mr, const int* table, const int* row_lane, const int* row_pos,
-                     const int* tiles, const int* offs, int n_tiles, const void* bias, int64_t bias_len, const void* sink, float cap, void* out, int max_pages, int n_pages, int H, int G,
+                     const int* tiles, const int* offs, int n_tiles, const void* bias, int64_t bias_len, const void* sink, float cap, void* out,
+                     const void* gate, int64_t gate_row, int max_pages, int n_pages, int H, int G,
                      int dim, int vdim, int rot, int k_page, int k_head, int window, float scale, void* status, cudaStream_t stream) {
   if (n_tiles < 1 || n_tiles > 65535 || G < 1 || H % G || dim % 8 || vdim % 8 || dim < 8 || dim > 128 || vdim < 8 || vdim > 128 || rot % 8 || rot > 64 ||
-      (rot > 0) != (mr != nullptr) || (rot && bias) || (cap > 0.f && (bias || rot)) || window < 1)
+      (rot > 0) != (mr != nullptr) || (rot && bias) || (cap > 0.f && (bias || rot)) || window < 1 || (gate && (gate_row % 8 || (uintptr_t)gate % 16)))
     return (int)cudaErrorInvalidValue;
-  Args a{tiles, table, row_lane, row_pos, offs, (const float*)bias, bias_len, (const float*)sink, cap, (__nv_bfloat16*)out, max_pages, n_pages, H, G, dim, vdim, rot, k_page, k_head,
+  Args a{tiles, table, row_lane, row_pos, offs, (const float*)bias, bias_len, (const float*)sink, cap, (__nv_bfloat16*)out, (const __nv_bfloat16*)gate, gate_row, max_pages, n_pages, H, G, dim, vdim, rot, k_page, k_head,
          window, scale, (Status*)status};
   const CUtensorMap *q = (const CUtensorMap*)mq, *k = (const CUtensorMap*)mk, *v = (const CUtensorMap*)mv, *r = mr ? (const CUtensorMap*)mr : k;
   if (rot) {

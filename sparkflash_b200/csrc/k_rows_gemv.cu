@@ -1,5 +1,5 @@
 // Matrix products of one to four rows, bf16 weights streamed once: out = x W^T (+ bias), to bf16 or 32-bit, or act(x Wg^T) * (x Wu^T)
-// with gate and up stacked, or gelu(x W^T) times the token's row of a table.  Paced by memory: a warp (or two, four, eight of them, each on a share of K) owns two weight rows, whose first
+// with gate and up stacked, or act(x W^T), or gelu(x W^T) times the token's row of a table.  Paced by memory: a warp (or two, four, eight of them, each on a share of K) owns two weight rows, whose first
 // 16-byte words are requested before the previous kernel has finished - weights do not depend on it; x sits in shared memory.
 #include "k_rows.cuh"
 
@@ -13,9 +13,9 @@ struct Args {
   const __nv_bfloat16* x;     // [n, K]
   const __nv_bfloat16* bias;  // [M] or null
   void* out;                  // [n, M] bf16 (or float)
-  int M, K, n, wk, f32, act;
+  int M, K, n, wk, f32, act, single;     // act: of gate and up; single: of one product
   int64_t out_stride;         // elements between the rows of out
-  float alpha, limit;         // of the clamped gate
+  float alpha, limit;         // of the clamped gate; the single activation's numbers
   const __nv_bfloat16* table; // [vocab, table_stride] or null: out = gelu(x W^T) * table[token][col0 + .]
   int64_t table_stride;
   const int* tokens;
@@ -120,6 +120,7 @@ __global__ void __launch_bounds__(256, 2) gemv_kernel(Args a) {
       } else {
         const int r0 = 2 * o, r1 = r0 + 1;
         if (a.bias) { if (r0 < a.M) s0 += __bfloat162float(a.bias[r0]); if (r1 < a.M) s1 += __bfloat162float(a.bias[r1]); }
+        if (a.single) { s0 = rows::act_single<float>(s0, a.single, a.alpha, a.limit); s1 = rows::act_single<float>(s1, a.single, a.alpha, a.limit); }
         if (a.table) {
           int tok = a.tokens[lane];
           if (tok < 0 || tok >= a.vocab) { status_set(a.status, ST_BOUNDS, 76, tok, a.vocab); tok = 0; }
@@ -171,12 +172,15 @@ static int run(Args a, cudaStream_t stream) {
 
 extern "C" {
 
-// n <= 4 rows, K a multiple of 8, n K bounded by shared memory (4 K rows of 200 KB).  act (1 silu, 2 gelu, 3 clamped): w holds 2 M rows.
+// n <= 4 rows, K a multiple of 8, n K bounded by shared memory (4 K rows of 200 KB).  act (1 silu, 2 gelu, 3 clamped): w holds 2 M rows; the
+// ungated ones (4, 5): M rows.
 int sfb_rows_gemv(const void* w, const void* x, const void* bias, void* out, int64_t out_stride, int n, int M, int K, int f32, int act, float alpha, float limit,
                   cudaStream_t stream) {
   Args a{};
   a.w = (const __nv_bfloat16*)w; a.x = (const __nv_bfloat16*)x; a.bias = (const __nv_bfloat16*)bias; a.out = out; a.M = M; a.K = K; a.n = n; a.f32 = f32;
-  a.act = act; a.out_stride = out_stride; a.alpha = alpha; a.limit = limit;
+  if (act == rows::ACT_RELU2 || act == rows::ACT_XIELU) a.single = act;
+  else a.act = act;
+  a.out_stride = out_stride; a.alpha = alpha; a.limit = limit;
   return run(a, stream);
 }
 

@@ -1,14 +1,16 @@
-// Mixture of experts on a step's rows: every row goes through `top` of E gated feed-forwards, and through a shared one.
+// Mixture of experts on a step's rows: every row goes through `top` of E feed-forwards (gated, or with one activation), and through a
+// shared one.
 //
-//   moe_route   the chosen experts of a row and their weights (softmax over the chosen logits), and the shared expert's weight
-//               (sigmoid of one more logit); one warp per row
+//   moe_route   the chosen experts of a row and their weights, and the shared expert's weight (sigmoid of one more logit); one warp per row.
+//               Either the largest logits and the softmax over them; or scores s = sigmoid(logit), the largest s + correction among the
+//               groups of neighbouring experts whose two best sum highest, weighted by their s over its sum
 //   moe_plan    (row, choice) pairs in order of their expert, cut into tiles of `tile` pairs of one expert; chooses as well when rows are few
 //   moe_tile    one tile x 64 output columns on CUDA cores: any sizes, bf16 or 32-bit (k_rows_moe_tc.cu takes bf16 on tcgen05)
 //   moe_gemv    one to four rows, bf16: a block per (pair, share of the output), weights streamed; the shared expert's rows beside the
 //               pairs; every block of the first product chooses for its row
 //
-// Both products of an expert go through the same kernels: `gated` (gate and up rows stacked, act(gate) * up, rows picked by the plan) and
-// down (rows of the first product in plan order, results at [row][choice], where the seam sums them with their weights).
+// Both products of an expert go through the same kernels: the first (rows picked by the plan; gate and up rows stacked, act(gate) * up, or one
+// matrix and act) and down (rows of the first product in plan order, results at [row][choice], where the seam sums them with their weights).
 #include "k_rows.cuh"
 
 namespace sfb {
@@ -24,21 +26,76 @@ struct RouteArgs {
   int* ids;                 // [n, top]
   float* wts;               // [n, top + shared]
   int n, E, top, shared;
+  const float* corr;        // [E]: choice by sigmoid(logit) + corr, weights by the sigmoids; null: by logits and their softmax
+  int groups, keep;         // (corr) only experts of the best `keep` of `groups` equal groups of neighbours
+  float scale;              // (corr) of the weights
 };
-// One warp, one row: lane j ends up with choice j and its weight (the lower number wins among equal logits); `shared_w`: the shared expert's.
-constexpr int HELD = 8;     // logits a lane holds, the rest is read again
+constexpr int HELD = 8;     // scores a lane holds, the rest is read again
+constexpr int MAX_GROUPS = 256;
 // bits that compare as the numbers do; above 0 for every number
 __device__ __forceinline__ uint32_t rank_bits(float v) {
   const uint32_t b = __float_as_uint(v);
   return b & 0x80000000u ? ~b : b | 0x80000000u;
 }
+__device__ __forceinline__ float choice_score(const RouteArgs& a, const float* z, int e) { return a.corr ? sigmoid_f(z[e]) + a.corr[e] : z[e]; }
+
+// The warp's largest of v[k] (number k * 32 + lane; 0: none), the lower number among equal ones; it becomes 0.
+template <int N> __device__ __forceinline__ int take_best(uint32_t (&v)[N], int none) {
+  const int lane = threadIdx.x & 31;
+  uint32_t best = 0;
+  int at = none;
+#pragma unroll
+  for (int k = 0; k < N; ++k)
+    if (v[k] > best) { best = v[k]; at = k * 32 + lane; }
+  const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+  at = (int)__reduce_min_sync(0xffffffffu, (unsigned)(best == top ? at : none));
+#pragma unroll
+  for (int k = 0; k < N; ++k)
+    if (at == k * 32 + lane) v[k] = 0u;
+  return at;
+}
+
+// Groups: bit k of the result: this lane's expert k * 32 + lane cannot be chosen.
+__device__ __forceinline__ uint32_t shut_experts(const RouteArgs& a, const float* z) {
+  const int lane = threadIdx.x & 31, size = a.E / a.groups;
+  constexpr int N = MAX_GROUPS / 32;
+  uint32_t v[N];
+#pragma unroll
+  for (int k = 0; k < N; ++k) v[k] = 0u;
+  for (int g = 0; g < a.groups; ++g) {
+    float m0 = -INFINITY, m1 = -INFINITY;       // the two largest of the group
+    for (int e = lane; e < size; e += 32) {
+      const float s = choice_score(a, z, g * size + e);
+      m1 = fmaxf(m1, fminf(m0, s));
+      m0 = fmaxf(m0, s);
+    }
+    for (int o = 1; o < 32 && o < size; o <<= 1) {
+      const float x0 = __shfl_xor_sync(0xffffffffu, m0, o), x1 = __shfl_xor_sync(0xffffffffu, m1, o);
+      m1 = fmaxf(fmaxf(m1, x1), fminf(m0, x0));
+      m0 = fmaxf(m0, x0);
+    }
+    const uint32_t bits = __shfl_sync(0xffffffffu, rank_bits(size > 1 ? m0 + m1 : m0), 0);
+#pragma unroll
+    for (int k = 0; k < N; ++k)
+      if (g == k * 32 + lane) v[k] = bits;
+  }
+  uint32_t shut = 0xffffffffu;
+  for (int i = 0; i < a.keep; ++i) {
+    const int g = take_best<N>(v, a.groups - 1);
+    for (int k = 0, e = lane; e < a.E; ++k, e += 32)
+      if (e / size == g) shut &= ~(1u << k);
+  }
+  return shut;
+}
+
+// One warp, one row: lane j ends up with choice j and its weight (the lower number wins among equal scores); `shared_w`: the shared expert's.
 __device__ __forceinline__ void choose(const RouteArgs& a, const float* z, int& id, float& weight, float& shared_w) {
   const int lane = threadIdx.x & 31;
+  uint32_t taken = a.corr && a.keep < a.groups ? shut_experts(a, z) : 0u;      // bit k: this lane's expert k * 32 + lane
   uint32_t v[HELD];         // 0: taken, or past the end
 #pragma unroll
-  for (int k = 0; k < HELD; ++k) v[k] = k * 32 + lane < a.E ? rank_bits(z[k * 32 + lane]) : 0u;
+  for (int k = 0; k < HELD; ++k) v[k] = k * 32 + lane < a.E && !(taken >> k & 1) ? rank_bits(choice_score(a, z, k * 32 + lane)) : 0u;
   const float zs = a.shared ? z[a.E] : 0.f;
-  uint32_t taken = 0, mine = 0;      // taken: of this lane's experts beyond those it holds; mine: lane j: logit of choice j
   id = 0;
   for (int j = 0; j < a.top; ++j) {
     uint32_t best = 0;
@@ -47,7 +104,7 @@ __device__ __forceinline__ void choose(const RouteArgs& a, const float* z, int& 
     for (int k = 0; k < HELD; ++k)
       if (v[k] > best) { best = v[k]; at = k * 32 + lane; }
     for (int e = HELD * 32 + lane, k = HELD; e < a.E; e += 32, ++k) {
-      const uint32_t x = taken >> k & 1 ? 0u : rank_bits(z[e]);
+      const uint32_t x = taken >> k & 1 ? 0u : rank_bits(choice_score(a, z, e));
       if (x > best) { best = x; at = e; }
     }
     const uint32_t top = __reduce_max_sync(0xffffffffu, best);
@@ -58,11 +115,16 @@ __device__ __forceinline__ void choose(const RouteArgs& a, const float* z, int& 
       for (int k = 0; k < HELD; ++k)
         if (at >> 5 == k) v[k] = 0u;
     }
-    if (lane == j) { mine = top; id = at; }
+    if (lane == j) id = at;
   }
-  const float mz = __uint_as_float(mine & 0x80000000u ? mine ^ 0x80000000u : ~mine);
-  const float top = __shfl_sync(0xffffffffu, mz, 0), e = lane < a.top ? expf(mz - top) : 0.f;
-  weight = e / warp_sum(e);
+  const float mz = lane < a.top ? z[id] : 0.f;
+  if (a.corr) {
+    const float s = lane < a.top ? sigmoid_f(mz) : 0.f;
+    weight = s / (warp_sum(s) + 1e-20f) * a.scale;
+  } else {
+    const float top = __shfl_sync(0xffffffffu, mz, 0), e = lane < a.top ? expf(mz - top) : 0.f;
+    weight = e / warp_sum(e);
+  }
   shared_w = sigmoid_f(zs);
 }
 __device__ __forceinline__ void route_row(const RouteArgs& a, int row) {
@@ -144,11 +206,11 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(PlanArgs a) {
 
 // ---- tiles on CUDA cores ----------------------------------------------------------------------------------------------------
 struct TileArgs {
-  const void* x;            // gated: [n, K] rows; down: [pairs, K] in plan order
-  const void* w;            // [E, (2) M, K]
-  void* out;                // gated: [pairs, M] in plan order; down: [n, slots, M]
+  const void* x;            // first: [n, K] rows; down: [pairs, K] in plan order
+  const void* w;            // [E, M, K], gated: [E, 2 M, K]
+  void* out;                // first: [pairs, M] in plan order; down: [n, slots, M]
   const int *order, *tiles, *count;
-  int M, K, top, slots, gated;
+  int M, K, top, slots, act, gated;      // act: 0 down, ACT_CLAMP (gated), or an ungated one
   float alpha, limit;
 };
 constexpr int TR = 32, TC = 64, TK = 16;
@@ -164,7 +226,7 @@ __global__ void __launch_bounds__(256) moe_tile_kernel(TileArgs a) {
   const int tr = tid >> 4, tc = tid & 15;            // rows tr, tr + 16; columns tc + 16 i
   const int xr = tid >> 3, xk = (tid & 7) * 2;       // staged: row xr, two of its elements
   const int place = p0 + min(xr, rows - 1);
-  const T* xp = (const T*)a.x + (size_t)(a.gated ? a.order[place] / a.top : place) * a.K;
+  const T* xp = (const T*)a.x + (size_t)(a.act ? a.order[place] / a.top : place) * a.K;
   const T* wp = (const T*)a.w + (size_t)e * (a.gated ? 2 : 1) * a.M * a.K;
   float acc[2][2][4] = {};
   for (int k0 = 0; k0 < a.K; k0 += TK) {
@@ -197,12 +259,14 @@ __global__ void __launch_bounds__(256) moe_tile_kernel(TileArgs a) {
     const int row = tr + 16 * r;
     if (row >= rows) continue;
     size_t o;
-    if (a.gated) o = (size_t)(p0 + row);
+    if (a.act) o = (size_t)(p0 + row);
     else { const int pair = a.order[p0 + row]; o = (size_t)(pair / a.top) * a.slots + pair % a.top; }
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int c = c0 + tc + 16 * i;
-      if (c < a.M) ((T*)a.out)[o * a.M + c] = from_f<T>(a.gated ? gate_clamp<T>(acc[0][r][i], acc[1][r][i], a.alpha, a.limit) : acc[0][r][i]);
+      if (c >= a.M) continue;
+      const float f = acc[0][r][i];
+      ((T*)a.out)[o * a.M + c] = from_f<T>(a.gated ? gate_clamp<T>(f, acc[1][r][i], a.alpha, a.limit) : a.act ? act_single<T>(f, a.act, a.alpha, a.limit) : f);
     }
   }
 }
@@ -210,12 +274,12 @@ __global__ void __launch_bounds__(256) moe_tile_kernel(TileArgs a) {
 // ---- few rows -----------------------------------------------------------------------------------------------------------------
 struct GemvArgs {
   RouteArgs r;                // r.z: the first product chooses the experts (and leaves them in r.ids and r.wts)
-  const __nv_bfloat16* x;     // gated: [n, K]; down: [pairs, K]
-  const __nv_bfloat16* w;     // [E, (2) M, K]
-  __nv_bfloat16* out;         // gated: [pairs, M]; down: [n, slots, M]
-  const __nv_bfloat16 *sx, *sw;     // the shared expert: gated [n, SK], down [n, SK]; null: none
-  __nv_bfloat16* sout;        // gated: [n, SM]
-  int pairs, n, M, K, SM, SK, top, slots, gated;
+  const __nv_bfloat16* x;     // first: [n, K]; down: [pairs, K]
+  const __nv_bfloat16* w;     // [E, M, K], gated: [E, 2 M, K]
+  __nv_bfloat16* out;         // first: [pairs, M]; down: [n, slots, M]
+  const __nv_bfloat16 *sx, *sw;     // the shared expert: first [n, SK], down [n, SK]; null: none
+  __nv_bfloat16* sout;        // first: [n, SM]
+  int pairs, n, M, K, SM, SK, top, slots, act, gated;      // act: 0 down, ACT_CLAMP (gated), or an ungated one
   float alpha, limit, slimit;
 };
 constexpr int GU = 4;         // 256-element steps in flight per weight row
@@ -245,8 +309,8 @@ __global__ void __launch_bounds__(256) moe_gemv_kernel(GemvArgs a) {
   const int expert = sh ? 0 : a.r.z ? chosen : a.r.ids[job];
   const int row = sh ? job - a.pairs : job / a.top, M = sh ? a.SM : a.M, K = sh ? a.SK : a.K, words = K / 8;
   const __nv_bfloat16* w = sh ? a.sw : a.w + (size_t)expert * (a.gated ? 2 : 1) * M * K;
-  const __nv_bfloat16* x = a.gated ? (sh ? a.sx : a.x) + (size_t)row * K : (sh ? a.sx + (size_t)row * K : a.x + (size_t)job * K);
-  __nv_bfloat16* out = a.gated ? (sh ? a.sout + (size_t)row * M : a.out + (size_t)job * M)
+  const __nv_bfloat16* x = a.act ? (sh ? a.sx : a.x) + (size_t)row * K : (sh ? a.sx + (size_t)row * K : a.x + (size_t)job * K);
+  __nv_bfloat16* out = a.act ? (sh ? a.sout + (size_t)row * M : a.out + (size_t)job * M)
                                : a.out + ((size_t)row * a.slots + (sh ? a.top : job % a.top)) * M;
   const int outs = a.gated ? M : (M + 1) / 2, stride = gridDim.x * 8;
   uint4 c0[GU], c1[GU];
@@ -295,6 +359,7 @@ __global__ void __launch_bounds__(256) moe_gemv_kernel(GemvArgs a) {
     if (lane == 0) {
       if (a.gated) out[o] = __float2bfloat16_rn(gate_clamp<float>(s0, s1, a.alpha, sh ? a.slimit : a.limit));
       else {
+        if (a.act) { s0 = act_single<float>(s0, a.act, a.alpha, a.limit); s1 = act_single<float>(s1, a.act, a.alpha, a.limit); }
         out[2 * o] = __float2bfloat16_rn(s0);
         if (2 * o + 1 < M) out[2 * o + 1] = __float2bfloat16_rn(s1);
       }
@@ -308,40 +373,52 @@ __global__ void __launch_bounds__(256) moe_gemv_kernel(GemvArgs a) {
 using namespace sfb;
 using namespace sfb::rmoe;
 
+static bool route_ok(const RouteArgs& a) {
+  return a.n >= 1 && a.E >= 1 && a.E <= MAX_E && a.top >= 1 && a.top <= MAX_TOP && a.top <= a.E &&
+         (!a.corr || (a.groups >= 1 && a.groups <= MAX_GROUPS && a.E % a.groups == 0 && a.keep >= 1 && a.keep <= a.groups && a.top <= a.E / a.groups * a.keep));
+}
+// a first product's activation (0: down)
+static bool act_ok(int act) { return act == 0 || act == ACT_CLAMP || act == ACT_RELU2 || act == ACT_XIELU; }
+
 extern "C" {
 
-int sfb_rows_moe_route(const void* z, int64_t ld, void* ids, void* wts, int n, int E, int top, int shared, cudaStream_t stream) {
-  if (n < 1 || E < 1 || E > MAX_E || top < 1 || top > MAX_TOP || top > E) return (int)cudaErrorInvalidValue;
-  RouteArgs a{(const float*)z, ld, (int*)ids, (float*)wts, n, E, top, shared};
+// corr, groups, keep, scale: see RouteArgs
+int sfb_rows_moe_route(const void* z, int64_t ld, void* ids, void* wts, int n, int E, int top, int shared, const void* corr, int groups, int keep, float scale,
+                       cudaStream_t stream) {
+  RouteArgs a{(const float*)z, ld, (int*)ids, (float*)wts, n, E, top, shared, (const float*)corr, groups, keep, scale};
+  if (!route_ok(a)) return (int)cudaErrorInvalidValue;
   return (int)sfb_launch(moe_route_kernel, dim3((n + 7) / 8), dim3(256), 0, stream, a);
 }
 
 // tiles: 4 ints each, at most pairs / tile + min(E, pairs) of them.  z: the choice is made here (few rows), null: ids are there.
 int sfb_rows_moe_plan(const void* z, int64_t ld, void* ids, void* wts, void* order, void* tiles, void* count, int n, int E, int top, int shared, int tile,
-                      cudaStream_t stream) {
-  if (n < 1 || E < 1 || E > MAX_E || top < 1 || top > MAX_TOP || top > E || tile < 1 || (long long)n * top >= 1 << 20) return (int)cudaErrorInvalidValue;
-  PlanArgs a{{(const float*)z, ld, (int*)ids, (float*)wts, n, E, top, shared}, (int*)order, (int*)tiles, (int*)count, n * top, E, tile};
+                      const void* corr, int groups, int keep, float scale, cudaStream_t stream) {
+  RouteArgs r{(const float*)z, ld, (int*)ids, (float*)wts, n, E, top, shared, (const float*)corr, groups, keep, scale};
+  if (!route_ok(r) || tile < 1 || (long long)n * top >= 1 << 20) return (int)cudaErrorInvalidValue;
+  PlanArgs a{r, (int*)order, (int*)tiles, (int*)count, n * top, E, tile};
   return (int)sfb_launch(moe_plan_kernel, dim3(1), dim3(E > 256 || n * top > 2048 ? 1024 : 256), 0, stream, a);
 }
 
 // tiles of at most 32 pairs
 int sfb_rows_moe_tile(const void* x, const void* w, void* out, const void* order, const void* tiles, const void* count, int max_tiles, int M, int K, int top,
-                      int slots, int gated, float alpha, float limit, int fp32, cudaStream_t stream) {
-  if (max_tiles < 1 || max_tiles > 65535 || M < 1 || K < 1) return (int)cudaErrorInvalidValue;
-  TileArgs a{x, w, out, (const int*)order, (const int*)tiles, (const int*)count, M, K, top, slots, gated, alpha, limit};
+                      int slots, int act, float alpha, float limit, int fp32, cudaStream_t stream) {
+  if (!act_ok(act) || max_tiles < 1 || max_tiles > 65535 || M < 1 || K < 1) return (int)cudaErrorInvalidValue;
+  TileArgs a{x, w, out, (const int*)order, (const int*)tiles, (const int*)count, M, K, top, slots, act, act == ACT_CLAMP, alpha, limit};
   const dim3 g((M + TC - 1) / TC, max_tiles), b(256);
   return (int)(fp32 ? sfb_launch(moe_tile_kernel<float>, g, b, 0, stream, a) : sfb_launch(moe_tile_kernel<__nv_bfloat16>, g, b, 0, stream, a));
 }
 
-// bf16, K and SK multiples of 8; z: the choice of E experts is made here, null: ids are there
-int sfb_rows_moe_gemv(const void* z, int64_t ld, int E, void* ids, void* wts, const void* x, const void* w, void* out, const void* sx, const void* sw, void* sout, int pairs, int n, int M, int K, int SM,
-                      int SK, int top, int slots, int gated, float alpha, float limit, float slimit, cudaStream_t stream) {
-  const int kmax = sw && SK > K ? SK : K;
-  if (n < 1 || pairs != n * top || pairs + n > 65535 || M < 1 || K < 8 || K % 8 || (sw && (SM < 1 || SK < 8 || SK % 8)) || kmax * 2 > 200 * 1024)
+// bf16, K and SK multiples of 8; z: the choice of E experts is made here (first product), null: ids are there
+int sfb_rows_moe_gemv(const void* z, int64_t ld, int E, void* ids, void* wts, const void* corr, int groups, int keep, float scale, const void* x, const void* w, void* out,
+                      const void* sx, const void* sw, void* sout, int pairs, int n, int M, int K, int SM, int SK, int top, int slots, int act, float alpha, float limit,
+                      float slimit, cudaStream_t stream) {
+  const int kmax = sw && SK > K ? SK : K, gated = act == ACT_CLAMP;
+  if (n < 1 || pairs != n * top || pairs + n > 65535 || M < 1 || K < 8 || K % 8 || (sw && (SM < 1 || SK < 8 || SK % 8)) || kmax * 2 > 200 * 1024 || !act_ok(act))
     return (int)cudaErrorInvalidValue;
-  if (z && (!gated || E < top || E > MAX_E || top > MAX_TOP || slots < top)) return (int)cudaErrorInvalidValue;
-  GemvArgs a{{(const float*)z, ld, (int*)ids, (float*)wts, n, E, top, slots - top}, (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, (const __nv_bfloat16*)sx, (const __nv_bfloat16*)sw,
-             (__nv_bfloat16*)sout, pairs, n, M, K, SM, SK, top, slots, gated, alpha, limit, slimit};
+  RouteArgs r{(const float*)z, ld, (int*)ids, (float*)wts, n, E, top, slots - top, (const float*)corr, groups, keep, scale};
+  if (z && (!act || slots < top || !route_ok(r))) return (int)cudaErrorInvalidValue;
+  GemvArgs a{r, (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, (const __nv_bfloat16*)sx, (const __nv_bfloat16*)sw,
+             (__nv_bfloat16*)sout, pairs, n, M, K, SM, SK, top, slots, act, gated, alpha, limit, slimit};
   const int jobs = pairs + (sw ? n : 0), big = sw && SM > M ? SM : M, outs = gated ? big : (big + 1) / 2;
   int bx = (outs + 7) / 8, cap = (148 * 4 + jobs - 1) / jobs;
   if (bx > cap) bx = cap;

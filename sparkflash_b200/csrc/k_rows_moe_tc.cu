@@ -3,6 +3,7 @@
 //
 //   gated   act(x Wg^T, x Wu^T): 128 pairs x 128 gate columns beside their 128 up columns; results in plan order.  With few rows the pairs' rows
 //           are gathered by TMA straight from the layer's input (four rows a copy); many are brought into plan order first (`pick`)
+//   single  act(x W^T): the same with 256 columns of one matrix
 //   down    128 pairs x 256 columns; rows in plan order; every result row goes to its [row][choice]
 //
 // The shared expert's rows (all of the step, in order, with sizes of their own) are tiles of the same launches, ahead of the others.
@@ -19,10 +20,12 @@ using namespace tc;
 
 constexpr int THREADS = 192, ROWS = 128, COLS = 256, KS = 64, ST = 4, XSLAB = ROWS * 128, WSLAB = COLS * 128;
 
+constexpr int DOWN = 0, GATED = 1, SINGLE = 2;
+
 struct Args {
   const int *order, *tiles, *count;
-  __nv_bfloat16 *out, *sout; // gated: [pairs, M], the shared expert's [n, SM]; down: [n, slots, M]
-  int M, K, SM, SK, top, slots, cblocks, sblocks;     // cblocks, sblocks: blocks of 128 (gated) or 256 columns
+  __nv_bfloat16 *out, *sout; // first product: [pairs, M], the shared expert's [n, SM]; down: [n, slots, M]
+  int M, K, SM, SK, top, slots, act, cblocks, sblocks;     // cblocks, sblocks: blocks of 128 (gated) or 256 columns
   int stotal, n;             // tiles x column blocks of the shared expert (0: none), its rows
   float alpha, limit, slimit;
   Status* status;
@@ -33,13 +36,13 @@ struct Job {
   int4 t;                    // expert, first place (shared: row), pairs, -
   int c0, M, K, shared;
 };
-template <bool GATED>
+template <int KIND>
 __device__ __forceinline__ Job job(const Args& a, int b) {
   Job j;
   j.shared = b < a.stotal;
   const int x = j.shared ? b : b - a.stotal, blocks = j.shared ? a.sblocks : a.cblocks, ti = x / blocks;
   j.t = j.shared ? make_int4(0, ti * 128, min(128, a.n - ti * 128), 0) : reinterpret_cast<const int4*>(a.tiles)[ti];
-  j.c0 = (x % blocks) * (GATED ? 128 : 256);
+  j.c0 = (x % blocks) * (KIND == GATED ? 128 : 256);
   j.M = j.shared ? a.SM : a.M;
   j.K = j.shared ? a.SK : a.K;
   return j;
@@ -78,7 +81,7 @@ __global__ void __launch_bounds__(256) moe_pick_kernel(const uint4* x, const int
   }
 }
 
-template <bool GATED, bool GATHER>
+template <int KIND, bool GATHER>
 __global__ void __launch_bounds__(THREADS, 1)
 moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ CUtensorMap mw, const __grid_constant__ CUtensorMap msx,
                 const __grid_constant__ CUtensorMap msw, Args a) {
@@ -107,7 +110,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
   if (warp == 0) {
     int it = 0;              // stages filled so far
     for (int b = blockIdx.x; b < total && !*dead; b += gridDim.x) {
-      const Job j = job<GATED>(a, b);
+      const Job j = job<KIND>(a, b);
       const int4 t = j.t;
       const bool gather = GATHER && !j.shared;
       int4 rows = make_int4(0, 0, 0, 0);      // a lane gathers four rows, the tile's last one again past its end; lanes past it none
@@ -116,7 +119,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
 #pragma unroll
         for (int k = 0; k < 4; ++k) r[k] = a.order[t.y + min(lane * 4 + k, t.z - 1)] / a.top;
       }
-      const int wrow = t.x * (GATED ? 2 : 1) * j.M + j.c0, steps = (j.K + KS - 1) / KS;
+      const int wrow = t.x * (KIND == GATED ? 2 : 1) * j.M + j.c0, steps = (j.K + KS - 1) / KS;
       const CUtensorMap *x = j.shared ? &msx : &mx, *w = j.shared ? &msw : &mw;
       for (int k = 0; k < steps; ++k, ++it) {
         const int st = it % ST, ph = (it / ST) & 1;
@@ -128,7 +131,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
         if (lane == 0) {
           if (!gather) tma2d(S.x + st * XSLAB, x, k * KS, t.y, &S.full[st]);
           tma2d(S.w + st * WSLAB, w, k * KS, wrow, &S.full[st]);
-          tma2d(S.w + st * WSLAB + XSLAB, w, k * KS, wrow + (GATED ? j.M : 128), &S.full[st]);
+          tma2d(S.w + st * WSLAB + XSLAB, w, k * KS, wrow + (KIND == GATED ? j.M : 128), &S.full[st]);
         }
       }
     }
@@ -165,24 +168,24 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
     const uint32_t lanes = (uint32_t)(w4 * 32) << 16;
     int n = 0;
     for (int b = blockIdx.x; b < total; b += gridDim.x, ++n) {
-      const Job j = job<GATED>(a, b);
+      const Job j = job<KIND>(a, b);
       const int acc = n & 1;
       const bool in = r < j.t.z;
       size_t row = 0;
-      if (GATED) row = (size_t)(j.t.y + r);
+      if (KIND != DOWN) row = (size_t)(j.t.y + r);
       else if (j.shared) row = (size_t)(j.t.y + r) * a.slots + a.top;
       else if (in) { const int pair = a.order[j.t.y + r]; row = (size_t)(pair / a.top) * a.slots + pair % a.top; }
-      __nv_bfloat16* o = (GATED && j.shared ? a.sout : a.out) + row * j.M + j.c0;
+      __nv_bfloat16* o = (KIND != DOWN && j.shared ? a.sout : a.out) + row * j.M + j.c0;
       const float limit = j.shared ? a.slimit : a.limit;
       const bool ok = mbar_wait(&S.acc_full[acc], (n >> 1) & 1, dead);
       if (!__all_sync(0xffffffffu, ok)) break;
       fence_after();
       const uint32_t ta = tmem + acc * COLS + lanes;
-      const int width = min(GATED ? 128 : 256, j.M - j.c0);
+      const int width = min(KIND == GATED ? 128 : 256, j.M - j.c0);
       for (int c = 0; c < width; c += 32) {
         float f[32];
         ld32(ta + c, f);
-        if constexpr (GATED) {
+        if constexpr (KIND == GATED) {
           float u[32];
           ld32(ta + 128 + c, u);
           wait_ld();
@@ -190,6 +193,15 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
           for (int k = 0; k < 32; ++k) f[k] = rows::gate_clamp<__nv_bfloat16>(f[k], u[k], a.alpha, limit);
         } else {
           wait_ld();
+          if constexpr (KIND == SINGLE) {
+            if (a.act == rows::ACT_RELU2) {
+#pragma unroll
+              for (int k = 0; k < 32; ++k) { const float p = fmaxf(f[k], 0.f); f[k] = p * p; }
+            } else {
+#pragma unroll
+              for (int k = 0; k < 32; ++k) f[k] = rows::act_single<__nv_bfloat16>(f[k], rows::ACT_XIELU, a.alpha, limit);
+            }
+          }
         }
         if (in) {
 #pragma unroll
@@ -203,16 +215,16 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap mx, const __grid_constant__ 
   }
   fence_before();
   __syncthreads();
-  if (tid == 0 && *dead) status_set(a.status, ST_TIMEOUT, 75, blockIdx.x, GATED);
+  if (tid == 0 && *dead) status_set(a.status, ST_TIMEOUT, 75, blockIdx.x, KIND);
   if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, 512;" ::"r"(tmem) : "memory");
 }
 
-template <bool GATED, bool GATHER>
+template <int KIND, bool GATHER>
 static int launch(const CUtensorMap* mx, const CUtensorMap* mw, const CUtensorMap* msx, const CUtensorMap* msw, const Args& a, int most, cudaStream_t st) {
   const size_t smem = sizeof(Smem) + 1024;
   static bool done = false;
   if (!done) {
-    const cudaError_t e = cudaFuncSetAttribute(moe_gemm_kernel<GATED, GATHER>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const cudaError_t e = cudaFuncSetAttribute(moe_gemm_kernel<KIND, GATHER>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     done = true;
   }
@@ -220,7 +232,7 @@ static int launch(const CUtensorMap* mx, const CUtensorMap* mw, const CUtensorMa
   cudaGetDevice(&dev);
   cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
   const long long blocks = (long long)most * a.cblocks + a.stotal;
-  return (int)sfb_launch(moe_gemm_kernel<GATED, GATHER>, dim3((unsigned)(blocks < sms ? blocks : sms)), dim3(THREADS), smem, st, *mx, *mw, *msx, *msw, a);
+  return (int)sfb_launch(moe_gemm_kernel<KIND, GATHER>, dim3((unsigned)(blocks < sms ? blocks : sms)), dim3(THREADS), smem, st, *mx, *mw, *msx, *msw, a);
 }
 
 }  // namespace rmoetc
@@ -239,20 +251,21 @@ int sfb_rows_moe_pick(const void* x, const void* order, void* out, int pairs, in
 
 // mx: rows [pairs, K] in plan order, box 128 rows, or (gather) rows [n, K], box of one row; mw: weights [E (2) M, K], box 128 rows.  msx, msw: the
 // same of the shared expert (rows in order), or null.  M, K, SM and SK: multiples of 8; most: the most tiles (of up to 128 pairs) that the plan
-// can hold.
+// can hold.  act: 0 down, ACT_CLAMP (gated) or an ungated activation with the numbers alpha, limit.
 int sfb_rows_moe_gemm(const void* mx, const void* mw, const void* msx, const void* msw, const void* order, const void* tiles, const void* count, void* out, void* sout,
-                      int most, int n, int M, int K, int SM, int SK, int top, int slots, int gated, int gather, float alpha, float limit, float slimit, void* status,
+                      int most, int n, int M, int K, int SM, int SK, int top, int slots, int act, int gather, float alpha, float limit, float slimit, void* status,
                       cudaStream_t stream) {
-  if (most < 1 || n < 1 || M < 8 || M % 8 || K < 8 || K % 8 || top < 1 || (gather && !gated) || (msx && (SM < 8 || SM % 8 || SK < 8 || SK % 8 || slots <= top)) ||
+  if (most < 1 || n < 1 || M < 8 || M % 8 || K < 8 || K % 8 || top < 1 || (gather && !act) || (act && act != rows::ACT_CLAMP && act != rows::ACT_RELU2 && act != rows::ACT_XIELU) || (msx && (SM < 8 || SM % 8 || SK < 8 || SK % 8 || slots <= top)) ||
       (uintptr_t)out % 16 || (uintptr_t)sout % 16)
     return (int)cudaErrorInvalidValue;
-  const int per = gated ? 128 : 256;
-  Args a{(const int*)order, (const int*)tiles, (const int*)count, (__nv_bfloat16*)out, (__nv_bfloat16*)sout, M, K, SM, SK, top, slots, (M + per - 1) / per,
+  const int gated = act == rows::ACT_CLAMP, per = gated ? 128 : 256;
+  Args a{(const int*)order, (const int*)tiles, (const int*)count, (__nv_bfloat16*)out, (__nv_bfloat16*)sout, M, K, SM, SK, top, slots, act, (M + per - 1) / per,
          (SM + per - 1) / per, 0, n, alpha, limit, slimit, (Status*)status};
   if (msx) a.stotal = (n + 127) / 128 * a.sblocks;
   const CUtensorMap *x = (const CUtensorMap*)mx, *w = (const CUtensorMap*)mw, *sx = msx ? (const CUtensorMap*)msx : x, *sw = msw ? (const CUtensorMap*)msw : w;
-  if (gather) return launch<true, true>(x, w, sx, sw, a, most, stream);
-  return gated ? launch<true, false>(x, w, sx, sw, a, most, stream) : launch<false, false>(x, w, sx, sw, a, most, stream);
+  if (gather) return gated ? launch<GATED, true>(x, w, sx, sw, a, most, stream) : launch<SINGLE, true>(x, w, sx, sw, a, most, stream);
+  if (act) return gated ? launch<GATED, false>(x, w, sx, sw, a, most, stream) : launch<SINGLE, false>(x, w, sx, sw, a, most, stream);
+  return launch<DOWN, false>(x, w, sx, sw, a, most, stream);
 }
 
 }  // extern "C"

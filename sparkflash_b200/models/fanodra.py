@@ -16,7 +16,7 @@ from dataclasses import dataclass, field
 import torch
 
 from ..ops import rows as R
-from .layered import CONFIG_META, LayeredModel, check_keys
+from .layered import CONFIG_META, LayeredModel, check_keys, check_loop, loop_runs
 from .mixers import DenseFF, ParallelMixer, RecurrentMixer, W
 
 ARCHITECTURE = "Fanodra"
@@ -82,9 +82,8 @@ class FanodraConfig:
                     raise ValueError(f"layer {i}: unknown mlp kind {ff['kind']!r}")
             layers.append(LayerSpec(L["type"], m, ff["ff"] if ff is not None else None))
         loop = d.get("loop") or {"start": 0, "stop": 0, "times": 0}
-        check_keys(loop, {"start", "stop", "times"}, "loop")
-        if loop["times"] and not 0 <= loop["start"] < loop["stop"] <= len(layers):
-            raise ValueError("config.json: loop range outside the layers")
+        if loop["times"]:
+            check_loop(loop, len(layers))
         if not 1 <= d["canon"]["taps"] <= R.MAX_TAPS:
             raise ValueError(f"convolutions of 1..{R.MAX_TAPS} taps are implemented")
         return cls(d["vocab"], d["width"], float(d["norm"]["eps"]), d["canon"]["taps"], layers, loop["start"], loop["stop"], loop["times"],
@@ -92,12 +91,8 @@ class FanodraConfig:
 
     def runs(self) -> list[tuple[int, int | None]]:
         """(layer, pass that begins right before it or None) in the order the layers run."""
-        if not self.loop_times:
-            return [(i, None) for i in range(len(self.layers))]
-        out = [(i, None) for i in range(self.loop_start)]
-        for t in range(self.loop_times):
-            out += [(i, t if i == self.loop_start else None) for i in range(self.loop_start, self.loop_stop)]
-        return out + [(i, None) for i in range(self.loop_stop, len(self.layers))]
+        order = loop_runs(len(self.layers), {"start": self.loop_start, "stop": self.loop_stop, "times": self.loop_times} if self.loop_times else None)
+        return [(i, t if i == self.loop_start else None) for i, t in order]
 
     def shapes(self) -> dict[str, tuple[int, ...]]:
         """Every tensor of a checkpoint."""

@@ -12,7 +12,8 @@ row selection and the sampler - and speaks the contract of serve/driver.py.  A m
     bind(engine)                       reserve scratch, register state tensors
     forward(step) -> [head rows, vocab] float32 logits (None without a head)
 
-and writes no loop, cache or batching of its own (models/fanodra.py, models/gudutar.py and models/lifulorn.py; ``LayeredModel`` has what they share).
+and writes no loop, cache or batching of its own (models/fanodra.py, models/gudutar.py, models/lifulorn.py and models/dironex.py; ``LayeredModel`` has
+what they share).
 """
 from __future__ import annotations
 
@@ -75,6 +76,24 @@ class Step:
 
     single = False            # every segment is one row (a decode step)
     taps: list | None = None  # debug: collects the residual after every layer run
+
+    def single_rows(self, tc: bool):
+        """(rows, count) that a sublayer takes one by one: all of them, or those that its tensor-core arm does not (None: all, in order)."""
+        return (self.short_rows, self.short) if tc else (None, self.n)
+
+
+def loop_runs(layers: int, loop: dict | None) -> list[tuple[int, int | None]]:
+    """Layers in the order they run, each with its pass (None outside the loop): layers start .. stop - 1 run ``times`` times."""
+    if not loop:
+        return [(i, None) for i in range(layers)]
+    a, b, times = loop["start"], loop["stop"], loop["times"]
+    return [(i, None) for i in range(a)] + [(i, t) for t in range(times) for i in range(a, b)] + [(i, None) for i in range(b, layers)]
+
+
+def check_loop(loop: dict, layers: int) -> None:
+    check_keys(loop, {"start", "stop", "times"}, "loop")
+    if not (0 <= loop["start"] < loop["stop"] <= layers and loop["times"] >= 1):
+        raise ValueError("config.json: loop out of range")
 
 
 class LayeredModel:

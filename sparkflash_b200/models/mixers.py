@@ -1,7 +1,7 @@
 """Sublayers of the layered decoders (models/layered.py): attention with a distance bias, attention with rotated keys in a window (sinks,
-capped scores, values mixed across layers), the real-gated linear recurrence, two mixers side by side, matrix-state recurrences
-(state-space duality, retention, the gated delta rule), latent attention in a window, the dense gated feed-forward, the mixture of
-experts, and the per-layer token input.  Each takes its sizes and constants as arguments, reads its weights by
+capped scores, values mixed across layers), attention with normed heads in a window, the real-gated linear recurrence, two mixers side by side, matrix-state recurrences
+(state-space duality, retention, the gated delta rule), latent attention, the dense feed-forward (gated or with one activation), the
+mixture of experts, the per-layer token input, and the weights of residual streams.  Each takes its sizes and constants as arguments, reads its weights by
 name, keeps its caches in the engine's page pool or state slots, and runs on a step's rows through the kernels of ops/rows.py.
 
 A sublayer is built once per layer (``weights``) and bound once per run of the layer (``bind_run``): a looped layer shares its
@@ -83,18 +83,19 @@ class PagedAttention:
     def attend(self, s, q, kv, o) -> None:
         """q [n, H dim] against this run's pools, whose rows of the step have been appended; kv from R.attn_pools."""
         k, v, opts = kv[0], kv[1], dict(window=self.window, sink=self.sink, cap=self.cap)
-        if s.ntiles:
+        rows, m = s.single_rows(self.tc)
+        if s.ntiles and self.tc:
             R.attn_tc(q, kv, s.table, s.row_lane, s.row_pos, s.tiles, s.ntiles, self.bias, o, self.H, self.scale, s.status, **opts)
-        if s.short and self.stream and s.short <= R.STREAM_ROWS:
+        if m and self.stream and m <= R.STREAM_ROWS:
             pages = min(s.pages, (self.window + R.PAGE - 2) // R.PAGE + 1)
-            R.attn_stream(q, k, v, s.table, s.row_lane, s.row_pos, s.short_rows, s.short, self.bias, o, s.scratch.buf["attn_part"],
-                          s.scratch.buf["attn_ml"], self.H, self.scale, s.short * pages, s.status, **opts)
-        elif s.short:
+            R.attn_stream(q, k, v, s.table, s.row_lane, s.row_pos, rows, m, self.bias, o, s.scratch.buf["attn_part"],
+                          s.scratch.buf["attn_ml"], self.H, self.scale, m * pages, s.status, **opts)
+        elif m:
             blocks = R.attn_blocks(self.H, self.G)
-            sp = s.engine.splits(s, s.short, blocks, self.window)
+            sp = s.engine.splits(s, m, blocks, self.window)
             part = s.scratch.buf["attn_part"] if sp > 1 else None
             ml = s.scratch.buf["attn_ml"] if sp > 1 else None
-            R.attn(q, k, v, s.table, s.row_lane, s.row_pos, s.short_rows, s.short, self.bias, o, part, ml, self.H, self.scale, sp, s.status, **opts)
+            R.attn(q, k, v, s.table, s.row_lane, s.row_pos, rows, m, self.bias, o, part, ml, self.H, self.scale, sp, s.status, **opts)
 
 
 class BiasedAttention(PagedAttention):
@@ -281,6 +282,32 @@ class RotaryAttention(PagedAttention):
         q, o = s.scratch.get("attn_q", n, self.H * self.dim), s.scratch.get("attn_o", n, self.H * self.vdim)
         first = s.scratch.get("v_first", n, self.mix.cols) if self.mix is not None else None
         R.rot_append(proj, self.cs, self.dims, q, kv[0], kv[1], first, self.lam, s.table, s.row_lane, s.row_pos, n, self.H, s.status)
+        self.attend(s, q, kv, o)
+        return R.linear(o, self.wo, None, s.scratch.get("y", n, h.shape[1])), None
+
+
+class HeadNormAttention(PagedAttention):
+    """Queries and keys RMS-normed head by head (weights that the heads share), no rotation, a sliding window.  A layer's only mixer."""
+
+    def __init__(self, w: W, spec: dict, eps: float, max_context: int):
+        super().__init__(w, spec)
+        self.eps, self.window = eps, min(int(spec["mask"]["size"]), max_context)
+        self.q_norm, self.k_norm = w.f32("q.norm"), w.f32("k.norm")
+        self.w_in, self.wo = w.act(*self.PROJ, pad=8), w.act("o")
+        self.merge, self.kv_run = (None, None), (self.G, self.dim, self.vdim)
+
+    def reserve(self, e) -> None:
+        super().reserve(e)
+        e.scratch.reserve("proj", e.max_rows * self.w_in.shape[0], self.dtype)
+
+    def bind_run(self, e, tag: str, kv_index):
+        return {"kv": R.attn_pools(e.kv, kv_index, self.tc)}
+
+    def run(self, s, h, run):
+        n, kv = s.n, run["kv"]
+        proj = R.linear(h, self.w_in, None, s.scratch.get("proj", n, self.w_in.shape[0]))
+        q, o = s.scratch.get("attn_q", n, self.H * self.dim), s.scratch.get("attn_o", n, self.H * self.vdim)
+        R.head_append(proj, self.q_norm, self.k_norm, q, kv[0], kv[1], s.table, s.row_lane, s.row_pos, n, self.H, self.eps, s.status)
         self.attend(s, q, kv, o)
         return R.linear(o, self.wo, None, s.scratch.get("y", n, h.shape[1])), None
 
@@ -477,19 +504,27 @@ class DeltaMixer:
 
 class LatentAttention:
     """Attention whose keys and values are products of one cached vector per token (DeepSeek-AI, "DeepSeek-V2: A Strong, Economical, and
-    Efficient Mixture-of-Experts Language Model"): the RMS-normed latent c, beside one rotated key part that the heads share.  A
-    position sees the last ``window`` ones.  Single rows and short runs score in the latent space (W_uk on the query, W_uv on the output);
-    long runs multiply the window's keys and values out and take the tensor-core attention."""
+    Efficient Mixture-of-Experts Language Model"): the RMS-normed latent c, beside one rotated key part that the heads share.  Queries are a
+    product of the input, or (``q_rank``) of a normed latent of their own; the rotation may turn neighbours or halves, at scaled frequencies;
+    ``gated``: the heads' outputs times sigmoid(W_g h).  A position sees the last ``mask.size`` ones, or all of them.  Single rows and short
+    runs score in the latent space (W_uk on the query, W_uv on the output); long runs multiply the visible keys and values out and take the
+    tensor-core attention."""
 
-    PROJ = ("q", "dkv")
-
-    def __init__(self, w: W, spec: dict, eps: float, max_context: int):
+    def __init__(self, w: W, spec: dict, eps: float, max_context: int, halves: bool = False, gated: bool = False):
         self.H, self.dim, self.rot, self.vdim, self.rank = spec["heads"], spec["dim"], spec["rot_dim"], spec["vdim"], spec["kv_rank"]
-        self.scale, self.eps, self.window = float(spec["scale"]), eps, min(int(spec["mask"]["size"]), max_context)
-        self.w_in, self.w_out, self.norm = w.act(*self.PROJ, pad=8), w.act("o"), w.f32("dkv.norm")
+        self.q_rank, self.halves, self.gated = spec.get("q_rank", 0), halves, gated
+        self.scale, self.eps = float(spec["scale"]), eps
+        self.window = min(int(spec["mask"]["size"]), max_context) if spec.get("mask") else max_context
+        names = (["g"] if gated else []) + (["dkv", "dq"] if self.q_rank else ["q", "dkv"])
+        self.w_in, self.w_out, self.norm = w.act(*names, pad=8), w.act("o"), w.f32("dkv.norm")
+        # columns of the stacked projection: gate, then queries and latent, or latent and the queries' latent
+        self.col_q = H_out = self.H * self.vdim if gated else 0
+        self.col_c = H_out + (0 if self.q_rank else self.H * (self.dim + self.rot))
+        self.col_cq = self.col_c + self.rank + self.rot
+        self.uq, self.q_norm = (w.act("uq"), w.f32("dq.norm")) if self.q_rank else (None, None)
         self.uk = w.act("uk").view(self.H, self.dim, self.rank)
         self.uv = w.act("uv").view(self.H, self.vdim, self.rank).transpose(1, 2).contiguous()       # [H, rank, vdim]
-        self.cs = rotation_table(spec["rot"]["base"], self.rot, max_context, w.device)
+        self.cs = rotation_table(spec["rot"]["base"], self.rot, max_context, w.device, spec["rot"].get("scaling"))
         self.tc = R.latent_tc_supports(w.dtype, self.dim, self.rot, self.vdim, self.rank)
         self.dec = R.latent_decode_supports(w.dtype, self.rot, self.rank)
         self.merge, self.kv_run = (None, None), (1, self.rank + self.rot, 0)
@@ -498,6 +533,9 @@ class LatentAttention:
         n, dt, key = e.max_rows, self.w_in.dtype, self.rank + self.rot
         e.scratch.reserve("proj", n * self.w_in.shape[0], dt)
         e.scratch.reserve("mix_o", n * self.H * self.vdim, dt)
+        if self.q_rank:
+            e.scratch.reserve("lat_cq", n * self.q_rank, dt)
+            e.scratch.reserve("lat_heads", n * self.H * (self.dim + self.rot), dt)
         short = min(n, e.short_rows(self.tc))
         e.scratch.reserve("lat_q", short * self.H * key, dt)
         e.scratch.reserve("lat_o", short * self.H * self.rank, dt)
@@ -517,40 +555,57 @@ class LatentAttention:
     def bind_run(self, e, tag: str, kv_index):
         return {"kv": e.kv.k[kv_index]}
 
+    def queries(self, s, h, pool):
+        """Projections, norms and the cache append; (heads' queries [n, .], what head_proj still has to turn, gate or None)."""
+        n, H, dim, rot = s.n, self.H, self.dim, self.rot
+        proj = R.linear(h, self.w_in, None, s.scratch.get("proj", n, self.w_in.shape[0]))
+        gate = proj[:, :H * self.vdim] if self.gated else None
+        where, sizes = (s.table, s.row_lane, s.row_pos, n), (H, dim, rot, self.rank)
+        if not self.q_rank:
+            q = proj[:, self.col_q:]
+            R.latent_append(q, proj[:, self.col_c:], self.norm, self.cs, pool, *where, *sizes, self.eps, s.status, self.halves)
+            return q, None, gate
+        cq = s.scratch.get("lat_cq", n, self.q_rank)
+        R.latent_append(None, proj[:, self.col_c:], self.norm, self.cs, pool, *where, *sizes, self.eps, s.status, self.halves, proj[:, self.col_cq:], self.q_norm, cq)
+        q = R.linear(cq, self.uq, None, s.scratch.get("lat_heads", n, H * (dim + rot)))
+        if (s.ntiles and self.tc) or not self.halves:
+            R.latent_turn(q, self.cs, s.row_pos, n, H, dim, rot, self.halves)
+            return q, None, gate
+        return q, (self.cs, s.row_pos), gate
+
     def run(self, s, h, run):
         n, H, dim, rot, key, pool = s.n, self.H, self.dim, self.rot, self.rank + self.rot, run["kv"]
-        proj = R.linear(h, self.w_in, None, s.scratch.get("proj", n, self.w_in.shape[0]))
-        R.latent_append(proj, self.norm, self.cs, pool, s.table, s.row_lane, s.row_pos, n, H, dim, rot, self.rank, self.eps, s.status)
+        heads, turn, gate = self.queries(s, h, pool)
         o = s.scratch.get("mix_o", n, H * self.vdim)
-        if s.ntiles:
+        short_rows, m = s.single_rows(self.tc)
+        if s.ntiles and self.tc:
             pages, count, offs = s.expand[self.window]
-            m = count * 64
-            rows = s.scratch.get("lat_rows", m, key)
-            kx, vx = s.scratch.get("lat_k", H, m, dim), s.scratch.get("lat_v", H, m, self.vdim)
+            seen = count * 64
+            rows = s.scratch.get("lat_rows", seen, key)
+            kx, vx = s.scratch.get("lat_k", H, seen, dim), s.scratch.get("lat_v", H, seen, self.vdim)
             R.gather_pages(pool, pages, rows, count, s.status)
             R.expand(rows[:, :self.rank], self.uk.transpose(1, 2), kx)
             R.expand(rows[:, :self.rank], self.uv, vx)
-            R.latent_attn_tc(proj, proj.shape[1], kx, vx, rows, self.rank, s.row_pos, s.tiles, offs, s.ntiles, o, H, dim, rot, self.vdim, self.window,
-                             self.scale, s.status)
-        if s.short:
-            m = s.short
+            R.latent_attn_tc(heads, heads.stride(0), kx, vx, rows, self.rank, s.row_pos, s.tiles, offs, s.ntiles, o, H, dim, rot, self.vdim, self.window,
+                             self.scale, s.status, gate)
+        if m:
             q, c = s.scratch.get("lat_q", m, H * key), s.scratch.get("lat_o", m, H * self.rank)
-            R.head_proj(proj, dim + rot, self.uk, q, key, m, s.short_rows, 1, rot)
-        if s.short and self.dec:
+            R.head_proj(heads, dim + rot, self.uk, q, key, m, short_rows, 1, rot, turn=turn)
+        if m and self.dec:
             part, ml = s.scratch.buf["attn_part"], s.scratch.buf["attn_ml"]
             blocks = R.latent_blocks(self.window, min(s.pages * 64, s.engine.max_context) - 1)
-            idx = s.short_rows if s.short_rows is not None else s.engine._iota[:m]
+            idx = short_rows if short_rows is not None else s.engine._iota[:m]
             for a in range(0, m, self.slice):
                 b = min(m, a + self.slice)
                 R.latent_decode(q[a:b], pool, self.rank, rot, s.table, s.row_lane, s.row_pos, idx[a:b], b - a, H, part, ml, self.window, blocks,
                                 self.scale, s.status)
-                R.head_proj(None, 0, self.uv, o, self.vdim, b - a, idx[a:b], 2, merge=(part, ml, s.row_pos, self.window, blocks))
-        elif s.short:
+                R.head_proj(None, 0, self.uv, o, self.vdim, b - a, idx[a:b], 2, merge=(part, ml, s.row_pos, self.window, blocks), gate=gate)
+        elif m:
             blocks = R.attn_blocks(H, 1)
             sp = s.engine.splits(s, m, blocks, self.window)
             part, ml = (s.scratch.buf["attn_part"], s.scratch.buf["attn_ml"]) if sp > 1 else (None, None)
-            R.attn(q, pool, None, s.table, s.row_lane, s.row_pos, s.short_rows, m, None, c, part, ml, H, self.scale, sp, s.status, self.window, self.rank, True)
-            R.head_proj(c, self.rank, self.uv, o, self.vdim, m, s.short_rows, 2)
+            R.attn(q, pool, None, s.table, s.row_lane, s.row_pos, short_rows, m, None, c, part, ml, H, self.scale, sp, s.status, self.window, self.rank, True)
+            R.head_proj(c, self.rank, self.uv, o, self.vdim, m, short_rows, 2, gate=gate)
         return R.linear(o, self.w_out, None, s.scratch.get("y", n, h.shape[1])), None
 
 
@@ -571,21 +626,39 @@ class DenseFF:
         return R.linear(act, self.w_out, None, s.scratch.get("y", s.n, h.shape[1]))
 
 
-class MixtureFF:
-    """Every row through ``top`` of ``experts`` small feed-forwards, weighted by the softmax over their router logits, and through a shared one,
-    weighted by the sigmoid of a logit of its own.  An expert: W_down (g sigmoid(alpha g) (u + 1)), g = min(W_gate h, limit), u = W_up h within
-    +-limit.  ``run`` returns the parts [n, top + shared, width] and their weights; the seam adds them up."""
+class SingleFF:
+    """W_down act(W_up h); act of one input, with up to two numbers: relu2, or xielu."""
 
-    def __init__(self, w: W, spec: dict, alpha: float):
+    def __init__(self, w: W, act: str, a: float = 0.0, b: float = 0.0):
+        self.act, self.a, self.b = act, a, b
+        self.w_in, self.w_out = w.act("up"), w.act("down")
+        self.ff = self.w_out.shape[1]
+
+    def reserve(self, e) -> None:
+        e.scratch.reserve("ff_act", e.max_rows * self.ff, self.w_in.dtype)
+
+    def run(self, s, h):
+        act = R.act_linear(h, self.w_in, s.scratch.get("ff_act", s.n, self.ff), self.act, self.a, self.b)
+        return R.linear(act, self.w_out, None, s.scratch.get("y", s.n, h.shape[1]))
+
+
+class MixtureFF:
+    """Every row through ``top`` of ``experts`` small feed-forwards, chosen and weighted as ``choice`` says (R.Choice), and through a shared one,
+    weighted by the sigmoid of a logit of its own.  An expert with the "clamp" activation: W_down (g sigmoid(alpha g) (u + 1)), g = min(W_gate h,
+    limit), u = W_up h within +-limit; with one of R.SINGLE_ACT: W_down act(W_up h).  ``run`` returns the parts [n, top + shared, width] and
+    their weights; the seam adds them up."""
+
+    def __init__(self, w: W, spec: dict, alpha: float = 0.0, act: str = "clamp", choice: R.Choice = R.SOFTMAX):
         self.E, self.top = spec["router"]["experts"], spec["router"]["top"]
-        self.ff, self.limit, self.alpha = spec["expert"]["ff"], float(spec["expert"]["limit"]), alpha
+        self.ff, self.limit, self.alpha, self.act, self.choice = spec["expert"]["ff"], float(spec["expert"].get("limit", 0.0)), alpha, act, choice
+        first = ("gate", "up") if act == "clamp" else ("up",)
         sh = spec.get("shared")
-        self.shared, self.shared_ff, self.shared_limit = int(sh is not None), sh["ff"] if sh else 0, float(sh["limit"]) if sh else 0.0
+        self.shared, self.shared_ff, self.shared_limit = int(sh is not None), sh["ff"] if sh else 0, float(sh.get("limit", 0.0)) if sh else 0.0
         self.slots = self.top + self.shared
-        self.w_in = torch.stack([w.act(f"e{i}.gate", f"e{i}.up") for i in range(self.E)]).contiguous()        # [E, 2 ff, width]
+        self.w_in = torch.stack([w.act(*(f"e{i}.{n}" for n in first)) for i in range(self.E)]).contiguous()   # [E, ff, width], gated: [E, 2 ff, width]
         self.w_out = torch.stack([w.act(f"e{i}.down") for i in range(self.E)]).contiguous()                   # [E, width, ff]
         self.router = w.act("router", *(["shared.sg"] if sh else []), pad=8)
-        self.s_in, self.s_out = (w.act("shared.gate", "shared.up"), w.act("shared.down")) if sh else (None, None)
+        self.s_in, self.s_out = (w.act(*(f"shared.{n}" for n in first)), w.act("shared.down")) if sh else (None, None)
 
     def reserve(self, e) -> None:
         n, dt, d = e.max_rows, self.router.dtype, self.router.shape[1]
@@ -613,25 +686,28 @@ class MixtureFF:
         first = (h, self.s_in, s_act, self.shared_ff, self.shared_limit) if self.shared else None        # the shared expert's part in both products
         second = (s_act, self.s_out, None, d, 0.0) if self.shared else None
         if R.moe_gemv_takes(h, self.ff, self.shared_ff):
-            R.moe_gemv(z, ids, wts, h, self.w_in, act, first, n, self.ff, top, slots, True, self.alpha, self.limit)
-            R.moe_gemv(None, ids, wts, act, self.w_out, parts, second, n, d, top, slots, False)
+            R.moe_gemv(z, ids, wts, h, self.w_in, act, first, n, self.ff, top, slots, self.act, self.alpha, self.limit, self.choice)
+            R.moe_gemv(None, ids, wts, act, self.w_out, parts, second, n, d, top, slots, None)
             return parts, wts
         plan = (s.scratch.get("moe_order", n * top), s.scratch.get("moe_tiles", R.moe_tiles(n, self.E, top, self.tile), 4), s.scratch.get("moe_count", 4),
                 R.moe_tiles(n, self.E, top, self.tile))
         if n > R.MOE_PLAN_ROWS:
-            R.moe_route(z, ids, wts, self.E, top, self.shared)
-        R.moe_plan(z if n <= R.MOE_PLAN_ROWS else None, ids, wts, *plan[:3], self.E, top, self.shared, self.tile)
+            R.moe_route(z, ids, wts, self.E, top, self.shared, self.choice)
+        R.moe_plan(z if n <= R.MOE_PLAN_ROWS else None, ids, wts, *plan[:3], self.E, top, self.shared, self.tile, self.choice)
         if self.tc:
             few, x = n <= R.MOE_GATHER_ROWS, h
             if not few:
                 x = s.scratch.get("moe_x", n * top, d)
                 R.moe_pick(h, plan[0], x, top)
-            R.moe_gemm(x, self.w_in, act, plan, first, n, self.ff, top, slots, True, s.status, self.alpha, self.limit, few)
-            R.moe_gemm(act, self.w_out, parts, plan, second, n, d, top, slots, False, s.status)
+            R.moe_gemm(x, self.w_in, act, plan, first, n, self.ff, top, slots, self.act, s.status, self.alpha, self.limit, few)
+            R.moe_gemm(act, self.w_out, parts, plan, second, n, d, top, slots, None, s.status)
             return parts, wts
-        R.moe_tile(h, self.w_in, act, plan, self.ff, top, slots, True, self.alpha, self.limit)
-        R.moe_tile(act, self.w_out, parts, plan, d, top, slots, False)
-        if self.shared:
+        R.moe_tile(h, self.w_in, act, plan, self.ff, top, slots, self.act, self.alpha, self.limit)
+        R.moe_tile(act, self.w_out, parts, plan, d, top, slots, None)
+        if self.shared and self.act != "clamp":
+            R.act_linear(h, self.s_in, s_act, self.act, self.alpha, self.shared_limit)
+            R.linear(s_act, self.s_out, None, parts[:, top])
+        elif self.shared:
             R.gated_linear(h, self.s_in, s.scratch.get("proj", n, 2 * self.shared_ff), s_act, "clamp", self.alpha, self.shared_limit)
             R.linear(s_act, self.s_out, None, parts[:, top])
         return parts, wts
@@ -655,3 +731,11 @@ class TokenInput:
         z, g = s.scratch.get("side_z", n, self.dim), s.scratch.get("side_g", n, self.dim)
         R.token_linear(h, self.gate, self.table, self.col0, s.tokens, z, g, s.status)
         return R.linear(g, self.proj, None, s.scratch.get("y", n, h.shape[1]))
+
+
+class StreamMix:
+    """How a sublayer reads the residual's streams and how its output goes back into them (R.stream_seam): ``into`` [streams], ``mix`` [from, to],
+    ``out`` [streams], with the residual's factor ``m`` on the output."""
+
+    def __init__(self, w: W, m: float):
+        self.into, self.mix, self.out = w.f32("in"), w.f32("mix"), (m * w.f32("out")).contiguous()

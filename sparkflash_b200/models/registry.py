@@ -29,12 +29,13 @@ MODELS = {m.name: m for m in [
     ModelEntry("fanodra", "fanodra", "device", "gated linear recurrence, alone or beside attention with a distance bias; looped layers, input convolution; layered engine (bf16 or 32-bit)", "sparkflash_b200.models.fanodra"),
     ModelEntry("gudutar", "gudutar", "device", "state-space duality, retention and latent attention in a window; norms on sublayer outputs, layers that share weights; layered engine (bf16 or 32-bit)", "sparkflash_b200.models.gudutar"),
     ModelEntry("lifulorn", "lifulorn", "device", "gated delta rule and windowed attention with sinks, capped scores and mixed values; mixture of experts, per-layer token input; layered engine (bf16 or 32-bit)", "sparkflash_b200.models.lifulorn"),
+    ModelEntry("dironex", "dironex", "device", "latent attention with a latent for the queries and an output gate, windowed attention with normed heads; several residual streams, looped layers, grouped experts; layered engine (bf16 or 32-bit)", "sparkflash_b200.models.dironex"),
     ModelEntry("dflash-block-drafter", "drafter", "oracle", "one-forward block drafter over a ring of captured target features", "sparkflash_b200.models.dflash"),
 ]}
 
 # config.json "architecture" -> (module, class) of the models that run on the layered engine (models/layered.py)
 LAYERED = {"Fanodra": ("sparkflash_b200.models.fanodra", "Fanodra"), "Gudutar": ("sparkflash_b200.models.gudutar", "Gudutar"),
-           "Lifulorn": ("sparkflash_b200.models.lifulorn", "Lifulorn")}
+           "Lifulorn": ("sparkflash_b200.models.lifulorn", "Lifulorn"), "Dironex": ("sparkflash_b200.models.dironex", "Dironex")}
 
 
 def architecture(path: str) -> str:

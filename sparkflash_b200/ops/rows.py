@@ -42,6 +42,23 @@ def seam(x, n, *, h=None, y=None, y2=None, merge_w=(None, None), post=(None, Non
                                      c_int(embed.shape[0] if embed is not None else 0), c_float(eps), c_float(embed_scale), _fp32(act), _p(status), _stream()), "rows_seam")
 
 
+MAX_STREAMS = 8
+
+
+def stream_seam(x, n, *, h, norm, y=None, parts_w=None, mix=None, out=None, into=None, embed=None, tokens=None, embed_scale=1.0, tap=None, row_map=None, conv=None,
+                keep=True, eps=1e-6, status=None):
+    """Several residual streams x [rows, streams, d]: x_t = sum_s mix[s, t] x_s + out[t] y (y None: every stream is the scaled embedding), then
+    h = RMS(sum_t into[t] x_t; norm) (``into`` None: ones).  ``parts_w`` [rows, parts]: y is [rows, parts, d] and its weighted sum the output.
+    ``conv``: (weight [taps, d], history, src, dst) applies h + conv(h) on a step of single-row segments.  ``keep`` False: the streams end here."""
+    cw, hist, src, dst = conv if conv is not None else (None, None, None, None)
+    S, d = x.shape[1], x.shape[2]
+    _check(_lib.rows().sfb_rows_streams(_p(x), _p(y), _p(parts_w), _p(mix), _p(out), _p(embed), _p(tokens), _p(tap), _p(into), _p(norm), _p(h), _p(row_map), _p(cw),
+                                        _p(hist), _p(src), _p(dst), c_int(S), c_int(parts_w.shape[1] if parts_w is not None else 0),
+                                        c_int(cw.shape[0] if cw is not None else 0), c_int(keep), c_int(n), c_int(d),
+                                        c_int(embed.shape[0] if embed is not None else 0), c_float(eps), c_float(embed_scale), _fp32(h), _p(status), _stream()),
+           "rows_streams")
+
+
 CONV_PLAIN, CONV_RESIDUAL, CONV_SILU = 0, 1, 2
 
 
@@ -57,6 +74,14 @@ def qk_append(proj, qw, kw, q, kpool, vpool, table, row_lane, row_pos, n, heads,
     _check(_lib.rows().sfb_rows_qk_append(_p(proj), c_int64(proj.stride(0)), _p(qw), _p(kw), _p(q), _p(kpool), _p(vpool), _p(table), _p(row_lane),
                                           _p(row_pos), c_int(table.shape[1]), c_int(kpool.shape[0]), c_int(n), c_int(heads), c_int(G), c_int(dim),
                                           c_int(vdim), c_float(eps), _fp32(q), _p(status), _stream()), "rows_qk_append")
+
+
+def head_append(proj, qw, kw, q, kpool, vpool, table, row_lane, row_pos, n, heads, eps, status):
+    """q | k | v of ``proj``: RMS norm of every query and key head (weights [dim]), queries to ``q``, the rest to the pools."""
+    G, dim, vdim = kpool.shape[1], kpool.shape[3], vpool.shape[3]
+    _check(_lib.rows().sfb_rows_head_append(*_strides(proj), _p(qw), _p(kw), _p(q), _p(kpool), _p(vpool), _p(table), _p(row_lane), _p(row_pos),
+                                            c_int(table.shape[1]), c_int(kpool.shape[0]), c_int(n), c_int(heads), c_int(G), c_int(dim), c_int(vdim),
+                                            c_float(eps), _fp32(q), _p(status), _stream()), "rows_head_append")
 
 
 def rot_append(proj, cs, dims, q, kpool, vpool, v_first, lam, table, row_lane, row_pos, n, heads, status):
@@ -122,6 +147,23 @@ def act_mul(gate_up, out, n, act="silu", alpha=0.0, limit=0.0):
     """out = act(gate) * up; "clamp": g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = up within +-limit."""
     _check(_lib.rows().sfb_rows_act_mul(_p(gate_up), *_strides(out), c_int(n), c_int(out.shape[1]), c_int(ACT[act]), c_float(alpha), c_float(limit), _fp32(out),
                                         _stream()), "rows_act_mul")
+
+
+SINGLE_ACT = {"relu2": 4, "xielu": 5}          # activations of one input, with up to two numbers
+
+
+def act_linear(x, w, out, act, a=0.0, b=0.0):
+    """out = act(x w^T): one kernel for few rows, else a product and an element-wise pass over it."""
+    if _gemv_takes(x):
+        _gemv(x, w, None, out, SINGLE_ACT[act], a, b)
+        return out
+    linear(x, w, None, out)
+    return act_rows(out, out, act, a, b)
+
+
+def act_rows(z, out, act, a=0.0, b=0.0):
+    _check(_lib.rows().sfb_rows_act(_p(z), _p(out), c_int64(out.numel()), c_int(SINGLE_ACT[act]), c_float(a), c_float(b), _fp32(out), _stream()), "rows_act")
+    return out
 
 
 def _strides(t) -> tuple:
@@ -208,21 +250,33 @@ def gated_norm(y, gate, w, out, part, before, eps):
                                            c_float(eps), _fp32(y), _stream()), "rows_gated_norm")
 
 
-def latent_append(proj, w, cs, pool, table, row_lane, row_pos, n, heads, dim, rot, rank, eps, status):
-    """Norm and rotation of q | latent | shared key part in ``proj``: queries in place, the rest to the pool [pages, 1, 64, rank + rot]."""
-    _check(_lib.rows().sfb_rows_latent_append(*_strides(proj), _p(w), _p(cs), _p(pool), _p(table), _p(row_lane), _p(row_pos), c_int(table.shape[1]),
-                                              c_int(pool.shape[0]), c_int(n), c_int(heads), c_int(dim), c_int(rot), c_int(rank), c_float(eps), _fp32(pool),
-                                              _p(status), _stream()), "rows_latent_append")
+def latent_append(q, c, w, cs, pool, table, row_lane, row_pos, n, heads, dim, rot, rank, eps, status, halves=False, cq=None, wq=None, cq_out=None):
+    """``c`` [n, stride] view of latent | shared key part: normed and turned into the pool [pages, 1, 64, rank + rot].  ``q`` [n, stride] view of the
+    queries, turned in place, or None.  ``cq``, ``wq``: latent of the queries, a view with c's stride, normed to ``cq_out`` [n, q_rank].
+    ``halves``: element i turns with i + rot / 2, else neighbours do."""
+    _check(_lib.rows().sfb_rows_latent_append(*_strides(q), _p(c), _p(cq), _p(cq_out), c_int64(c.stride(0)), _p(w), _p(wq), _p(cs), _p(pool), _p(table), _p(row_lane), _p(row_pos),
+                                              c_int(table.shape[1]), c_int(pool.shape[0]), c_int(n), c_int(heads), c_int(dim), c_int(rot), c_int(rank),
+                                              c_int(wq.shape[0] if wq is not None else 0), c_int(halves), c_float(eps), _fp32(pool), _p(status), _stream()),
+           "rows_latent_append")
 
 
-def head_proj(x, x_head, w, out, out_head, n, rows=None, lists=0, tail=0, merge=None):
+def latent_turn(q, cs, row_pos, n, heads, dim, rot, halves):
+    """The last ``rot`` of every head of q [n, heads (dim + rot)], turned in place (``halves``: element i with i + rot / 2, else neighbours)."""
+    _check(_lib.rows().sfb_rows_latent_turn(*_strides(q), _p(cs), _p(row_pos), c_int(n), c_int(heads), c_int(dim), c_int(rot), c_int(halves), _fp32(q),
+                                            _stream()), "rows_latent_turn")
+
+
+def head_proj(x, x_head, w, out, out_head, n, rows=None, lists=0, tail=0, merge=None, turn=None, gate=None):
     """out[row][h] = x[row][h] w[h], w [heads, K, M]; heads ``x_head`` / ``out_head`` elements apart.  ``rows`` names rows of x (lists=1) or
-    of out (lists=2); ``tail`` elements behind x's K are copied behind out's M.  ``merge``: (part, ml, row_pos, window, blocks) of
-    latent_decode; x is then the merged attention output."""
+    of out (lists=2); ``tail`` elements behind x's K are copied behind out's M, turned by ``turn`` = (cs, row_pos) (element i with i + tail / 2).
+    ``merge``: (part, ml, row_pos, window, blocks) of latent_decode; x is then the merged attention output.  ``gate`` [rows of out, heads M]
+    view: outputs are multiplied by its sigmoid."""
     part, ml, pos, window, blocks = merge or (None, None, None, 1, 0)
+    cs, pos = turn if turn is not None else (None, pos)
     H, K, M = w.shape
     _check(_lib.rows().sfb_rows_head_proj(*_strides(x), c_int64(x_head), _p(w), *_strides(out), c_int64(out_head), _p(rows), c_int(lists if rows is not None else 0),
-                                          _p(part), _p(ml), _p(pos), c_int(window), c_int(blocks), c_int(n), c_int(H), c_int(K), c_int(M), c_int(tail), _fp32(w), _stream()), "rows_head_proj")
+                                          _p(part), _p(ml), _p(pos), c_int(window), c_int(blocks), c_int(n), c_int(H), c_int(K), c_int(M), c_int(tail), _p(cs),
+                                          *_strides(gate), _fp32(w), _stream()), "rows_head_proj")
 
 
 def gather_pages(pool, pages, out, count, status):
@@ -394,8 +448,8 @@ def attn_tc(q, kv, table, row_lane, row_pos, tiles, n_tiles, bias, out, heads, s
     mq = tensor_map(q, q.shape[1], 128)
     G = k.shape[1]
     _check(_lib.rows().sfb_rows_attn_tc(mq.ptr, mk.ptr, mv.ptr, None, _p(table), _p(row_lane), _p(row_pos), _p(tiles), None, c_int(n_tiles), _p(bias),
-                                        c_int64(bias.shape[1] if bias is not None else 0), _p(sink), c_float(cap), _p(out), c_int(table.shape[1]),
-                                        c_int(k.shape[0]), c_int(heads), c_int(G), c_int(k.shape[3]), c_int(v.shape[3]), c_int(0), c_int(G * 64), c_int(64),
+                                        c_int64(bias.shape[1] if bias is not None else 0), _p(sink), c_float(cap), _p(out), None, c_int64(0),
+                                        c_int(table.shape[1]), c_int(k.shape[0]), c_int(heads), c_int(G), c_int(k.shape[3]), c_int(v.shape[3]), c_int(0), c_int(G * 64), c_int(64),
                                         c_int(window), c_float(scale), _p(status), _stream()), "rows_attn_tc")
 
 
@@ -430,14 +484,15 @@ def expand(c: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
     return out
 
 
-def latent_attn_tc(q, q_stride, kx, vx, rows, rank, row_pos, tiles, offs, n_tiles, out, heads, dim, rot, vdim, window, scale, status):
+def latent_attn_tc(q, q_stride, kx, vx, rows, rank, row_pos, tiles, offs, n_tiles, out, heads, dim, rot, vdim, window, scale, status, gate=None):
     """Tensor-core arm over keys kx [heads, m, dim] and values vx [heads, m, vdim] that were multiplied out, and the shared key part: the
-    last columns of ``rows`` [m, rank + rot].  q: [n, q_stride] with a head's dim + rot columns side by side."""
+    last columns of ``rows`` [m, rank + rot].  q: [n, q_stride] with a head's dim + rot columns side by side.
+    ``gate`` [n, heads vdim] view: outputs are multiplied by its sigmoid."""
     m = kx.shape[1]
-    mq, mk, mv = tensor_map(q, heads * (dim + rot), 128, q_stride), tensor_map(kx, dim, 64), tensor_map(vx, vdim, 64)
+    mq, mk, mv = tensor_map(q, heads * (dim + rot), 128, q_stride, q.storage_offset()), tensor_map(kx, dim, 64), tensor_map(vx, vdim, 64)
     mr = tensor_map(rows, rot, 64, rank + rot, rank)
     _check(_lib.rows().sfb_rows_attn_tc(mq.ptr, mk.ptr, mv.ptr, mr.ptr, None, None, _p(row_pos), _p(tiles), _p(offs), c_int(n_tiles), None, c_int64(0), None, c_float(0.0),
-                                        _p(out), c_int(0), c_int(m // 64), c_int(heads), c_int(heads), c_int(dim), c_int(vdim), c_int(rot), c_int(64),
+                                        _p(out), *_strides(gate), c_int(0), c_int(m // 64), c_int(heads), c_int(heads), c_int(dim), c_int(vdim), c_int(rot), c_int(64),
                                         c_int(m), c_int(window), c_float(scale), _p(status), _stream()), "rows_attn_tc")
 
 
@@ -451,28 +506,46 @@ def moe_tiles(n: int, experts: int, top: int, tile: int) -> int:
     return n * top // tile + min(experts, n * top)
 
 
-def moe_route(z, ids, wts, experts, top, shared):
+class Choice:
+    """How a row's experts are chosen and weighted.  ``corr`` None: the largest logits, the softmax over them.  Else s = sigmoid(logit): the largest
+    s + corr [E] among the ``keep`` of ``groups`` groups of neighbours whose two largest sum highest, weighted by s over their sum, times ``scale``."""
+
+    def __init__(self, corr=None, groups: int = 1, keep: int = 1, scale: float = 1.0):
+        self.corr, self.groups, self.keep, self.scale = corr, groups, keep, scale
+
+    def args(self) -> tuple:
+        return _p(self.corr), c_int(self.groups), c_int(self.keep), c_float(self.scale)
+
+
+SOFTMAX = Choice()
+MOE_MAX_GROUPS = 256
+
+
+def moe_route(z, ids, wts, experts, top, shared, choice=SOFTMAX):
     """Choices [n, top] and weights [n, top + shared] of logits z [n, >= experts + shared]."""
-    _check(_lib.rows().sfb_rows_moe_route(*_strides(z), _p(ids), _p(wts), c_int(z.shape[0]), c_int(experts), c_int(top), c_int(shared), _stream()),
+    _check(_lib.rows().sfb_rows_moe_route(*_strides(z), _p(ids), _p(wts), c_int(z.shape[0]), c_int(experts), c_int(top), c_int(shared), *choice.args(), _stream()),
            "rows_moe_route")
 
 
 MOE_PLAN_ROWS = 128        # up to this many rows the plan makes the choice itself
 
 
-def moe_plan(z, ids, wts, order, tiles, count, experts, top, shared, tile):
+def moe_plan(z, ids, wts, order, tiles, count, experts, top, shared, tile, choice=SOFTMAX):
     """``z``: logits (few rows: the choice is made here), or None: ``ids`` are there."""
     zp, ld = _strides(z)
     _check(_lib.rows().sfb_rows_moe_plan(zp, ld, _p(ids), _p(wts), _p(order), _p(tiles), _p(count), c_int(ids.shape[0]), c_int(experts), c_int(top),
-                                         c_int(shared), c_int(tile), _stream()), "rows_moe_plan")
+                                         c_int(shared), c_int(tile), *choice.args(), _stream()), "rows_moe_plan")
 
 
-def moe_tile(x, w, out, plan, M, top, slots, gated, alpha=0.0, limit=0.0):
-    """One product of every expert on its pairs; ``plan``: (order, tiles, count, most tiles).  gated: x [n, K], w [E, 2 M, K], out [pairs, M] in
-    plan order; else x [pairs, K], w [E, M, K], out [n, slots, M]."""
+MOE_ACT = {None: 0, "clamp": 3, **SINGLE_ACT}          # of an expert's first product: gated (gate and up stacked), or of one product; None: the second
+
+
+def moe_tile(x, w, out, plan, M, top, slots, act, alpha=0.0, limit=0.0):
+    """One product of every expert on its pairs; ``plan``: (order, tiles, count, most tiles).  ``act`` (see MOE_ACT): x [n, K], w [E, M, K] (gated:
+    [E, 2 M, K]), out [pairs, M] in plan order; None: x [pairs, K], w [E, M, K], out [n, slots, M]."""
     order, tiles, count, most = plan
     _check(_lib.rows().sfb_rows_moe_tile(_p(x), _p(w), _p(out), _p(order), _p(tiles), _p(count), c_int(most), c_int(M), c_int(w.shape[2]), c_int(top),
-                                         c_int(slots), c_int(gated), c_float(alpha), c_float(limit), _fp32(out), _stream()), "rows_moe_tile")
+                                         c_int(slots), c_int(MOE_ACT[act]), c_float(alpha), c_float(limit), _fp32(out), _stream()), "rows_moe_tile")
 
 
 def moe_tc_supports(dtype: torch.dtype, width: int, ff: int, shared_ff: int) -> bool:
@@ -488,7 +561,7 @@ def moe_pick(x, order, out, top):
     _check(_lib.rows().sfb_rows_moe_pick(_p(x), _p(order), _p(out), c_int(out.shape[0]), c_int(top), c_int(x.shape[1]), _stream()), "rows_moe_pick")
 
 
-def moe_gemm(x, w, out, plan, shared, n, M, top, slots, gated, status, alpha=0.0, limit=0.0, gather=False):
+def moe_gemm(x, w, out, plan, shared, n, M, top, slots, act, status, alpha=0.0, limit=0.0, gather=False):
     """``moe_tile`` on the tensor cores (tiles of up to 128 pairs); w and out in bf16; x in plan order, or ``gather``: the layer's rows.
     ``shared``: (x, w, out, M, limit) of the shared expert, whose rows are done beside the pairs, or None."""
     order, tiles, count, most = plan
@@ -496,7 +569,7 @@ def moe_gemm(x, w, out, plan, shared, n, M, top, slots, gated, status, alpha=0.0
     msx, msw = (tensor_map(sx, sx.shape[1], 128).ptr, tensor_map(sw, sw.shape[1], 128).ptr) if shared is not None else (None, None)
     mx, mw = tensor_map(x, x.shape[1], 1 if gather else 128), tensor_map(w, w.shape[2], 128)
     _check(_lib.rows().sfb_rows_moe_gemm(mx.ptr, mw.ptr, msx, msw, _p(order), _p(tiles), _p(count), _p(out), _p(sout), c_int(most), c_int(n), c_int(M),
-                                         c_int(w.shape[2]), c_int(sm), c_int(sw.shape[1] if sw is not None else 0), c_int(top), c_int(slots), c_int(gated),
+                                         c_int(w.shape[2]), c_int(sm), c_int(sw.shape[1] if sw is not None else 0), c_int(top), c_int(slots), c_int(MOE_ACT[act]),
                                          c_int(gather), c_float(alpha), c_float(limit), c_float(sl), _p(status), _stream()), "rows_moe_gemm")
 
 
@@ -505,10 +578,10 @@ def moe_gemv_takes(x: torch.Tensor, ff: int, shared_ff: int) -> bool:
     return x.dtype == torch.bfloat16 and n <= GEMV_ROWS and K % 8 == 0 and ff % 8 == 0 and shared_ff % 8 == 0 and max(K, ff, shared_ff) * 2 <= 200 * 1024
 
 
-def moe_gemv(z, ids, wts, x, w, out, shared, n, M, top, slots, gated, alpha=0.0, limit=0.0):
+def moe_gemv(z, ids, wts, x, w, out, shared, n, M, top, slots, act, alpha=0.0, limit=0.0, choice=SOFTMAX):
     """Few rows; ``z``: logits, the experts are chosen here and left in ``ids`` and ``wts``; None: ``ids`` are there.  ``shared``: (x, w, out, M,
     limit) of the shared expert or None."""
     sx, sw, sout, sm, sl = shared if shared is not None else (None, None, None, 0, 0.0)
-    _check(_lib.rows().sfb_rows_moe_gemv(*_strides(z), c_int(w.shape[0]), _p(ids), _p(wts), _p(x), _p(w), _p(out), _p(sx), _p(sw), _p(sout), c_int(ids.numel()), c_int(n), c_int(M), c_int(w.shape[2]),
-                                         c_int(sm), c_int(sw.shape[1] if sw is not None else 0), c_int(top), c_int(slots), c_int(gated), c_float(alpha),
+    _check(_lib.rows().sfb_rows_moe_gemv(*_strides(z), c_int(w.shape[0]), _p(ids), _p(wts), *choice.args(), _p(x), _p(w), _p(out), _p(sx), _p(sw), _p(sout), c_int(ids.numel()), c_int(n), c_int(M), c_int(w.shape[2]),
+                                         c_int(sm), c_int(sw.shape[1] if sw is not None else 0), c_int(top), c_int(slots), c_int(MOE_ACT[act]), c_float(alpha),
                                          c_float(limit), c_float(sl), _stream()), "rows_moe_gemv")

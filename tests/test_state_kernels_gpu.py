@@ -238,7 +238,7 @@ def test_latent_append(H, dim, rot, rank, dtype):
     x = proj.cpu().double()
     pool, table, read = _pool(rank, rot, [200], dtype)
     cs, first = rotation_table(50.0, rot, 256, "cuda"), 100
-    R.latent_append(proj, w, cs, pool, table, torch.zeros(n, dtype=torch.int32, device="cuda"), _i32(list(range(first, first + n))), n, H, dim, rot, rank, 1e-2,
+    R.latent_append(proj, proj[:, H * (dim + rot):], w, cs, pool, table, torch.zeros(n, dtype=torch.int32, device="cuda"), _i32(list(range(first, first + n))), n, H, dim, rot, rank, 1e-2,
                     _status())
     turned = lambda t: P.rotate(torch.cat([torch.zeros(first, *t.shape[1:], dtype=torch.float64), t]), 50.0, rot, "pairs")[first:]
     tol = 1e-5 if dtype == torch.float32 else 1e-2
