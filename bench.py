@@ -510,7 +510,7 @@ def main() -> None:
     ap.add_argument("--prefill-chunk", type=int, default=4096, help="rows per prompt chunk (the reference prefills 4,096-row chunks)")
     ap.add_argument("--no-mtp", action="store_true", help="skip the DSpark draft-path section")
     ap.add_argument("--no-ep", action="store_true", help="skip the expert-parallel section (2+ GPUs)")
-    ap.add_argument("--design", default="", choices=["", "fanodra", "gudutar", "lifulorn"], help="benchmark a layered design instead of the headline model: prefill and "
+    ap.add_argument("--design", default="", choices=["", "fanodra", "gudutar", "lifulorn", "dironex"], help="benchmark a layered design instead of the headline model: prefill and "
                     "decode throughput and per-kernel roofline fractions, beside the closest model (one JSON line)")
     ap.add_argument("--design-sizes", default="w1024,w2048,w4096", help="sizes of --design (sparkflash_b200/utils/layered_bench.py)")
     args = ap.parse_args()

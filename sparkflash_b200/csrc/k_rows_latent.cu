@@ -163,9 +163,10 @@ struct HeadProjArgs {
   void* out;                // (T)
   int64_t out_row, out_head;
   const int* rows;          // row of x (x_list) or of out (out_list) for every launch row, or null: identity
-  const float *part, *ml;   // or x is to be merged: [launch rows, H, blocks, K] and (log2 maximum, sum) of every block
-  const int* row_pos;
-  int window, blocks;
+  const float *part, *ml;   // or x is to be merged: [places, H, K] and (log2 maximum, sum) of every partial result
+  const int2* parts;        // first place and number of places of every launch row
+  int most;                 // at least the places of a row
+  const int* row_pos;       // (cs)
   int x_list, out_list, n, H, K, M, tail;   // tail: elements after x's K that are copied after out's M
   const float2* cs;         // [positions, tail / 2]: the tail is turned (element i with i + tail / 2) by its row's position, or null
   const void* gate;         // (T) outputs are multiplied by sigmoid(gate[row of out][h M + m]), or null
@@ -199,37 +200,48 @@ __global__ void __launch_bounds__(HP_T) head_proj_kernel(HeadProjArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   if (a.part) {
-    __shared__ int wn[HP_R];
-    float* wt = red;                                   // [HP_R][blocks]
+    __shared__ int wn[HP_R], w0[HP_R];
+    float* wt = red;                                   // [HP_R][most], then the groups' sums [groups][HP_R][K]
     const int warp = tid >> 5, lane = tid & 31;
     if (warp < nr) {
-      const int row = a.rows ? a.rows[r0 + warp] : r0 + warp, pos = a.row_pos[row], first = max(0, pos - a.window + 1);
-      const int nb = min(a.blocks, (pos / 64 - first / 64) / 2 + 1);
-      const float* ml = a.ml + ((size_t)(r0 + warp) * a.H + h) * a.blocks * 2;
+      const int2 places = a.parts[r0 + warp];
+      const int place = places.x, nb = places.y;
+      const float* ml = a.ml + ((size_t)place * a.H + h) * 2;
+      const size_t step = (size_t)a.H * 2;
       float m = -INFINITY, l = 0.f;
-      for (int b = lane; b < nb; b += 32) m = fmaxf(m, ml[2 * b]);
+      for (int b = lane; b < nb; b += 32) m = fmaxf(m, ml[b * step]);
       m = warp_max(m);
-      for (int b = lane; b < nb; b += 32) l += ml[2 * b + 1] * exp2f(ml[2 * b] - m);
+      for (int b = lane; b < nb; b += 32) l += ml[b * step + 1] * exp2f(ml[b * step] - m);
       const float inv = 1.f / warp_sum(l);
-      for (int b = lane; b < nb; b += 32) wt[warp * a.blocks + b] = exp2f(ml[2 * b] - m) * inv;
-      if (lane == 0) wn[warp] = nb;
+      for (int b = lane; b < nb; b += 32) wt[warp * a.most + b] = exp2f(ml[b * step] - m) * inv;
+      if (lane == 0) { wn[warp] = nb; w0[warp] = place; }
     }
     __syncthreads();
-    const int K4 = a.K >> 2;                           // K (the latent's size) is a multiple of eight
-    for (int i = tid; i < HP_R * K4; i += HP_T) {
-      const int r = i / K4, k = (i - r * K4) * 4;
-      float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (r < nr) {
-        const int nb = wn[r];
-        const float* p = a.part + ((size_t)(r0 + r) * a.H + h) * a.blocks * a.K + k;
+    const int K4 = a.K >> 2, groups = HP_T / K4;       // K (the latent's size) is a multiple of eight, up to 512
+    const int grp = tid / K4, k = (tid - grp * K4) * 4;
+    float* gs = red + ((HP_R * a.most + 3) & ~3);
+    if (grp < groups) {
+      for (int r = 0; r < HP_R; ++r) {
+        float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (r < nr) {
+          const int nb = wn[r];
+          const float* p = a.part + ((size_t)w0[r] * a.H + h) * a.K + k;
+          const size_t step = (size_t)a.H * a.K;
 #pragma unroll 8
-        for (int b = 0; b < nb; ++b) {
-          const float wb = wt[r * a.blocks + b];
-          const float4 v = *reinterpret_cast<const float4*>(p + (size_t)b * a.K);
-          f.x = fmaf(wb, v.x, f.x); f.y = fmaf(wb, v.y, f.y); f.z = fmaf(wb, v.z, f.z); f.w = fmaf(wb, v.w, f.w);
+          for (int b = grp; b < nb; b += groups) {
+            const float wb = wt[r * a.most + b];
+            const float4 v = *reinterpret_cast<const float4*>(p + b * step);
+            f.x = fmaf(wb, v.x, f.x); f.y = fmaf(wb, v.y, f.y); f.z = fmaf(wb, v.z, f.z); f.w = fmaf(wb, v.w, f.w);
+          }
         }
+        *reinterpret_cast<float4*>(gs + (size_t)(grp * HP_R + r) * a.K + k) = f;
       }
-      *reinterpret_cast<float4*>(xs + r * a.K + k) = f;
+    }
+    __syncthreads();
+    for (int i = tid; i < HP_R * a.K; i += HP_T) {
+      float f = 0.f;
+      for (int q = 0; q < groups; ++q) f += gs[(size_t)q * HP_R * a.K + i];
+      xs[i] = f;
     }
   } else {
     for (int i = tid; i < HP_R * a.K; i += HP_T) {
@@ -313,7 +325,7 @@ __global__ void __launch_bounds__(256) gather_pages_kernel(const uint4* pool, co
 
 template <typename T, int V, int MG>
 static int launch_head_proj(const HeadProjArgs& a, cudaStream_t st) {
-  const size_t red = (size_t)HP_T * HP_R * 8, wts = (size_t)HP_R * a.blocks;
+  const size_t red = (size_t)HP_T * HP_R * 8, wts = ((size_t)HP_R * a.most + 3) / 4 * 4 + HP_T * 4 * HP_R;
   const size_t smem = (((size_t)HP_R * a.K + 3) / 4 * 4 + (red > wts ? red : wts)) * sizeof(float);
   if (smem > 220 * 1024) return (int)cudaErrorInvalidValue;
   static size_t granted = 48 * 1024;
@@ -380,12 +392,12 @@ int sfb_rows_latent_turn(void* q, int64_t stride, const void* cs, const int* row
 // list: 0 = rows ignored, 1 = it names x's rows, 2 = it names out's rows.  part (then x is null), cs, gate: see HeadProjArgs; with part, list
 // is 2 or 0.
 int sfb_rows_head_proj(const void* x, int64_t x_row, int64_t x_head, const void* w, void* out, int64_t out_row, int64_t out_head, const int* rows, int list,
-                       const void* part, const void* ml, const int* row_pos, int window, int blocks, int n, int H, int K, int M, int tail, const void* cs,
+                       const void* part, const void* ml, const void* parts, int most, const int* row_pos, int n, int H, int K, int M, int tail, const void* cs,
                        const void* gate, int64_t gate_row, int fp32, cudaStream_t stream) {
-  if (n < 1 || n > 65535 * HP_R || H < 1 || K < 1 || M < 1 || K > 8192 || (part && (K % 8 || blocks < 1 || tail || list == 1)) ||
+  if (n < 1 || n > 65535 * HP_R || H < 1 || K < 1 || M < 1 || K > 8192 || (part && (K % 8 || K > 512 || most < 1 || !parts || tail || list == 1)) ||
       (cs && (tail < 2 || tail % 2 || !row_pos)))
     return (int)cudaErrorInvalidValue;
-  HeadProjArgs a{x, x_row, x_head, w, out, out_row, out_head, list ? rows : nullptr, (const float*)part, (const float*)ml, row_pos, window, part ? blocks : 0,
+  HeadProjArgs a{x, x_row, x_head, w, out, out_row, out_head, list ? rows : nullptr, (const float*)part, (const float*)ml, (const int2*)parts, part ? most : 0, row_pos,
                  list == 1, list == 2, n, H, K, M, tail, (const float2*)cs, gate, gate_row};
   return fp32 ? launch_head_proj_t<float>(a, stream) : launch_head_proj_t<__nv_bfloat16>(a, stream);
 }

@@ -111,9 +111,9 @@ __device__ __forceinline__ uint64_t desc(uint32_t saddr, uint32_t lbo) {
   return (uint64_t)((saddr >> 4) & 0x3fff) | (uint64_t)((lbo >> 4) & 0x3fff) << 16 | (uint64_t)(1024 >> 4) << 32 | (uint64_t)1 << 46 |
          (uint64_t)2 << 61;
 }
-// kind::f16: bf16 operands, 32-bit accumulator, M = 128
-__device__ __forceinline__ uint32_t idesc(int N, int a_mn, int b_mn) {
-  return 1u << 4 | 1u << 7 | 1u << 10 | (uint32_t)a_mn << 15 | (uint32_t)b_mn << 16 | (uint32_t)(N >> 3) << 17 | (128u >> 4) << 24;
+// kind::f16: bf16 operands, 32-bit accumulator.  M = 128: accumulator row = lane; M = 64: rows 16 w .. 16 w + 15 in the first lanes of warp w
+__device__ __forceinline__ uint32_t idesc(int N, int a_mn, int b_mn, uint32_t M = 128) {
+  return 1u << 4 | 1u << 7 | 1u << 10 | (uint32_t)a_mn << 15 | (uint32_t)b_mn << 16 | (uint32_t)(N >> 3) << 17 | (M >> 4) << 24;
 }
 // one 32-bit value as two bf16 terms, for pairs of neighbours: hi = the upper halves, lo = the rounded rest
 __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {

@@ -16,7 +16,6 @@ import torch.nn.functional as F
 
 from ..ops import rows as R
 
-DECODE_ROWS = 64           # single rows of latent attention whose partial results are held at a time
 CONV_STEP_ROWS = 4         # up to this many single rows the matrix-state kernel applies the convolution itself (every head does B and C again)
 GATED_STEP_ROWS = 16       # up to this many single rows run convolution, gates and recurrence as one kernel
 
@@ -540,8 +539,9 @@ class LatentAttention:
         e.scratch.reserve("lat_q", short * self.H * key, dt)
         e.scratch.reserve("lat_o", short * self.H * self.rank, dt)
         if self.dec:
-            self.slice = min(short, DECODE_ROWS)
-            parts = self.slice * self.H * R.latent_blocks(self.window, e.max_context - 1)
+            self.slice = min(short, R.LATENT_ROWS)
+            e.scratch.reserve("lat_parts", 2 * self.slice, torch.int32)
+            parts = R.latent_places(self.slice, self.H) * self.H
         else:
             parts = max(1, self.H // R.attn_blocks(self.H, 1)) * 1024 + self.H * 64
         e.scratch.reserve("attn_part", parts * self.rank, torch.float32)
@@ -593,13 +593,14 @@ class LatentAttention:
             R.head_proj(heads, dim + rot, self.uk, q, key, m, short_rows, 1, rot, turn=turn)
         if m and self.dec:
             part, ml = s.scratch.buf["attn_part"], s.scratch.buf["attn_ml"]
-            blocks = R.latent_blocks(self.window, min(s.pages * 64, s.engine.max_context) - 1)
+            parts, seen = s.scratch.get("lat_parts", self.slice, 2), min(s.pages, -(-s.engine.max_context // R.PAGE), (self.window + R.PAGE - 2) // R.PAGE + 1)
             idx = short_rows if short_rows is not None else s.engine._iota[:m]
             for a in range(0, m, self.slice):
                 b = min(m, a + self.slice)
-                R.latent_decode(q[a:b], pool, self.rank, rot, s.table, s.row_lane, s.row_pos, idx[a:b], b - a, H, part, ml, self.window, blocks,
-                                self.scale, s.status)
-                R.head_proj(None, 0, self.uv, o, self.vdim, b - a, idx[a:b], 2, merge=(part, ml, s.row_pos, self.window, blocks), gate=gate)
+                ctas = R.latent_ctas(H, (b - a) * seen)
+                R.latent_decode(q[a:b], pool, self.rank, rot, s.table, s.row_lane, s.row_pos, idx[a:b], b - a, H, part, ml, parts, self.window, ctas,
+                                (b - a) * seen, self.scale, s.status)
+                R.head_proj(None, 0, self.uv, o, self.vdim, b - a, idx[a:b], 2, merge=(part, ml, parts, ctas), gate=gate)
         elif m:
             blocks = R.attn_blocks(H, 1)
             sp = s.engine.splits(s, m, blocks, self.window)

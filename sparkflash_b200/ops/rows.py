@@ -269,13 +269,13 @@ def latent_turn(q, cs, row_pos, n, heads, dim, rot, halves):
 def head_proj(x, x_head, w, out, out_head, n, rows=None, lists=0, tail=0, merge=None, turn=None, gate=None):
     """out[row][h] = x[row][h] w[h], w [heads, K, M]; heads ``x_head`` / ``out_head`` elements apart.  ``rows`` names rows of x (lists=1) or
     of out (lists=2); ``tail`` elements behind x's K are copied behind out's M, turned by ``turn`` = (cs, row_pos) (element i with i + tail / 2).
-    ``merge``: (part, ml, row_pos, window, blocks) of latent_decode; x is then the merged attention output.  ``gate`` [rows of out, heads M]
+    ``merge``: (part, ml, parts, ctas) of latent_decode; x is then the merged attention output.  ``gate`` [rows of out, heads M]
     view: outputs are multiplied by its sigmoid."""
-    part, ml, pos, window, blocks = merge or (None, None, None, 1, 0)
-    cs, pos = turn if turn is not None else (None, pos)
+    part, ml, parts, most = merge or (None, None, None, 0)
+    cs, pos = turn if turn is not None else (None, None)
     H, K, M = w.shape
     _check(_lib.rows().sfb_rows_head_proj(*_strides(x), c_int64(x_head), _p(w), *_strides(out), c_int64(out_head), _p(rows), c_int(lists if rows is not None else 0),
-                                          _p(part), _p(ml), _p(pos), c_int(window), c_int(blocks), c_int(n), c_int(H), c_int(K), c_int(M), c_int(tail), _p(cs),
+                                          _p(part), _p(ml), _p(parts), c_int(most), _p(pos), c_int(n), c_int(H), c_int(K), c_int(M), c_int(tail), _p(cs),
                                           *_strides(gate), _fp32(w), _stream()), "rows_head_proj")
 
 
@@ -462,19 +462,29 @@ def latent_decode_supports(dtype: torch.dtype, rot: int, rank: int) -> bool:
     return dtype == torch.bfloat16 and rot % 8 == 0 and 0 < rot <= 64 and rank % 8 == 0 and rank <= 512
 
 
-def latent_blocks(window: int, max_pos: int) -> int:
-    """Pairs of pages that the window of a position up to ``max_pos`` can touch."""
-    return -(-min((window + 62) // 64 + 1, max_pos // 64 + 1) // 2)
+LATENT_ROWS = 256          # most rows of a launch of latent_decode (csrc/k_rows_latent_dec.cu)
+SMS = 148
 
 
-def latent_decode(q, pool, rank, rot, table, row_lane, row_pos, rows, n, heads, part, ml, window, blocks, scale, status):
-    """Attention of single rows over the cached latents, per block of two pages: (log2 maximum, sum, output) to ml and part.  q: [n, heads
-    (rank + rot)] of the launch's rows."""
+def latent_ctas(heads: int, pages: int) -> int:
+    """CTAs that share up to ``pages`` pages of a launch: at most one per SM over the groups of heads."""
+    return max(1, min(SMS // -(-heads // (16 if heads <= 16 else 32)), pages if pages <= 64 else (pages + 1) // 2))
+
+
+def latent_places(n: int, heads: int) -> int:
+    """Partial results (a row, every head) that a launch of n rows leaves at most."""
+    return SMS // -(-heads // (16 if heads <= 16 else 32)) + 1 + n
+
+
+def latent_decode(q, pool, rank, rot, table, row_lane, row_pos, rows, n, heads, part, ml, parts, window, ctas, pages, scale, status):
+    """Attention of single rows over the cached latents, the pages of all rows (``pages`` at most) shared equally among ``ctas``: (log2 maximum, sum, output) of every
+    share of a row to ml and part, ctas + n places; a row's first place and number of places to parts [n, 2].  q: [n, heads (rank + rot)] of the
+    launch's rows."""
     key, box = rank + rot, _lib.rows().sfb_rows_latent_heads(heads)
     maps = (tensor_map(q, rank, box, key), tensor_map(q, rot, box, key, rank), tensor_map(pool, rank, 64, key), tensor_map(pool, rot, 64, key, rank))
-    _check(_lib.rows().sfb_rows_latent_decode(*(m.ptr for m in maps), _p(table), _p(row_lane), _p(row_pos), _p(rows), _p(part), _p(ml),
+    _check(_lib.rows().sfb_rows_latent_decode(*(m.ptr for m in maps), _p(table), _p(row_lane), _p(row_pos), _p(rows), _p(part), _p(ml), _p(parts),
                                               c_int(table.shape[1]), c_int(pool.shape[0]), c_int(n), c_int(heads), c_int(rank), c_int(rot), c_int(window),
-                                              c_int(blocks), c_int(q.storage_offset() // key), c_float(scale), _p(status), _stream()), "rows_latent_decode")
+                                              c_int(ctas), c_int(pages), c_int(q.storage_offset() // key), c_float(scale), _p(status), _stream()), "rows_latent_decode")
 
 
 def expand(c: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:

@@ -1,7 +1,8 @@
-"""Throughput of a layered decoder (models/fanodra.py, models/gudutar.py, models/lifulorn.py) at sizes that resemble a real model's layers,
+"""Throughput of a layered decoder (models/fanodra.py, models/gudutar.py, models/lifulorn.py, models/dironex.py) at sizes that resemble a real model's layers,
 per-kernel roofline fractions, and the same for the closest model of the package: for Fanodra the hybrid decoder of models/qwen.py (linear
 attention three layers in four, softmax attention in the fourth), for Gudutar the Fanodra of the same width, head size, feed-forward
-width and number of layer runs, for Lifulorn the Gudutar of the same width, number of layers, head size and active feed-forward width.  ``python bench.py --design NAME`` prints it as one JSON line.
+width and number of layer runs, for Lifulorn the Gudutar of the same width, number of layers, head size and active feed-forward width, for
+Dironex the Lifulorn (windowed attention, experts) and the Gudutar (latent attention) of the same sizes.  ``python bench.py --design NAME`` prints it as one JSON line.
 
 Everything is timed on the device with CUDA events after warm-up; inputs are larger than L2, or L2 is flushed in between.
 """
@@ -11,7 +12,8 @@ import statistics
 
 import torch
 
-from ..models import fanodra, gudutar, lifulorn
+from ..models import dironex, fanodra, gudutar, lifulorn
+from ..models.dironex import DironexConfig
 from ..models.fanodra import FanodraConfig
 from ..models.gudutar import GudutarConfig
 from ..models.lifulorn import LifulornConfig
@@ -76,8 +78,28 @@ def lifulorn_config(name: str) -> LifulornConfig:
                                      "layers": [{"type": t, "mixer": mixers[t], "mlp": mlp} for t in (RULES[i % 4] for i in range(len(gudutar_config(name).layers)))]})
 
 
+STREAMS, GROUPS, KEEP = 4, 8, 4
+SUBLAYERS = (("attention", "moe"), ("latent_attention", "dense"), ("attention", "dense"), ("latent_attention", "moe"))
+
+
+def dironex_config(name: str) -> DironexConfig:
+    """The Fanodra's layers and loop; attention with the other designs' heads and window, latent attention with their heads, latent and rotated part,
+    over the whole context.  A feed-forward has two matrices instead of three and is half as wide again, so that a row uses as many weights."""
+    w, n, H, G, dim, _, _, _, ff, vocab, loop = SIZES[name]
+    wide = ff * 3 // 2
+    mlp = {"dense": {"kind": "dense", "ff": wide},
+           "moe": {"kind": "moe", "router": {"experts": EXPERTS, "top": TOP, "groups": {"count": GROUPS, "keep": KEEP}, "scale": 1.0}, "expert": {"ff": wide // TOP}}}
+    yarn = {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    mixers = {"attention": {"heads": H, "kv_heads": G, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "mask": {"size": WINDOW}},
+              "latent_attention": {"heads": H, "dim": dim, "rot_dim": ROT, "vdim": dim, "kv_rank": RANK, "q_rank": min(w // 2, 1536), "scale": (dim + ROT) ** -0.5,
+                                   "rot": {"base": 500000.0, "dims": ROT, "scaling": yarn}}}
+    return DironexConfig.from_dict({"architecture": "Dironex", "name": f"dironex-{name}", "vocab": vocab, "width": w, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+                                    "residual_mult": 0.5, "streams": STREAMS, "canon": {"taps": 4}, "loop": dict(zip(("start", "stop", "times"), loop)) if loop else None,
+                                    "layers": [{"type": t, "mixer": mixers[t], "mlp": mlp[f]} for t, f in (SUBLAYERS[i % 4] for i in range(n))]})
+
+
 CONFIGS = {"fanodra": (fanodra_config, fanodra.Fanodra, fanodra.random_tensors), "gudutar": (gudutar_config, gudutar.Gudutar, gudutar.random_tensors),
-           "lifulorn": (lifulorn_config, lifulorn.Lifulorn, lifulorn.random_tensors)}
+           "lifulorn": (lifulorn_config, lifulorn.Lifulorn, lifulorn.random_tensors), "dironex": (dironex_config, dironex.Dironex, dironex.random_tensors)}
 
 
 def engine(design: str, name: str, lanes: int, context: int, rows: int) -> LayeredEngine:
@@ -283,6 +305,81 @@ def lifulorn_work(cfg: LifulornConfig, n: int, ctx: int, head_rows: int, decode:
     return out
 
 
+def dironex_work(cfg: DironexConfig, n: int, ctx: int, head_rows: int, decode: bool) -> dict[str, roofline.ClassWork]:
+    """The same accounting for Dironex.  Seam: every stream in and out once per sublayer."""
+    d, W, few = cfg.width, roofline.ClassWork, n <= 4
+    out = {k: W() for k in ("rows_streams", "rows_conv", "rows_head_append", "rows_attn_stream", "rows_attn_tc", "rows_latent_append", "rows_latent_turn",
+                            "rows_head_proj", "rows_latent_decode", "rows_gather_pages", "rows_act", "rows_moe_gemm", "rows_moe_gemv", "rows_moe_route", "rows_moe_plan",
+                            "rows_moe_pick", "linear", "router", "head")}
+
+    def linear(k, m, rows=n, name="linear"):
+        out[name].flops += 2.0 * rows * k * m
+        out[name].bytes += 2.0 * (k * m + rows * (k + m))
+
+    def seam(parts=1):
+        out["rows_streams"].bytes += n * d * (8.0 * cfg.streams + 2.0 * parts + 2.0)
+        out["rows_conv"].bytes += 0.0 if decode else 4.0 * n * d
+    out["rows_streams"].bytes += n * d * (4.0 * cfg.streams + 4.0) + head_rows * d * (4.0 * cfg.streams + 4.0)
+    out["rows_conv"].bytes += 0.0 if decode else 4.0 * n * d
+    for at, i in enumerate(cfg.runs()):
+        L = cfg.layers[i]
+        m, H, dim, vdim = L.mixer, L.mixer["heads"], L.mixer["dim"], L.mixer["vdim"]
+        inner = H * vdim
+        linear(inner, d)
+        if L.type == "attention":
+            G = m["kv_heads"]
+            cols, win = H * dim + G * (dim + vdim), min(m["mask"]["size"], ctx)
+            linear(d, cols)
+            out["rows_head_append"].bytes += 4.0 * n * cols
+            if decode:
+                out["rows_attn_stream"].bytes += 2.0 * n * (win * G * (dim + vdim) + H * (dim + vdim))
+            else:
+                seen, keys = n * win if ctx - n >= win else n * (ctx - n) + n * (n + 1) / 2, n + min(ctx - n, win - 1)
+                out["rows_attn_tc"].flops += 2.0 * H * seen * (dim + vdim)
+                out["rows_attn_tc"].bytes += 2.0 * (n * H * (dim + vdim) + keys * G * (dim + vdim))
+        else:
+            r, rot, qr = m["kv_rank"], m["rot_dim"], m["q_rank"]
+            key, qd = r + rot, dim + rot
+            linear(d, inner + key + qr)
+            linear(qr, H * qd)
+            out["rows_latent_append"].bytes += 4.0 * n * (key + qr)
+            if decode:
+                out["rows_head_proj"].bytes += 2.0 * H * r * (dim + vdim) + 2.0 * n * H * (dim + 2 * vdim + r + key)
+                out["rows_latent_decode"].bytes += 2.0 * n * (ctx * key + H * (key + r))
+                out["rows_latent_decode"].flops += 2.0 * n * H * ctx * (key + r)
+            else:
+                out["rows_latent_turn"].bytes += 4.0 * n * H * rot
+                out["rows_gather_pages"].bytes += 4.0 * ctx * key
+                linear(r, H * (dim + vdim), ctx)
+                seen = n * (ctx - n) + n * (n + 1) / 2
+                out["rows_attn_tc"].flops += 2.0 * H * seen * (qd + vdim)
+                out["rows_attn_tc"].bytes += 2.0 * (n * H * (qd + 2 * vdim) + ctx * H * (dim + vdim))
+        if L.mlp is not None and L.mlp["kind"] == "dense":
+            ff = L.mlp["ff"]
+            seam()
+            linear(d, ff)
+            linear(ff, d)
+            out["rows_act"].bytes += 0.0 if few else 4.0 * n * ff
+        elif L.mlp is not None:
+            E, top, ff = L.mlp["router"]["experts"], L.mlp["router"]["top"], L.mlp["expert"]["ff"]
+            used = E * (1 - (1 - top / E) ** n)              # experts that n rows touch, on average
+            seam()
+            linear(d, E, name="router")
+            out["rows_moe_route"].bytes += n * (4.0 * E + 8.0 * top)
+            out["rows_moe_plan"].bytes += n * top * 16.0
+            if few:
+                out["rows_moe_gemv"].bytes += 2.0 * 2 * d * n * top * ff
+            else:
+                out["rows_moe_gemm"].bytes += 2.0 * (2 * d * used * ff + n * (d + top * (2 * ff + d)))
+                out["rows_moe_pick"].bytes += 0.0 if decode else 2.0 * n * d * (1 + top)
+                out["rows_moe_gemm"].flops += 2.0 * n * 2 * d * top * ff
+        if at + 1 < len(cfg.runs()):
+            seam(L.mlp["router"]["top"] if L.mlp is not None and L.mlp["kind"] == "moe" else 1)
+    out["head"].flops += 2.0 * head_rows * cfg.vocab * d
+    out["head"].bytes += 2.0 * cfg.vocab * d
+    return out
+
+
 def fanodra_work(cfg: FanodraConfig, n: int, ctx: int, head_rows: int, decode: bool) -> dict[str, roofline.ClassWork]:
     """Bytes that must move and FLOPs that must be done by a step of n rows that ends at ``ctx`` cached positions (prefill: one
     segment; decode: one row in each of n lanes), per launch name."""
@@ -350,8 +447,8 @@ def _fractions(timings: list[list[tuple[str, float]]], wk: dict[str, roofline.Cl
     return out
 
 
-WORK = {"fanodra": fanodra_work, "gudutar": gudutar_work, "lifulorn": lifulorn_work}
-CLOSEST = {"gudutar": "fanodra", "lifulorn": "gudutar"}
+WORK = {"fanodra": fanodra_work, "gudutar": gudutar_work, "lifulorn": lifulorn_work, "dironex": dironex_work}
+CLOSEST = {"gudutar": ("fanodra",), "lifulorn": ("gudutar",), "dironex": ("lifulorn", "gudutar")}
 
 
 def kernel_table(design: str, name: str, rows: int = 4096, ctx: int = 8192, reps: int = 5) -> list[dict]:
@@ -456,6 +553,10 @@ def run(design: str, sizes: list[str], steps: int, compare: bool = True) -> dict
     for name in sizes:
         out[name] = measure(design, name, steps)
         if compare:
-            out[name]["closest_model"] = closest(name) if design == "fanodra" else measure(CLOSEST[design], name, steps)
+            if design == "fanodra":
+                out[name]["closest_model"] = closest(name)
+            else:
+                for key, other in zip(("closest_model", "second_closest_model"), CLOSEST[design]):
+                    out[name][key] = {"design": other, **measure(other, name, steps)}
         torch.cuda.empty_cache()
     return out

@@ -114,8 +114,8 @@ def dense(h, w, p):
     return xielu(h @ w[p + "up"].t(), *w[p + "act"]) @ w[p + "down"].t()
 
 
-def route(z, correction, r):
-    """Chosen experts and weights of every row of logits."""
+def route(z, correction, r, margins=None):
+    """Chosen experts and weights of every row of logits; ``margins`` collects how far each row is from another choice."""
     s, E = sigmoid(z), z.shape[1]
     choice = s + correction
     g = r.get("groups") or {"count": 1, "keep": 1}
@@ -124,22 +124,33 @@ def route(z, correction, r):
     for t in range(z.shape[0]):
         row = choice[t].tolist()
         score = [sum(sorted(row[a * per:(a + 1) * per], reverse=True)[:2]) for a in range(g["count"])]
-        kept = sorted(range(g["count"]), key=lambda a: -score[a])[:g["keep"]]
-        open_ = [e for a in kept for e in range(a * per, (a + 1) * per)]
-        best = sorted(open_, key=lambda e: (-row[e], e))[:r["top"]]
+        groups = sorted(range(g["count"]), key=lambda a: (-score[a], a))
+        open_ = [e for a in groups[:g["keep"]] for e in range(a * per, (a + 1) * per)]
+        ranked = sorted(open_, key=lambda e: (-row[e], e))
+        best = ranked[:r["top"]]
         v = s[t, best]
         ids.append(best)
         wts.append(v / (v.sum() + 1e-20) * r["scale"])
+        if margins is not None:
+            gap = [score[groups[g["keep"] - 1]] - score[groups[g["keep"]]]] if g["keep"] < g["count"] else []
+            gap += [row[best[-1]] - row[ranked[r["top"]]]] if r["top"] < len(ranked) else []
+            margins.append(min(gap, default=float("inf")))
     return ids, wts
 
 
-def mixture(h, w, p, r):
-    ids, wts = route(h @ w[p + "router"].t(), w[p + "correction"], r)
+def expert(h, w, p):
+    u = (h @ w[p + "up"].t()).clamp(min=0)
+    return (u * u) @ w[p + "down"].t()
+
+
+def mixture(h, w, p, r, margins=None):
+    ids, wts = route(h @ w[p + "router"].t(), w[p + "correction"], r, margins)
     out = torch.zeros_like(h)
-    for t in range(h.shape[0]):
-        for e, v in zip(ids[t], wts[t]):
-            u = (w[f"{p}e{e}.up"] @ h[t]).clamp(min=0)
-            out[t] += v * (w[f"{p}e{e}.down"] @ (u * u))
+    for e in range(r["experts"]):
+        at = [(t, k) for t in range(h.shape[0]) for k in range(r["top"]) if ids[t][k] == e]
+        if at:
+            rows = [t for t, _ in at]
+            out[rows] += torch.stack([wts[t][k] for t, k in at])[:, None] * expert(h[rows], w, f"{p}e{e}.")
     return out
 
 
@@ -152,8 +163,9 @@ def order(cfg):
     return list(range(loop["start"])) + list(range(loop["start"], loop["stop"])) * loop["times"] + list(range(loop["stop"], n))
 
 
-def forward(cfg, tensors, tokens, taps=None, dtype=torch.float64):
-    """Logits [T, vocab] of one sequence; ``taps`` collects the sum of the streams after every layer run."""
+def forward(cfg, tensors, tokens, taps=None, dtype=torch.float64, margins=None):
+    """Logits [T, vocab] of one sequence; ``taps`` collects the sum of the streams after every layer run, ``margins`` every mixture's [T] distances
+    from another choice of experts."""
     w = {k: v.to(dtype) for k, v in tensors.items()}
     eps, m = cfg["norm"]["eps"], cfg["residual_mult"]
     X = (w["embed"][torch.as_tensor(tokens)] * cfg["embedding"]["scale"]).expand(cfg["streams"], -1, -1)
@@ -167,8 +179,82 @@ def forward(cfg, tensors, tokens, taps=None, dtype=torch.float64):
             if q == 1:
                 y = (window_attention if L["type"] == "attention" else latent_attention)(h, w, p + "mix.", L["mixer"], eps)
             else:
-                y = dense(h, w, p + "mlp.") if L["mlp"]["kind"] == "dense" else mixture(h, w, p + "mlp.", L["mlp"]["router"])
+                near = []
+                y = dense(h, w, p + "mlp.") if L["mlp"]["kind"] == "dense" else mixture(h, w, p + "mlp.", L["mlp"]["router"], near)
+                if margins is not None and near:
+                    margins.append(torch.tensor(near))
             X = spread(X, w[f"{p}hc{q}.mix"], w[f"{p}hc{q}.out"], m, y)
         if taps is not None:
             taps.append(X.sum(0))
     return rms(X.sum(0), w["final.norm"], eps) @ w["head"].t()
+
+
+# ---- models for tests ---------------------------------------------------------------------------------------------------
+def windowed(heads, kv_heads, dim, vdim, window, scale, mlp=None):
+    return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "mask": {"size": window}}, "mlp": mlp}
+
+
+def latent(heads, dim, rot, vdim, rank, q_rank, scale, base, scaling=None, mlp=None):
+    turned = {"base": base, "dims": rot}
+    if scaling:
+        turned["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    return {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "kv_rank": rank, "q_rank": q_rank,
+                                                              "scale": scale, "rot": turned}}
+
+
+def ff(width):
+    return {"kind": "dense", "ff": width}
+
+
+def moe(experts, top, width, count, keep, scale):
+    return {"kind": "moe", "router": {"experts": experts, "top": top, "groups": {"count": count, "keep": keep}, "scale": scale}, "expert": {"ff": width}}
+
+
+def make_config(vocab, width, streams, taps, mult, embed, layers, loop=None, eps=1e-5):
+    out = {"architecture": "Dironex", "vocab": vocab, "width": width, "streams": streams, "canon": {"taps": taps}, "residual_mult": mult,
+           "embedding": {"scale": embed}, "norm": {"eps": eps}, "layers": layers}
+    if loop:
+        out["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return out
+
+
+def make_weights(cfg, seed=0, spread=False):
+    """Random bf16 tensors; norm weights, mixes, corrections and activations' numbers differ from 1 and 0, so that leaving one out shows.
+    ``spread``: corrections so far apart that no rounding turns a choice of experts over."""
+    g = torch.Generator().manual_seed(seed)
+    w, d, S = {}, cfg["width"], cfg["streams"]
+
+    def put(name, *shape, s=None, mean=0.0):
+        w[name] = (mean + torch.randn(*shape, generator=g) * (shape[-1] ** -0.5 if s is None else s)).to(torch.bfloat16)
+    put("embed", cfg["vocab"], d, s=1.0)
+    put("head", cfg["vocab"], d)
+    put("final.norm", d, s=0.3, mean=1.0)
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        q, H, dim, vdim = p + "mix.", m["heads"], m["dim"], m["vdim"]
+        for k in (1, 2) if L.get("mlp") else (1,):
+            put(f"{p}norm{k}", d, s=0.3, mean=1.0)
+            put(f"{p}canon{k}", d, cfg["canon"]["taps"], s=0.4)
+            put(f"{p}hc{k}.in", S, s=0.3, mean=1 / S)
+            put(f"{p}hc{k}.out", S, s=0.4, mean=0.8)
+            put(f"{p}hc{k}.mix", S, S, s=0.25)
+            w[f"{p}hc{k}.mix"] = (w[f"{p}hc{k}.mix"].float() + 0.8 * torch.eye(S)).to(torch.bfloat16)
+        put(q + "o", d, H * vdim)
+        if L["type"] == "attention":
+            G = m["kv_heads"]
+            put(q + "q", H * dim, d); put(q + "k", G * dim, d); put(q + "v", G * vdim, d)
+            put(q + "q.norm", dim, s=0.4, mean=1.2); put(q + "k.norm", dim, s=0.4, mean=1.2)
+        else:
+            r, qr, rot = m["kv_rank"], m["q_rank"], m["rot_dim"]
+            put(q + "dq", qr, d); put(q + "dq.norm", qr, s=0.4, mean=1.2); put(q + "uq", H * (dim + rot), qr)
+            put(q + "dkv", r + rot, d); put(q + "dkv.norm", r, s=0.4, mean=1.2)
+            put(q + "uk", H * dim, r); put(q + "uv", H * vdim, r); put(q + "g", H * vdim, d)
+        f = L.get("mlp")
+        if f and f["kind"] == "dense":
+            put(p + "mlp.up", f["ff"], d); put(p + "mlp.down", d, f["ff"]); put(p + "mlp.act", 2, s=1.0)
+        elif f:
+            E, e_ff = f["router"]["experts"], f["expert"]["ff"]
+            put(p + "mlp.router", E, d, s=2 * d ** -0.5); put(p + "mlp.correction", E, s=20.0 if spread else 0.3, mean=-0.3)
+            for e in range(E):
+                put(f"{p}mlp.e{e}.up", e_ff, d); put(f"{p}mlp.e{e}.down", d, e_ff)
+    return w

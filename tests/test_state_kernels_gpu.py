@@ -281,13 +281,15 @@ def test_single_rows_in_the_latent_space(H, rank, rot, window, dtype):
     R.head_proj(c, rank, uv, o, 12, n)
     _close(o, out, tol)
     if R.latent_decode_supports(dtype, rot, rank):
-        blocks, o = R.latent_blocks(window, max(lens) - 1), torch.zeros_like(o)
-        part, ml = torch.zeros(n * H * blocks * rank, device="cuda"), torch.zeros(n * H * blocks * 2, device="cuda")
-        for a in (0, 4):                             # in slices of the rows
-            b = 4 if a == 0 else n
-            R.latent_decode(q[a:b], pool, rank, rot, table, lane, pos, lane[a:b], b - a, H, part, ml, window, blocks, scale, st)
-            R.head_proj(None, 0, uv, o, 12, b - a, lane[a:b], 2, merge=(part, ml, pos, window, blocks))
-        _close(o, out, tol)
+        parts = torch.zeros(n, 2, dtype=torch.int32, device="cuda")
+        for ctas in (1, 2, 5, 11, 148):              # shares that end inside rows, at their ends, and hold several rows
+            o = torch.zeros_like(o)
+            part, ml = torch.full(((n + ctas) * H * rank,), float("nan"), device="cuda"), torch.full(((n + ctas) * H * 2,), float("nan"), device="cuda")
+            for a in (0, 4):                         # in slices of the rows
+                b = 4 if a == 0 else n
+                R.latent_decode(q[a:b], pool, rank, rot, table, lane, pos, lane[a:b], b - a, H, part, ml, parts, window, ctas, sum(-(-x // 64) for x in lens), scale, st)
+                R.head_proj(None, 0, uv, o, 12, b - a, lane[a:b], 2, merge=(part, ml, parts, ctas))
+            _close(o, out, tol)
     assert st.tolist()[0] == 0
 
 
@@ -342,12 +344,12 @@ def test_a_key_that_stands_out_at_the_windows_edge():
     rows = [at, at + 1, at + window - 2, at + window - 1, at + window, at + window + 1]
     q = q1.repeat(len(rows), H).cuda()
     pos, lane, st = _i32(rows), torch.zeros(len(rows), dtype=torch.int32, device="cuda"), _status()
-    blocks, eye = R.latent_blocks(window, 299), torch.eye(rank, dtype=torch.bfloat16, device="cuda").repeat(H, 1, 1)
-    part, ml = torch.zeros(len(rows) * H * blocks * rank, device="cuda"), torch.zeros(len(rows) * H * blocks * 2, device="cuda")
+    ctas, parts, eye = 7, torch.zeros(len(rows), 2, dtype=torch.int32, device="cuda"), torch.eye(rank, dtype=torch.bfloat16, device="cuda").repeat(H, 1, 1)
+    part, ml = torch.zeros((len(rows) + ctas) * H * rank, device="cuda"), torch.zeros((len(rows) + ctas) * H * 2, device="cuda")
     a, b = torch.zeros(len(rows), H * rank, dtype=torch.bfloat16, device="cuda"), torch.zeros(len(rows), H * rank, dtype=torch.bfloat16, device="cuda")
     R.attn(q, pool, None, table, lane, pos, None, len(rows), None, a, None, None, H, 1.0, 1, st, window, rank, True)
-    R.latent_decode(q, pool, rank, rot, table, lane, pos, torch.arange(len(rows), dtype=torch.int32, device="cuda"), len(rows), H, part, ml, window, blocks, 1.0, st)
-    R.head_proj(None, 0, eye, b, rank, len(rows), None, 0, merge=(part, ml, pos, window, blocks))
+    R.latent_decode(q, pool, rank, rot, table, lane, pos, torch.arange(len(rows), dtype=torch.int32, device="cuda"), len(rows), H, part, ml, parts, window, ctas, 6 * 5, 1.0, st)
+    R.head_proj(None, 0, eye, b, rank, len(rows), None, 0, merge=(part, ml, parts, ctas))
     for got in (a, b):
         d = (got.float().view(-1, H, rank) - 4 * q1[:rank].float().cuda()).abs().amax((1, 2))
         assert (d[:4] < 0.1).all() and (d[4:] > 1).all(), d
