@@ -217,31 +217,34 @@ __global__ void __launch_bounds__(HP_T) head_proj_kernel(HeadProjArgs a) {
       if (lane == 0) { wn[warp] = nb; w0[warp] = place; }
     }
     __syncthreads();
+    // threads in groups of K / 4: a group per row, several on the places of a row where there are more groups than rows
     const int K4 = a.K >> 2, groups = HP_T / K4;       // K (the latent's size) is a multiple of eight, up to 512
-    const int grp = tid / K4, k = (tid - grp * K4) * 4;
-    float* gs = red + ((HP_R * a.most + 3) & ~3);
-    if (grp < groups) {
-      for (int r = 0; r < HP_R; ++r) {
+    const int across = min(groups, nr), along = groups / across;
+    const int grp = tid / K4, k = (tid - grp * K4) * 4, part0 = grp / across;
+    float* gs = along > 1 ? red + ((HP_R * a.most + 3) & ~3) : xs;      // [along][HP_R][K]
+    if (part0 < along) {
+      for (int r = grp % across; r < nr; r += across) {
         float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (r < nr) {
-          const int nb = wn[r];
-          const float* p = a.part + ((size_t)w0[r] * a.H + h) * a.K + k;
-          const size_t step = (size_t)a.H * a.K;
+        const int nb = wn[r];
+        const float* p = a.part + ((size_t)w0[r] * a.H + h) * a.K + k;
+        const size_t step = (size_t)a.H * a.K;
 #pragma unroll 8
-          for (int b = grp; b < nb; b += groups) {
-            const float wb = wt[r * a.most + b];
-            const float4 v = *reinterpret_cast<const float4*>(p + b * step);
-            f.x = fmaf(wb, v.x, f.x); f.y = fmaf(wb, v.y, f.y); f.z = fmaf(wb, v.z, f.z); f.w = fmaf(wb, v.w, f.w);
-          }
+        for (int b = part0; b < nb; b += along) {
+          const float wb = wt[r * a.most + b];
+          const float4 v = *reinterpret_cast<const float4*>(p + b * step);
+          f.x = fmaf(wb, v.x, f.x); f.y = fmaf(wb, v.y, f.y); f.z = fmaf(wb, v.z, f.z); f.w = fmaf(wb, v.w, f.w);
         }
-        *reinterpret_cast<float4*>(gs + (size_t)(grp * HP_R + r) * a.K + k) = f;
+        *reinterpret_cast<float4*>(gs + (size_t)(part0 * HP_R + r) * a.K + k) = f;
       }
     }
-    __syncthreads();
-    for (int i = tid; i < HP_R * a.K; i += HP_T) {
-      float f = 0.f;
-      for (int q = 0; q < groups; ++q) f += gs[(size_t)q * HP_R * a.K + i];
-      xs[i] = f;
+    for (int i = nr * a.K + tid; i < HP_R * a.K; i += HP_T) xs[i] = 0.f;
+    if (along > 1) {
+      __syncthreads();
+      for (int i = tid; i < nr * a.K; i += HP_T) {
+        float f = 0.f;
+        for (int q = 0; q < along; ++q) f += gs[(size_t)q * HP_R * a.K + i];
+        xs[i] = f;
+      }
     }
   } else {
     for (int i = tid; i < HP_R * a.K; i += HP_T) {

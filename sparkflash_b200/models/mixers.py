@@ -594,13 +594,13 @@ class LatentAttention:
         if m and self.dec:
             part, ml = s.scratch.buf["attn_part"], s.scratch.buf["attn_ml"]
             parts, seen = s.scratch.get("lat_parts", self.slice, 2), min(s.pages, -(-s.engine.max_context // R.PAGE), (self.window + R.PAGE - 2) // R.PAGE + 1)
-            idx = short_rows if short_rows is not None else s.engine._iota[:m]
             for a in range(0, m, self.slice):
                 b = min(m, a + self.slice)
+                rows = None if short_rows is None and a == 0 else (short_rows if short_rows is not None else s.engine._iota)[a:b]
                 ctas = R.latent_ctas(H, (b - a) * seen)
-                R.latent_decode(q[a:b], pool, self.rank, rot, s.table, s.row_lane, s.row_pos, idx[a:b], b - a, H, part, ml, parts, self.window, ctas,
+                R.latent_decode(q[a:b], pool, self.rank, rot, s.table, s.row_lane, s.row_pos, rows, b - a, H, part, ml, parts, self.window, ctas,
                                 (b - a) * seen, self.scale, s.status)
-                R.head_proj(None, 0, self.uv, o, self.vdim, b - a, idx[a:b], 2, merge=(part, ml, parts, ctas), gate=gate)
+                R.head_proj(None, 0, self.uv, o, self.vdim, b - a, rows, 2, merge=(part, ml, parts, ctas), gate=gate)
         elif m:
             blocks = R.attn_blocks(H, 1)
             sp = s.engine.splits(s, m, blocks, self.window)
