@@ -855,17 +855,24 @@ __global__ void __launch_bounds__(256) act_mul_kernel(const T* gu, T* out, int f
 }
 
 // ---- ungated activations ---------------------------------------------------------------------------------------------------
+constexpr int ACT_U = 2;    // groups of V per thread, requested together
 template <typename T, int V>
 __global__ void __launch_bounds__(256) act_kernel(const T* z, T* out, int64_t count, int act, float p0, float p1) {
   pdl_launch_dependents();
   pdl_wait();
-  const int64_t c = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * V;
-  if (c >= count) return;
-  float f[V];
-  load_v<T, V>(z + c, f);
+  const int64_t c0 = ((int64_t)blockIdx.x * ACT_U * blockDim.x + threadIdx.x) * V;
+  float f[ACT_U][V];
 #pragma unroll
-  for (int k = 0; k < V; ++k) f[k] = act_single<T>(f[k], act, p0, p1);
-  store_v<T, V>(out + c, f);
+  for (int u = 0; u < ACT_U; ++u)
+    if (c0 + (int64_t)u * 256 * V < count) load_v<T, V>(z + c0 + (int64_t)u * 256 * V, f[u]);
+#pragma unroll
+  for (int u = 0; u < ACT_U; ++u) {
+    const int64_t c = c0 + (int64_t)u * 256 * V;
+    if (c >= count) break;
+#pragma unroll
+    for (int k = 0; k < V; ++k) f[u][k] = act_single<T>(f[u][k], act, p0, p1);
+    store_v<T, V>(out + c, f[u]);
+  }
 }
 
 // ---- dispatch ---------------------------------------------------------------------------------------------------------------
@@ -1052,7 +1059,7 @@ int sfb_rows_act_mul(const void* gu, void* out, int64_t out_stride, int n, int f
 int sfb_rows_act(const void* z, void* out, int64_t count, int act, float p0, float p1, int fp32, cudaStream_t stream) {
   if (count < 1 || (act != ACT_RELU2 && act != ACT_XIELU)) return (int)cudaErrorInvalidValue;
   const int V = count % 4 ? 1 : fp32 || count % 8 ? 4 : 8;
-  const int64_t blocks = (count + 256 * V - 1) / (256 * V);
+  const int64_t blocks = (count + 256 * ACT_U * V - 1) / (256 * ACT_U * V);
   if (blocks > 0x7fffffff) return (int)cudaErrorInvalidValue;
   const dim3 g((unsigned)blocks), b(256);
   if (fp32) return (int)(V == 4 ? sfb_launch(act_kernel<float, 4>, g, b, 0, stream, (const float*)z, (float*)out, count, act, p0, p1)

@@ -101,15 +101,18 @@ template <typename T> __device__ __forceinline__ float gate_clamp(float g, float
   return g * gate_sigmoid<T>(alpha * g) * (u + 1.f);
 }
 
-// exp(z) - 1 - z for z <= 0: the series near 0, where the difference would cancel (the first term left out is below 2^-28 of the sum)
+// exp(z) - 1 - z for z <= 0: the series near 0, where the difference would cancel.  32-bit activations: the first term left out is below 2^-28 of
+// the sum; bf16: the difference is taken from where it is good to 2^-13.
 template <typename T> __device__ __forceinline__ float expm1_minus(float z) {
-  float p = 1.f / 3628800.f;
-  p = fmaf(p, z, 1.f / 362880.f); p = fmaf(p, z, 1.f / 40320.f); p = fmaf(p, z, 1.f / 5040.f); p = fmaf(p, z, 1.f / 720.f); p = fmaf(p, z, 1.f / 120.f);
-  p = fmaf(p, z, 1.f / 24.f); p = fmaf(p, z, 1.f / 6.f); p = fmaf(p, z, 0.5f);
-  float e;
-  if constexpr (sizeof(T) == 4) e = expf(z);
-  else e = __expf(z);
-  return z > -0.75f ? z * z * p : e - 1.f - z;
+  if constexpr (sizeof(T) == 4) {
+    float p = 1.f / 3628800.f;
+    p = fmaf(p, z, 1.f / 362880.f); p = fmaf(p, z, 1.f / 40320.f); p = fmaf(p, z, 1.f / 5040.f); p = fmaf(p, z, 1.f / 720.f); p = fmaf(p, z, 1.f / 120.f);
+    p = fmaf(p, z, 1.f / 24.f); p = fmaf(p, z, 1.f / 6.f); p = fmaf(p, z, 0.5f);
+    return z > -0.75f ? z * z * p : expf(z) - 1.f - z;
+  } else {
+    const float p = fmaf(fmaf(fmaf(1.f / 120.f, z, 1.f / 24.f), z, 1.f / 6.f), z, 0.5f);
+    return z > -0.0625f ? z * z * p : __expf(z) - 1.f - z;
+  }
 }
 
 // One input.  RELU2: max(z, 0)^2.  XIELU (Huang and Schlag, "Deriving Activation Functions Using Integration"): a z^2 + z / 2 above 0,

@@ -55,7 +55,39 @@ template <int N> __device__ __forceinline__ int take_best(uint32_t (&v)[N], int 
   return at;
 }
 
-// Groups: bit k of the result: this lane's expert k * 32 + lane cannot be chosen.
+// Groups of 2, 4 .. 32 experts whose scores c the lanes hold: a group is a run of lanes, and its two largest meet in it.  Bit k of the result: this
+// lane's expert k * 32 + lane cannot be chosen.
+__device__ __forceinline__ uint32_t shut_held(const RouteArgs& a, const float (&c)[HELD], int size) {
+  const int lane = threadIdx.x & 31;
+  uint32_t v[HELD];
+#pragma unroll
+  for (int k = 0; k < HELD; ++k) {
+    v[k] = 0u;
+    if (k * 32 >= a.E) continue;
+    float m0 = c[k], m1 = -INFINITY;
+    for (int o = 1; o < size; o <<= 1) {
+      const float x0 = __shfl_xor_sync(0xffffffffu, m0, o), x1 = __shfl_xor_sync(0xffffffffu, m1, o);
+      m1 = fmaxf(fmaxf(m1, x1), fminf(m0, x0));
+      m0 = fmaxf(m0, x0);
+    }
+    if (k * 32 + lane < a.E) v[k] = rank_bits(m0 + m1);
+  }
+  uint32_t shut = 0xffffffffu;
+  for (int i = 0; i < a.keep; ++i) {
+    uint32_t best = 0;
+    int at = a.groups - 1;
+#pragma unroll
+    for (int k = 0; k < HELD; ++k)
+      if (v[k] > best) { best = v[k]; at = (k * 32 + lane) / size; }
+    const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+    at = (int)__reduce_min_sync(0xffffffffu, (unsigned)(best == top ? at : a.groups - 1));
+#pragma unroll
+    for (int k = 0; k < HELD; ++k)
+      if (k * 32 + lane < a.E && (k * 32 + lane) / size == at) { v[k] = 0u; shut &= ~(1u << k); }
+  }
+  return shut;
+}
+// The same for groups of any size.
 __device__ __forceinline__ uint32_t shut_experts(const RouteArgs& a, const float* z) {
   const int lane = threadIdx.x & 31, size = a.E / a.groups;
   constexpr int N = MAX_GROUPS / 32;
@@ -91,10 +123,17 @@ __device__ __forceinline__ uint32_t shut_experts(const RouteArgs& a, const float
 // One warp, one row: lane j ends up with choice j and its weight (the lower number wins among equal scores); `shared_w`: the shared expert's.
 __device__ __forceinline__ void choose(const RouteArgs& a, const float* z, int& id, float& weight, float& shared_w) {
   const int lane = threadIdx.x & 31;
-  uint32_t taken = a.corr && a.keep < a.groups ? shut_experts(a, z) : 0u;      // bit k: this lane's expert k * 32 + lane
+  float c[HELD];
+#pragma unroll
+  for (int k = 0; k < HELD; ++k) c[k] = k * 32 + lane < a.E ? choice_score(a, z, k * 32 + lane) : -INFINITY;
+  uint32_t taken = 0u;      // bit k: this lane's expert k * 32 + lane
+  if (a.corr && a.keep < a.groups) {
+    const int size = a.E / a.groups;
+    taken = a.E <= HELD * 32 && size > 1 && size <= 32 && (size & (size - 1)) == 0 ? shut_held(a, c, size) : shut_experts(a, z);
+  }
   uint32_t v[HELD];         // 0: taken, or past the end
 #pragma unroll
-  for (int k = 0; k < HELD; ++k) v[k] = k * 32 + lane < a.E && !(taken >> k & 1) ? rank_bits(choice_score(a, z, k * 32 + lane)) : 0u;
+  for (int k = 0; k < HELD; ++k) v[k] = k * 32 + lane < a.E && !(taken >> k & 1) ? rank_bits(c[k]) : 0u;
   const float zs = a.shared ? z[a.E] : 0.f;
   id = 0;
   for (int j = 0; j < a.top; ++j) {

@@ -112,7 +112,7 @@ def test_append_norms_every_head(H, G, dim, vdim, dt):
 @pytest.mark.parametrize("dt", DTYPES)
 @pytest.mark.parametrize("p,q", [(0.3, -0.7), (-4.0, 3.0)])
 def test_xielu_near_zero_and_far_out(p, q, dt):
-    z = torch.cat([torch.linspace(-30, 8, 1001), torch.tensor([-0.75, -0.7501, -0.7499, 0.0, -0.0, 1e-6, -1e-6, -1e-4, -3e-3, -100.0])]).to(dt)
+    z = torch.cat([torch.linspace(-30, 8, 1001), torch.tensor([-0.75, -0.7501, -0.7499, -0.0625, -0.0628, -0.062, 0.0, -0.0, 1e-6, -1e-6, -1e-4, -3e-3, -100.0])]).to(dt)
     P_, Q_ = torch.tensor(p, dtype=torch.float64), torch.tensor(q, dtype=torch.float64)
     want = P.xielu(z.double(), P_, Q_)
     got = R.act_rows(_dev(z, dt), torch.empty(len(z), dtype=dt, device="cuda"), "xielu", float(P.softplus(P_)), 0.5 + float(P.softplus(Q_))).double().cpu()
@@ -160,7 +160,8 @@ class _Step:
 # ---- experts -----------------------------------------------------------------------------------------------------------------
 # width, experts, choices, ff, groups, kept
 MOES = [(64, 16, 2, 24, 4, 2), (96, 6, 6, 200, 1, 1), (40, 40, 3, 136, 20, 2), (37, 6, 2, 11, 3, 2), (320, 4, 1, 64, 2, 1), (520, 130, 8, 264, 10, 3), (24, 512, 4, 8, 8, 5),
-        (32, 320, 2, 16, 160, 7), (64, 5, 2, 40, 5, 3), (48, 64, 8, 520, 1, 1)]
+        (32, 320, 2, 16, 160, 7), (64, 5, 2, 40, 5, 3), (48, 64, 8, 520, 1, 1), (64, 32, 4, 16, 8, 4),
+        (32, 256, 6, 16, 8, 3), (32, 40, 3, 24, 10, 4)]
 
 
 def _moe(d, E, top, ff, count, keep, n, dt, scale=1.7):
