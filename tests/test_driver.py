@@ -26,8 +26,10 @@ async def collect(drv, req):
 
 def run(drv, reqs):
     async def go():
-        return await asyncio.gather(*[collect(drv, r) for r in reqs])
-    drv.start()
+        tasks = [asyncio.ensure_future(collect(drv, r)) for r in reqs]
+        await asyncio.sleep(0)               # every request is in the queue before the loop runs: they share steps however fast it is
+        drv.start()
+        return await asyncio.gather(*tasks)
     try:
         return asyncio.run(go())
     finally:
