@@ -27,7 +27,7 @@ struct RouteArgs {
   float* wts;               // [n, top + shared]
   int n, E, top, shared;
   const float* corr;        // [E]: choice by sigmoid(logit) + corr, weights by the sigmoids; null: by logits and their softmax
-  int groups, keep;         // (corr) only experts of the best `keep` of `groups` equal groups of neighbours
+  int groups, keep;         // (corr) runs of E / groups experts, of which the best `keep` are open
   float scale;              // (corr) of the weights
 };
 constexpr int HELD = 8;     // scores a lane holds, the rest is read again

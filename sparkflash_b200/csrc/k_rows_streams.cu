@@ -1,7 +1,7 @@
 // Seam of the layered decoders whose residual is several streams (hyper-connections: Zhu et al., "Hyper-Connections"): one pass over a row
 // brings a sublayer's output into the streams and makes the next sublayer's input.
 //
-//   x_t  <- sum_s mix[s][t] x_s + out[t] y      all streams at once from the old ones; y may be a weighted sum of several parts
+//   x_t  <- sum_s mix[s][t] x_s + out[t] y      (the right side holds the streams before the pass); y may be a weighted sum of several parts
 //   u     = sum_t in[t] x_t                     the streams as the next sublayer reads them (in null: their sum)
 //   h     = RMS(u) w                            with, on a step of single-row segments, the input convolution h + conv(h)
 //

@@ -628,7 +628,7 @@ class DenseFF:
 
 
 class SingleFF:
-    """W_down act(W_up h); act of one input, with up to two numbers: relu2, or xielu."""
+    """act(h W_up^T) W_down^T; act of one input, with up to two numbers: relu2, or xielu."""
 
     def __init__(self, w: W, act: str, a: float = 0.0, b: float = 0.0):
         self.act, self.a, self.b = act, a, b
@@ -646,7 +646,7 @@ class SingleFF:
 class MixtureFF:
     """Every row through ``top`` of ``experts`` small feed-forwards, chosen and weighted as ``choice`` says (R.Choice), and through a shared one,
     weighted by the sigmoid of a logit of its own.  An expert with the "clamp" activation: W_down (g sigmoid(alpha g) (u + 1)), g = min(W_gate h,
-    limit), u = W_up h within +-limit; with one of R.SINGLE_ACT: W_down act(W_up h).  ``run`` returns the parts [n, top + shared, width] and
+    limit), u = W_up h within +-limit; with one of R.SINGLE_ACT: act(h W_up^T) W_down^T.  ``run`` returns the parts [n, top + shared, width] and
     their weights; the seam adds them up."""
 
     def __init__(self, w: W, spec: dict, alpha: float = 0.0, act: str = "clamp", choice: R.Choice = R.SOFTMAX):

@@ -35,7 +35,7 @@ def spread(X, mix, out, m, y):
 
 
 def input_convolution(h, w):
-    """h_t + sum_j w[:, j] h_(t - taps + 1 + j), zeros before the start."""
+    """Every row plus its channels' weighted sum over itself (last column of w) and the rows before it; rows that do not exist count as zero."""
     T, taps, out = h.shape[0], w.shape[1], h.clone()
     for j in range(taps):
         back = taps - 1 - j
